@@ -6,6 +6,9 @@ Two libraries are produced:
 * ``liblsb200_kernels.so``  - all ``csrc/kernels/*.cu`` (device code, sm_100a only)
 * ``liblsb200_runtime.so``  - all ``csrc/runtime/*.cpp`` (host-only C++20 runtime)
 
+A tool that runs one kind of model builds only what that model launches: ``ensure_for(cfg)`` returns the full kernel library when it is up to
+date and otherwise compiles the kernel files of the model's family into ``liblsb200_kernels_<family>.so``.
+
 The libraries expose a plain C ABI and are loaded with ``ctypes`` (see
 ``layerstorm_b200/ops/_native.py`` and ``layerstorm_b200/runtime/_native.py``), so no
 Python headers are needed and a full rebuild takes well under a minute.  Objects are
@@ -38,10 +41,21 @@ CXX_FLAGS = ["-O2", "-g", "-std=c++20", "-fPIC", "-Wall", "-Wno-unused-function"
              "-I", str(CSRC / "include"), "-I", str(CSRC / "runtime")]
 
 
+# kernel files of a model family (models described layer by layer run without the MLA, indexer, hyper-connection and expert-parallel kernels)
+FAMILIES = {"blocks": ("attn", "delta", "gemm_tc", "gemv", "moe", "moe_tc", "norm", "sampling")}
+
+
+def _rel(p) -> str:
+    """Path as it counts for the cache keys: relative to the package, so that a checkout can move."""
+    p = Path(p)
+    return str(p.relative_to(ROOT)) if p.is_relative_to(ROOT) else str(p)
+
+
 def _hash(paths, flags) -> str:
     h = hashlib.sha256()
+    flags = [f.replace(str(ROOT), "") for f in flags]
     for p in paths:
-        h.update(str(p).encode())
+        h.update(_rel(p).encode())
         h.update(Path(p).read_bytes())
     h.update(" ".join(flags).encode())
     return h.hexdigest()[:16]
@@ -52,10 +66,13 @@ def _headers():
     return hs
 
 
+def _obj_path(src: Path, kind: str) -> Path:
+    return OBJ / f"{src.stem}.{_hash([src] + _headers(), NVCC_FLAGS if kind == 'cu' else CXX_FLAGS)}.o"
+
+
 def _compile_one(src: Path, kind: str, verbose: bool) -> Path:
     flags = NVCC_FLAGS if kind == "cu" else CXX_FLAGS
-    key = _hash([src] + _headers(), flags)
-    obj = OBJ / f"{src.stem}.{key}.o"
+    obj = _obj_path(src, kind)
     if obj.exists():
         return obj
     for old in OBJ.glob(f"{src.stem}.*.o"):
@@ -72,10 +89,18 @@ def _compile_one(src: Path, kind: str, verbose: bool) -> Path:
     return obj
 
 
-def _link(objs, out: Path, kind: str):
+def _link_key(objs) -> str:
+    return hashlib.sha256(" ".join(sorted(_rel(o) for o in objs)).encode()).hexdigest()
+
+
+def _linked(objs, out: Path) -> bool:
     stamp = out.with_suffix(".stamp")
-    key = hashlib.sha256(" ".join(sorted(str(o) for o in objs)).encode()).hexdigest()
-    if out.exists() and stamp.exists() and stamp.read_text() == key:
+    return out.exists() and stamp.exists() and stamp.read_text() == _link_key(objs)
+
+
+def _link(objs, out: Path, kind: str):
+    stamp, key = out.with_suffix(".stamp"), _link_key(objs)
+    if _linked(objs, out):
         return
     if kind == "cu":
         cmd = [NVCC, "-shared", "-o", str(out)] + [str(o) for o in objs] + []
@@ -87,12 +112,12 @@ def _link(objs, out: Path, kind: str):
     stamp.write_text(key)
 
 
-def build_all(verbose: bool = False, only: str | None = None) -> dict:
-    """Build both libraries; returns {name: path}."""
+def build_all(verbose: bool = False, only: str | None = None, family: str | None = None) -> dict:
+    """Build both libraries; returns {name: path}.  ``family``: only the kernel files of that model family, into a library of their own."""
     OBJ.mkdir(parents=True, exist_ok=True)
     out = {}
     jobs = []
-    cu = sorted((CSRC / "kernels").glob("*.cu"))
+    cu = _kernel_sources(family)
     cpp = sorted((CSRC / "runtime").glob("*.cpp"))
     with cf.ThreadPoolExecutor(max_workers=max(2, (os.cpu_count() or 4))) as ex:
         if only in (None, "kernels"):
@@ -103,7 +128,7 @@ def build_all(verbose: bool = False, only: str | None = None) -> dict:
         for kind, fut in jobs:
             objs[kind].append(fut.result())
     if objs["cu"]:
-        p = LIB / "liblsb200_kernels.so"
+        p = LIB / (f"liblsb200_kernels_{family}.so" if family else "liblsb200_kernels.so")
         _link(objs["cu"], p, "cu")
         out["kernels"] = p
     if objs["cpp"]:
@@ -111,6 +136,25 @@ def build_all(verbose: bool = False, only: str | None = None) -> dict:
         _link(objs["cpp"], p, "cpp")
         out["runtime"] = p
     return out
+
+
+def _kernel_sources(family: str | None = None):
+    cu = sorted((CSRC / "kernels").glob("*.cu"))
+    return [s for s in cu if family is None or s.stem in FAMILIES[family]]
+
+
+def ensure_for(cfg) -> Path:
+    """Compile what the model needs (nothing when it is there already) and make the bindings load it; returns the kernel library's path."""
+    from .ops import _native
+    full = LIB / "liblsb200_kernels.so"
+    family = "blocks" if cfg.blocks else None
+    if family and not _linked([_obj_path(s, "cu") for s in _kernel_sources()], full):
+        out = build_all(family=family)
+    else:
+        out = build_all(only="runtime") if family else build_all()
+        out.setdefault("kernels", full)
+    _native.use_library(out["kernels"])
+    return out["kernels"]
 
 
 def build_sanitized(sanitizers: str = "address,undefined") -> Path:

@@ -1,0 +1,544 @@
+// Grouped-query softmax attention over the paged cache, with an optional sliding window, a per-head linear distance bias, query / key norms
+// over the whole projection, value mixing across layers and an output gate - every one of them a parameter.
+//
+//   q = RMSNorm_all(W_q h), k = RMSNorm_all(W_k h)        one norm over all rows of the projection (w = null: no norm)
+//   v = (1 - lambda) W_v h + lambda v_first                (mix = 2), v_first = the values of the first mixing layer (mix = 1 stores them)
+//   s_ij = scale q_i . k_j - slope_h (i - j),  0 <= i - j < window (window 0: the whole prefix);  o_i = softmax_j(s_ij) v_j
+//   out = o * sigmoid(gate)                                (gate offset < 0: none)
+//
+// Cache row of a token: [G * dkp keys | G * dvp values], head widths padded with zeros to dkp / dvp.
+//   attn_prep      norms, value mixing, append to the cache
+//   attn_decode    few rows: one block per (row, kv head, split of the visible keys); the heads of a group are the rows of mma.sync tiles, each
+//                  warp walks its own 16-key tiles; attn_combine merges the splits
+//   attn_prefill   runs of rows: 128 (token, head) rows of a sequence per block against 64-key tiles shared by eight warps
+//   attn_exact     fp32 cache and activations (and bf16 caches whose head widths the tensor-core kernels do not cover): CUDA cores
+// Scores, weights and the output sum are fp32; the tensor-core kernels split the weights into a bf16 (hi | lo) pair for the value product.
+#include "common.cuh"
+
+namespace lsb {
+
+struct AttnParams {
+    const void* q;                    // [rows, H, dkp] bf16 / fp32
+    const void* cache; const int* block_table; int max_pages, page;
+    const int* row_seq; const int* row_pos;
+    const float* proj; int ldp, off_gate;
+    void* out; int ldo;               // [rows, ldo]
+    float* o_part; float* ml_part;    // [rows, H, NS, dvp], [rows, H, NS, 2]
+    int rows, H, G, dk, dv, dkp, dvp, NS, window;
+    float scale;
+    const float* slope;               // [H] (log2 units are applied in the kernels) or null
+};
+
+template <typename T> __device__ __forceinline__ T to_act(float v);
+template <> __device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16(v); }
+template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
+__device__ __forceinline__ float act_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float act_f(float v) { return v; }
+__device__ __forceinline__ float gate_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+
+// ------------------------------------------------------------------------------------------------ projection -> q, cache row
+template <typename T>
+__global__ void __launch_bounds__(256) attn_prep_kernel(const float* __restrict__ proj, int ldp, int off_q, int off_k, int off_v, const float* __restrict__ wq,
+                                                        const float* __restrict__ wk, float eps, float* __restrict__ vfirst, int mix,
+                                                        const float* __restrict__ lambda, T* __restrict__ q_out, T* __restrict__ cache,
+                                                        const int* __restrict__ block_table, int max_pages, const int* __restrict__ row_seq,
+                                                        const int* __restrict__ row_pos, int H, int G, int dk, int dv, int dkp, int dvp, int page) {
+    __shared__ float red[33];
+    const int r = blockIdx.x, t = threadIdx.x;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = row_seq[r], pos = row_pos[r];
+    if (seq < 0) return;
+    const float* pr = proj + (size_t)r * ldp;
+    float qr = 1.f, kr = 1.f;
+    if (wq) {
+        float s = 0.f;
+        for (int i = t; i < H * dk; i += 256) { const float x = pr[off_q + i]; s = fmaf(x, x, s); }
+        qr = 1.f / sqrtf(block_sum(s, red) / (float)(H * dk) + eps);
+        s = 0.f;
+        for (int i = t; i < G * dk; i += 256) { const float x = pr[off_k + i]; s = fmaf(x, x, s); }
+        kr = 1.f / sqrtf(block_sum(s, red) / (float)(G * dk) + eps);
+    }
+    for (int i = t; i < H * dkp; i += 256) {
+        const int h = i / dkp, c = i - h * dkp, s = h * dk + c;
+        q_out[(size_t)r * H * dkp + i] = to_act<T>(c < dk ? pr[off_q + s] * qr * (wq ? wq[s] : 1.f) : 0.f);
+    }
+    T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * (dkp + dvp));
+    for (int i = t; i < G * dkp; i += 256) {
+        const int g = i / dkp, c = i - g * dkp, s = g * dk + c;
+        row[i] = to_act<T>(c < dk ? pr[off_k + s] * kr * (wk ? wk[s] : 1.f) : 0.f);
+    }
+    const float lam = mix == 2 ? *lambda : 0.f;
+    for (int i = t; i < G * dvp; i += 256) {
+        const int g = i / dvp, c = i - g * dvp, s = g * dv + c;
+        float v = 0.f;
+        if (c < dv) {
+            v = pr[off_v + s];
+            if (mix == 1) vfirst[(size_t)r * G * dv + s] = v;
+            if (mix == 2) v = (1.f - lam) * v + lam * vfirst[(size_t)r * G * dv + s];
+        }
+        row[G * dkp + i] = to_act<T>(v);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ CUDA-core kernel
+// One block per (row, head): 128 keys at a time, one thread per key for the scores, one per value channel for the sum.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_exact_kernel(AttnParams p) {
+    extern __shared__ __align__(16) float esm[];
+    float* s_q = esm;                                     // [dkp]
+    float* s_p = s_q + p.dkp;                             // [128]
+    int* s_row = reinterpret_cast<int*>(s_p + 128);       // [128] cache row of the tile's keys
+    float* s_o = reinterpret_cast<float*>(s_row + 128);   // [dv]
+    __shared__ float red[33];
+    const int r = blockIdx.x, h = blockIdx.y, t = threadIdx.x, g = h / (p.H / p.G);
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = p.row_seq[r], pos = p.row_pos[r];
+    if (seq < 0) return;
+    const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)r * p.H + h) * p.dkp;
+    for (int i = t; i < p.dkp; i += 128) s_q[i] = act_f(q[i]);
+    for (int i = t; i < p.dv; i += 128) s_o[i] = 0.f;
+    const float slope = p.slope ? p.slope[h] : 0.f;
+    const size_t ldc = (size_t)p.G * (p.dkp + p.dvp);
+    const T* cache = reinterpret_cast<const T*>(p.cache);
+    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    float m = -INFINITY, l = 0.f;
+    for (int k0 = lo; k0 <= pos; k0 += 128) {
+        const int j = k0 + t;
+        float s = -INFINITY;
+        int row = 0;
+        __syncthreads();
+        if (j <= pos) {
+            row = p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page;
+            const T* k = cache + (size_t)row * ldc + (size_t)g * p.dkp;
+            float a = 0.f;
+#pragma unroll 8
+            for (int c = 0; c < p.dk; ++c) a = fmaf(s_q[c], act_f(k[c]), a);
+            s = a * p.scale - slope * (float)(pos - j);
+        }
+        s_row[t] = row;
+        const float mt = fmaxf(m, block_max(s, red));
+        const float e = j <= pos ? expf(s - mt) : 0.f;
+        const float corr = m == -INFINITY ? 0.f : expf(m - mt);
+        s_p[t] = e;
+        l = l * corr + block_sum(e, red);
+        m = mt;
+        __syncthreads();
+        const int n = min(128, pos - k0 + 1);
+        for (int c = t; c < p.dv; c += 128) {
+            float a = s_o[c] * corr;
+            for (int i = 0; i < n; ++i) a = fmaf(s_p[i], act_f(cache[(size_t)s_row[i] * ldc + (size_t)p.G * p.dkp + (size_t)g * p.dvp + c]), a);
+            s_o[c] = a;
+        }
+    }
+    for (int c = t; c < p.dv; c += 128) {
+        float o = s_o[c] / l;
+        if (p.off_gate >= 0) o *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + (size_t)h * p.dv + c]);
+        reinterpret_cast<T*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = to_act<T>(o);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ tensor-core pieces (mma.sync m16n8k16)
+__device__ __forceinline__ uint32_t sm_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(sm_addr(p)));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const bf16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(sm_addr(p)));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(bf16* dst, const bf16* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sm_addr(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// two weights -> packed bf16 (hi) and the packed remainders (lo)
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const bf162 h = __floats2bfloat162_rn(a, b);
+    const bf162 r = __floats2bfloat162_rn(a - __low2float(h), b - __high2float(h));
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&r);
+}
+constexpr float kLog2e = 1.4426950408889634f;
+
+// One warp's 16 query rows against NT 16-key tiles held in shared memory.  K: [keys][ldk], V: [keys][ldv]; row r of the warp sits at
+// position pos[r / 8 half]; scores are in log2 units.  m, l: running maximum and sum of the thread's two rows.
+template <int NV, int NT>
+__device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* sk, int ldk, const bf16* sv, int ldv, int dkp, int key0, int key_end,
+                                           const int (&pos)[2], int window, float scale2, const float (&slope2)[2], float (&m)[2], float (&l)[2],
+                                           float (&o)[NV][4]) {
+    const int lane = threadIdx.x & 31;
+    float s[2 * NT][4];
+#pragma unroll
+    for (int i = 0; i < 2 * NT; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+    const bf16* qp = sq + (lane & 15) * ldq + (lane >> 4) * 8;
+    const bf16* kp = sk + ((lane & 7) + (lane >> 4) * 8) * ldk + ((lane >> 3) & 1) * 8;
+#pragma unroll 2
+    for (int k = 0; k < dkp; k += 16) {
+        uint32_t a[4];
+        ldsm4(a, qp + k);
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            uint32_t b[4];
+            ldsm4(b, kp + t * 16 * ldk + k);
+            mma_bf16(s[2 * t], a, b[0], b[1]);
+            mma_bf16(s[2 * t + 1], a, b[2], b[3]);
+        }
+    }
+    float mt[2] = {m[0], m[1]};
+#pragma unroll
+    for (int i = 0; i < 2 * NT; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int row = j >> 1, key = key0 + (i >> 1) * 16 + (i & 1) * 8 + (lane & 3) * 2 + (j & 1), dist = pos[row] - key;
+            const bool seen = dist >= 0 && (window <= 0 || dist < window) && key < key_end;
+            s[i][j] = seen ? s[i][j] * scale2 - slope2[row] * (float)dist : -INFINITY;
+            mt[row] = fmaxf(mt[row], s[i][j]);
+        }
+    float corr[2], base[2];
+#pragma unroll
+    for (int row = 0; row < 2; ++row) {
+        mt[row] = fmaxf(mt[row], __shfl_xor_sync(0xffffffffu, mt[row], 1));
+        mt[row] = fmaxf(mt[row], __shfl_xor_sync(0xffffffffu, mt[row], 2));
+        base[row] = mt[row] == -INFINITY ? 0.f : mt[row];
+        corr[row] = ex2(m[row] - base[row]);               // m = -inf: 0
+        m[row] = mt[row];
+        l[row] *= corr[row];
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+    const bf16* vp = sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8;
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+        float e[2][4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) { e[u][j] = ex2(s[2 * t + u][j] - base[j >> 1]); l[j >> 1] += e[u][j]; }
+        uint32_t hi[4], lo[4];
+        split2(e[0][0], e[0][1], hi[0], lo[0]);
+        split2(e[0][2], e[0][3], hi[1], lo[1]);
+        split2(e[1][0], e[1][1], hi[2], lo[2]);
+        split2(e[1][2], e[1][3], hi[3], lo[3]);
+#pragma unroll
+        for (int i = 0; i < NV; i += 2) {
+            uint32_t b[4];
+            ldsm4_t(b, vp + t * 16 * ldv + i * 8);
+            mma_bf16(o[i], hi, b[0], b[1]);
+            mma_bf16(o[i], lo, b[0], b[1]);
+            mma_bf16(o[i + 1], hi, b[2], b[3]);
+            mma_bf16(o[i + 1], lo, b[2], b[3]);
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ decode
+constexpr int kDecStages = 3;
+template <int DVP>
+__global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
+    constexpr int NV = DVP / 8;
+    extern __shared__ __align__(16) bf16 asm_[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = threadIdx.x;
+    const int r = blockIdx.x / p.G, g = blockIdx.x % p.G, split = blockIdx.y, hg = p.H / p.G, h0 = blockIdx.z * 16;
+    const int ldk = p.dkp + 8, ldv = DVP + 8;
+    bf16* sq = asm_;                                              // [16][ldk]
+    bf16* st = sq + 16 * ldk + (size_t)warp * kDecStages * 16 * (ldk + ldv);
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = p.row_seq[r], pos = p.row_pos[r];
+    if (seq < 0) return;
+    const bf16* q = reinterpret_cast<const bf16*>(p.q) + ((size_t)r * p.H + (size_t)g * hg + h0) * p.dkp;
+    const int nh = min(16, hg - h0);
+    for (int i = t; i < 16 * (p.dkp / 8); i += 128) {
+        const int hh = i / (p.dkp / 8), c = i % (p.dkp / 8);
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (hh < nh) v = *reinterpret_cast<const uint4*>(q + (size_t)hh * p.dkp + c * 8);
+        *reinterpret_cast<uint4*>(sq + hh * ldk + c * 8) = v;
+    }
+    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    const int ntile = (pos - lo + 16) / 16;                       // 16-key tiles of the visible range
+    const int per = (ntile + p.NS - 1) / p.NS, t0 = split * per, t1 = min(ntile, t0 + per);
+    const size_t ldc = (size_t)p.G * (p.dkp + p.dvp);
+    const bf16* cache = reinterpret_cast<const bf16*>(p.cache);
+    const int kc = p.dkp / 8, vc = DVP / 8;
+    auto issue = [&](int tile, int buf) {
+        if (tile < t1) {
+            bf16* dk_ = st + (size_t)buf * 16 * (ldk + ldv);
+            bf16* dv_ = dk_ + 16 * ldk;
+            // two lanes per key, alternating 16-byte pieces; keys past the position are clamped (masked later)
+            const int kr = lane >> 1, j = min(lo + tile * 16 + kr, pos);
+            const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
+            for (int c = lane & 1; c < kc; c += 2) cp16(dk_ + kr * ldk + c * 8, src + (size_t)g * p.dkp + c * 8);
+            for (int c = lane & 1; c < vc; c += 2) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.G * p.dkp + (size_t)g * p.dvp + c * 8);
+        }
+        cp_commit();
+    };
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[NV][4];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    const int hr0 = g * hg + h0 + min(lane >> 2, nh - 1), hr1 = g * hg + h0 + min((lane >> 2) + 8, nh - 1);
+    const float slope2[2] = {p.slope ? p.slope[hr0] * kLog2e : 0.f, p.slope ? p.slope[hr1] * kLog2e : 0.f};
+    const int pp[2] = {pos, pos};
+#pragma unroll
+    for (int s = 0; s < kDecStages - 1; ++s) issue(t0 + warp + 4 * s, s);
+    __syncthreads();
+    int buf = 0;
+    for (int tile = t0 + warp; tile < t1; tile += 4) {
+        issue(tile + 4 * (kDecStages - 1), (buf + kDecStages - 1) % kDecStages);
+        cp_wait<kDecStages - 1>();
+        __syncwarp();
+        const bf16* dk_ = st + (size_t)buf * 16 * (ldk + ldv);
+        attn_tiles<NV, 1>(sq, ldk, dk_, ldk, dk_ + 16 * ldk, ldv, p.dkp, lo + tile * 16, pos + 1, pp, p.window, p.scale * kLog2e, slope2, m, l, o);
+        __syncwarp();
+        buf = (buf + 1) % kDecStages;
+    }
+    cp_wait<0>();
+#pragma unroll
+    for (int row = 0; row < 2; ++row) {
+        l[row] += __shfl_xor_sync(0xffffffffu, l[row], 1);
+        l[row] += __shfl_xor_sync(0xffffffffu, l[row], 2);
+    }
+    // merge the four warps through shared memory (fixed order)
+    __syncthreads();
+    float* so = reinterpret_cast<float*>(asm_);                   // [4][16][DVP + 2]
+    constexpr int LDO = DVP + 2;
+#pragma unroll
+    for (int row = 0; row < 2; ++row) {
+        float* d = so + ((size_t)warp * 16 + (lane >> 2) + 8 * row) * LDO;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) { d[i * 8 + (lane & 3) * 2] = o[i][2 * row]; d[i * 8 + (lane & 3) * 2 + 1] = o[i][2 * row + 1]; }
+        if ((lane & 3) == 0) { d[DVP] = m[row]; d[DVP + 1] = l[row]; }
+    }
+    __syncthreads();
+    for (int i = t; i < nh * p.dv; i += 128) {
+        const int hh = i / p.dv, c = i - hh * p.dv, h = g * hg + h0 + hh;
+        float M = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) M = fmaxf(M, so[((size_t)w * 16 + hh) * LDO + DVP]);
+        float L = 0.f, O = 0.f;
+        if (M != -INFINITY) {
+#pragma unroll
+            for (int w = 0; w < 4; ++w) {
+                const float* d = so + ((size_t)w * 16 + hh) * LDO;
+                const float f = ex2(d[DVP] - M);
+                L = fmaf(d[DVP + 1], f, L);
+                O = fmaf(d[c], f, O);
+            }
+        }
+        if (p.NS == 1) {
+            O /= L;
+            if (p.off_gate >= 0) O *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + (size_t)h * p.dv + c]);
+            reinterpret_cast<bf16*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = __float2bfloat16(O);
+        } else {
+            const size_t k = ((size_t)r * p.H + h) * p.NS + split;
+            p.o_part[k * p.dvp + c] = O;
+            if (c == 0) { p.ml_part[2 * k] = M; p.ml_part[2 * k + 1] = L; }
+        }
+    }
+}
+
+__global__ void __launch_bounds__(128) attn_combine_kernel(AttnParams p) {
+    const int r = blockIdx.x, h = blockIdx.y;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (p.row_seq[r] < 0) return;
+    const size_t k0 = ((size_t)r * p.H + h) * p.NS;
+    float M = -INFINITY;
+    for (int s = 0; s < p.NS; ++s) M = fmaxf(M, p.ml_part[2 * (k0 + s)]);
+    float L = 0.f;
+    for (int s = 0; s < p.NS; ++s) L = fmaf(p.ml_part[2 * (k0 + s) + 1], ex2(p.ml_part[2 * (k0 + s)] - M), L);
+    for (int c = threadIdx.x; c < p.dv; c += 128) {
+        float O = 0.f;
+        for (int s = 0; s < p.NS; ++s) O = fmaf(p.o_part[(k0 + s) * p.dvp + c], ex2(p.ml_part[2 * (k0 + s)] - M), O);
+        O /= L;
+        if (p.off_gate >= 0) O *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + (size_t)h * p.dv + c]);
+        reinterpret_cast<bf16*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = __float2bfloat16(O);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ prefill
+constexpr int kPreKeys = 64;
+template <int DVP>
+__global__ void __launch_bounds__(256) attn_prefill_kernel(AttnParams p, const int* __restrict__ seq_row0, const int* __restrict__ seq_nrows, int nseq,
+                                                           int tq) {
+    constexpr int NV = DVP / 8;
+    extern __shared__ __align__(16) bf16 asm_[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = threadIdx.x, g = blockIdx.y, hg = p.H / p.G;
+    const int ldk = p.dkp + 8, ldv = DVP + 8;
+    bf16* sq = asm_;                                              // [128][ldk]
+    bf16* skv = sq + 128 * ldk;                                   // [2][64][ldk + ldv]
+    pdl_wait();
+    pdl_launch_dependents();
+    // tile -> rows [r0, r0 + n) of one sequence
+    int r0 = 0, n = 0;
+    for (int s = 0, base = 0; s < nseq; ++s) {
+        const int ns = seq_nrows[s], nt = (ns + tq - 1) / tq;
+        if ((int)blockIdx.x < base + nt) { const int k = blockIdx.x - base; r0 = seq_row0[s] + k * tq; n = min(tq, ns - k * tq); break; }
+        base += nt;
+    }
+    if (n <= 0) return;
+    const int seq = p.row_seq[r0], pos0 = p.row_pos[r0];
+    if (seq < 0) return;
+    const bf16* q = reinterpret_cast<const bf16*>(p.q);
+    for (int i = t; i < 128 * (p.dkp / 8); i += 256) {
+        const int m = i / (p.dkp / 8), c = i % (p.dkp / 8), tok = m / hg;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (tok < n) v = *reinterpret_cast<const uint4*>(q + ((size_t)(r0 + tok) * p.H + (size_t)g * hg + m % hg) * p.dkp + c * 8);
+        *reinterpret_cast<uint4*>(sq + m * ldk + c * 8) = v;
+    }
+    const int pos_last = pos0 + n - 1;
+    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) / kPreKeys * kPreKeys : 0;
+    const int ntile = (pos_last - lo) / kPreKeys + 1;
+    const size_t ldc = (size_t)p.G * (p.dkp + p.dvp);
+    const bf16* cache = reinterpret_cast<const bf16*>(p.cache);
+    const int kc = p.dkp / 8, vc = DVP / 8;
+    auto issue = [&](int tile) {
+        if (tile < ntile) {
+            bf16* dk_ = skv + (size_t)(tile & 1) * kPreKeys * (ldk + ldv);
+            bf16* dv_ = dk_ + kPreKeys * ldk;
+            const int kr = t >> 2, j = min(lo + tile * kPreKeys + kr, pos_last);     // four threads per key
+            const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
+            for (int c = t & 3; c < kc; c += 4) cp16(dk_ + kr * ldk + c * 8, src + (size_t)g * p.dkp + c * 8);
+            for (int c = t & 3; c < vc; c += 4) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.G * p.dkp + (size_t)g * p.dvp + c * 8);
+        }
+        cp_commit();
+    };
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[NV][4];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    int mr[2], pp[2];
+    float slope2[2];
+#pragma unroll
+    for (int row = 0; row < 2; ++row) {
+        mr[row] = warp * 16 + (lane >> 2) + 8 * row;
+        const int tok = mr[row] / hg;
+        pp[row] = tok < n ? pos0 + tok : -1;                      // -1: an idle row sees nothing
+        slope2[row] = p.slope ? p.slope[g * hg + mr[row] % hg] * kLog2e : 0.f;
+    }
+    // positions this warp's rows span: tiles outside their windows are skipped
+    const int wfirst = pos0 + min((warp * 16) / hg, n - 1), wlast = pos0 + min((warp * 16 + 15) / hg, n - 1);
+    const bool wlive = (warp * 16) / hg < n;
+    issue(0);
+    for (int tile = 0; tile < ntile; ++tile) {
+        issue(tile + 1);
+        cp_wait<1>();
+        __syncthreads();
+        const int k0 = lo + tile * kPreKeys;
+        if (wlive && k0 <= wlast && (p.window <= 0 || k0 + kPreKeys - 1 > wfirst - p.window)) {
+            const bf16* dk_ = skv + (size_t)(tile & 1) * kPreKeys * (ldk + ldv);
+            attn_tiles<NV, kPreKeys / 16>(sq + warp * 16 * ldk, ldk, dk_, ldk, dk_ + kPreKeys * ldk, ldv, p.dkp, k0, pos_last + 1, pp, p.window,
+                                          p.scale * kLog2e, slope2, m, l, o);
+        }
+        __syncthreads();                                          // the buffer is refilled next
+    }
+    cp_wait<0>();
+#pragma unroll
+    for (int row = 0; row < 2; ++row) {
+        l[row] += __shfl_xor_sync(0xffffffffu, l[row], 1);
+        l[row] += __shfl_xor_sync(0xffffffffu, l[row], 2);
+        const int tok = mr[row] / hg, h = g * hg + mr[row] % hg;
+        if (tok >= n) continue;
+        const float inv = 1.f / l[row];
+        const size_t rr = (size_t)(r0 + tok);
+        bf16* d = reinterpret_cast<bf16*>(p.out) + rr * p.ldo + (size_t)h * p.dv;
+        const float* gt = p.proj + rr * p.ldp + p.off_gate + (size_t)h * p.dv;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int c = i * 8 + (lane & 3) * 2 + u;
+                if (c < p.dv) {
+                    float v = o[i][2 * row + u] * inv;
+                    if (p.off_gate >= 0) v *= gate_sigmoid(gt[c]);
+                    d[c] = __float2bfloat16(v);
+                }
+            }
+    }
+}
+
+template <int DVP>
+static int launch_decode(const AttnParams& p, cudaStream_t st) {
+    const int ldk = p.dkp + 8, ldv = DVP + 8;
+    size_t smem = (size_t)(16 * ldk + 4 * kDecStages * 16 * (ldk + ldv)) * 2;
+    const size_t merge = (size_t)4 * 16 * (DVP + 2) * 4;
+    if (merge > smem) smem = merge;
+    static bool attr = false;
+    if (!attr) { cudaFuncSetAttribute(attn_decode_kernel<DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024); attr = true; }
+    launch_pdl((attn_decode_kernel<DVP>), dim3(p.rows * p.G, p.NS, (p.H / p.G + 15) / 16), 128, smem, st, p);
+    if (p.NS > 1) launch_pdl((attn_combine_kernel), dim3(p.rows, p.H), 128, 0, st, p);
+    return (int)cudaGetLastError();
+}
+template <int DVP>
+static int launch_prefill(const AttnParams& p, const int* row0, const int* nrows, int nseq, cudaStream_t st) {
+    const int ldk = p.dkp + 8, ldv = DVP + 8, tq = 128 / (p.H / p.G);
+    const size_t smem = (size_t)(128 * ldk + 2 * kPreKeys * (ldk + ldv)) * 2;
+    static bool attr = false;
+    if (!attr) { cudaFuncSetAttribute(attn_prefill_kernel<DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024); attr = true; }
+    launch_pdl((attn_prefill_kernel<DVP>), dim3(p.rows / tq + nseq, p.G), 256, smem, st, p, row0, nrows, nseq, tq);
+    return (int)cudaGetLastError();
+}
+
+}  // namespace lsb
+using namespace lsb;
+
+// padded head width of the cache and of the query buffer
+LSB_API int lsb_attn_head_pad(int d) { return d <= 32 ? 32 : (d <= 64 ? 64 : (d <= 128 ? 128 : (d + 127) / 128 * 128)); }
+
+// Query / key norms (wq / wk null: none), value mixing (mix 0 none, 1 store v_first, 2 mix with lambda) and the cache append of every row.
+LSB_API int lsb_attn_prep(const void* proj, int ldp, int off_q, int off_k, int off_v, const void* wq, const void* wk, float eps, void* vfirst, int mix,
+                          const void* lambda, void* q_out, void* cache, const void* block_table, int max_pages, const void* row_seq, const void* row_pos,
+                          int rows, int H, int G, int dk, int dv, int dkp, int dvp, int page, int f32, void* stream) {
+    if (H % G || dkp < dk || dvp < dv || dkp % 16 || dvp % 16 || (mix && !vfirst) || (mix == 2 && !lambda)) return -1;
+    cudaStream_t st = (cudaStream_t)stream;
+#define LSB_PREP(T) launch_pdl((attn_prep_kernel<T>), rows, 256, 0, st, (const float*)proj, ldp, off_q, off_k, off_v, (const float*)wq, (const float*)wk, eps, \
+                               (float*)vfirst, mix, (const float*)lambda, (T*)q_out, (T*)cache, (const int*)block_table, max_pages, (const int*)row_seq, \
+                               (const int*)row_pos, H, G, dk, dv, dkp, dvp, page)
+    if (f32) LSB_PREP(float); else LSB_PREP(bf16);
+#undef LSB_PREP
+    LSB_CHECK_LAUNCH();
+}
+
+// Attention of the step's rows.  run_rows: the largest number of rows a sequence has in this step (host knowledge; it selects the kernel form).
+// NS: key splits of the few-row form (o_part / ml_part sized for it).  off_gate < 0: no output gate.  slope null: no distance bias.
+LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
+                     const void* seq_row0, const void* seq_nrows, int nseq, int run_rows, const void* proj, int ldp, int off_gate, void* out, int ldo,
+                     void* o_part, void* ml_part, int NS, int rows, int H, int G, int dk, int dv, int dkp, int dvp, int window, float scale,
+                     const void* slope, int f32, void* stream) {
+    if (rows < 1 || H % G || dkp % 16 || dvp % 16 || NS < 1 || (NS > 1 && (!o_part || !ml_part))) return -1;
+    AttnParams p;
+    p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
+    p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.out = out; p.ldo = ldo;
+    p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.rows = rows; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = dkp; p.dvp = dvp;
+    p.NS = NS; p.window = window; p.scale = scale; p.slope = (const float*)slope;
+    cudaStream_t st = (cudaStream_t)stream;
+    const int hg = H / G;
+    const bool tc = !f32 && dkp <= 256 && dvp <= 256;
+    const bool prefill = tc && run_rows >= 8 && hg <= 128;
+    if (!tc) {
+        const size_t smem = (size_t)(dkp + 256 + dv) * 4;
+        if (smem > 48 * 1024) return -1;
+        if (f32) launch_pdl((attn_exact_kernel<float>), dim3(rows, H), 128, smem, st, p);
+        else launch_pdl((attn_exact_kernel<bf16>), dim3(rows, H), 128, smem, st, p);
+        LSB_CHECK_LAUNCH();
+    }
+    switch (dvp) {
+        case 32: return prefill ? launch_prefill<32>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<32>(p, st);
+        case 64: return prefill ? launch_prefill<64>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<64>(p, st);
+        case 128: return prefill ? launch_prefill<128>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<128>(p, st);
+        case 256: return prefill ? launch_prefill<256>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<256>(p, st);
+    }
+    return -1;
+}
+
+LSB_API int lsb_trace_set_attn(void* buf) { return lsb_trace_install(buf); }

@@ -354,7 +354,8 @@ namespace lsb {
 // Many-row product with fp32 weights (router logits of a prefill chunk): out[m][n] = alpha * sum_k x[m][k] * W[n][k] + bias[n].
 // 64 x 64 output tile per block, 4 x 4 outputs per thread, K in steps of 16 through shared memory; fp32 FMAs in a fixed
 // k order (the routing decision must not depend on the launch shape).
-__global__ void __launch_bounds__(256) sgemm_f32w_kernel(void* __restrict__ out, const bf16* __restrict__ x, const float* __restrict__ w,
+template <typename XT>
+__global__ void __launch_bounds__(256) sgemm_f32w_kernel(void* __restrict__ out, const XT* __restrict__ x, const float* __restrict__ w,
                                                          const float* __restrict__ bias, int M, int N, int K, int ldx, int ldw, int ldo,
                                                          float alpha, int out_bf16) {
     __shared__ float xs[16][64 + 4], ws[16][64 + 4];
@@ -369,8 +370,13 @@ __global__ void __launch_bounds__(256) sgemm_f32w_kernel(void* __restrict__ out,
             const int m = m0 + lr, n = n0 + lr;
             float xv[4] = {0, 0, 0, 0}, wv[4] = {0, 0, 0, 0};
             if (m < M && k0 + lk < K) {
-                const uint2 u = *reinterpret_cast<const uint2*>(x + (size_t)m * ldx + k0 + lk);
-                xv[0] = bf16_lo(u.x); xv[1] = bf16_hi(u.x); xv[2] = bf16_lo(u.y); xv[3] = bf16_hi(u.y);
+                if constexpr (std::is_same<XT, float>::value) {
+                    const float4 f = *reinterpret_cast<const float4*>(x + (size_t)m * ldx + k0 + lk);
+                    xv[0] = f.x; xv[1] = f.y; xv[2] = f.z; xv[3] = f.w;
+                } else {
+                    const uint2 u = *reinterpret_cast<const uint2*>(x + (size_t)m * ldx + k0 + lk);
+                    xv[0] = bf16_lo(u.x); xv[1] = bf16_hi(u.x); xv[2] = bf16_lo(u.y); xv[3] = bf16_hi(u.y);
+                }
             }
             if (n < N && k0 + lk < K) {
                 const float4 f = *reinterpret_cast<const float4*>(w + (size_t)n * ldw + k0 + lk);
@@ -417,12 +423,20 @@ LSB_API int lsb_gemv_f32w(void* out, const void* x, const void* w, const void* b
     // blocks (5 blocks for 288 router rows and 32 tokens: 378 us measured), while passes of the weight-streaming kernel over
     // four rows at a time keep the whole GPU busy (about 3 us per pass).
     if (M >= 128) {
-        launch_pdl((sgemm_f32w_kernel), dim3((N + 63) / 64, (M + 63) / 64), 256, 0, (cudaStream_t)stream, out, (const bf16*)x, (const float*)w,
+        launch_pdl((sgemm_f32w_kernel<bf16>), dim3((N + 63) / 64, (M + 63) / 64), 256, 0, (cudaStream_t)stream, out, (const bf16*)x, (const float*)w,
                    (const float*)bias, M, N, K, ldx, ldw, ldo, alpha, out_bf16);
         LSB_CHECK_LAUNCH();
     }
     return launch_gemv(MatF32{(const float*)w, ldw}, (const bf16*)x, ldx, out, ldo, M, N, K, alpha, (const float*)bias,
                        out_bf16, (cudaStream_t)stream);
+}
+
+// Full-precision product: x fp32 [M, ldx], w fp32 [N, ldw], out fp32 [M, ldo], fp32 FMAs.  K, ldx, ldw multiples of 4, 16-byte aligned.
+LSB_API int lsb_gemm_f32(void* out, const void* x, const void* w, int M, int N, int K, int ldx, int ldw, int ldo, void* stream) {
+    if (K % 4 || ldw % 4 || ldx % 4 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return -1;
+    launch_pdl((sgemm_f32w_kernel<float>), dim3((N + 63) / 64, (M + 63) / 64), 256, 0, (cudaStream_t)stream, out, (const float*)x, (const float*)w, nullptr,
+               M, N, K, ldx, ldw, ldo, 1.f, 0);
+    LSB_CHECK_LAUNCH();
 }
 
 // W: e4m3 [N, K] with fp32 scales [ceil(N/128), ceil(K/128)] (128x128 blocks). K % 16 == 0.

@@ -427,6 +427,14 @@ __global__ void __launch_bounds__(kD) kda_recur_kernel(KdaParams p, KdaScratch w
 
 #include "kda_chunk.cuh"
 
+// the chunk scan's tail: this head's convolution history moves on to the last three raw rows
+struct KdaTail {
+    KdaParams p;
+    __device__ void operator()(int h, int vs, int tid, int row0, int nrows, int slot) const {
+        if (vs == 0 && tid < kD) kda_update_conv_history(p, row0, nrows, slot, h * kD + tid);
+    }
+};
+
 __global__ void __launch_bounds__(kD) kda_out_kernel(KdaParams p, KdaScratch w) {
     __shared__ float s_red[33];
     const int row = blockIdx.x, h = blockIdx.y, t = threadIdx.x;
@@ -495,18 +503,19 @@ static int kda_forward_impl(const void* proj, int ldp, int off_q, int off_k, int
             launch_pdl((kda_prep_kernel), dim3((total_rows + kPrepRows - 1) / kPrepRows, H), kD, prep_smem, st, p, w, nseq, total_rows);
         // chunk-parallel recurrence: one sequence per step (its rows are the step's rows), a workspace for W, B and the chunk decays
         const int nch = (total_rows + kCh - 1) / kCh;
-        const long long need = (long long)nch * H * (2 * kCh * kCh + kD);
+        const long long need = (long long)nch * H * ChunkDims<kD>::kWsFloats;
         if (chunk_ws && nseq == 1 && total_rows >= 2 * kCh && need <= chunk_ws_floats && ((uintptr_t)chunk_ws & 15) == 0) {
             static bool chunk_attr = false;
             if (!chunk_attr) {
-                cudaFuncSetAttribute(kda_chunk_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kChunkPrepSmem);
-                cudaFuncSetAttribute(kda_chunk_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kChunkScanSmem);
+                cudaFuncSetAttribute(delta_chunk_prep_kernel<kD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ChunkDims<kD>::kPrepSmem);
+                cudaFuncSetAttribute(delta_chunk_scan_kernel<kD, KdaTail>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ChunkDims<kD>::kScanSmem);
                 chunk_attr = true;
             }
             float* cb = (float*)chunk_ws;
-            KdaChunkWs cw{cb, cb + (size_t)nch * H * kCh * kCh, cb + (size_t)2 * nch * H * kCh * kCh};
-            launch_pdl((kda_chunk_prep_kernel), dim3(nch, H), 256, kChunkPrepSmem, st, p, w, cw);
-            launch_pdl((kda_chunk_scan_kernel), dim3(H, kD / kCh), 256, kChunkScanSmem, st, p, w, cw);
+            DeltaChunkArgs ca{w.qn, w.kn, w.decay, w.vo, w.beta, p.state, p.seq_row0, p.seq_nrows, p.seq_slot, 1, 1, H, kD, 0,
+                              cb, cb + (size_t)nch * H * kCh * kCh, cb + (size_t)2 * nch * H * kCh * kCh};
+            launch_pdl((delta_chunk_prep_kernel<kD>), dim3(nch, H), 256, ChunkDims<kD>::kPrepSmem, st, ca);
+            launch_pdl((delta_chunk_scan_kernel<kD, KdaTail>), dim3(H, kD / kCh, 1), 256, ChunkDims<kD>::kScanSmem, st, ca, KdaTail{p});
         } else {
             launch_pdl((kda_recur_kernel), dim3(nseq, H), kD, 0, st, p, w);
         }

@@ -1,27 +1,39 @@
 #pragma once
 // ------------------------------------------------------------------------------------------------ chunk-parallel recurrence
-// The same recurrence in chunks of 64 tokens (one sequence per step, prefill chunks).  With G_t = sum_{s<=t} log d_s inside a chunk:
+// The gated delta rule in chunks of 64 tokens of one sequence (prefill chunks), for any head sizes: key channels padded to DK (32, 64 or
+// 128), value channels in tiles of 64.  With G_t = sum_{s<=t} log d_s inside a chunk:
 //   A[t][s] = sum_c k_t k_s exp(G_t - G_s) (s < t),  B[t][s] = sum_c q_t k_s exp(G_t - G_s) (s <= t)    every exponent <= 0
 //   W = (I + diag(beta) tril(A,-1))^-1 diag(beta),  U = W (V - Kp S0^T),  O = Qp S0^T + tril(B) U,  S = S0 diag(gC) + U^T Km
 //   Kp = K exp(G), Qp = Q exp(G), Km = K exp(G_last - G), gC = exp(G_last)
-// kda_chunk_prep: everything that does not depend on the state, one block per (chunk, head); rewrites qn -> Qp, decay -> Kp, kn -> Km in
-// place.  kda_chunk_scan: sequential over the chunks, one block per (head, half of the value channels) - value channels are independent.
-// fp32 on the CUDA cores (same precision as kda_recur); opt-in (lsb_kda_forward_chunked).
+// delta_chunk_prep: everything that does not depend on the state, one block per (chunk, head); rewrites qn -> Qp, decay -> Kp, kn -> Km in
+// place.  delta_chunk_scan: sequential over the chunks, one block per (head, value tile, sequence) - value channels are independent.
+// A step may hold several sequences; those with fewer than `min_rows` rows are left to the token recurrence.  fp32 on the CUDA cores.
 constexpr int kCh = 64;            // tokens per chunk
-constexpr int kLdK = kD + 4;       // shared-memory row stride (floats) of [*, 128] tiles: 16-byte aligned rows, conflict-free float4 columns
 constexpr int kLdC = kCh + 4;      // row stride of [*, 64] tiles
 constexpr int kSub = 16;           // tokens per sub-chunk of the A / B factorisation
-constexpr int kLdR = kD + 1;       // odd row stride of the rescaled tiles: lanes that read different rows at the same column hit different banks
-constexpr size_t kChunkPrepSmem = (size_t)(3 * kCh * kLdK + 3 * kCh * kLdC + kCh + (2 * kSub + kCh - kSub) * kLdR) * sizeof(float);
-constexpr size_t kChunkScanSmem = (size_t)(4 * kCh * kLdK + 4 * kCh * kLdC) * sizeof(float);
-
-struct KdaChunkWs {
-    float* W;     // [chunks, H, 64, 64]
-    float* B;     // [chunks, H, 64, 64] lower triangle incl. diagonal, zero above
-    float* gC;    // [chunks, H, 128]
+template <int DK> struct ChunkDims {
+    static constexpr int kLdK = DK + 4;       // shared-memory row stride (floats) of [*, DK] tiles: 16-byte aligned rows, conflict-free float4 columns
+    static constexpr int kLdR = DK + 1;       // odd row stride of the rescaled tiles: lanes that read different rows at the same column hit different banks
+    static constexpr size_t kPrepSmem = (size_t)(3 * kCh * kLdK + 3 * kCh * kLdC + kCh + (2 * kSub + kCh - kSub) * kLdR) * sizeof(float);
+    static constexpr size_t kScanSmem = (size_t)(4 * kCh * kLdK + 4 * kCh * kLdC) * sizeof(float);
+    static constexpr int kWsFloats = 2 * kCh * kCh + DK;      // workspace floats per (chunk, head)
 };
 
-__global__ void __launch_bounds__(256) kda_chunk_prep_kernel(KdaParams p, KdaScratch w, KdaChunkWs cw) {
+struct DeltaChunkArgs {
+    float* qn; float* kn; float* decay;      // [rows, H, DK]; decay: the factors, or their logarithms with `log_decay`
+    float* vo;                               // [rows, H, dv]  v in, o out
+    const float* beta;                       // [rows, H]
+    float* state;                            // [slots, H, dv, DK]
+    const int* seq_row0; const int* seq_nrows; const int* seq_slot;
+    int nseq, min_rows, H, dv, log_decay;
+    float* W;     // [chunks, H, 64, 64]
+    float* B;     // [chunks, H, 64, 64] lower triangle incl. diagonal, zero above
+    float* gC;    // [chunks, H, DK]
+};
+
+template <int kD>
+__global__ void __launch_bounds__(256) delta_chunk_prep_kernel(DeltaChunkArgs a_) {
+    constexpr int kLdK = ChunkDims<kD>::kLdK, kLdR = ChunkDims<kD>::kLdR;
     extern __shared__ __align__(16) float csm[];
     float* sK = csm;
     float* sQ = sK + kCh * kLdK;
@@ -36,28 +48,34 @@ __global__ void __launch_bounds__(256) kda_chunk_prep_kernel(KdaParams p, KdaScr
     const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     pdl_wait();
     pdl_launch_dependents();
-    const int row0 = p.seq_row0[0], nrows = p.seq_nrows[0];
-    const int c0 = chunk * kCh;
-    const int cc = min(kCh, nrows - c0);                     // tokens of this chunk
+    // this block's sequence and its chunk inside it (chunks are numbered over the chunked sequences in order)
+    int row0 = 0, cc = 0, c0 = 0;
+    for (int s_ = 0, base = 0; s_ < a_.nseq; ++s_) {
+        const int n = a_.seq_nrows[s_];
+        if (n < a_.min_rows) continue;
+        const int nc = (n + kCh - 1) / kCh;
+        if (chunk < base + nc) { row0 = a_.seq_row0[s_]; c0 = (chunk - base) * kCh; cc = min(kCh, n - c0); break; }
+        base += nc;
+    }
     if (cc <= 0) return;
-    const int C = p.H * kD;
+    const int C = a_.H * kD;
     // 1. k, q and log-decay tiles (rows past the chunk: zeros, i.e. no decay and no write)
     for (int idx = tid; idx < kCh * (kD / 4); idx += 256) {
         const int t = idx / (kD / 4), c4 = idx % (kD / 4);
         float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4, g4 = k4;
         if (t < cc) {
             const size_t off = (size_t)(row0 + c0 + t) * C + h * kD + c4 * 4;
-            k4 = *reinterpret_cast<const float4*>(w.kn + off);
-            q4 = *reinterpret_cast<const float4*>(w.qn + off);
-            const float4 d = *reinterpret_cast<const float4*>(w.decay + off);
-            g4 = make_float4(logf(d.x), logf(d.y), logf(d.z), logf(d.w));
+            k4 = *reinterpret_cast<const float4*>(a_.kn + off);
+            q4 = *reinterpret_cast<const float4*>(a_.qn + off);
+            const float4 d = *reinterpret_cast<const float4*>(a_.decay + off);
+            g4 = a_.log_decay ? d : make_float4(logf(d.x), logf(d.y), logf(d.z), logf(d.w));
         }
         *reinterpret_cast<float4*>(sK + t * kLdK + c4 * 4) = k4;
         *reinterpret_cast<float4*>(sQ + t * kLdK + c4 * 4) = q4;
         *reinterpret_cast<float4*>(sG + t * kLdK + c4 * 4) = g4;
     }
     for (int idx = tid; idx < kCh * kLdC; idx += 256) { sA[idx] = 0.f; sB[idx] = 0.f; sW[idx] = 0.f; }
-    if (tid < kCh) sBeta[tid] = tid < cc ? w.beta[(size_t)(row0 + c0 + tid) * p.H + h] : 0.f;
+    if (tid < kCh) sBeta[tid] = tid < cc ? a_.beta[(size_t)(row0 + c0 + tid) * a_.H + h] : 0.f;
     __syncthreads();
     // 2. cumulative log-decay per channel (non-increasing in t)
     if (tid < kD) {
@@ -78,16 +96,14 @@ __global__ void __launch_bounds__(256) kda_chunk_prep_kernel(KdaParams p, KdaScr
             while (ds > dt) { ds -= dt + 1; ++dt; }
             const int t = t0 + dt, s_ = t0 + ds;
             if (t >= cc) continue;                            // warp-uniform
-            const float4 kt = *reinterpret_cast<const float4*>(sK + t * kLdK + lane * 4);
-            const float4 qt = *reinterpret_cast<const float4*>(sQ + t * kLdK + lane * 4);
-            const float4 gt = *reinterpret_cast<const float4*>(sG + t * kLdK + lane * 4);
-            const float4 ks = *reinterpret_cast<const float4*>(sK + s_ * kLdK + lane * 4);
-            const float4 gs = *reinterpret_cast<const float4*>(sG + s_ * kLdK + lane * 4);
-            const float e0 = __expf(fminf(gt.x - gs.x, 0.f)), e1 = __expf(fminf(gt.y - gs.y, 0.f));
-            const float e2 = __expf(fminf(gt.z - gs.z, 0.f)), e3 = __expf(fminf(gt.w - gs.w, 0.f));
-            const float k0 = ks.x * e0, k1 = ks.y * e1, k2 = ks.z * e2, k3 = ks.w * e3;
-            float a = kt.x * k0 + kt.y * k1 + kt.z * k2 + kt.w * k3;
-            float b = qt.x * k0 + qt.y * k1 + qt.z * k2 + qt.w * k3;
+            float a = 0.f, b = 0.f;
+#pragma unroll
+            for (int i = 0; i < kD / 32; ++i) {
+                const int c = lane + 32 * i;
+                const float kse = sK[s_ * kLdK + c] * __expf(fminf(sG[t * kLdK + c] - sG[s_ * kLdK + c], 0.f));
+                a = fmaf(sK[t * kLdK + c], kse, a);
+                b = fmaf(sQ[t * kLdK + c], kse, b);
+            }
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) {
                 a += __shfl_xor_sync(0xffffffffu, a, o);
@@ -138,8 +154,8 @@ __global__ void __launch_bounds__(256) kda_chunk_prep_kernel(KdaParams p, KdaScr
     }
     __syncthreads();
     // 5. results: W, tril(B), the rescaled tiles in place, the chunk's total decay
-    float* Wg = cw.W + ((size_t)chunk * p.H + h) * kCh * kCh;
-    float* Bg = cw.B + ((size_t)chunk * p.H + h) * kCh * kCh;
+    float* Wg = a_.W + ((size_t)chunk * a_.H + h) * kCh * kCh;
+    float* Bg = a_.B + ((size_t)chunk * a_.H + h) * kCh * kCh;
     for (int idx = tid; idx < kCh * kCh; idx += 256) {
         const int t = idx / kCh, s = idx % kCh;
         Wg[idx] = sW[t * kLdC + s];
@@ -156,11 +172,11 @@ __global__ void __launch_bounds__(256) kda_chunk_prep_kernel(KdaParams p, KdaScr
         const float4 el = make_float4(expf(fminf(l4.x - g4.x, 0.f)), expf(fminf(l4.y - g4.y, 0.f)), expf(fminf(l4.z - g4.z, 0.f)),
                                       expf(fminf(l4.w - g4.w, 0.f)));
         const size_t off = (size_t)(row0 + c0 + t) * C + h * kD + c4 * 4;
-        *reinterpret_cast<float4*>(w.qn + off) = make_float4(q4.x * eg.x, q4.y * eg.y, q4.z * eg.z, q4.w * eg.w);
-        *reinterpret_cast<float4*>(w.decay + off) = make_float4(k4.x * eg.x, k4.y * eg.y, k4.z * eg.z, k4.w * eg.w);
-        *reinterpret_cast<float4*>(w.kn + off) = make_float4(k4.x * el.x, k4.y * el.y, k4.z * el.z, k4.w * el.w);
+        *reinterpret_cast<float4*>(a_.qn + off) = make_float4(q4.x * eg.x, q4.y * eg.y, q4.z * eg.z, q4.w * eg.w);
+        *reinterpret_cast<float4*>(a_.decay + off) = make_float4(k4.x * eg.x, k4.y * eg.y, k4.z * eg.z, k4.w * eg.w);
+        *reinterpret_cast<float4*>(a_.kn + off) = make_float4(k4.x * el.x, k4.y * el.y, k4.z * el.z, k4.w * el.w);
     }
-    if (tid < kD) cw.gC[((size_t)chunk * p.H + h) * kD + tid] = expf(gl[tid]);
+    if (tid < kD) a_.gC[((size_t)chunk * a_.H + h) * kD + tid] = expf(gl[tid]);
 }
 
 // acc[ii][jj] += sum_k A[ty + 16 ii][k] B[tx + 16 jj][k]  (both operands row-major with k contiguous, K a multiple of 4)
@@ -183,7 +199,11 @@ __device__ __forceinline__ void kda_mm_nt(const float* __restrict__ A, int lda, 
     }
 }
 
-__global__ void __launch_bounds__(256) kda_chunk_scan_kernel(KdaParams p, KdaScratch w, KdaChunkWs cw) {
+// `tail(h, value tile, thread, row0, nrows, slot)` runs after the block's last chunk (convolution histories of the caller).
+template <int kD, class Tail>
+__global__ void __launch_bounds__(256) delta_chunk_scan_kernel(DeltaChunkArgs a_, Tail tail) {
+    constexpr int kLdK = ChunkDims<kD>::kLdK;
+    constexpr int NK = kD / 16;                               // key columns per thread
     extern __shared__ __align__(16) float csm[];
     float* sS = csm;                         // [64 value channels][128 key channels] state slice
     float* sKp = sS + kCh * kLdK;            // [t][k]
@@ -196,13 +216,21 @@ __global__ void __launch_bounds__(256) kda_chunk_scan_kernel(KdaParams p, KdaScr
     const int h = blockIdx.x, vs = blockIdx.y, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     pdl_wait();
     pdl_launch_dependents();
-    const int row0 = p.seq_row0[0], nrows = p.seq_nrows[0], slot = p.seq_slot[0];
-    if (nrows <= 0) return;
-    const int C = p.H * kD, vbase = h * kD + vs * kCh;
-    float* sp = p.state + (((size_t)slot * p.H + h) * kD + vs * kCh) * kD;
+    const int seq = blockIdx.z;
+    const int row0 = a_.seq_row0[seq], nrows = a_.seq_nrows[seq], slot = a_.seq_slot[seq];
+    if (nrows <= 0 || nrows < a_.min_rows) return;
+    int chunk0 = 0;                                           // first chunk of this sequence in the workspace
+    for (int s_ = 0; s_ < seq; ++s_) {
+        const int n = a_.seq_nrows[s_];
+        if (n >= a_.min_rows) chunk0 += (n + kCh - 1) / kCh;
+    }
+    const int C = a_.H * kD, Cv = a_.H * a_.dv, vbase = h * a_.dv + vs * kCh;
+    const int nv = min(kCh, a_.dv - vs * kCh);                // value channels of this tile
+    float* sp = a_.state + (((size_t)slot * a_.H + h) * a_.dv + vs * kCh) * kD;
     for (int idx = tid; idx < kCh * (kD / 4); idx += 256) {
         const int v = idx / (kD / 4), c4 = idx % (kD / 4);
-        *reinterpret_cast<float4*>(sS + v * kLdK + c4 * 4) = *reinterpret_cast<const float4*>(sp + (size_t)v * kD + c4 * 4);
+        *reinterpret_cast<float4*>(sS + v * kLdK + c4 * 4) =
+            v < nv ? *reinterpret_cast<const float4*>(sp + (size_t)v * kD + c4 * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     const int nchunks = (nrows + kCh - 1) / kCh;
     for (int chunk = 0; chunk < nchunks; ++chunk) {
@@ -212,31 +240,31 @@ __global__ void __launch_bounds__(256) kda_chunk_scan_kernel(KdaParams p, KdaScr
             float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a, c = a;
             if (t < cc) {
                 const size_t off = (size_t)(row0 + c0 + t) * C + h * kD + c4 * 4;
-                a = *reinterpret_cast<const float4*>(w.decay + off);     // Kp
-                b = *reinterpret_cast<const float4*>(w.qn + off);        // Qp
-                c = *reinterpret_cast<const float4*>(w.kn + off);        // Km
+                a = *reinterpret_cast<const float4*>(a_.decay + off);     // Kp
+                b = *reinterpret_cast<const float4*>(a_.qn + off);        // Qp
+                c = *reinterpret_cast<const float4*>(a_.kn + off);        // Km
             }
             *reinterpret_cast<float4*>(sKp + t * kLdK + c4 * 4) = a;
             *reinterpret_cast<float4*>(sQp + t * kLdK + c4 * 4) = b;
             *reinterpret_cast<float4*>(sKm + t * kLdK + c4 * 4) = c;
         }
-        const float* Wg = cw.W + ((size_t)chunk * p.H + h) * kCh * kCh;
-        const float* Bg = cw.B + ((size_t)chunk * p.H + h) * kCh * kCh;
+        const float* Wg = a_.W + ((size_t)(chunk0 + chunk) * a_.H + h) * kCh * kCh;
+        const float* Bg = a_.B + ((size_t)(chunk0 + chunk) * a_.H + h) * kCh * kCh;
         for (int idx = tid; idx < kCh * (kCh / 4); idx += 256) {
             const int t = idx / (kCh / 4), c4 = idx % (kCh / 4);
             *reinterpret_cast<float4*>(sW + t * kLdC + c4 * 4) = *reinterpret_cast<const float4*>(Wg + t * kCh + c4 * 4);
             *reinterpret_cast<float4*>(sBm + t * kLdC + c4 * 4) = *reinterpret_cast<const float4*>(Bg + t * kCh + c4 * 4);
         }
-        float vreg[4][4], gc[8];
+        float vreg[4][4], gc[NK];
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int t = ty + 16 * i;
-                vreg[i][j] = t < cc ? w.vo[(size_t)(row0 + c0 + t) * C + vbase + tx + 16 * j] : 0.f;
+                vreg[i][j] = (t < cc && tx + 16 * j < nv) ? a_.vo[(size_t)(row0 + c0 + t) * Cv + vbase + tx + 16 * j] : 0.f;
             }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) gc[j] = cw.gC[((size_t)chunk * p.H + h) * kD + tx + 16 * j];
+        for (int j = 0; j < NK; ++j) gc[j] = a_.gC[((size_t)(chunk0 + chunk) * a_.H + h) * kD + tx + 16 * j];
         __syncthreads();
         float acc[4][4];
         // a. X = V - Kp S^T, stored transposed
@@ -273,32 +301,33 @@ __global__ void __launch_bounds__(256) kda_chunk_scan_kernel(KdaParams p, KdaScr
             const int t = ty + 16 * i;
             if (t < cc) {
 #pragma unroll
-                for (int j = 0; j < 4; ++j) w.vo[(size_t)(row0 + c0 + t) * C + vbase + tx + 16 * j] = acc[i][j];
+                for (int j = 0; j < 4; ++j)
+                    if (tx + 16 * j < nv) a_.vo[(size_t)(row0 + c0 + t) * Cv + vbase + tx + 16 * j] = acc[i][j];
             }
         }
         __syncthreads();                                     // every thread has read S before it changes
         // d. S = S diag(gC) + U^T Km : value rows ty + 16 i, key columns tx + 16 j
-        float a2[4][8];
+        float a2[4][NK];
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int j = 0; j < 8; ++j) a2[i][j] = 0.f;
+            for (int j = 0; j < NK; ++j) a2[i][j] = 0.f;
 #pragma unroll 2
         for (int t = 0; t < kCh; ++t) {
-            float u[4], km[8];
+            float u[4], km[NK];
 #pragma unroll
             for (int i = 0; i < 4; ++i) u[i] = sU[(ty + 16 * i) * kLdC + t];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) km[j] = sKm[t * kLdK + tx + 16 * j];
+            for (int j = 0; j < NK; ++j) km[j] = sKm[t * kLdK + tx + 16 * j];
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 8; ++j) a2[i][j] = fmaf(u[i], km[j], a2[i][j]);
+                for (int j = 0; j < NK; ++j) a2[i][j] = fmaf(u[i], km[j], a2[i][j]);
         }
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
+            for (int j = 0; j < NK; ++j) {
                 const int idx = (ty + 16 * i) * kLdK + tx + 16 * j;
                 sS[idx] = fmaf(sS[idx], gc[j], a2[i][j]);
             }
@@ -306,8 +335,8 @@ __global__ void __launch_bounds__(256) kda_chunk_scan_kernel(KdaParams p, KdaScr
     }
     for (int idx = tid; idx < kCh * (kD / 4); idx += 256) {
         const int v = idx / (kD / 4), c4 = idx % (kD / 4);
-        *reinterpret_cast<float4*>(sp + (size_t)v * kD + c4 * 4) = *reinterpret_cast<const float4*>(sS + v * kLdK + c4 * 4);
+        if (v < nv) *reinterpret_cast<float4*>(sp + (size_t)v * kD + c4 * 4) = *reinterpret_cast<const float4*>(sS + v * kLdK + c4 * 4);
     }
-    if (vs == 0 && tid < kD) kda_update_conv_history(p, row0, nrows, slot, h * kD + tid);
+    tail(h, vs, tid, row0, nrows, slot);
     pdl_launch_dependents();
 }

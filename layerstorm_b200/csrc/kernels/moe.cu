@@ -24,12 +24,12 @@ namespace lsb {
 // One block per row.
 __global__ void __launch_bounds__(1024) router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids,
                                                            float* __restrict__ wts, int E, int topk, int n_group, int topk_group, int scoring,
-                                                           int norm_topk, float scale, int n_shared, int ld_logits) {
+                                                           int norm_topk, float scale, int n_shared, int ld_logits, int group_score) {
     extern __shared__ float sm[];
     pdl_wait();
     pdl_launch_dependents();
     router_topk_block<false>(logits + (size_t)blockIdx.x * ld_logits, bias, ids + (size_t)blockIdx.x * (topk + n_shared),
-                             wts + (size_t)blockIdx.x * (topk + n_shared), E, topk, n_group, topk_group, scoring, norm_topk, scale, n_shared, sm);
+                             wts + (size_t)blockIdx.x * (topk + n_shared), E, topk, n_group, topk_group, scoring, norm_topk, scale, n_shared, sm, group_score);
 }
 
 // Router projection and top-k in one launch for decode-sized steps (rows <= 8): one block per expert computes its fp32 logit
@@ -341,6 +341,39 @@ __global__ void __launch_bounds__(256) moe_down_kernel(const bf16* __restrict__ 
 }
 
 
+// fp32 experts over fp32 activations (full-precision mode): one warp per output row and group, gate / up with SwiGLU or down.
+template <bool GATEUP>
+__global__ void __launch_bounds__(256) moe_f32_kernel(const float* __restrict__ in, const uint8_t* __restrict__ arena, const int* __restrict__ slot_of,
+                                                      ExpertFmt ef, const int* __restrict__ group_expert, const int* __restrict__ group_n,
+                                                      const int* __restrict__ group_pairs, const int* __restrict__ n_groups, float* __restrict__ out,
+                                                      int S, float limit, int* __restrict__ miss_flag) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int g = blockIdx.y;
+    if (g >= n_groups[0]) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_out = blockIdx.x * 8 + warp;
+    const int K = GATEUP ? ef.H : ef.F, N = GATEUP ? ef.F : ef.H;
+    if (n_out >= N) return;
+    const int e = group_expert[g], n = group_n[g], slot = slot_of[e];
+    if (slot < 0) { if (GATEUP && miss_flag && threadIdx.x == 0 && blockIdx.x == 0) atomicExch(miss_flag, e + 1); return; }
+    const uint8_t* base = arena + (size_t)slot * ef.stride;
+    const float* w0 = reinterpret_cast<const float*>(base + (GATEUP ? ef.off_gate : ef.off_down)) + (size_t)n_out * K;
+    const float* w1 = reinterpret_cast<const float*>(base + ef.off_up) + (size_t)n_out * K;
+    for (int m = 0; m < n; ++m) {
+        const int pr = group_pairs[g * 4 + m];
+        const float* x = in + (size_t)(GATEUP ? pr / S : pr) * K;
+        float a = 0.f, b = 0.f;
+        for (int k = lane; k < K; k += 32) { a = fmaf(w0[k], x[k], a); if (GATEUP) b = fmaf(w1[k], x[k], b); }
+        a = warp_sum(a);
+        if (GATEUP) {
+            b = warp_sum(b);
+            if (limit > 0.f) { a = fminf(a, limit); b = fminf(fmaxf(b, -limit), limit); }
+            a = a / (1.f + expf(-a)) * b;
+        }
+        if (lane == 0) out[(size_t)pr * N + n_out] = a;
+    }
+}
+
 // ---- NVFP4 fast path (hidden and expert width multiples of 128) -----------------------------
 // Row order inside a 128-row tile follows the scale-atom layout: a block covers 8 (gate/up) or 16
 // (down) consecutive values of n%32 for all four 32-row quads, so every 32-byte sector of scale
@@ -529,15 +562,23 @@ __global__ void swiglu_kernel(bf16* __restrict__ out, const float* __restrict__ 
 }  // namespace lsb
 using namespace lsb;
 
-LSB_API int lsb_router_topk(const void* logits, const void* bias, void* ids, void* wts, int rows, int E, int topk,
-                            int n_group, int topk_group, int scoring, int norm_topk, float scale, int n_shared,
-                            int ld_logits, void* stream) {
+// group_score: 0 a group counts as the sum of its two best biased scores, 1 as its best one.
+LSB_API int lsb_router_topk_grouped(const void* logits, const void* bias, void* ids, void* wts, int rows, int E, int topk,
+                                    int n_group, int topk_group, int scoring, int norm_topk, float scale, int n_shared,
+                                    int ld_logits, int group_score, void* stream) {
     if (topk > 32 || n_group > 64 || E > 4096 || n_shared > 32) return -1;
     int threads = (E + 31) / 32 * 32;
     threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
     launch_pdl((router_topk_kernel), rows, threads, (size_t)router_topk_smem_floats(E) * 4, (cudaStream_t)stream, (const float*)logits, (const float*)bias,
-               (int*)ids, (float*)wts, E, topk, n_group, topk_group, scoring, norm_topk, scale, n_shared, ld_logits);
+               (int*)ids, (float*)wts, E, topk, n_group, topk_group, scoring, norm_topk, scale, n_shared, ld_logits, group_score);
     LSB_CHECK_LAUNCH();
+}
+
+LSB_API int lsb_router_topk(const void* logits, const void* bias, void* ids, void* wts, int rows, int E, int topk,
+                            int n_group, int topk_group, int scoring, int norm_topk, float scale, int n_shared,
+                            int ld_logits, void* stream) {
+    return lsb_router_topk_grouped(logits, bias, ids, wts, rows, E, topk, n_group, topk_group, scoring, norm_topk, scale, n_shared, ld_logits,
+                                   kGroupTop2, stream);
 }
 
 // Router projection + top-k in one launch (rows <= 8, H % 16 == 0).  w: fp32 [E, H]; x: bf16 [rows, H]; logits: fp32 scratch
@@ -595,6 +636,12 @@ LSB_API int lsb_moe_gateup(const void* x, const void* arena, const void* slot_of
                                                                         (int*)miss_flag, run);
         LSB_CHECK_LAUNCH();
     }
+    if (ef.fmt == 7) {
+        if (!group_n) return -1;
+        launch_pdl((moe_f32_kernel<true>), dim3((ef.F + 7) / 8, max_groups), 256, 0, st, (const float*)x, (const uint8_t*)arena, (const int*)slot_of, ef,
+                   (const int*)group_expert, (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (float*)act, S, limit, (int*)miss_flag);
+        LSB_CHECK_LAUNCH();
+    }
     if (!group_n) return -1;   // pair mode is only implemented for the NVFP4 fast path
     dim3 grid((ef.F + 7) / 8, max_groups);
 #define ARGS (const bf16*)x, (const uint8_t*)arena, (const int*)slot_of, ef, (const int*)group_expert, (const int*)group_n, \
@@ -635,6 +682,11 @@ LSB_API int lsb_moe_down(const void* act, const void* arena, const void* slot_of
         LSB_CHECK_LAUNCH();
     }
     if (!group_n) return -1;
+    if (ef.fmt == 7) {
+        launch_pdl((moe_f32_kernel<false>), dim3((ef.H + 7) / 8, max_groups), 256, 0, st, (const float*)act, (const uint8_t*)arena, (const int*)slot_of, ef,
+                   (const int*)group_expert, (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (float*)y, 1, 0.f, nullptr);
+        LSB_CHECK_LAUNCH();
+    }
     dim3 grid((ef.H + 15) / 16, max_groups);
 #define ARGS (const bf16*)act, (const uint8_t*)arena, (const int*)slot_of, ef, (const int*)group_expert, (const int*)group_n, \
              (const int*)group_pairs, (const int*)n_groups, (float*)y

@@ -6,7 +6,7 @@
 namespace lsb {
 
 struct ExpertFmt {
-    int fmt;                 // gate / up: 0 bf16, 1 fp8 block-128, 2 nvfp4, 3 GGUF Q4_K, 4 Q5_K, 5 Q6_K (224-byte blocks), 6 Q8_0 (planar rows)
+    int fmt;                 // gate / up: 0 bf16, 1 fp8 block-128, 2 nvfp4, 3 GGUF Q4_K, 4 Q5_K, 5 Q6_K (224-byte blocks), 6 Q8_0 (planar rows), 7 fp32 (fp32 activations)
     int H, F;                // hidden, expert intermediate
     long long stride;        // bytes between slots
     long long off_gate, off_up, off_down;        // weights

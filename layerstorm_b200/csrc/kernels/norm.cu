@@ -722,4 +722,131 @@ LSB_API int lsb_cosine_sim(const void* a, const void* b, int rows, int dim, int 
     LSB_CHECK_LAUNCH();
 }
 
+namespace lsb {
+// ---- norm on a sublayer's output (post-norm residual streams), RMS or layer norm with bias ----
+struct NormW { const float* w; const float* b; int dim; float eps; int layer; };      // layer 0: RMS norm; b may be null
+
+// row[0..dim) (shared memory) -> scale and shift of its normalisation: n(x) = (x - mean) * rstd
+__device__ __forceinline__ void norm_moments(const float* row, const NormW& n, float* red, float& mean, float& rstd) {
+    mean = 0.f;
+    if (n.layer) {
+        float s = 0.f;
+        for (int i = threadIdx.x; i < n.dim; i += blockDim.x) s += row[i];
+        mean = block_sum(s, red) / (float)n.dim;
+    }
+    float v = 0.f;
+    for (int i = threadIdx.x; i < n.dim; i += blockDim.x) { const float d = row[i] - mean; v = fmaf(d, d, v); }
+    rstd = 1.f / sqrtf(block_sum(v, red) / (float)n.dim + n.eps);
+}
+template <typename T> __device__ __forceinline__ T as_act(float v);
+template <> __device__ __forceinline__ bf16 as_act<bf16>(float v) { return __float2bfloat16(v); }
+template <> __device__ __forceinline__ float as_act<float>(float v) { return v; }
+
+// The weighted sum of a row's expert outputs, slots in order: slot s holds expert ids[s]; ids below `experts` take their row of y (none when the
+// expert is not resident), the others are identity experts and take the residual stream itself.
+struct MoeSum { const float* y; const float* wts; const int* ids; const int* slot_of; int S, experts, ldy; };
+
+// resid[r] += norm(sub[r]) (or norm of the MoE sum), x[r] = the new residual in the activation type
+template <typename T, bool MOE>
+__global__ void __launch_bounds__(512) post_norm_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
+                                                        NormW n, MoeSum mo) {
+    __shared__ float red[33], s_w[32];
+    __shared__ int s_id[32];
+    extern __shared__ float row[];
+    const int r = blockIdx.x;
+    float* rr = resid + (size_t)r * ldr;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (MOE) {
+        if (threadIdx.x < mo.S) {
+            int id = mo.ids[(size_t)r * mo.S + threadIdx.x];
+            if (id >= 0 && id < mo.experts && mo.slot_of[id] < 0) id = -1;
+            s_id[threadIdx.x] = id;
+            s_w[threadIdx.x] = mo.wts[(size_t)r * mo.S + threadIdx.x];
+        }
+        __syncthreads();
+        const float* yr = mo.y + (size_t)r * mo.S * mo.ldy;
+        if (n.dim % 4 == 0 && mo.ldy % 4 == 0 && ldr % 4 == 0) {
+            for (int i = threadIdx.x * 4; i < n.dim; i += blockDim.x * 4) {
+                float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+                for (int s = 0; s < mo.S; ++s) {
+                    const int id = s_id[s];
+                    if (id < 0) continue;
+                    const float4 v = *reinterpret_cast<const float4*>(id < mo.experts ? yr + (size_t)s * mo.ldy + i : rr + i);
+                    const float w = s_w[s];
+                    a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+                }
+                *reinterpret_cast<float4*>(row + i) = a;
+            }
+        } else {
+            for (int i = threadIdx.x; i < n.dim; i += blockDim.x) {
+                float a = 0.f;
+                for (int s = 0; s < mo.S; ++s) {
+                    const int id = s_id[s];
+                    if (id >= 0) a = fmaf(s_w[s], id < mo.experts ? yr[(size_t)s * mo.ldy + i] : rr[i], a);
+                }
+                row[i] = a;
+            }
+        }
+    } else {
+        const float* sr = sub + (size_t)r * lds;
+        for (int i = threadIdx.x; i < n.dim; i += blockDim.x) row[i] = sr[i];
+    }
+    __syncthreads();
+    float mean, rstd;
+    norm_moments(row, n, red, mean, rstd);
+    T* xr = x + (size_t)r * ldx;
+    for (int i = threadIdx.x; i < n.dim; i += blockDim.x) {
+        const float v = rr[i] + ((row[i] - mean) * rstd * n.w[i] + (n.b ? n.b[i] : 0.f));
+        rr[i] = v;
+        xr[i] = as_act<T>(v);
+    }
+}
+
+// out[j] = norm(resid[rows ? rows[j] : row0 + j])
+template <typename T>
+__global__ void __launch_bounds__(512) norm_rows_kernel(T* __restrict__ out, int ldo, const float* __restrict__ resid, int ldr, const int* __restrict__ rows,
+                                                        int row0, NormW n) {
+    __shared__ float red[33];
+    extern __shared__ float row[];
+    pdl_wait();
+    pdl_launch_dependents();
+    const float* rr = resid + (size_t)(rows ? rows[blockIdx.x] : row0 + (int)blockIdx.x) * ldr;
+    for (int i = threadIdx.x; i < n.dim; i += blockDim.x) row[i] = rr[i];
+    __syncthreads();
+    float mean, rstd;
+    norm_moments(row, n, red, mean, rstd);
+    for (int i = threadIdx.x; i < n.dim; i += blockDim.x)
+        out[(size_t)blockIdx.x * ldo + i] = as_act<T>((row[i] - mean) * rstd * n.w[i] + (n.b ? n.b[i] : 0.f));
+}
+static int norm_threads(int dim) { return dim >= 2048 ? 512 : (dim >= 512 ? 256 : 128); }
+}  // namespace lsb
+
+// Post-norm residual update: resid += norm(sub), x = resid in the activation type (f32: fp32, else bf16).  layer 1: layer norm with bias b,
+// 0: RMS norm.  y non-null: `sub` is the weighted sum of the row's S expert outputs instead (ids >= experts: identity experts).
+LSB_API int lsb_post_norm(void* x, int ldx, void* resid, int ldr, const void* sub, int lds, const void* w, const void* b, int rows, int dim, float eps,
+                          int layer, const void* y, const void* wts, const void* ids, const void* slot_of, int S, int experts, int ldy, int f32,
+                          void* stream) {
+    if (dim < 1 || dim > 12000 || (y && S > 32)) return -1;
+    NormW n{(const float*)w, (const float*)b, dim, eps, layer};
+    MoeSum mo{(const float*)y, (const float*)wts, (const int*)ids, (const int*)slot_of, S, experts, ldy};
+    cudaStream_t st = (cudaStream_t)stream;
+#define LSB_PN(T, M) launch_pdl((post_norm_kernel<T, M>), rows, norm_threads(dim), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, n, mo)
+    if (f32) { if (y) LSB_PN(float, true); else LSB_PN(float, false); }
+    else { if (y) LSB_PN(bf16, true); else LSB_PN(bf16, false); }
+#undef LSB_PN
+    LSB_CHECK_LAUNCH();
+}
+
+LSB_API int lsb_norm_rows(void* out, int ldo, const void* resid, int ldr, const void* row_idx, int row0, const void* w, const void* b, int rows, int dim,
+                          float eps, int layer, int f32, void* stream) {
+    if (dim < 1 || dim > 12000) return -1;
+    NormW n{(const float*)w, (const float*)b, dim, eps, layer};
+    cudaStream_t st = (cudaStream_t)stream;
+    if (f32) launch_pdl((norm_rows_kernel<float>), rows, norm_threads(dim), (size_t)dim * 4, st, (float*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
+    else launch_pdl((norm_rows_kernel<bf16>), rows, norm_threads(dim), (size_t)dim * 4, st, (bf16*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
+    LSB_CHECK_LAUNCH();
+}
+
 LSB_API int lsb_trace_set_norm(void* buf) { return lsb_trace_install(buf); }

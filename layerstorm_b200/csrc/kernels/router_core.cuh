@@ -12,6 +12,7 @@
 namespace lsb {
 
 enum { kScoreSigmoid = 0, kScoreSoftmax = 1, kScoreSqrtSoftplus = 2 };
+enum { kGroupTop2 = 0, kGroupMax = 1 };       // a group's score: the sum of its two best biased scores, or its best one
 
 // floats of shared memory router_topk_block needs for E experts
 __host__ __device__ constexpr int router_topk_smem_floats(int E) { return 2 * E + 64 + 64 + 32 + 32 + 34; }
@@ -21,7 +22,7 @@ __host__ __device__ constexpr int router_topk_smem_floats(int E) { return 2 * E 
 template <bool CG = true>
 __device__ __forceinline__ void router_topk_block(const float* __restrict__ lg, const float* __restrict__ bias, int* __restrict__ ids,
                                                   float* __restrict__ wts, int E, int topk, int n_group, int topk_group, int scoring,
-                                                  int norm_topk, float scale, int n_shared, float* sm) {
+                                                  int norm_topk, float scale, int n_shared, float* sm, int group_score = kGroupTop2) {
     float* score = sm;                         // [E] unbiased
     float* sel = sm + E;                       // [E] biased, -inf when the group is masked
     float* gscore = sel + E;                   // [64]
@@ -52,14 +53,14 @@ __device__ __forceinline__ void router_topk_block(const float* __restrict__ lg, 
     __syncthreads();
     if (n_group > 1) {
         const int gs = E / n_group;
-        // group score = sum of the two best biased scores; keep topk_group groups (ties -> lower group)
+        // keep the topk_group groups with the best scores (ties -> lower group)
         for (int g = t; g < n_group; g += nt) {
             float a = -INFINITY, b2 = -INFINITY;
             for (int i = 0; i < gs; ++i) {
                 const float v = sel[g * gs + i];
                 if (v > a) { b2 = a; a = v; } else if (v > b2) b2 = v;
             }
-            gscore[g] = a + b2;
+            gscore[g] = group_score == kGroupMax ? a : a + b2;
         }
         __syncthreads();
         for (int g = t; g < n_group; g += nt) {

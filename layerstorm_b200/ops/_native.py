@@ -59,6 +59,14 @@ def lib_path() -> Path:
     return _LIB_PATH
 
 
+def use_library(path) -> None:
+    """Load another build of the kernel library (a model family's subset) instead of the full one; before the first call."""
+    global _LIB_PATH
+    if _LIB is not None and Path(path) != _LIB_PATH:
+        raise RuntimeError(f"the kernel library {_LIB_PATH} is loaded already")
+    _LIB_PATH = Path(path)
+
+
 def available() -> bool:
     return _LIB_PATH.exists()
 
@@ -72,7 +80,9 @@ def load():
             f"native kernel library not built: {_LIB_PATH} (run `python -m layerstorm_b200.build`)")
     lib = ctypes.CDLL(str(_LIB_PATH), mode=os.RTLD_GLOBAL if hasattr(os, "RTLD_GLOBAL") else ctypes.DEFAULT_MODE)
     for name, (sig, has_stream) in SIGS.items():
-        fn = getattr(lib, name)
+        fn = getattr(lib, name, None)
+        if fn is None:
+            continue                     # a family's subset of the kernels; calling a missing launcher raises
         fn.argtypes = [_CT[c] for c in sig] + ([ctypes.c_void_p] if has_stream else [])
         fn.restype = ctypes.c_int
     _LIB = lib

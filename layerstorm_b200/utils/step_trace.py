@@ -27,7 +27,7 @@ def install_trace(buf) -> None:
     ``None`` switches tracing off."""
     from ..ops import _native as nat
     for name in nat.SIGS:
-        if name.startswith("lsb_trace_set_"):
+        if name.startswith("lsb_trace_set_") and hasattr(nat.load(), name):
             rc = nat.call(name, buf)
             if rc != 0:
                 raise RuntimeError(f"{name} failed with status {rc}")

@@ -47,8 +47,15 @@ static inline void pdl_launch_dependents() {}
 #include "kda_types.cuh"
 #include "kda_chunk.cuh"
 
+struct Tail {
+    KdaParams p;
+    void operator()(int h, int vs, int tid, int row0, int nrows, int slot) const {
+        if (vs == 0 && tid < kD) kda_update_conv_history(p, row0, nrows, slot, h * kD + tid);
+    }
+};
+
 template <class K>
-static void launch(K kernel, int gx, int gy, int nthreads, const KdaParams& p, const KdaScratch& w, const KdaChunkWs& cw) {
+static void launch(K kernel, int gx, int gy, int nthreads) {
     for (int by = 0; by < gy; ++by)
         for (int bx = 0; bx < gx; ++bx) {
             std::barrier<> bar(nthreads);
@@ -57,9 +64,9 @@ static void launch(K kernel, int gx, int gy, int nthreads, const KdaParams& p, c
             for (int i = 0; i < 8; ++i) { wb.emplace_back(new std::barrier<>(32)); g_warp_bar[i] = wb.back().get(); }
             std::vector<std::thread> th;
             for (int t = 0; t < nthreads; ++t)
-                th.emplace_back([=, &p, &w, &cw] {
+                th.emplace_back([=] {
                     threadIdx.x = t; blockIdx.x = bx; blockIdx.y = by;
-                    kernel(p, w, cw);
+                    kernel();
                 });
             for (auto& x : th) x.join();
         }
@@ -114,13 +121,13 @@ int main(int argc, char** argv) {
     KdaParams p{};
     p.proj = proj.data(); p.ldp = ldp; p.off_q = 0; p.off_k = C; p.off_v = 2 * C; p.state = state.data(); p.conv_state = conv.data();
     p.seq_row0 = &h_row0; p.seq_nrows = &h_nrows; p.seq_slot = &h_slot; p.H = H;
-    KdaScratch w{qn.data(), kn.data(), vo.data(), decay.data(), gate.data(), beta.data(), nullptr, nullptr};
     const int nch = (rows + kCh - 1) / kCh;                  // the host sizes the grid from the step's row count (>= the sequence's rows)
-    std::vector<float> ws((size_t)nch * H * (2 * kCh * kCh + kD), -777.f);
-    KdaChunkWs cw{ws.data(), ws.data() + (size_t)nch * H * kCh * kCh, ws.data() + (size_t)2 * nch * H * kCh * kCh};
-    if (kChunkPrepSmem > sizeof(csm) || kChunkScanSmem > sizeof(csm)) { printf("shared memory buffer too small\n"); return 2; }
-    launch(kda_chunk_prep_kernel, nch, H, 256, p, w, cw);
-    launch(kda_chunk_scan_kernel, H, kD / kCh, 256, p, w, cw);
+    std::vector<float> ws((size_t)nch * H * ChunkDims<kD>::kWsFloats, -777.f);
+    DeltaChunkArgs ca{qn.data(), kn.data(), decay.data(), vo.data(), beta.data(), state.data(), &h_row0, &h_nrows, &h_slot, 1, 1, H, kD, 0,
+                      ws.data(), ws.data() + (size_t)nch * H * kCh * kCh, ws.data() + (size_t)2 * nch * H * kCh * kCh};
+    if (ChunkDims<kD>::kPrepSmem > sizeof(csm) || ChunkDims<kD>::kScanSmem > sizeof(csm)) { printf("shared memory buffer too small\n"); return 2; }
+    launch([=] { delta_chunk_prep_kernel<kD>(ca); }, nch, H, 256);
+    launch([=] { delta_chunk_scan_kernel<kD>(ca, Tail{p}); }, H, kD / kCh, 256);
     double eo = 0, mo = 0, es = 0, ms = 0;
     for (int t = 0; t < T; ++t)
         for (int c = 0; c < C; ++c) {
