@@ -269,6 +269,12 @@ def fill_model_from_checkpoint(cfg: dict) -> dict:
     hf = json.load(open(cj))
     hf = hf.get("text_config", hf)
     m = cfg["model"]
+    from ..models.config import NATIVE_CONFIGS
+    if str(hf.get("architecture", "")).lower() in NATIVE_CONFIGS:
+        # described by keys of its own: the section carries the shape's summary, the layers themselves stay in the checkpoint's config.json
+        from ..models.config import from_hf_config
+        m.update({k: v for k, v in model_section_from(from_hf_config(hf)).items() if k in m})
+        return cfg
     for k, v in hf.items():
         if k in m and isinstance(SCHEMA["model"].get(k), F) and m[k] in (0, None, [], ""):
             m[k] = v
@@ -284,6 +290,13 @@ def model_config_from(cfg: dict) -> ModelConfig:
     """The engine's ModelConfig for the ``model`` + ``quantization`` sections."""
     m = cfg["model"]
     q = cfg["quantization"]
+    from ..models.config import NATIVE_CONFIGS, from_hf_config
+    if m["architecture"] in NATIVE_CONFIGS:
+        d = m["weights_path"]
+        cj = os.path.join(d if os.path.isdir(d) else os.path.dirname(d), "config.json") if d else ""
+        if not os.path.exists(cj):
+            raise ConfigError([f"model.architecture {m['architecture']}: the layers are read from config.json in model.weights_path"])
+        return from_hf_config(cj)
     n = m["num_hidden_layers"]
     if not n or not m["hidden_size"]:
         raise ConfigError(["model: num_hidden_layers / hidden_size are not set and no checkpoint config.json was found"])

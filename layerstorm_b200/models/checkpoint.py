@@ -63,6 +63,17 @@ _GGUF_LAYER = {
     "mtp.enorm": "nextn.enorm.weight", "mtp.hnorm": "nextn.hnorm.weight", "mtp.eh_proj": "nextn.eh_proj.weight",
     "mtp.final_norm": "nextn.shared_head_norm.weight",
 }
+# canonical suffix -> tensor name behind "l<N>." (Gazutar)
+_GAZUTAR_LAYER = {
+    "mix_norm.weight": "norm1", "mix_norm.bias": "norm1.b", "ffn_norm.weight": "norm2", "ffn_norm.bias": "norm2.b",
+    "attn.q": "mix.q", "attn.k": "mix.k", "attn.v": "mix.v", "attn.g": "mix.g", "attn.o": "mix.o", "attn.q_norm": "mix.q.norm",
+    "attn.k_norm": "mix.k.norm", "attn.v_mix": "mix.vmix",
+    "kda.q": "mix.q", "kda.k": "mix.k", "kda.v": "mix.v", "kda.beta": "mix.b", "kda.f_a": "mix.a1", "kda.f_b": "mix.a2", "kda.g_a": "mix.g1",
+    "kda.g_b": "mix.g2", "kda.conv_q": "mix.q.conv", "kda.conv_k": "mix.k.conv", "kda.conv_v": "mix.v.conv", "kda.a_log": "mix.A_log",
+    "kda.dt_bias": "mix.dt_bias", "kda.o_norm": "mix.norm", "kda.o": "mix.o",
+    "moe.router": "mlp.router", "moe.router_bias": "mlp.correction",
+}
+_GAZUTAR_TOP = {"embed.weight": "embed", "head.weight": "head", "final_norm.weight": "final.norm", "final_norm.bias": "final.norm.b"}
 _LAYER_RE = re.compile(r"^layers\.(\d+)\.(.+)$")
 _EXPERT_RE = re.compile(r"^moe\.(experts|shared)\.(\d+)\.(gate|up|down)$")
 
@@ -199,7 +210,17 @@ class LazyCheckpoint(Mapping):
 
     # ---- resolution ----
     def _resolve(self, key: str) -> Optional[Callable[[], torch.Tensor]]:
-        return self._resolve_hf(key) if self.kind == "hf" else self._resolve_gguf(key)
+        return {"hf": self._resolve_hf, "gguf": self._resolve_gguf, "gazutar": self._resolve_gazutar}[self.kind](key)
+
+    def _resolve_gazutar(self, key: str):
+        m = _LAYER_RE.match(key)
+        if m is None:
+            name = _GAZUTAR_TOP.get(key)
+        else:
+            e = _EXPERT_RE.match(m.group(2))
+            rest = f"mlp.e{e.group(2)}.{e.group(3)}" if e and e.group(1) == "experts" else _GAZUTAR_LAYER.get(m.group(2))
+            name = f"l{m.group(1)}.{rest}" if rest else None
+        return (lambda: self.src.load(name)) if name and self.src.has(name) else None
 
     def _lin(self, path: str):
         s = self.src
@@ -472,6 +493,8 @@ def open_checkpoint(path: str, cfg: Optional[ModelConfig] = None) -> tuple[Model
     if cfg is None:
         cfg = from_hf_config(os.path.join(d, "config.json"))
     src = SafetensorsSource(d)
+    if cfg.architecture == "gazutar":
+        return cfg, LazyCheckpoint(cfg, src, "gazutar")
     skip = QuantSkipList.from_model_dir(d)
     if skip is not None and skip.quant_method in ("fp8", ""):
         dts, shp = {}, {}

@@ -16,7 +16,40 @@ import math
 from dataclasses import dataclass, field, asdict
 from typing import List, Optional
 
-ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next")
+ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar")
+
+
+@dataclass
+class BlockSpec:
+    """One layer of a model that is described layer by layer (``ModelConfig.blocks``): a mixer and an optional mixture-of-experts
+    feed-forward, each with sizes of its own."""
+    kind: str = "attention"           # "attention" | "channel_delta" (gated delta rule with a decay per key channel)
+    heads: int = 0                    # query heads (attention) / value heads (delta)
+    kv_heads: int = 0                 # key-value heads (attention) / query-key heads (delta); divides `heads`
+    dim: int = 0                      # query / key head width
+    vdim: int = 0                     # value head width
+    # attention
+    scale: float = 0.0
+    window: int = 0                   # sliding window: 0 <= i - j < window (0 = the whole prefix)
+    qk_norm: bool = False             # RMS norm over all rows of the q (and of the k) projection
+    alibi: bool = False               # linear distance bias, slope 2^(-8 (h + 1) / heads)
+    out_gate: bool = False            # heads times sigmoid(W_g h) in front of the output projection
+    v_mix: bool = False               # values mixed with those of the first such layer
+    # delta rule
+    conv: int = 0                     # taps of the short causal convolutions
+    decay: str = "softplus"           # log decay: "softplus" -exp(A) softplus(x) | "bounded" decay_bound * sigmoid(exp(A) x)
+    decay_bound: float = -5.0
+    # feed-forward (experts 0: none)
+    experts: int = 0
+    identity: int = 0                 # router outputs behind the experts whose "expert" is the input itself
+    top: int = 0
+    groups: int = 1
+    keep: int = 1                     # groups a token may choose from
+    ff: int = 0
+
+    @property
+    def recurrent(self) -> bool:
+        return self.kind == "channel_delta"
 
 
 @dataclass
@@ -81,8 +114,16 @@ class ModelConfig:
     expert_quant: str = "bf16"        # bf16 | fp8_e4m3 | nvfp4 | gguf_q4_k ...
     dense_quant: str = "bf16"         # attention / dense FFN / shared expert
     eos_token_ids: List[int] = field(default_factory=list)
+    # models described layer by layer (models/block_model.py); empty for the MLA family
+    blocks: List[BlockSpec] = field(default_factory=list)
+    norm_kind: str = "rms"            # "rms" | "layer" (with bias): the norms of the residual stream
+    logit_scale: float = 1.0
 
     def __post_init__(self):
+        self.blocks = [b if isinstance(b, BlockSpec) else BlockSpec(**b) for b in self.blocks]
+        if self.blocks:
+            self.n_layers = len(self.blocks)
+            self.layer_types = [b.kind for b in self.blocks]
         if not self.layer_types:
             self.layer_types = ["mla"] * self.n_layers
         assert len(self.layer_types) == self.n_layers
@@ -102,6 +143,8 @@ class ModelConfig:
         return self.hc_mult > 1
 
     def is_moe_layer(self, i: int) -> bool:
+        if self.blocks:
+            return i < len(self.blocks) and self.blocks[i].experts > 0
         return i >= self.first_k_dense and self.n_routed > 0
 
     def is_hash_layer(self, i: int) -> bool:
@@ -109,7 +152,8 @@ class ModelConfig:
         return self.is_moe_layer(i) and i < self.num_hash_layers
 
     def is_kda_layer(self, i: int) -> bool:
-        return i < len(self.layer_types) and self.layer_types[i] == "kda"       # multi-token-prediction blocks (i >= n_layers) are MLA layers
+        """The layer keeps a recurrent state per sequence (KDA, or a delta-rule block) instead of a KV cache."""
+        return i < len(self.layer_types) and self.layer_types[i] in ("kda", "channel_delta")       # multi-token-prediction blocks (i >= n_layers) are MLA layers
 
     def mla_layers(self) -> List[int]:
         return [i for i in range(self.n_layers) if not self.is_kda_layer(i)]
@@ -229,7 +273,31 @@ def glm_5_3_flash() -> ModelConfig:
         eos_token_ids=[154820, 154827, 154829])
 
 
+def _gazutar(name, width, n_layers, vocab, attn, delta, router, ff, every=3, scale=None) -> ModelConfig:
+    """A Gazutar shape: every ``every``-th layer is attention, the others are delta-rule layers."""
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": router}
+    layers = [{"type": "attention", "mixer": attn, "mlp": mlp} if i % every == every - 1 else {"type": "channel_delta", "mixer": delta, "mlp": mlp}
+              for i in range(n_layers)]
+    return gazutar_config({"name": name, "layers": layers, "logit_scale": scale or 1.0, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width})
+
+
+def tiny_gazutar() -> ModelConfig:
+    """A small Gazutar shape for tests and smoke runs."""
+    return _gazutar("tiny-gazutar", 192, 5, 320, {"heads": 6, "kv_heads": 2, "dim": 32, "vdim": 48, "scale": 0.2, "mask": {"size": 40}, "v_mix": True},
+                    {"heads": 4, "kv_heads": 2, "dim": 48, "vdim": 32, "conv": 3},
+                    {"experts": 6, "identity": 2, "top": 2, "groups": {"count": 4, "keep": 2}}, 80, every=2, scale=0.5)
+
+
+def gazutar_flash() -> ModelConfig:
+    """A Gazutar shape with layers of a real model's size (the hidden size, KDA heads and expert width of the GLM-5.3-Flash shape)."""
+    return _gazutar("gazutar-flash", 4096, 8, 154880, {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 4096}, "v_mix": True},
+                    {"heads": 64, "kv_heads": 64, "dim": 128, "vdim": 128, "conv": 4},
+                    {"experts": 64, "identity": 8, "top": 8, "groups": {"count": 8, "keep": 4}}, 2048, every=4)
+
+
 PRESETS = {
+    "tiny-gazutar": tiny_gazutar,
+    "gazutar-flash": gazutar_flash,
     "tiny-mla-moe": tiny_mla_moe,
     "tiny-glm5-next": tiny_glm5_next,
     "tiny-deepseek-v32": tiny_deepseek_v32,
@@ -243,9 +311,50 @@ def get_preset(name: str) -> ModelConfig:
     return PRESETS[name.lower()]()
 
 
+def gazutar_config(c: dict) -> ModelConfig:
+    """Gazutar: post-norm residual stream with layer norms; windowed ALiBi attention with whole-projection query / key norms, value mixing
+    and an output gate, or gated delta-rule layers with a decay per key channel; grouped softmax routing with identity experts."""
+    blocks = []
+    for i, L in enumerate(c["layers"]):
+        m = L["mixer"]
+        b = BlockSpec(kind=L["type"], heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"])
+        if L["type"] == "attention":
+            b.scale, b.window, b.v_mix = float(m["scale"]), int((m.get("mask") or {}).get("size", 0)), bool(m.get("v_mix", False))
+            b.qk_norm = b.alibi = b.out_gate = True
+        elif L["type"] == "channel_delta":
+            b.conv = int(m["conv"])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
+        mlp = L.get("mlp")
+        if mlp:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            r = mlp["router"]
+            g = r.get("groups") or {}
+            b.experts, b.top, b.identity, b.ff = int(r["experts"]), int(r["top"]), int(r.get("identity", 0) or 0), int(mlp["expert"]["ff"])
+            b.groups, b.keep = int(g.get("count", 1)), int(g.get("keep", 1))
+        blocks.append(b)
+    moe = [b for b in blocks if b.experts]
+    att = [b for b in blocks if not b.recurrent]
+    rec = [b for b in blocks if b.recurrent]
+    return ModelConfig(
+        name=c.get("name", "Gazutar"), architecture="gazutar", hidden=c["width"], vocab=c["vocab"], rms_eps=float(c["norm"]["eps"]), norm_kind="layer",
+        logit_scale=float(c.get("logit_scale", 1.0)), blocks=blocks, n_heads=max((b.heads for b in att), default=1), q_lora=0, kv_lora=0, qk_nope=0, qk_rope=0,
+        v_head=max((b.vdim for b in att), default=0), dense_inter=0, first_k_dense=0, n_routed=max((b.experts for b in moe), default=0),
+        top_k=max((b.top for b in moe), default=0), n_shared=0, moe_inter=max((b.ff for b in moe), default=0), norm_topk_prob=False, router_bias=True,
+        kda_heads=max((b.heads for b in rec), default=0), kda_head_dim=max((b.dim for b in rec), default=0), max_position=int(c.get("max_position", 1 << 20)))
+
+
+# architectures whose config.json is described by its own keys ("architecture": name) rather than HuggingFace ones
+NATIVE_CONFIGS = {"gazutar": gazutar_config}
+
+
 def from_hf_config(path_or_dict) -> ModelConfig:
-    """Build a ModelConfig from a HuggingFace ``config.json`` (path or dict)."""
+    """Build a ModelConfig from a ``config.json`` (path or dict): HuggingFace keys, or the keys of a natively described architecture."""
     c = json.load(open(path_or_dict)) if isinstance(path_or_dict, str) else dict(path_or_dict)
+    native = NATIVE_CONFIGS.get(str(c.get("architecture", "")).lower())
+    if native is not None:
+        return native(c)
     c = c.get("text_config", c)
     mt = c.get("model_type", "")
     arch = {"deepseek_v3": "deepseek_v3", "deepseek_v32": "deepseek_v3", "glm_moe_dsa": "glm_moe_dsa",

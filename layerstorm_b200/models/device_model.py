@@ -26,7 +26,7 @@ from ..ops import _native as nat
 from .config import ModelConfig
 
 KV_FMT = {"bf16": 0, "fp8": 1, "tq4": 2}
-EXPERT_FMT = {"bf16": 0, "fp8_e4m3": 1, "nvfp4": 2, "gguf_q4_k": 3, "gguf_q5_k": 4, "gguf_q6_k": 5, "gguf_q8_0": 6}
+EXPERT_FMT = {"bf16": 0, "fp8_e4m3": 1, "nvfp4": 2, "gguf_q4_k": 3, "gguf_q5_k": 4, "gguf_q6_k": 5, "gguf_q8_0": 6, "f32": 7}
 _FMT_NAME = {v: k for k, v in EXPERT_FMT.items()}
 GGML_OF = {"gguf_q4_k": 12, "gguf_q5_k": 13, "gguf_q6_k": 14, "gguf_q8_0": 8}      # storage formats that are GGUF block types
 
@@ -64,8 +64,8 @@ def expert_layout(fmt: str, H: int, F: int, down_fmt: Optional[str] = None) -> E
         return ef
     if down_fmt not in (None, fmt):
         raise ValueError("a separate down format is only supported between GGUF block types")
-    if fmt == "bf16":
-        wb = H * F * 2
+    if fmt in ("bf16", "f32"):
+        wb = H * F * (2 if fmt == "bf16" else 4)
         ef.off_gate, ef.off_up, ef.off_down = 0, wb, 2 * wb
         ef.off_sg = ef.off_su = ef.off_sd = ef.off_tail = 3 * wb
         end = 3 * wb
@@ -364,7 +364,12 @@ class QLinear:
             self(out, x, M, ldx, ldo, bias, None)
             nat.call("lsb_comm_push_rows", out, M, self.N, ldo, comm)
             return
-        if self.fmt == "bf16" and M >= 8:
+        if x.dtype == torch.float32:
+            # full-precision mode: fp32 activations, weights and FMAs
+            if self.fmt != "f32" or ob or bias is not None or comm is not None:
+                raise RuntimeError("fp32 activations need fp32 weights and an fp32 output on one GPU")
+            nat.call("lsb_gemm_f32", out, x, self.w, M, self.N, self.K, ldx, self.K, ldo)
+        elif self.fmt == "bf16" and M >= 8:
             sc = TcScratch.get(self.w.device)
             nat.call("lsb_gemm_bf16_tc", out, x, self.w, bias, M, self.N, self.K, ldx, self.K, ldo, ob, sc.partial, sc.cap, sc.err, comm)
         elif (self.fmt == "nvfp4" and MOE_BLOCK_SCALED and M >= 16 and comm is None and bias is None and ldx == self.K and self.K % 256 == 0
@@ -494,6 +499,8 @@ class ExpertArena:
                                    ("down", (H, F), ef.off_down, ef.off_sd)):
             if fmt == "bf16":
                 out.append(v[ow: ow + N * K * 2].view(torch.bfloat16).view(N, K).float())
+            elif fmt == "f32":
+                out.append(v[ow: ow + N * K * 4].view(torch.float32).view(N, K).clone())
             elif fmt in GGML_OF:
                 from ..formats import gguf as _gguf
                 t = GGML_OF[fmt] if (nm != "down" or not ef.fmt_down1) else GGML_OF[_FMT_NAME[ef.fmt_down1 - 1]]
@@ -511,23 +518,67 @@ class ExpertArena:
         return out
 
 
-class Workspace:
+class StepBuffers:
+    """What every step of up to ``R`` rows has, whatever the model: the packed step inputs and the logits of ``n_logit_rows`` rows."""
+
+    def __init__(self, m: "ModelBase", R: int, n_logit_rows: int):
+        self.R, self.dev = R, m.device
+        # step inputs: one packed int32 buffer so a step needs a single host->device copy
+        self.inp = self.z(9, R, dtype=torch.int32)
+        self.inp[1].fill_(-1)
+        (self.tok, self.row_seq, self.row_pos, self.row_len, self.row_slot, self.n_entries,
+         self.seq_row0, self.seq_nrows, self.seq_slot) = (self.inp[j] for j in range(9))
+        # host-side facts of the staged step (Engine._stage): largest index-entry count of a row, one sequence or several, rows per sequence
+        self.ne_hint, self.single_seq, self.seq_rows = 0, False, [1] * R
+        # outputs
+        self.n_logit_rows = n_logit_rows
+        self.logits = self.z(n_logit_rows, m.V_local)
+        self.amax_part = self.z(n_logit_rows, 64, dtype=torch.int64)
+        self.out_tok = self.z(n_logit_rows, dtype=torch.int32)
+        self.out_val = self.z(n_logit_rows)
+
+    def z(self, *shape, dtype=torch.float32):
+        return torch.zeros(*shape, dtype=dtype, device=self.dev)
+
+
+class MoeBuffers:
+    """Buffers of a routed feed-forward over up to ``R`` rows with ``S`` slots per row and ``E`` expert ids: routing, the 4-row groups of the
+    weight-streaming kernels and - with ``tc`` - the expert-sorted operands of the tensor-core grouped kernel."""
+
+    def alloc_moe(self, z, R: int, S: int, E: int, n_logits: int, H: int, F: int, tc: bool, act_dtype=torch.bfloat16):
+        i32 = torch.int32
+        self.S = S
+        self.logits_r = z(R, n_logits)
+        self.ids = z(R, S, dtype=i32); self.wts = z(R, S)
+        self.max_groups = min(R * S, (R * S + 3) // 4 + E)
+        self.group_expert = z(self.max_groups, dtype=i32); self.group_n = z(self.max_groups, dtype=i32)
+        self.group_pairs = z(self.max_groups * 4, dtype=i32); self.n_groups = z(1, dtype=i32)
+        self.counts = z(2 * E + 2, dtype=i32)
+        self.act = z(R * S, F, dtype=act_dtype)
+        self.y = z(R * S, H)
+        self.miss = z(1, dtype=i32)
+        # tensor-core grouped path (many rows): expert-sorted fp16 operands and the device-built tile list
+        self.tc_ok = tc and R >= TC_MOE_MIN_ROWS and H % 128 == 0 and F % 128 == 0
+        self.bs_ok = self.bs_fp8 = False
+        if self.tc_ok:
+            P = R * S
+            avg = P / max(1, min(E, P))
+            self.tc_bn = 32 if avg <= 32 else (64 if avg <= 96 else 128)
+            self.tc_tiles = P // self.tc_bn + E + 1
+            self.tc_sorted = z(P, dtype=i32)
+            self.tc_tile_e = z(self.tc_tiles, dtype=i32); self.tc_tile_r0 = z(self.tc_tiles, dtype=i32)
+            self.tc_tile_n = z(self.tc_tiles, dtype=i32); self.tc_cnt = z(2, dtype=i32)
+
+
+class Workspace(StepBuffers, MoeBuffers):
     """Static activation buffers for steps of up to ``R`` rows."""
 
     def __init__(self, m: "DeviceModel", R: int, n_logit_rows: int, max_ctx: int):
         cfg, dev = m.cfg, m.device
         f32, b16, i32 = torch.float32, torch.bfloat16, torch.int32
         H, n = cfg.hidden, cfg.hc_mult
-        self.R = R
-
-        def z(*shape, dtype=f32):
-            return torch.zeros(*shape, dtype=dtype, device=dev)
-
-        # step inputs: one packed int32 buffer so a step needs a single host->device copy
-        self.inp = z(9, R, dtype=i32)
-        self.inp[1].fill_(-1)
-        (self.tok, self.row_seq, self.row_pos, self.row_len, self.row_slot, self.n_entries,
-         self.seq_row0, self.seq_nrows, self.seq_slot) = (self.inp[j] for j in range(9))
+        super().__init__(m, R, n_logit_rows)
+        z = self.z
         # activations
         self.x = z(R, H, dtype=b16)
         self.mtp_cat = z(R, 2 * H, dtype=b16) if m.mtp_layers else None       # [RMSNorm(embedding) ; RMSNorm(stream)] of an MTP block
@@ -582,7 +633,6 @@ class Workspace:
                 self.idx_kbf_rows = (self.max_entries + 127) // 128 * 128
                 self.idx_kbf = z(self.idx_kbf_rows, 128, dtype=b16)
                 self.idx_kscale = z(self.idx_kbf_rows)
-            self.ne_hint, self.single_seq = 0, False
             self.idx_w = z(R, cfg.index_n_heads)
             self.kstash = z(R, cfg.index_head_dim, dtype=b16)
         # FFN
@@ -592,26 +642,8 @@ class Workspace:
         if cfg.n_routed > 0:
             S = cfg.top_k + cfg.n_shared
             E_total = cfg.n_routed + cfg.n_shared
-            self.S = S
-            self.logits_r = z(R, cfg.n_routed)
-            self.ids = z(R, S, dtype=i32); self.wts = z(R, S)
-            self.max_groups = min(R * S, (R * S + 3) // 4 + E_total)
-            self.group_expert = z(self.max_groups, dtype=i32); self.group_n = z(self.max_groups, dtype=i32)
-            self.group_pairs = z(self.max_groups * 4, dtype=i32); self.n_groups = z(1, dtype=i32)
-            self.counts = z(2 * E_total + 2, dtype=i32)
-            self.act = z(R * S, cfg.moe_inter, dtype=b16)
-            self.y = z(R * S, H)
-            self.miss = z(1, dtype=i32)
-            # tensor-core grouped path (many rows): expert-sorted fp16 operands and the device-built tile list
-            self.tc_ok = R >= TC_MOE_MIN_ROWS and H % 64 == 0 and H % 128 == 0 and m.Fe % 128 == 0
+            self.alloc_moe(z, R, S, E_total, cfg.n_routed, H, cfg.moe_inter, tc=m.Fe % 128 == 0)
             if self.tc_ok:
-                P = R * S
-                avg = P / max(1, min(E_total, P))
-                self.tc_bn = 32 if avg <= 32 else (64 if avg <= 96 else 128)
-                self.tc_tiles = P // self.tc_bn + E_total + 1
-                self.tc_sorted = z(P, dtype=i32)
-                self.tc_tile_e = z(self.tc_tiles, dtype=i32); self.tc_tile_r0 = z(self.tc_tiles, dtype=i32)
-                self.tc_tile_n = z(self.tc_tiles, dtype=i32); self.tc_cnt = z(2, dtype=i32)
                 # block-scaled path (NVFP4 experts): both operands stay 4-bit, the activations are quantised in tile order
                 fmts = {L["arena"].ef.fmt for L in m.layers if L.get("arena") is not None}
                 self.bs_can = fmts == {2} and H % 256 == 0 and m.Fe % 256 == 0 and H <= 8192 and m.Fe <= 8192
@@ -620,15 +652,7 @@ class Workspace:
                 self.bs_fp8 = (fmts == {1} and H % 128 == 0 and m.Fe % 128 == 0 and H <= 8192 and m.Fe <= 8192 and m.streamer is None
                                and all(L["arena"].bs_scale_atoms() is not None for L in m.layers if L.get("arena") is not None))
                 self.bs_can = self.bs_can or self.bs_fp8
-                self.bs_ok = False
                 self._m, self._z = m, z
-        # outputs
-        self.n_logit_rows = n_logit_rows
-        self.logits = z(n_logit_rows, m.V_local)
-        self.amax_part = torch.zeros(n_logit_rows, 64, dtype=torch.int64, device=dev)
-        self.out_tok = z(n_logit_rows, dtype=i32)
-        self.out_val = z(n_logit_rows)
-
         if getattr(self, "tc_ok", False):
             self.set_block_scaled(MOE_BLOCK_SCALED)
 
@@ -655,44 +679,25 @@ class Workspace:
         return on
 
 
-class DeviceModel:
-    def __init__(self, cfg: ModelConfig, device="cuda", kv_fmt: str = "fp8", page: int = 64, tp_rank: int = 0, tp_size: int = 1,
-                 expert_shard: Optional[str] = None):
-        """``expert_shard``: how the experts are spread over ``tp_size`` GPUs - ``"ep"`` routed expert e lives whole on GPU e % N (the
-        shared expert of layer i on GPU i % N), ``"tp"`` every GPU holds a 1/N slice of EVERY expert (gate / up rows, down columns).
-        Both end in the same cross-rank sum.  ``"tp"`` gives every GPU the same work whatever the router picks, which is what a
-        decode step wants (with ``"ep"`` a token's 8 experts land 4-0-3-1 on 4 GPUs and the step waits for the fullest one);
-        default: ``LSB_EXPERT_SHARD``, else ``"tp"`` whenever the expert width divides into slices of 128."""
+class ModelBase:
+    """What the engine needs of any model on the device: the weight list, the paged / per-slot cache tables, greedy selection and the
+    step hooks.  ``kv_cache`` / ``idx_cache`` hold [pages, page, ...] tensors by layer, ``kda_state`` / ``kda_conv`` / ``idx_tail`` [slots, ...]
+    tensors of recurrent layers; forks, anchors, hibernation and spilling work on these tables whatever the layer kinds are."""
+
+    mixed_steps = False      # the server may run a joining prompt's slice and the running requests' tokens as one step
+
+    def _init_base(self, cfg: ModelConfig, device, kv_fmt: str, page: int, tp_rank: int, tp_size: int):
         self.cfg, self.device = cfg, torch.device(device)
-        if expert_shard is None:
-            expert_shard = os.environ.get("LSB_EXPERT_SHARD") or ("tp" if (tp_size > 1 and cfg.n_routed and cfg.moe_inter % (128 * tp_size) == 0) else "ep")
-        if expert_shard == "tp" and (tp_size == 1 or cfg.moe_inter % tp_size):
-            expert_shard = "ep"
-        self.expert_shard = expert_shard
-        self.Fe = cfg.moe_inter // tp_size if expert_shard == "tp" else cfg.moe_inter        # expert width held by this GPU
         self.kv_fmt, self.page = kv_fmt, page
-        assert page % max(cfg.index_kpool, 1) == 0
-        # Tensor / expert parallel layout (one process per GPU): attention heads, KDA heads, dense FFN
-        # columns and the LM-head vocabulary are split over the ranks; routed experts are owned by rank
-        # e % tp_size, the shared expert of layer i by rank i % tp_size; small projections are replicated.
         self.tp_rank, self.tp_size = tp_rank, tp_size
-        for v, nm in ((cfg.n_heads, "n_heads"), (cfg.dense_inter, "dense_inter"), (cfg.vocab, "vocab")):
-            assert v % tp_size == 0, f"{nm}={v} not divisible by tp={tp_size}"
-        assert cfg.kda_heads % tp_size == 0
-        self.Hh = cfg.n_heads // tp_size
-        self.Hk = cfg.kda_heads // tp_size
-        self.Fd = cfg.dense_inter // tp_size
         self.V_local = cfg.vocab // tp_size
-        self._fused = False
         self.dcp = None
-        self.idx_identity = False  # the indexer's key cache keeps a page table of its own (row-granular KV tiering: its pages never leave HBM)
-        self.skip_layers = frozenset()   # layers whose attention + FFN a step leaves out (self-speculative drafting; never the first or last)
+        self.skip_layers = frozenset()   # layers whose mixer + FFN a step leaves out (self-speculative drafting; never the first or last)
         self.probe = None                # {"prev": bf16 [1, hidden], "sims": fp32 [n_layers]} while layer-input similarities are recorded
         self.aux_capture = None          # {"slots": {layer: column}, "buf": bf16 [rows, n_aux, hidden]}: layer inputs kept for a block draft model
         self.row_tier = None      # RowTiering (runtime/kv_tiering.py) when old KV pages of active sequences live in pinned host memory
         self.streamer = None      # ExpertStreamer when the VRAM expert cache is capped (runtime/streaming.py)
         self.drift = None         # dict: eager steps store every layer's output rows here (input of utils/determinism_probe.py drift)
-        self.tq_centroids = None  # TurboQuant reconstruction levels (kv_fmt "tq4")
         self.comm = None          # PeerComm for the fused all-reduces
         self.comm_amax = None     # PeerComm for the argmax exchange
         self.layers: List[dict] = []
@@ -701,13 +706,6 @@ class DeviceModel:
         self.head: Optional[QLinear] = None
         self.final_norm = None
         self.max_proj = 1
-        self.max_qb = 1
-        self.kv_row_bytes = nat.call("lsb_kv_row_bytes", KV_FMT[kv_fmt], cfg.kv_lora, cfg.qk_rope)
-        self.idx_row_bytes = nat.call("lsb_indexer_row_bytes")
-        inv = cfg.rope_inv_freq()
-        self.inv_freq = torch.tensor(inv if inv else [0.0], dtype=torch.float32, device=self.device)
-        inv_i = cfg.rope_inv_freq(cfg.index_rope_dim) if cfg.index_rope_dim else [0.0]
-        self.inv_freq_idx = torch.tensor(inv_i, dtype=torch.float32, device=self.device)
         # caches (allocated by alloc_cache)
         self.kv_cache: Dict[int, torch.Tensor] = {}
         self.idx_cache: Dict[int, torch.Tensor] = {}
@@ -716,6 +714,199 @@ class DeviceModel:
         self.kda_conv: Dict[int, torch.Tensor] = {}
         self.block_table = None
         self.kernel_launches = 0
+
+    def reset_slot(self, slot: int):
+        for t in self.kda_state.values():
+            t[slot].zero_()
+        for t in self.kda_conv.values():
+            t[slot].zero_()
+
+    def weight_bytes(self) -> int:
+        tot = self.head.nbytes() + (self.embed.numel() * 2 if self.embed.is_cuda else 0)
+        for L in self.layers + self.mtp_layers:
+            for v in L.values():
+                if isinstance(v, QLinear):
+                    tot += v.nbytes()
+                elif isinstance(v, ExpertArena):
+                    tot += v.data.numel()
+                elif isinstance(v, torch.Tensor):
+                    tot += v.numel() * v.element_size()
+                elif isinstance(v, tuple):
+                    tot += sum(t.numel() * t.element_size() for t in v if t is not None)
+        return tot
+
+    # ------------------------------------------------------------------ routed experts of a step
+    def moe_mode(self, arena: "ExpertArena", ws, R: int) -> str:
+        if getattr(ws, "tc_ok", False) and R >= TC_MOE_MIN_ROWS and arena.ef.fmt <= 3 and not arena.ef.fmt_down1:
+            return "tc"
+        fast_fp4 = arena.ef.fmt == 2 and arena.ef.F % 128 == 0 and arena.ef.H % 128 == 0
+        return "pairs" if (fast_fp4 and R * ws.S <= 72) else "groups"
+
+    def moe_prepare(self, arena: "ExpertArena", ws, x, R: int, E: int):
+        """Group the step's (row, slot) pairs by expert (once per layer, independent of residency).  Ids outside [0, E) take no part."""
+        S, H = ws.S, arena.ef.H
+        mode = self.moe_mode(arena, ws, R)
+        if mode == "tc":
+            P = R * S
+            nat.call("lsb_moe_tc_sort", ws.ids, P, E, ws.tc_bn, ws.tc_sorted, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt)
+            if ws.bs_ok:
+                nat.call("lsb_quant_fp8_tiles" if ws.bs_fp8 else "lsb_quant_nvfp4_tiles", x, 0, ws.tc_sorted, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt,
+                         S, H, ws.tc_bn, min(ws.tc_tiles, P // ws.tc_bn + E + 1), ws.bs_xq, ws.bs_xsf, ws.bs_xa)
+            else:
+                nat.call("lsb_moe_tc_gather", x, ws.tc_sorted, ws.tc_cnt, ws.tc_xs, P, S, H)
+        elif mode == "groups":
+            nat.call("lsb_moe_build_groups", ws.ids, R * S, E, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups, ws.counts)
+
+    def moe_experts(self, arena: "ExpertArena", ws, x, R: int, E: int, limit: float, miss):
+        """gate/up + SwiGLU and down projections of every pair whose expert is resident (``arena.slot_of[e] >= 0``)."""
+        S = ws.S
+        efp = ctypes.addressof(arena.ef)
+        mode = self.moe_mode(arena, ws, R)
+        if mode == "tc":
+            P = R * S
+            err = TcScratch.get(self.device).err
+            tiles = min(ws.tc_tiles, P // ws.tc_bn + E + 1)
+            if ws.bs_ok and ws.bs_fp8:
+                wsf, og, ou, od = arena.bs_scale_atoms()
+                a = (arena.data, arena.slot_of, efp, wsf, wsf.shape[1], og, ou, od, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, ws.tc_sorted)
+                nat.call("lsb_moe_bs_ffn_fp8", 1, ws.bs_xq, ws.bs_xsf, ws.bs_xa, *a, ws.bs_act, ws.tc_bn, tiles, limit, miss, err)
+                nat.call("lsb_quant_fp8_tiles", ws.bs_act, 1, None, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, S, arena.ef.F, ws.tc_bn, tiles,
+                         ws.bs_aq, ws.bs_asf, ws.bs_aa)
+                nat.call("lsb_moe_bs_ffn_fp8", 0, ws.bs_aq, ws.bs_asf, ws.bs_aa, *a, ws.y, ws.tc_bn, tiles, 0.0, None, err)
+                return
+            if ws.bs_ok:
+                a = (arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, ws.tc_sorted)
+                nat.call("lsb_moe_bs_ffn", 1, ws.bs_xq, ws.bs_xsf, ws.bs_xa, *a, ws.bs_act, ws.tc_bn, tiles, limit, miss, err)
+                nat.call("lsb_quant_nvfp4_tiles", ws.bs_act, 1, None, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, S, arena.ef.F, ws.tc_bn, tiles,
+                         ws.bs_aq, ws.bs_asf, ws.bs_aa)
+                nat.call("lsb_moe_bs_ffn", 0, ws.bs_aq, ws.bs_asf, ws.bs_aa, *a, ws.y, ws.tc_bn, tiles, 0.0, None, err)
+                return
+            nat.call("lsb_moe_tc_ffn", 1, ws.tc_xs, ws.tc_xs.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
+                     ws.tc_cnt, ws.tc_sorted, ws.tc_act, ws.tc_bn, tiles, limit, miss, err, None)
+            nat.call("lsb_moe_tc_ffn", 0, ws.tc_act, ws.tc_act.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
+                     ws.tc_cnt, ws.tc_sorted, ws.y, ws.tc_bn, tiles, 0.0, None, err, None)
+        elif mode == "pairs":
+            # small batch: every (row, slot) pair streams its expert on its own - no grouping pass
+            # blocks per expert: finer when this GPU holds only a share of the step's experts (expert parallel), see the kernels
+            # (sliced experts keep every expert on every GPU with 1/N of the rows of gate / up and 1/N of the columns of down: the
+            # down projection keeps its row count, so it keeps the widest block)
+            run_gu = MOE_RUN_GU or (8 if self.tp_size == 1 else (4 if self.tp_size == 2 else 2))
+            run_dn = MOE_RUN_DN or (16 if self.tp_size == 1 or self.expert_shard == "tp" else (8 if self.tp_size == 2 else 4))
+            nat.call("lsb_moe_gateup", x, arena.data, arena.slot_of, efp, ws.ids, None, None, None, ws.act, S, R * S, limit, miss, run_gu)
+            nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.ids, None, None, None, ws.y, R * S, run_dn)
+        else:
+            mg = min(ws.max_groups, min(R * S, (R * S + 3) // 4 + E))
+            nat.call("lsb_moe_gateup", x, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,
+                     ws.act, S, mg, limit, miss, 0)
+            nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,
+                     ws.y, mg, 0)
+
+    # ------------------------------------------------------------------ step hooks
+    @staticmethod
+    def _resid_rows(ws, R: int, H: int) -> torch.Tensor:
+        return ws.resid.view(-1)[: ws.R * H].view(ws.R, H)[:R]
+
+    def set_aux_capture(self, layer_ids=(), rows: int = 0):
+        """Keep, for every step from now on, the stream that ENTERS each layer of ``layer_ids`` (hyper-connection models: the mean over
+        the residual streams; ``n_layers`` = the stream leaving the last layer, models without hyper-connections only) for the step's
+        rows: ``aux_capture["buf"][:R].view(R, -1)`` is the concatenation in the order of ``layer_ids`` - the features a block draft
+        model is conditioned on (``speculation/dspark.py``).  The copies are part of the step (and of its CUDA graph): the caller
+        drops graphs captured before.  An empty ``layer_ids`` switches the capture off.
+        Reference: the aux-hidden export hook in front of every layer's attention (src/daemon/dispatch_forward.cpp)."""
+        ids = [int(l) for l in layer_ids]
+        if not ids:
+            self.aux_capture = None
+            return
+        n = self.cfg.n_layers
+        if self.tp_size > 1:
+            raise NotImplementedError("aux hidden capture is built for one GPU")
+        if any(l < 0 or l > n or (l == n and self.cfg.mhc) for l in ids) or len(set(ids)) != len(ids):
+            raise ValueError(f"aux layers {ids} do not fit a model of {n} layers" + (" with hyper-connections (no un-normalised final stream)" if self.cfg.mhc else ""))
+        self.aux_capture = {"slots": {l: j for j, l in enumerate(ids)},
+                            "buf": torch.zeros(max(1, int(rows)), len(ids), self.cfg.hidden, dtype=torch.bfloat16, device=self.device)}
+
+    def _capture_aux(self, i: int, ws, R: int):
+        ac = self.aux_capture
+        j = ac["slots"].get(i)
+        if j is None:
+            return
+        if R > ac["buf"].shape[0]:
+            raise RuntimeError(f"a step of {R} rows exceeds the aux capture buffer ({ac['buf'].shape[0]} rows)")
+        H = self.cfg.hidden
+        if self.cfg.mhc:
+            ac["buf"][:R, j].copy_(ws.resid[:R].mean(1))
+        else:
+            ac["buf"][:R, j].copy_(self._resid_rows(ws, R, H))
+
+    def set_layer_skip(self, skip=(), probe: bool = False):
+        """Layer skipping for draft passes: ``skip`` = layers to leave out (the first and the last layer are never skipped), ``probe`` =
+        record, per executed layer l, the cosine similarity between the normalised input of l and of the next executed layer (row 0 of
+        the step) in ``self.probe["sims"][l]`` - "how much did layer l change its input".  Reference: layer skip during the
+        self-speculative draft (python/orchestrator/layer_skip.py; src/compute/kernels/similarity/cosine_sim.h)."""
+        n = self.cfg.n_layers
+        self.skip_layers = frozenset(int(l) for l in skip if 0 < int(l) < n - 1)
+        if probe and self.probe is None:
+            self.probe = {"prev": torch.zeros(1, self.cfg.hidden, dtype=torch.bfloat16, device=self.device),
+                          "sims": torch.zeros(n, dtype=torch.float32, device=self.device)}
+        if not probe:
+            self.probe = None
+
+    def _probe_input(self, i: int, ws, last: int) -> int:
+        """Called when ``ws.x`` holds the input of layer i; ``last`` = the previously executed layer (-1 for none)."""
+        pr = self.probe
+        if pr is None:
+            return i
+        H = self.cfg.hidden
+        if last >= 0:
+            nat.call("lsb_cosine_sim", pr["prev"], ws.x, 1, H, H, H, pr["sims"][last: last + 1])
+        pr["prev"].copy_(ws.x[:1])
+        return i
+
+    def argmax(self, ws, n_rows: int):
+        """Greedy token per row; with a vocabulary-parallel head the per-rank winners are exchanged
+        in-kernel over NVLink (8 bytes per row per rank)."""
+        nat.call("lsb_argmax", ws.logits, self.V_local, n_rows, self.V_local, ws.amax_part, ws.out_tok, ws.out_val,
+                 self.tp_rank * self.V_local, self.comm_amax.ptr if self.comm_amax is not None else None)
+
+
+class DeviceModel(ModelBase):
+    def __init__(self, cfg: ModelConfig, device="cuda", kv_fmt: str = "fp8", page: int = 64, tp_rank: int = 0, tp_size: int = 1,
+                 expert_shard: Optional[str] = None):
+        """``expert_shard``: how the experts are spread over ``tp_size`` GPUs - ``"ep"`` routed expert e lives whole on GPU e % N (the
+        shared expert of layer i on GPU i % N), ``"tp"`` every GPU holds a 1/N slice of EVERY expert (gate / up rows, down columns).
+        Both end in the same cross-rank sum.  ``"tp"`` gives every GPU the same work whatever the router picks, which is what a
+        decode step wants (with ``"ep"`` a token's 8 experts land 4-0-3-1 on 4 GPUs and the step waits for the fullest one);
+        default: ``LSB_EXPERT_SHARD``, else ``"tp"`` whenever the expert width divides into slices of 128."""
+        self._init_base(cfg, device, kv_fmt, page, tp_rank, tp_size)
+        if expert_shard is None:
+            expert_shard = os.environ.get("LSB_EXPERT_SHARD") or ("tp" if (tp_size > 1 and cfg.n_routed and cfg.moe_inter % (128 * tp_size) == 0) else "ep")
+        if expert_shard == "tp" and (tp_size == 1 or cfg.moe_inter % tp_size):
+            expert_shard = "ep"
+        self.expert_shard = expert_shard
+        self.Fe = cfg.moe_inter // tp_size if expert_shard == "tp" else cfg.moe_inter        # expert width held by this GPU
+        assert page % max(cfg.index_kpool, 1) == 0
+        # Tensor / expert parallel layout (one process per GPU): attention heads, KDA heads, dense FFN
+        # columns and the LM-head vocabulary are split over the ranks; routed experts are owned by rank
+        # e % tp_size, the shared expert of layer i by rank i % tp_size; small projections are replicated.
+        for v, nm in ((cfg.n_heads, "n_heads"), (cfg.dense_inter, "dense_inter"), (cfg.vocab, "vocab")):
+            assert v % tp_size == 0, f"{nm}={v} not divisible by tp={tp_size}"
+        assert cfg.kda_heads % tp_size == 0
+        self.Hh = cfg.n_heads // tp_size
+        self.Hk = cfg.kda_heads // tp_size
+        self.Fd = cfg.dense_inter // tp_size
+        self._fused = False
+        self.idx_identity = False  # the indexer's key cache keeps a page table of its own (row-granular KV tiering: its pages never leave HBM)
+        self.tq_centroids = None  # TurboQuant reconstruction levels (kv_fmt "tq4")
+        self.max_qb = 1
+        self.kv_row_bytes = nat.call("lsb_kv_row_bytes", KV_FMT[kv_fmt], cfg.kv_lora, cfg.qk_rope)
+        self.idx_row_bytes = nat.call("lsb_indexer_row_bytes")
+        inv = cfg.rope_inv_freq()
+        self.inv_freq = torch.tensor(inv if inv else [0.0], dtype=torch.float32, device=self.device)
+        inv_i = cfg.rope_inv_freq(cfg.index_rope_dim) if cfg.index_rope_dim else [0.0]
+        self.inv_freq_idx = torch.tensor(inv_i, dtype=torch.float32, device=self.device)
+
+    def make_workspace(self, R: int, n_logit_rows: int, max_ctx: int) -> Workspace:
+        return Workspace(self, R, n_logit_rows, max_ctx)
 
     def attach_comm(self, comm, comm_amax):
         self.comm, self.comm_amax = comm, comm_amax
@@ -1100,20 +1291,6 @@ class DeviceModel:
                 self.max_qb = max(self.max_qb, L["mla_qb"].N)
         self._ef_bytes = {}
 
-    def weight_bytes(self) -> int:
-        tot = self.head.nbytes() + (self.embed.numel() * 2 if self.embed.is_cuda else 0)
-        for L in self.layers + self.mtp_layers:
-            for v in L.values():
-                if isinstance(v, QLinear):
-                    tot += v.nbytes()
-                elif isinstance(v, ExpertArena):
-                    tot += v.data.numel()
-                elif isinstance(v, torch.Tensor):
-                    tot += v.numel() * v.element_size()
-                elif isinstance(v, tuple):
-                    tot += sum(t.numel() * t.element_size() for t in v)
-        return tot
-
     # ------------------------------------------------------------------ caches
     def alloc_cache(self, num_pages: int, n_slots: int, max_pages_per_seq: int):
         cfg, dev = self.cfg, self.device
@@ -1140,12 +1317,6 @@ class DeviceModel:
         for k in range(len(self.mtp_layers)):
             # a multi-token-prediction block keeps its own latent cache over the same pages (same positions, same page table)
             self.kv_cache[cfg.n_layers + k] = torch.zeros(num_pages, self.page, self.kv_row_bytes, dtype=torch.uint8, device=dev)
-
-    def reset_slot(self, slot: int):
-        for t in self.kda_state.values():
-            t[slot].zero_()
-        for t in self.kda_conv.values():
-            t[slot].zero_()
 
     def cache_bytes_per_token(self) -> int:
         cfg = self.cfg
@@ -1201,73 +1372,11 @@ class DeviceModel:
         self._reduce(ws, R)
         return False
 
-    def _moe_mode(self, arena: ExpertArena, ws: Workspace, R: int) -> str:
-        cfg = self.cfg
-        if getattr(ws, "tc_ok", False) and R >= TC_MOE_MIN_ROWS and arena.ef.fmt <= 3 and not arena.ef.fmt_down1:
-            return "tc"
-        fast_fp4 = arena.ef.fmt == 2 and self.Fe % 128 == 0 and cfg.hidden % 128 == 0
-        return "pairs" if (fast_fp4 and R * ws.S <= 72) else "groups"
-
     def _moe_prepare(self, arena: ExpertArena, ws: Workspace, R: int):
-        """Group the step's (row, slot) pairs by expert (once per layer, independent of residency)."""
-        cfg, S = self.cfg, ws.S
-        E_total = cfg.n_routed + cfg.n_shared
-        mode = self._moe_mode(arena, ws, R)
-        if mode == "tc":
-            P = R * S
-            nat.call("lsb_moe_tc_sort", ws.ids, P, E_total, ws.tc_bn, ws.tc_sorted, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt)
-            if ws.bs_ok:
-                nat.call("lsb_quant_fp8_tiles" if ws.bs_fp8 else "lsb_quant_nvfp4_tiles", ws.x, 0, ws.tc_sorted, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt,
-                         S, cfg.hidden, ws.tc_bn, min(ws.tc_tiles, P // ws.tc_bn + E_total + 1), ws.bs_xq, ws.bs_xsf, ws.bs_xa)
-            else:
-                nat.call("lsb_moe_tc_gather", ws.x, ws.tc_sorted, ws.tc_cnt, ws.tc_xs, P, S, cfg.hidden)
-        elif mode == "groups":
-            nat.call("lsb_moe_build_groups", ws.ids, R * S, E_total, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups, ws.counts)
+        self.moe_prepare(arena, ws, ws.x, R, self.cfg.n_routed + self.cfg.n_shared)
 
     def _moe_experts(self, arena: ExpertArena, ws: Workspace, R: int, miss):
-        """gate/up + SwiGLU and down projections of every pair whose expert is resident (``arena.slot_of[e] >= 0``)."""
-        cfg, S = self.cfg, ws.S
-        E_total = cfg.n_routed + cfg.n_shared
-        efp = ctypes.addressof(arena.ef)
-        mode = self._moe_mode(arena, ws, R)
-        if mode == "tc":
-            P = R * S
-            err = TcScratch.get(self.device).err
-            tiles = min(ws.tc_tiles, P // ws.tc_bn + E_total + 1)
-            if ws.bs_ok and ws.bs_fp8:
-                wsf, og, ou, od = arena.bs_scale_atoms()
-                a = (arena.data, arena.slot_of, efp, wsf, wsf.shape[1], og, ou, od, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, ws.tc_sorted)
-                nat.call("lsb_moe_bs_ffn_fp8", 1, ws.bs_xq, ws.bs_xsf, ws.bs_xa, *a, ws.bs_act, ws.tc_bn, tiles, cfg.swiglu_limit, miss, err)
-                nat.call("lsb_quant_fp8_tiles", ws.bs_act, 1, None, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, S, self.Fe, ws.tc_bn, tiles,
-                         ws.bs_aq, ws.bs_asf, ws.bs_aa)
-                nat.call("lsb_moe_bs_ffn_fp8", 0, ws.bs_aq, ws.bs_asf, ws.bs_aa, *a, ws.y, ws.tc_bn, tiles, 0.0, None, err)
-                return
-            if ws.bs_ok:
-                a = (arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, ws.tc_sorted)
-                nat.call("lsb_moe_bs_ffn", 1, ws.bs_xq, ws.bs_xsf, ws.bs_xa, *a, ws.bs_act, ws.tc_bn, tiles, cfg.swiglu_limit, miss, err)
-                nat.call("lsb_quant_nvfp4_tiles", ws.bs_act, 1, None, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, S, self.Fe, ws.tc_bn, tiles,
-                         ws.bs_aq, ws.bs_asf, ws.bs_aa)
-                nat.call("lsb_moe_bs_ffn", 0, ws.bs_aq, ws.bs_asf, ws.bs_aa, *a, ws.y, ws.tc_bn, tiles, 0.0, None, err)
-                return
-            nat.call("lsb_moe_tc_ffn", 1, ws.tc_xs, ws.tc_xs.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
-                     ws.tc_cnt, ws.tc_sorted, ws.tc_act, ws.tc_bn, tiles, cfg.swiglu_limit, miss, err, None)
-            nat.call("lsb_moe_tc_ffn", 0, ws.tc_act, ws.tc_act.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
-                     ws.tc_cnt, ws.tc_sorted, ws.y, ws.tc_bn, tiles, 0.0, None, err, None)
-        elif mode == "pairs":
-            # small batch: every (row, slot) pair streams its expert on its own - no grouping pass
-            # blocks per expert: finer when this GPU holds only a share of the step's experts (expert parallel), see the kernels
-            # (sliced experts keep every expert on every GPU with 1/N of the rows of gate / up and 1/N of the columns of down: the
-            # down projection keeps its row count, so it keeps the widest block)
-            run_gu = MOE_RUN_GU or (8 if self.tp_size == 1 else (4 if self.tp_size == 2 else 2))
-            run_dn = MOE_RUN_DN or (16 if self.tp_size == 1 or self.expert_shard == "tp" else (8 if self.tp_size == 2 else 4))
-            nat.call("lsb_moe_gateup", ws.x, arena.data, arena.slot_of, efp, ws.ids, None, None, None, ws.act, S, R * S, cfg.swiglu_limit, miss, run_gu)
-            nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.ids, None, None, None, ws.y, R * S, run_dn)
-        else:
-            mg = min(ws.max_groups, min(R * S, (R * S + 3) // 4 + E_total))
-            nat.call("lsb_moe_gateup", ws.x, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,
-                     ws.act, S, mg, cfg.swiglu_limit, miss, 0)
-            nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,
-                     ws.y, mg, 0)
+        self.moe_experts(arena, ws, ws.x, R, self.cfg.n_routed + self.cfg.n_shared, self.cfg.swiglu_limit, miss)
 
     def _kda(self, i: int, L: dict, ws: Workspace, R: int, nseq: int):
         cfg = self.cfg
@@ -1388,62 +1497,6 @@ class DeviceModel:
         nat.call("lsb_mhc_post_pre", ws.x, ws.resid, ws.sub, ws.post, ws.comb, fn, sc, base, norm_w, ws.part, R, H, n,
                  mode, cfg.hc_sinkhorn_iters, cfg.hc_eps, cfg.rms_eps, cfg.hc_post_mult, ws.hc_done, ws.hc_pre, self._cp)
 
-    def set_aux_capture(self, layer_ids=(), rows: int = 0):
-        """Keep, for every step from now on, the stream that ENTERS each layer of ``layer_ids`` (hyper-connection models: the mean over
-        the residual streams; ``n_layers`` = the stream leaving the last layer, models without hyper-connections only) for the step's
-        rows: ``aux_capture["buf"][:R].view(R, -1)`` is the concatenation in the order of ``layer_ids`` - the features a block draft
-        model is conditioned on (``speculation/dspark.py``).  The copies are part of the step (and of its CUDA graph): the caller
-        drops graphs captured before.  An empty ``layer_ids`` switches the capture off.
-        Reference: the aux-hidden export hook in front of every layer's attention (src/daemon/dispatch_forward.cpp)."""
-        ids = [int(l) for l in layer_ids]
-        if not ids:
-            self.aux_capture = None
-            return
-        n = self.cfg.n_layers
-        if self.tp_size > 1:
-            raise NotImplementedError("aux hidden capture is built for one GPU")
-        if any(l < 0 or l > n or (l == n and self.cfg.mhc) for l in ids) or len(set(ids)) != len(ids):
-            raise ValueError(f"aux layers {ids} do not fit a model of {n} layers" + (" with hyper-connections (no un-normalised final stream)" if self.cfg.mhc else ""))
-        self.aux_capture = {"slots": {l: j for j, l in enumerate(ids)},
-                            "buf": torch.zeros(max(1, int(rows)), len(ids), self.cfg.hidden, dtype=torch.bfloat16, device=self.device)}
-
-    def _capture_aux(self, i: int, ws: Workspace, R: int):
-        ac = self.aux_capture
-        j = ac["slots"].get(i)
-        if j is None:
-            return
-        if R > ac["buf"].shape[0]:
-            raise RuntimeError(f"a step of {R} rows exceeds the aux capture buffer ({ac['buf'].shape[0]} rows)")
-        H = self.cfg.hidden
-        if self.cfg.mhc:
-            ac["buf"][:R, j].copy_(ws.resid[:R].mean(1))
-        else:
-            ac["buf"][:R, j].copy_(ws.resid.view(-1)[: ws.R * H].view(ws.R, H)[:R])
-
-    def set_layer_skip(self, skip=(), probe: bool = False):
-        """Layer skipping for draft passes: ``skip`` = layers to leave out (the first and the last layer are never skipped), ``probe`` =
-        record, per executed layer l, the cosine similarity between the normalised input of l and of the next executed layer (row 0 of
-        the step) in ``self.probe["sims"][l]`` - "how much did layer l change its input".  Reference: layer skip during the
-        self-speculative draft (python/orchestrator/layer_skip.py; src/compute/kernels/similarity/cosine_sim.h)."""
-        n = self.cfg.n_layers
-        self.skip_layers = frozenset(int(l) for l in skip if 0 < int(l) < n - 1)
-        if probe and self.probe is None:
-            self.probe = {"prev": torch.zeros(1, self.cfg.hidden, dtype=torch.bfloat16, device=self.device),
-                          "sims": torch.zeros(n, dtype=torch.float32, device=self.device)}
-        if not probe:
-            self.probe = None
-
-    def _probe_input(self, i: int, ws: Workspace, last: int) -> int:
-        """Called when ``ws.x`` holds the input of layer i; ``last`` = the previously executed layer (-1 for none)."""
-        pr = self.probe
-        if pr is None:
-            return i
-        H = self.cfg.hidden
-        if last >= 0:
-            nat.call("lsb_cosine_sim", pr["prev"], ws.x, 1, H, H, H, pr["sims"][last: last + 1])
-        pr["prev"].copy_(ws.x[:1])
-        return i
-
     def forward(self, ws: Workspace, R: int, nseq: int, logit_row0: int, n_logit_rows: int):
         """Run one step over the first ``R`` rows of the workspace (inputs already staged in
         ``ws``).  Writes logits for rows [logit_row0, logit_row0 + n_logit_rows)."""
@@ -1514,11 +1567,16 @@ class DeviceModel:
                     self.drift[f"layer{i:03d}.resid"] = resid[:R].float().cpu()
             if self.aux_capture is not None:
                 self._capture_aux(cfg.n_layers, ws, R)
-        xr = ws.x[logit_row0: logit_row0 + n_logit_rows]
-        self.head(ws.logits, xr, n_logit_rows)
+        if n_logit_rows:
+            self.emit_logits(ws, logit_row0, n_logit_rows)
+
+    def emit_logits(self, ws: Workspace, row0: int, n: int, rows: Optional[torch.Tensor] = None):
+        """Logits of step rows [row0, row0 + n), or of the ``n`` rows listed in ``rows`` (int32, device), after :meth:`forward`."""
+        xr = ws.x[row0: row0 + n] if rows is None else ws.x.index_select(0, rows[:n])
+        self.head(ws.logits, xr, n)
         if self.drift is not None:
             self.drift["final_norm_out"] = xr.float().cpu()
-            self.drift["logits"] = ws.logits[:n_logit_rows].float().cpu()
+            self.drift["logits"] = ws.logits[:n].float().cpu()
 
     def forward_mtp(self, ws: Workspace, R: int, k: int = 0, logit_row0: int = 0, n_logit_rows: int = 0):
         """Multi-token-prediction block ``k`` over the staged rows.  In: ``ws.resid`` rows = the stream of the previous depth at the
@@ -1551,12 +1609,6 @@ class DeviceModel:
         nat.call("lsb_add_rmsnorm", ws.x, resid, ws.sub, L["mtp_final_norm"], R, H, cfg.rms_eps, None)
         if n_logit_rows:
             self.head(ws.logits, ws.x[logit_row0: logit_row0 + n_logit_rows], n_logit_rows)
-
-    def argmax(self, ws: Workspace, n_rows: int):
-        """Greedy token per row; with a vocabulary-parallel head the per-rank winners are exchanged
-        in-kernel over NVLink (8 bytes per row per rank)."""
-        nat.call("lsb_argmax", ws.logits, self.V_local, n_rows, self.V_local, ws.amax_part, ws.out_tok, ws.out_val,
-                 self.tp_rank * self.V_local, self.comm_amax.ptr if self.comm_amax is not None else None)
 
     # ------------------------------------------------------------------ oracle support
     def effective_state_dict(self) -> Dict[str, torch.Tensor]:

@@ -28,6 +28,10 @@ from .config import ModelConfig
 
 
 def init_weights(cfg: ModelConfig, seed: int = 0, std: float = 0.02) -> Dict[str, torch.Tensor]:
+    if cfg.blocks:
+        from .block_model import RandomBlockWeights
+        rw = RandomBlockWeights(cfg, seed)
+        return {name: rw[name] for name in rw.shapes}
     g = torch.Generator().manual_seed(seed)
 
     def mat(*shape, s=std):

@@ -1,8 +1,8 @@
 """Step engine: sequences, paged-cache bookkeeping, step staging, CUDA-graph decode.
 
-One ``Engine`` drives one ``DeviceModel`` on one GPU.  A step is a batch of rows (decode: one
+One ``Engine`` drives one device model on one GPU.  A step is a batch of rows (decode: one
 row per sequence; prefill: a chunk of consecutive tokens of one sequence; verify: a few
-consecutive rows).  All per-step inputs are packed into one pinned host buffer and copied
+consecutive rows; mixed: portions of some sequences beside single tokens of others).  All per-step inputs are packed into one pinned host buffer and copied
 with a single cudaMemcpyAsync; decode steps replay a captured CUDA graph per batch size,
 so the host issues one copy + one graph launch + one 4-byte readback per generated token.
 
@@ -21,7 +21,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..models.config import ModelConfig
-from ..models.device_model import DeviceModel, Workspace
+from ..models.device_model import ModelBase, StepBuffers
 from ..ops import _native as nat
 from . import native as rt
 from .native import KvPoolExhausted  # noqa: F401  (re-exported: no free KV pages, the reference's kKvPoolExhausted)
@@ -54,6 +54,14 @@ class SequenceState:
 
 
 @dataclass
+class Portion:
+    """One sequence's part of a mixed step: its next tokens and the places among them whose next token (and logits) are asked for."""
+    sid: int
+    tokens: List[int]
+    want: List[int] = field(default_factory=list)
+
+
+@dataclass
 class SamplingParams:
     temperature: float = 0.0
     top_k: int = 0
@@ -63,7 +71,7 @@ class SamplingParams:
 
 
 class Engine:
-    def __init__(self, model: DeviceModel, max_seqs: int = 4, max_ctx: int = 4096, prefill_chunk: int = 256,
+    def __init__(self, model: ModelBase, max_seqs: int = 4, max_ctx: int = 4096, prefill_chunk: int = 256,
                  max_batch: int = 4, num_pages: Optional[int] = None, use_graph: bool = True, row_tiering: Optional[dict] = None):
         """``row_tiering``: ``{"hot_window_tokens": n, "cold_pages": m}`` keeps only the last n tokens of every sequence in HBM pages;
         older pages move to pinned host memory and single rows come back when the indexer selects them (eager steps, sparse-attention
@@ -82,11 +90,12 @@ class Engine:
         self.free_slots = list(range(max_seqs - 1, -1, -1))
         self.seqs: Dict[int, SequenceState] = {}
         self.use_graph = use_graph and self.dev.type == "cuda"
-        self.ws_decode: Dict[int, Workspace] = {}
-        self.ws_prefill: Optional[Workspace] = None
+        self.ws_decode: Dict[int, StepBuffers] = {}
+        self.ws_prefill: Optional[StepBuffers] = None
+        self.ws_mixed: Optional[StepBuffers] = None
         self.graphs: Dict[int, torch.cuda.CUDAGraph] = {}
         self.graph_launches: Dict[int, int] = {}
-        Rmax = max(prefill_chunk, max_batch)
+        Rmax = max(prefill_chunk, max_batch, 64)
         self.h_bt = torch.zeros(max_seqs, self.max_pages, dtype=torch.int32).pin_memory()
         self.h_out = torch.zeros(Rmax, dtype=torch.int32).pin_memory()
         self.stream = torch.cuda.Stream(device=self.dev)
@@ -424,12 +433,12 @@ class Engine:
             for i, t in dst.items():
                 t[s.slot].copy_(self._anchor_buf[key][i], non_blocking=True)
 
-    def _ws_rows(self, R: int) -> Workspace:
+    def _ws_rows(self, R: int) -> StepBuffers:
         """Cached workspace for verify / replay steps of R consecutive rows of one sequence (logits for every row)."""
         if not hasattr(self, "ws_verify"):
-            self.ws_verify: Dict[int, Workspace] = {}
+            self.ws_verify: Dict[int, StepBuffers] = {}
         if R not in self.ws_verify:
-            self.ws_verify[R] = Workspace(self.model, R, R, self.max_ctx)
+            self.ws_verify[R] = self.model.make_workspace(R, R, self.max_ctx)
         return self.ws_verify[R]
 
     def rewind(self, sid: int, length: int):
@@ -487,7 +496,7 @@ class Engine:
             self._sync_block_table(s)
 
     # ------------------------------------------------------------------ staging
-    def _stage(self, ws: Workspace, rows: List[tuple], seq_groups: List[tuple]):
+    def _stage(self, ws: StepBuffers, rows: List[tuple], seq_groups: List[tuple]):
         """rows: (token, slot, pos); seq_groups: (row0, nrows, slot)."""
         R = len(rows)
         P = max(self.cfg.index_kpool, 1)
@@ -513,6 +522,7 @@ class Engine:
             h[6, j] = r0; h[7, j] = n; h[8, j] = slot
         # host-side facts about the step that size kernels' grids: the largest index-entry count of a row, one sequence or several
         ws.ne_hint = max((pos + 1) // P for (_, _, pos) in rows) if rows else 0
+        ws.seq_rows = [n for (_, n, _) in seq_groups]
         ws.single_seq = len(seq_groups) == 1 and len({slot for (_, slot, _) in rows}) == 1
         ws.inp.copy_(h, non_blocking=True)
         ev = torch.cuda.Event()
@@ -520,9 +530,9 @@ class Engine:
         ws.h_ev[k] = ev
         self.h2d_bytes += 9 * ws.R * 4
 
-    def _ws_decode(self, B: int) -> Workspace:
+    def _ws_decode(self, B: int) -> StepBuffers:
         if B not in self.ws_decode:
-            self.ws_decode[B] = Workspace(self.model, B, B, self.max_ctx)
+            self.ws_decode[B] = self.model.make_workspace(B, B, self.max_ctx)
         return self.ws_decode[B]
 
     # ------------------------------------------------------------------ steps
@@ -533,7 +543,7 @@ class Engine:
         s = self.seqs[sid]
         tokens = [int(t) for t in tokens]
         if self.ws_prefill is None:
-            self.ws_prefill = Workspace(self.model, self.prefill_chunk, 1, self.max_ctx)
+            self.ws_prefill = self.model.make_workspace(self.prefill_chunk, 1, self.max_ctx)
         ws = self.ws_prefill
         nxt, logits = None, None
         if self.mtp is not None and tokens:
@@ -570,6 +580,92 @@ class Engine:
         if self.row_tier is not None:
             self.row_tier.slide_window(sid)
         return (nxt, logits) if want_logits else nxt
+
+    @property
+    def supports_mixed_steps(self) -> bool:
+        """Whether :meth:`step` serves running requests and a joining prompt's slice well in one pass (the model's recurrent layers take
+        several sequences of unequal length at full speed, and nothing rides on a single-sequence prefill)."""
+        return self.model.mixed_steps and self.mtp is None and self.row_tier is None and getattr(self.model, "dcp", None) is None
+
+    def step(self, portions: Sequence[Portion], return_logits: bool = False):
+        """One batch of unequal portions: prompt slices of some sequences beside single tokens of others, every token appended to its
+        sequence.  Returns per portion the greedy next tokens at its wanted places - with ``return_logits`` ``(tokens, logits
+        [n_wanted, vocab])``.  A step of single tokens is the captured decode step; otherwise the portions' rows run together, in passes of
+        at most ``prefill_chunk`` rows (+ one per sequence) when the step is larger than that."""
+        if not portions or len({p.sid for p in portions}) != len(portions):
+            raise ValueError("a step takes one portion per sequence, at least one")
+        if any(not p.tokens or any(not 0 <= k < len(p.tokens) for k in p.want) for p in portions):
+            raise ValueError("a portion has at least one token, and wanted places are places among its tokens")
+        if self.mtp is not None or self.row_tier is not None or getattr(self.model, "dcp", None) is not None:
+            raise NotImplementedError("mixed steps with a multi-token-prediction block, tiered rows or a sharded cache")
+        if all(len(p.tokens) == 1 for p in portions) and len(portions) <= self.max_batch:
+            out = self.decode([p.sid for p in portions], [p.tokens[0] for p in portions], return_logits=return_logits)
+            toks, lg = out if return_logits else (out, None)
+            pick = [[t] * len(p.want) for p, t in zip(portions, toks)]
+            return [(t, lg[j: j + 1].expand(len(t), -1)) for j, t in enumerate(pick)] if return_logits else pick
+        for p in portions:
+            self._require_hot(p.sid)
+        if self.ws_mixed is None:
+            self.ws_mixed = self.model.make_workspace(self.prefill_chunk + self.max_seqs, max(self.max_batch, min(64, self.prefill_chunk)), self.max_ctx)
+            self.h_want = torch.zeros(self.ws_mixed.n_logit_rows, dtype=torch.int32).pin_memory()
+            self.d_want = torch.zeros(self.ws_mixed.n_logit_rows, dtype=torch.int32, device=self.dev)
+        ws, nl = self.ws_mixed, self.ws_mixed.n_logit_rows
+        toks: List[List[int]] = [[] for _ in portions]
+        lgs: List[List[torch.Tensor]] = [[] for _ in portions]
+        at = [0] * len(portions)                                     # tokens of each portion that have run
+        with torch.cuda.stream(self.stream):
+            # all pages of the step up front: a step that runs out of pages fails before it has committed anything
+            for p in portions:
+                self._ensure_pages(self.seqs[p.sid], self.seqs[p.sid].length + len(p.tokens))
+            while True:
+                left = [(j, len(p.tokens) - at[j]) for j, p in enumerate(portions) if at[j] < len(p.tokens)]
+                if not left:
+                    break
+                # the shortest remainders first, so that single tokens never wait for a second pass; every portion gets at least one row
+                take, room = {}, ws.R - len(left)
+                for j, n in sorted(left, key=lambda x: x[1]):
+                    take[j] = 1 + min(n - 1, room)
+                    room -= take[j] - 1
+                rows, groups, wanted = [], [], []
+                for j, n in sorted(take.items()):
+                    p, s = portions[j], self.seqs[portions[j].sid]
+                    wanted += [(j, len(rows) + k - at[j]) for k in p.want if at[j] <= k < at[j] + n]
+                    groups.append((len(rows), n, s.slot))
+                    rows += [(int(t), s.slot, s.length + c) for c, t in enumerate(p.tokens[at[j]: at[j] + n])]
+                self._stage(ws, rows, groups)
+                n0 = nat.launch_count()
+                self.model.forward(ws, len(rows), len(groups), 0, 0)
+                for w0 in range(0, len(wanted), nl):
+                    part = wanted[w0: w0 + nl]
+                    n = len(part)
+                    self.h_want[:n] = torch.tensor([r for _, r in part], dtype=torch.int32)
+                    self.d_want[:n].copy_(self.h_want[:n], non_blocking=True)
+                    self.model.emit_logits(ws, 0, n, self.d_want)
+                    self.model.argmax(ws, n)
+                    self.h_out[:n].copy_(ws.out_tok[:n], non_blocking=True)
+                    self.h2d_bytes += 4 * n
+                    self.d2h_bytes += 4 * n
+                    self.stream.synchronize()
+                    lg = ws.logits[:n].float().cpu() if return_logits else None
+                    for c, (j, _) in enumerate(part):
+                        toks[j].append(int(self.h_out[c]))
+                        if return_logits:
+                            lgs[j].append(lg[c])
+                self.kernel_launches += nat.launch_count() - n0
+                for (r0, n, _), j in zip(groups, sorted(take)):
+                    s, run = self.seqs[portions[j].sid], [int(t) for t in portions[j].tokens[at[j]: at[j] + n]]
+                    if self.aux_listener is not None:
+                        self._aux_rows(s.slot, r0, n, s.length, run)
+                    s.length += n
+                    s.tokens.extend(run)
+                    at[j] += n
+            self._queue_error_readback()
+            self.stream.synchronize()
+            self._check_errors()
+        if not return_logits:
+            return toks
+        V = ws.logits.shape[1]
+        return [(t, torch.stack(l) if l else torch.zeros(0, V)) for t, l in zip(toks, lgs)]
 
     def sample_last_prefill(self, sid: int, sample) -> int:
         """Draw the first generated token of a sampled request from the logits the sequence's prefill left in the prefill
@@ -804,7 +900,7 @@ class Engine:
             return out, conf
         return out
 
-    def _capture(self, B: int, ws: Workspace, gk=None):
+    def _capture(self, B: int, ws: StepBuffers, gk=None):
         gk = B if gk is None else gk
         # warm-up run outside capture (sets function attributes, touches every buffer); the KDA
         # state it perturbs is restored by snapshotting the affected slots first.
