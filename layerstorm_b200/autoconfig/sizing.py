@@ -33,6 +33,8 @@ def _align(x: int, a: int) -> int:
 def expert_slot_bytes(mc: ModelConfig, quant: str | None = None) -> int:
     """One routed expert (gate, up, down) in its cache slot, 4096-aligned."""
     q = quant or mc.expert_quant
+    if mc.blocks:                              # bf16, width padded to the tensor-core tile
+        return _align(3 * mc.hidden * _align(mc.moe_inter, 128) * 2, 4096)
     bits = QUANT_BITS.get(q, 16.0)
     return _align(int(3 * mc.hidden * mc.moe_inter * bits / 8) + 64, 4096)
 
@@ -54,8 +56,15 @@ def indexer_row_bytes(mc: ModelConfig) -> float:
     return (mc.index_head_dim + 16) / max(1, mc.index_kpool)
 
 
+def _head_pad(d: int) -> int:
+    """Cache width of an attention head of a model described layer by layer (csrc/kernels/attn.cu)."""
+    return next((p for p in (32, 64, 128) if d <= p), _align(d, 128))
+
+
 def kv_bytes_per_token(mc: ModelConfig, backend: str = "snapmla", tp: int = 1, kv_mode: str = "sharded") -> float:
-    """All MLA layers, one token, on one GPU.  Sharded mode keeps 1/tp of the rows per rank."""
+    """All attention layers, one token, on one GPU.  Sharded mode keeps 1/tp of the rows per rank."""
+    if mc.blocks:
+        return float(sum(b.kv_heads * (_head_pad(b.dim) + _head_pad(b.vdim)) * 2 for b in mc.blocks if not b.recurrent))
     mla = mc.mla_layers()
     idx_layers = len({mc.index_source_layer(i) for i in mla}) if mc.has_indexer else 0
     per = len(mla) * kv_row_bytes(mc, backend) + idx_layers * indexer_row_bytes(mc)
@@ -64,6 +73,9 @@ def kv_bytes_per_token(mc: ModelConfig, backend: str = "snapmla", tp: int = 1, k
 
 def recurrent_state_bytes_per_seq(mc: ModelConfig, tp: int = 1) -> int:
     """KDA state (fp32 [heads, 128, 128]) and conv history per sequence on one GPU (heads split over tp)."""
+    if mc.blocks:
+        pad = lambda d: next((p for p in (32, 64, 128) if d <= p), 256)
+        return sum(b.heads * (b.vdim * pad(b.dim) + (2 * b.dim + b.vdim) * (b.conv - 1)) * 4 for b in mc.blocks if b.recurrent)
     n_kda = sum(1 for t in mc.layer_types if t == "kda")
     if not n_kda:
         return 0
@@ -93,7 +105,17 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
     H = mc.hidden
     r = ResidentBytes()
     n = mc.hc_mult
-    for i in range(mc.n_layers):
+    for b in mc.blocks:
+        if b.recurrent:
+            rank = b.dim                                                 # the low-rank width is only in the tensors; this is its usual size
+            w = (2 * b.kv_heads * b.dim + 2 * b.heads * b.vdim + b.heads + 2 * rank) * H + 3 * b.heads * (b.dim + b.vdim) * rank
+            r.attention += w * 2 + ((2 * b.kv_heads * b.dim + b.heads * b.vdim) * b.conv + b.heads * b.dim) * 4
+        else:
+            r.attention += (b.heads * (b.dim + b.vdim * (2 if b.out_gate else 1)) + b.kv_heads * (b.dim + b.vdim)) * H * 2
+        if b.experts:
+            r.router += (b.experts + b.identity) * (2 * H + 4)
+        r.norms += (4 if b.experts else 2) * H * 4
+    for i in range(0 if mc.blocks else mc.n_layers):
         if mc.is_kda_layer(i):
             C = mc.kda_heads * mc.kda_head_dim
             sharded = 3 * C * H + C * H                                  # q, k, v in; o out (dense format)

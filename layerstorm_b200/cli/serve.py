@@ -167,7 +167,7 @@ def build_engine(cfg: dict, shape: ModelConfig, ckpt: Optional[str], args: argpa
         return NullEngine(vocab=max(512, min(shape.vocab, 65536)), max_seqs=sv["max_concurrent_requests"] + 4,
                           max_ctx=sv["max_sequence_length"], page=page)
     import torch
-    from ..models.device_model import DeviceModel
+    from ..models.block_model import model_class
     from ..runtime.engine import Engine
     if not torch.cuda.is_available():
         raise RuntimeError("no CUDA device is visible; use --test-engine to serve from the null engine")
@@ -186,7 +186,9 @@ def build_engine(cfg: dict, shape: ModelConfig, ckpt: Optional[str], args: argpa
     streamer = None
     ratio = float((cfg.get("autoconfig") or {}).get("vram_expert_ratio") or 1.0)
     if ratio < 1.0 and shape.n_routed > 0:
-        if world > 1:
+        if shape.blocks:
+            log.warning("expert streaming is built for the MLA family; autoconfig.vram_expert_ratio = %.2f ignored", ratio)
+        elif world > 1:
             log.warning("expert streaming is wired for one GPU per model; autoconfig.vram_expert_ratio = %.2f ignored with %d ranks", ratio, world)
         else:
             from ..runtime.streaming import ExpertStreamer
@@ -208,11 +210,11 @@ def build_engine(cfg: dict, shape: ModelConfig, ckpt: Optional[str], args: argpa
     if ckpt and not args.random_weights:
         from ..models.checkpoint import open_checkpoint
         _, w = open_checkpoint(ckpt, shape)
-        model = DeviceModel.from_state_dict(shape, w, dev, kv_fmt, page, tp_rank=rank, tp_size=world, with_mtp=want_mtp, layer_hook=hook,
+        model = model_class(shape).from_state_dict(shape, w, dev, kv_fmt, page, tp_rank=rank, tp_size=world, with_mtp=want_mtp, layer_hook=hook,
                                             skip_experts=streamer.covers if (streamer is not None and streamer.live_source is not None) else None)
     else:
         log.warning("serving RANDOM weights of shape %s", shape.name)
-        model = DeviceModel.random_init(shape, dev, kv_fmt, page, expert_slots="auto", embed_on_host=shape.vocab * shape.hidden > (1 << 28),
+        model = model_class(shape).random_init(shape, dev, kv_fmt, page, expert_slots="auto", embed_on_host=shape.vocab * shape.hidden > (1 << 28),
                                         tp_rank=rank, tp_size=world, with_mtp=want_mtp, layer_hook=hook)
     if streamer is not None:
         streamer.attach(model)

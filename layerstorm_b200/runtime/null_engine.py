@@ -45,6 +45,7 @@ class NullEngine:
         self.kernel_launches = 0
         self.steps = 0
         self.prefill_tokens = 0
+        self.supports_mixed_steps = False      # tests set it to serve joining slices beside running requests (``step``)
 
     # ---- model ----
     def _next(self, toks: Sequence[int]) -> int:
@@ -130,6 +131,23 @@ class NullEngine:
             lgs.append(lg)
         self.steps += 1
         return (outs, torch.stack(lgs)) if return_logits else outs
+
+    def step(self, portions, return_logits: bool = False):
+        """One batch of unequal portions (``runtime.engine.Portion``): greedy next tokens (and logits) at each portion's wanted places."""
+        for p in portions:
+            self._grow(p.sid, len(p.tokens))
+        out = []
+        for p in portions:
+            s = self.seqs[p.sid]
+            lgs = []
+            for k, t in enumerate(p.tokens):
+                s.tokens.append(int(t))
+                if k in p.want:
+                    lgs.append(self._logits(s.tokens))
+            toks = [int(lg.argmax()) for lg in lgs]
+            out.append((toks, torch.stack(lgs) if lgs else torch.zeros(0, self.vocab)) if return_logits else toks)
+        self.steps += 1
+        return out
 
     def forward_rows(self, sid: int, tokens: Sequence[int], commit: bool = True) -> torch.Tensor:
         """Logits for every row of a run of consecutive tokens (speculative verify shape)."""

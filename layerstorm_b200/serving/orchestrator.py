@@ -162,6 +162,10 @@ class _DegradedRetry(Exception):
     step without it): the attempt is abandoned before a single token is emitted, so even a streaming request can be run again."""
 
 
+class _MixedStepFailed(RuntimeError):
+    """A step that carried a joining slice beside the running requests failed: none of them can go on."""
+
+
 class Orchestrator:
     """Serves InferenceRequests on one engine.  ``draft`` is an optional proposer with
     ``propose(context_ids, gamma) -> List[int]`` (speculative decoding)."""
@@ -193,7 +197,7 @@ class Orchestrator:
         self.admission_waits = 0
         self.preemptions = 0
         self.joining: Optional[list] = None       # [request, sequence id, prompt, tokens already in the sequence, degraded steps before]
-        self.prefill_slices = 0
+        self.prefill_slices = self.mixed_steps = 0
         self.eos = set(int(t) for t in eos_token_ids)
         self.prefix = PrefixCache(engine, prefix_cache or PrefixCacheConfig())
         self.draft, self.gamma = draft, speculation_depth if draft is not None else 0
@@ -386,11 +390,15 @@ class Orchestrator:
                             self._wait_for_capacity(head)
                         else:
                             self._fail(head, exc)
+        mixed: Optional[List[int]] = None                  # next tokens of the running requests when the joining slice ran in their step
         if self.joining is not None:
             did = True
             req, sid, prompt, _, d0 = self.joining
             try:
-                done_prefill, tok = self._prefill_slice(self.joining)
+                if self.running and getattr(eng, "supports_mixed_steps", False):
+                    done_prefill, tok, mixed = self._mixed_step(self.joining)
+                else:
+                    done_prefill, tok = self._prefill_slice(self.joining)
                 if req.cancelled.is_set():
                     eng.free_sequence(sid)
                     self._finish(req, "cancelled")
@@ -420,13 +428,20 @@ class Orchestrator:
                 if self.running and self._is_capacity_error(exc):
                     self._wait_for_capacity(req)          # nothing was emitted during the join: the prompt is simply fed again later
                 else:
-                    self._fail(req, exc)
+                    cause = exc.__cause__ if isinstance(exc, _MixedStepFailed) and exc.__cause__ is not None else exc
+                    self._fail(req, cause)
+                    if isinstance(exc, _MixedStepFailed):  # the running requests were part of the step: their tokens may be in the cache
+                        for r, s_, _ in self.running:
+                            eng.free_sequence(s_)
+                            self._fail(r, cause)
+                        self.running = []
         # 2. one token for every running request
         if self.running:
             did = True
-            sids, toks = [r[1] for r in self.running], [r[2] for r in self.running]
+            batch = self.running[: len(mixed)] if mixed is not None else list(self.running)      # a request that joined in this very step waits for the next
+            sids, toks = [r[1] for r in batch], [r[2] for r in batch]
             try:
-                outs = self._with_pool_evict_retry(self.running[0][0], lambda: eng.decode(sids, toks))
+                outs = mixed if mixed is not None else self._with_pool_evict_retry(batch[0][0], lambda: eng.decode(sids, toks))
             except Exception as exc:  # noqa: BLE001 - the step failed for the whole batch
                 if len(self.running) > 1 and self._is_capacity_error(exc):
                     # out of KV pages in mid-decode: the youngest request gives its pages back and joins again later, its prompt
@@ -445,7 +460,7 @@ class Orchestrator:
                 return True
             self.batched_steps += 1
             keep = []
-            for entry, tok in zip(self.running, outs):
+            for entry, tok in zip(batch, outs):
                 req, sid, _ = entry
                 if self._emit(req, int(tok), None):
                     eng.free_sequence(sid)
@@ -454,7 +469,7 @@ class Orchestrator:
                 else:
                     entry[2] = int(tok)
                     keep.append(entry)
-            self.running = keep
+            self.running = keep + self.running[len(batch):]
         return did
 
     @staticmethod
@@ -490,6 +505,27 @@ class Orchestrator:
         joining[3] = fed + n
         self.prefill_slices += 1
         return joining[3] >= len(prompt), tok
+
+    def _mixed_step(self, joining: list):
+        """One engine step of the joining request's next slice beside one token of every running request: (prompt complete, the engine's
+        next token after the slice, the running requests' next tokens).  Without the pages for all of it the slice runs on its own
+        (third item None), where the capacity rules for joining and for running requests apply one by one."""
+        from ..runtime.engine import Portion
+        req, sid, prompt, fed = joining[:4]
+        n = min(self.prefill_slice, getattr(self.engine, "prefill_chunk", self.prefill_slice), len(prompt) - fed)
+        last = fed + n >= len(prompt)
+        portions = [Portion(sid, prompt[fed: fed + n], [n - 1] if last else [])] + [Portion(s, [t], [0]) for _, s, t in self.running]
+        try:
+            res = self._with_pool_evict_retry(req, lambda: self.engine.step(portions))
+        except KvPoolExhausted:
+            done, tok = self._prefill_slice(joining)
+            return done, tok, None
+        except Exception as exc:  # noqa: BLE001
+            raise _MixedStepFailed(str(exc)) from exc
+        joining[3] = fed + n
+        self.prefill_slices += 1
+        self.mixed_steps += 1
+        return last, (res[0][0] if last else None), [r[0] for r in res[1:]]
 
     def _finish(self, req: InferenceRequest, reason: str):
         req.finish_reason = req.finish_reason or reason

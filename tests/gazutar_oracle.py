@@ -174,3 +174,80 @@ def save_model(path, cfg, w):
     hj = json.dumps(head).encode()
     (path / "model.safetensors").write_bytes(struct.pack("<Q", len(hj)) + hj + b"".join(blobs))
     return held
+
+
+# ------------------------------------------------------------------------------------------------ random models
+def random_model(cfg, seed=0, rank=20, sharp=1.0):
+    """Tensors for a configuration, spread so that every mechanism matters.  ``sharp`` scales the query norms: large values make single
+    keys stand out of the softmax."""
+    g = torch.Generator().manual_seed(seed)
+    n = lambda *s: torch.randn(*s, generator=g)
+    u = lambda lo, hi, *s: lo + (hi - lo) * torch.rand(s, generator=g)
+    H, V, w = cfg["width"], cfg["vocab"], {}
+    lin = lambda o, i: n(o, i) / i ** 0.5
+
+    def ln(p):
+        w[p], w[p + ".b"] = 1.0 + 0.2 * n(H), 0.2 * n(H)
+
+    w["embed"], w["head"] = n(V, H), lin(V, H)
+    ln("final.norm")
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        x = p + "mix."
+        ln(p + "norm1")
+        h, k, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        if L["type"] == "attention":
+            w[x + "q"], w[x + "k"], w[x + "v"], w[x + "g"], w[x + "o"] = lin(h * d, H), lin(k * d, H), lin(k * e, H), lin(h * e, H), lin(H, h * e)
+            w[x + "q.norm"], w[x + "k.norm"] = sharp * (1.0 + 0.2 * n(h * d)), 1.0 + 0.2 * n(k * d)
+            if m.get("v_mix"):
+                w[x + "vmix"] = u(0.3, 0.7)
+        else:
+            w[x + "q"], w[x + "k"], w[x + "v"], w[x + "b"], w[x + "o"] = lin(k * d, H), lin(k * d, H), lin(h * e, H), lin(h, H), lin(H, h * e)
+            for t, c in (("q", k * d), ("k", k * d), ("v", h * e)):
+                w[x + t + ".conv"] = u(-1.0, 1.0, c, m["conv"])
+            w[x + "A_log"], w[x + "dt_bias"], w[x + "norm"] = u(-3.0, 0.5, h), u(-3.0, 0.0, h * d), 1.0 + 0.2 * n(e)
+            w[x + "a1"], w[x + "a2"], w[x + "g1"], w[x + "g2"] = lin(rank, H), lin(h * d, rank), lin(rank + 3, H), lin(h * e, rank + 3)
+        if L.get("mlp"):
+            ln(p + "norm2")
+            r, f = L["mlp"]["router"], L["mlp"]["expert"]["ff"]
+            z = p + "mlp."
+            tot = r["experts"] + (r.get("identity") or 0)
+            w[z + "router"], w[z + "correction"] = 1.5 * lin(tot, H), -1.5 + 0.3 * n(tot)
+            for j in range(r["experts"]):
+                w[z + f"e{j}.gate"], w[z + f"e{j}.up"], w[z + f"e{j}.down"] = lin(f, H), lin(f, H), lin(H, f)
+    return w
+
+
+def att(heads, kv_heads, dim, vdim, window=0, v_mix=False, scale=None, mlp=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or round(1.7 / dim ** 0.5, 4), "v_mix": v_mix}
+    if window:
+        m["mask"] = {"size": window}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def delta(heads, kv_heads, dim, vdim, conv, mlp=None):
+    return {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": mlp}
+
+
+def moe_spec(experts, identity, top, count=1, keep=1, ff=40):
+    r = {"experts": experts, "top": top, "groups": {"count": count, "keep": keep}}
+    if identity:
+        r["identity"] = identity
+    return {"kind": "moe", "expert": {"ff": ff}, "router": r}
+
+
+def model_cfg(width, vocab, layers, eps=1e-5, logit_scale=0.5):
+    return {"architecture": "Gazutar", "layers": layers, "logit_scale": logit_scale, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+# several geometries: unequal layers, layers without a feed-forward, groups of one head, sizes off the kernels' tiles and on them
+MODELS = {
+    "odd": lambda: model_cfg(136, 301, [delta(6, 2, 24, 40, 3, moe_spec(5, 1, 2, 3, 2, 40)), att(6, 2, 24, 40, 21, True, mlp=moe_spec(7, 0, 3, 1, 1, 24)),
+                                        delta(2, 1, 40, 20, 5), att(4, 4, 36, 40, 9, False), att(4, 2, 20, 40, 33, True, mlp=moe_spec(4, 4, 4, 2, 1, 56))], 3e-4, 0.3),
+    "attention first": lambda: model_cfg(96, 128, [att(3, 1, 32, 32, 50, True, mlp=moe_spec(6, 2, 1, 4, 2, 48)), delta(1, 1, 16, 16, 1, moe_spec(6, 2, 2, 2, 1, 48)),
+                                                   att(3, 1, 16, 32, 0, True), delta(5, 5, 64, 48, 2)], 1e-6, 1.0),
+    "tiles": lambda: model_cfg(384, 520, [delta(3, 3, 128, 128, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(16, 1, 128, 64, 130, True, mlp=moe_spec(12, 4, 4, 4, 2, 128)),
+                                          delta(4, 2, 64, 96, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(8, 4, 64, 64, 70, True)], 1e-5, 0.25),
+    "wide": lambda: model_cfg(256, 200, [delta(2, 1, 160, 160, 4), att(20, 1, 192, 256, 65, True, mlp=moe_spec(3, 3, 2, 1, 1, 64)), delta(2, 2, 48, 200, 4),
+                                         att(2, 2, 260, 24, 40, False)], 1e-5, 2.0),
+}
