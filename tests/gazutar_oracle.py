@@ -177,9 +177,9 @@ def save_model(path, cfg, w):
 
 
 # ------------------------------------------------------------------------------------------------ random models
-def random_model(cfg, seed=0, rank=20, sharp=1.0):
+def random_model(cfg, seed=0, rank=20, sharp=1.0, close_calls=True):
     """Tensors for a configuration, spread so that every mechanism matters.  ``sharp`` scales the query norms: large values make single
-    keys stand out of the softmax."""
+    keys stand out of the softmax.  Without ``close_calls`` the router's correction decides the choice alone (rounding cannot turn it)."""
     g = torch.Generator().manual_seed(seed)
     n = lambda *s: torch.randn(*s, generator=g)
     u = lambda lo, hi, *s: lo + (hi - lo) * torch.rand(s, generator=g)
@@ -213,6 +213,8 @@ def random_model(cfg, seed=0, rank=20, sharp=1.0):
             z = p + "mlp."
             tot = r["experts"] + (r.get("identity") or 0)
             w[z + "router"], w[z + "correction"] = 1.5 * lin(tot, H), -1.5 + 0.3 * n(tot)
+            if not close_calls:
+                w[z + "correction"] = 2.0 * torch.randperm(tot, generator=g).float() - tot
             for j in range(r["experts"]):
                 w[z + f"e{j}.gate"], w[z + f"e{j}.up"], w[z + f"e{j}.down"] = lin(f, H), lin(f, H), lin(H, f)
     return w
@@ -247,7 +249,7 @@ MODELS = {
     "attention first": lambda: model_cfg(96, 128, [att(3, 1, 32, 32, 50, True, mlp=moe_spec(6, 2, 1, 4, 2, 48)), delta(1, 1, 16, 16, 1, moe_spec(6, 2, 2, 2, 1, 48)),
                                                    att(3, 1, 16, 32, 0, True), delta(5, 5, 64, 48, 2)], 1e-6, 1.0),
     "tiles": lambda: model_cfg(384, 520, [delta(3, 3, 128, 128, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(16, 1, 128, 64, 130, True, mlp=moe_spec(12, 4, 4, 4, 2, 128)),
-                                          delta(4, 2, 64, 96, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(8, 4, 64, 64, 70, True)], 1e-5, 0.25),
+                                          delta(4, 2, 64, 96, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(8, 2, 64, 32, 70, True)], 1e-5, 0.25),
     "wide": lambda: model_cfg(256, 200, [delta(2, 1, 160, 160, 4), att(20, 1, 192, 256, 65, True, mlp=moe_spec(3, 3, 2, 1, 1, 64)), delta(2, 2, 48, 200, 4),
                                          att(2, 2, 260, 24, 40, False)], 1e-5, 2.0),
 }

@@ -60,7 +60,7 @@ def test_server_resolves_a_native_checkpoint_directory(tmp_path):
     assert shape.blocks and ckpt == str(tmp_path) and cfg["model"]["architecture"] == "gazutar" and cfg["model"]["vocab_size"] == 520
     from layerstorm_b200.config import model_config_from
     assert model_config_from(cfg).blocks == shape.blocks
-    assert sizing.kv_bytes_per_token(shape) == 2 * (128 + 64) + 2 * 4 * (64 + 64)
+    assert sizing.kv_bytes_per_token(shape) == 2 * (128 + 64) + 2 * 2 * (64 + 32)
     assert sizing.recurrent_state_bytes_per_seq(shape) == 4 * (3 * (128 * 128 + 384 * 3) + 4 * (96 * 64 + 224 * 3))
 
 
