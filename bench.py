@@ -134,9 +134,16 @@ def main():
     ap.add_argument("--dcp-chunk", type=int, default=0,
                     help="N > 1 GPUs: shard the latent KV cache over the ranks in chunks of this many tokens (context parallel); 0 = replicated")
     ap.add_argument("--layers", type=int, default=0, help="smoke runs only: keep the first N layers (the JSON line is then marked invalid)")
+    ap.add_argument("--design", default="", choices=["", "gazutar"],
+                    help="instead of the headline workload: prefill and decode of this design at a few layer sizes beside the closest other design")
+    ap.add_argument("--design-sizes", default="2048,4096", help="hidden sizes of --design")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.design:
+        from layerstorm_b200.utils import design_bench
+        print(json.dumps(design_bench.run(args.design, [int(x) for x in args.design_sizes.split(",")], sampler=ClockSampler(int(os.environ.get("LOCAL_RANK", 0))))))
+        return 0
     if args.moe_block_scaled:
         os.environ["LSB_MOE_BLOCK_SCALED"] = "1"
     if args.warmup < 3:

@@ -1,0 +1,198 @@
+"""Prefill and decode throughput of a model design at layer sizes of a real model (random weights), beside the framework's closest other
+design at equal size, with the device time of every kernel launcher.
+
+    python bench.py --design gazutar [--design-sizes 2048,4096]
+
+Gazutar's neighbour is a KDA + MLA model of the same width, heads, experts and layer pattern (plain residual stream, dense latent attention).
+Per launcher: all its calls of one step, recorded from an eager pass and replayed back to back in a CUDA graph (other layers' operands in
+between, so that a layer's weights are not left over in L2), divided by the number of calls.  Fractions are of the measured peaks
+(MEASURED_PEAKS.json): bytes or FLOPs that the operation has to move or do, over the launcher's time.
+"""
+from __future__ import annotations
+
+import json
+import os
+import statistics
+
+import torch
+
+from ..models.block_model import model_class
+from ..models.config import ModelConfig, gazutar_config
+from ..ops import _native as nat
+from ..runtime.engine import Engine
+
+N_LAYERS, EVERY, TOP = 8, 4, 8
+
+
+def design_pair(hidden: int, window: int):
+    """(Gazutar, neighbour) of one size: 128-wide heads, experts of half the width, every fourth layer attention."""
+    heads, att_heads, kv, experts, ff, vocab = hidden // 64, hidden // 128, max(1, hidden // 512), hidden // 64, hidden // 2, 65536
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": 8, "top": TOP, "groups": {"count": 8, "keep": 4}}}
+    att = {"heads": att_heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window}, "v_mix": True}
+    dlt = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}
+    g = gazutar_config({"name": f"gazutar-{hidden}", "vocab": vocab, "width": hidden, "norm": {"eps": 1e-5}, "logit_scale": 0.5, "layers": [
+        {"type": "attention", "mixer": att, "mlp": mlp} if i % EVERY == EVERY - 1 else {"type": "channel_delta", "mixer": dlt, "mlp": mlp} for i in range(N_LAYERS)]})
+    k = ModelConfig(name=f"kda-mla-{hidden}", architecture="glm5_next", hidden=hidden, n_layers=N_LAYERS, vocab=vocab, rms_eps=1e-5, n_heads=att_heads,
+                    q_lora=hidden * 3 // 8, kv_lora=512, qk_nope=128, qk_rope=0, v_head=128, dense_inter=1024, first_k_dense=0, n_routed=experts, top_k=TOP,
+                    n_shared=0, moe_inter=ff, scoring="softmax", n_group=8, topk_group=4, norm_topk_prob=False, router_bias=True,
+                    layer_types=["mla" if i % EVERY == EVERY - 1 else "kda" for i in range(N_LAYERS)], kda_heads=heads, kda_head_dim=128, kda_rank=128)
+    return g, k
+
+
+def _peaks():
+    p = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    if os.path.exists(p):
+        d = json.load(open(p))
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12
+    return 6.65e12, 1.59e15
+
+
+def _events(fn, stream, reps):
+    out = []
+    with torch.cuda.stream(stream):
+        for _ in range(3):
+            fn()
+        for _ in range(reps):
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(stream)
+            fn()
+            b.record(stream)
+            stream.synchronize()
+            out.append(a.elapsed_time(b))
+    return statistics.median(out)
+
+
+def launcher_times(eng, run, reps=5) -> dict:
+    """{launcher: (calls per step, microseconds per call)} of the step that ``run`` launches eagerly."""
+    calls, orig = [], nat.call
+
+    def rec(name, *a, **k):
+        if nat.SIGS[name][1]:
+            calls.append((name, a))
+        return orig(name, *a, **k)
+
+    with torch.cuda.stream(eng.stream):
+        run()
+        nat.call = rec
+        try:
+            run()
+        finally:
+            nat.call = orig
+        eng.stream.synchronize()
+        out = {}
+        for name in dict.fromkeys(n for n, _ in calls):
+            mine = [a for n, a in calls if n == name]
+            g = torch.cuda.CUDAGraph()
+            loops = 1 if len(mine) > 4 else 4
+            with torch.cuda.graph(g, stream=eng.stream):
+                for _ in range(loops):
+                    for a in mine:
+                        orig(name, *a)
+            out[name] = (len(mine), round(_events(g.replay, eng.stream, reps) * 1e3 / (len(mine) * loops), 2))
+            del g
+    return out
+
+
+def work(cfg, rows: int, ctx: int, batch: int) -> dict:
+    """{launcher: ("bytes" | "flops", amount per call)} of the operations that have a clear floor."""
+    H = cfg.hidden
+    heads = cfg.kda_heads
+    out = {}
+    state = 2 * batch * heads * 128 * 128 * 4                       # read and write the recurrent state once
+    gates = 2 * heads * 128 * 128 * 2
+    per_tok = heads * (4 * 128 * 128 + 6 * 64 * 128) * 2            # chunk form: state products, pair products
+    rec = ("bytes", state + gates + rows * heads * 128 * 18) if rows == batch else ("flops", rows * per_tok)
+    if cfg.blocks:
+        b = next(x for x in cfg.blocks if not x.recurrent)
+        seen = min(ctx, b.window)
+        out["lsb_delta_forward"] = rec
+        kv = b.kv_heads * (b.dim + b.vdim) * 2
+        out["lsb_attn"] = ("bytes", batch * seen * kv + rows * b.heads * b.vdim * 6) if rows == batch else ("flops", 2 * rows * seen * b.heads * (b.dim + b.vdim))
+        out["lsb_attn_prep"] = ("bytes", rows * ((b.heads + b.kv_heads) * b.dim + b.kv_heads * b.vdim) * 6)
+        out["lsb_post_norm"] = ("bytes", rows * H * (14 + TOP * 4) // 2 + rows * H * 7)
+    else:
+        out["lsb_kda_forward"] = out["lsb_kda_forward_chunked"] = rec
+        lat = cfg.kv_lora
+        out["lsb_mla_decode"] = ("bytes", batch * ctx * lat * 2 + rows * cfg.n_heads * lat * 4) if rows == batch else ("flops", 4 * rows * ctx * cfg.n_heads * lat)
+        out["lsb_add_rmsnorm"] = ("bytes", rows * H * 14)
+        out["lsb_moe_combine"] = ("bytes", rows * H * (TOP + 1) * 4)
+        out["lsb_mla_prep"] = ("bytes", rows * (cfg.q_lora + lat) * 6)
+    if rows == 1:                          # (how many experts a batch touches is the router's affair)
+        by = TOP * 3 * H * cfg.moe_inter * 2
+        out["lsb_moe_gateup"], out["lsb_moe_down"] = ("bytes", by * 2 / 3), ("bytes", by / 3)
+    elif rows > 1024:
+        out["lsb_moe_tc_ffn"] = ("flops", 3 * rows * TOP * H * cfg.moe_inter)
+    return out
+
+
+def measure(cfg, ctx: int, chunk: int, batches, clocks=None) -> dict:
+    hbm, tf = _peaks()
+    dev = torch.device("cuda", torch.cuda.current_device())
+    m = model_class(cfg).random_init(cfg, dev, "bf16", 64, seed=5)
+    bmax = max(batches)
+    eng = Engine(m, max_seqs=bmax, max_ctx=ctx + chunk + 256, prefill_chunk=chunk, max_batch=bmax)
+    g = torch.Generator().manual_seed(1)
+    tok = lambda n: torch.randint(0, cfg.vocab, (n,), generator=g).tolist()
+    res: dict = {"model": cfg.name, "weight_gib": round(m.weight_bytes() / 2 ** 30, 2)}
+
+    def table(times, rows, batch):
+        w = work(cfg, rows, ctx, batch)
+        t = {}
+        for k, (n, us) in sorted(times.items(), key=lambda x: -x[1][0] * x[1][1]):
+            e = {"calls": n, "us": us}
+            if k in w:
+                kind, amount = w[k]
+                e["of_measured_" + ("hbm" if kind == "bytes" else "bf16")] = round(amount / (us * 1e-6) / (hbm if kind == "bytes" else tf), 4)
+            t[k] = e
+        return t
+
+    warm = eng.create_sequence()
+    eng.prefill(warm, tok(chunk))
+    eng.free_sequence(warm)
+    s0 = eng.create_sequence()
+    eng.prefill(s0, tok(ctx - chunk))
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record(eng.stream)
+    nxt = eng.prefill(s0, tok(chunk))
+    e1.record(eng.stream)
+    torch.cuda.synchronize()
+    ms = e0.elapsed_time(e1)
+    res["prefill"] = {"chunk": chunk, "context": ctx, "ms": round(ms, 3), "tok_s": round(chunk / ms * 1e3, 1)}
+    ws = eng.ws_prefill                       # still staged with the last chunk
+    res["prefill"]["launchers"] = table(launcher_times(eng, lambda: m.forward(ws, chunk, 1, chunk - 1, 1)), chunk, 1)
+    sids, toks = [s0], [nxt]
+    res["decode"] = {}
+    for B in batches:
+        while len(sids) < B:
+            sids.append(eng.create_sequence())
+            toks.append(eng.prefill(sids[-1], tok(ctx)))
+        for _ in range(4):
+            toks = eng.decode(sids, toks)
+        n = 32
+        e0.record(eng.stream)
+        for _ in range(n):
+            toks = eng.decode(sids, toks)
+        e1.record(eng.stream)
+        torch.cuda.synchronize()
+        e2e = e0.elapsed_time(e1) / n
+        wd = eng.ws_decode[B]
+        dev_ms = _events(eng.graphs[B].replay, eng.stream, 20)
+        res["decode"][str(B)] = {"ms_per_step": round(dev_ms, 4), "tok_s": round(B / dev_ms * 1e3, 1), "e2e_tok_s": round(B / e2e * 1e3, 1),
+                                 "launchers": table(launcher_times(eng, lambda: m.forward(wd, B, B, 0, B)), B, B)}
+    del eng, m
+    torch.cuda.empty_cache()
+    return res
+
+
+def run(design: str, sizes, ctx: int = 8192, chunk: int = 2048, batches=(1, 32), sampler=None) -> dict:
+    if design != "gazutar":
+        raise ValueError(f"no comparison for design {design!r}")
+    out = {"metric": "prefill and decode throughput beside the closest design", "design": design, "data": "random weights, synthetic token ids", "dtype": "bf16",
+           "context": ctx, "window": 4096, "l2": "decode and prefill steps stream more weights than L2 holds", "sizes": {}}
+    if sampler is not None:
+        sampler.start()
+    for h in sizes:
+        out["sizes"][str(h)] = [measure(c, ctx, chunk, list(batches)) for c in design_pair(h, 4096)]
+    if sampler is not None:
+        out["clocks"] = sampler.stop()
+    return out

@@ -250,6 +250,8 @@ MODELS = {
                                                    att(3, 1, 16, 32, 0, True), delta(5, 5, 64, 48, 2)], 1e-6, 1.0),
     "tiles": lambda: model_cfg(384, 520, [delta(3, 3, 128, 128, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(16, 1, 128, 64, 130, True, mlp=moe_spec(12, 4, 4, 4, 2, 128)),
                                           delta(4, 2, 64, 96, 4, moe_spec(12, 4, 4, 4, 2, 128)), att(8, 2, 64, 32, 70, True)], 1e-5, 0.25),
+    "narrow": lambda: model_cfg(100, 67, [att(5, 5, 8, 8, 3, True, mlp=moe_spec(3, 2, 5, 5, 5, 12)), delta(5, 5, 8, 12, 7, moe_spec(3, 2, 2, 5, 4, 12)),
+                                          att(10, 5, 16, 8, 1, True), delta(4, 1, 20, 8, 4)], 1e-4, 0.7),
     "wide": lambda: model_cfg(256, 200, [delta(2, 1, 160, 160, 4), att(20, 1, 192, 256, 65, True, mlp=moe_spec(3, 3, 2, 1, 1, 64)), delta(2, 2, 48, 200, 4),
                                          att(2, 2, 260, 24, 40, False)], 1e-5, 2.0),
 }
