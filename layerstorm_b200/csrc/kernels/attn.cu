@@ -37,39 +37,46 @@ __device__ __forceinline__ float act_f(float v) { return v; }
 __device__ __forceinline__ float gate_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
 // ------------------------------------------------------------------------------------------------ projection -> q, cache row
-template <typename T>
-__global__ void __launch_bounds__(256) attn_prep_kernel(const float* __restrict__ proj, int ldp, int off_q, int off_k, int off_v, const float* __restrict__ wq,
+template <typename T, int NT>
+__global__ void __launch_bounds__(NT) attn_prep_kernel(const float* __restrict__ proj, int ldp, int off_q, int off_k, int off_v, const float* __restrict__ wq,
                                                         const float* __restrict__ wk, float eps, float* __restrict__ vfirst, int mix,
                                                         const float* __restrict__ lambda, T* __restrict__ q_out, T* __restrict__ cache,
                                                         const int* __restrict__ block_table, int max_pages, const int* __restrict__ row_seq,
                                                         const int* __restrict__ row_pos, int H, int G, int dk, int dv, int dkp, int dvp, int page) {
-    __shared__ float red[33];
+    __shared__ float red[2][32];
+    constexpr int nt = NT;
     const int r = blockIdx.x, t = threadIdx.x;
     pdl_wait();
     pdl_launch_dependents();
     const int seq = row_seq[r], pos = row_pos[r];
     if (seq < 0) return;
     const float* pr = proj + (size_t)r * ldp;
+    T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * (dkp + dvp));
     float qr = 1.f, kr = 1.f;
     if (wq) {
-        float s = 0.f;
-        for (int i = t; i < H * dk; i += 256) { const float x = pr[off_q + i]; s = fmaf(x, x, s); }
-        qr = 1.f / sqrtf(block_sum(s, red) / (float)(H * dk) + eps);
-        s = 0.f;
-        for (int i = t; i < G * dk; i += 256) { const float x = pr[off_k + i]; s = fmaf(x, x, s); }
-        kr = 1.f / sqrtf(block_sum(s, red) / (float)(G * dk) + eps);
+        float a = 0.f, b = 0.f;
+#pragma unroll 4
+        for (int i = t; i < H * dk; i += nt) { const float x = pr[off_q + i]; a = fmaf(x, x, a); }
+#pragma unroll 4
+        for (int i = t; i < G * dk; i += nt) { const float x = pr[off_k + i]; b = fmaf(x, x, b); }
+        a = warp_sum(a); b = warp_sum(b);
+        if ((t & 31) == 0) { red[0][t >> 5] = a; red[1][t >> 5] = b; }
+        __syncthreads();
+        a = (t & 31) < NT / 32 ? red[0][t & 31] : 0.f;            // every warp adds the warps' partials on its own
+        b = (t & 31) < NT / 32 ? red[1][t & 31] : 0.f;
+        qr = 1.f / sqrtf(warp_sum(a) / (float)(H * dk) + eps);
+        kr = 1.f / sqrtf(warp_sum(b) / (float)(G * dk) + eps);
     }
-    for (int i = t; i < H * dkp; i += 256) {
+    for (int i = t; i < H * dkp; i += nt) {
         const int h = i / dkp, c = i - h * dkp, s = h * dk + c;
         q_out[(size_t)r * H * dkp + i] = to_act<T>(c < dk ? pr[off_q + s] * qr * (wq ? wq[s] : 1.f) : 0.f);
     }
-    T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * (dkp + dvp));
-    for (int i = t; i < G * dkp; i += 256) {
+    for (int i = t; i < G * dkp; i += nt) {
         const int g = i / dkp, c = i - g * dkp, s = g * dk + c;
         row[i] = to_act<T>(c < dk ? pr[off_k + s] * kr * (wk ? wk[s] : 1.f) : 0.f);
     }
     const float lam = mix == 2 ? *lambda : 0.f;
-    for (int i = t; i < G * dvp; i += 256) {
+    for (int i = t; i < G * dvp; i += nt) {
         const int g = i / dvp, c = i - g * dvp, s = g * dv + c;
         float v = 0.f;
         if (c < dv) {
@@ -501,10 +508,11 @@ LSB_API int lsb_attn_prep(const void* proj, int ldp, int off_q, int off_k, int o
                           int rows, int H, int G, int dk, int dv, int dkp, int dvp, int page, int f32, void* stream) {
     if (H % G || dkp < dk || dvp < dv || dkp % 16 || dvp % 16 || (mix && !vfirst) || (mix == 2 && !lambda)) return -1;
     cudaStream_t st = (cudaStream_t)stream;
-#define LSB_PREP(T) launch_pdl((attn_prep_kernel<T>), rows, 256, 0, st, (const float*)proj, ldp, off_q, off_k, off_v, (const float*)wq, (const float*)wk, eps, \
+    const bool wide = rows <= 64 && (H + 2 * G) * dk >= 2048;                   // few rows: a row's latency counts, not the blocks per SM
+#define LSB_PREP(T, N) launch_pdl((attn_prep_kernel<T, N>), rows, N, 0, st, (const float*)proj, ldp, off_q, off_k, off_v, (const float*)wq, (const float*)wk, eps, \
                                (float*)vfirst, mix, (const float*)lambda, (T*)q_out, (T*)cache, (const int*)block_table, max_pages, (const int*)row_seq, \
                                (const int*)row_pos, H, G, dk, dv, dkp, dvp, page)
-    if (f32) LSB_PREP(float); else LSB_PREP(bf16);
+    if (f32) LSB_PREP(float, 256); else if (wide) LSB_PREP(bf16, 1024); else LSB_PREP(bf16, 256);
 #undef LSB_PREP
     LSB_CHECK_LAUNCH();
 }

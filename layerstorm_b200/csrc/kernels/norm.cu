@@ -748,7 +748,7 @@ struct MoeSum { const float* y; const float* wts; const int* ids; const int* slo
 
 // resid[r] += norm(sub[r]) (or norm of the MoE sum), x[r] = the new residual in the activation type
 template <typename T, bool MOE>
-__global__ void __launch_bounds__(512) post_norm_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
+__global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
                                                         NormW n, MoeSum mo) {
     __shared__ float red[33], s_w[32];
     __shared__ int s_id[32];
@@ -806,7 +806,7 @@ __global__ void __launch_bounds__(512) post_norm_kernel(T* __restrict__ x, int l
 
 // out[j] = norm(resid[rows ? rows[j] : row0 + j])
 template <typename T>
-__global__ void __launch_bounds__(512) norm_rows_kernel(T* __restrict__ out, int ldo, const float* __restrict__ resid, int ldr, const int* __restrict__ rows,
+__global__ void __launch_bounds__(1024) norm_rows_kernel(T* __restrict__ out, int ldo, const float* __restrict__ resid, int ldr, const int* __restrict__ rows,
                                                         int row0, NormW n) {
     __shared__ float red[33];
     extern __shared__ float row[];
@@ -820,7 +820,7 @@ __global__ void __launch_bounds__(512) norm_rows_kernel(T* __restrict__ out, int
     for (int i = threadIdx.x; i < n.dim; i += blockDim.x)
         out[(size_t)blockIdx.x * ldo + i] = as_act<T>((row[i] - mean) * rstd * n.w[i] + (n.b ? n.b[i] : 0.f));
 }
-static int norm_threads(int dim) { return dim >= 2048 ? 512 : (dim >= 512 ? 256 : 128); }
+static int norm_threads(int dim, int rows) { return dim >= 2048 ? (rows <= 64 ? 1024 : 512) : (dim >= 512 ? 256 : 128); }
 }  // namespace lsb
 
 // Post-norm residual update: resid += norm(sub), x = resid in the activation type (f32: fp32, else bf16).  layer 1: layer norm with bias b,
@@ -832,7 +832,7 @@ LSB_API int lsb_post_norm(void* x, int ldx, void* resid, int ldr, const void* su
     NormW n{(const float*)w, (const float*)b, dim, eps, layer};
     MoeSum mo{(const float*)y, (const float*)wts, (const int*)ids, (const int*)slot_of, S, experts, ldy};
     cudaStream_t st = (cudaStream_t)stream;
-#define LSB_PN(T, M) launch_pdl((post_norm_kernel<T, M>), rows, norm_threads(dim), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, n, mo)
+#define LSB_PN(T, M) launch_pdl((post_norm_kernel<T, M>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, n, mo)
     if (f32) { if (y) LSB_PN(float, true); else LSB_PN(float, false); }
     else { if (y) LSB_PN(bf16, true); else LSB_PN(bf16, false); }
 #undef LSB_PN
@@ -844,8 +844,8 @@ LSB_API int lsb_norm_rows(void* out, int ldo, const void* resid, int ldr, const 
     if (dim < 1 || dim > 12000) return -1;
     NormW n{(const float*)w, (const float*)b, dim, eps, layer};
     cudaStream_t st = (cudaStream_t)stream;
-    if (f32) launch_pdl((norm_rows_kernel<float>), rows, norm_threads(dim), (size_t)dim * 4, st, (float*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
-    else launch_pdl((norm_rows_kernel<bf16>), rows, norm_threads(dim), (size_t)dim * 4, st, (bf16*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
+    if (f32) launch_pdl((norm_rows_kernel<float>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (float*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
+    else launch_pdl((norm_rows_kernel<bf16>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (bf16*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
     LSB_CHECK_LAUNCH();
 }
 

@@ -476,3 +476,16 @@ def test_random_full_size_layers_run():
     eng = engine(BlockModel.random_init(get_preset("tiny-gazutar"), DEV, seed=1))
     out = eng.generate(list(range(2, 40)), 6)
     assert len(out) == 6 and eng.kernel_launches > 0
+
+
+def test_the_server_boots_a_checkpoint_directory(tmp_path_factory):
+    from layerstorm_b200.cli import serve
+    c, m, toks, ref = load(tmp_path_factory, "odd", "bfloat16")
+    d = _cache["odd", "bfloat16", "files"][1]
+    args = serve.build_parser().parse_args(["--model", str(d), "--max-sequence-length", "512", "--max-concurrent", "3", "--tokenizer-mode", "byte"])
+    cfg, shape, ckpt, _ = serve.resolve_config(args)
+    eng = serve.build_engine(cfg, shape, ckpt, args)
+    assert isinstance(eng.model, BlockModel) and eng.supports_mixed_steps and eng.model.kv_fmt == "bf16"
+    s = eng.create_sequence()
+    _, lg = eng.prefill(s, toks[1], want_logits=True)
+    assert rms(lg[None], ref[1][-1:]) < TOL["bfloat16"]
