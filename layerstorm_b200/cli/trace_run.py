@@ -2,7 +2,7 @@
 
 Reads one JSON object per line from standard input,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "x", "tokens": [11, 4], "want": [1]}, {"id": "y", "tokens": [9]}], "end": ["y"]}
 
 and runs all entries of a line as one batch (``Engine.step``): each request's next tokens, appended to what earlier steps left in the
 cache and state.  ``want`` lists the places among an entry's tokens whose logits are asked for; a step that wants any writes
@@ -27,7 +27,7 @@ def build_parser() -> argparse.ArgumentParser:
     p.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                    help="bfloat16: the precisions this model is served with; float32: everything in fp32")
     p.add_argument("--out", required=True, help="directory for <step>.f32")
-    p.add_argument("--max-tokens", type=int, required=True, help="tokens that live requests hold at any time (the cache pool is made for these)")
+    p.add_argument("--max-tokens", type=int, required=True, help="size of the cache pool: tokens of all unfinished requests together")
     return p
 
 
