@@ -64,7 +64,8 @@ def _head_pad(d: int) -> int:
 def kv_bytes_per_token(mc: ModelConfig, backend: str = "snapmla", tp: int = 1, kv_mode: str = "sharded") -> float:
     """All attention layers, one token, on one GPU.  Sharded mode keeps 1/tp of the rows per rank."""
     if mc.blocks:
-        return float(sum(b.kv_heads * (_head_pad(b.dim) + _head_pad(b.vdim)) * 2 for b in mc.blocks if not b.recurrent))
+        lat = lambda b: _align(b.kv_rank, 16) + _align(b.rot_dim, 16) if b.kv_from < 0 else 0       # (layers may read another layer's rows)
+        return float(sum(2 * (lat(b) if b.latent else b.kv_heads * (_head_pad(b.dim) + _head_pad(b.vdim))) for b in mc.blocks if not b.recurrent))
     mla = mc.mla_layers()
     idx_layers = len({mc.index_source_layer(i) for i in mla}) if mc.has_indexer else 0
     per = len(mla) * kv_row_bytes(mc, backend) + idx_layers * indexer_row_bytes(mc)
@@ -110,11 +111,16 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
             rank = b.dim                                                 # the low-rank width is only in the tensors; this is its usual size
             w = (2 * b.kv_heads * b.dim + 2 * b.heads * b.vdim + b.heads + 2 * rank) * H + 3 * b.heads * (b.dim + b.vdim) * rank
             r.attention += w * 2 + ((2 * b.kv_heads * b.dim + b.heads * b.vdim) * b.conv + b.heads * b.dim) * 4
+        elif b.latent:
+            own = b.kv_rank + b.rot_dim if b.kv_from < 0 else 0
+            r.attention += ((b.heads * (b.dim + b.rot_dim + b.vdim + (1 if b.head_gate else 0)) + own) * H + b.heads * (b.dim + b.vdim) * b.kv_rank) * 2
         else:
             r.attention += (b.heads * (b.dim + b.vdim * (2 if b.out_gate else 1)) + b.kv_heads * (b.dim + b.vdim)) * H * 2
+        r.dense_ffn += 3 * b.dense_ff * H * 2 + mc.side_dim * H * 2 * 2
         if b.experts:
             r.router += (b.experts + b.identity) * (2 * H + 4)
-        r.norms += (4 if b.experts else 2) * H * 4
+            r.shared_expert += (3 * b.shared_ff + (1 if b.shared_ff else 0)) * H * 2
+        r.norms += (4 if b.has_ff else 2) * H * 4 * (2 if mc.norm_place == "sandwich" else 1) + (H * 4 if mc.side_dim else 0)
     for i in range(0 if mc.blocks else mc.n_layers):
         if mc.is_kda_layer(i):
             C = mc.kda_heads * mc.kda_head_dim
@@ -148,7 +154,7 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
             # two hyper-connection passes per layer: mixing matrix [(2n + n^2), n H] fp32, its base vector and three scales
             r.norms += 2 * ((2 * n + n * n) * (n * H + 1) + 3) * 4
     r.norms += H * 4                                                     # output norm
-    r.embedding = 0 if embed_on_host else mc.vocab * H * 2
+    r.embedding = (0 if embed_on_host else mc.vocab * H * 2) + mc.vocab * mc.n_layers * mc.side_dim * 2
     r.head = int(mc.vocab * H * 2 / tp)
     return r
 

@@ -41,8 +41,8 @@ CXX_FLAGS = ["-O2", "-g", "-std=c++20", "-fPIC", "-Wall", "-Wno-unused-function"
              "-I", str(CSRC / "include"), "-I", str(CSRC / "runtime")]
 
 
-# kernel files of a model family (models described layer by layer run without the MLA, indexer, hyper-connection and expert-parallel kernels)
-FAMILIES = {"blocks": ("attn", "delta", "gemm_tc", "gemv", "moe", "moe_tc", "norm", "sampling")}
+# kernel files of a model family (models described layer by layer run without the MLA-family, indexer, hyper-connection and expert-parallel kernels)
+FAMILIES = {"blocks": ("attn", "delta", "gemm_tc", "gemv", "latent", "moe", "moe_tc", "norm", "sampling")}
 
 
 def _rel(p) -> str:

@@ -220,13 +220,13 @@ template <> struct RowOf<6> {
     static __device__ __forceinline__ T make(const uint8_t* w, const uint8_t*, int n, int K) { return T{w + (size_t)n * (K + (K >> 4)), K}; }
 };
 
-// act[pair][f] = silu(min(g,limit)) * clamp(u) ; g = x[row] . Wgate[f], u = x[row] . Wup[f]
+// act[pair][f] = glu_act(g, u) ; g = x[row] . Wgate[f], u = x[row] . Wup[f]
 template <int FMT>
 __global__ void __launch_bounds__(256) moe_gateup_kernel(const bf16* __restrict__ x, const uint8_t* __restrict__ arena,
                                                          const int* __restrict__ slot_of, ExpertFmt ef,
                                                          const int* __restrict__ group_expert, const int* __restrict__ group_n,
                                                          const int* __restrict__ group_pairs, const int* __restrict__ n_groups,
-                                                         bf16* __restrict__ act, int S, float limit, int* __restrict__ miss_flag) {
+                                                         bf16* __restrict__ act, int S, GluAct ga, int* __restrict__ miss_flag) {
     pdl_wait();
     pdl_launch_dependents();
     const int g = blockIdx.y;
@@ -273,9 +273,11 @@ __global__ void __launch_bounds__(256) moe_gateup_kernel(const bf16* __restrict_
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
         if (m < n) {
-            float gv = warp_sum(ag[m]) * sg, uv = warp_sum(au[m]) * su;
-            if (limit > 0.f) { gv = fminf(gv, limit); uv = fminf(fmaxf(uv, -limit), limit); }
-            if (lane == 0) act[(size_t)pr[m] * ef.F + f] = __float2bfloat16(siluf_(gv) * uv);
+            const float gv = warp_sum(ag[m]) * sg, uv = warp_sum(au[m]) * su;
+            if (lane == 0) {
+                const float c = glu_in_scale(ga, pr[m]);
+                act[(size_t)pr[m] * ef.F + f] = __float2bfloat16(glu_act(gv * c, uv * c, ga));
+            }
         }
     }
     pdl_launch_dependents();
@@ -346,7 +348,7 @@ template <bool GATEUP>
 __global__ void __launch_bounds__(256) moe_f32_kernel(const float* __restrict__ in, const uint8_t* __restrict__ arena, const int* __restrict__ slot_of,
                                                       ExpertFmt ef, const int* __restrict__ group_expert, const int* __restrict__ group_n,
                                                       const int* __restrict__ group_pairs, const int* __restrict__ n_groups, float* __restrict__ out,
-                                                      int S, float limit, int* __restrict__ miss_flag) {
+                                                      int S, GluAct ga, int* __restrict__ miss_flag) {
     pdl_wait();
     pdl_launch_dependents();
     const int g = blockIdx.y;
@@ -367,8 +369,8 @@ __global__ void __launch_bounds__(256) moe_f32_kernel(const float* __restrict__ 
         a = warp_sum(a);
         if (GATEUP) {
             b = warp_sum(b);
-            if (limit > 0.f) { a = fminf(a, limit); b = fminf(fmaxf(b, -limit), limit); }
-            a = a / (1.f + expf(-a)) * b;
+            const float c = glu_in_scale(ga, pr);
+            a = glu_act<true>(a * c, b * c, ga);
         }
         if (lane == 0) out[(size_t)pr * N + n_out] = a;
     }
@@ -383,7 +385,7 @@ __global__ void __launch_bounds__(256) moe_gateup_fp4_kernel(const bf16* __restr
                                                              const int* __restrict__ slot_of, ExpertFmt ef,
                                                              const int* __restrict__ group_expert, const int* __restrict__ group_n,
                                                              const int* __restrict__ group_pairs, const int* __restrict__ n_groups,
-                                                             bf16* __restrict__ act, int S, float limit, int* __restrict__ miss_flag, int run) {
+                                                             bf16* __restrict__ act, int S, GluAct ga, int* __restrict__ miss_flag, int run) {
     extern __shared__ __align__(16) uint8_t smraw[];
     __half* xs = reinterpret_cast<__half*>(smraw);
     __shared__ const bf16* rows[4];
@@ -431,9 +433,11 @@ __global__ void __launch_bounds__(256) moe_gateup_fp4_kernel(const bf16* __restr
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
             if (m < n) {
-                float gv = warp_sum(ag[m]) * sg, uv = warp_sum(au[m]) * su;
-                if (limit > 0.f) { gv = fminf(gv, limit); uv = fminf(fmaxf(uv, -limit), limit); }
-                if (lane == 0) act[(size_t)pr[m] * ef.F + f] = __float2bfloat16(siluf_(gv) * uv);
+                const float gv = warp_sum(ag[m]) * sg, uv = warp_sum(au[m]) * su;
+                if (lane == 0) {
+                    const float c = glu_in_scale(ga, pr[m]);
+                    act[(size_t)pr[m] * ef.F + f] = __float2bfloat16(glu_act(gv * c, uv * c, ga));
+                }
             }
         }
     }
@@ -547,16 +551,40 @@ __global__ void moe_combine_kernel(float* __restrict__ out, const float* __restr
     pdl_launch_dependents();
 }
 
-// Dense SwiGLU on a fused [rows, 2F] fp32 projection (gate | up) -> bf16 [rows, F].
-__global__ void swiglu_kernel(bf16* __restrict__ out, const float* __restrict__ gu, int F, float limit) {
+// Dense gated unit over a fused fp32 projection (gate columns at off_g, up columns at off_u of rows of ld) -> [rows, ldo] bf16 / fp32; columns F .. ldo
+// are zeroed.  off_s >= 0: the row's result times sigmoid of the projection's column off_s.
+template <typename T>
+__global__ void glu_kernel(T* __restrict__ out, int ldo, const float* __restrict__ z, int ld, int off_g, int off_u, int off_s, int F, GluAct ga) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.y, f = blockIdx.x * blockDim.x + threadIdx.x;
-    if (f >= F) return;
-    float g = gu[(size_t)r * 2 * F + f], u = gu[(size_t)r * 2 * F + F + f];
-    if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
-    out[(size_t)r * F + f] = __float2bfloat16(siluf_(g) * u);
+    if (f >= ldo) return;
+    const float* zr = z + (size_t)r * ld;
+    float v = 0.f;
+    if (f < F) {
+        v = glu_act<sizeof(T) == 4>(zr[off_g + f], zr[off_u + f], ga);
+        if (off_s >= 0) v *= 1.f / (1.f + expf(-zr[off_s]));
+    }
+    if constexpr (sizeof(T) == 2) out[(size_t)r * ldo + f] = __float2bfloat16(v);
+    else out[(size_t)r * ldo + f] = v;
     pdl_launch_dependents();
+}
+
+// Gate of a per-token side input: out[r][c] = gelu_tanh(z[r][c]) * table[tok[r]][off + c], columns dim .. ldo zeroed.
+template <typename T>
+__global__ void side_gate_kernel(T* __restrict__ out, int ldo, const float* __restrict__ z, int ldz, const bf16* __restrict__ table, long long ldt, int off, int dim,
+                                 const int* __restrict__ tok, int vocab) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int r = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x, id = tok[r];
+    if (c >= ldo) return;
+    float v = 0.f;
+    if (c < dim && id >= 0 && id < vocab) {
+        const float x = z[(size_t)r * ldz + c], u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
+        v = 0.5f * x * (1.f + tanhf(u)) * __bfloat162float(table[(size_t)id * ldt + off + c]);
+    }
+    if constexpr (sizeof(T) == 2) out[(size_t)r * ldo + c] = __float2bfloat16(v);
+    else out[(size_t)r * ldo + c] = v;
 }
 
 }  // namespace lsb
@@ -611,9 +639,9 @@ LSB_API int lsb_moe_build_groups(const void* ids, int npairs, int E_total, void*
 
 // Pair mode (group_n == null): every (row, slot) pair is its own group - group_expert is the
 // routing id array itself, group g is pair g; used for small batches where no build pass is needed.
-LSB_API int lsb_moe_gateup(const void* x, const void* arena, const void* slot_of, const void* fmt_struct,
-                           const void* group_expert, const void* group_n, const void* group_pairs, const void* n_groups,
-                           void* act, int S, int max_groups, float limit, void* miss_flag, int run, void* stream) {
+static int moe_gateup(const void* x, const void* arena, const void* slot_of, const void* fmt_struct, const void* group_expert, const void* group_n,
+                      const void* group_pairs, const void* n_groups, void* act, int S, int max_groups, GluAct ga, void* miss_flag, int run,
+                      void* stream) {
     ExpertFmt ef = *reinterpret_cast<const ExpertFmt*>(fmt_struct);
     cudaStream_t st = (cudaStream_t)stream;
     if (ef.fmt == 2 && ef.F % 128 == 0 && ef.H % 128 == 0) {   // K % 64 == 0 follows
@@ -629,23 +657,23 @@ LSB_API int lsb_moe_gateup(const void* x, const void* arena, const void* slot_of
         }
         if (!group_n)
             launch_pdl((moe_gateup_fp4_kernel<1>), g2, 256, (size_t)ef.H * 2 + sc_bytes, st, (const bf16*)x, (const uint8_t*)arena, (const int*)slot_of, ef, (const int*)group_expert,
-                                                                        nullptr, nullptr, nullptr, (bf16*)act, S, limit, (int*)miss_flag, run);
+                                                                        nullptr, nullptr, nullptr, (bf16*)act, S, ga, (int*)miss_flag, run);
         else
             launch_pdl((moe_gateup_fp4_kernel<4>), g2, 256, (size_t)ef.H * 8 + sc_bytes, st, (const bf16*)x, (const uint8_t*)arena, (const int*)slot_of, ef, (const int*)group_expert,
-                                                                        (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (bf16*)act, S, limit,
+                                                                        (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (bf16*)act, S, ga,
                                                                         (int*)miss_flag, run);
         LSB_CHECK_LAUNCH();
     }
     if (ef.fmt == 7) {
         if (!group_n) return -1;
         launch_pdl((moe_f32_kernel<true>), dim3((ef.F + 7) / 8, max_groups), 256, 0, st, (const float*)x, (const uint8_t*)arena, (const int*)slot_of, ef,
-                   (const int*)group_expert, (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (float*)act, S, limit, (int*)miss_flag);
+                   (const int*)group_expert, (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (float*)act, S, ga, (int*)miss_flag);
         LSB_CHECK_LAUNCH();
     }
     if (!group_n) return -1;   // pair mode is only implemented for the NVFP4 fast path
     dim3 grid((ef.F + 7) / 8, max_groups);
 #define ARGS (const bf16*)x, (const uint8_t*)arena, (const int*)slot_of, ef, (const int*)group_expert, (const int*)group_n, \
-             (const int*)group_pairs, (const int*)n_groups, (bf16*)act, S, limit, (int*)miss_flag
+             (const int*)group_pairs, (const int*)n_groups, (bf16*)act, S, ga, (int*)miss_flag
     if (ef.fmt == 0) launch_pdl((moe_gateup_kernel<0>), grid, 256, 0, st, ARGS);
     else if (ef.fmt == 1) launch_pdl((moe_gateup_kernel<1>), grid, 256, 0, st, ARGS);
     else if (ef.fmt == 2) launch_pdl((moe_gateup_kernel<2>), grid, 256, 0, st, ARGS);
@@ -656,6 +684,22 @@ LSB_API int lsb_moe_gateup(const void* x, const void* arena, const void* slot_of
     else return -1;
 #undef ARGS
     LSB_CHECK_LAUNCH();
+}
+
+LSB_API int lsb_moe_gateup(const void* x, const void* arena, const void* slot_of, const void* fmt_struct,
+                           const void* group_expert, const void* group_n, const void* group_pairs, const void* n_groups,
+                           void* act, int S, int max_groups, float limit, void* miss_flag, int run, void* stream) {
+    return moe_gateup(x, arena, slot_of, fmt_struct, group_expert, group_n, group_pairs, n_groups, act, S, max_groups, GluAct{limit, 1.f, 0.f, nullptr}, miss_flag,
+                      run, stream);
+}
+
+// The same with another gated unit (GluAct): sigmoid slope alpha, linear half shifted by `shift`, in_scale [rows * S] on the experts' inputs (or null).
+LSB_API int lsb_moe_gateup_act(const void* x, const void* arena, const void* slot_of, const void* fmt_struct,
+                               const void* group_expert, const void* group_n, const void* group_pairs, const void* n_groups,
+                               void* act, int S, int max_groups, float limit, float alpha, float shift, const void* in_scale, void* miss_flag, int run,
+                               void* stream) {
+    return moe_gateup(x, arena, slot_of, fmt_struct, group_expert, group_n, group_pairs, n_groups, act, S, max_groups,
+                      GluAct{limit, alpha, shift, (const float*)in_scale}, miss_flag, run, stream);
 }
 
 LSB_API int lsb_moe_down(const void* act, const void* arena, const void* slot_of, const void* fmt_struct,
@@ -684,7 +728,7 @@ LSB_API int lsb_moe_down(const void* act, const void* arena, const void* slot_of
     if (!group_n) return -1;
     if (ef.fmt == 7) {
         launch_pdl((moe_f32_kernel<false>), dim3((ef.H + 7) / 8, max_groups), 256, 0, st, (const float*)act, (const uint8_t*)arena, (const int*)slot_of, ef,
-                   (const int*)group_expert, (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (float*)y, 1, 0.f, nullptr);
+                   (const int*)group_expert, (const int*)group_n, (const int*)group_pairs, (const int*)n_groups, (float*)y, 1, GluAct{0.f, 1.f, 0.f, nullptr}, nullptr);
         LSB_CHECK_LAUNCH();
     }
     dim3 grid((ef.H + 15) / 16, max_groups);
@@ -716,8 +760,30 @@ LSB_API int lsb_moe_combine(void* out, const void* y, const void* wts, const voi
 }
 
 LSB_API int lsb_swiglu(void* out, const void* gu, int rows, int F, float limit, void* stream) {
-    dim3 grid((F + 255) / 256, rows);
-    launch_pdl((swiglu_kernel), grid, 256, 0, (cudaStream_t)stream, (bf16*)out, (const float*)gu, F, limit);
+    launch_pdl((glu_kernel<bf16>), dim3((F + 255) / 256, rows), 256, 0, (cudaStream_t)stream, (bf16*)out, F, (const float*)gu, 2 * F, 0, F, -1, F,
+               GluAct{limit, 1.f, 0.f, nullptr});
+    LSB_CHECK_LAUNCH();
+}
+
+// Gated unit of any two column blocks of a projection: see glu_kernel.  f32: fp32 output.
+LSB_API int lsb_glu(void* out, int ldo, const void* z, int ld, int off_g, int off_u, int off_s, int rows, int F, float limit, float alpha, float shift, int f32,
+                    void* stream) {
+    if (rows < 1 || rows > 65535 || F < 1 || ldo < F) return -1;
+    const dim3 grid((ldo + 255) / 256, rows);
+    const GluAct ga{limit, alpha, shift, nullptr};
+    if (f32) launch_pdl((glu_kernel<float>), grid, 256, 0, (cudaStream_t)stream, (float*)out, ldo, (const float*)z, ld, off_g, off_u, off_s, F, ga);
+    else launch_pdl((glu_kernel<bf16>), grid, 256, 0, (cudaStream_t)stream, (bf16*)out, ldo, (const float*)z, ld, off_g, off_u, off_s, F, ga);
+    LSB_CHECK_LAUNCH();
+}
+
+LSB_API int lsb_side_gate(void* out, int ldo, const void* z, int ldz, const void* table, long long ld_table, int off, int dim, const void* tok, int vocab,
+                          int rows, int f32, void* stream) {
+    if (rows < 1 || rows > 65535 || dim < 1 || ldo < dim) return -1;
+    const dim3 grid((ldo + 127) / 128, rows);
+    if (f32) launch_pdl((side_gate_kernel<float>), grid, 128, 0, (cudaStream_t)stream, (float*)out, ldo, (const float*)z, ldz, (const bf16*)table, ld_table, off, dim,
+                        (const int*)tok, vocab);
+    else launch_pdl((side_gate_kernel<bf16>), grid, 128, 0, (cudaStream_t)stream, (bf16*)out, ldo, (const float*)z, ldz, (const bf16*)table, ld_table, off, dim,
+                    (const int*)tok, vocab);
     LSB_CHECK_LAUNCH();
 }
 

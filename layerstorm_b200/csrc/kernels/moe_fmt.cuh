@@ -17,4 +17,17 @@ struct ExpertFmt {
     __host__ __device__ int down_fmt() const { return fmt_down1 ? fmt_down1 - 1 : fmt; }
 };
 
+// Activation of a gated unit: g = min(g, limit), u = clamp(u, -limit, limit) (limit 0: as they are), then g sigmoid(alpha g) (u + shift).
+// in_scale: one factor per (row, slot) pair on the unit's input - the products are linear in it, so it multiplies g and u in fp32 - or null.
+struct GluAct { float limit, alpha, shift; const float* in_scale; };
+
+#ifdef __CUDACC__
+template <bool EXACT = false> __device__ __forceinline__ float glu_act(float g, float u, const GluAct& a) {
+    if (a.limit > 0.f) { g = fminf(g, a.limit); u = fminf(fmaxf(u, -a.limit), a.limit); }
+    const float e = EXACT ? expf(-a.alpha * g) : __expf(-a.alpha * g);
+    return g / (1.f + e) * (u + a.shift);
+}
+__device__ __forceinline__ float glu_in_scale(const GluAct& a, int pair) { return a.in_scale ? a.in_scale[pair] : 1.f; }
+#endif
+
 }  // namespace lsb

@@ -239,7 +239,7 @@ struct MoeTcParams {
     const int* sorted_pair;
     __half* act;          // gate/up output, [pairs, F] fp16 in sorted order
     float* y;             // down output, [npairs, H] fp32 in pair order
-    float limit;
+    GluAct ga;
     int* miss_flag; int* err;
     // expert-parallel mode (ep.nranks > 0): the gate/up kernel waits for the peers' token rows (phase 1) before its
     // first load, the down kernel stores its rows straight into the token owners' buffers and publishes phase 2
@@ -604,9 +604,8 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                     for (int j = 0; j < 16; ++j) {
                         if (c0 + j < ncols && n < NOUT) {
                             if (GATEUP) {
-                                float gv = gq[j] * sg, uv = uq[j] * su;
-                                if (p.limit > 0.f) { gv = fminf(gv, p.limit); uv = fminf(fmaxf(uv, -p.limit), p.limit); }
-                                p.act[(size_t)(row0 + c0 + j) * NOUT + n] = __float2half_rn(siluf_(gv) * uv);
+                                const float c = p.ga.in_scale ? p.ga.in_scale[p.sorted_pair[row0 + c0 + j]] : 1.f;
+                                p.act[(size_t)(row0 + c0 + j) * NOUT + n] = __float2half_rn(glu_act(gq[j] * sg * c, uq[j] * su * c, p.ga));
                             } else if (ep_mode) {
                                 const int2 ra = p.ep.ret[p.ep.rank][row0 + c0 + j];      // (token owner, pair index there)
                                 p.ep.y[ra.x][(size_t)ra.y * NOUT + n] = gq[j] * sg;       // NVLink store into the owner's buffer
@@ -738,9 +737,9 @@ LSB_API int lsb_moe_tc_gather(const void* x, const void* sorted_pair, const void
 // gateup != 0: act[pos][f] = SwiGLU(xs[pos] . Wgate[f], xs[pos] . Wup[f]) for every sorted position (fp16, [cap_rows, F]).
 // gateup == 0: y[pair][h] = act[pos] . Wdown[h]  (fp32, [npairs, H], rows in pair order).
 // `b` is the fp16 token operand ([cap_rows, K], K = H for gate/up and F for down), 16-byte aligned.
-LSB_API int lsb_moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* arena, const void* slot_of, const void* fmt_struct,
+static int moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* arena, const void* slot_of, const void* fmt_struct,
                            const void* tile_expert, const void* tile_row0, const void* tile_n, const void* counters,
-                           const void* sorted_pair, void* out, int BN, int max_tiles, float limit, void* miss_flag, void* err,
+                           const void* sorted_pair, void* out, int BN, int max_tiles, GluAct ga, void* miss_flag, void* err,
                            const void* ep, void* stream) {
     const ExpertFmt* ef = (const ExpertFmt*)fmt_struct;
     const int K = gateup ? ef->H : ef->F, nout = gateup ? ef->F : ef->H;
@@ -755,7 +754,7 @@ LSB_API int lsb_moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* 
     p.tile_expert = (const int*)tile_expert; p.tile_row0 = (const int*)tile_row0; p.tile_n = (const int*)tile_n;
     p.counters = (const int*)counters; p.sorted_pair = (const int*)sorted_pair;
     p.act = gateup ? (__half*)out : nullptr; p.y = gateup ? nullptr : (float*)out;
-    p.limit = limit; p.miss_flag = (int*)miss_flag; p.err = (int*)err;
+    p.ga = ga; p.miss_flag = (int*)miss_flag; p.err = (int*)err;
     if (ep) p.ep = *(const EpComm*)ep; else { memset(&p.ep, 0, sizeof(p.ep)); }
     p.ldo = nout; p.out_bf16 = 0; p.down_scale = 0.f;
     cudaStream_t st = (cudaStream_t)stream;
@@ -773,6 +772,23 @@ LSB_API int lsb_moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* 
         }
     }
     return -1;
+}
+
+LSB_API int lsb_moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* arena, const void* slot_of, const void* fmt_struct,
+                           const void* tile_expert, const void* tile_row0, const void* tile_n, const void* counters,
+                           const void* sorted_pair, void* out, int BN, int max_tiles, float limit, void* miss_flag, void* err,
+                           const void* ep, void* stream) {
+    return moe_tc_ffn(gateup, b, cap_rows, arena, slot_of, fmt_struct, tile_expert, tile_row0, tile_n, counters, sorted_pair, out, BN, max_tiles,
+                      GluAct{limit, 1.f, 0.f, nullptr}, miss_flag, err, ep, stream);
+}
+
+// The gate/up half with another gated unit (GluAct): in_scale [npairs] in pair order, or null.
+LSB_API int lsb_moe_tc_gateup_act(const void* b, int cap_rows, const void* arena, const void* slot_of, const void* fmt_struct,
+                                  const void* tile_expert, const void* tile_row0, const void* tile_n, const void* counters,
+                                  const void* sorted_pair, void* out, int BN, int max_tiles, float limit, float alpha, float shift, const void* in_scale,
+                                  void* miss_flag, void* err, void* stream) {
+    return moe_tc_ffn(1, b, cap_rows, arena, slot_of, fmt_struct, tile_expert, tile_row0, tile_n, counters, sorted_pair, out, BN, max_tiles,
+                      GluAct{limit, alpha, shift, (const float*)in_scale}, miss_flag, err, nullptr, stream);
 }
 
 // Dense linear layer with quantised weights on the tensor cores: out[m][n] = alpha * sum_k x16[m][k] * W[n][k].

@@ -723,13 +723,17 @@ LSB_API int lsb_cosine_sim(const void* a, const void* b, int rows, int dim, int 
 }
 
 namespace lsb {
-// ---- norm on a sublayer's output (post-norm residual streams), RMS or layer norm with bias ----
-struct NormW { const float* w; const float* b; int dim; float eps; int layer; };      // layer 0: RMS norm; b may be null
+// ---- norms of the residual stream, on a sublayer's output and in front of the next sublayer ----
+enum { kNormRms = 0, kNormLayer = 1, kNormTanh = 2, kNormNone = 3 };    // kNormTanh: dynamic tanh, b + w tanh(alpha x), element-wise
+struct NormW { const float* w; const float* b; const float* alpha; int dim; float eps; int kind; };      // b may be null
+__host__ __device__ __forceinline__ bool norm_moments_needed(int kind) { return kind == kNormRms || kind == kNormLayer; }
 
 // row[0..dim) (shared memory) -> scale and shift of its normalisation: n(x) = (x - mean) * rstd
 __device__ __forceinline__ void norm_moments(const float* row, const NormW& n, float* red, float& mean, float& rstd) {
     mean = 0.f;
-    if (n.layer) {
+    rstd = 1.f;
+    if (!norm_moments_needed(n.kind)) return;
+    if (n.kind == kNormLayer) {
         float s = 0.f;
         for (int i = threadIdx.x; i < n.dim; i += blockDim.x) s += row[i];
         mean = block_sum(s, red) / (float)n.dim;
@@ -738,69 +742,122 @@ __device__ __forceinline__ void norm_moments(const float* row, const NormW& n, f
     for (int i = threadIdx.x; i < n.dim; i += blockDim.x) { const float d = row[i] - mean; v = fmaf(d, d, v); }
     rstd = 1.f / sqrtf(block_sum(v, red) / (float)n.dim + n.eps);
 }
+// element i of the normalised row; alpha: *n.alpha (dynamic tanh)
+__device__ __forceinline__ float norm_apply(float v, int i, const NormW& n, float mean, float rstd, float alpha) {
+    if (n.kind == kNormNone) return v;
+    const float y = n.kind == kNormTanh ? tanhf(alpha * v) : (v - mean) * rstd;
+    return y * n.w[i] + (n.b ? n.b[i] : 0.f);
+}
 template <typename T> __device__ __forceinline__ T as_act(float v);
 template <> __device__ __forceinline__ bf16 as_act<bf16>(float v) { return __float2bfloat16(v); }
 template <> __device__ __forceinline__ float as_act<float>(float v) { return v; }
 
-// The weighted sum of a row's expert outputs, slots in order: slot s holds expert ids[s]; ids below `experts` take their row of y (none when the
-// expert is not resident), the others are identity experts and take the residual stream itself.
+// The sum of a row's expert outputs, slots in order: slot s holds expert ids[s]; ids below `experts` take their row of y (none when the expert is not
+// resident), the others are identity experts and take the residual stream itself.  wts null: every weight is 1.
 struct MoeSum { const float* y; const float* wts; const int* ids; const int* slot_of; int S, experts, ldy; };
 
-// resid[r] += norm(sub[r]) (or norm of the MoE sum), x[r] = the new residual in the activation type
+__device__ __forceinline__ void load_slots(const MoeSum& mo, int r, int* s_id, float* s_w) {
+    if ((int)threadIdx.x < mo.S) {
+        int id = mo.ids[(size_t)r * mo.S + threadIdx.x];
+        if (id >= 0 && id < mo.experts && mo.slot_of[id] < 0) id = -1;
+        s_id[threadIdx.x] = id;
+        s_w[threadIdx.x] = mo.wts ? mo.wts[(size_t)r * mo.S + threadIdx.x] : 1.f;
+    }
+    __syncthreads();
+}
+__device__ __forceinline__ float4 sum_slots4(float4 a, const MoeSum& mo, const float* yr, const float* rr, int i, const int* s_id, const float* s_w) {
+#pragma unroll 4
+    for (int s = 0; s < mo.S; ++s) {
+        const int id = s_id[s];
+        if (id < 0) continue;
+        const float4 v = *reinterpret_cast<const float4*>(id < mo.experts ? yr + (size_t)s * mo.ldy + i : rr + i);
+        const float w = s_w[s];
+        a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+    }
+    return a;
+}
+__device__ __forceinline__ float sum_slots(float a, const MoeSum& mo, const float* yr, const float* rr, int i, const int* s_id, const float* s_w) {
+    for (int s = 0; s < mo.S; ++s) {
+        const int id = s_id[s];
+        if (id >= 0) a = fmaf(s_w[s], id < mo.experts ? yr[(size_t)s * mo.ldy + i] : rr[i], a);
+    }
+    return a;
+}
+
+// resid[r] += post(sub[r] + MoE sum of the row), x[r] = pre(the new residual) in the activation type.  sub may be null.  Whole rows per block.
 template <typename T, bool MOE>
 __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
-                                                        NormW n, MoeSum mo) {
+                                                        NormW post, NormW pre, MoeSum mo) {
     __shared__ float red[33], s_w[32];
     __shared__ int s_id[32];
     extern __shared__ float row[];
-    const int r = blockIdx.x;
+    const int r = blockIdx.x, dim = post.dim;
     float* rr = resid + (size_t)r * ldr;
     pdl_wait();
     pdl_launch_dependents();
+    const float* sr = sub ? sub + (size_t)r * lds : nullptr;
     if (MOE) {
-        if (threadIdx.x < mo.S) {
-            int id = mo.ids[(size_t)r * mo.S + threadIdx.x];
-            if (id >= 0 && id < mo.experts && mo.slot_of[id] < 0) id = -1;
-            s_id[threadIdx.x] = id;
-            s_w[threadIdx.x] = mo.wts[(size_t)r * mo.S + threadIdx.x];
-        }
-        __syncthreads();
+        load_slots(mo, r, s_id, s_w);
         const float* yr = mo.y + (size_t)r * mo.S * mo.ldy;
-        if (n.dim % 4 == 0 && mo.ldy % 4 == 0 && ldr % 4 == 0) {
-            for (int i = threadIdx.x * 4; i < n.dim; i += blockDim.x * 4) {
-                float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-                for (int s = 0; s < mo.S; ++s) {
-                    const int id = s_id[s];
-                    if (id < 0) continue;
-                    const float4 v = *reinterpret_cast<const float4*>(id < mo.experts ? yr + (size_t)s * mo.ldy + i : rr + i);
-                    const float w = s_w[s];
-                    a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
-                }
-                *reinterpret_cast<float4*>(row + i) = a;
-            }
+        if (dim % 4 == 0 && mo.ldy % 4 == 0 && ldr % 4 == 0 && lds % 4 == 0) {
+            for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4)
+                *reinterpret_cast<float4*>(row + i) = sum_slots4(sr ? *reinterpret_cast<const float4*>(sr + i) : make_float4(0.f, 0.f, 0.f, 0.f), mo, yr, rr, i, s_id, s_w);
         } else {
-            for (int i = threadIdx.x; i < n.dim; i += blockDim.x) {
-                float a = 0.f;
-                for (int s = 0; s < mo.S; ++s) {
-                    const int id = s_id[s];
-                    if (id >= 0) a = fmaf(s_w[s], id < mo.experts ? yr[(size_t)s * mo.ldy + i] : rr[i], a);
-                }
-                row[i] = a;
-            }
+            for (int i = threadIdx.x; i < dim; i += blockDim.x) row[i] = sum_slots(sr ? sr[i] : 0.f, mo, yr, rr, i, s_id, s_w);
         }
     } else {
-        const float* sr = sub + (size_t)r * lds;
-        for (int i = threadIdx.x; i < n.dim; i += blockDim.x) row[i] = sr[i];
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) row[i] = sr ? sr[i] : 0.f;
     }
     __syncthreads();
     float mean, rstd;
-    norm_moments(row, n, red, mean, rstd);
+    norm_moments(row, post, red, mean, rstd);
+    const float a_post = post.alpha ? *post.alpha : 0.f, a_pre = pre.alpha ? *pre.alpha : 0.f;
     T* xr = x + (size_t)r * ldx;
-    for (int i = threadIdx.x; i < n.dim; i += blockDim.x) {
-        const float v = rr[i] + ((row[i] - mean) * rstd * n.w[i] + (n.b ? n.b[i] : 0.f));
+    const bool again = norm_moments_needed(pre.kind);
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+        const float v = rr[i] + norm_apply(row[i], i, post, mean, rstd, a_post);
         rr[i] = v;
-        xr[i] = as_act<T>(v);
+        if (again) row[i] = v;
+        else xr[i] = as_act<T>(norm_apply(v, i, pre, 0.f, 1.f, a_pre));
+    }
+    if (!again) return;
+    __syncthreads();
+    norm_moments(row, pre, red, mean, rstd);
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) xr[i] = as_act<T>(norm_apply(row[i], i, pre, mean, rstd, a_pre));
+}
+
+// The same with element-wise norms on both sides: columns spread over blocks, four per thread, nothing exchanged.
+template <typename T, bool MOE>
+__global__ void __launch_bounds__(128) post_norm_wide_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
+                                                            NormW post, NormW pre, MoeSum mo) {
+    __shared__ float s_w[32];
+    __shared__ int s_id[32];
+    const int r = blockIdx.y, i = (blockIdx.x * 128 + threadIdx.x) * 4;
+    // the norms' vectors do not depend on the previous kernel: have them here before the dependency wait
+    const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool in = i < post.dim;
+    auto vec = [&](const float* v, float4 other) { return v && in ? *reinterpret_cast<const float4*>(v + i) : other; };
+    const float4 w0 = vec(post.w, one), b0 = vec(post.b, zero), w1 = vec(pre.w, one), b1 = vec(pre.b, zero);
+    const float a_post = post.alpha ? *post.alpha : 0.f, a_pre = pre.alpha ? *pre.alpha : 0.f;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (MOE) load_slots(mo, r, s_id, s_w);
+    if (!in) return;
+    float* rr = resid + (size_t)r * ldr;
+    float4 a = sub ? *reinterpret_cast<const float4*>(sub + (size_t)r * lds + i) : zero;
+    const float4 x0 = *reinterpret_cast<const float4*>(rr + i);
+    if (MOE) a = sum_slots4(a, mo, mo.y + (size_t)r * mo.S * mo.ldy, rr, i, s_id, s_w);
+    auto ew = [](float v, int kind, float alpha, float w, float b) { return kind == kNormTanh ? fmaf(tanhf(alpha * v), w, b) : v; };
+    const float4 v = make_float4(x0.x + ew(a.x, post.kind, a_post, w0.x, b0.x), x0.y + ew(a.y, post.kind, a_post, w0.y, b0.y),
+                                 x0.z + ew(a.z, post.kind, a_post, w0.z, b0.z), x0.w + ew(a.w, post.kind, a_post, w0.w, b0.w));
+    *reinterpret_cast<float4*>(rr + i) = v;
+    T* xr = x + (size_t)r * ldx + i;
+    const float y[4] = {ew(v.x, pre.kind, a_pre, w1.x, b1.x), ew(v.y, pre.kind, a_pre, w1.y, b1.y), ew(v.z, pre.kind, a_pre, w1.z, b1.z), ew(v.w, pre.kind, a_pre, w1.w, b1.w)};
+    if constexpr (sizeof(T) == 2) {
+        *reinterpret_cast<bf162*>(xr) = __floats2bfloat162_rn(y[0], y[1]);
+        *reinterpret_cast<bf162*>(xr + 2) = __floats2bfloat162_rn(y[2], y[3]);
+    } else {
+        *reinterpret_cast<float4*>(xr) = make_float4(y[0], y[1], y[2], y[3]);
     }
 }
 
@@ -817,32 +874,52 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(T* __restrict__ out, in
     __syncthreads();
     float mean, rstd;
     norm_moments(row, n, red, mean, rstd);
+    const float alpha = n.alpha ? *n.alpha : 0.f;
     for (int i = threadIdx.x; i < n.dim; i += blockDim.x)
-        out[(size_t)blockIdx.x * ldo + i] = as_act<T>((row[i] - mean) * rstd * n.w[i] + (n.b ? n.b[i] : 0.f));
+        out[(size_t)blockIdx.x * ldo + i] = as_act<T>(norm_apply(row[i], i, n, mean, rstd, alpha));
 }
 static int norm_threads(int dim, int rows) { return dim >= 2048 ? (rows <= 64 ? 1024 : 512) : (dim >= 512 ? 256 : 128); }
-}  // namespace lsb
 
-// Post-norm residual update: resid += norm(sub), x = resid in the activation type (f32: fp32, else bf16).  layer 1: layer norm with bias b,
-// 0: RMS norm.  y non-null: `sub` is the weighted sum of the row's S expert outputs instead (ids >= experts: identity experts).
-LSB_API int lsb_post_norm(void* x, int ldx, void* resid, int ldr, const void* sub, int lds, const void* w, const void* b, int rows, int dim, float eps,
-                          int layer, const void* y, const void* wts, const void* ids, const void* slot_of, int S, int experts, int ldy, int f32,
-                          void* stream) {
-    if (dim < 1 || dim > 12000 || (y && S > 32)) return -1;
-    NormW n{(const float*)w, (const float*)b, dim, eps, layer};
-    MoeSum mo{(const float*)y, (const float*)wts, (const int*)ids, (const int*)slot_of, S, experts, ldy};
-    cudaStream_t st = (cudaStream_t)stream;
-#define LSB_PN(T, M) launch_pdl((post_norm_kernel<T, M>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, n, mo)
-    if (f32) { if (y) LSB_PN(float, true); else LSB_PN(float, false); }
-    else { if (y) LSB_PN(bf16, true); else LSB_PN(bf16, false); }
+static int residual_update(void* x, int ldx, void* resid, int ldr, const void* sub, int lds, const NormW& post, const NormW& pre, const MoeSum& mo, int rows,
+                           int f32, cudaStream_t st) {
+    const int dim = post.dim;
+    if (dim < 1 || dim > 12000 || rows < 1 || (mo.y && mo.S > 32)) return -1;
+    for (const NormW* n : {&post, &pre})
+        if (n->kind < 0 || n->kind > kNormNone || (n->kind != kNormNone && !n->w) || (n->kind == kNormTanh && !n->alpha)) return -1;
+    if (!norm_moments_needed(post.kind) && !norm_moments_needed(pre.kind) && dim % 4 == 0 && ldx % 4 == 0 && ldr % 4 == 0 && lds % 4 == 0 && mo.ldy % 4 == 0 && rows < 65536) {
+        const dim3 grid((dim / 4 + 127) / 128, rows);
+#define LSB_PW(T, M) launch_pdl((post_norm_wide_kernel<T, M>), grid, 128, 0, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
+        if (f32) { if (mo.y) LSB_PW(float, true); else LSB_PW(float, false); }
+        else { if (mo.y) LSB_PW(bf16, true); else LSB_PW(bf16, false); }
+#undef LSB_PW
+        LSB_CHECK_LAUNCH();
+    }
+#define LSB_PN(T, M) launch_pdl((post_norm_kernel<T, M>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
+    if (f32) { if (mo.y) LSB_PN(float, true); else LSB_PN(float, false); }
+    else { if (mo.y) LSB_PN(bf16, true); else LSB_PN(bf16, false); }
 #undef LSB_PN
     LSB_CHECK_LAUNCH();
 }
+}  // namespace lsb
 
-LSB_API int lsb_norm_rows(void* out, int ldo, const void* resid, int ldr, const void* row_idx, int row0, const void* w, const void* b, int rows, int dim,
-                          float eps, int layer, int f32, void* stream) {
-    if (dim < 1 || dim > 12000) return -1;
-    NormW n{(const float*)w, (const float*)b, dim, eps, layer};
+// Residual update with a norm on either side: resid += post(sub + sum of the row's S expert outputs), x = pre(resid).  Kinds: 0 RMS, 1 layer norm,
+// 2 dynamic tanh (w, b, alpha: one number), 3 none (post: the sum as it is).  sub null: no dense part; y null: no experts; wts null: experts are
+// added as they are; ids >= experts: identity experts.
+LSB_API int lsb_resid_update(void* x, int ldx, void* resid, int ldr, const void* sub, int lds, int post_kind, const void* post_w, const void* post_b,
+                             const void* post_alpha, int pre_kind, const void* pre_w, const void* pre_b, const void* pre_alpha, int rows, int dim,
+                             float eps, const void* y, const void* wts, const void* ids, const void* slot_of, int S, int experts, int ldy, int f32,
+                             void* stream) {
+    const NormW post{(const float*)post_w, (const float*)post_b, (const float*)post_alpha, dim, eps, post_kind};
+    const NormW pre{(const float*)pre_w, (const float*)pre_b, (const float*)pre_alpha, dim, eps, pre_kind};
+    const MoeSum mo{(const float*)y, (const float*)wts, (const int*)ids, (const int*)slot_of, S, experts, ldy};
+    return residual_update(x, ldx, resid, ldr, sub, lds, post, pre, mo, rows, f32, (cudaStream_t)stream);
+}
+
+// out[j] = norm(resid[row]); kind as above.
+LSB_API int lsb_norm_rows(void* out, int ldo, const void* resid, int ldr, const void* row_idx, int row0, const void* w, const void* b, const void* alpha,
+                          int rows, int dim, float eps, int kind, int f32, void* stream) {
+    if (dim < 1 || dim > 12000 || kind < 0 || kind > kNormTanh || (kind == kNormTanh && !alpha)) return -1;
+    NormW n{(const float*)w, (const float*)b, (const float*)alpha, dim, eps, kind};
     cudaStream_t st = (cudaStream_t)stream;
     if (f32) launch_pdl((norm_rows_kernel<float>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (float*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);
     else launch_pdl((norm_rows_kernel<bf16>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (bf16*)out, ldo, (const float*)resid, ldr, (const int*)row_idx, row0, n);

@@ -18,7 +18,7 @@ __device__ __forceinline__ uint32_t sortable_key(float x) {
 // out[r] = table[ids[r]] (bf16 table; rows outside [vocab_lo, vocab_hi) give zeros, which is
 // what a vocabulary-sharded table contributes before the cross-rank sum).
 __global__ void embedding_kernel(float* __restrict__ out_f32, bf16* __restrict__ out_bf16, const bf16* __restrict__ table,
-                                 const int* __restrict__ ids, int hidden, int vocab_lo, int vocab_hi) {
+                                 const int* __restrict__ ids, int hidden, int vocab_lo, int vocab_hi, float scale) {
     const int r = blockIdx.x;
     pdl_wait();
     pdl_launch_dependents();
@@ -27,8 +27,9 @@ __global__ void embedding_kernel(float* __restrict__ out_f32, bf16* __restrict__
     const bf16* src = table + (size_t)(own ? id - vocab_lo : 0) * hidden;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         const bf16 v = own ? src[i] : __float2bfloat16(0.f);
-        if (out_f32) out_f32[(size_t)r * hidden + i] = __bfloat162float(v);
-        if (out_bf16) out_bf16[(size_t)r * hidden + i] = v;
+        const float f = __bfloat162float(v) * scale;
+        if (out_f32) out_f32[(size_t)r * hidden + i] = f;
+        if (out_bf16) out_bf16[(size_t)r * hidden + i] = scale == 1.f ? v : __float2bfloat16(f);
     }
     pdl_launch_dependents();
 }
@@ -270,11 +271,16 @@ __global__ void spec_verify_kernel(const int* __restrict__ draft, const int* __r
 }  // namespace lsb
 using namespace lsb;
 
+// out = scale * table[id] (scale 1: the table's rows as they are)
+LSB_API int lsb_embedding_scaled(void* out_f32, void* out_bf16, const void* table, const void* ids, int rows, int hidden,
+                                 int vocab_lo, int vocab_hi, float scale, void* stream) {
+    launch_pdl((embedding_kernel), rows, 256, 0, (cudaStream_t)stream, (float*)out_f32, (bf16*)out_bf16, (const bf16*)table, (const int*)ids,
+               hidden, vocab_lo, vocab_hi, scale);
+    LSB_CHECK_LAUNCH();
+}
 LSB_API int lsb_embedding(void* out_f32, void* out_bf16, const void* table, const void* ids, int rows, int hidden,
                           int vocab_lo, int vocab_hi, void* stream) {
-    launch_pdl((embedding_kernel), rows, 256, 0, (cudaStream_t)stream, (float*)out_f32, (bf16*)out_bf16, (const bf16*)table, (const int*)ids,
-                                                           hidden, vocab_lo, vocab_hi);
-    LSB_CHECK_LAUNCH();
+    return lsb_embedding_scaled(out_f32, out_bf16, table, ids, rows, hidden, vocab_lo, vocab_hi, 1.f, stream);
 }
 
 // part: scratch u64 [rows, 64].  out_val may be null.  `base` is added to the index (vocab shard offset).

@@ -1,13 +1,18 @@
-"""Models described layer by layer (``ModelConfig.blocks``) on the device: every layer is a mixer (grouped-query attention or a gated delta
-rule) and an optional routed feed-forward, each with its own sizes, around a post-norm fp32 residual stream
+"""Models described layer by layer (``ModelConfig.blocks``) on the device: every layer is a mixer (grouped-query attention, latent attention or
+a gated delta rule) and an optional feed-forward (a dense gated unit or routed experts), each with its own sizes, around an fp32 residual stream.
+The norms stand on every sublayer's output (``norm_place`` "post") or on both its sides ("sandwich"; n_in is the identity for "post"):
 
-    x <- x + norm1(mixer(x)),    x <- x + norm2(ffn(x)),    logits = head(norm(x)) * logit_scale.
+    x <- x + n_out(mixer(n_in(x))),    x <- x + n_out(ffn(n_in(x))),    logits = head(norm(x)) * logit_scale,
+
+and a layer may end with an update from its slice e of a per-token table: x <- x + rms(W_p (gelu(W_g x) * e)).
 
 Same engine, caches and step protocol as :class:`DeviceModel`: attention layers keep a paged cache (one row of all heads' keys and values per
-token), delta-rule layers an fp32 state and convolution history per sequence slot.  Steps are any mixture of prompt portions and single tokens.
+token; latent layers one row for all heads, which later layers may read instead of keeping their own), delta-rule layers an fp32 state and
+convolution history per sequence slot.  Steps are any mixture of prompt portions and single tokens.
 
 Two precisions.  ``bfloat16``: weights, activations and the cache in bf16, products accumulated in fp32; the residual stream, norms, routing,
-attention scores and weights and the whole recurrence in fp32.  ``float32``: everything in fp32 (FMA units, no reduced-precision products).
+attention scores and weights, rotations and the whole recurrence in fp32.  ``float32``: everything in fp32 (FMA units, no reduced-precision
+products).
 
 Sizes are padded where kernels want it: the residual width to a multiple of 8, projection blocks to multiples of 8 rows, head widths and
 expert widths to the kernels' tiles; padding holds zeros and never reaches a result.
@@ -25,23 +30,38 @@ from .device_model import ExpertArena, ModelBase, MoeBuffers, QLinear, StepBuffe
 
 FEW_ROWS = 8            # rows per sequence up to which a delta-rule layer runs as one kernel
 LONG_ROWS = 64          # rows of a sequence from which its recurrence runs chunk-parallel
+NORM_KIND = {"rms": 0, "layer": 1, "tanh": 2}        # as the kernels number them; 3: none
+NO_NORM = (3, None, None, None)
 
 
 def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = None) -> Dict[str, tuple]:
     """Canonical tensor names and shapes.  ``ranks``: {layer: (decay rank, gate rank)} of delta-rule layers (default: the key head width)."""
     H, out = cfg.hidden, {}
-    norm = lambda p: out.update({p + ".weight": (H,)} | ({p + ".bias": (H,)} if cfg.norm_kind == "layer" else {}))
+    extra = {"rms": (), "layer": ("bias",), "tanh": ("bias", "alpha")}[cfg.norm_kind]
+    norm = lambda p: out.update({p + ".weight": (H,)} | {f"{p}.{k}": () if k == "alpha" else (H,) for k in extra})
     out["embed.weight"] = out["head.weight"] = (cfg.vocab, H)
+    if cfg.side_dim:
+        out["side_embed.weight"] = (cfg.vocab, cfg.n_layers * cfg.side_dim)
     norm("final_norm")
     for i, b in enumerate(cfg.blocks):
         p = f"layers.{i}."
         norm(p + "mix_norm")
+        if cfg.norm_place == "sandwich":
+            norm(p + "mix_post_norm")
         if b.recurrent:
             k, kw, vw = p + "kda.", b.kv_heads * b.dim, b.heads * b.vdim
             ra, rg = (ranks or {}).get(i, (b.dim, b.dim))
             out.update({k + "q": (kw, H), k + "k": (kw, H), k + "v": (vw, H), k + "beta": (b.heads, H), k + "f_a": (ra, H), k + "g_a": (rg, H),
                         k + "f_b": (b.heads * b.dim, ra), k + "g_b": (vw, rg), k + "conv_q": (kw, b.conv), k + "conv_k": (kw, b.conv), k + "conv_v": (vw, b.conv),
                         k + "a_log": (b.heads,), k + "dt_bias": (b.heads * b.dim,), k + "o_norm": (b.vdim,), k + "o": (H, vw)})
+        elif b.latent:
+            a = p + "attn."
+            out.update({a + "q": (b.heads * (b.dim + b.rot_dim), H), a + "k_b": (b.heads * b.dim, b.kv_rank), a + "v_b": (b.heads * b.vdim, b.kv_rank),
+                        a + "o": (H, b.heads * b.vdim)})
+            if b.kv_from < 0:
+                out.update({a + "kv_a": (b.kv_rank + b.rot_dim, H), a + "kv_a_norm": (b.kv_rank,)})
+            if b.head_gate:
+                out[a + "g"] = (b.heads, H)
         else:
             a, qw, kw, vw = p + "attn.", b.heads * b.dim, b.kv_heads * b.dim, b.kv_heads * b.vdim
             out.update({a + "q": (qw, H), a + "k": (kw, H), a + "v": (vw, H), a + "o": (H, b.heads * b.vdim)})
@@ -51,12 +71,25 @@ def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = No
                 out[a + "g"] = (b.heads * b.vdim, H)
             if b.v_mix:
                 out[a + "v_mix"] = ()
-        if b.experts:
+        if b.has_ff:
             norm(p + "ffn_norm")
+            if cfg.norm_place == "sandwich":
+                norm(p + "ffn_post_norm")
+        glu = lambda m, ff: out.update({m + "gate": (ff, H), m + "up": (ff, H), m + "down": (H, ff)})
+        if b.dense_ff:
+            glu(p + "mlp.", b.dense_ff)
+        if b.experts:
             m = p + "moe."
-            out[m + "router"], out[m + "router_bias"] = (b.experts + b.identity, H), (b.experts + b.identity,)
+            out[m + "router"] = (b.experts + b.identity, H)
+            if b.correction:
+                out[m + "router_bias"] = (b.experts + b.identity,)
             for e in range(b.experts):
-                out.update({m + f"experts.{e}.gate": (b.ff, H), m + f"experts.{e}.up": (b.ff, H), m + f"experts.{e}.down": (H, b.ff)})
+                glu(m + f"experts.{e}.", b.ff)
+            if b.shared_ff:
+                glu(m + "shared.0.", b.shared_ff)
+                out[m + "shared_gate"] = (1, H)
+        if cfg.side_dim:
+            out.update({p + "side.gate": (cfg.side_dim, H), p + "side.proj": (H, cfg.side_dim), p + "side.norm": (H,)})
     return out
 
 
@@ -76,8 +109,10 @@ def random_block_tensor(name: str, shape: tuple, gen: torch.Generator, device="c
         return t.uniform_(0.2, 0.6, generator=gen)
     if leaf in ("bias", "router_bias"):
         return t.normal_(0.0, 0.1, generator=gen)
-    if leaf == "weight":                                     # embedding, head
-        return t.normal_(0.0, 1.0 if name.startswith("embed") else 0.5 / shape[1] ** 0.5, generator=gen)
+    if leaf == "alpha":
+        return t.uniform_(0.4, 1.0, generator=gen)
+    if leaf == "weight":                                     # token tables, head
+        return t.normal_(0.0, 1.0 if "embed" in name else 0.5 / shape[1] ** 0.5, generator=gen)
     return t.normal_(0.0, 1.0 / shape[1] ** 0.5, generator=gen)
 
 
@@ -107,18 +142,31 @@ class BlockWorkspace(StepBuffers):
         self.xh = z(n_logit_rows, Hp, dtype=act)
         self.proj = z(R, m.max_proj)
         self.mix = z(R, m.max_mix, dtype=act)        # a mixer's output in front of its output projection
-        att = [b for b in m.cfg.blocks if not b.recurrent]
+        lat = [b for b in m.cfg.blocks if b.latent]
+        att = [b for b in m.cfg.blocks if not b.recurrent and not b.latent]
+        if lat:
+            self.q_lat = z(R * max(b.heads * m.latent_row(b) for b in lat), dtype=act)
+            self.q_nope = z(R * max(b.heads * _align(b.dim, 8) for b in lat), dtype=torch.bfloat16) if not m.f32 and R >= 8 else None
+            self.o_lat = z(R * max(b.heads * m.latent_pad(b.kv_rank) for b in lat), dtype=act)
+            self.lat_splits = {i: 1 if R > 64 else int(nat.call("lsb_latent_splits", R, b.heads, b.kv_rank, b.rot_dim, max_ctx, int(m.f32)))
+                               for i, b in enumerate(m.cfg.blocks) if b.latent}
+            ns = [(b.heads * self.lat_splits[i], m.latent_pad(b.kv_rank)) for i, b in enumerate(m.cfg.blocks) if b.latent and self.lat_splits[i] > 1]
+            self.lat_o_part = z(R * max((n * w for n, w in ns), default=1))
+            self.lat_ml_part = z(2 * R * max((n for n, _ in ns), default=1))
+        dense = max((_align(max(b.dense_ff, b.shared_ff), 8) for b in m.cfg.blocks), default=0)
+        self.glu = z(R * dense, dtype=act) if dense else None
+        self.side = z(R, _align(m.cfg.side_dim, 8), dtype=act) if m.cfg.side_dim else None
         if att:
             self.q = z(R * max(b.heads * m.head_pad(b.dim) for b in att), dtype=act)
             self.v_first = z(R, max([b.kv_heads * b.vdim for b in att if b.v_mix], default=1))
             # key splits of the few-row attention: about two blocks per SM, no split shorter than 64 visible keys
             self.splits = {}
             for i, b in enumerate(m.cfg.blocks):
-                if not b.recurrent:
+                if not b.recurrent and not b.latent:
                     seen = min(b.window or max_ctx, max_ctx)
                     blocks = R * b.kv_heads * ((b.heads // b.kv_heads + 15) // 16)
                     self.splits[i] = 1 if (m.f32 or R > 64) else max(1, min(32, 296 // blocks, (seen + 63) // 64))
-            ns = [(b.heads * self.splits[i], m.head_pad(b.vdim)) for i, b in enumerate(m.cfg.blocks) if not b.recurrent and self.splits[i] > 1]
+            ns = [(b.heads * self.splits[i], m.head_pad(b.vdim)) for i, b in enumerate(m.cfg.blocks) if self.splits.get(i, 1) > 1]
             self.o_part = z(R * max((n * w for n, w in ns), default=1))
             self.ml_part = z(2 * R * max((n for n, _ in ns), default=1))
         self.moe: Dict[tuple, MoeBuffers] = {}
@@ -165,13 +213,15 @@ class BlockModel(ModelBase):
         self.expert_shard = "ep"
         self.Hp = _align(cfg.hidden, 8)
         self.max_mix = 8
-        mixing = [i for i, b in enumerate(cfg.blocks) if b.v_mix and not b.recurrent]
+        mixing = [i for i, b in enumerate(cfg.blocks) if b.v_mix and b.kind == "attention"]
         self.v_first_layer = mixing[0] if mixing else -1
         if len({cfg.blocks[i].kv_heads * cfg.blocks[i].vdim for i in mixing}) > 1:
             raise ValueError("layers that mix values must have the same number of value channels")
         for i, b in enumerate(cfg.blocks):
             if b.heads % max(b.kv_heads, 1) or min(b.heads, b.kv_heads, b.dim, b.vdim) < 1:
                 raise ValueError(f"layer {i}: {b.heads} heads over {b.kv_heads} groups of widths {b.dim} / {b.vdim}")
+            if b.latent and (b.kv_rank < 1 or b.rot_dim < 2 or b.rot_dim % 2):
+                raise ValueError(f"layer {i}: latent rows of {b.kv_rank} + {b.rot_dim} channels")
             if b.recurrent and b.dim > 256:
                 raise ValueError(f"layer {i}: key heads of up to 256 channels, not {b.dim}")
             if b.experts and (b.top > min(32, b.experts + b.identity) or (b.experts + b.identity) % b.groups or b.groups > 64):
@@ -180,6 +230,14 @@ class BlockModel(ModelBase):
     @staticmethod
     def head_pad(d: int) -> int:
         return int(nat.call("lsb_attn_head_pad", d))
+
+    @staticmethod
+    def latent_pad(d: int) -> int:
+        return _align(d, 16)
+
+    def latent_row(self, b: BlockSpec) -> int:
+        """Elements of a token's cached row (and of a head's query) in a latent layer."""
+        return self.latent_pad(b.kv_rank) + self.latent_pad(b.rot_dim)
 
     def moe_key(self, i: int) -> tuple:
         b = self.cfg.blocks[i]
@@ -213,9 +271,20 @@ class BlockModel(ModelBase):
         m = cls(cfg, device, kv_fmt, page, tp_rank, tp_size, dtype)
         H, Hp, dev = cfg.hidden, m.Hp, m.device
 
+        kind, sandwich = NORM_KIND[cfg.norm_kind], cfg.norm_place == "sandwich"
+
         def norm(p, scale=1.0):
-            b = p + ".bias"
-            return m._vec(w[p + ".weight"]) * scale, (m._vec(w[b]) * scale if b in w else None)
+            """(kind, weight, bias, alpha) of a norm of the residual stream"""
+            b, al = p + ".bias", p + ".alpha"
+            return kind, m._vec(w[p + ".weight"]) * scale, (m._vec(w[b]) * scale if b in w else None), (m._vec(w[al]) if al in w else None)
+
+        def stacked(parts, cols=Hp):
+            """The parts as one projection and the row at which each starts."""
+            offs, o = [], 0
+            for t in parts:
+                offs.append(o)
+                o += _align(t.shape[0], 8)
+            return m._mat(*parts, cols=cols), offs
 
         e = torch.zeros(cfg.vocab, Hp, dtype=torch.bfloat16, device=dev)
         e[:, :H] = w["embed.weight"].to(dev)
@@ -223,21 +292,19 @@ class BlockModel(ModelBase):
         hw = w["head.weight"].to(dev)
         m.head = m._mat(hw, cols=Hp)
         m.head.N = cfg.vocab                                   # padding rows of the matrix are never computed
-        m.final_norm, m.final_bias = norm("final_norm", cfg.logit_scale)      # the scale of the logits rides on the last norm
+        m.final_norm = norm("final_norm", cfg.logit_scale)     # the scale of the logits rides on the last norm
+        if cfg.side_dim:
+            m.side_embed = w["side_embed.weight"].to(dev).to(torch.bfloat16).contiguous()
         for i, b in enumerate(cfg.blocks):
             p = f"layers.{i}."
-            L: dict = {"norm1": norm(p + "mix_norm")}
+            L: dict = {"mix_in": norm(p + "mix_norm"), "mix_out": norm(p + "mix_post_norm")} if sandwich else {"mix_in": NO_NORM, "mix_out": norm(p + "mix_norm")}
             if b.recurrent:
                 k = p + "kda."
                 fb, gb = w[k + "f_b"].to(dev), w[k + "g_b"].to(dev)
                 ra, rg = _align(fb.shape[1], 8), _align(gb.shape[1], 8)
                 kw, vw = b.kv_heads * b.dim, b.heads * b.vdim
                 parts = [w[k + n].to(dev) for n in ("q", "k", "v", "beta", "f_a", "g_a")]
-                L["in"] = m._mat(*parts, cols=Hp)
-                offs, o = [], 0
-                for t in parts:
-                    offs.append(o)
-                    o += _align(t.shape[0], 8)
+                L["in"], offs = stacked(parts)
                 L["meta"] = _Meta(offs=offs, ra=ra, rg=rg)
                 pad = lambda t, n: torch.nn.functional.pad(t.float(), (0, n - t.shape[1])).to(m.act_dtype).contiguous()
                 L["w_a"], L["w_g"] = pad(fb, ra), pad(gb, rg)
@@ -251,15 +318,26 @@ class BlockModel(ModelBase):
                     L[n] = t
                 L["a_exp"], L["dt_bias"], L["o_norm"] = torch.exp(m._vec(w[k + "a_log"])), m._vec(w[k + "dt_bias"]), m._vec(w[k + "o_norm"])
                 L["out"] = m._mat(w[k + "o"].to(dev), cols=_align(vw, 8))
-                L["out"].N = Hp
+            elif b.latent:
+                a, own = p + "attn.", b.kv_from < 0
+                names = ["q"] + (["kv_a"] if own else []) + (["g"] if b.head_gate else [])
+                L["in"], offs = stacked([w[a + n].to(dev) for n in names])
+                at = dict(zip(names, offs))
+                L["meta"] = _Meta(offs=[at["q"], at.get("kv_a", -1), at.get("g", -1)])
+                dnp, dlp = _align(b.dim, 8), m.latent_pad(b.kv_rank)
+                uk, uv = w[a + "k_b"].to(dev).view(b.heads, b.dim, b.kv_rank), w[a + "v_b"].to(dev).view(b.heads, b.vdim, b.kv_rank)
+                L["w_uk"] = torch.zeros(b.heads, dlp, dnp, dtype=m.act_dtype, device=dev)
+                L["w_uk"][:, : b.kv_rank, : b.dim] = uk.transpose(1, 2)
+                L["w_uv"] = torch.zeros(b.heads, b.vdim, dlp, dtype=m.act_dtype, device=dev)
+                L["w_uv"][:, :, : b.kv_rank] = uv
+                if own:
+                    L["kv_norm"] = m._vec(w[a + "kv_a_norm"])
+                L["inv_freq"] = torch.tensor([b.rot_base ** (-2.0 * j / b.rot_dim) for j in range(b.rot_dim // 2)], dtype=torch.float64, device=dev)
+                L["out"] = m._mat(w[a + "o"].to(dev), cols=_align(b.heads * b.vdim, 8))
             else:
                 a = p + "attn."
                 parts = [w[a + n].to(dev) for n in ("q", "k", "v")] + ([w[a + "g"].to(dev)] if b.out_gate else [])
-                L["in"] = m._mat(*parts, cols=Hp)
-                offs, o = [], 0
-                for t in parts:
-                    offs.append(o)
-                    o += _align(t.shape[0], 8)
+                L["in"], offs = stacked(parts)
                 L["meta"] = _Meta(offs=offs + ([] if b.out_gate else [-1]))
                 if b.qk_norm:
                     L["q_norm"], L["k_norm"] = m._vec(w[a + "q_norm"]), m._vec(w[a + "k_norm"])
@@ -268,14 +346,27 @@ class BlockModel(ModelBase):
                 if b.v_mix:
                     L["v_mix"] = m._vec(w[a + "v_mix"])
                 L["out"] = m._mat(w[a + "o"].to(dev), cols=_align(b.heads * b.vdim, 8))
+            L["out"].N = Hp
             m.max_proj = max(m.max_proj, L["in"].N)
             m.max_mix = max(m.max_mix, L["out"].K)
+            if b.has_ff:
+                L["ff_in"], L["ff_out"] = (norm(p + "ffn_norm"), norm(p + "ffn_post_norm")) if sandwich else (NO_NORM, norm(p + "ffn_norm"))
+            if b.dense_ff:
+                L["ff"], L["ff_offs"] = stacked([w[p + f"mlp.{n}"].to(dev) for n in ("gate", "up")])
+                L["ff_down"] = m._mat(w[p + "mlp.down"].to(dev))
+                L["ff_down"].N = Hp
+                m.max_proj = max(m.max_proj, L["ff"].N)
             if b.experts:
                 mo = p + "moe."
-                L["norm2"] = norm(p + "ffn_norm")
-                L["router"] = m._mat(w[mo + "router"].to(dev), cols=Hp)        # values of the file's type: fp32-accumulated products are exact in them
-                L["router"].N = b.experts + b.identity
-                L["router_bias"] = m._vec(w[mo + "router_bias"]) if (mo + "router_bias") in w else None
+                # the router and - where there is one - the shared expert's gate, up and output-gate rows are one product (values of the file's
+                # type: fp32-accumulated products are exact in them)
+                parts = [w[mo + "router"].to(dev)] + ([w[mo + n].to(dev) for n in ("shared.0.gate", "shared.0.up", "shared_gate")] if b.shared_ff else [])
+                L["router"], L["ff_offs"] = stacked(parts)
+                L["router_bias"] = m._vec(w[mo + "router_bias"]) if b.correction and (mo + "router_bias") in w else None
+                if b.shared_ff:
+                    L["ff_down"] = m._mat(w[mo + "shared.0.down"].to(dev))
+                    L["ff_down"].N = Hp
+                m.max_proj = max(m.max_proj, L["router"].N)
                 # expert width padded to the tensor-core tile where the residual width allows that path
                 F = _align(b.ff, 128) if Hp % 128 == 0 else _align(b.ff, 8)
                 arena = ExpertArena(expert_layout(m.w_fmt, Hp, F), b.experts, b.experts, dev)
@@ -285,6 +376,12 @@ class BlockModel(ModelBase):
                     arena.write_expert(x, QLinear(m.w_fmt, F, Hp, g), QLinear(m.w_fmt, F, Hp, u), QLinear(m.w_fmt, Hp, F, d))
                     arena.slot_of[x] = x
                 L["arena"] = arena
+            if cfg.side_dim:
+                L["side_gate"] = m._mat(w[p + "side.gate"].to(dev), cols=Hp)
+                L["side_proj"] = m._mat(w[p + "side.proj"].to(dev))
+                L["side_proj"].N = Hp
+                L["side_norm"] = (NORM_KIND["rms"], m._vec(w[p + "side.norm"]), None, None)
+                m.max_proj = max(m.max_proj, L["side_gate"].N)
             m.layers.append(L)
         m.max_proj, m.max_mix = _align(m.max_proj, 8), _align(m.max_mix, 8)
         return m
@@ -310,11 +407,15 @@ class BlockModel(ModelBase):
             if b.recurrent:
                 self.kda_state[i] = z(n_slots, b.heads, b.vdim, int(nat.call("lsb_delta_key_pad", b.dim)))
                 self.kda_conv[i] = z(n_slots, b.heads, 2 * b.dim + b.vdim, b.conv - 1)
+            elif b.latent:
+                if b.kv_from < 0:
+                    self.kv_cache[i] = z(num_pages, self.page, self.latent_row(b), dtype=self.act_dtype)
             else:
                 self.kv_cache[i] = z(num_pages, self.page, b.kv_heads * (self.head_pad(b.dim) + self.head_pad(b.vdim)), dtype=self.act_dtype)
 
     def cache_bytes_per_token(self) -> int:
-        return sum(b.kv_heads * (self.head_pad(b.dim) + self.head_pad(b.vdim)) * (4 if self.f32 else 2) for b in self.cfg.blocks if not b.recurrent)
+        width = lambda b: ((self.latent_row(b) if b.kv_from < 0 else 0) if b.latent else b.kv_heads * (self.head_pad(b.dim) + self.head_pad(b.vdim)))
+        return sum(width(b) * (4 if self.f32 else 2) for b in self.cfg.blocks if not b.recurrent)
 
     # ------------------------------------------------------------------ forward
     def _resid_rows(self, ws, R: int, H: int) -> torch.Tensor:
@@ -331,6 +432,18 @@ class BlockModel(ModelBase):
         nat.call("lsb_attn", ws.q, self.kv_cache[i], self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
                  max(ws.seq_rows), ws.proj, ldp, og, ws.mix, L["out"].K, ws.o_part, ws.ml_part, ws.splits[i], R, b.heads, b.kv_heads, b.dim, b.vdim, dkp, dvp,
                  b.window, b.scale, L.get("slope"), int(self.f32))
+
+    def _latent(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
+        oq, okv, og = L["meta"].offs
+        cache = self.kv_cache[i if b.kv_from < 0 else b.kv_from]
+        L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
+        err = TcScratch.get(self.device).err
+        nat.call("lsb_latent_query", ws.proj, self.max_proj, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], ws.q_lat, ws.q_nope, cache,
+                 self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, R, b.heads, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank,
+                 int(self.f32), err)
+        nat.call("lsb_latent_attn", ws.q_lat, cache, self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
+                 max(ws.seq_rows), ws.proj, self.max_proj, og, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], L["w_uv"], ws.mix, L["out"].K, R,
+                 b.heads, b.kv_rank, b.rot_dim, b.vdim, b.scale, int(self.f32), err)
 
     def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
         mt = L["meta"]
@@ -350,42 +463,76 @@ class BlockModel(ModelBase):
                  b.dim ** -0.5, b.decay_bound, self.cfg.rms_eps, int(self.f32), int(few), scratch, len(rows) - len(long_), len(long_), chunks, LONG_ROWS,
                  chunk_ws, TcScratch.get(self.device).err)
 
+    def _glu(self, L: dict, ws: BlockWorkspace, R: int, ff: int, offs, limit=0.0, alpha=1.0, shift=0.0):
+        """Gated unit over columns of the projection in ``ws.proj`` and its down product into ``ws.sub``; ``offs``: gate, up, output gate (-1: none)."""
+        K = L["ff_down"].K
+        nat.call("lsb_glu", ws.glu, K, ws.proj, self.max_proj, *offs, R, ff, limit, alpha, shift, int(self.f32))
+        L["ff_down"](ws.sub, ws.glu, R, ldo=self.Hp)
+
     def _moe(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int) -> MoeBuffers:
-        mb = ws.moe[self.moe_key(i)]
+        mb, cfg = ws.moe[self.moe_key(i)], self.cfg
         n = b.experts + b.identity
-        L["router"](mb.logits_r, ws.x, R, ldo=n)
-        nat.call("lsb_router_topk_grouped", mb.logits_r, L["router_bias"], mb.ids, mb.wts, R, n, b.top, b.groups, b.keep, 1, int(self.cfg.norm_topk_prob),
-                 self.cfg.routed_scale, 0, n, 1)
+        L["router"](ws.proj, ws.x, R, ldo=self.max_proj)
+        nat.call("lsb_router_topk_grouped", ws.proj, L["router_bias"], mb.ids, mb.wts, R, n, b.top, b.groups, b.keep, {"sigmoid": 0, "softmax": 1}[b.scoring],
+                 int(cfg.norm_topk_prob), cfg.routed_scale, 0, self.max_proj, 1)
+        if b.shared_ff:
+            self._glu(L, ws, R, b.shared_ff, L["ff_offs"][1:], b.shared_limit, b.act_alpha, b.act_shift)
         self.moe_prepare(L["arena"], mb, ws.x, R, b.experts)
-        self.moe_experts(L["arena"], mb, ws.x, R, b.experts, self.cfg.swiglu_limit, mb.miss)
+        plain = b.act_alpha == 1.0 and b.act_shift == 0.0 and not b.scale_input
+        act = None if plain else (b.act_alpha, b.act_shift, mb.wts if b.scale_input else None)
+        self.moe_experts(L["arena"], mb, ws.x, R, b.experts, b.limit, mb.miss, act)
         return mb
+
+    def _update(self, ws: BlockWorkspace, R: int, post: tuple, pre: tuple, sub=None, mb: Optional[MoeBuffers] = None, b: Optional[BlockSpec] = None,
+                L: Optional[dict] = None):
+        """resid += post(sub + expert sum), x = pre(resid)."""
+        Hp, y = self.Hp, (None, None, None, None, 0, 0, 0)
+        if mb is not None:
+            y = (mb.y, None if b.scale_input else mb.wts, mb.ids, L["arena"].slot_of, b.top, b.experts, L["arena"].ef.H)
+        nat.call("lsb_resid_update", ws.x, Hp, ws.resid, Hp, sub, Hp, *post, *pre, R, self.cfg.hidden, self.cfg.rms_eps, *y, int(self.f32))
+
+    def _side(self, i: int, L: dict, ws: BlockWorkspace, R: int):
+        """The layer's per-token input: gate product on the stream, table slice, projection into ``ws.sub``."""
+        d, K = self.cfg.side_dim, L["side_proj"].K
+        L["side_gate"](ws.proj, ws.x, R, ldo=self.max_proj)
+        nat.call("lsb_side_gate", ws.side, K, ws.proj, self.max_proj, self.side_embed, self.side_embed.shape[1], i * d, d, ws.tok, self.cfg.vocab, R, int(self.f32))
+        L["side_proj"](ws.sub, ws.side, R, ldo=self.Hp)
 
     def set_layer_skip(self, skip=(), probe: bool = False):
         if probe:
             raise NotImplementedError("layer-input similarity probing is built for the MLA family")
-        super().set_layer_skip([l for l in skip if int(l) != self.v_first_layer], False)
+        keep = {self.v_first_layer} | {b.kv_from for b in self.cfg.blocks}          # layers whose values or cached rows others read
+        super().set_layer_skip([l for l in skip if int(l) not in keep], False)
 
     def forward(self, ws: BlockWorkspace, R: int, nseq: int, logit_row0: int, n_logit_rows: int):
         """One step over the first ``R`` staged rows; logits of rows [logit_row0, logit_row0 + n_logit_rows)."""
         cfg, H, Hp, f32 = self.cfg, self.cfg.hidden, self.Hp, int(self.f32)
-        layer = int(cfg.norm_kind == "layer")
-        nat.call("lsb_embedding", ws.resid, None if f32 else ws.x, self.embed, ws.tok, R, Hp, 0, cfg.vocab)
-        if f32:
-            ws.x[:R].copy_(ws.resid[:R])
-        for i, (b, L) in enumerate(zip(cfg.blocks, self.layers)):
+        run = [i for i in range(cfg.n_layers) if i not in self.skip_layers]
+        enters = dict(zip([-1] + run, [self.layers[i]["mix_in"] for i in run] + [NO_NORM]))       # norm in front of the layer that follows
+        plain = enters[-1] is NO_NORM
+        nat.call("lsb_embedding_scaled", ws.resid, ws.x if plain and not f32 else None, self.embed, ws.tok, R, Hp, 0, cfg.vocab, cfg.embed_scale)
+        if not plain or f32:
+            self._update(ws, R, NO_NORM, enters[-1])
+        for i in range(cfg.n_layers):
             if self.aux_capture is not None:
                 self._capture_aux(i, ws, R)
-            if i in self.skip_layers:
+            if i not in enters:
                 continue
-            (self._delta if b.recurrent else self._attention)(i, b, L, ws, R, nseq)
+            b, L = cfg.blocks[i], self.layers[i]
+            (self._delta if b.recurrent else (self._latent if b.latent else self._attention))(i, b, L, ws, R, nseq)
             L["out"](ws.sub, ws.mix, R, ldo=Hp)
-            nw, nb = L["norm1"]
-            nat.call("lsb_post_norm", ws.x, Hp, ws.resid, Hp, ws.sub, Hp, nw, nb, R, H, cfg.rms_eps, layer, None, None, None, None, 0, 0, 0, f32)
+            last = NO_NORM if cfg.side_dim else enters[i]
+            self._update(ws, R, L["mix_out"], L["ff_in"] if b.has_ff else last, ws.sub)
             if b.experts:
                 mb = self._moe(i, b, L, ws, R)
-                nw, nb = L["norm2"]
-                nat.call("lsb_post_norm", ws.x, Hp, ws.resid, Hp, None, 0, nw, nb, R, H, cfg.rms_eps, layer, mb.y, mb.wts, mb.ids, L["arena"].slot_of, b.top,
-                         b.experts, L["arena"].ef.H, f32)
+                self._update(ws, R, L["ff_out"], last, ws.sub if b.shared_ff else None, mb, b, L)
+            elif b.dense_ff:
+                L["ff"](ws.proj, ws.x, R, ldo=self.max_proj)
+                self._glu(L, ws, R, b.dense_ff, (*L["ff_offs"], -1))
+                self._update(ws, R, L["ff_out"], last, ws.sub)
+            if cfg.side_dim:
+                self._side(i, L, ws, R)
+                self._update(ws, R, L["side_norm"], enters[i], ws.sub)
             if self.drift is not None:
                 self.drift[f"layer{i:03d}.resid"] = ws.resid[:R, :H].float().cpu()
         if self.aux_capture is not None:
@@ -395,8 +542,8 @@ class BlockModel(ModelBase):
 
     def emit_logits(self, ws: BlockWorkspace, row0: int, n: int, rows: Optional[torch.Tensor] = None):
         """Logits of step rows [row0, row0 + n), or of the ``n`` rows listed in ``rows`` (int32, device), after :meth:`forward`."""
-        nat.call("lsb_norm_rows", ws.xh, self.Hp, ws.resid, self.Hp, rows, row0, self.final_norm, self.final_bias, n, self.cfg.hidden, self.cfg.rms_eps,
-                 int(self.cfg.norm_kind == "layer"), int(self.f32))
+        kind, nw, nb, alpha = self.final_norm
+        nat.call("lsb_norm_rows", ws.xh, self.Hp, ws.resid, self.Hp, rows, row0, nw, nb, alpha, n, self.cfg.hidden, self.cfg.rms_eps, kind, int(self.f32))
         self.head(ws.logits, ws.xh, n)
 
 

@@ -74,6 +74,17 @@ _GAZUTAR_LAYER = {
     "moe.router": "mlp.router", "moe.router_bias": "mlp.correction",
 }
 _GAZUTAR_TOP = {"embed.weight": "embed", "head.weight": "head", "final_norm.weight": "final.norm", "final_norm.bias": "final.norm.b"}
+# canonical suffix -> tensor name behind "l<N>." (Rubasun)
+_RUBASUN_LAYER = {f"{c}.{k}": f + s for c, f in (("mix_norm", "norm1"), ("mix_post_norm", "norm1b"), ("ffn_norm", "norm2"), ("ffn_post_norm", "norm2b"))
+                  for k, s in (("weight", ""), ("bias", ".b"), ("alpha", ".alpha"))} | {
+    "attn.q": "mix.q", "attn.kv_a": "mix.dkv", "attn.kv_a_norm": "mix.dkv.norm", "attn.k_b": "mix.uk", "attn.v_b": "mix.uv", "attn.g": "mix.g", "attn.o": "mix.o",
+    "mlp.gate": "mlp.gate", "mlp.up": "mlp.up", "mlp.down": "mlp.down", "moe.router": "mlp.router", "moe.shared_gate": "mlp.shared.sg",
+    "moe.shared.0.gate": "mlp.shared.gate", "moe.shared.0.up": "mlp.shared.up", "moe.shared.0.down": "mlp.shared.down",
+    "side.gate": "side.gate", "side.proj": "side.proj", "side.norm": "side.norm",
+}
+_RUBASUN_TOP = _GAZUTAR_TOP | {"final_norm.alpha": "final.norm.alpha", "side_embed.weight": "side.embed"}
+# checkpoints with tensor names of their own: architecture -> (layer names, names outside the layers)
+_NATIVE_NAMES = {"gazutar": (_GAZUTAR_LAYER, _GAZUTAR_TOP), "rubasun": (_RUBASUN_LAYER, _RUBASUN_TOP)}
 _LAYER_RE = re.compile(r"^layers\.(\d+)\.(.+)$")
 _EXPERT_RE = re.compile(r"^moe\.(experts|shared)\.(\d+)\.(gate|up|down)$")
 
@@ -210,15 +221,16 @@ class LazyCheckpoint(Mapping):
 
     # ---- resolution ----
     def _resolve(self, key: str) -> Optional[Callable[[], torch.Tensor]]:
-        return {"hf": self._resolve_hf, "gguf": self._resolve_gguf, "gazutar": self._resolve_gazutar}[self.kind](key)
+        return {"hf": self._resolve_hf, "gguf": self._resolve_gguf, "native": self._resolve_native}[self.kind](key)
 
-    def _resolve_gazutar(self, key: str):
+    def _resolve_native(self, key: str):
+        layer, top = _NATIVE_NAMES[self.cfg.architecture]
         m = _LAYER_RE.match(key)
         if m is None:
-            name = _GAZUTAR_TOP.get(key)
+            name = top.get(key)
         else:
             e = _EXPERT_RE.match(m.group(2))
-            rest = f"mlp.e{e.group(2)}.{e.group(3)}" if e and e.group(1) == "experts" else _GAZUTAR_LAYER.get(m.group(2))
+            rest = f"mlp.e{e.group(2)}.{e.group(3)}" if e and e.group(1) == "experts" else layer.get(m.group(2))
             name = f"l{m.group(1)}.{rest}" if rest else None
         return (lambda: self.src.load(name)) if name and self.src.has(name) else None
 
@@ -493,8 +505,8 @@ def open_checkpoint(path: str, cfg: Optional[ModelConfig] = None) -> tuple[Model
     if cfg is None:
         cfg = from_hf_config(os.path.join(d, "config.json"))
     src = SafetensorsSource(d)
-    if cfg.architecture == "gazutar":
-        return cfg, LazyCheckpoint(cfg, src, "gazutar")
+    if cfg.architecture in _NATIVE_NAMES:
+        return cfg, LazyCheckpoint(cfg, src, "native")
     skip = QuantSkipList.from_model_dir(d)
     if skip is not None and skip.quant_method in ("fp8", ""):
         dts, shp = {}, {}

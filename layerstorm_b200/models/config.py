@@ -16,14 +16,14 @@ import math
 from dataclasses import dataclass, field, asdict
 from typing import List, Optional
 
-ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar")
+ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun")
 
 
 @dataclass
 class BlockSpec:
-    """One layer of a model that is described layer by layer (``ModelConfig.blocks``): a mixer and an optional mixture-of-experts
-    feed-forward, each with sizes of its own."""
-    kind: str = "attention"           # "attention" | "channel_delta" (gated delta rule with a decay per key channel)
+    """One layer of a model that is described layer by layer (``ModelConfig.blocks``): a mixer and an optional feed-forward, dense or a
+    mixture of experts, each with sizes of its own."""
+    kind: str = "attention"           # "attention" | "latent_attention" | "channel_delta" (gated delta rule with a decay per key channel)
     heads: int = 0                    # query heads (attention) / value heads (delta)
     kv_heads: int = 0                 # key-value heads (attention) / query-key heads (delta); divides `heads`
     dim: int = 0                      # query / key head width
@@ -35,21 +35,46 @@ class BlockSpec:
     alibi: bool = False               # linear distance bias, slope 2^(-8 (h + 1) / heads)
     out_gate: bool = False            # heads times sigmoid(W_g h) in front of the output projection
     v_mix: bool = False               # values mixed with those of the first such layer
+    # latent attention (one cached row of kv_rank + rot_dim per token for all heads)
+    kv_rank: int = 0
+    rot_dim: int = 0                  # rotated query / key channels per head, behind `dim` unrotated ones
+    rot_base: float = 10000.0
+    kv_from: int = -1                 # layer whose cached rows are attended over (-1: the layer's own)
+    head_gate: bool = False           # head h times sigmoid((W_g h)_h)
     # delta rule
     conv: int = 0                     # taps of the short causal convolutions
     decay: str = "softplus"           # log decay: "softplus" -exp(A) softplus(x) | "bounded" decay_bound * sigmoid(exp(A) x)
     decay_bound: float = -5.0
-    # feed-forward (experts 0: none)
+    # feed-forward (dense_ff 0 and experts 0: none)
+    dense_ff: int = 0                 # width of a dense gated unit
     experts: int = 0
     identity: int = 0                 # router outputs behind the experts whose "expert" is the input itself
     top: int = 0
     groups: int = 1
     keep: int = 1                     # groups a token may choose from
     ff: int = 0
+    # router: scores, selection correction; where a chosen expert's weight goes
+    scoring: str = "softmax"          # softmax | sigmoid
+    correction: bool = True
+    scale_input: bool = False         # the weight multiplies the expert's input instead of its output
+    # the experts' gated unit min(g, limit) sigmoid(act_alpha g) (clamp(u, -limit, limit) + act_shift); limit 0: no clamps
+    limit: float = 0.0
+    act_alpha: float = 1.0
+    act_shift: float = 0.0
+    shared_ff: int = 0                # an expert for every token (same unit, own limit) times sigmoid of one number per token
+    shared_limit: float = 0.0
 
     @property
     def recurrent(self) -> bool:
         return self.kind == "channel_delta"
+
+    @property
+    def latent(self) -> bool:
+        return self.kind == "latent_attention"
+
+    @property
+    def has_ff(self) -> bool:
+        return self.dense_ff > 0 or self.experts > 0
 
 
 @dataclass
@@ -116,8 +141,11 @@ class ModelConfig:
     eos_token_ids: List[int] = field(default_factory=list)
     # models described layer by layer (models/block_model.py); empty for the MLA family
     blocks: List[BlockSpec] = field(default_factory=list)
-    norm_kind: str = "rms"            # "rms" | "layer" (with bias): the norms of the residual stream
+    norm_kind: str = "rms"            # "rms" | "layer" (with bias) | "tanh" (dynamic tanh, element-wise): the norms of the residual stream
+    norm_place: str = "post"          # "post": on every sublayer's output | "sandwich": in front of every sublayer and on its output
     logit_scale: float = 1.0
+    embed_scale: float = 1.0
+    side_dim: int = 0                 # width of a layer's slice of the per-token side table (0: no such table)
 
     def __post_init__(self):
         self.blocks = [b if isinstance(b, BlockSpec) else BlockSpec(**b) for b in self.blocks]
@@ -128,6 +156,11 @@ class ModelConfig:
             self.layer_types = ["mla"] * self.n_layers
         assert len(self.layer_types) == self.n_layers
         assert self.architecture in ARCHITECTURES
+        for i, b in enumerate(self.blocks):
+            if b.kv_from >= 0:
+                src = self.blocks[b.kv_from] if b.kv_from < i else None
+                if src is None or not src.latent or src.kv_from >= 0 or (src.kv_rank, src.rot_dim, src.rot_base) != (b.kv_rank, b.rot_dim, b.rot_base):
+                    raise ValueError(f"layer {i}: layer {b.kv_from} has no latent rows of its kind to share")
 
     # ---- derived ----
     @property
@@ -295,7 +328,34 @@ def gazutar_flash() -> ModelConfig:
                     {"experts": 64, "identity": 8, "top": 8, "groups": {"count": 8, "keep": 4}}, 2048, every=4)
 
 
+def _rubasun(name, width, vocab, mixer, dense_ff, experts, top, ff, shared, limits, n_layers, share=2, side=0, scale=1.0) -> ModelConfig:
+    """A Rubasun shape: a dense first layer, then expert layers of which every ``share``-th makes latent rows that the ones behind it use."""
+    layers = []
+    for i in range(n_layers):
+        m, src = dict(mixer), 1 + (i - 1) // share * share if i else 0
+        if src != i:
+            m["kv_from"] = src
+        mlp = {"kind": "dense", "ff": dense_ff} if i == 0 else {"kind": "moe", "expert": {"ff": ff, "limit": limits[0]}, "router": {"experts": experts, "top": top},
+                                                               "shared": {"ff": shared, "limit": limits[1]}}
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+    return rubasun_config({"name": name, "width": width, "vocab": vocab, "layers": layers, "norm": {"eps": 1e-5}, "embedding": {"scale": scale}, "token_side": {"dim": side}})
+
+
+def tiny_rubasun() -> ModelConfig:
+    """A small Rubasun shape for tests and smoke runs."""
+    return _rubasun("tiny-rubasun", 192, 320, {"heads": 6, "dim": 40, "rot_dim": 16, "vdim": 24, "kv_rank": 80, "rot": {"base": 5000.0, "dims": 16}, "scale": 0.15}, 256,
+                    6, 2, 80, 72, (3.0, 2.0), 5, side=20, scale=2.0)
+
+
+def rubasun_flash() -> ModelConfig:
+    """A Rubasun shape with layers of a real model's size."""
+    return _rubasun("rubasun-flash", 4096, 154880, {"heads": 32, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "rot": {"base": 1e6, "dims": 64}, "scale": 192 ** -0.5},
+                    12288, 64, 8, 2048, 2048, (7.0, 7.0), 8, side=256)
+
+
 PRESETS = {
+    "tiny-rubasun": tiny_rubasun,
+    "rubasun-flash": rubasun_flash,
     "tiny-gazutar": tiny_gazutar,
     "gazutar-flash": gazutar_flash,
     "tiny-mla-moe": tiny_mla_moe,
@@ -345,8 +405,43 @@ def gazutar_config(c: dict) -> ModelConfig:
         kda_heads=max((b.heads for b in rec), default=0), kda_head_dim=max((b.dim for b in rec), default=0), max_position=int(c.get("max_position", 1 << 20)))
 
 
+def rubasun_config(c: dict) -> ModelConfig:
+    """Rubasun: dynamic-tanh norms around every sublayer; latent attention with rotary positions, a gate per head and cached rows that later layers
+    may share; dense or expert feed-forwards (sigmoid scores on the experts' inputs, clamped and shifted gated units, a gated shared expert); a
+    table of per-token inputs for every layer."""
+    blocks = []
+    for i, L in enumerate(c["layers"]):
+        if L["type"] != "latent_attention":
+            raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
+        m, src = L["mixer"], L["mixer"].get("kv_from")
+        rot = m.get("rot") or {}
+        if int(rot.get("dims", m["rot_dim"])) != m["rot_dim"]:
+            raise ValueError(f"layer {i}: {rot['dims']} rotary channels in a rotated part of {m['rot_dim']}")
+        b = BlockSpec(kind=L["type"], heads=m["heads"], kv_heads=1, dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]), kv_rank=m["kv_rank"], rot_dim=m["rot_dim"],
+                      rot_base=float(rot.get("base", 10000.0)), kv_from=-1 if src is None else int(src), head_gate=True)
+        mlp = L.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            b.dense_ff = int(mlp["ff"])
+        elif mlp and mlp["kind"] == "moe":
+            sh = mlp.get("shared") or {}
+            b.experts, b.top, b.ff, b.limit = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"]), float(mlp["expert"]["limit"])
+            b.scoring, b.correction, b.scale_input, b.act_alpha, b.act_shift = "sigmoid", False, True, 1.702, 1.0
+            b.shared_ff, b.shared_limit = int(sh.get("ff", 0)), float(sh.get("limit", 0.0))
+        elif mlp:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        blocks.append(b)
+    moe = [b for b in blocks if b.experts]
+    top = lambda key, of=blocks: max((getattr(b, key) for b in of), default=0)
+    return ModelConfig(
+        name=c.get("name", "Rubasun"), architecture="rubasun", hidden=c["width"], vocab=c["vocab"], rms_eps=float(c["norm"]["eps"]), norm_kind="tanh",
+        norm_place="sandwich", embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)), side_dim=int((c.get("token_side") or {}).get("dim", 0)),
+        blocks=blocks, n_heads=max(1, top("heads")), q_lora=0, kv_lora=top("kv_rank"), qk_nope=top("dim"), qk_rope=top("rot_dim"), v_head=top("vdim"),
+        rope_theta=blocks[0].rot_base if blocks else 10000.0, dense_inter=top("dense_ff"), first_k_dense=0, n_routed=top("experts", moe), top_k=top("top", moe),
+        n_shared=0, moe_inter=top("ff", moe), scoring="sigmoid", norm_topk_prob=False, max_position=int(c.get("max_position", 1 << 20)))
+
+
 # architectures whose config.json is described by its own keys ("architecture": name) rather than HuggingFace ones
-NATIVE_CONFIGS = {"gazutar": gazutar_config}
+NATIVE_CONFIGS = {"gazutar": gazutar_config, "rubasun": rubasun_config}
 
 
 def from_hf_config(path_or_dict) -> ModelConfig:

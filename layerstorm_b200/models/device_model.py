@@ -732,7 +732,7 @@ class ModelBase:
                 elif isinstance(v, torch.Tensor):
                     tot += v.numel() * v.element_size()
                 elif isinstance(v, tuple):
-                    tot += sum(t.numel() * t.element_size() for t in v if t is not None)
+                    tot += sum(t.numel() * t.element_size() for t in v if isinstance(t, torch.Tensor))
         return tot
 
     # ------------------------------------------------------------------ routed experts of a step
@@ -757,11 +757,14 @@ class ModelBase:
         elif mode == "groups":
             nat.call("lsb_moe_build_groups", ws.ids, R * S, E, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups, ws.counts)
 
-    def moe_experts(self, arena: "ExpertArena", ws, x, R: int, E: int, limit: float, miss):
-        """gate/up + SwiGLU and down projections of every pair whose expert is resident (``arena.slot_of[e] >= 0``)."""
+    def moe_experts(self, arena: "ExpertArena", ws, x, R: int, E: int, limit: float, miss, act=None):
+        """gate/up + gated unit and down projections of every pair whose expert is resident (``arena.slot_of[e] >= 0``).  ``act``: (sigmoid slope,
+        shift of the linear half, input scale per pair or None) of another unit than SwiGLU."""
         S = ws.S
         efp = ctypes.addressof(arena.ef)
         mode = self.moe_mode(arena, ws, R)
+        if act is not None and (mode == "pairs" or ws.bs_ok):
+            raise NotImplementedError("block-scaled and 4-bit pair experts are built for SwiGLU")
         if mode == "tc":
             P = R * S
             err = TcScratch.get(self.device).err
@@ -781,8 +784,12 @@ class ModelBase:
                          ws.bs_aq, ws.bs_asf, ws.bs_aa)
                 nat.call("lsb_moe_bs_ffn", 0, ws.bs_aq, ws.bs_asf, ws.bs_aa, *a, ws.y, ws.tc_bn, tiles, 0.0, None, err)
                 return
-            nat.call("lsb_moe_tc_ffn", 1, ws.tc_xs, ws.tc_xs.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
-                     ws.tc_cnt, ws.tc_sorted, ws.tc_act, ws.tc_bn, tiles, limit, miss, err, None)
+            up = (ws.tc_xs, ws.tc_xs.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, ws.tc_sorted, ws.tc_act,
+                  ws.tc_bn, tiles, limit)
+            if act is None:
+                nat.call("lsb_moe_tc_ffn", 1, *up, miss, err, None)
+            else:
+                nat.call("lsb_moe_tc_gateup_act", *up, *act, miss, err)
             nat.call("lsb_moe_tc_ffn", 0, ws.tc_act, ws.tc_act.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
                      ws.tc_cnt, ws.tc_sorted, ws.y, ws.tc_bn, tiles, 0.0, None, err, None)
         elif mode == "pairs":
@@ -796,8 +803,11 @@ class ModelBase:
             nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.ids, None, None, None, ws.y, R * S, run_dn)
         else:
             mg = min(ws.max_groups, min(R * S, (R * S + 3) // 4 + E))
-            nat.call("lsb_moe_gateup", x, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,
-                     ws.act, S, mg, limit, miss, 0)
+            up = (x, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups, ws.act, S, mg, limit)
+            if act is None:
+                nat.call("lsb_moe_gateup", *up, miss, 0)
+            else:
+                nat.call("lsb_moe_gateup_act", *up, *act, miss, 0)
             nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,
                      ws.y, mg, 0)
 

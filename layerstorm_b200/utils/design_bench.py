@@ -109,7 +109,7 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
         kv = b.kv_heads * (b.dim + b.vdim) * 2
         out["lsb_attn"] = ("bytes", batch * seen * kv + rows * b.heads * b.vdim * 6) if rows == batch else ("flops", 2 * rows * seen * b.heads * (b.dim + b.vdim))
         out["lsb_attn_prep"] = ("bytes", rows * ((b.heads + b.kv_heads) * b.dim + b.kv_heads * b.vdim) * 6)
-        out["lsb_post_norm"] = ("bytes", rows * H * (14 + TOP * 4) // 2 + rows * H * 7)
+        out["lsb_resid_update"] = ("bytes", rows * H * (14 + TOP * 4) // 2 + rows * H * 7)
     else:
         out["lsb_kda_forward"] = out["lsb_kda_forward_chunked"] = rec
         lat = cfg.kv_lora

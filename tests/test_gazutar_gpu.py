@@ -248,13 +248,14 @@ def test_post_norm_update_and_gathered_norm_rows(layer, bias, dim):
         resid, ds = torch.zeros(R, ld, device=DEV), torch.zeros(R, ld, device=DEV)
         resid[:, :dim], ds[:, :dim] = x.to(DEV), sub.to(DEV)
         act = torch.zeros(R, ld, dtype=F32 if f32 else B16, device=DEV)
-        nat.call("lsb_post_norm", act, ld, resid, ld, ds, ld, w.to(DEV), b.to(DEV) if bias else None, R, dim, eps, layer, None, None, None, None, 0, 0, 0, f32)
+        nat.call("lsb_resid_update", act, ld, resid, ld, ds, ld, layer, w.to(DEV), b.to(DEV) if bias else None, None, 3, None, None, None, R, dim, eps, None, None,
+                 None, None, 0, 0, 0, f32)
         want = x + nrm(sub)
         assert err(resid[:, :dim], want) < 1e-6 and err(act[:, :dim], want) < (1e-6 if f32 else 5e-3) and float(act[:, dim:].float().abs().sum()) == 0
         out = torch.zeros(3, ld, dtype=act.dtype, device=DEV)
-        nat.call("lsb_norm_rows", out, ld, resid, ld, i32([4, 0, 4]), 0, w.to(DEV), b.to(DEV) if bias else None, 3, dim, eps, layer, f32)
+        nat.call("lsb_norm_rows", out, ld, resid, ld, i32([4, 0, 4]), 0, w.to(DEV), b.to(DEV) if bias else None, None, 3, dim, eps, layer, f32)
         assert err(out[:, :dim], nrm(want[[4, 0, 4]])) < (1e-5 if f32 else 5e-3)
-        nat.call("lsb_norm_rows", out, ld, resid, ld, None, 2, w.to(DEV), b.to(DEV) if bias else None, 3, dim, eps, layer, f32)
+        nat.call("lsb_norm_rows", out, ld, resid, ld, None, 2, w.to(DEV), b.to(DEV) if bias else None, None, 3, dim, eps, layer, f32)
         assert err(out[:, :dim], nrm(want[2:5])) < (1e-5 if f32 else 5e-3)
 
 
@@ -273,7 +274,8 @@ def test_grouped_router_and_identity_experts(E, ident, top, count, keep):
     val = torch.where((ids < E)[..., None], y, x[:, None, :].expand(-1, top, -1))
     want = x + O.layer_norm((wt[..., None] * val).sum(1), w, b, 1e-5)
     resid, act = x.to(DEV).contiguous(), torch.zeros(R, H, device=DEV)
-    nat.call("lsb_post_norm", act, H, resid, H, None, 0, w.to(DEV), b.to(DEV), R, H, 1e-5, 1, y.to(DEV), dw, di, torch.arange(E, dtype=I32, device=DEV), top, E, H, 1)
+    nat.call("lsb_resid_update", act, H, resid, H, None, 0, 1, w.to(DEV), b.to(DEV), None, 3, None, None, None, R, H, 1e-5, y.to(DEV), dw, di,
+             torch.arange(E, dtype=I32, device=DEV), top, E, H, 1)
     assert err(resid, want) < 1e-5 and torch.equal(resid, act)
 
 
