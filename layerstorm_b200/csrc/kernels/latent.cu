@@ -175,7 +175,7 @@ struct LatentAttn {
     const float* proj; int ldp, off_gate;
     bf16* out;                        // [rows, H, dlp]
     float* o_part; float* ml_part;    // [rows, H, NS, dlp], [rows, H, NS, 2]
-    int H, dl, dlp, drp, NS;
+    int H, dlp, drp, NS;
     float scale2;                     // log2 units
 };
 
@@ -549,49 +549,54 @@ LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, c
     LSB_CHECK_LAUNCH();
 }
 
-// Attention of the step's rows and the value up-projection: out [rows, ldo] = W_uv (gate * attention), heads side by side.
-// w_uv: [H, dv, dlp].  o_lat: scratch [rows, H, dlp].  seq_row0 / seq_nrows: the step's sequences (consecutive positions each); run_rows: the largest
-// number of rows one of them has; NS: key splits (o_part / ml_part sized for it; runs use 1).
+// Attention of the step's rows.  NS 1: o_lat [rows, H, dlp], gated; NS > 1 (key splits, for steps of few rows): partial sums in o_part / ml_part, merged
+// by lsb_latent_out.  seq_row0 / seq_nrows: the step's sequences (consecutive positions each); run_rows: the largest number of rows one of them has.
 LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
                             const void* seq_row0, const void* seq_nrows, int nseq, int run_rows, const void* proj, int ldp, int off_gate, void* o_lat,
-                            void* o_part, void* ml_part, int NS, const void* w_uv, void* out, int ldo, int rows, int H, int dl, int dr, int dv,
-                            float scale, int f32, void* err, void* stream) {
+                            void* o_part, void* ml_part, int NS, int rows, int H, int dl, int dr, float scale, int f32, void* stream) {
     if (rows < 1 || NS < 1 || NS > 32 || (NS > 1 && (!o_part || !ml_part)) || dl < 1 || dr < 1) return -1;
     const int dlp = lsb_latent_pad(dl), drp = lsb_latent_pad(dr), D = dlp + drp;
     cudaStream_t st = (cudaStream_t)stream;
-    int rc = 0;
     if (latent_tc(dlp, drp, f32)) {
         LatentAttn p;
         p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page;
         p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos; p.seq_row0 = (const int*)seq_row0; p.seq_nrows = (const int*)seq_nrows;
         p.nseq = nseq; p.run_rows = run_rows; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.out = (bf16*)o_lat;
-        p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.H = H; p.dl = dl; p.dlp = dlp; p.drp = drp; p.NS = NS; p.scale2 = scale * kLog2e;
+        p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.H = H; p.dlp = dlp; p.drp = drp; p.NS = NS; p.scale2 = scale * kLog2e;
         const int mg = row_tiles(run_rows, H), bm = 16 * mg;
         const long long tiles = run_rows == 1 ? (long long)rows * ((H + bm - 1) / bm) : (long long)rows * H / bm + nseq;
         if (tiles > 0x7fffffff) return -1;
         const int nv = dlp <= 64 ? 1 : (dlp <= 128 ? 2 : (dlp <= 256 ? 4 : 8));
-        if (nv == 1) rc = launch_latent_rows<1>(p, mg, (int)tiles, st);
-        else if (nv == 2) rc = launch_latent_rows<2>(p, mg, (int)tiles, st);
-        else if (nv == 4) rc = launch_latent_rows<4>(p, mg, (int)tiles, st);
-        else rc = launch_latent_rows<8>(p, mg, (int)tiles, st);
-        if (rc) return rc;
-    } else {
-        if (NS != 1) return -1;
-        AttnParams p;
-        p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
-        p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.ldc = D; p.off_v = 0;
-        p.out = o_lat; p.ldo = H * dlp; p.o_part = p.ml_part = nullptr; p.rows = rows; p.H = H; p.G = 1; p.dk = p.dkp = D; p.dv = p.dvp = dlp; p.NS = 1;
-        p.window = 0; p.scale = scale; p.slope = nullptr;
-        const size_t smem = (size_t)(D + 256 + dlp) * 4;
-        if (smem > 48 * 1024) return -1;
-        if (f32) launch_pdl((attn_exact_kernel<float>), dim3(rows, H), 128, smem, st, p);
-        else launch_pdl((attn_exact_kernel<bf16>), dim3(rows, H), 128, smem, st, p);
+        if (nv == 1) return launch_latent_rows<1>(p, mg, (int)tiles, st);
+        if (nv == 2) return launch_latent_rows<2>(p, mg, (int)tiles, st);
+        if (nv == 4) return launch_latent_rows<4>(p, mg, (int)tiles, st);
+        return launch_latent_rows<8>(p, mg, (int)tiles, st);
     }
+    if (NS != 1) return -1;
+    AttnParams p;
+    p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
+    p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.ldc = D; p.off_v = 0;
+    p.out = o_lat; p.ldo = H * dlp; p.o_part = p.ml_part = nullptr; p.rows = rows; p.H = H; p.G = 1; p.dk = p.dkp = D; p.dv = p.dvp = dlp; p.NS = 1;
+    p.window = 0; p.scale = scale; p.slope = nullptr;
+    const size_t smem = (size_t)(D + 256 + dlp) * 4;
+    if (smem > 48 * 1024) return -1;
+    if (f32) launch_pdl((attn_exact_kernel<float>), dim3(rows, H), 128, smem, st, p);
+    else launch_pdl((attn_exact_kernel<bf16>), dim3(rows, H), 128, smem, st, p);
+    LSB_CHECK_LAUNCH();
+}
+
+// Value up-projection: out [rows, ldo] = W_uv o_lat, heads side by side; NS > 1: o_lat is first made from the splits' partial sums (and gated).
+// w_uv: [H, dv, dlp].
+LSB_API int lsb_latent_out(void* out, int ldo, void* o_lat, const void* o_part, const void* ml_part, int NS, const void* w_uv, const void* proj, int ldp,
+                           int off_gate, const void* row_seq, int rows, int H, int dl, int dv, int f32, void* err, void* stream) {
+    if (rows < 1 || NS < 1 || NS > 32 || (NS > 1 && (!o_part || !ml_part || f32)) || dl < 1 || dv < 1) return -1;
+    const int dlp = lsb_latent_pad(dl);
+    cudaStream_t st = (cudaStream_t)stream;
     LatentOut o{o_lat, (const float*)o_part, (const float*)ml_part, NS, (const float*)proj, ldp, off_gate, (const int*)row_seq, rows, H, dlp, dv};
     if (!f32 && rows >= 8) {
         if (NS > 1) launch_pdl((latent_combine_kernel), dim3(rows, H), 128, 0, st, o, (bf16*)o_lat);
         if (dv % 8 == 0 && ldo % 8 == 0) {
-            rc = lsb_gemm_bf16_tc_batched(out, o_lat, w_uv, rows, dv, dlp, H, H * dlp, dlp, dlp, (long long)dv * dlp, ldo, dv, 1, err, stream);
+            const int rc = lsb_gemm_bf16_tc_batched(out, o_lat, w_uv, rows, dv, dlp, H, H * dlp, dlp, dlp, (long long)dv * dlp, ldo, dv, 1, err, stream);
             return rc ? rc : (int)cudaGetLastError();
         }
         o.NS = 1;

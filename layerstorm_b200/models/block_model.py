@@ -442,8 +442,10 @@ class BlockModel(ModelBase):
                  self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, R, b.heads, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank,
                  int(self.f32), err)
         nat.call("lsb_latent_attn", ws.q_lat, cache, self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
-                 max(ws.seq_rows), ws.proj, self.max_proj, og, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], L["w_uv"], ws.mix, L["out"].K, R,
-                 b.heads, b.kv_rank, b.rot_dim, b.vdim, b.scale, int(self.f32), err)
+                 max(ws.seq_rows), ws.proj, self.max_proj, og, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], R, b.heads, b.kv_rank, b.rot_dim,
+                 b.scale, int(self.f32))
+        nat.call("lsb_latent_out", ws.mix, L["out"].K, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], L["w_uv"], ws.proj, self.max_proj, og,
+                 ws.row_seq, R, b.heads, b.kv_rank, b.vdim, int(self.f32), err)
 
     def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
         mt = L["meta"]

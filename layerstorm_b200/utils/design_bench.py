@@ -1,9 +1,10 @@
 """Prefill and decode throughput of a model design at layer sizes of a real model (random weights), beside the framework's closest other
 design at equal size, with the device time of every kernel launcher.
 
-    python bench.py --design gazutar [--design-sizes 2048,4096]
+    python bench.py --design gazutar|rubasun [--design-sizes 2048,4096]
 
-Gazutar's neighbour is a KDA + MLA model of the same width, heads, experts and layer pattern (plain residual stream, dense latent attention).
+Gazutar's neighbour is a KDA + MLA model of the same width, heads, experts and layer pattern (plain residual stream, dense latent attention),
+Rubasun's an MLA + MoE model of the same width, heads, latent rows, experts and shared expert.
 Per launcher: all its calls of one step, recorded from an eager pass and replayed back to back in a CUDA graph (other layers' operands in
 between, so that a layer's weights are not left over in L2), divided by the number of calls.  Fractions are of the measured peaks
 (MEASURED_PEAKS.json): bytes or FLOPs that the operation has to move or do, over the launcher's time.
@@ -17,18 +18,18 @@ import statistics
 import torch
 
 from ..models.block_model import model_class
-from ..models.config import ModelConfig, gazutar_config
+from ..models.config import ModelConfig, gazutar_config, rubasun_config
 from ..ops import _native as nat
 from ..runtime.engine import Engine
 
 N_LAYERS, EVERY, TOP = 8, 4, 8
 
 
-def design_pair(hidden: int, window: int):
+def gazutar_pair(hidden: int):
     """(Gazutar, neighbour) of one size: 128-wide heads, experts of half the width, every fourth layer attention."""
     heads, att_heads, kv, experts, ff, vocab = hidden // 64, hidden // 128, max(1, hidden // 512), hidden // 64, hidden // 2, 65536
     mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": 8, "top": TOP, "groups": {"count": 8, "keep": 4}}}
-    att = {"heads": att_heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window}, "v_mix": True}
+    att = {"heads": att_heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 4096}, "v_mix": True}
     dlt = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}
     g = gazutar_config({"name": f"gazutar-{hidden}", "vocab": vocab, "width": hidden, "norm": {"eps": 1e-5}, "logit_scale": 0.5, "layers": [
         {"type": "attention", "mixer": att, "mlp": mlp} if i % EVERY == EVERY - 1 else {"type": "channel_delta", "mixer": dlt, "mlp": mlp} for i in range(N_LAYERS)]})
@@ -37,6 +38,23 @@ def design_pair(hidden: int, window: int):
                     n_shared=0, moe_inter=ff, scoring="softmax", n_group=8, topk_group=4, norm_topk_prob=False, router_bias=True,
                     layer_types=["mla" if i % EVERY == EVERY - 1 else "kda" for i in range(N_LAYERS)], kda_heads=heads, kda_head_dim=128, kda_rank=128)
     return g, k
+
+
+def rubasun_pair(hidden: int):
+    """(Rubasun, neighbour) of one size: 128 + 64 wide heads over rows of 512 + 64, experts of half the width, a dense first layer; every second
+    Rubasun layer reads the rows of the one before it, and every layer takes a per-token input of 256 channels."""
+    heads, experts, ff, vocab = hidden // 128, hidden // 64, hidden // 2, 65536
+    mixer = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "rot": {"base": 10000.0, "dims": 64}, "scale": 192 ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": TOP}, "shared": {"ff": ff, "limit": 7.0}}
+    g = rubasun_config({"name": f"rubasun-{hidden}", "vocab": vocab, "width": hidden, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "token_side": {"dim": 256}, "layers": [
+        {"type": "latent_attention", "mixer": mixer | ({"kv_from": i - 1} if i % 2 else {}), "mlp": moe if i else {"kind": "dense", "ff": 3 * hidden}} for i in range(N_LAYERS)]})
+    k = ModelConfig(name=f"mla-moe-{hidden}", architecture="deepseek_v3", hidden=hidden, n_layers=N_LAYERS, vocab=vocab, rms_eps=1e-5, n_heads=heads,
+                    q_lora=hidden * 3 // 8, kv_lora=512, qk_nope=128, qk_rope=64, v_head=128, dense_inter=3 * hidden, first_k_dense=1, n_routed=experts, top_k=TOP,
+                    n_shared=1, moe_inter=ff, scoring="sigmoid", norm_topk_prob=False)
+    return g, k
+
+
+DESIGNS = {"gazutar": gazutar_pair, "rubasun": rubasun_pair}
 
 
 def _peaks():
@@ -101,27 +119,42 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
     state = 2 * batch * heads * 128 * 128 * 4                       # read and write the recurrent state once
     gates = 2 * heads * 128 * 128 * 2
     per_tok = heads * (4 * 128 * 128 + 6 * 64 * 128) * 2            # chunk form: state products, pair products
-    rec = ("bytes", state + gates + rows * heads * 128 * 18) if rows == batch else ("flops", rows * per_tok)
-    if cfg.blocks:
-        b = next(x for x in cfg.blocks if not x.recurrent)
+    decode = rows == batch
+    rec = ("bytes", state + gates + rows * heads * 128 * 18) if decode else ("flops", rows * per_tok)
+    att = next((x for x in cfg.blocks if not x.recurrent), None)
+    lat, rot, ah, dn, dv = cfg.kv_lora, cfg.qk_rope, cfg.n_heads, cfg.qk_nope, cfg.v_head
+    seen = ctx - rows // 2                                          # keys a row of the chunk sees on average
+    latent = ("bytes", batch * ctx * (lat + rot) * 2 + rows * ah * (2 * lat + rot) * 2) if decode else ("flops", 2 * rows * seen * ah * (2 * lat + rot))
+    # the queries' way into the latent space and the values' way out of it: weights and activations, or products
+    absorb, up = ((("bytes", ah * lat * d * 2 + rows * ah * (lat + d) * 2) if decode else ("flops", 2 * rows * ah * lat * d)) for d in (dn, dv))
+    experts = TOP + cfg.n_shared
+    if att is not None and att.latent:
+        out["lsb_latent_attn"], out["lsb_latent_query"], out["lsb_latent_out"] = latent, absorb, up
+        out["lsb_resid_update"] = ("bytes", rows * H * 14)
+        out["lsb_glu"] = ("bytes", rows * cfg.moe_inter * 10)
+    elif att is not None:
+        b = att
         seen = min(ctx, b.window)
         out["lsb_delta_forward"] = rec
         kv = b.kv_heads * (b.dim + b.vdim) * 2
-        out["lsb_attn"] = ("bytes", batch * seen * kv + rows * b.heads * b.vdim * 6) if rows == batch else ("flops", 2 * rows * seen * b.heads * (b.dim + b.vdim))
+        out["lsb_attn"] = ("bytes", batch * seen * kv + rows * b.heads * b.vdim * 6) if decode else ("flops", 2 * rows * seen * b.heads * (b.dim + b.vdim))
         out["lsb_attn_prep"] = ("bytes", rows * ((b.heads + b.kv_heads) * b.dim + b.kv_heads * b.vdim) * 6)
         out["lsb_resid_update"] = ("bytes", rows * H * (14 + TOP * 4) // 2 + rows * H * 7)
     else:
         out["lsb_kda_forward"] = out["lsb_kda_forward_chunked"] = rec
-        lat = cfg.kv_lora
-        out["lsb_mla_decode"] = ("bytes", batch * ctx * lat * 2 + rows * cfg.n_heads * lat * 4) if rows == batch else ("flops", 4 * rows * ctx * cfg.n_heads * lat)
+        out["lsb_mla_decode"] = latent
+        out["lsb_batched_gemv_bf16"] = (absorb[0], (absorb[1] + up[1]) / 2)
         out["lsb_add_rmsnorm"] = ("bytes", rows * H * 14)
-        out["lsb_moe_combine"] = ("bytes", rows * H * (TOP + 1) * 4)
-        out["lsb_mla_prep"] = ("bytes", rows * (cfg.q_lora + lat) * 6)
+        out["lsb_moe_combine"] = ("bytes", rows * H * (experts + 1) * 4)
+        out["lsb_mla_prep"] = ("bytes", rows * (cfg.q_lora + lat + rot) * 6)
     if rows == 1:                          # (how many experts a batch touches is the router's affair)
-        by = TOP * 3 * H * cfg.moe_inter * 2
-        out["lsb_moe_gateup"], out["lsb_moe_down"] = ("bytes", by * 2 / 3), ("bytes", by / 3)
+        by = experts * 3 * H * cfg.moe_inter * 2
+        out["lsb_moe_gateup"] = out["lsb_moe_gateup_act"] = ("bytes", by * 2 / 3)
+        out["lsb_moe_down"] = ("bytes", by / 3)
     elif rows > 1024:
-        out["lsb_moe_tc_ffn"] = ("flops", 3 * rows * TOP * H * cfg.moe_inter)
+        own = att is not None and att.scale_input                    # gate/up and down are launchers of their own, else halves of one launcher's calls
+        out["lsb_moe_tc_ffn"] = ("flops", (2 if own else 3) * rows * experts * H * cfg.moe_inter)
+        out["lsb_moe_tc_gateup_act"] = ("flops", 4 * rows * experts * H * cfg.moe_inter)
     return out
 
 
@@ -185,14 +218,13 @@ def measure(cfg, ctx: int, chunk: int, batches, clocks=None) -> dict:
 
 
 def run(design: str, sizes, ctx: int = 8192, chunk: int = 2048, batches=(1, 32), sampler=None) -> dict:
-    if design != "gazutar":
-        raise ValueError(f"no comparison for design {design!r}")
+    pair = DESIGNS[design]
     out = {"metric": "prefill and decode throughput beside the closest design", "design": design, "data": "random weights, synthetic token ids", "dtype": "bf16",
-           "context": ctx, "window": 4096, "l2": "decode and prefill steps stream more weights than L2 holds", "sizes": {}}
+           "context": ctx, "l2": "decode and prefill steps stream more weights than L2 holds", "sizes": {}}
     if sampler is not None:
         sampler.start()
     for h in sizes:
-        out["sizes"][str(h)] = [measure(c, ctx, chunk, list(batches)) for c in design_pair(h, 4096)]
+        out["sizes"][str(h)] = [measure(c, ctx, chunk, list(batches)) for c in pair(h)]
     if sampler is not None:
         out["clocks"] = sampler.stop()
     return out
