@@ -10,15 +10,18 @@
 //   latent_query    few rows (and fp32): rotation, absorption and the cache append in one launch
 //   latent_prep     many rows: rotation, append and the bf16 operand of the absorbing product, which then runs on the tcgen05 GEMM
 //   latent_attn     (token, head) rows of a sequence in tiles of 16 MG against key tiles shared by all of them; any mixture of prompt runs and
-//                   single tokens; key splits for small batches
-//   latent_combine  merge of the splits;  latent_out: the same together with the value up-projection (few rows)
+//                   single tokens; key splits for small batches: up to eight splits are a thread-block cluster that merges its sums through
+//                   distributed shared memory, what is left (one partial sum per cluster) goes through global memory
+//   latent_combine  merge of those partial sums;  latent_out: the same together with the value up-projection (few rows)
 // The value of a key is the head of its cache row, so a key tile is loaded once for both products.
 #include "attn_core.cuh"
+#include <cooperative_groups.h>
 
 extern "C" int lsb_gemm_bf16_tc_batched(void* out, const void* x, const void* w, int M, int N, int K, int B, int ldx, long long xs_b, int ldw,
                                         long long ws_b, int ldo, long long os_b, int out_bf16, void* err, void* stream);
 
 namespace lsb {
+namespace cg = cooperative_groups;
 
 struct LatentPrep {
     const float* proj; int ldp, off_q, off_kv;        // off_kv < 0: the layer has no latent projection of its own
@@ -100,12 +103,22 @@ __device__ __forceinline__ void small_products(const T* w, int K, int n0, int n1
     }
 }
 
+// Weights do not depend on the previous kernel: on their way to L2 before the dependency wait (first block of a column range only).
+template <typename T>
+__device__ __forceinline__ void prefetch_rows(const T* w, size_t n) {
+    if (blockIdx.z) return;
+    const char* b = reinterpret_cast<const char*>(w);
+    for (size_t i = (size_t)threadIdx.x * 128; i < n * sizeof(T); i += 256 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(b + i));
+}
+
 constexpr int kQueryCols = 128;       // latent columns per block of latent_query
 template <typename T, int MT>
 __global__ void __launch_bounds__(256) latent_query_kernel(LatentPrep p) {
     extern __shared__ __align__(16) float lsm[];              // [MT][dnp]
     __shared__ float red[33];
     const int h = blockIdx.y, r0 = blockIdx.z * MT, nr = min(MT, p.rows - r0), t = threadIdx.x, D = p.dlp + p.drp;
+    const int n0 = blockIdx.x * kQueryCols, n1 = min(p.dlp, n0 + kQueryCols);
+    if (n0 < n1) prefetch_rows(reinterpret_cast<const T*>(p.w_uk) + ((size_t)h * p.dlp + n0) * p.dnp, (size_t)(n1 - n0) * p.dnp);
     pdl_wait();
     pdl_launch_dependents();
     T* q = reinterpret_cast<T*>(p.q) + ((size_t)r0 * p.H + h) * D;
@@ -122,7 +135,6 @@ __global__ void __launch_bounds__(256) latent_query_kernel(LatentPrep p) {
         lsm[i] = m < nr && c < p.dn ? src[(size_t)m * p.ldp + c] : 0.f;
     }
     __syncthreads();
-    const int n0 = blockIdx.x * kQueryCols, n1 = min(p.dlp, n0 + kQueryCols);
     small_products<T, MT>(reinterpret_cast<const T*>(p.w_uk) + (size_t)h * p.dlp * p.dnp, p.dnp, n0, n1, lsm, p.dnp, [&](int n, const float (&a)[MT]) {
 #pragma unroll
         for (int m = 0; m < MT; ++m)
@@ -174,8 +186,8 @@ struct LatentAttn {
     const int* row_seq; const int* row_pos; const int* seq_row0; const int* seq_nrows; int nseq, run_rows;
     const float* proj; int ldp, off_gate;
     bf16* out;                        // [rows, H, dlp]
-    float* o_part; float* ml_part;    // [rows, H, NS, dlp], [rows, H, NS, 2]
-    int H, dlp, drp, NS;
+    float* o_part; float* ml_part;    // [rows, H, NS / C, dlp], [rows, H, NS / C, 2]
+    int H, dlp, drp, NS, C;           // key splits, and how many of them form a cluster
     float scale2;                     // log2 units
 };
 
@@ -185,6 +197,8 @@ template <int NV, int MG> struct LatentCfg {
     static constexpr int RANGES = 8 / MG, KW = KT / RANGES, NT = KW / 8, LDP = KT + 8;      // score phase: a warp owns 16 rows x KW keys
     static __host__ __device__ int ld(int D) { return (D > NV * 64 ? D : NV * 64) + 8; }     // an odd multiple of 16 bytes
     static size_t smem(int D) { return (size_t)(BM + STAGES * KT) * ld(D) * 2 + (size_t)2 * BM * LDP * 2 + (size_t)(RANGES + 1) * BM * 4; }
+    // the cluster merge reuses the query and key tiles
+    static_assert((size_t)BM * (NV * 64 + 4) * 4 + 8 * BM * 4 <= (size_t)(BM + STAGES * KT) * (NV * 64 + 8) * 2, "merge scratch");
 };
 __device__ __forceinline__ void ldsm2(uint32_t (&r)[2], const bf16* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(sm_addr(p)));
@@ -233,12 +247,18 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
     const int ntile = pos_last / KT + 1, per = (ntile + p.NS - 1) / p.NS, t0 = (int)blockIdx.y * per, t1 = min(ntile, t0 + per);
     constexpr int TPK = 256 / KT;                                 // threads per key of a tile copy
     const int kr = t / TPK;
+    const int* bt = p.block_table + (size_t)seq * p.max_pages;
+    auto locate = [&](int kt) {                                   // cache row of this thread's key in tile kt
+        const int j = min(kt * KT + kr, pos_last);                // keys past the tile's last position are clamped (masked later)
+        return kt < t1 ? (size_t)bt[j / p.page] * p.page + j % p.page : 0;
+    };
+    size_t ahead = locate(t0);                                    // looked up one tile early: the copies do not wait for the table
     auto issue = [&](int kt) {
         if (kt < t1) {
-            const int j = min(kt * KT + kr, pos_last);            // keys past the tile's last position are clamped (masked later)
-            const bf16* src = p.cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * D;
+            const bf16* src = p.cache + ahead * D;
             bf16* dst = sk + ((size_t)((kt - t0) % C::STAGES) * KT + kr) * ld;
             for (int c = t % TPK; c < chunks; c += TPK) cp16(dst + c * 8, src + c * 8);
+            ahead = locate(kt + 1);
         }
         cp_commit();
     };
@@ -286,7 +306,7 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
             }
         };
         int k = 0;
-#pragma unroll 2
+#pragma unroll(MG == 4 ? 2 : 4)
         for (; k + 32 <= D; k += 32) { step(k, s[0]); step(k + 16, s[1]); }
         if (k < D) step(k, s[0]);
         float mt[2] = {-INFINITY, -INFINITY};
@@ -381,35 +401,92 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
         }
     }
     __syncthreads();
+    float L = 0.f;
+    if (t < BM) {
 #pragma unroll
-    for (int a = 0; a < MG; ++a)
+        for (int r = 0; r < C::RANGES; ++r) L += s_max[r * BM + t];
+    }
+    __syncthreads();
+    if (t < BM) s_max[t] = L;                                     // sums and maxima of the tile's rows: s_max[m], s_corr[m]
+    auto gate = [&](int m) {
+        return p.off_gate >= 0 ? gate_sigmoid(p.proj[(size_t)(row0 + (f0 + m) / p.H) * p.ldp + p.off_gate + (f0 + m) % p.H]) : 1.f;
+    };
+    if (p.C == 1) {
+        __syncthreads();
 #pragma unroll
-        for (int u = 0; u < 2; ++u) {
-            const int m = a * 16 + (lane >> 2) + 8 * u;
-            if (m >= nf) continue;
-            float L = 0.f;
+        for (int a = 0; a < MG; ++a)
 #pragma unroll
-            for (int r = 0; r < C::RANGES; ++r) L += s_max[r * BM + m];
-            const size_t rh = (size_t)row0 * p.H + f0 + m;
-            if (p.NS == 1) {
-                const int h = (f0 + m) % p.H;
-                float f = 1.f / L;
-                if (p.off_gate >= 0) f *= gate_sigmoid(p.proj[(size_t)(row0 + (f0 + m) / p.H) * p.ldp + p.off_gate + h]);
+            for (int u = 0; u < 2; ++u) {
+                const int m = a * 16 + (lane >> 2) + 8 * u;
+                if (m >= nf) continue;
+                const size_t rh = (size_t)row0 * p.H + f0 + m;
+                const float f = gate(m) / s_max[m];
 #pragma unroll
                 for (int b = 0; b < NV; ++b) {
                     const int c = (warp * NV + b) * 8 + (lane & 3) * 2;
                     if (c < p.dlp) *reinterpret_cast<bf162*>(p.out + rh * p.dlp + c) = __floats2bfloat162_rn(o[a][b][2 * u] * f, o[a][b][2 * u + 1] * f);
                 }
-            } else {
-                const size_t k = rh * p.NS + blockIdx.y;
-#pragma unroll
-                for (int b = 0; b < NV; ++b) {
-                    const int c = (warp * NV + b) * 8 + (lane & 3) * 2;
-                    if (c < p.dlp) *reinterpret_cast<float2*>(p.o_part + k * p.dlp + c) = make_float2(o[a][b][2 * u], o[a][b][2 * u + 1]);
-                }
-                if (warp == 0 && (lane & 3) == 0) { p.ml_part[2 * k] = s_corr[m]; p.ml_part[2 * k + 1] = L; }
             }
+        return;
+    }
+    // merge inside the cluster: every CTA shows its sums, and takes an equal share of the columns of all of them
+    constexpr int LDO = NV * 64 + 4;
+    float* so = reinterpret_cast<float*>(asm_);                   // [BM][LDO], over the query and key tiles
+    float* s_w = so + BM * LDO;                                   // [8][BM] weights of the CTAs, then the row's factor
+#pragma unroll
+    for (int a = 0; a < MG; ++a)
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            float* d = so + (a * 16 + (lane >> 2) + 8 * u) * LDO + warp * NV * 8 + (lane & 3) * 2;
+#pragma unroll
+            for (int b = 0; b < NV; ++b) *reinterpret_cast<float2*>(d + b * 8) = make_float2(o[a][b][2 * u], o[a][b][2 * u + 1]);
         }
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();
+    const int rank = (int)cluster.block_rank(), NSo = p.NS / p.C, so_i = (int)blockIdx.y / p.C;
+    if (t < nf) {
+        float mm[8], ll[8], M = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            mm[j] = j < p.C ? cluster.map_shared_rank(s_corr, j)[t] : -INFINITY;
+            ll[j] = j < p.C ? cluster.map_shared_rank(s_max, j)[t] : 0.f;
+            M = fmaxf(M, mm[j]);
+        }
+        float S = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            mm[j] = mm[j] == -INFINITY ? 0.f : ex2(mm[j] - M);
+            S = fmaf(mm[j], ll[j], S);
+        }
+        const float f = NSo == 1 ? gate(t) / S : 1.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s_w[j * BM + t] = mm[j] * f;
+        if (NSo > 1 && rank == 0) {
+            const size_t k = ((size_t)row0 * p.H + f0 + t) * NSo + so_i;
+            p.ml_part[2 * k] = M; p.ml_part[2 * k + 1] = S;
+        }
+    }
+    __syncthreads();
+    const int quads = NV * 16 / p.C;                              // groups of four columns per CTA
+    for (int i = t; i < nf * quads; i += 256) {
+        const int m = i / quads, c = (rank * quads + i - m * quads) * 4;
+        float4 v[8], a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (j < p.C) v[j] = *reinterpret_cast<const float4*>(cluster.map_shared_rank(so, j) + m * LDO + c);
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (j < p.C) { const float w = s_w[j * BM + m]; a.x = fmaf(w, v[j].x, a.x); a.y = fmaf(w, v[j].y, a.y); a.z = fmaf(w, v[j].z, a.z); a.w = fmaf(w, v[j].w, a.w); }
+        if (c >= p.dlp) continue;
+        const size_t rh = (size_t)row0 * p.H + f0 + m;
+        if (NSo == 1) {
+            bf162* d = reinterpret_cast<bf162*>(p.out + rh * p.dlp + c);
+            d[0] = __floats2bfloat162_rn(a.x, a.y); d[1] = __floats2bfloat162_rn(a.z, a.w);
+        } else {
+            *reinterpret_cast<float4*>(p.o_part + (rh * NSo + so_i) * p.dlp + c) = a;
+        }
+    }
+    cluster.sync();                                               // nobody leaves while its sums may still be read
 }
 
 // ------------------------------------------------------------------------------------------------ split merge, value up-projection
@@ -433,7 +510,7 @@ __device__ __forceinline__ void split_weights(const LatentOut& p, int r, int h, 
 __device__ __forceinline__ float4 merged4(const LatentOut& p, int r, int h, int c, const float* w) {
     const float* op = p.o_part + ((size_t)r * p.H + h) * p.NS * p.dlp + c;
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
+#pragma unroll 16
     for (int s = 0; s < p.NS; ++s) {
         const float4 v = *reinterpret_cast<const float4*>(op + (size_t)s * p.dlp);
         a.x = fmaf(w[s], v.x, a.x); a.y = fmaf(w[s], v.y, a.y); a.z = fmaf(w[s], v.z, a.z); a.w = fmaf(w[s], v.w, a.w);
@@ -461,7 +538,8 @@ template <typename T, int MT>
 __global__ void __launch_bounds__(256) latent_out_kernel(LatentOut p, const T* __restrict__ w_uv, T* __restrict__ out, int ldo) {
     extern __shared__ __align__(16) float lsm[];              // [MT][dlp]
     __shared__ float w[MT][32];
-    const int h = blockIdx.y, r0 = blockIdx.z * MT, nr = min(MT, p.rows - r0), t = threadIdx.x;
+    const int h = blockIdx.y, r0 = blockIdx.z * MT, nr = min(MT, p.rows - r0), t = threadIdx.x, n0 = blockIdx.x * kOutCols, n1 = min(p.dv, n0 + kOutCols);
+    prefetch_rows(w_uv + ((size_t)h * p.dv + n0) * p.dlp, (size_t)(n1 - n0) * p.dlp);
     pdl_wait();
     pdl_launch_dependents();
     if (p.NS > 1) {
@@ -481,7 +559,6 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentOut p, const T* _
         }
     }
     __syncthreads();
-    const int n0 = blockIdx.x * kOutCols, n1 = min(p.dv, n0 + kOutCols);
     small_products<T, MT>(w_uv + (size_t)h * p.dv * p.dlp, p.dlp, n0, n1, lsm, p.dlp, [&](int n, const float (&a)[MT]) {
 #pragma unroll
         for (int m = 0; m < MT; ++m)
@@ -495,14 +572,28 @@ static int launch_latent(const LatentAttn& p, int tiles, cudaStream_t st) {
     if (smem > 226 * 1024) return -1;
     static bool attr = false;
     if (!attr) { cudaFuncSetAttribute(latent_attn_kernel<NV, MG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024); attr = true; }
-    launch_pdl((latent_attn_kernel<NV, MG>), dim3(tiles, p.NS), 256, smem, st, p);
-    return (int)cudaGetLastError();
+    if (p.C == 1) {
+        launch_pdl((latent_attn_kernel<NV, MG>), dim3(tiles, p.NS), 256, smem, st, p);
+        return (int)cudaGetLastError();
+    }
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(tiles, p.NS); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = 1; at[0].val.clusterDim.y = p.C; at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at; cfg.numAttrs = pdl_enabled_flag() ? 2 : 1;
+    return (int)cudaLaunchKernelEx(&cfg, latent_attn_kernel<NV, MG>, p);
 }
 template <int NV>
 static int launch_latent_rows(const LatentAttn& p, int mg, int tiles, cudaStream_t st) {
     return mg == 1 ? launch_latent<NV, 1>(p, tiles, st) : (mg == 2 ? launch_latent<NV, 2>(p, tiles, st) : launch_latent<NV, 4>(p, tiles, st));
 }
 static int row_tiles(int run_rows, int H) { return run_rows * H <= 16 ? 1 : (run_rows * H <= 32 ? 2 : 4); }
+constexpr int kMaxSplits = 128;
+static int cluster_of(int NS) { return NS >= 8 ? 8 : NS; }
+static bool splits_ok(int NS) { return NS == 1 || NS == 2 || NS == 4 || (NS >= 8 && NS % 8 == 0 && NS <= kMaxSplits); }
 // the tensor-core kernel covers latents of up to 512 channels whose tiles fit an SM's shared memory
 static bool latent_tc(int dlp, int drp, int f32) { return !f32 && dlp <= 512 && dlp + drp <= 656; }
 
@@ -512,14 +603,17 @@ using namespace lsb;
 // padded width of the latent and of the rotated part in cache rows and queries
 LSB_API int lsb_latent_pad(int d) { return (d + 15) / 16 * 16; }
 
-// Key splits worth having for steps of `rows` single tokens over up to `seen` keys (o_part / ml_part are sized with it).
+// Key splits worth having for steps of `rows` single tokens over up to `seen` keys: 1, 2, 4 or a multiple of 8.
 LSB_API int lsb_latent_splits(int rows, int H, int dl, int dr, int seen, int f32) {
     if (!latent_tc((dl + 15) / 16 * 16, (dr + 15) / 16 * 16, f32)) return 1;
     const int mg = row_tiles(1, H), blocks = rows * ((H + 16 * mg - 1) / (16 * mg)), kt = mg == 4 ? 32 : 64;
     int ns = 148 / blocks;
     if (ns > (seen + kt - 1) / kt) ns = (seen + kt - 1) / kt;
-    return ns < 1 ? 1 : (ns > 32 ? 32 : ns);
+    if (ns > kMaxSplits) ns = kMaxSplits;
+    return ns >= 8 ? ns / 8 * 8 : (ns >= 4 ? 4 : (ns >= 2 ? 2 : 1));
 }
+// Partial sums per (row, head) that NS splits leave to lsb_latent_out (1: none, the attention kernel writes its result): o_part [rows, H, this, dlp].
+LSB_API int lsb_latent_partials(int NS) { return NS / cluster_of(NS); }
 
 // Queries in the latent space and the cache append.  w_uk: [H, dlp, dnp] (dn padded to dnp % 8 == 0 with zeros).  off_kv < 0: nothing is appended.
 LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_uk,
@@ -549,12 +643,12 @@ LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, c
     LSB_CHECK_LAUNCH();
 }
 
-// Attention of the step's rows.  NS 1: o_lat [rows, H, dlp], gated; NS > 1 (key splits, for steps of few rows): partial sums in o_part / ml_part, merged
-// by lsb_latent_out.  seq_row0 / seq_nrows: the step's sequences (consecutive positions each); run_rows: the largest number of rows one of them has.
+// Attention of the step's rows.  NS: key splits (lsb_latent_splits; runs of rows use 1).  One partial sum: o_lat [rows, H, dlp], gated; more: o_part /
+// ml_part, merged by lsb_latent_out.  seq_row0 / seq_nrows: the step's sequences (consecutive positions each); run_rows: the largest number of rows one of them has.
 LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
                             const void* seq_row0, const void* seq_nrows, int nseq, int run_rows, const void* proj, int ldp, int off_gate, void* o_lat,
                             void* o_part, void* ml_part, int NS, int rows, int H, int dl, int dr, float scale, int f32, void* stream) {
-    if (rows < 1 || NS < 1 || NS > 32 || (NS > 1 && (!o_part || !ml_part)) || dl < 1 || dr < 1) return -1;
+    if (rows < 1 || !splits_ok(NS) || (lsb_latent_partials(NS) > 1 && (!o_part || !ml_part)) || dl < 1 || dr < 1) return -1;
     const int dlp = lsb_latent_pad(dl), drp = lsb_latent_pad(dr), D = dlp + drp;
     cudaStream_t st = (cudaStream_t)stream;
     if (latent_tc(dlp, drp, f32)) {
@@ -562,7 +656,7 @@ LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_
         p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page;
         p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos; p.seq_row0 = (const int*)seq_row0; p.seq_nrows = (const int*)seq_nrows;
         p.nseq = nseq; p.run_rows = run_rows; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.out = (bf16*)o_lat;
-        p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.H = H; p.dlp = dlp; p.drp = drp; p.NS = NS; p.scale2 = scale * kLog2e;
+        p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.H = H; p.dlp = dlp; p.drp = drp; p.NS = NS; p.C = cluster_of(NS); p.scale2 = scale * kLog2e;
         const int mg = row_tiles(run_rows, H), bm = 16 * mg;
         const long long tiles = run_rows == 1 ? (long long)rows * ((H + bm - 1) / bm) : (long long)rows * H / bm + nseq;
         if (tiles > 0x7fffffff) return -1;
@@ -585,7 +679,7 @@ LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_
     LSB_CHECK_LAUNCH();
 }
 
-// Value up-projection: out [rows, ldo] = W_uv o_lat, heads side by side; NS > 1: o_lat is first made from the splits' partial sums (and gated).
+// Value up-projection: out [rows, ldo] = W_uv o_lat, heads side by side; NS (partial sums) > 1: o_lat is first made from them (and gated).
 // w_uv: [H, dv, dlp].
 LSB_API int lsb_latent_out(void* out, int ldo, void* o_lat, const void* o_part, const void* ml_part, int NS, const void* w_uv, const void* proj, int ldp,
                            int off_gate, const void* row_seq, int rows, int H, int dl, int dv, int f32, void* err, void* stream) {

@@ -579,6 +579,11 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
             const int n = jn * kTBM + q * 32 + lane;
             const uint8_t* base = p.arena + (size_t)slot * p.ef.stride;
             const uint32_t buf = lt % C::NBUF;
+            // the columns' factors on the experts' inputs, fetched while the tile is being computed
+            float in_scale[BN / 32];
+#pragma unroll
+            for (int g = 0; g < BN / 32; ++g)
+                in_scale[g] = GATEUP && p.ga.in_scale && g * 32 + lane < ncols ? p.ga.in_scale[p.sorted_pair[row0 + g * 32 + lane]] : 1.f;
             int okw = 1;
             if (lane == 0) { if (q == 0) PROF_SCOPE(0, okw = mbar_wait_relaxed(&acc_full[buf], (lt / C::NBUF) & 1u, p.err, 14) ? 1 : 0); else okw = mbar_wait_relaxed(&acc_full[buf], (lt / C::NBUF) & 1u, p.err, 14) ? 1 : 0; }
             ok = __shfl_sync(0xffffffffu, okw, 0) != 0;
@@ -600,11 +605,14 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                     float gq[16], uq[16];
                     tmem_ld16(lane_addr + (uint32_t)c0, gq);
                     if (GATEUP) tmem_ld16(lane_addr + (uint32_t)(BN + c0), uq);
+                    float cs = in_scale[0];                                // factors of this group of 32 columns, one per lane
+#pragma unroll
+                    for (int g = 1; g < BN / 32; ++g) cs = (c0 >> 5) == g ? in_scale[g] : cs;
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
+                        const float c = GATEUP ? __shfl_sync(0xffffffffu, cs, (c0 + j) & 31) : 1.f;
                         if (c0 + j < ncols && n < NOUT) {
                             if (GATEUP) {
-                                const float c = p.ga.in_scale ? p.ga.in_scale[p.sorted_pair[row0 + c0 + j]] : 1.f;
                                 p.act[(size_t)(row0 + c0 + j) * NOUT + n] = __float2half_rn(glu_act(gq[j] * sg * c, uq[j] * su * c, p.ga));
                             } else if (ep_mode) {
                                 const int2 ra = p.ep.ret[p.ep.rank][row0 + c0 + j];      // (token owner, pair index there)

@@ -150,7 +150,8 @@ class BlockWorkspace(StepBuffers):
             self.o_lat = z(R * max(b.heads * m.latent_pad(b.kv_rank) for b in lat), dtype=act)
             self.lat_splits = {i: 1 if R > 64 else int(nat.call("lsb_latent_splits", R, b.heads, b.kv_rank, b.rot_dim, max_ctx, int(m.f32)))
                                for i, b in enumerate(m.cfg.blocks) if b.latent}
-            ns = [(b.heads * self.lat_splits[i], m.latent_pad(b.kv_rank)) for i, b in enumerate(m.cfg.blocks) if b.latent and self.lat_splits[i] > 1]
+            self.lat_parts = {i: int(nat.call("lsb_latent_partials", n)) for i, n in self.lat_splits.items()}
+            ns = [(b.heads * self.lat_parts[i], m.latent_pad(b.kv_rank)) for i, b in enumerate(m.cfg.blocks) if self.lat_parts.get(i, 1) > 1]
             self.lat_o_part = z(R * max((n * w for n, w in ns), default=1))
             self.lat_ml_part = z(2 * R * max((n for n, _ in ns), default=1))
         dense = max((_align(max(b.dense_ff, b.shared_ff), 8) for b in m.cfg.blocks), default=0)
@@ -444,7 +445,7 @@ class BlockModel(ModelBase):
         nat.call("lsb_latent_attn", ws.q_lat, cache, self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
                  max(ws.seq_rows), ws.proj, self.max_proj, og, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], R, b.heads, b.kv_rank, b.rot_dim,
                  b.scale, int(self.f32))
-        nat.call("lsb_latent_out", ws.mix, L["out"].K, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], L["w_uv"], ws.proj, self.max_proj, og,
+        nat.call("lsb_latent_out", ws.mix, L["out"].K, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_parts[i], L["w_uv"], ws.proj, self.max_proj, og,
                  ws.row_seq, R, b.heads, b.kv_rank, b.vdim, int(self.f32), err)
 
     def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):

@@ -201,6 +201,6 @@ MODELS = {
                                           lat(40, 64, 32, 64, 256, mlp=moe_spec(8, 2, 256, 3.0, 128, 1.0), base=1e5), lat(8, 96, 32, 128, 256, 2, base=1e5)], 1e-5, 2.0, 64),
     "ones": lambda: model_cfg(48, 40, [lat(1, 1, 2, 1, 1, mlp=moe_spec(1, 1, 1, shared=1)), lat(1, 8, 2, 8, 8, mlp=moe_spec(3, 3, 8, 2.0)), lat(16, 1, 2, 3, 1, 0, dense(1))],
                               1e-6, 1.0, 1),
-    "wide": lambda: model_cfg(256, 200, [lat(33, 24, 16, 16, 600, mlp=moe_spec(4, 1, 96, 1.0)), lat(5, 200, 16, 136, 600, 0, dense(136), scale=0.05),
+    "wide": lambda: model_cfg(250, 200, [lat(33, 24, 16, 16, 600, mlp=moe_spec(4, 1, 96, 1.0)), lat(5, 200, 16, 136, 600, 0, dense(136), scale=0.05),
                                          lat(70, 8, 8, 8, 128, mlp=moe_spec(6, 2, 64, 0.6, 200))], 1e-4, 3.0),
 }
