@@ -165,7 +165,9 @@ def workspace_bytes(mc: ModelConfig, max_rows: int, max_ctx: int) -> int:
     per_row = H * 4 * (2 + 2 * mc.hc_mult) + mc.n_heads * (mc.qk_head + mc.kv_lora + mc.v_head) * 4 + mc.top_k * (2 * mc.moe_inter + H) * 4
     per_row += 3 * mc.kda_heads * mc.kda_head_dim * 4 + mc.dense_inter * 2 * 4
     score = mc.index_n_heads and max_ctx * 4 * min(max_rows, 256)
-    return int(per_row * max_rows + score + (64 << 20))
+    # latent layers write keys and values of all positions out per head for long prompt runs, while that stays within a bound
+    wide = max((b.heads * (_align(b.dim, 16) + _head_pad(b.vdim)) + _align(b.rot_dim, 16) + b.kv_rank for b in mc.blocks if b.latent), default=0)
+    return int(per_row * max_rows + score + min(2 * wide * max_ctx, 5 << 28) + (64 << 20))
 
 
 @dataclass

@@ -299,7 +299,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
     const int pos_last = pos0 + n - 1;
     const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) / kPreKeys * kPreKeys : 0;
     const int ntile = (pos_last - lo) / kPreKeys + 1;
-    const size_t ldc = (size_t)p.G * (p.dkp + p.dvp);
+    const size_t ldc = (size_t)p.ldc;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache);
     const int kc = p.dkp / 8, vc = DVP / 8;
     auto issue = [&](int tile) {
@@ -308,8 +308,8 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
             bf16* dv_ = dk_ + kPreKeys * ldk;
             const int kr = t / kTpk, j = min(lo + tile * kPreKeys + kr, pos_last);
             const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
-            for (int c = t % kTpk; c < kc; c += kTpk) cp16(dk_ + kr * ldk + c * 8, src + (size_t)g * p.dkp + c * 8);
-            for (int c = t % kTpk; c < vc; c += kTpk) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.G * p.dkp + (size_t)g * p.dvp + c * 8);
+            for (int c = t % kTpk; c < kc; c += kTpk) cp16(dk_ + kr * ldk + c * 8, src + (c * 8 < p.dkh ? (size_t)g * p.dkh + c * 8 : (size_t)p.off_ks + c * 8 - p.dkh));
+            for (int c = t % kTpk; c < vc; c += kTpk) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)g * p.dvp + c * 8);
         }
         cp_commit();
     };
@@ -348,8 +348,8 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         l[row] += __shfl_xor_sync(0xffffffffu, l[row], 2);
         const int tok = mr[row] / hg, h = g * hg + mr[row] % hg;
         if (tok >= n) continue;
-        const float inv = 1.f / l[row];
         const size_t rr = (size_t)(r0 + tok);
+        const float inv = (p.off_gate >= 0 && p.head_gate ? gate_sigmoid(p.proj[rr * p.ldp + p.off_gate + h]) : 1.f) / l[row];
         bf16* d = reinterpret_cast<bf16*>(p.out) + rr * p.ldo + (size_t)h * p.dv;
         const float* gt = p.proj + rr * p.ldp + p.off_gate + (size_t)h * p.dv;
 #pragma unroll
@@ -359,7 +359,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
                 const int c = i * 8 + (lane & 3) * 2 + u;
                 if (c < p.dv) {
                     float v = o[i][2 * row + u] * inv;
-                    if (p.off_gate >= 0) v *= gate_sigmoid(gt[c]);
+                    if (p.off_gate >= 0 && !p.head_gate) v *= gate_sigmoid(gt[c]);
                     d[c] = __float2bfloat16(v);
                 }
             }
@@ -420,7 +420,7 @@ LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, 
     p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
     p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 0; p.out = out; p.ldo = ldo;
     p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.rows = rows; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = dkp; p.dvp = dvp;
-    p.ldc = G * (dkp + dvp); p.off_v = G * dkp; p.NS = NS; p.window = window; p.scale = scale; p.slope = (const float*)slope;
+    p.ldc = G * (dkp + dvp); p.off_v = G * dkp; p.dkh = dkp; p.off_ks = 0; p.NS = NS; p.window = window; p.scale = scale; p.slope = (const float*)slope;
     cudaStream_t st = (cudaStream_t)stream;
     const int hg = H / G;
     const bool tc = !f32 && dkp <= 256 && dvp <= 256;
@@ -437,6 +437,27 @@ LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, 
         case 64: return prefill ? launch_prefill<64>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<64>(p, st);
         case 128: return prefill ? launch_prefill<128>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<128>(p, st);
         case 256: return prefill ? launch_prefill<256>(p, (const int*)seq_row0, (const int*)seq_nrows, nseq, st) : launch_decode<256>(p, st);
+    }
+    return -1;
+}
+
+// Attention of one run of rows (positions row_pos, causal) over keys and values written out per head and position: kv [positions, H dkh keys | H dvp values |
+// dks key channels shared by all heads].  q: [rows, H, dkh + dks].  seq_row0 / seq_nrows: the run, as the other kernels take it; page0: a zero (the rows
+// are one page); off_gate: one gate per head (-1: none).
+LSB_API int lsb_attn_run(const void* q, const void* kv, int positions, const void* page0, const void* row_seq, const void* row_pos, const void* seq_row0,
+                         const void* seq_nrows, const void* proj, int ldp, int off_gate, void* out, int ldo, int rows, int H, int dkh, int dks, int dv, int dvp,
+                         float scale, void* stream) {
+    if (rows < 1 || dkh % 16 || dks % 16 || dkh + dks > 256 || dv > dvp) return -1;
+    AttnParams p;
+    p.q = q; p.cache = kv; p.block_table = (const int*)page0; p.max_pages = 0; p.page = positions; p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos;
+    p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.out = out; p.ldo = ldo; p.o_part = p.ml_part = nullptr; p.rows = rows;
+    p.H = p.G = H; p.dk = p.dkp = dkh + dks; p.dv = dv; p.dvp = dvp; p.dkh = dkh; p.off_ks = H * (dkh + dvp); p.ldc = H * (dkh + dvp) + dks; p.off_v = H * dkh;
+    p.NS = 1; p.window = 0; p.scale = scale; p.slope = nullptr;
+    switch (dvp) {
+        case 32: return launch_prefill<32>(p, (const int*)seq_row0, (const int*)seq_nrows, 1, (cudaStream_t)stream);
+        case 64: return launch_prefill<64>(p, (const int*)seq_row0, (const int*)seq_nrows, 1, (cudaStream_t)stream);
+        case 128: return launch_prefill<128>(p, (const int*)seq_row0, (const int*)seq_nrows, 1, (cudaStream_t)stream);
+        case 256: return launch_prefill<256>(p, (const int*)seq_row0, (const int*)seq_nrows, 1, (cudaStream_t)stream);
     }
     return -1;
 }

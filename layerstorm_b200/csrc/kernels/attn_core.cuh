@@ -11,6 +11,7 @@ struct AttnParams {
     const int* row_seq; const int* row_pos;
     const float* proj; int ldp, off_gate, head_gate;     // gate per value channel, or (head_gate) one per head
     int ldc, off_v;                   // cache row: elements, and where the values start (latent rows: 0, the values are the head of the key row)
+    int dkh, off_ks;                  // key channels from dkh on are shared by all heads and start at element off_ks of the row (dkh = dkp: none)
     void* out; int ldo;               // [rows, ldo]
     float* o_part; float* ml_part;    // [rows, H, NS, dvp], [rows, H, NS, 2]
     int rows, H, G, dk, dv, dkp, dvp, NS, window;

@@ -12,6 +12,9 @@
 //   latent_attn     (token, head) rows of a sequence in tiles of 16 MG against key tiles shared by all of them; any mixture of prompt runs and
 //                   single tokens; key splits for small batches: up to eight splits are a thread-block cluster that merges its sums through
 //                   distributed shared memory, what is left (one partial sum per cluster) goes through global memory
+//   latent_rows / latent_gather   long runs of one sequence: keys and values are written out per head for all its positions (one tcgen05
+//                   product over the gathered latents; the rotated part stays shared), and the run goes through the grouped-query prefill kernel (attn.cu) - a third of the
+//                   arithmetic per (query, key) of the absorbed form, for products that do not depend on the number of queries
 //   latent_combine  merge of those partial sums;  latent_out: the same together with the value up-projection (few rows)
 // The value of a key is the head of its cache row, so a key tile is loaded once for both products.
 #include "attn_core.cuh"
@@ -19,6 +22,8 @@
 
 extern "C" int lsb_gemm_bf16_tc_batched(void* out, const void* x, const void* w, int M, int N, int K, int B, int ldx, long long xs_b, int ldw,
                                         long long ws_b, int ldo, long long os_b, int out_bf16, void* err, void* stream);
+extern "C" int lsb_gemm_bf16_tc(void* out, const void* x, const void* w, const void* bias, int M, int N, int K, int ldx, int ldw, int ldo, int out_bf16,
+                                void* partial, long long partial_cap, void* err, const void* comm, void* stream);
 
 namespace lsb {
 namespace cg = cooperative_groups;
@@ -142,6 +147,20 @@ __global__ void __launch_bounds__(256) latent_query_kernel(LatentPrep p) {
     });
 }
 
+// Rotated parts of all heads of a row (dst: rows of ld, src: rows of dn + dr); a thread keeps its rotary pair over the heads: one angle per pair.
+__device__ __forceinline__ void rotated_heads(bf16* dst, int ld, const float* src, const LatentPrep& p, int pos, int hp) {
+    const int t = threadIdx.x, w = min(hp, 256), step = 256 / w, h0 = t / w;
+    for (int i = h0 < step ? t % w : hp; i < hp; i += w) {
+        float cs = 1.f, sn = 0.f;
+        if (2 * i < p.dr) rotate_pair(cs, sn, pos, p.inv_freq[i]);
+        for (int h = h0; h < p.H; h += step) {
+            float a = 0.f, b = 0.f;
+            if (2 * i < p.dr) { const float* s = src + (size_t)h * (p.dn + p.dr) + 2 * i; a = s[0]; b = s[1]; }
+            *reinterpret_cast<bf162*>(dst + (size_t)h * ld + 2 * i) = __floats2bfloat162_rn(a * cs - b * sn, b * cs + a * sn);
+        }
+    }
+}
+
 __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrep p) {
     __shared__ float red[33];
     const int r = blockIdx.x, t = threadIdx.x, D = p.dlp + p.drp, hp = p.drp / 2;
@@ -164,19 +183,43 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrep p) {
             qn[i] = __float2bfloat16(c < p.dn ? src[(size_t)h * (p.dn + p.dr) + c] : 0.f);
         }
     }
-    // a thread keeps its rotary pair over the heads: one angle per pair
-    bf16* q = reinterpret_cast<bf16*>(p.q) + (size_t)r * p.H * D + p.dlp;
-    const int w = min(hp, 256), step = 256 / w, h0 = t / w;
-    for (int i = h0 < step ? t % w : hp; i < hp; i += w) {
-        float cs = 1.f, sn = 0.f;
-        if (2 * i < p.dr) rotate_pair(cs, sn, pos, p.inv_freq[i]);
-        for (int h = h0; h < p.H; h += step) {
-            float a = 0.f, b = 0.f;
-            if (2 * i < p.dr) { const float* s = src + (size_t)h * (p.dn + p.dr) + p.dn + 2 * i; a = s[0]; b = s[1]; }
-            *reinterpret_cast<bf162*>(q + (size_t)h * D + 2 * i) = __floats2bfloat162_rn(a * cs - b * sn, b * cs + a * sn);
-        }
-    }
+    rotated_heads(reinterpret_cast<bf16*>(p.q) + (size_t)r * p.H * D + p.dlp, D, src + p.dn, p, pos, hp);
     if (p.off_kv >= 0) append_row<bf16>(p, r, red);
+}
+
+// ------------------------------------------------------------------------------------------------ keys and values written out per head
+// Row r: q [H, dnw + drp] (unrotated part padded to dnw, rotated part behind it), cache append.
+__global__ void __launch_bounds__(256) latent_rows_kernel(LatentPrep p, int dnw) {
+    __shared__ float red[33];
+    const int r = blockIdx.x, t = threadIdx.x, K = dnw + p.drp, hp = p.drp / 2;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int pos = p.row_pos[r];
+    const float* src = p.proj + (size_t)r * p.ldp + p.off_q;
+    bf16* q = reinterpret_cast<bf16*>(p.q) + (size_t)r * p.H * K;
+    for (int i = t; i < p.H * (dnw / 2); i += 256) {
+        const int h = i / (dnw / 2), c = (i - h * (dnw / 2)) * 2;
+        const float* s = src + (size_t)h * (p.dn + p.dr) + c;
+        *reinterpret_cast<bf162*>(q + (size_t)h * K + c) = __floats2bfloat162_rn(c < p.dn ? s[0] : 0.f, c + 1 < p.dn ? s[1] : 0.f);
+    }
+    rotated_heads(q + dnw, K, src + p.dn, p, pos, hp);
+    if (p.off_kv >= 0) append_row<bf16>(p, r, red);
+}
+
+// Cached rows of positions [0, T) of one sequence: the latents to lat [T, dlp], the rotated part to column off_rot of kv's rows.  One warp per position.
+__global__ void __launch_bounds__(128) latent_gather_kernel(const bf16* __restrict__ cache, const int* __restrict__ block_table, int max_pages, int page,
+                                                            const int* __restrict__ row_seq, int T, int dlp, int drp, bf16* __restrict__ lat,
+                                                            bf16* __restrict__ kv, int ldkv, int off_rot) {
+    const int j = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = row_seq[0];
+    if (seq < 0 || j >= T) return;
+    const uint4* src = reinterpret_cast<const uint4*>(cache + ((size_t)block_table[(size_t)seq * max_pages + j / page] * page + j % page) * (dlp + drp));
+    for (int i = lane; i < (dlp + drp) / 8; i += 32) {
+        if (i < dlp / 8) reinterpret_cast<uint4*>(lat + (size_t)j * dlp)[i] = src[i];
+        else reinterpret_cast<uint4*>(kv + (size_t)j * ldkv + off_rot)[i - dlp / 8] = src[i];
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ attention (mma.sync m16n8k16)
@@ -591,6 +634,16 @@ static int launch_latent_rows(const LatentAttn& p, int mg, int tiles, cudaStream
     return mg == 1 ? launch_latent<NV, 1>(p, tiles, st) : (mg == 2 ? launch_latent<NV, 2>(p, tiles, st) : launch_latent<NV, 4>(p, tiles, st));
 }
 static int row_tiles(int run_rows, int H) { return run_rows * H <= 16 ? 1 : (run_rows * H <= 32 ? 2 : 4); }
+static LatentPrep latent_prep_params(const void* proj, int ldp, int off_q, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_uk, void* q,
+                                     void* q_nope, void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
+                                     int rows, int H, int dn, int dnp, int dr, int dl) {
+    LatentPrep p;
+    p.proj = (const float*)proj; p.ldp = ldp; p.off_q = off_q; p.off_kv = off_kv; p.kv_norm = (const float*)kv_norm; p.eps = eps;
+    p.inv_freq = (const double*)inv_freq; p.w_uk = w_uk; p.q = q; p.q_nope = (bf16*)q_nope; p.cache = cache; p.block_table = (const int*)block_table;
+    p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos; p.rows = rows; p.H = H; p.dn = dn;
+    p.dnp = dnp; p.dr = dr; p.drp = (dr + 15) / 16 * 16; p.dl = dl; p.dlp = (dl + 15) / 16 * 16;
+    return p;
+}
 constexpr int kMaxSplits = 128;
 static int cluster_of(int NS) { return NS >= 8 ? 8 : NS; }
 static bool splits_ok(int NS) { return NS == 1 || NS == 2 || NS == 4 || (NS >= 8 && NS % 8 == 0 && NS <= kMaxSplits); }
@@ -620,11 +673,8 @@ LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, c
                              void* q, void* q_nope, void* cache, const void* block_table, int max_pages, int page, const void* row_seq,
                              const void* row_pos, int rows, int H, int dn, int dnp, int dr, int dl, int f32, void* err, void* stream) {
     if (rows < 1 || dnp % 8 || dnp < dn || dr % 2 || dr < 1 || dl < 1) return -1;
-    LatentPrep p;
-    p.proj = (const float*)proj; p.ldp = ldp; p.off_q = off_q; p.off_kv = off_kv; p.kv_norm = (const float*)kv_norm; p.eps = eps;
-    p.inv_freq = (const double*)inv_freq; p.w_uk = w_uk; p.q = q; p.q_nope = (bf16*)q_nope; p.cache = cache; p.block_table = (const int*)block_table;
-    p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos; p.rows = rows; p.H = H; p.dn = dn;
-    p.dnp = dnp; p.dr = dr; p.drp = lsb_latent_pad(dr); p.dl = dl; p.dlp = lsb_latent_pad(dl);
+    const LatentPrep p = latent_prep_params(proj, ldp, off_q, off_kv, kv_norm, eps, inv_freq, w_uk, q, q_nope, cache, block_table, max_pages, page, row_seq, row_pos,
+                                            rows, H, dn, dnp, dr, dl);
     cudaStream_t st = (cudaStream_t)stream;
     if (!f32 && rows >= 8) {
         const int D = p.dlp + p.drp;
@@ -641,6 +691,24 @@ LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, c
     else { if (mt == 4) LSB_LQ(bf16, 4); else if (mt == 2) LSB_LQ(bf16, 2); else LSB_LQ(bf16, 1); }
 #undef LSB_LQ
     LSB_CHECK_LAUNCH();
+}
+
+// A run of rows of one sequence (row_pos consecutive, T positions in all after the append) with keys and values written out per head: q [rows, H, dnw + drp];
+// kv [Tm, H dnw unrotated keys | H dvp values | drp shared rotated part], read by lsb_attn_run.  w_kv: [H dnw + H dvp, dlp], padding rows and columns zero;
+// lat: scratch [Tm, dlp].  Tm >= T: positions the product runs over (those past T are never read).
+LSB_API int lsb_latent_expand(const void* proj, int ldp, int off_q, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_kv,
+                              void* q, void* lat, void* kv, void* cache, const void* block_table, int max_pages, int page, const void* row_seq,
+                              const void* row_pos, int rows, int T, int Tm, int H, int dn, int dnw, int dr, int dl, int dvp, void* err, void* stream) {
+    if (rows < 1 || T < rows || Tm < T || dnw % 16 || dnw < dn || dvp % 16 || dr % 2 || dr < 1 || dl < 1) return -1;
+    const LatentPrep p = latent_prep_params(proj, ldp, off_q, off_kv, kv_norm, eps, inv_freq, nullptr, q, nullptr, cache, block_table, max_pages, page, row_seq, row_pos,
+                                            rows, H, dn, dnw, dr, dl);
+    cudaStream_t st = (cudaStream_t)stream;
+    const int N = H * (dnw + dvp), ldkv = N + p.drp;
+    launch_pdl((latent_rows_kernel), rows, 256, 0, st, p, dnw);
+    launch_pdl((latent_gather_kernel), (T + 3) / 4, 128, 0, st, (const bf16*)cache, (const int*)block_table, max_pages, page, (const int*)row_seq, T, p.dlp, p.drp,
+               (bf16*)lat, (bf16*)kv, ldkv, N);
+    const int rc = lsb_gemm_bf16_tc(kv, lat, w_kv, nullptr, Tm, N, p.dlp, p.dlp, p.dlp, ldkv, 1, nullptr, 0, err, nullptr, stream);
+    return rc ? rc : (int)cudaGetLastError();
 }
 
 // Attention of the step's rows.  NS: key splits (lsb_latent_splits; runs of rows use 1).  One partial sum: o_lat [rows, H, dlp], gated; more: o_part /
@@ -669,7 +737,7 @@ LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_
     if (NS != 1) return -1;
     AttnParams p;
     p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
-    p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.ldc = D; p.off_v = 0;
+    p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.ldc = p.dkh = D; p.off_v = p.off_ks = 0;
     p.out = o_lat; p.ldo = H * dlp; p.o_part = p.ml_part = nullptr; p.rows = rows; p.H = H; p.G = 1; p.dk = p.dkp = D; p.dv = p.dvp = dlp; p.NS = 1;
     p.window = 0; p.scale = scale; p.slope = nullptr;
     const size_t smem = (size_t)(D + 256 + dlp) * 4;

@@ -30,6 +30,8 @@ from .device_model import ExpertArena, ModelBase, MoeBuffers, QLinear, StepBuffe
 
 FEW_ROWS = 8            # rows per sequence up to which a delta-rule layer runs as one kernel
 LONG_ROWS = 64          # rows of a sequence from which its recurrence runs chunk-parallel
+EXPAND_ROWS = 128       # rows of a step of one sequence from which latent layers write keys and values out per head ...
+EXPAND_BYTES = 1 << 30  # ... while those of all its positions fit this much scratch
 NORM_KIND = {"rms": 0, "layer": 1, "tanh": 2}        # as the kernels number them; 3: none
 NO_NORM = (3, None, None, None)
 
@@ -213,6 +215,7 @@ class BlockModel(ModelBase):
         self.w_fmt = "f32" if self.f32 else "bf16"
         self.expert_shard = "ep"
         self.Hp = _align(cfg.hidden, 8)
+        self.zero, self._expand = torch.zeros(1, dtype=torch.int32, device=self.device), None
         self.max_mix = 8
         mixing = [i for i, b in enumerate(cfg.blocks) if b.v_mix and b.kind == "attention"]
         self.v_first_layer = mixing[0] if mixing else -1
@@ -331,6 +334,12 @@ class BlockModel(ModelBase):
                 L["w_uk"][:, : b.kv_rank, : b.dim] = uk.transpose(1, 2)
                 L["w_uv"] = torch.zeros(b.heads, b.vdim, dlp, dtype=m.act_dtype, device=dev)
                 L["w_uv"][:, :, : b.kv_rank] = uv
+                if not m.f32:
+                    # the same two, one after the other per position: what long prompt runs make keys and values with
+                    dnw, dvp = _align(b.dim, 16), m.head_pad(b.vdim)
+                    L["w_kv"] = torch.zeros(b.heads * (dnw + dvp), dlp, dtype=m.act_dtype, device=dev)
+                    L["w_kv"][: b.heads * dnw].view(b.heads, dnw, dlp)[:, : b.dim, : b.kv_rank] = uk
+                    L["w_kv"][b.heads * dnw:].view(b.heads, dvp, dlp)[:, : b.vdim, : b.kv_rank] = uv
                 if own:
                     L["kv_norm"] = m._vec(w[a + "kv_a_norm"])
                 L["inv_freq"] = torch.tensor([b.rot_base ** (-2.0 * j / b.rot_dim) for j in range(b.rot_dim // 2)], dtype=torch.float64, device=dev)
@@ -439,6 +448,17 @@ class BlockModel(ModelBase):
         cache = self.kv_cache[i if b.kv_from < 0 else b.kv_from]
         L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
         err = TcScratch.get(self.device).err
+        T = ws.ne_hint                                             # positions of the step's (longest) sequence
+        if nseq == 1 and self._expands(b, R, T):
+            # the run attends over keys and values of every head, made for this step from the cached rows
+            dnw, dvp, drp = _align(b.dim, 16), self.head_pad(b.vdim), self.latent_pad(b.rot_dim)
+            Tm, width = _align(T, 256), b.heads * (dnw + dvp) + drp
+            q, lat, kv = self._expand_scratch(R * b.heads * (dnw + drp), Tm * self.latent_pad(b.kv_rank), Tm * width)
+            nat.call("lsb_latent_expand", ws.proj, self.max_proj, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_kv"], q, lat, kv, cache,
+                     self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, R, T, Tm, b.heads, b.dim, dnw, b.rot_dim, b.kv_rank, dvp, err)
+            nat.call("lsb_attn_run", q, kv, Tm, self.zero, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, ws.proj, self.max_proj, og, ws.mix, L["out"].K, R,
+                     b.heads, dnw, drp, b.vdim, dvp, b.scale)
+            return
         nat.call("lsb_latent_query", ws.proj, self.max_proj, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], ws.q_lat, ws.q_nope, cache,
                  self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, R, b.heads, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank,
                  int(self.f32), err)
@@ -447,6 +467,23 @@ class BlockModel(ModelBase):
                  b.scale, int(self.f32))
         nat.call("lsb_latent_out", ws.mix, L["out"].K, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_parts[i], L["w_uv"], ws.proj, self.max_proj, og,
                  ws.row_seq, R, b.heads, b.kv_rank, b.vdim, int(self.f32), err)
+
+    def _expands(self, b: BlockSpec, R: int, T: int) -> bool:
+        """Whether a run of R rows over T positions is worth writing keys and values out for (and the kernels take the sizes): fewer operations per
+        (query, key), against a product over all positions that runs about four times as fast per operation."""
+        dnw, dvp = _align(b.dim, 16), self.head_pad(b.vdim)
+        row = b.heads * (dnw + dvp) + self.latent_pad(b.rot_dim)
+        return (not self.f32 and R >= EXPAND_ROWS and dnw + self.latent_pad(b.rot_dim) <= 256 and dvp <= 256 and 2 * T * row <= EXPAND_BYTES
+                and R * (2 * b.kv_rank - b.dim - b.vdim) * 4 > (b.dim + b.vdim) * b.kv_rank)
+
+    def _expand_scratch(self, *sizes: int) -> list:
+        """bf16 scratch of long prompt runs, shared by the layers (made when the first such run comes)."""
+        at = [0]
+        for n in sizes:
+            at.append(at[-1] + _align(n, 64))
+        if self._expand is None or self._expand.numel() < at[-1]:
+            self._expand = torch.empty(at[-1] * 5 // 4, dtype=torch.bfloat16, device=self.device)
+        return [self._expand[a: a + n] for a, n in zip(at, sizes)]
 
     def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
         mt = L["meta"]

@@ -515,11 +515,14 @@ class Engine:
         h = ws.h_ring[k]
         h.zero_()
         h[1].fill_(-1)
-        for r, (tok, slot, pos) in enumerate(rows):
-            h[0, r] = tok; h[1, r] = slot; h[2, r] = pos; h[3, r] = pos + 1; h[4, r] = slot
-            h[5, r] = (pos + 1) // P
-        for j, (r0, n, slot) in enumerate(seq_groups):
-            h[6, j] = r0; h[7, j] = n; h[8, j] = slot
+        if rows:
+            t = torch.tensor(rows, dtype=torch.int32).T             # token, slot, position
+            h[0:3, :R] = t
+            h[3, :R] = t[2] + 1
+            h[4, :R] = t[1]
+            h[5, :R] = (t[2] + 1) // P
+        if seq_groups:
+            h[6:9, : len(seq_groups)] = torch.tensor(seq_groups, dtype=torch.int32).T
         # host-side facts about the step that size kernels' grids: the largest index-entry count of a row, one sequence or several
         ws.ne_hint = max((pos + 1) // P for (_, _, pos) in rows) if rows else 0
         ws.seq_rows = [n for (_, n, _) in seq_groups]

@@ -130,6 +130,8 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
     experts = TOP + cfg.n_shared
     if att is not None and att.latent:
         out["lsb_latent_attn"], out["lsb_latent_query"], out["lsb_latent_out"] = latent, absorb, up
+        out["lsb_latent_expand"] = ("flops", 2 * ctx * ah * lat * (dn + dv))
+        out["lsb_attn_run"] = ("flops", 2 * rows * seen * ah * (dn + rot + dv))
         out["lsb_resid_update"] = ("bytes", rows * H * 14)
         out["lsb_glu"] = ("bytes", rows * cfg.moe_inter * 10)
     elif att is not None:

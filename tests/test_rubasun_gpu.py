@@ -150,6 +150,35 @@ def test_latent_attention_sees_far_keys_and_nothing_ahead(H, dn, dr, dv, dl, f32
     assert err(out.view(2, H, dv) * gt, ref[0][88:90].view(2, H, dv)) < tol
 
 
+@pytest.mark.parametrize("H,dn,dr,dv,dl", [g for g in GEOMETRIES if g[1] + g[2] <= 230])
+def test_long_runs_over_written_out_keys_and_values(H, dn, dr, dv, dl):
+    """The same standing keys through per-head keys and values: a whole prompt, then portions that start inside a page, on rows that were appended
+    before and rows of another layer."""
+    T, page, base, scale = 150, 16, 300.0, 0.9
+    (d,), (uk, uv, kvn) = standing_keys(H, dn, dr, dv, dl, [T], False, base, page, torch.Generator().manual_seed(H * 100 + dn))
+    ref = reference(H, dn, dr, dv, dl, *d, uk, uv, kvn, scale, base)
+    P = Paged(H, dn, dr, dv, dl, page, [T, T], False, base).weights(uk, uv, kvn)
+    up = lambda n: (n + 15) // 16 * 16
+    dnw, dvp, drp = up(dn), nat.call("lsb_attn_head_pad", dv), up(dr)
+    w = torch.zeros(H * (dnw + dvp), P.dlp, dtype=B16, device=DEV)
+    w[: H * dnw].view(H, dnw, P.dlp)[:, :dn, :dl] = uk.view(H, dn, dl).to(DEV)
+    w[H * dnw:].view(H, dvp, P.dlp)[:, :dv, :dl] = uv.view(H, dv, dl).to(DEV)
+    e, ldo = torch.zeros(1, dtype=I32, device=DEV), (H * dv + 7) // 8 * 8
+    for a, b, own in ((0, T, True), (0, 70, True), (70, 73, True), (73, T, True), (20, 101, False)):
+        proj = torch.cat([t[a:b] for t in d], 1).to(DEV).contiguous()
+        R, Tm = b - a, (b + 255) // 256 * 256
+        z = lambda *s: torch.full(s, float("nan"), dtype=B16, device=DEV)
+        q, lat, kv, out = z(R, H, dnw + drp), z(Tm, P.dlp), z(Tm, H * (dnw + dvp) + drp), z(R, ldo)
+        seq, pos = i32([1] * R), i32(list(range(a, b)))
+        oq, oy, og = 0, H * (dn + dr), H * (dn + dr) + dl + dr
+        nat.call("lsb_latent_expand", proj, proj.shape[1], oq, oy if own else -1, P.kv_norm, 1e-5, P.inv_freq, w, q, lat, kv, P.cache, P.bt, P.max_pages, page,
+                 seq, pos, R, b, Tm, H, dn, dnw, dr, dl, dvp, e)
+        nat.call("lsb_attn_run", q, kv, Tm, i32([0]), seq, pos, i32([0]), i32([R]), proj, proj.shape[1], og, out, ldo, R, H, dnw, drp, dv, dvp, scale)
+        torch.cuda.synchronize()
+        assert int(e[0]) == 0
+        assert err(out[:, : H * dv], ref[a:b]) < (2e-2 if dl > 32 else 6e-2), (a, b)
+
+
 @pytest.mark.parametrize("f32", [True, False])
 def test_rotations_stay_exact_at_far_positions(f32):
     """Queries and rows from position 250 000 on: angles of every pair against fp64."""
@@ -348,6 +377,24 @@ def test_prompts_portions_and_decoding_match_the_oracle(tmp_path_factory, name, 
         assert e < TOL[dtype], (cuts, dec, e)
         assert eng.seq_len(sid) == LONG
         eng.free_sequence(sid)
+
+
+@pytest.mark.parametrize("name", ["odd", "tiles", "wide"])
+def test_long_portions_match_the_oracle(tmp_path_factory, name):
+    """Portions of 128 rows and more beside shorter ones, alone and with another request's tokens in the step."""
+    c, m, toks, ref = load(tmp_path_factory, name, "bfloat16")
+    eng = engine(m, prefill_chunk=256)
+    assert sum(m._expands(b, 140, LONG) for b in m.cfg.blocks) >= 1
+    for cuts in ([LONG], [140, 60], [33, 129, 38], [128, 1, 2, 69]):
+        sid = eng.create_sequence()
+        e = rms(feed(eng, sid, toks[0], cuts), ref[0])
+        assert e < TOL["bfloat16"], (cuts, e)
+        eng.free_sequence(sid)
+    a, b = eng.create_sequence(), eng.create_sequence()
+    res = eng.step([Portion(a, toks[0][:150], list(range(150))), Portion(b, toks[1][:9], [8])], return_logits=True)
+    assert rms(res[0][1], ref[0][:150]) < TOL["bfloat16"] and rms(res[1][1], ref[1][8:9]) < TOL["bfloat16"]
+    _, lg = eng.prefill(b, toks[1][9:], want_logits=True)
+    assert rms(lg[None], ref[1][-1:]) < TOL["bfloat16"]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
