@@ -644,7 +644,7 @@ static LatentPrep latent_prep_params(const void* proj, int ldp, int off_q, int o
     p.dnp = dnp; p.dr = dr; p.drp = (dr + 15) / 16 * 16; p.dl = dl; p.dlp = (dl + 15) / 16 * 16;
     return p;
 }
-constexpr int kMaxSplits = 128;
+constexpr int kMaxSplits = 128;       // sixteen clusters' partial sums
 static int cluster_of(int NS) { return NS >= 8 ? 8 : NS; }
 static bool splits_ok(int NS) { return NS == 1 || NS == 2 || NS == 4 || (NS >= 8 && NS % 8 == 0 && NS <= kMaxSplits); }
 // the tensor-core kernel covers latents of up to 512 channels whose tiles fit an SM's shared memory
@@ -660,10 +660,13 @@ LSB_API int lsb_latent_pad(int d) { return (d + 15) / 16 * 16; }
 LSB_API int lsb_latent_splits(int rows, int H, int dl, int dr, int seen, int f32) {
     if (!latent_tc((dl + 15) / 16 * 16, (dr + 15) / 16 * 16, f32)) return 1;
     const int mg = row_tiles(1, H), blocks = rows * ((H + 16 * mg - 1) / (16 * mg)), kt = mg == 4 ? 32 : 64;
-    int ns = 148 / blocks;
-    if (ns > (seen + kt - 1) / kt) ns = (seen + kt - 1) / kt;
-    if (ns > kMaxSplits) ns = kMaxSplits;
-    return ns >= 8 ? ns / 8 * 8 : (ns >= 4 ? 4 : (ns >= 2 ? 2 : 1));
+    const int most = (seen + kt - 1) / kt;                        // no split shorter than a key tile
+    // clusters of eight: 14 of them are resident at a time, 16 are not; 12 leave the merge less to add up (one row of 16 heads, 8192 keys, both kernels:
+    // 20.8 us with 64 splits, 22.0 with 96, 22.8 with 112, 27.3 with 128; a few keys more and 64 splits have three tiles each instead of two)
+    int ns = 96 / blocks < most ? 96 / blocks : most;
+    if (ns >= 8) return ns / 8 * 8;
+    ns = 148 / blocks < most ? 148 / blocks : most;
+    return ns >= 4 ? 4 : (ns >= 2 ? 2 : 1);
 }
 // Partial sums per (row, head) that NS splits leave to lsb_latent_out (1: none, the attention kernel writes its result): o_part [rows, H, this, dlp].
 LSB_API int lsb_latent_partials(int NS) { return NS / cluster_of(NS); }

@@ -24,8 +24,8 @@ struct GluAct { float limit, alpha, shift; const float* in_scale; };
 #ifdef __CUDACC__
 template <bool EXACT = false> __device__ __forceinline__ float glu_act(float g, float u, const GluAct& a) {
     if (a.limit > 0.f) { g = fminf(g, a.limit); u = fminf(fmaxf(u, -a.limit), a.limit); }
-    const float e = EXACT ? expf(-a.alpha * g) : __expf(-a.alpha * g);
-    return g / (1.f + e) * (u + a.shift);
+    if (EXACT) return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);
+    return __fdividef(g, 1.f + __expf(-a.alpha * g)) * (u + a.shift);
 }
 __device__ __forceinline__ float glu_in_scale(const GluAct& a, int pair) { return a.in_scale ? a.in_scale[pair] : 1.f; }
 #endif

@@ -580,10 +580,11 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
             const uint8_t* base = p.arena + (size_t)slot * p.ef.stride;
             const uint32_t buf = lt % C::NBUF;
             // the columns' factors on the experts' inputs, fetched while the tile is being computed
+            const bool scaled = GATEUP && p.ga.in_scale != nullptr;
             float in_scale[BN / 32];
 #pragma unroll
             for (int g = 0; g < BN / 32; ++g)
-                in_scale[g] = GATEUP && p.ga.in_scale && g * 32 + lane < ncols ? p.ga.in_scale[p.sorted_pair[row0 + g * 32 + lane]] : 1.f;
+                in_scale[g] = scaled && g * 32 + lane < ncols ? p.ga.in_scale[p.sorted_pair[row0 + g * 32 + lane]] : 1.f;
             int okw = 1;
             if (lane == 0) { if (q == 0) PROF_SCOPE(0, okw = mbar_wait_relaxed(&acc_full[buf], (lt / C::NBUF) & 1u, p.err, 14) ? 1 : 0); else okw = mbar_wait_relaxed(&acc_full[buf], (lt / C::NBUF) & 1u, p.err, 14) ? 1 : 0; }
             ok = __shfl_sync(0xffffffffu, okw, 0) != 0;
@@ -610,7 +611,7 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                     for (int g = 1; g < BN / 32; ++g) cs = (c0 >> 5) == g ? in_scale[g] : cs;
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        const float c = GATEUP ? __shfl_sync(0xffffffffu, cs, (c0 + j) & 31) : 1.f;
+                        const float c = GATEUP && scaled ? __shfl_sync(0xffffffffu, cs, (c0 + j) & 31) : 1.f;
                         if (c0 + j < ncols && n < NOUT) {
                             if (GATEUP) {
                                 p.act[(size_t)(row0 + c0 + j) * NOUT + n] = __float2half_rn(glu_act(gq[j] * sg * c, uq[j] * su * c, p.ga));

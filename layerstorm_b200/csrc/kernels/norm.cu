@@ -785,7 +785,8 @@ __device__ __forceinline__ float sum_slots(float a, const MoeSum& mo, const floa
 }
 
 // resid[r] += post(sub[r] + MoE sum of the row), x[r] = pre(the new residual) in the activation type.  sub may be null.  Whole rows per block.
-template <typename T, bool MOE>
+// PLAIN: post is an RMS or layer norm and there is no pre norm.
+template <typename T, bool MOE, bool PLAIN>
 __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
                                                         NormW post, NormW pre, MoeSum mo) {
     __shared__ float red[33], s_w[32];
@@ -813,6 +814,14 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int 
     norm_moments(row, post, red, mean, rstd);
     const float a_post = post.alpha ? *post.alpha : 0.f, a_pre = pre.alpha ? *pre.alpha : 0.f;
     T* xr = x + (size_t)r * ldx;
+    if constexpr (PLAIN) {
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+            const float v = rr[i] + ((row[i] - mean) * rstd * post.w[i] + (post.b ? post.b[i] : 0.f));
+            rr[i] = v;
+            xr[i] = as_act<T>(v);
+        }
+        return;
+    }
     const bool again = norm_moments_needed(pre.kind);
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
         const float v = rr[i] + norm_apply(row[i], i, post, mean, rstd, a_post);
@@ -894,10 +903,13 @@ static int residual_update(void* x, int ldx, void* resid, int ldr, const void* s
 #undef LSB_PW
         LSB_CHECK_LAUNCH();
     }
-#define LSB_PN(T, M) launch_pdl((post_norm_kernel<T, M>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
-    if (f32) { if (mo.y) LSB_PN(float, true); else LSB_PN(float, false); }
-    else { if (mo.y) LSB_PN(bf16, true); else LSB_PN(bf16, false); }
+    const bool plain = norm_moments_needed(post.kind) && pre.kind == kNormNone;
+#define LSB_PN(T, M) if (plain) LSB_PM(T, M, true); else LSB_PM(T, M, false)
+#define LSB_PM(T, M, P) launch_pdl((post_norm_kernel<T, M, P>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
+    if (f32) { if (mo.y) { LSB_PN(float, true); } else { LSB_PN(float, false); } }
+    else { if (mo.y) { LSB_PN(bf16, true); } else { LSB_PN(bf16, false); } }
 #undef LSB_PN
+#undef LSB_PM
     LSB_CHECK_LAUNCH();
 }
 }  // namespace lsb

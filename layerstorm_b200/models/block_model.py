@@ -215,7 +215,7 @@ class BlockModel(ModelBase):
         self.w_fmt = "f32" if self.f32 else "bf16"
         self.expert_shard = "ep"
         self.Hp = _align(cfg.hidden, 8)
-        self.zero, self._expand = torch.zeros(1, dtype=torch.int32, device=self.device), None
+        self.zero, self._expand, self._expand_rows = torch.zeros(1, dtype=torch.int32, device=self.device), None, 0
         self.max_mix = 8
         mixing = [i for i, b in enumerate(cfg.blocks) if b.v_mix and b.kind == "attention"]
         self.v_first_layer = mixing[0] if mixing else -1
@@ -444,29 +444,46 @@ class BlockModel(ModelBase):
                  b.window, b.scale, L.get("slope"), int(self.f32))
 
     def _latent(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
-        oq, okv, og = L["meta"].offs
         cache = self.kv_cache[i if b.kv_from < 0 else b.kv_from]
         L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
-        err = TcScratch.get(self.device).err
-        T = ws.ne_hint                                             # positions of the step's (longest) sequence
-        if nseq == 1 and self._expands(b, R, T):
-            # the run attends over keys and values of every head, made for this step from the cached rows
-            dnw, dvp, drp = _align(b.dim, 16), self.head_pad(b.vdim), self.latent_pad(b.rot_dim)
-            Tm, width = _align(T, 256), b.heads * (dnw + dvp) + drp
-            q, lat, kv = self._expand_scratch(R * b.heads * (dnw + drp), Tm * self.latent_pad(b.kv_rank), Tm * width)
-            nat.call("lsb_latent_expand", ws.proj, self.max_proj, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_kv"], q, lat, kv, cache,
-                     self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, R, T, Tm, b.heads, b.dim, dnw, b.rot_dim, b.kv_rank, dvp, err)
-            nat.call("lsb_attn_run", q, kv, Tm, self.zero, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, ws.proj, self.max_proj, og, ws.mix, L["out"].K, R,
-                     b.heads, dnw, drp, b.vdim, dvp, b.scale)
-            return
-        nat.call("lsb_latent_query", ws.proj, self.max_proj, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], ws.q_lat, ws.q_nope, cache,
-                 self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, R, b.heads, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank,
-                 int(self.f32), err)
-        nat.call("lsb_latent_attn", ws.q_lat, cache, self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
-                 max(ws.seq_rows), ws.proj, self.max_proj, og, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], R, b.heads, b.kv_rank, b.rot_dim,
-                 b.scale, int(self.f32))
-        nat.call("lsb_latent_out", ws.mix, L["out"].K, ws.o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_parts[i], L["w_uv"], ws.proj, self.max_proj, og,
-                 ws.row_seq, R, b.heads, b.kv_rank, b.vdim, int(self.f32), err)
+        # long runs one by one, what lies between them together
+        rows, row0, j = ws.seq_rows, 0, 0
+        while j < nseq:
+            k, n = j + 1, rows[j]
+            if self._expands(b, rows[j], ws.seq_end[j]):
+                self._latent_run(b, L, ws, cache, row0, n, j)
+            else:
+                while k < nseq and not self._expands(b, rows[k], ws.seq_end[k]):
+                    n, k = n + rows[k], k + 1
+                self._latent_rows(i, b, L, ws, cache, row0, n, j, k)
+            row0, j = row0 + n, k
+
+    def _latent_rows(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, r0: int, R: int, j: int, k: int):
+        """Step rows [r0, r0 + R) (sequences j .. k - 1 of the step) in the latent space."""
+        oq, okv, og = L["meta"].offs
+        H, ld, K, f32, err = b.heads, self.max_proj, L["out"].K, int(self.f32), TcScratch.get(self.device).err
+        q, o_lat, proj, seq, pos = ws.q_lat[r0 * H * self.latent_row(b):], ws.o_lat[r0 * H * L["w_uv"].shape[2]:], ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
+        nat.call("lsb_latent_query", proj, ld, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], q, ws.q_nope, cache, self.block_table,
+                 self.max_pages, self.page, seq, pos, R, H, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank, f32, err)
+        # seq_row0 holds row numbers of the step, so runs get the whole buffers (steps with key splits have no long runs: r0 is 0)
+        run = max(ws.seq_rows[j:k])
+        rows = (q, proj, seq, pos, o_lat) if run == 1 else (ws.q_lat, ws.proj, ws.row_seq, ws.row_pos, ws.o_lat)
+        nat.call("lsb_latent_attn", rows[0], cache, self.block_table, self.max_pages, self.page, rows[2], rows[3], ws.seq_row0[j:], ws.seq_nrows[j:], k - j, run,
+                 rows[1], ld, og, rows[4], ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], R, H, b.kv_rank, b.rot_dim, b.scale, f32)
+        nat.call("lsb_latent_out", ws.mix.view(-1)[r0 * K:], K, o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_parts[i], L["w_uv"], proj, ld, og, seq, R, H, b.kv_rank,
+                 b.vdim, f32, err)
+
+    def _latent_run(self, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, r0: int, R: int, j: int):
+        """Step rows [r0, r0 + R), a run of sequence j, over keys and values of every head, made for this step from the cached rows."""
+        oq, okv, og = L["meta"].offs
+        H, ld, K, err, T = b.heads, self.max_proj, L["out"].K, TcScratch.get(self.device).err, ws.seq_end[j]
+        dnw, dvp, drp = _align(b.dim, 16), self.head_pad(b.vdim), self.latent_pad(b.rot_dim)
+        Tm, proj, seq, pos = _align(T, 256), ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
+        q, lat, kv = self._expand_scratch(ws.R, R * H * (dnw + drp), Tm * self.latent_pad(b.kv_rank), Tm * (H * (dnw + dvp) + drp))
+        nat.call("lsb_latent_expand", proj, ld, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_kv"], q, lat, kv, cache, self.block_table,
+                 self.max_pages, self.page, seq, pos, R, T, Tm, H, b.dim, dnw, b.rot_dim, b.kv_rank, dvp, err)
+        nat.call("lsb_attn_run", q, kv, Tm, self.zero, seq, pos, self.zero, ws.seq_nrows[j:], proj, ld, og, ws.mix.view(-1)[r0 * K:], K, R, H, dnw, drp, b.vdim, dvp,
+                 b.scale)
 
     def _expands(self, b: BlockSpec, R: int, T: int) -> bool:
         """Whether a run of R rows over T positions is worth writing keys and values out for (and the kernels take the sizes): fewer operations per
@@ -476,13 +493,20 @@ class BlockModel(ModelBase):
         return (not self.f32 and R >= EXPAND_ROWS and dnw + self.latent_pad(b.rot_dim) <= 256 and dvp <= 256 and 2 * T * row <= EXPAND_BYTES
                 and R * (2 * b.kv_rank - b.dim - b.vdim) * 4 > (b.dim + b.vdim) * b.kv_rank)
 
-    def _expand_scratch(self, *sizes: int) -> list:
-        """bf16 scratch of long prompt runs, shared by the layers (made when the first such run comes)."""
+    def _expand_scratch(self, R: int, *sizes: int) -> list:
+        """bf16 scratch of long prompt runs, shared by the layers: made once, for the most rows and positions such runs can have."""
+        if self._expand is None or R > self._expand_rows:
+            need = 0
+            for b in self.cfg.blocks:
+                if b.latent:
+                    dnw, drp, dlp = _align(b.dim, 16), self.latent_pad(b.rot_dim), self.latent_pad(b.kv_rank)
+                    row = b.heads * (dnw + self.head_pad(b.vdim)) + drp
+                    T = _align(min(self.max_pages * self.page, EXPAND_BYTES // (2 * row)), 256)
+                    need = max(need, R * b.heads * (dnw + drp) + T * (dlp + row))
+            self._expand, self._expand_rows = torch.empty(need + 192, dtype=torch.bfloat16, device=self.device), R
         at = [0]
         for n in sizes:
             at.append(at[-1] + _align(n, 64))
-        if self._expand is None or self._expand.numel() < at[-1]:
-            self._expand = torch.empty(at[-1] * 5 // 4, dtype=torch.bfloat16, device=self.device)
         return [self._expand[a: a + n] for a, n in zip(at, sizes)]
 
     def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):

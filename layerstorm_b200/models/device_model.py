@@ -528,8 +528,9 @@ class StepBuffers:
         self.inp[1].fill_(-1)
         (self.tok, self.row_seq, self.row_pos, self.row_len, self.row_slot, self.n_entries,
          self.seq_row0, self.seq_nrows, self.seq_slot) = (self.inp[j] for j in range(9))
-        # host-side facts of the staged step (Engine._stage): largest index-entry count of a row, one sequence or several, rows per sequence
-        self.ne_hint, self.single_seq, self.seq_rows = 0, False, [1] * R
+        # host-side facts of the staged step (Engine._stage): largest index-entry count of a row, one sequence or several, rows per sequence and
+        # positions each has after the step
+        self.ne_hint, self.single_seq, self.seq_rows, self.seq_end = 0, False, [1] * R, [1] * R
         # outputs
         self.n_logit_rows = n_logit_rows
         self.logits = self.z(n_logit_rows, m.V_local)

@@ -526,6 +526,7 @@ class Engine:
         # host-side facts about the step that size kernels' grids: the largest index-entry count of a row, one sequence or several
         ws.ne_hint = max((pos + 1) // P for (_, _, pos) in rows) if rows else 0
         ws.seq_rows = [n for (_, n, _) in seq_groups]
+        ws.seq_end = [rows[r0 + n - 1][2] + 1 for (r0, n, _) in seq_groups]
         ws.single_seq = len(seq_groups) == 1 and len({slot for (_, slot, _) in rows}) == 1
         ws.inp.copy_(h, non_blocking=True)
         ev = torch.cuda.Event()

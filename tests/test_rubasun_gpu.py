@@ -390,10 +390,17 @@ def test_long_portions_match_the_oracle(tmp_path_factory, name):
         e = rms(feed(eng, sid, toks[0], cuts), ref[0])
         assert e < TOL["bfloat16"], (cuts, e)
         eng.free_sequence(sid)
-    a, b = eng.create_sequence(), eng.create_sequence()
-    res = eng.step([Portion(a, toks[0][:150], list(range(150))), Portion(b, toks[1][:9], [8])], return_logits=True)
-    assert rms(res[0][1], ref[0][:150]) < TOL["bfloat16"] and rms(res[1][1], ref[1][8:9]) < TOL["bfloat16"]
-    _, lg = eng.prefill(b, toks[1][9:], want_logits=True)
+    eng = engine(m, prefill_chunk=400)
+    a, b, d, f = (eng.create_sequence() for _ in range(4))
+    eng.step([Portion(d, toks[2][:3], [])])
+    res = eng.step([Portion(b, toks[1][:9], [8]), Portion(a, toks[0][:150], list(range(150))), Portion(d, toks[2][3:4], [0]), Portion(f, toks[0][:130], [3, 129])],
+                   return_logits=True)
+    for (_, lg), want in zip(res, (ref[1][8:9], ref[0][:150], ref[2][3:4], ref[0][[3, 129]])):
+        assert rms(lg, want) < TOL["bfloat16"]
+    res = eng.step([Portion(a, toks[0][150:151], [0]), Portion(b, toks[1][9:10], [0]), Portion(d, toks[2][4:5], [0]), Portion(f, toks[0][130:], [0, 69])], return_logits=True)
+    for (_, lg), want in zip(res, (ref[0][150:151], ref[1][9:10], ref[2][4:5], ref[0][[130, 199]])):
+        assert rms(lg, want) < TOL["bfloat16"]
+    _, lg = eng.prefill(b, toks[1][10:], want_logits=True)
     assert rms(lg[None], ref[1][-1:]) < TOL["bfloat16"]
 
 
