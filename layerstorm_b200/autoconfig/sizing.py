@@ -34,7 +34,8 @@ def expert_slot_bytes(mc: ModelConfig, quant: str | None = None) -> int:
     """One routed expert (gate, up, down) in its cache slot, 4096-aligned."""
     q = quant or mc.expert_quant
     if mc.blocks:                              # bf16, width padded to the tensor-core tile
-        return _align(3 * mc.hidden * _align(mc.moe_inter, 128) * 2, 4096)
+        mats = 3 if all(b.unit == "glu" for b in mc.blocks if b.experts) else 2
+        return _align(mats * mc.hidden * _align(mc.moe_inter, 128) * 2, 4096)
     bits = QUANT_BITS.get(q, 16.0)
     return _align(int(3 * mc.hidden * mc.moe_inter * bits / 8) + 64, 4096)
 
@@ -65,7 +66,7 @@ def kv_bytes_per_token(mc: ModelConfig, backend: str = "snapmla", tp: int = 1, k
     """All attention layers, one token, on one GPU.  Sharded mode keeps 1/tp of the rows per rank."""
     if mc.blocks:
         lat = lambda b: _align(b.kv_rank, 16) + _align(b.rot_dim, 16) if b.kv_from < 0 else 0       # (layers may read another layer's rows)
-        return float(sum(2 * (lat(b) if b.latent else b.kv_heads * (_head_pad(b.dim) + _head_pad(b.vdim))) for b in mc.blocks if not b.recurrent))
+        return float(sum(2 * (lat(b) if b.latent else b.kv_heads * (_head_pad(b.dim) + _head_pad(b.vdim))) for L in mc.blocks for b in L.mixers if not b.recurrent))
     mla = mc.mla_layers()
     idx_layers = len({mc.index_source_layer(i) for i in mla}) if mc.has_indexer else 0
     per = len(mla) * kv_row_bytes(mc, backend) + idx_layers * indexer_row_bytes(mc)
@@ -76,7 +77,8 @@ def recurrent_state_bytes_per_seq(mc: ModelConfig, tp: int = 1) -> int:
     """KDA state (fp32 [heads, 128, 128]) and conv history per sequence on one GPU (heads split over tp)."""
     if mc.blocks:
         pad = lambda d: next((p for p in (32, 64, 128) if d <= p), 256)
-        return sum(b.heads * (b.vdim * pad(b.dim) + (2 * b.dim + b.vdim) * (b.conv - 1)) * 4 for b in mc.blocks if b.recurrent)
+        kept = lambda b: _align(mc.hidden, 8) if b.kind == "time_mix" else b.heads * (2 * b.dim + b.vdim) * (b.conv - 1)      # previous input / convolutions
+        return sum((b.heads * b.vdim * pad(b.dim) + kept(b)) * 4 for L in mc.blocks for b in L.mixers if b.recurrent)
     n_kda = sum(1 for t in mc.layer_types if t == "kda")
     if not n_kda:
         return 0
@@ -106,8 +108,14 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
     H = mc.hidden
     r = ResidentBytes()
     n = mc.hc_mult
-    for b in mc.blocks:
-        if b.recurrent:
+    for b in [m for L in mc.blocks for m in L.mixers]:
+        if b.kind == "time_mix":
+            kw, vw, rank = b.heads * b.dim, b.heads * b.vdim, b.dim          # (the rank is only in the tensors)
+            r.attention += ((2 * kw + 3 * vw + rank) * H + 3 * kw * rank) * 2 + (5 * H + 2 * kw + vw) * 4
+        elif b.kind == "head_delta":
+            kw, vw = b.kv_heads * b.dim, b.heads * b.vdim
+            r.attention += (2 * kw + 3 * vw + 2 * b.heads) * H * 2 + ((2 * kw + vw) * b.conv + 2 * b.heads + b.vdim) * 4
+        elif b.recurrent:
             rank = b.dim                                                 # the low-rank width is only in the tensors; this is its usual size
             w = (2 * b.kv_heads * b.dim + 2 * b.heads * b.vdim + b.heads + 2 * rank) * H + 3 * b.heads * (b.dim + b.vdim) * rank
             r.attention += w * 2 + ((2 * b.kv_heads * b.dim + b.heads * b.vdim) * b.conv + b.heads * b.dim) * 4
@@ -115,12 +123,15 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
             own = b.kv_rank + b.rot_dim if b.kv_from < 0 else 0
             r.attention += ((b.heads * (b.dim + b.rot_dim + b.vdim + (1 if b.head_gate else 0)) + own) * H + b.heads * (b.dim + b.vdim) * b.kv_rank) * 2
         else:
-            r.attention += (b.heads * (b.dim + b.vdim * (2 if b.out_gate else 1)) + b.kv_heads * (b.dim + b.vdim)) * H * 2
+            r.attention += (b.heads * (b.dim + b.vdim * (2 if b.out_gate else 1) + (1 if b.head_gate else 0)) + b.kv_heads * (b.dim + b.vdim)) * H * 2
+            r.attention += (b.heads * (b.bias_max + 1) * 4 if b.bias_rows else 0) + ((b.heads * b.dim + b.kv_heads * (b.dim + b.vdim)) * 4 if b.qkv_bias else 0)
+    for b in mc.blocks:
         r.dense_ffn += 3 * b.dense_ff * H * 2 + mc.side_dim * H * 2 * 2
         if b.experts:
             r.router += (b.experts + b.identity) * (2 * H + 4)
             r.shared_expert += (3 * b.shared_ff + (1 if b.shared_ff else 0)) * H * 2
         r.norms += (4 if b.has_ff else 2) * H * 4 * (2 if mc.norm_place == "sandwich" else 1) + (H * 4 if mc.side_dim else 0)
+        r.norms += (2 if b.has_ff else 1) * mc.streams * (mc.streams + 2) * 4 + (2 * H * 4 if b.branches and b.join == "normed" else 0)
     for i in range(0 if mc.blocks else mc.n_layers):
         if mc.is_kda_layer(i):
             C = mc.kda_heads * mc.kda_head_dim

@@ -42,7 +42,7 @@ CXX_FLAGS = ["-O2", "-g", "-std=c++20", "-fPIC", "-Wall", "-Wno-unused-function"
 
 
 # kernel files of a model family (models described layer by layer run without the MLA-family, indexer, hyper-connection and expert-parallel kernels)
-FAMILIES = {"blocks": ("attn", "delta", "gemm_tc", "gemv", "latent", "moe", "moe_tc", "norm", "sampling")}
+FAMILIES = {"blocks": ("attn", "delta", "gemm_tc", "gemv", "latent", "moe", "moe_tc", "norm", "sampling", "tmix")}
 
 
 def _rel(p) -> str:

@@ -1,13 +1,16 @@
-// Grouped-query softmax attention over the paged cache, with an optional sliding window, a per-head linear distance bias, query / key norms
-// over the whole projection, value mixing across layers and an output gate - every one of them a parameter.
+// Grouped-query softmax attention over the paged cache, with an optional sliding window or chunked mask, a per-head linear or learned distance
+// bias, query / key norms over the whole projection or per head, rotary positions, value mixing across layers and an output gate per channel
+// or head - every one of them a parameter.
 //
 //   q = RMSNorm_all(W_q h), k = RMSNorm_all(W_k h)        one norm over all rows of the projection (w = null: no norm)
 //   v = (1 - lambda) W_v h + lambda v_first                (mix = 2), v_first = the values of the first mixing layer (mix = 1 stores them)
-//   s_ij = scale q_i . k_j - slope_h (i - j),  0 <= i - j < window (window 0: the whole prefix);  o_i = softmax_j(s_ij) v_j
+//   or per head: q, k = rot(RMSNorm_head(W h + b))         norm with or without a weight, "rotate half" over the leading channels
+//   s_ij = scale q_i . k_j - slope_h (i - j) + bias_h[i - j],  0 <= i - j < window (window 0: the whole prefix), i and j in one chunk;
+//   o_i = softmax_j(s_ij) v_j
 //   out = o * sigmoid(gate)                                (gate offset < 0: none)
 //
 // Cache row of a token: [G * dkp keys | G * dvp values], head widths padded with zeros to dkp / dvp.
-//   attn_prep      norms, value mixing, append to the cache
+//   attn_prep      norms, value mixing, append to the cache;  attn_head_prep: biases, per-head norms, rotation, append
 //   attn_decode    few rows: one block per (row, kv head, split of the visible keys); the heads of a group are the rows of mma.sync tiles, each
 //                  warp walks its own 16-key tiles; attn_combine merges the splits
 //   attn_prefill   runs of rows: 128 (token, head) rows of a sequence per block against 32-key tiles shared by eight warps
@@ -69,12 +72,66 @@ __global__ void __launch_bounds__(NT) attn_prep_kernel(const float* __restrict__
     }
 }
 
+// One block per row, one warp per head: q and k = rot(norm(proj + bias)), v = proj + bias.  norm 0 none, 1 without a weight, 2 with wq / wk [dk].
+template <typename T, int NT>
+__global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restrict__ proj, int ldp, int off_q, int off_k, int off_v, const float* __restrict__ bq,
+                                                             const float* __restrict__ bk, const float* __restrict__ bv, int norm, const float* __restrict__ wq,
+                                                             const float* __restrict__ wk, float eps, int rot, const double* __restrict__ inv_freq,
+                                                             T* __restrict__ q_out, T* __restrict__ cache, const int* __restrict__ block_table, int max_pages,
+                                                             const int* __restrict__ row_seq, const int* __restrict__ row_pos, int H, int G, int dk, int dv,
+                                                             int dkp, int dvp, int page) {
+    extern __shared__ float s_cs[];                                // [rot / 2] cosines | [rot / 2] sines
+    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = rot / 2;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = row_seq[r], pos = row_pos[r];
+    if (seq < 0) return;
+    for (int i = threadIdx.x; i < half; i += NT) rotary_angle(pos, inv_freq[i], s_cs[half + i], s_cs[i]);
+    __syncthreads();
+    const float* pr = proj + (size_t)r * ldp;
+    T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * (dkp + dvp));
+    for (int j = warp; j < H + 2 * G; j += NT / 32) {
+        if (j >= H + G) {
+            const int g = j - H - G;
+            for (int c = lane; c < dvp; c += 32)
+                row[G * dkp + g * dvp + c] = to_act<T>(c < dv ? pr[off_v + g * dv + c] + (bv ? bv[g * dv + c] : 0.f) : 0.f);
+            continue;
+        }
+        const bool isq = j < H;
+        const int h = isq ? j : j - H;
+        const float* x = pr + (isq ? off_q : off_k) + (size_t)h * dk;
+        const float* b = isq ? bq : bk;
+        const float* w = isq ? wq : wk;
+        if (b) b += (size_t)h * dk;
+        float rs = 1.f;
+        if (norm) {
+            float a = 0.f;
+#pragma unroll 4
+            for (int c = lane; c < dk; c += 32) { const float v = x[c] + (b ? b[c] : 0.f); a = fmaf(v, v, a); }
+            rs = 1.f / sqrtf(warp_sum(a) / (float)dk + eps);
+        }
+        auto at = [&](int c) { return (x[c] + (b ? b[c] : 0.f)) * rs * (norm == 2 ? w[c] : 1.f); };
+        T* d = isq ? q_out + ((size_t)r * H + h) * dkp : row + (size_t)h * dkp;
+#pragma unroll 4
+        for (int c = lane; c < dkp; c += 32) {
+            float v = 0.f;
+            if (c < dk) {
+                v = at(c);
+                if (c < half) v = v * s_cs[c] - at(c + half) * s_cs[half + c];
+                else if (c < rot) v = v * s_cs[c - half] + at(c - half) * s_cs[c];
+            }
+            d[c] = to_act<T>(v);
+        }
+    }
+}
+
 // One warp's 16 query rows against NT 16-key tiles held in shared memory.  K: [keys][ldk], V: [keys][ldv]; row r of the warp sits at
-// position pos[r / 8 half]; scores are in log2 units.  m, l: running maximum and sum of the thread's two rows.
-template <int NV, int NT>
+// position pos[r / 8 half] and sees keys from low[..] on; scores are in log2 units.  m, l: running maximum and sum of the thread's two rows.
+// BIAS 1: tab[row][distance] in log2 units; 2: as it is stored, distances clamped to bias_last.
+template <int NV, int NT, int BIAS>
 __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* sk, int ldk, const bf16* sv, int ldv, int dkp, int key0, int key_end,
-                                           const int (&pos)[2], int window, float scale2, const float (&slope2)[2], float (&m)[2], float (&l)[2],
-                                           float (&o)[NV][4]) {
+                                           const int (&pos)[2], const int (&low)[2], float scale2, const float (&slope2)[2], const float* const (&tab)[2],
+                                           int bias_last, float (&m)[2], float (&l)[2], float (&o)[NV][4]) {
     const int lane = threadIdx.x & 31;
     float s[2 * NT][4];
 #pragma unroll
@@ -101,8 +158,10 @@ __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int row = j >> 1, key = key0 + (i >> 1) * 16 + (i & 1) * 8 + (lane & 3) * 2 + (j & 1), dist = pos[row] - key;
-            const bool seen = dist >= 0 && (window <= 0 || dist < window) && key < key_end;
-            s[i][j] = seen ? s[i][j] * scale2 - slope2[row] * (float)dist : -INFINITY;
+            const bool seen = dist >= 0 && key >= low[row] && key < key_end;
+            if constexpr (BIAS == 0) s[i][j] = seen ? s[i][j] * scale2 - slope2[row] * (float)dist : -INFINITY;
+            else if constexpr (BIAS == 1) s[i][j] = seen ? fmaf(s[i][j], scale2, tab[row][dist]) : -INFINITY;
+            else s[i][j] = seen ? fmaf(s[i][j], scale2, __ldg(tab[row] + min(dist, bias_last)) * kLog2e) : -INFINITY;
             mt[row] = fmaxf(mt[row], s[i][j]);
         }
     float corr[2], base[2];
@@ -144,7 +203,7 @@ __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* 
 
 // ------------------------------------------------------------------------------------------------ decode
 constexpr int kDecStages = 3;
-template <int DVP>
+template <int DVP, int BIAS>
 __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     constexpr int NV = DVP / 8;
     extern __shared__ __align__(16) bf16 asm_[];
@@ -165,7 +224,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         if (hh < nh) v = *reinterpret_cast<const uint4*>(q + (size_t)hh * p.dkp + c * 8);
         *reinterpret_cast<uint4*>(sq + hh * ldk + c * 8) = v;
     }
-    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    const int lo = attn_low(p, pos);
     const int ntile = (pos - lo + 16) / 16;                       // 16-key tiles of the visible range
     const int per = (ntile + p.NS - 1) / p.NS, t0 = split * per, t1 = min(ntile, t0 + per);
     const size_t ldc = (size_t)p.G * (p.dkp + p.dvp);
@@ -188,7 +247,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     for (int i = 0; i < NV; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     const int hr0 = g * hg + h0 + min(lane >> 2, nh - 1), hr1 = g * hg + h0 + min((lane >> 2) + 8, nh - 1);
     const float slope2[2] = {p.slope ? p.slope[hr0] * kLog2e : 0.f, p.slope ? p.slope[hr1] * kLog2e : 0.f};
-    const int pp[2] = {pos, pos};
+    const int pp[2] = {pos, pos}, low[2] = {lo, lo};
+    const float* const tab[2] = {BIAS ? p.bias + (size_t)hr0 * p.bias_len : nullptr, BIAS ? p.bias + (size_t)hr1 * p.bias_len : nullptr};
 #pragma unroll
     for (int s = 0; s < kDecStages - 1; ++s) issue(t0 + warp + 4 * s, s);
     __syncthreads();
@@ -198,7 +258,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         cp_wait<kDecStages - 1>();
         __syncwarp();
         const bf16* dk_ = st + (size_t)buf * 16 * (ldk + ldv);
-        attn_tiles<NV, 1>(sq, ldk, dk_, ldk, dk_ + 16 * ldk, ldv, p.dkp, lo + tile * 16, pos + 1, pp, p.window, p.scale * kLog2e, slope2, m, l, o);
+        attn_tiles<NV, 1, BIAS ? 2 : 0>(sq, ldk, dk_, ldk, dk_ + 16 * ldk, ldv, p.dkp, lo + tile * 16, pos + 1, pp, low, p.scale * kLog2e, slope2, tab,
+                                        p.bias_len - 1, m, l, o);
         __syncwarp();
         buf = (buf + 1) % kDecStages;
     }
@@ -236,8 +297,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
             }
         }
         if (p.NS == 1) {
-            O /= L;
-            if (p.off_gate >= 0) O *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + (size_t)h * p.dv + c]);
+            O = O / L * attn_out_factor(p, r, h, c);
             reinterpret_cast<bf16*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = __float2bfloat16(O);
         } else {
             const size_t k = ((size_t)r * p.H + h) * p.NS + split;
@@ -260,15 +320,16 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(AttnParams p) {
     for (int c = threadIdx.x; c < p.dv; c += 128) {
         float O = 0.f;
         for (int s = 0; s < p.NS; ++s) O = fmaf(p.o_part[(k0 + s) * p.dvp + c], ex2(p.ml_part[2 * (k0 + s)] - M), O);
-        O /= L;
-        if (p.off_gate >= 0) O *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + (size_t)h * p.dv + c]);
+        O = O / L * attn_out_factor(p, r, h, c);
         reinterpret_cast<bf16*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = __float2bfloat16(O);
     }
 }
 
 // ------------------------------------------------------------------------------------------------ prefill
 constexpr int kPreKeys = 32;          // keys per tile: with 32, two 256-thread blocks fit an SM's registers (1.24 -> 0.97 ms for 2048 rows x 4096 keys x 32 heads)
-template <int DVP>
+// row stride of the prefill form's slices of the bias table: one slice per head and key tile, all distances a tile of tq tokens can have
+__host__ __device__ constexpr int attn_bias_ld(int tq) { return (tq + kPreKeys - 1 + 31) / 32 * 32 + 8; }
+template <int DVP, int BIAS>
 __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(AttnParams p, const int* __restrict__ seq_row0, const int* __restrict__ seq_nrows, int nseq,
                                                            int tq) {
     constexpr int NV = DVP / 8, kTpk = 256 / kPreKeys;             // threads per key of a tile copy
@@ -277,6 +338,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
     const int ldk = p.dkp + 8, ldv = DVP + 8;
     bf16* sq = asm_;                                              // [128][ldk]
     bf16* skv = sq + 128 * ldk;                                   // [2][kPreKeys][ldk + ldv]
+    float* sbias = reinterpret_cast<float*>(skv + 2 * kPreKeys * (ldk + ldv));     // [2][hg][attn_bias_ld]
     pdl_wait();
     pdl_launch_dependents();
     // tile -> rows [r0, r0 + n) of one sequence
@@ -297,7 +359,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         *reinterpret_cast<uint4*>(sq + m * ldk + c * 8) = v;
     }
     const int pos_last = pos0 + n - 1;
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) / kPreKeys * kPreKeys : 0;
+    const int lo = attn_low(p, pos0) / kPreKeys * kPreKeys;
     const int ntile = (pos_last - lo) / kPreKeys + 1;
     const size_t ldc = (size_t)p.ldc;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache);
@@ -310,23 +372,32 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
             const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
             for (int c = t % kTpk; c < kc; c += kTpk) cp16(dk_ + kr * ldk + c * 8, src + (c * 8 < p.dkh ? (size_t)g * p.dkh + c * 8 : (size_t)p.off_ks + c * 8 - p.dkh));
             for (int c = t % kTpk; c < vc; c += kTpk) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)g * p.dvp + c * 8);
+            if constexpr (BIAS) {
+                const int ldb = attn_bias_ld(tq), d0 = pos0 - (lo + tile * kPreKeys) - (kPreKeys - 1);       // distance of column 0
+                float* sb = sbias + (tile & 1) * hg * ldb;
+                for (int h = warp; h < hg; h += 8)
+                    for (int c = lane; c < tq + kPreKeys - 1; c += 32)
+                        sb[h * ldb + c] = __ldg(p.bias + (size_t)(g * hg + h) * p.bias_len + min(max(d0 + c, 0), p.bias_len - 1)) * kLog2e;
+            }
         }
         cp_commit();
     };
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[NV][4];
 #pragma unroll
     for (int i = 0; i < NV; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
-    int mr[2], pp[2];
+    int mr[2], pp[2], low[2];
     float slope2[2];
 #pragma unroll
     for (int row = 0; row < 2; ++row) {
         mr[row] = warp * 16 + (lane >> 2) + 8 * row;
         const int tok = mr[row] / hg;
         pp[row] = tok < n ? pos0 + tok : -1;                      // -1: an idle row sees nothing
+        low[row] = tok < n ? attn_low(p, pos0 + tok) : 0;
         slope2[row] = p.slope ? p.slope[g * hg + mr[row] % hg] * kLog2e : 0.f;
     }
     // positions this warp's rows span: tiles outside their windows are skipped
     const int wfirst = pos0 + min((warp * 16) / hg, n - 1), wlast = pos0 + min((warp * 16 + 15) / hg, n - 1);
+    const int wlow = attn_low(p, wfirst);
     const bool wlive = (warp * 16) / hg < n;
     issue(0);
     for (int tile = 0; tile < ntile; ++tile) {
@@ -334,10 +405,16 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         cp_wait<1>();
         __syncthreads();
         const int k0 = lo + tile * kPreKeys;
-        if (wlive && k0 <= wlast && (p.window <= 0 || k0 + kPreKeys - 1 > wfirst - p.window)) {
+        if (wlive && k0 <= wlast && k0 + kPreKeys - 1 >= wlow) {
             const bf16* dk_ = skv + (size_t)(tile & 1) * kPreKeys * (ldk + ldv);
-            attn_tiles<NV, kPreKeys / 16>(sq + warp * 16 * ldk, ldk, dk_, ldk, dk_ + kPreKeys * ldk, ldv, p.dkp, k0, pos_last + 1, pp, p.window,
-                                          p.scale * kLog2e, slope2, m, l, o);
+            const float* tab[2] = {nullptr, nullptr};
+            if constexpr (BIAS) {
+                const int ldb = attn_bias_ld(tq), d0 = pos0 - k0 - (kPreKeys - 1);
+#pragma unroll
+                for (int row = 0; row < 2; ++row) tab[row] = sbias + ((tile & 1) * hg + mr[row] % hg) * ldb - d0;      // read at seen distances only
+            }
+            attn_tiles<NV, kPreKeys / 16, BIAS>(sq + warp * 16 * ldk, ldk, dk_, ldk, dk_ + kPreKeys * ldk, ldv, p.dkp, k0, pos_last + 1, pp, low,
+                                                p.scale * kLog2e, slope2, tab, 0, m, l, o);
         }
         __syncthreads();                                          // the buffer is refilled next
     }
@@ -349,7 +426,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         const int tok = mr[row] / hg, h = g * hg + mr[row] % hg;
         if (tok >= n) continue;
         const size_t rr = (size_t)(r0 + tok);
-        const float inv = (p.off_gate >= 0 && p.head_gate ? gate_sigmoid(p.proj[rr * p.ldp + p.off_gate + h]) : 1.f) / l[row];
+        const float inv = (p.off_gate >= 0 && p.head_gate ? gate_sigmoid(p.proj[rr * p.ldp + p.off_gate + h]) : 1.f) * p.out_scale / l[row];
         bf16* d = reinterpret_cast<bf16*>(p.out) + rr * p.ldo + (size_t)h * p.dv;
         const float* gt = p.proj + rr * p.ldp + p.off_gate + (size_t)h * p.dv;
 #pragma unroll
@@ -373,18 +450,30 @@ static int launch_decode(const AttnParams& p, cudaStream_t st) {
     const size_t merge = (size_t)4 * 16 * (DVP + 2) * 4;
     if (merge > smem) smem = merge;
     static bool attr = false;
-    if (!attr) { cudaFuncSetAttribute(attn_decode_kernel<DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024); attr = true; }
-    launch_pdl((attn_decode_kernel<DVP>), dim3(p.rows * p.G, p.NS, (p.H / p.G + 15) / 16), 128, smem, st, p);
+    if (!attr) {
+        cudaFuncSetAttribute(attn_decode_kernel<DVP, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<DVP, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        attr = true;
+    }
+    const dim3 grid(p.rows * p.G, p.NS, (p.H / p.G + 15) / 16);
+    if (p.bias) launch_pdl((attn_decode_kernel<DVP, 1>), grid, 128, smem, st, p);
+    else launch_pdl((attn_decode_kernel<DVP, 0>), grid, 128, smem, st, p);
     if (p.NS > 1) launch_pdl((attn_combine_kernel), dim3(p.rows, p.H), 128, 0, st, p);
     return (int)cudaGetLastError();
 }
 template <int DVP>
 static int launch_prefill(const AttnParams& p, const int* row0, const int* nrows, int nseq, cudaStream_t st) {
     const int ldk = p.dkp + 8, ldv = DVP + 8, tq = 128 / (p.H / p.G);
-    const size_t smem = (size_t)(128 * ldk + 2 * kPreKeys * (ldk + ldv)) * 2;
+    const size_t smem = (size_t)(128 * ldk + 2 * kPreKeys * (ldk + ldv)) * 2, sb = (size_t)2 * (p.H / p.G) * attn_bias_ld(tq) * 4;
     static bool attr = false;
-    if (!attr) { cudaFuncSetAttribute(attn_prefill_kernel<DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024); attr = true; }
-    launch_pdl((attn_prefill_kernel<DVP>), dim3(p.rows / tq + nseq, p.G), 256, smem, st, p, row0, nrows, nseq, tq);
+    if (!attr) {
+        cudaFuncSetAttribute(attn_prefill_kernel<DVP, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(attn_prefill_kernel<DVP, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        attr = true;
+    }
+    const dim3 grid(p.rows / tq + nseq, p.G);
+    if (p.bias) launch_pdl((attn_prefill_kernel<DVP, 1>), grid, 256, smem + sb, st, p, row0, nrows, nseq, tq);
+    else launch_pdl((attn_prefill_kernel<DVP, 0>), grid, 256, smem, st, p, row0, nrows, nseq, tq);
     return (int)cudaGetLastError();
 }
 
@@ -409,16 +498,37 @@ LSB_API int lsb_attn_prep(const void* proj, int ldp, int off_q, int off_k, int o
     LSB_CHECK_LAUNCH();
 }
 
+// Biases (null: none), per-head norms (norm 0 none, 1 plain, 2 with wq / wk [dk]), rotation of the leading `rot` channels (inv_freq: fp64 [rot / 2]) and
+// the cache append of every row.
+LSB_API int lsb_attn_head_prep(const void* proj, int ldp, int off_q, int off_k, int off_v, const void* bias_q, const void* bias_k, const void* bias_v, int norm,
+                               const void* wq, const void* wk, float eps, int rot, const void* inv_freq, void* q_out, void* cache, const void* block_table,
+                               int max_pages, const void* row_seq, const void* row_pos, int rows, int H, int G, int dk, int dv, int dkp, int dvp, int page,
+                               int f32, void* stream) {
+    if (rows < 1 || H % G || dkp < dk || dvp < dv || dkp % 16 || dvp % 16 || rot < 0 || rot % 2 || rot > dk || (rot && !inv_freq) || norm < 0 || norm > 2 ||
+        (norm == 2 && (!wq || !wk)) || rot > 8192)
+        return -1;
+    cudaStream_t st = (cudaStream_t)stream;
+    const bool wide = rows <= 64 && H + 2 * G >= 12;
+#define LSB_PREP(T, N) launch_pdl((attn_head_prep_kernel<T, N>), rows, N, (size_t)rot * 4, st, (const float*)proj, ldp, off_q, off_k, off_v, (const float*)bias_q, \
+                               (const float*)bias_k, (const float*)bias_v, norm, (const float*)wq, (const float*)wk, eps, rot, (const double*)inv_freq, (T*)q_out, \
+                               (T*)cache, (const int*)block_table, max_pages, (const int*)row_seq, (const int*)row_pos, H, G, dk, dv, dkp, dvp, page)
+    if (f32) LSB_PREP(float, 256); else if (wide) LSB_PREP(bf16, 1024); else LSB_PREP(bf16, 256);
+#undef LSB_PREP
+    LSB_CHECK_LAUNCH();
+}
+
 // Attention of the step's rows.  run_rows: the largest number of rows a sequence has in this step (host knowledge; it selects the kernel form).
-// NS: key splits of the few-row form (o_part / ml_part sized for it).  off_gate < 0: no output gate.  slope null: no distance bias.
+// NS: key splits of the few-row form (o_part / ml_part sized for it).  off_gate < 0: no output gate; head_gate: one gate per head.  slope null: no linear
+// distance bias; bias [H, bias_len] (null: none): learned distance bias, not together with slopes.  chunk: size of the mask's chunks (0: none).
 LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
                      const void* seq_row0, const void* seq_nrows, int nseq, int run_rows, const void* proj, int ldp, int off_gate, void* out, int ldo,
                      void* o_part, void* ml_part, int NS, int rows, int H, int G, int dk, int dv, int dkp, int dvp, int window, float scale,
-                     const void* slope, int f32, void* stream) {
-    if (rows < 1 || H % G || dkp % 16 || dvp % 16 || NS < 1 || (NS > 1 && (!o_part || !ml_part))) return -1;
+                     const void* slope, int head_gate, int chunk, const void* bias, int bias_len, float out_scale, int f32, void* stream) {
+    if (rows < 1 || H % G || dkp % 16 || dvp % 16 || NS < 1 || (NS > 1 && (!o_part || !ml_part)) || chunk < 0 || (bias && (slope || bias_len < 1))) return -1;
     AttnParams p;
+    p.chunk = chunk; p.bias = (const float*)bias; p.bias_len = bias_len; p.out_scale = out_scale;
     p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
-    p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 0; p.out = out; p.ldo = ldo;
+    p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = head_gate; p.out = out; p.ldo = ldo;
     p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.rows = rows; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = dkp; p.dvp = dvp;
     p.ldc = G * (dkp + dvp); p.off_v = G * dkp; p.dkh = dkp; p.off_ks = 0; p.NS = NS; p.window = window; p.scale = scale; p.slope = (const float*)slope;
     cudaStream_t st = (cudaStream_t)stream;

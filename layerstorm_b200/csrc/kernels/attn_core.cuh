@@ -17,7 +17,17 @@ struct AttnParams {
     int rows, H, G, dk, dv, dkp, dvp, NS, window;
     float scale;
     const float* slope;               // [H] (log2 units are applied in the kernels) or null
+    int chunk = 0;                    // a position sees the keys of its own chunk of this many (0: no chunks)
+    const float* bias = nullptr;      // [H, bias_len] added to the scores by distance, the last entry for all further ones; or null
+    int bias_len = 0;
+    float out_scale = 1.f;            // on the heads' outputs
 };
+
+// first key that position `pos` sees
+__device__ __forceinline__ int attn_low(const AttnParams& p, int pos) {
+    const int w = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    return p.chunk > 0 ? max(w, pos / p.chunk * p.chunk) : w;
+}
 
 template <typename T> __device__ __forceinline__ T to_act(float v);
 template <> __device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16(v); }
@@ -25,6 +35,17 @@ template <> __device__ __forceinline__ float to_act<float>(float v) { return v; 
 __device__ __forceinline__ float act_f(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float act_f(float v) { return v; }
 __device__ __forceinline__ float gate_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+// factor on value channel c of head h: output gate (if any) and constant
+__device__ __forceinline__ float attn_out_factor(const AttnParams& p, size_t r, int h, int c) {
+    return p.off_gate >= 0 ? p.out_scale * gate_sigmoid(p.proj[r * p.ldp + p.off_gate + (p.head_gate ? (size_t)h : (size_t)h * p.dv + c)]) : p.out_scale;
+}
+
+// cosine and sine of pos * freq; the angle is reduced in fp64 so that far positions keep their phase
+__device__ __forceinline__ void rotary_angle(int pos, double freq, float& s, float& c) {
+    constexpr double kTwoPi = 6.283185307179586476925;
+    const double x = (double)pos * freq;
+    sincosf((float)(x - kTwoPi * rint(x * (1.0 / kTwoPi))), &s, &c);
+}
 
 // ------------------------------------------------------------------------------------------------ CUDA-core kernel
 // One block per (row, head): 128 keys at a time, one thread per key for the scores, one per value channel for the sum.
@@ -47,7 +68,8 @@ static __global__ void __launch_bounds__(128) attn_exact_kernel(AttnParams p) {
     const float slope = p.slope ? p.slope[h] : 0.f;
     const size_t ldc = (size_t)p.ldc;
     const T* cache = reinterpret_cast<const T*>(p.cache);
-    const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    const int lo = attn_low(p, pos);
+    const float* bias = p.bias ? p.bias + (size_t)h * p.bias_len : nullptr;
     float m = -INFINITY, l = 0.f;
     for (int k0 = lo; k0 <= pos; k0 += 128) {
         const int j = k0 + t;
@@ -60,7 +82,7 @@ static __global__ void __launch_bounds__(128) attn_exact_kernel(AttnParams p) {
             float a = 0.f;
 #pragma unroll 8
             for (int c = 0; c < p.dk; ++c) a = fmaf(s_q[c], act_f(k[c]), a);
-            s = a * p.scale - slope * (float)(pos - j);
+            s = a * p.scale - slope * (float)(pos - j) + (bias ? bias[min(pos - j, p.bias_len - 1)] : 0.f);
         }
         s_row[t] = row;
         const float mt = fmaxf(m, block_max(s, red));
@@ -78,8 +100,7 @@ static __global__ void __launch_bounds__(128) attn_exact_kernel(AttnParams p) {
         }
     }
     for (int c = t; c < p.dv; c += 128) {
-        float o = s_o[c] / l;
-        if (p.off_gate >= 0) o *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + (p.head_gate ? (size_t)h : (size_t)h * p.dv + c)]);
+        const float o = s_o[c] / l * attn_out_factor(p, r, h, c);
         reinterpret_cast<T*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = to_act<T>(o);
     }
 }

@@ -1,5 +1,6 @@
-// Gated delta rule with one decay per key channel, for any head geometry: `H` value heads of `dv` channels over `G` query / key heads of
-// `dk` channels (head h reads query / key head h / (H / G)), short causal convolutions of any length, low-rank decay and output gates.
+// Gated delta rule with one decay per key channel or per head, for any head geometry: `H` value heads of `dv` channels over `G` query / key
+// heads of `dk` channels (head h reads query / key head h / (H / G)), short causal convolutions of any length, low-rank decay and output gates.
+// Rank 0 of the decay: one decay per head, x = its column of the projection.  Rank 0 of the output gate: SiLU of a full-rank projection.
 //
 //   q, k, v = SiLU(conv(raw));  q = q / sqrt(sum q^2 + 1e-6) * q_scale;  k = k / sqrt(sum k^2 + 1e-6)
 //   log g = decay(a_exp[h], W_a a + dt_bias)      one per head and key channel; mode 0: -a_exp softplus(x), mode 1: bound * sigmoid(a_exp x)
@@ -47,6 +48,15 @@ __device__ __forceinline__ float sigmoid_acc(float x) { return 1.f / (1.f + expf
 __device__ __forceinline__ float delta_log_decay(int mode, float a_exp, float x, float bound) {
     if (mode == 0) return -a_exp * (x > 20.f ? x : log1pf(expf(x)));
     return bound * sigmoid_acc(a_exp * x);
+}
+
+// rank_a 0: the head's log decay at a row of the projection;  rank_g 0: the output gate of value channel v
+__device__ __forceinline__ float delta_head_decay(const DeltaParams& p, const float* pr, int h, float a_exp) {
+    return delta_log_decay(p.decay_mode, a_exp, pr[p.off_a + h] + p.dt_bias[h], p.decay_bound);
+}
+__device__ __forceinline__ float delta_full_gate(const DeltaParams& p, const float* pr, int h, int v) {
+    const float x = pr[p.off_g + (size_t)h * p.dv + v];
+    return x * sigmoid_acc(x);
 }
 
 // channel c of a head: [0, dk) query, [dk, 2 dk) key, [2 dk, 2 dk + dv) value -> projection column and convolution taps
@@ -196,9 +206,13 @@ __global__ void __launch_bounds__(MAXT, 1) delta_step_kernel(DeltaParams p, int 
         qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
         const float qi = p.q_scale / sqrtf(qq + 1e-6f), ki = 1.f / sqrtf(kk + 1e-6f);
         float gate = 0.f;
-        if (p.dv == (T >> 2) || __any_sync(0xffffffffu, has_v))
-            gate = quad_dot<WT>(wg + (size_t)(has_v ? v : 0) * srg, s_ga, p.rank_g, ks);
-        for (int c0 = 0; c0 < p.dk; c0 += T >> 2) {
+        if (p.rank_g == 0) gate = delta_full_gate(p, pr, h, has_v ? v : 0);
+        else if (p.dv == (T >> 2) || __any_sync(0xffffffffu, has_v))
+            gate = sigmoid_acc(quad_dot<WT>(wg + (size_t)(has_v ? v : 0) * srg, s_ga, p.rank_g, ks));
+        if (p.rank_a == 0) {
+            const float gh = expf(delta_head_decay(p, pr, h, a_exp));
+            for (int c = t; c < p.dk; c += T) s_g[c] = gh;
+        } else for (int c0 = 0; c0 < p.dk; c0 += T >> 2) {
             const int c = c0 + v;
             const float x = quad_dot<WT>(wa + (size_t)min(c, p.dk - 1) * sra, s_fa, p.rank_a, ks);
             if (ks == 0 && c < p.dk) s_g[c] = expf(delta_log_decay(p.decay_mode, a_exp, x + p.dt_bias[(size_t)h * p.dk + c], p.decay_bound));
@@ -226,7 +240,7 @@ __global__ void __launch_bounds__(MAXT, 1) delta_step_kernel(DeltaParams p, int 
             S[j].x = fmaf(uk, k.x, S[j].x); S[j].y = fmaf(uk, k.y, S[j].y); S[j].z = fmaf(uk, k.z, S[j].z); S[j].w = fmaf(uk, k.w, S[j].w);
         }
         const float os = block_sum(ks == 0 ? o * o : 0.f, s_red);
-        if (ks == 0 && has_v) store_act<OT>(p.out, (size_t)(row0 + i) * p.ldo + (size_t)h * p.dv + v, o / sqrtf(os / (float)p.dv + p.eps) * ow * sigmoid_acc(gate));
+        if (ks == 0 && has_v) store_act<OT>(p.out, (size_t)(row0 + i) * p.ldo + (size_t)h * p.dv + v, o / sqrtf(os / (float)p.dv + p.eps) * ow * gate);
         __syncthreads();
     }
     if (has_v) {
@@ -291,7 +305,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(DeltaParams p, DeltaScr
             const int c = lane + 32 * j;
             w.qn[o + c] = q[j] * qi;
             w.kn[o + c] = k[j] * ki;
-            w.ld[o + c] = c < p.dk ? delta_log_decay(p.decay_mode, a_exp, w.rawa[((size_t)row * p.H + h) * p.dk + c] + p.dt_bias[(size_t)h * p.dk + c], p.decay_bound) : 0.f;
+            if (p.rank_a == 0) w.ld[o + c] = c < p.dk ? delta_head_decay(p, p.proj + (size_t)row * p.ldp, h, a_exp) : 0.f;
+            else w.ld[o + c] = c < p.dk ? delta_log_decay(p.decay_mode, a_exp, w.rawa[((size_t)row * p.H + h) * p.dk + c] + p.dt_bias[(size_t)h * p.dk + c], p.decay_bound) : 0.f;
         }
         for (int c = lane; c < p.dv; c += 32) w.vo[((size_t)row * p.H + h) * p.dv + c] = delta_conv(p, h, 2 * p.dk + c, slot, row0, i);
         if (lane == 0) {
@@ -391,8 +406,10 @@ __global__ void __launch_bounds__(128) delta_out_kernel(DeltaParams p, DeltaScra
     float ss = 0.f;
     for (int c = lane; c < p.dv; c += 32) ss = fmaf(o[c], o[c], ss);
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
-    for (int c = lane; c < p.dv; c += 32)
-        store_act<OT>(p.out, (size_t)row * p.ldo + (size_t)h * p.dv + c, o[c] * r * p.onorm[c] * sigmoid_acc(w.rawg[(size_t)rh * p.dv + c]));
+    for (int c = lane; c < p.dv; c += 32) {
+        const float gate = p.rank_g == 0 ? delta_full_gate(p, p.proj + (size_t)row * p.ldp, h, c) : sigmoid_acc(w.rawg[(size_t)rh * p.dv + c]);
+        store_act<OT>(p.out, (size_t)row * p.ldo + (size_t)h * p.dv + c, o[c] * r * p.onorm[c] * gate);
+    }
 }
 
 static int delta_pad(int dk) { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : 256)); }
@@ -466,7 +483,7 @@ LSB_API int lsb_delta_chunk_floats(int chunks, int H, int dk) {
     return n > 0x7fffffffLL ? -1 : (int)n;
 }
 
-// One layer body over the step's rows: proj (the fused input projection) -> out.  f32: weights w_a / w_g and `out` are fp32, otherwise bf16;
+// One layer body over the step's rows: proj (the fused input projection) -> out.  rank_a = rank_g = 0: decays per head (dt_bias [H]), full-rank gate.  f32: weights w_a / w_g and `out` are fp32, otherwise bf16;
 // w_a2 / w_g2 = [W | W] (bf16 only).  few: the host's choice of the one-kernel form (dv <= lsb_delta_few_max_dv(dk)).  Otherwise scratch is required, with
 // `short_seqs` / `long_seqs` = how many sequences have fewer / at least `long_min` rows and `nchunks` = 64-token chunks of the latter
 // (long sequences need dk <= 128 and chunk_ws).  gemm_err: error word of the tensor-core products.
@@ -477,6 +494,7 @@ LSB_API int lsb_delta_forward(const void* proj, int ldp, int off_q, int off_k, i
                               int G, int dk, int dv, int taps, int decay_mode, float q_scale, float decay_bound, float eps, int f32, int few,
                               void* scratch, int short_seqs, int long_seqs, int nchunks, int long_min, void* chunk_ws, void* gemm_err, void* stream) {
     if (dk < 1 || dk > 256 || dv < 1 || H < 1 || G < 1 || H % G || taps < 1 || rank_a % 8 || rank_g % 8 || total_rows < 1 || nseq < 1) return -1;
+    if ((rank_a == 0) != (rank_g == 0)) return -1;
     if (few && dv > delta_step_max_dv(delta_pad(dk))) return -1;
     if (!few && (!scratch || (long_seqs && (dk > 128 || !chunk_ws || long_min < 1)))) return -1;
     cudaStream_t st = (cudaStream_t)stream;
@@ -499,7 +517,9 @@ LSB_API int lsb_delta_forward(const void* proj, int ldp, int off_q, int off_k, i
     w.vo = w.ld + n * DKP; w.beta = w.vo + n * dv; w.kq = w.beta + n; w.rawa = w.kq + n; w.rawg = w.rawa + n * dk;
     float* rest = w.rawg + n * dv;
     int rc;
-    if (f32) {
+    if (rank_a == 0 && rank_g == 0) {
+        rc = 0;                                                    // nothing low-rank: decays and gates are columns of the projection
+    } else if (f32) {
         rc = lsb_gemm_f32(w.rawa, (const float*)proj + off_a, w_a, total_rows, H * dk, rank_a, ldp, rank_a, H * dk, stream);
         if (rc) return rc;
         rc = lsb_gemm_f32(w.rawg, (const float*)proj + off_g, w_g, total_rows, H * dv, rank_g, ldp, rank_g, H * dv, stream);

@@ -134,6 +134,9 @@ struct WRowBf16S {
     }
 };
 
+// Weight rows in up to eight runs, each with an input row of its own: rows from `row[j]` on multiply x + j * stride (n 0: one input for all).
+struct XSegs { int n; int row[8]; long long stride; };
+
 static __device__ int g_gemv_err = 0;      // first bulk-copy wait that ran out (0 = none); read through lsb_gemv_error
 
 // bf16 weights, same work split as gemv_kernel, but every warp asks the copy engine for its two row slices (<= 4 KB each) with
@@ -143,7 +146,7 @@ static __device__ int g_gemv_err = 0;      // first bulk-copy wait that ran out 
 template <int MT, bool OUT_BF16, int KS>
 __global__ void __launch_bounds__(256) gemv_bf16_bulk_kernel(MatBf16 mat, const bf16* __restrict__ x, int ldx, void* __restrict__ out,
                                                              int ldo, int N, int K, int kper, float alpha, const float* __restrict__ bias,
-                                                             PeerComm comm) {
+                                                             PeerComm comm, XSegs xs) {
     __shared__ float red[8][2 * MT];
     __shared__ __align__(8) uint64_t bars[8];
     extern __shared__ __align__(128) uint8_t slices[];       // [8 warps][2 rows][kper] bf16
@@ -167,6 +170,12 @@ __global__ void __launch_bounds__(256) gemv_bf16_bulk_kernel(MatBf16 mat, const 
         tc::bulk_load_1d(s1, mat.w + (size_t)n1 * mat.ldw + k0, bytes, &bars[warp]);
     }
     __syncwarp();
+    if (xs.n) {
+        int s = 0;
+#pragma unroll
+        for (int j = 1; j < 8; ++j) s += j < xs.n && n0 >= xs.row[j];
+        x += s * xs.stride;
+    }
     pdl_wait();
     pdl_launch_dependents();
     unsigned next_epoch = 0;
@@ -220,7 +229,7 @@ __global__ void __launch_bounds__(256) gemv_bf16_bulk_kernel(MatBf16 mat, const 
 
 template <int MT, bool OB, int KS>
 static void launch_bulk_one(MatBf16 mat, const bf16* xp, int ldx, void* op, int ldo, int N, int K, int kper, float alpha, const float* bias,
-                            PeerComm comm, cudaStream_t st) {
+                            PeerComm comm, cudaStream_t st, const XSegs& xs) {
     const int rows_per_block = (8 / KS) * 2;
     static bool once = false;
     if (!once) {
@@ -235,16 +244,16 @@ static void launch_bulk_one(MatBf16 mat, const bf16* xp, int ldx, void* op, int 
     size_t smem = (size_t)16 * kper * 2;
     if (smem >= 64 * 1024) smem += (size_t)pad_kb * 1024;
     launch_pdl((gemv_bf16_bulk_kernel<MT, OB, KS>), (N + rows_per_block - 1) / rows_per_block, 256, smem, st, mat, xp, ldx, op, ldo,
-               N, K, kper, alpha, bias, comm);
+               N, K, kper, alpha, bias, comm, xs);
 }
 
 template <int MT, bool OB>
 static void launch_bulk_ks(int ks, MatBf16 mat, const bf16* xp, int ldx, void* op, int ldo, int N, int K, int kper, float alpha, const float* bias,
-                           PeerComm comm, cudaStream_t st) {
-    if (ks == 1) launch_bulk_one<MT, OB, 1>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st);
-    else if (ks == 2) launch_bulk_one<MT, OB, 2>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st);
-    else if (ks == 4) launch_bulk_one<MT, OB, 4>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st);
-    else launch_bulk_one<MT, OB, 8>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st);
+                           PeerComm comm, cudaStream_t st, const XSegs& xs) {
+    if (ks == 1) launch_bulk_one<MT, OB, 1>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st, xs);
+    else if (ks == 2) launch_bulk_one<MT, OB, 2>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st, xs);
+    else if (ks == 4) launch_bulk_one<MT, OB, 4>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st, xs);
+    else launch_bulk_one<MT, OB, 8>(mat, xp, ldx, op, ldo, N, K, kper, alpha, bias, comm, st, xs);
 }
 
 // LSB_GEMV_BULK=0: bf16 GEMVs keep the register-streaming kernel
@@ -288,7 +297,7 @@ static int choose_ks(int N, int K, int epl) {
 
 template <class Mat>
 static int launch_gemv(Mat mat, const bf16* x, int ldx, void* out, int ldo, int M, int N, int K, float alpha,
-                       const float* bias, int out_bf16, cudaStream_t st, const void* comm_host = nullptr) {
+                       const float* bias, int out_bf16, cudaStream_t st, const void* comm_host = nullptr, const XSegs& xs = XSegs{0, {0}, 0}) {
     PeerComm comm;
     comm.nranks = 0;
     if (comm_host) {
@@ -307,6 +316,7 @@ static int launch_gemv(Mat mat, const bf16* x, int ldx, void* out, int ldo, int 
             if (kper <= 2048) { ks = kb; bulk_kper = kper; }
         }
     }
+    if (xs.n && !bulk_kper) return -1;
     for (int m0 = 0; m0 < M;) {
         const int rem = M - m0;
         const int mt = rem >= 4 ? 4 : (rem >= 2 ? 2 : 1);
@@ -315,8 +325,8 @@ static int launch_gemv(Mat mat, const bf16* x, int ldx, void* out, int ldo, int 
 #define LSB_GEMV_CASE(MT_)                                                                              \
     if constexpr (std::is_same<Mat, MatBf16>::value) {                                                  \
         if (bulk_kper) {                                                                                \
-            if (out_bf16) launch_bulk_ks<MT_, true>(ks, mat, xp, ldx, op, ldo, N, K, bulk_kper, alpha, bias, comm, st);  \
-            else launch_bulk_ks<MT_, false>(ks, mat, xp, ldx, op, ldo, N, K, bulk_kper, alpha, bias, comm, st);          \
+            if (out_bf16) launch_bulk_ks<MT_, true>(ks, mat, xp, ldx, op, ldo, N, K, bulk_kper, alpha, bias, comm, st, xs);  \
+            else launch_bulk_ks<MT_, false>(ks, mat, xp, ldx, op, ldo, N, K, bulk_kper, alpha, bias, comm, st, xs);      \
             m0 += mt;                                                                                   \
             continue;                                                                                   \
         }                                                                                               \
@@ -348,6 +358,19 @@ LSB_API int lsb_gemv_bf16(void* out, const void* x, const void* w, const void* b
     if (K % 8 || ldw % 8 || ldx % 8) return -1;
     return launch_gemv(MatBf16{(const bf16*)w, ldw}, (const bf16*)x, ldx, out, ldo, M, N, K, alpha, (const float*)bias,
                        out_bf16, (cudaStream_t)stream, comm);
+}
+
+// The same with an input of its own for each of `nseg` runs of weight rows: run j starts at row seg_rows[j] (host array, [0] = 0, multiples of 2) and
+// multiplies x + j * seg_stride (elements).  fp32 output; K such that a row slice fits the bulk-copy form.
+LSB_API int lsb_gemv_bf16_segs(void* out, const void* x, const void* w, int M, int N, int K, int ldx, int ldw, int ldo, const void* seg_rows, int nseg,
+                               long long seg_stride, void* stream) {
+    if (K % 8 || ldw % 8 || ldx % 8 || seg_stride % 8 || nseg < 1 || nseg > 8) return -1;
+    XSegs xs{nseg, {0}, seg_stride};
+    for (int j = 0; j < nseg; ++j) {
+        xs.row[j] = reinterpret_cast<const int*>(seg_rows)[j];
+        if (xs.row[j] % 2 || (j == 0 ? xs.row[j] != 0 : xs.row[j] < xs.row[j - 1])) return -1;
+    }
+    return launch_gemv(MatBf16{(const bf16*)w, ldw}, (const bf16*)x, ldx, out, ldo, M, N, K, 1.f, nullptr, 0, (cudaStream_t)stream, nullptr, xs);
 }
 
 namespace lsb {

@@ -40,12 +40,10 @@ struct LatentPrep {
     int rows, H, dn, dnp, dr, drp, dl, dlp;
 };
 
-// (a, b) turned by pos * freq; the angle is reduced in fp64 so that far positions keep their phase
+// (a, b) turned by pos * freq
 __device__ __forceinline__ void rotate_pair(float& a, float& b, int pos, double freq) {
-    constexpr double kTwoPi = 6.283185307179586476925;
-    const double x = (double)pos * freq;
     float s, c;
-    sincosf((float)(x - kTwoPi * rint(x * (1.0 / kTwoPi))), &s, &c);
+    rotary_angle(pos, freq, s, c);
     const float u = a * c - b * s, v = b * c + a * s;
     a = u; b = v;
 }

@@ -220,8 +220,8 @@ template <> struct RowOf<6> {
     static __device__ __forceinline__ T make(const uint8_t* w, const uint8_t*, int n, int K) { return T{w + (size_t)n * (K + (K >> 4)), K}; }
 };
 
-// act[pair][f] = glu_act(g, u) ; g = x[row] . Wgate[f], u = x[row] . Wup[f]
-template <int FMT>
+// act[pair][f] = glu_act(g, u) ; g = x[row] . Wgate[f], u = x[row] . Wup[f]   (not GATED: relu(u)^2, no gate matrix)
+template <int FMT, bool GATED = true>
 __global__ void __launch_bounds__(256) moe_gateup_kernel(const bf16* __restrict__ x, const uint8_t* __restrict__ arena,
                                                          const int* __restrict__ slot_of, ExpertFmt ef,
                                                          const int* __restrict__ group_expert, const int* __restrict__ group_n,
@@ -249,7 +249,7 @@ __global__ void __launch_bounds__(256) moe_gateup_kernel(const bf16* __restrict_
 #pragma unroll 2
     for (int k = lane * E; k + E <= ef.H; k += 32 * E) {
         float a[E], b[E];
-        rg.load(k, a);
+        if constexpr (GATED) rg.load(k, a);
         ru.load(k, b);
 #pragma unroll
         for (int m = 0; m < 4; ++m) {
@@ -260,7 +260,7 @@ __global__ void __launch_bounds__(256) moe_gateup_kernel(const bf16* __restrict_
                     float xf[8];
                     unpack_bf16x8(__ldg(reinterpret_cast<const uint4*>(xp + e8)), xf);
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) { ag[m] = fmaf(a[e8 + i], xf[i], ag[m]); au[m] = fmaf(b[e8 + i], xf[i], au[m]); }
+                    for (int i = 0; i < 8; ++i) { if constexpr (GATED) ag[m] = fmaf(a[e8 + i], xf[i], ag[m]); au[m] = fmaf(b[e8 + i], xf[i], au[m]); }
                 }
             }
         }
@@ -273,10 +273,10 @@ __global__ void __launch_bounds__(256) moe_gateup_kernel(const bf16* __restrict_
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
         if (m < n) {
-            const float gv = warp_sum(ag[m]) * sg, uv = warp_sum(au[m]) * su;
+            const float gv = GATED ? warp_sum(ag[m]) * sg : 0.f, uv = warp_sum(au[m]) * su;
             if (lane == 0) {
                 const float c = glu_in_scale(ga, pr[m]);
-                act[(size_t)pr[m] * ef.F + f] = __float2bfloat16(glu_act(gv * c, uv * c, ga));
+                act[(size_t)pr[m] * ef.F + f] = __float2bfloat16(GATED ? glu_act(gv * c, uv * c, ga) : relu2_act(uv * c));
             }
         }
     }
@@ -359,18 +359,19 @@ __global__ void __launch_bounds__(256) moe_f32_kernel(const float* __restrict__ 
     const int e = group_expert[g], n = group_n[g], slot = slot_of[e];
     if (slot < 0) { if (GATEUP && miss_flag && threadIdx.x == 0 && blockIdx.x == 0) atomicExch(miss_flag, e + 1); return; }
     const uint8_t* base = arena + (size_t)slot * ef.stride;
-    const float* w0 = reinterpret_cast<const float*>(base + (GATEUP ? ef.off_gate : ef.off_down)) + (size_t)n_out * K;
+    const bool gated = GATEUP && ga.unit == 0;
     const float* w1 = reinterpret_cast<const float*>(base + ef.off_up) + (size_t)n_out * K;
+    const float* w0 = GATEUP && !gated ? w1 : reinterpret_cast<const float*>(base + (GATEUP ? ef.off_gate : ef.off_down)) + (size_t)n_out * K;
     for (int m = 0; m < n; ++m) {
         const int pr = group_pairs[g * 4 + m];
         const float* x = in + (size_t)(GATEUP ? pr / S : pr) * K;
         float a = 0.f, b = 0.f;
-        for (int k = lane; k < K; k += 32) { a = fmaf(w0[k], x[k], a); if (GATEUP) b = fmaf(w1[k], x[k], b); }
+        for (int k = lane; k < K; k += 32) { a = fmaf(w0[k], x[k], a); if (gated) b = fmaf(w1[k], x[k], b); }
         a = warp_sum(a);
         if (GATEUP) {
             b = warp_sum(b);
             const float c = glu_in_scale(ga, pr);
-            a = glu_act<true>(a * c, b * c, ga);
+            a = gated ? glu_act<true>(a * c, b * c, ga) : relu2_act(a * c);
         }
         if (lane == 0) out[(size_t)pr * N + n_out] = a;
     }
@@ -644,6 +645,7 @@ static int moe_gateup(const void* x, const void* arena, const void* slot_of, con
                       void* stream) {
     ExpertFmt ef = *reinterpret_cast<const ExpertFmt*>(fmt_struct);
     cudaStream_t st = (cudaStream_t)stream;
+    if (ga.unit && ef.fmt != 0 && ef.fmt != 7) return -1;      // experts without a gate: bf16 and fp32 weights
     if (ef.fmt == 2 && ef.F % 128 == 0 && ef.H % 128 == 0) {   // K % 64 == 0 follows
         // run: values of n % 32 per block (8, 4 or 2; 0 = 8) - see the kernel
         if (run != 2 && run != 4) run = 8;
@@ -674,7 +676,8 @@ static int moe_gateup(const void* x, const void* arena, const void* slot_of, con
     dim3 grid((ef.F + 7) / 8, max_groups);
 #define ARGS (const bf16*)x, (const uint8_t*)arena, (const int*)slot_of, ef, (const int*)group_expert, (const int*)group_n, \
              (const int*)group_pairs, (const int*)n_groups, (bf16*)act, S, ga, (int*)miss_flag
-    if (ef.fmt == 0) launch_pdl((moe_gateup_kernel<0>), grid, 256, 0, st, ARGS);
+    if (ef.fmt == 0 && ga.unit) launch_pdl((moe_gateup_kernel<0, false>), grid, 256, 0, st, ARGS);
+    else if (ef.fmt == 0) launch_pdl((moe_gateup_kernel<0>), grid, 256, 0, st, ARGS);
     else if (ef.fmt == 1) launch_pdl((moe_gateup_kernel<1>), grid, 256, 0, st, ARGS);
     else if (ef.fmt == 2) launch_pdl((moe_gateup_kernel<2>), grid, 256, 0, st, ARGS);
     else if (ef.fmt == 3) launch_pdl((moe_gateup_kernel<3>), grid, 256, 0, st, ARGS);
@@ -700,6 +703,13 @@ LSB_API int lsb_moe_gateup_act(const void* x, const void* arena, const void* slo
                                void* stream) {
     return moe_gateup(x, arena, slot_of, fmt_struct, group_expert, group_n, group_pairs, n_groups, act, S, max_groups,
                       GluAct{limit, alpha, shift, (const float*)in_scale}, miss_flag, run, stream);
+}
+
+// Experts without a gate: act = relu(up x)^2 (bf16 and fp32 weights).
+LSB_API int lsb_moe_up(const void* x, const void* arena, const void* slot_of, const void* fmt_struct, const void* group_expert, const void* group_n,
+                       const void* group_pairs, const void* n_groups, void* act, int S, int max_groups, void* miss_flag, void* stream) {
+    return moe_gateup(x, arena, slot_of, fmt_struct, group_expert, group_n, group_pairs, n_groups, act, S, max_groups, GluAct{0.f, 1.f, 0.f, nullptr, 1}, miss_flag, 0,
+                      stream);
 }
 
 LSB_API int lsb_moe_down(const void* act, const void* arena, const void* slot_of, const void* fmt_struct,

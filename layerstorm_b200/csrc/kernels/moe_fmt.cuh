@@ -19,9 +19,11 @@ struct ExpertFmt {
 
 // Activation of a gated unit: g = min(g, limit), u = clamp(u, -limit, limit) (limit 0: as they are), then g sigmoid(alpha g) (u + shift).
 // in_scale: one factor per (row, slot) pair on the unit's input - the products are linear in it, so it multiplies g and u in fp32 - or null.
-struct GluAct { float limit, alpha, shift; const float* in_scale; };
+// unit 1: no gate, the square of relu(u).
+struct GluAct { float limit, alpha, shift; const float* in_scale; int unit = 0; };
 
 #ifdef __CUDACC__
+__device__ __forceinline__ float relu2_act(float u) { const float r = fmaxf(u, 0.f); return r * r; }
 template <bool EXACT = false> __device__ __forceinline__ float glu_act(float g, float u, const GluAct& a) {
     if (a.limit > 0.f) { g = fminf(g, a.limit); u = fminf(fmaxf(u, -a.limit), a.limit); }
     if (EXACT) return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);

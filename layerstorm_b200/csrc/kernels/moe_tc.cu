@@ -247,6 +247,7 @@ struct MoeTcParams {
     // dense-linear mode of the down kernel (one "expert" = the whole matrix): row stride and type of the output and the
     // per-tensor scale (0 = read it from the slot tail)
     int ldo, out_bf16; float down_scale;
+    int up;               // one-matrix form of the kernel over the up matrices of experts without a gate: relu(up x)^2 into `act`
 };
 
 template <int FMT, int BN, bool GATEUP> struct MoeTcCfg {
@@ -347,8 +348,9 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
     uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(acc_empty + 2);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int K = GATEUP ? p.ef.H : p.ef.F;          // reduction length
-    const int NOUT = GATEUP ? p.ef.F : p.ef.H;       // weight rows
+    const bool up = !GATEUP && p.up;
+    const int K = GATEUP || up ? p.ef.H : p.ef.F;          // reduction length
+    const int NOUT = GATEUP || up ? p.ef.F : p.ef.H;       // weight rows
     const int NT = NOUT / kTBM;
     const int nkb = K / kTBK;
 
@@ -392,7 +394,7 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                 work_item(w, ntiles, NT, t, jn);
                 const int e = p.tile_expert[t];
                 if (!slot_ok(p.slot_of[e])) {
-                    if (GATEUP && p.miss_flag && jn == 0) atomicExch(p.miss_flag, e + 1);
+                    if ((GATEUP || up) && p.miss_flag && jn == 0) atomicExch(p.miss_flag, e + 1);
                     continue;
                 }
                 const int row0 = p.tile_row0[t];
@@ -422,7 +424,7 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                 const int slot = p.slot_of[p.tile_expert[t]];
                 if (!slot_ok(slot)) continue;
                 const uint8_t* base = p.arena + (size_t)slot * p.ef.stride;
-                const uint8_t* sf0 = base + (GATEUP ? p.ef.off_sg : p.ef.off_sd);
+                const uint8_t* sf0 = base + (GATEUP ? p.ef.off_sg : (up ? p.ef.off_su : p.ef.off_sd));
                 const uint8_t* sf1 = base + p.ef.off_su;
                 const int gtiles = ((K >> 4) + 3) >> 2;        // NVFP4: 512-byte scale atoms per 128-row tile
                 for (int it = 0; it < nkb; ++it, ++g) {
@@ -504,8 +506,8 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
             const int slot = p.slot_of[p.tile_expert[t]];
             if (!slot_ok(slot)) continue;
             const uint8_t* base = p.arena + (size_t)slot * p.ef.stride;
-            const uint8_t* wm = base + (GATEUP ? (part ? p.ef.off_up : p.ef.off_gate) : p.ef.off_down);
-            const uint8_t* sf = base + (GATEUP ? (part ? p.ef.off_su : p.ef.off_sg) : p.ef.off_sd);
+            const uint8_t* wm = base + (GATEUP ? (part ? p.ef.off_up : p.ef.off_gate) : (up ? p.ef.off_up : p.ef.off_down));
+            const uint8_t* sf = base + (GATEUP ? (part ? p.ef.off_su : p.ef.off_sg) : (up ? p.ef.off_su : p.ef.off_sd));
             const int n = jn * kTBM + row;                     // weight row in the expert matrix
             // side data that does not travel through the ring: the FP8 block scale (one float per 128 x 128 block, the
             // same for the whole tile) and the Q4_K super-block header (16 bytes per row and 256 elements), both read
@@ -593,7 +595,7 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                 float sg = 1.f, su = 1.f;
                 if (FMT == 2 && (GATEUP || p.down_scale == 0.f)) {
                     const float* tail = reinterpret_cast<const float*>(base + p.ef.off_tail);
-                    if (GATEUP) { sg = tail[0]; su = tail[1]; } else sg = tail[2];
+                    if (GATEUP) { sg = tail[0]; su = tail[1]; } else sg = tail[up ? 1 : 2];
                 } else if (FMT == 2) {
                     sg = p.down_scale;
                 } else if (FMT == 1) {
@@ -615,6 +617,9 @@ __global__ void __launch_bounds__(MoeTcCfg<FMT, BN, GATEUP>::THREADS) moe_tc_ffn
                         if (c0 + j < ncols && n < NOUT) {
                             if (GATEUP) {
                                 p.act[(size_t)(row0 + c0 + j) * NOUT + n] = __float2half_rn(glu_act(gq[j] * sg * c, uq[j] * su * c, p.ga));
+                            } else if (up) {
+                                // (fp16 range: far outside what normed inputs reach, kept finite all the same)
+                                p.act[(size_t)(row0 + c0 + j) * NOUT + n] = __float2half_rn(fminf(relu2_act(gq[j] * sg), 65504.f));
                             } else if (ep_mode) {
                                 const int2 ra = p.ep.ret[p.ep.rank][row0 + c0 + j];      // (token owner, pair index there)
                                 p.ep.y[ra.x][(size_t)ra.y * NOUT + n] = gq[j] * sg;       // NVLink store into the owner's buffer
@@ -676,7 +681,7 @@ static int sm_count() {
 template <int FMT, int BN, bool GATEUP>
 static int launch_moe_tc(const CUtensorMap& mb, const MoeTcParams& p, int nout, int max_tiles, cudaStream_t st) {
     using CVt = typename MoeTcCfg<FMT, BN, GATEUP>::CV;
-    const int Kred = GATEUP ? p.ef.H : p.ef.F;
+    const int Kred = GATEUP || p.up ? p.ef.H : p.ef.F;
     CUtensorMap mw0, mw1;
     {
         // byte views of the weight matrices over every slot of the arena (dense mode: one "slot")
@@ -684,7 +689,7 @@ static int launch_moe_tc(const CUtensorMap& mb, const MoeTcParams& p, int nout, 
         const bool dense = p.ef.stride == 0;
         const uint64_t sstride = dense ? pitch * (uint64_t)nout : (uint64_t)p.ef.stride;
         const uint64_t nslots = dense ? 1 : (uint64_t)kMaxSlots;
-        int rc = cached_map_w(&mw0, p.arena + (GATEUP ? p.ef.off_gate : p.ef.off_down), pitch, (uint64_t)nout, sstride, nslots, CVt::SBYTES);
+        int rc = cached_map_w(&mw0, p.arena + (GATEUP ? p.ef.off_gate : (p.up ? p.ef.off_up : p.ef.off_down)), pitch, (uint64_t)nout, sstride, nslots, CVt::SBYTES);
         if (rc) return rc;
         if (GATEUP) { rc = cached_map_w(&mw1, p.arena + p.ef.off_up, pitch, (uint64_t)nout, sstride, nslots, CVt::SBYTES); if (rc) return rc; }
         else mw1 = mw0;
@@ -745,6 +750,7 @@ LSB_API int lsb_moe_tc_gather(const void* x, const void* sorted_pair, const void
 
 // gateup != 0: act[pos][f] = SwiGLU(xs[pos] . Wgate[f], xs[pos] . Wup[f]) for every sorted position (fp16, [cap_rows, F]).
 // gateup == 0: y[pair][h] = act[pos] . Wdown[h]  (fp32, [npairs, H], rows in pair order).
+// gateup == 2: act[pos][f] = relu(xs[pos] . Wup[f])^2 (experts without a gate).
 // `b` is the fp16 token operand ([cap_rows, K], K = H for gate/up and F for down), 16-byte aligned.
 static int moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* arena, const void* slot_of, const void* fmt_struct,
                            const void* tile_expert, const void* tile_row0, const void* tile_n, const void* counters,
@@ -752,6 +758,7 @@ static int moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* arena
                            const void* ep, void* stream) {
     const ExpertFmt* ef = (const ExpertFmt*)fmt_struct;
     const int K = gateup ? ef->H : ef->F, nout = gateup ? ef->F : ef->H;
+    if (gateup == 2 && ep) return -1;
     if (K % kTBK || nout % kTBM || ((uintptr_t)b & 15)) return -1;
     if (ef->fmt == 1 && (K % 128)) return -1;
     if (ef->fmt == 3 && (K % 256)) return -1;
@@ -765,9 +772,9 @@ static int moe_tc_ffn(int gateup, const void* b, int cap_rows, const void* arena
     p.act = gateup ? (__half*)out : nullptr; p.y = gateup ? nullptr : (float*)out;
     p.ga = ga; p.miss_flag = (int*)miss_flag; p.err = (int*)err;
     if (ep) p.ep = *(const EpComm*)ep; else { memset(&p.ep, 0, sizeof(p.ep)); }
-    p.ldo = nout; p.out_bf16 = 0; p.down_scale = 0.f;
+    p.ldo = nout; p.out_bf16 = 0; p.down_scale = 0.f; p.up = gateup == 2;
     cudaStream_t st = (cudaStream_t)stream;
-    if (gateup) {
+    if (gateup == 1) {
         switch (BN) {
             case 32: return dispatch_fmt<32, true>(ef->fmt, mb, p, nout, max_tiles, st);
             case 64: return dispatch_fmt<64, true>(ef->fmt, mb, p, nout, max_tiles, st);

@@ -938,4 +938,146 @@ LSB_API int lsb_norm_rows(void* out, int ldo, const void* resid, int ldr, const 
     LSB_CHECK_LAUNCH();
 }
 
+namespace lsb {
+// ---- hyper-connections with static mixing: n copies of the residual stream per row ----
+// x_t <- sum_s mix[s][t] x_s + out[t] mult y for all t at once, u = sum_t in[t] x_t (in null: plain sum), next input = pre(u).
+// y: the sublayer's result sub; with norms (w_a) the mean of sub and sub2, each RMS-normed; plus the row's expert sum.
+struct StreamMix { const float* mix; const float* out; const float* in; float mult; };
+struct StreamSub { const float* a; const float* b; int ld; const float* w_a; const float* w_b; };
+
+template <int V> __device__ __forceinline__ void ldv(const float* p, float (&v)[V]) {
+    if constexpr (V == 4) { const float4 f = *reinterpret_cast<const float4*>(p); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+    else v[0] = *p;
+}
+template <int V> __device__ __forceinline__ void stv(float* p, const float (&v)[V]) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+}
+
+// first: [rows, ldr], the streams' common start (mix, out and y are not used).  sum: [rows, ldr] takes u (or null).  x may be null.
+template <typename T, int N, int V>
+__global__ void __launch_bounds__(1024) stream_update_kernel(T* __restrict__ x, int ldx, float* __restrict__ streams, int ldr, int n, const float* __restrict__ first,
+                                                            float* __restrict__ sum, StreamSub sub, StreamMix hc, NormW pre, MoeSum mo) {
+    constexpr int NS = N ? N : 8;
+    __shared__ float red[33], s_w[32], s_mix[NS * NS], s_out[NS], s_in[NS];
+    __shared__ int s_id[32];
+    extern __shared__ float row[];
+    const int r = blockIdx.x, dim = pre.dim, cnt = N ? N : n, t0 = threadIdx.x * V, dt = blockDim.x * V;
+    if ((int)threadIdx.x < cnt * cnt && !first) s_mix[threadIdx.x / cnt * NS + threadIdx.x % cnt] = hc.mix[threadIdx.x];
+    if ((int)threadIdx.x < cnt) { s_out[threadIdx.x] = first ? 0.f : hc.mult * hc.out[threadIdx.x]; s_in[threadIdx.x] = hc.in ? hc.in[threadIdx.x] : 1.f; }
+    pdl_wait();
+    pdl_launch_dependents();
+    if (mo.y) load_slots(mo, r, s_id, s_w);
+    __syncthreads();
+    const float* pa = sub.a ? sub.a + (size_t)r * sub.ld : nullptr;
+    const float* pb = sub.b ? sub.b + (size_t)r * sub.ld : nullptr;
+    float ra = 1.f, rb = 1.f;
+    if (sub.w_a) {
+        float qa = 0.f, qb = 0.f;
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) { qa = fmaf(pa[i], pa[i], qa); qb = fmaf(pb[i], pb[i], qb); }
+        ra = 0.5f / sqrtf(block_sum(qa, red) / (float)dim + pre.eps);
+        rb = 0.5f / sqrtf(block_sum(qb, red) / (float)dim + pre.eps);
+    }
+    float* st = streams + (size_t)r * cnt * ldr;
+    for (int i = t0; i < dim; i += dt) {
+        float nx[NS][V], u[V];
+        if (first) {
+            float f[V];
+            ldv<V>(first + (size_t)r * ldr + i, f);
+#pragma unroll
+            for (int t = 0; t < NS; ++t)
+#pragma unroll
+                for (int v = 0; v < V; ++v) nx[t][v] = f[v];
+        } else {
+            float y[V], o[V];
+#pragma unroll
+            for (int v = 0; v < V; ++v) y[v] = 0.f;
+            if (pa) ldv<V>(pa + i, y);
+            if (sub.w_a) {
+                float w[V];
+                ldv<V>(sub.w_a + i, w);
+#pragma unroll
+                for (int v = 0; v < V; ++v) y[v] = y[v] * ra * w[v];
+                ldv<V>(pb + i, o);
+                ldv<V>(sub.w_b + i, w);
+#pragma unroll
+                for (int v = 0; v < V; ++v) y[v] = fmaf(o[v] * rb, w[v], y[v]);
+            }
+            if (mo.y) {
+                const float* yr = mo.y + (size_t)r * mo.S * mo.ldy + i;
+#pragma unroll 4
+                for (int s = 0; s < mo.S; ++s) {
+                    if (s_id[s] < 0) continue;
+                    ldv<V>(yr + (size_t)s * mo.ldy, o);
+#pragma unroll
+                    for (int v = 0; v < V; ++v) y[v] = fmaf(s_w[s], o[v], y[v]);
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < NS; ++t)
+#pragma unroll
+                for (int v = 0; v < V; ++v) nx[t][v] = t < cnt ? s_out[t] * y[v] : 0.f;
+#pragma unroll
+            for (int s = 0; s < NS; ++s) {
+                if (s >= cnt) continue;
+                ldv<V>(st + (size_t)s * ldr + i, o);
+#pragma unroll
+                for (int t = 0; t < NS; ++t)
+#pragma unroll
+                    for (int v = 0; v < V; ++v) nx[t][v] = t < cnt ? fmaf(s_mix[s * NS + t], o[v], nx[t][v]) : 0.f;
+            }
+        }
+#pragma unroll
+        for (int v = 0; v < V; ++v) u[v] = 0.f;
+#pragma unroll
+        for (int t = 0; t < NS; ++t) {
+            if (t >= cnt) continue;
+            stv<V>(st + (size_t)t * ldr + i, nx[t]);
+#pragma unroll
+            for (int v = 0; v < V; ++v) u[v] = fmaf(s_in[t], nx[t][v], u[v]);
+        }
+        if (sum) stv<V>(sum + (size_t)r * ldr + i, u);
+        stv<V>(row + i, u);
+    }
+    if (!x) return;
+    __syncthreads();
+    float mean, rstd;
+    norm_moments(row, pre, red, mean, rstd);
+    const float alpha = pre.alpha ? *pre.alpha : 0.f;
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) x[(size_t)r * ldx + i] = as_act<T>(norm_apply(row[i], i, pre, mean, rstd, alpha));
+}
+
+template <typename T, int V>
+static void launch_streams(T* x, int ldx, float* streams, int ldr, int n, const float* first, float* sum, const StreamSub& sub, const StreamMix& hc, const NormW& pre,
+                           const MoeSum& mo, int rows, cudaStream_t st) {
+    const int dim = pre.dim, thr = norm_threads(dim, rows);
+#define LSB_SU(N) LSB_SUV(N, V)
+#define LSB_SUV(N, VV) launch_pdl((stream_update_kernel<T, N, VV>), rows, thr, (size_t)(dim + 3) / 4 * 16, st, x, ldx, streams, ldr, n, first, sum, sub, hc, pre, mo)
+    switch (n) { case 1: LSB_SU(1); break; case 2: LSB_SU(2); break; case 3: LSB_SU(3); break; case 4: LSB_SU(4); break; default: LSB_SUV(0, 1); }
+#undef LSB_SU
+#undef LSB_SUV
+}
+}  // namespace lsb
+
+// One step of the hyper-connections (see StreamMix): streams fp32 [rows, n, ldr].  `first` non-null starts them.  sub2 / w_a / w_b: the two results of mixers
+// side by side and their norms' weights; y .. ldy: the expert sum as in lsb_resid_update (wts null: as they are).  x null: no norm behind it.
+LSB_API int lsb_stream_update(void* x, int ldx, void* streams, int ldr, int n, const void* first, void* sum, const void* sub, const void* sub2, int lds,
+                              const void* w_a, const void* w_b, const void* mix, const void* out, float mult, const void* in_next, int pre_kind,
+                              const void* pre_w, const void* pre_b, const void* pre_alpha, int rows, int dim, float eps, const void* y, const void* wts,
+                              const void* ids, const void* slot_of, int S, int experts, int ldy, int f32, void* stream) {
+    if (rows < 1 || dim < 1 || dim > 12000 || n < 1 || n > 8 || (y && S > 32) || (!first && (!mix || !out)) || (w_a && (!sub || !sub2 || !w_b))) return -1;
+    if (pre_kind < 0 || pre_kind > kNormNone || (pre_kind != kNormNone && !pre_w) || (pre_kind == kNormTanh && !pre_alpha)) return -1;
+    const NormW pre{(const float*)pre_w, (const float*)pre_b, (const float*)pre_alpha, dim, eps, pre_kind};
+    const MoeSum mo{(const float*)y, (const float*)wts, (const int*)ids, (const int*)slot_of, S, experts, ldy};
+    const StreamMix hc{(const float*)mix, (const float*)out, (const float*)in_next, mult};
+    const StreamSub sb{(const float*)sub, (const float*)sub2, lds, (const float*)w_a, (const float*)w_b};
+    cudaStream_t st = (cudaStream_t)stream;
+    const bool vec = dim % 4 == 0 && ldr % 4 == 0 && lds % 4 == 0 && ldy % 4 == 0;
+#define LSB_SL(T, V) launch_streams<T, V>((T*)x, ldx, (float*)streams, ldr, n, (const float*)first, (float*)sum, sb, hc, pre, mo, rows, st)
+    if (f32) { if (vec) LSB_SL(float, 4); else LSB_SL(float, 1); }
+    else { if (vec) LSB_SL(bf16, 4); else LSB_SL(bf16, 1); }
+#undef LSB_SL
+    LSB_CHECK_LAUNCH();
+}
+
 LSB_API int lsb_trace_set_norm(void* buf) { return lsb_trace_install(buf); }

@@ -1,14 +1,18 @@
-"""Models described layer by layer (``ModelConfig.blocks``) on the device: every layer is a mixer (grouped-query attention, latent attention or
-a gated delta rule) and an optional feed-forward (a dense gated unit or routed experts), each with its own sizes, around an fp32 residual stream.
-The norms stand on every sublayer's output (``norm_place`` "post") or on both its sides ("sandwich"; n_in is the identity for "post"):
+"""Models described layer by layer (``ModelConfig.blocks``) on the device: every layer is a mixer (grouped-query attention, latent attention, a
+gated delta rule, time mixing, or two of them side by side) and an optional feed-forward (a dense gated unit or routed experts), each with its own
+sizes, around an fp32 residual stream.  The norms stand on every sublayer's output (``norm_place`` "post"), in front of it ("pre") or on both its
+sides ("sandwich"; n_in is the identity for "post", n_out for "pre"):
 
     x <- x + n_out(mixer(n_in(x))),    x <- x + n_out(ffn(n_in(x))),    logits = head(norm(x)) * logit_scale,
 
-and a layer may end with an update from its slice e of a per-token table: x <- x + rms(W_p (gelu(W_g x) * e)).
+and a layer may end with an update from its slice e of a per-token table: x <- x + rms(W_p (gelu(W_g x) * e)).  With ``streams`` there are n copies of
+the stream and every sublayer reads and updates them through learned static weights (in, out, mix):
+
+    u = sum_s in_s x_s,    y = residual_mult * f(n_in(u)),    x_t <- sum_s mix_st x_s + out_t y,    logits = head(norm(sum_t x_t)).
 
 Same engine, caches and step protocol as :class:`DeviceModel`: attention layers keep a paged cache (one row of all heads' keys and values per
-token; latent layers one row for all heads, which later layers may read instead of keeping their own), delta-rule layers an fp32 state and
-convolution history per sequence slot.  Steps are any mixture of prompt portions and single tokens.
+token; latent layers one row for all heads, which later layers may read instead of keeping their own), recurrent layers an fp32 state per sequence
+slot with the convolutions' history (delta rule) or the previous token's input (time mixing); layers with two mixers side by side have both.  Steps are any mixture of prompt portions and single tokens.
 
 Two precisions.  ``bfloat16``: weights, activations and the cache in bf16, products accumulated in fp32; the residual stream, norms, routing,
 attention scores and weights, rotations and the whole recurrence in fp32.  ``float32``: everything in fp32 (FMA units, no reduced-precision
@@ -34,6 +38,66 @@ EXPAND_ROWS = 128       # rows of a step of one sequence from which latent layer
 EXPAND_BYTES = 1 << 30  # ... while those of all its positions fit this much scratch
 NORM_KIND = {"rms": 0, "layer": 1, "tanh": 2}        # as the kernels number them; 3: none
 NO_NORM = (3, None, None, None)
+HEAD_NORM = {"": 0, "plain": 1, "weight": 2}
+
+
+def _sides(b: BlockSpec) -> list:
+    """[(name part, mixer)] of a layer: one mixer, or two side by side."""
+    return list(zip(("left.", "right."), b.branches)) if b.branches else [("", b)]
+
+
+def _mixer_shapes(out: dict, p: str, b: BlockSpec, H: int, ranks: tuple):
+    """Adds the tensors of a mixer, named behind ``p``."""
+    if b.delta:
+        k, kw, vw = p + "kda.", b.kv_heads * b.dim, b.heads * b.vdim
+        ra, rg = ranks
+        out.update({k + "q": (kw, H), k + "k": (kw, H), k + "v": (vw, H), k + "beta": (b.heads, H), k + "conv_q": (kw, b.conv), k + "conv_k": (kw, b.conv),
+                    k + "conv_v": (vw, b.conv), k + "a_log": (b.heads,), k + "o_norm": (b.vdim,), k + "o": (H, vw)})
+        if b.kind == "head_delta":
+            out.update({k + "a": (b.heads, H), k + "g": (vw, H), k + "dt_bias": (b.heads,)})
+        else:
+            out.update({k + "f_a": (ra, H), k + "g_a": (rg, H), k + "f_b": (b.heads * b.dim, ra), k + "g_b": (vw, rg), k + "dt_bias": (b.heads * b.dim,)})
+    elif b.kind == "time_mix":
+        k, kw, vw = p + "tmix.", b.heads * b.dim, b.heads * b.vdim
+        out.update({k + "r": (kw, H), k + "k": (kw, H), k + "v": (vw, H), k + "g": (vw, H), k + "w1": (ranks[0], H), k + "w2": (kw, ranks[0]), k + "w0": (kw,),
+                    k + "u": (b.heads, b.dim), k + "o_norm": (vw,), k + "o": (H, vw)} | {k + "mu_" + n: (H,) for n in "rkvgw"})
+    elif b.latent:
+        a = p + "attn."
+        out.update({a + "q": (b.heads * (b.dim + b.rot_dim), H), a + "k_b": (b.heads * b.dim, b.kv_rank), a + "v_b": (b.heads * b.vdim, b.kv_rank),
+                    a + "o": (H, b.heads * b.vdim)})
+        if b.kv_from < 0:
+            out.update({a + "kv_a": (b.kv_rank + b.rot_dim, H), a + "kv_a_norm": (b.kv_rank,)})
+        if b.head_gate:
+            out[a + "g"] = (b.heads, H)
+    else:
+        a, qw, kw, vw = p + "attn.", b.heads * b.dim, b.kv_heads * b.dim, b.kv_heads * b.vdim
+        out.update({a + "q": (qw, H), a + "k": (kw, H), a + "v": (vw, H), a + "o": (H, b.heads * b.vdim)})
+        if b.qkv_bias:
+            out.update({a + "q_bias": (qw,), a + "k_bias": (kw,), a + "v_bias": (vw,)})
+        if b.qk_norm:
+            out.update({a + "q_norm": (qw,), a + "k_norm": (kw,)})
+        if b.head_norm == "weight":
+            out.update({a + "q_norm": (b.dim,), a + "k_norm": (b.dim,)})
+        if b.bias_rows:
+            out[a + "rel"] = (b.bias_rows, b.heads)
+        if b.out_gate or b.head_gate:
+            out[a + "g"] = (b.heads * (b.vdim if b.out_gate else 1), H)
+        if b.v_mix:
+            out[a + "v_mix"] = ()
+
+
+def distance_buckets(rows: int, reach: int) -> List[int]:
+    """Rows of a learned distance bias table for distances 0 .. reach (further ones: the last): one each up to half the rows, then logarithmic,
+    half + floor(log(n / half) / log(reach / half) * (rows - half)).  In integers, so that distances on a border fall where the formula says."""
+    half = rows // 2
+    if half < 1 or reach <= half:
+        raise ValueError(f"a distance bias of {rows} rows up to distance {reach}")
+    m, out, k = rows - half, list(range(half)), 0
+    for n in range(half, reach + 1):
+        while k < m - 1 and n ** m * half ** (k + 1) >= reach ** (k + 1) * half ** m:
+            k += 1
+        out.append(half + k)
+    return out
 
 
 def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = None) -> Dict[str, tuple]:
@@ -50,29 +114,13 @@ def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = No
         norm(p + "mix_norm")
         if cfg.norm_place == "sandwich":
             norm(p + "mix_post_norm")
-        if b.recurrent:
-            k, kw, vw = p + "kda.", b.kv_heads * b.dim, b.heads * b.vdim
-            ra, rg = (ranks or {}).get(i, (b.dim, b.dim))
-            out.update({k + "q": (kw, H), k + "k": (kw, H), k + "v": (vw, H), k + "beta": (b.heads, H), k + "f_a": (ra, H), k + "g_a": (rg, H),
-                        k + "f_b": (b.heads * b.dim, ra), k + "g_b": (vw, rg), k + "conv_q": (kw, b.conv), k + "conv_k": (kw, b.conv), k + "conv_v": (vw, b.conv),
-                        k + "a_log": (b.heads,), k + "dt_bias": (b.heads * b.dim,), k + "o_norm": (b.vdim,), k + "o": (H, vw)})
-        elif b.latent:
-            a = p + "attn."
-            out.update({a + "q": (b.heads * (b.dim + b.rot_dim), H), a + "k_b": (b.heads * b.dim, b.kv_rank), a + "v_b": (b.heads * b.vdim, b.kv_rank),
-                        a + "o": (H, b.heads * b.vdim)})
-            if b.kv_from < 0:
-                out.update({a + "kv_a": (b.kv_rank + b.rot_dim, H), a + "kv_a_norm": (b.kv_rank,)})
-            if b.head_gate:
-                out[a + "g"] = (b.heads, H)
-        else:
-            a, qw, kw, vw = p + "attn.", b.heads * b.dim, b.kv_heads * b.dim, b.kv_heads * b.vdim
-            out.update({a + "q": (qw, H), a + "k": (kw, H), a + "v": (vw, H), a + "o": (H, b.heads * b.vdim)})
-            if b.qk_norm:
-                out.update({a + "q_norm": (qw,), a + "k_norm": (kw,)})
-            if b.out_gate:
-                out[a + "g"] = (b.heads * b.vdim, H)
-            if b.v_mix:
-                out[a + "v_mix"] = ()
+        for side, m in _sides(b):
+            _mixer_shapes(out, p + side, m, H, (ranks or {}).get(i, (m.dim, m.dim)))
+            if b.branches and b.join == "normed":
+                out[p + side + "out_norm"] = (H,)
+        if cfg.streams:
+            for q in ["mix_hc"] + (["ffn_hc"] if b.has_ff else []):
+                out.update({f"{p}{q}.in": (cfg.streams,), f"{p}{q}.out": (cfg.streams,), f"{p}{q}.mix": (cfg.streams, cfg.streams)})
         if b.has_ff:
             norm(p + "ffn_norm")
             if cfg.norm_place == "sandwich":
@@ -87,6 +135,8 @@ def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = No
                 out[m + "router_bias"] = (b.experts + b.identity,)
             for e in range(b.experts):
                 glu(m + f"experts.{e}.", b.ff)
+                if b.unit != "glu":
+                    del out[m + f"experts.{e}.gate"]
             if b.shared_ff:
                 glu(m + "shared.0.", b.shared_ff)
                 out[m + "shared_gate"] = (1, H)
@@ -107,9 +157,19 @@ def random_block_tensor(name: str, shape: tuple, gen: torch.Generator, device="c
         return t.uniform_(-3.0, -1.0, generator=gen)
     if leaf.startswith("conv_"):
         return t.uniform_(-0.7, 0.7, generator=gen)
+    if leaf.startswith("mu_"):
+        return t.uniform_(0.1, 0.9, generator=gen)
+    if leaf == "w0":
+        return t.uniform_(-5.0, 0.5, generator=gen)
+    if leaf in ("in", "out") and len(shape) == 1:
+        return t.uniform_(0.6, 1.2, generator=gen)
+    if leaf == "mix" and "_hc" in name:
+        return t.normal_(0.0, 0.15, generator=gen).add_(torch.eye(shape[0], device=device))
+    if leaf in ("rel", "u"):
+        return t.normal_(0.0, 0.5, generator=gen)
     if leaf == "v_mix":
         return t.uniform_(0.2, 0.6, generator=gen)
-    if leaf in ("bias", "router_bias"):
+    if leaf in ("bias", "router_bias", "q_bias", "k_bias", "v_bias"):
         return t.normal_(0.0, 0.1, generator=gen)
     if leaf == "alpha":
         return t.uniform_(0.4, 1.0, generator=gen)
@@ -145,7 +205,10 @@ class BlockWorkspace(StepBuffers):
         self.proj = z(R, m.max_proj)
         self.mix = z(R, m.max_mix, dtype=act)        # a mixer's output in front of its output projection
         lat = [b for b in m.cfg.blocks if b.latent]
-        att = [b for b in m.cfg.blocks if not b.recurrent and not b.latent]
+        att = [(i, b) for i, L in enumerate(m.cfg.blocks) for b in L.mixers if b.softmax]
+        self.streams = z(R, m.cfg.streams, Hp) if m.cfg.streams else None
+        self.sub2 = z(R, Hp) if any(b.join == "normed" and b.branches for b in m.cfg.blocks) else None
+        self.xs = z(5, R, Hp, dtype=act) if any(b.kind == "time_mix" for L in m.cfg.blocks for b in L.mixers) else None      # token-shifted inputs
         if lat:
             self.q_lat = z(R * max(b.heads * m.latent_row(b) for b in lat), dtype=act)
             self.q_nope = z(R * max(b.heads * _align(b.dim, 8) for b in lat), dtype=torch.bfloat16) if not m.f32 and R >= 8 else None
@@ -160,16 +223,15 @@ class BlockWorkspace(StepBuffers):
         self.glu = z(R * dense, dtype=act) if dense else None
         self.side = z(R, _align(m.cfg.side_dim, 8), dtype=act) if m.cfg.side_dim else None
         if att:
-            self.q = z(R * max(b.heads * m.head_pad(b.dim) for b in att), dtype=act)
-            self.v_first = z(R, max([b.kv_heads * b.vdim for b in att if b.v_mix], default=1))
+            self.q = z(R * max(b.heads * m.head_pad(b.dim) for _, b in att), dtype=act)
+            self.v_first = z(R, max([b.kv_heads * b.vdim for _, b in att if b.v_mix], default=1))
             # key splits of the few-row attention: about two blocks per SM, no split shorter than 64 visible keys
             self.splits = {}
-            for i, b in enumerate(m.cfg.blocks):
-                if not b.recurrent and not b.latent:
-                    seen = min(b.window or max_ctx, max_ctx)
-                    blocks = R * b.kv_heads * ((b.heads // b.kv_heads + 15) // 16)
-                    self.splits[i] = 1 if (m.f32 or R > 64) else max(1, min(32, 296 // blocks, (seen + 63) // 64))
-            ns = [(b.heads * self.splits[i], m.head_pad(b.vdim)) for i, b in enumerate(m.cfg.blocks) if self.splits.get(i, 1) > 1]
+            for i, b in att:
+                seen = min(b.window or max_ctx, b.chunk or max_ctx, max_ctx)
+                blocks = R * b.kv_heads * ((b.heads // b.kv_heads + 15) // 16)
+                self.splits[i] = 1 if (m.f32 or R > 64) else max(1, min(32, 296 // blocks, (seen + 63) // 64))
+            ns = [(b.heads * self.splits[i], m.head_pad(b.vdim)) for i, b in att if self.splits[i] > 1]
             self.o_part = z(R * max((n * w for n, w in ns), default=1))
             self.ml_part = z(2 * R * max((n for n, _ in ns), default=1))
         self.moe: Dict[tuple, MoeBuffers] = {}
@@ -182,7 +244,7 @@ class BlockWorkspace(StepBuffers):
                     mb.tc_xs = z(R * b.top, arena.ef.H, dtype=torch.float16)
                     mb.tc_act = z(R * b.top, arena.ef.F, dtype=torch.float16)
                 self.moe[m.moe_key(i)] = mb
-        self._delta = self._chunk = None
+        self._delta = self._chunk = self._tmix = None
 
     def delta_scratch(self, b: BlockSpec, R: int, ra: int, rg: int, chunks: int):
         """Scratch of the row-parallel form of a delta-rule layer (grown on first use; decode steps never ask for it)."""
@@ -195,6 +257,15 @@ class BlockWorkspace(StepBuffers):
         if c and (self._chunk is None or self._chunk.numel() < c):
             self._chunk = torch.empty(c, dtype=torch.float32, device=self.dev)
         return self._delta, self._chunk
+
+    def tmix_scratch(self, b: BlockSpec, R: int, chunks: int, rank: int):
+        """Scratch of the chunked form of a time-mixing layer (grown on first use)."""
+        n = int(nat.call("lsb_tmix_scratch_floats", R, chunks, b.heads, b.dim, b.vdim, rank))
+        if n < 0:
+            raise RuntimeError("the step's time-mixing scratch exceeds 2^31 floats: use a smaller prefill chunk")
+        if self._tmix is None or self._tmix.numel() < n:
+            self._tmix = torch.empty(n, dtype=torch.float32, device=self.dev)
+        return self._tmix
 
 
 class BlockModel(ModelBase):
@@ -221,13 +292,16 @@ class BlockModel(ModelBase):
         self.v_first_layer = mixing[0] if mixing else -1
         if len({cfg.blocks[i].kv_heads * cfg.blocks[i].vdim for i in mixing}) > 1:
             raise ValueError("layers that mix values must have the same number of value channels")
-        for i, b in enumerate(cfg.blocks):
+        if cfg.residual_mult != 1.0 and not cfg.streams or cfg.streams and cfg.norm_place != "pre" or cfg.streams > 8 or cfg.streams and cfg.side_dim:
+            raise ValueError("hyper-connections (up to 8 streams) come with norms in front of the sublayers, a residual factor comes with hyper-connections")
+        for i, b in [(i, m) for i, L in enumerate(cfg.blocks) for m in L.mixers]:
             if b.heads % max(b.kv_heads, 1) or min(b.heads, b.kv_heads, b.dim, b.vdim) < 1:
                 raise ValueError(f"layer {i}: {b.heads} heads over {b.kv_heads} groups of widths {b.dim} / {b.vdim}")
             if b.latent and (b.kv_rank < 1 or b.rot_dim < 2 or b.rot_dim % 2):
                 raise ValueError(f"layer {i}: latent rows of {b.kv_rank} + {b.rot_dim} channels")
             if b.recurrent and b.dim > 256:
                 raise ValueError(f"layer {i}: key heads of up to 256 channels, not {b.dim}")
+        for i, b in enumerate(cfg.blocks):
             if b.experts and (b.top > min(32, b.experts + b.identity) or (b.experts + b.identity) % b.groups or b.groups > 64):
                 raise ValueError(f"layer {i}: router with {b.experts} + {b.identity} outputs, top {b.top}, {b.groups} groups")
 
@@ -262,6 +336,92 @@ class BlockModel(ModelBase):
             r0 += n
         return QLinear(self.w_fmt, w.shape[0], cols, w)
 
+    def _build_mixer(self, w, p: str, b: BlockSpec, M: dict):
+        """Puts a mixer's device tensors into ``M``; returns the projections that read the layer's input as it is, and the output projection.
+        ``M["meta"]`` counts columns from the first of these projections."""
+        dev = self.device
+        if b.delta:
+            k = p + "kda."
+            kw, vw = b.kv_heads * b.dim, b.heads * b.vdim
+            low = b.kind == "channel_delta"
+            parts = [w[k + n].to(dev) for n in (("q", "k", "v", "beta", "f_a", "g_a") if low else ("q", "k", "v", "beta", "a", "g"))]
+            ra = rg = 0
+            if low:
+                fb, gb = w[k + "f_b"].to(dev), w[k + "g_b"].to(dev)
+                ra, rg = _align(fb.shape[1], 8), _align(gb.shape[1], 8)
+                pad = lambda t, n: torch.nn.functional.pad(t.float(), (0, n - t.shape[1])).to(self.act_dtype).contiguous()
+                M["w_a"], M["w_g"] = pad(fb, ra), pad(gb, rg)
+                if not self.f32:
+                    # [W | W]: many rows take the low-rank products on the tensor cores with (hi | lo) activations
+                    M["w_a2"], M["w_g2"] = torch.cat([M["w_a"]] * 2, 1).contiguous(), torch.cat([M["w_g"]] * 2, 1).contiguous()
+            M["meta"] = _Meta(_offsets(parts), ra, rg)
+            for n in ("conv_q", "conv_k", "conv_v"):
+                t = w[k + n].to(dev).float().contiguous()
+                if tuple(t.shape) != ((vw if n == "conv_v" else kw), b.conv):
+                    raise ValueError(f"{k + n}: shape {tuple(t.shape)}")
+                M[n] = t
+            M["a_exp"], M["dt_bias"], M["o_norm"] = torch.exp(self._vec(w[k + "a_log"])), self._vec(w[k + "dt_bias"]), self._vec(w[k + "o_norm"]) * b.out_scale
+            return parts, w[k + "o"].to(dev)
+        if b.kind == "time_mix":
+            k = p + "tmix."
+            own = [w[k + n].to(dev) for n in ("r", "k", "v", "g", "w1")]
+            M["shift"] = self._mat(*own, cols=self.Hp)
+            M["meta"] = _Meta(_offsets(own))
+            M["seg_rows"] = torch.tensor(M["meta"].offs, dtype=torch.int32)
+            M["segs"] = [t.shape[0] for t in own]
+            rank = _align(own[4].shape[0], 8)
+            w2 = w[k + "w2"].to(dev)
+            M["w2"] = torch.nn.functional.pad(w2.float(), (0, rank - w2.shape[1])).to(self.act_dtype).contiguous()
+            M["w22"] = None if self.f32 else torch.cat([M["w2"]] * 2, 1).contiguous()
+            mu = torch.zeros(5, self.Hp, device=dev)
+            for j, n in enumerate("rkvgw"):
+                mu[j, : self.cfg.hidden] = w[k + "mu_" + n].to(dev)
+            M["mu"], M["w0"], M["u"], M["o_norm"] = mu, self._vec(w[k + "w0"]), self._vec(w[k + "u"]), self._vec(w[k + "o_norm"]) * b.out_scale
+            return [], w[k + "o"].to(dev)
+        a = p + "attn."
+        if b.latent:
+            own = b.kv_from < 0
+            names = ["q"] + (["kv_a"] if own else []) + (["g"] if b.head_gate else [])
+            parts = [w[a + n].to(dev) for n in names]
+            at = dict(zip(names, _offsets(parts)))
+            M["meta"] = _Meta([at["q"], at.get("kv_a", -1), at.get("g", -1)])
+            dnp, dlp = _align(b.dim, 8), self.latent_pad(b.kv_rank)
+            uk, uv = w[a + "k_b"].to(dev).view(b.heads, b.dim, b.kv_rank), w[a + "v_b"].to(dev).view(b.heads, b.vdim, b.kv_rank)
+            M["w_uk"] = torch.zeros(b.heads, dlp, dnp, dtype=self.act_dtype, device=dev)
+            M["w_uk"][:, : b.kv_rank, : b.dim] = uk.transpose(1, 2)
+            M["w_uv"] = torch.zeros(b.heads, b.vdim, dlp, dtype=self.act_dtype, device=dev)
+            M["w_uv"][:, :, : b.kv_rank] = uv
+            if not self.f32:
+                # the same two, one after the other per position: what long prompt runs make keys and values with
+                dnw, dvp = _align(b.dim, 16), self.head_pad(b.vdim)
+                M["w_kv"] = torch.zeros(b.heads * (dnw + dvp), dlp, dtype=self.act_dtype, device=dev)
+                M["w_kv"][: b.heads * dnw].view(b.heads, dnw, dlp)[:, : b.dim, : b.kv_rank] = uk
+                M["w_kv"][b.heads * dnw:].view(b.heads, dvp, dlp)[:, : b.vdim, : b.kv_rank] = uv
+            if own:
+                M["kv_norm"] = self._vec(w[a + "kv_a_norm"])
+            M["inv_freq"] = self._inv_freq(b.rot_base, b.rot_dim)
+            return parts, w[a + "o"].to(dev)
+        gate = b.out_gate or b.head_gate
+        parts = [w[a + n].to(dev) for n in ("q", "k", "v")] + ([w[a + "g"].to(dev)] if gate else [])
+        M["meta"] = _Meta(_offsets(parts) + ([] if gate else [-1]))
+        if b.qkv_bias:
+            M["q_bias"], M["k_bias"], M["v_bias"] = (self._vec(w[a + n + "_bias"]) for n in "qkv")
+        if b.qk_norm or b.head_norm == "weight":
+            M["q_norm"], M["k_norm"] = self._vec(w[a + "q_norm"]), self._vec(w[a + "k_norm"])
+        if b.half_rot:
+            M["inv_freq"] = self._inv_freq(b.rot_base, b.half_rot)
+        if b.bias_rows:
+            rel = w[a + "rel"].to(dev).float()                 # one value per distance and head: the kernels know no buckets
+            M["bias"] = rel[torch.tensor(distance_buckets(rel.shape[0], b.bias_max), device=dev)].T.contiguous()
+        if b.alibi:
+            M["slope"] = torch.tensor([2.0 ** (-8.0 * (h + 1) / b.heads) for h in range(b.heads)], dtype=torch.float32, device=dev)
+        if b.v_mix:
+            M["v_mix"] = self._vec(w[a + "v_mix"])
+        return parts, w[a + "o"].to(dev)
+
+    def _inv_freq(self, base: float, dims: int) -> torch.Tensor:
+        return torch.tensor([base ** (-2.0 * j / dims) for j in range(dims // 2)], dtype=torch.float64, device=self.device)
+
     @classmethod
     def from_state_dict(cls, cfg: ModelConfig, w, device="cuda", kv_fmt=None, page=64, expert_quant=None, dense_quant=None, tp_rank: int = 0,
                         tp_size: int = 1, expert_shard=None, with_mtp: bool = False, layer_hook=None, skip_experts=None, dtype: str = "bfloat16") -> "BlockModel":
@@ -284,11 +444,7 @@ class BlockModel(ModelBase):
 
         def stacked(parts, cols=Hp):
             """The parts as one projection and the row at which each starts."""
-            offs, o = [], 0
-            for t in parts:
-                offs.append(o)
-                o += _align(t.shape[0], 8)
-            return m._mat(*parts, cols=cols), offs
+            return m._mat(*parts, cols=cols), _offsets(parts)
 
         e = torch.zeros(cfg.vocab, Hp, dtype=torch.bfloat16, device=dev)
         e[:, :H] = w["embed.weight"].to(dev)
@@ -302,65 +458,44 @@ class BlockModel(ModelBase):
         for i, b in enumerate(cfg.blocks):
             p = f"layers.{i}."
             L: dict = {"mix_in": norm(p + "mix_norm"), "mix_out": norm(p + "mix_post_norm")} if sandwich else {"mix_in": NO_NORM, "mix_out": norm(p + "mix_norm")}
-            if b.recurrent:
-                k = p + "kda."
-                fb, gb = w[k + "f_b"].to(dev), w[k + "g_b"].to(dev)
-                ra, rg = _align(fb.shape[1], 8), _align(gb.shape[1], 8)
-                kw, vw = b.kv_heads * b.dim, b.heads * b.vdim
-                parts = [w[k + n].to(dev) for n in ("q", "k", "v", "beta", "f_a", "g_a")]
-                L["in"], offs = stacked(parts)
-                L["meta"] = _Meta(offs=offs, ra=ra, rg=rg)
-                pad = lambda t, n: torch.nn.functional.pad(t.float(), (0, n - t.shape[1])).to(m.act_dtype).contiguous()
-                L["w_a"], L["w_g"] = pad(fb, ra), pad(gb, rg)
-                if not m.f32:
-                    # [W | W]: many rows take the low-rank products on the tensor cores with (hi | lo) activations
-                    L["w_a2"], L["w_g2"] = torch.cat([L["w_a"]] * 2, 1).contiguous(), torch.cat([L["w_g"]] * 2, 1).contiguous()
-                for n in ("conv_q", "conv_k", "conv_v"):
-                    t = w[k + n].to(dev).float().contiguous()
-                    if tuple(t.shape) != ((vw if n == "conv_v" else kw), b.conv):
-                        raise ValueError(f"{k + n}: shape {tuple(t.shape)}")
-                    L[n] = t
-                L["a_exp"], L["dt_bias"], L["o_norm"] = torch.exp(m._vec(w[k + "a_log"])), m._vec(w[k + "dt_bias"]), m._vec(w[k + "o_norm"])
-                L["out"] = m._mat(w[k + "o"].to(dev), cols=_align(vw, 8))
-            elif b.latent:
-                a, own = p + "attn.", b.kv_from < 0
-                names = ["q"] + (["kv_a"] if own else []) + (["g"] if b.head_gate else [])
-                L["in"], offs = stacked([w[a + n].to(dev) for n in names])
-                at = dict(zip(names, offs))
-                L["meta"] = _Meta(offs=[at["q"], at.get("kv_a", -1), at.get("g", -1)])
-                dnp, dlp = _align(b.dim, 8), m.latent_pad(b.kv_rank)
-                uk, uv = w[a + "k_b"].to(dev).view(b.heads, b.dim, b.kv_rank), w[a + "v_b"].to(dev).view(b.heads, b.vdim, b.kv_rank)
-                L["w_uk"] = torch.zeros(b.heads, dlp, dnp, dtype=m.act_dtype, device=dev)
-                L["w_uk"][:, : b.kv_rank, : b.dim] = uk.transpose(1, 2)
-                L["w_uv"] = torch.zeros(b.heads, b.vdim, dlp, dtype=m.act_dtype, device=dev)
-                L["w_uv"][:, :, : b.kv_rank] = uv
-                if not m.f32:
-                    # the same two, one after the other per position: what long prompt runs make keys and values with
-                    dnw, dvp = _align(b.dim, 16), m.head_pad(b.vdim)
-                    L["w_kv"] = torch.zeros(b.heads * (dnw + dvp), dlp, dtype=m.act_dtype, device=dev)
-                    L["w_kv"][: b.heads * dnw].view(b.heads, dnw, dlp)[:, : b.dim, : b.kv_rank] = uk
-                    L["w_kv"][b.heads * dnw:].view(b.heads, dvp, dlp)[:, : b.vdim, : b.kv_rank] = uv
-                if own:
-                    L["kv_norm"] = m._vec(w[a + "kv_a_norm"])
-                L["inv_freq"] = torch.tensor([b.rot_base ** (-2.0 * j / b.rot_dim) for j in range(b.rot_dim // 2)], dtype=torch.float64, device=dev)
-                L["out"] = m._mat(w[a + "o"].to(dev), cols=_align(b.heads * b.vdim, 8))
+            if cfg.norm_place == "pre":
+                L["mix_in"], L["mix_out"] = L["mix_out"], NO_NORM
+            sides, cols = _sides(b), 0
+            L["sides"] = [{} for _ in sides]
+            parts, outs, base = [], [], 0
+            for (side, x), M in zip(sides, L["sides"]):
+                own, out = m._build_mixer(w, p + side, x, M)
+                if "shift" not in M:
+                    M["meta"].shift(base)
+                M["col"], M["cols"] = cols, _align(out.shape[1], 8)
+                cols += M["cols"]
+                base += sum(_align(t.shape[0], 8) for t in own)
+                parts += own
+                outs.append(out)
+            L["mix_ld"] = cols
+            L["in"] = stacked(parts)[0] if parts else None
+            for M in L["sides"]:
+                if "shift" in M:                              # projections over inputs of their own, behind the others
+                    M["meta"].shift(base)
+                    M["at"] = base
+                    base += M["shift"].N
+            m.max_proj = max(m.max_proj, base)
+            if b.branches and b.join == "normed":
+                for (side, _), M, t in zip(sides, L["sides"], outs):
+                    M["out"], M["out_norm"] = m._mat(t, cols=M["cols"]), m._vec(w[p + side + "out_norm"])
+                    M["out"].N = Hp
             else:
-                a = p + "attn."
-                parts = [w[a + n].to(dev) for n in ("q", "k", "v")] + ([w[a + "g"].to(dev)] if b.out_gate else [])
-                L["in"], offs = stacked(parts)
-                L["meta"] = _Meta(offs=offs + ([] if b.out_gate else [-1]))
-                if b.qk_norm:
-                    L["q_norm"], L["k_norm"] = m._vec(w[a + "q_norm"]), m._vec(w[a + "k_norm"])
-                if b.alibi:
-                    L["slope"] = torch.tensor([2.0 ** (-8.0 * (h + 1) / b.heads) for h in range(b.heads)], dtype=torch.float32, device=dev)
-                if b.v_mix:
-                    L["v_mix"] = m._vec(w[a + "v_mix"])
-                L["out"] = m._mat(w[a + "o"].to(dev), cols=_align(b.heads * b.vdim, 8))
-            L["out"].N = Hp
-            m.max_proj = max(m.max_proj, L["in"].N)
-            m.max_mix = max(m.max_mix, L["out"].K)
+                pad = torch.nn.functional.pad
+                L["out"] = m._mat(torch.cat([pad(t, (0, M["cols"] - t.shape[1])) for t, M in zip(outs, L["sides"])], 1))
+                L["out"].N = Hp
+            m.max_mix = max(m.max_mix, cols)
+            if cfg.streams:
+                for q in ["mix_hc"] + (["ffn_hc"] if b.has_ff else []):
+                    L[q] = tuple(m._vec(w[f"{p}{q}.{k}"]) for k in ("in", "out", "mix"))
             if b.has_ff:
                 L["ff_in"], L["ff_out"] = (norm(p + "ffn_norm"), norm(p + "ffn_post_norm")) if sandwich else (NO_NORM, norm(p + "ffn_norm"))
+                if cfg.norm_place == "pre":
+                    L["ff_in"], L["ff_out"] = L["ff_out"], NO_NORM
             if b.dense_ff:
                 L["ff"], L["ff_offs"] = stacked([w[p + f"mlp.{n}"].to(dev) for n in ("gate", "up")])
                 L["ff_down"] = m._mat(w[p + "mlp.down"].to(dev))
@@ -379,11 +514,17 @@ class BlockModel(ModelBase):
                 m.max_proj = max(m.max_proj, L["router"].N)
                 # expert width padded to the tensor-core tile where the residual width allows that path
                 F = _align(b.ff, 128) if Hp % 128 == 0 else _align(b.ff, 8)
-                arena = ExpertArena(expert_layout(m.w_fmt, Hp, F), b.experts, b.experts, dev)
+                gated = b.unit == "glu"
+                arena = ExpertArena(expert_layout(m.w_fmt, Hp, F, gated=gated), b.experts, b.experts, dev)
                 for x in range(b.experts):
-                    g, u, d = (torch.zeros(n, k, dtype=m.act_dtype, device=dev) for n, k in ((F, Hp), (F, Hp), (Hp, F)))
-                    g[: b.ff, :H], u[: b.ff, :H], d[:H, : b.ff] = (w[mo + f"experts.{x}.{n}"].to(dev) for n in ("gate", "up", "down"))
-                    arena.write_expert(x, QLinear(m.w_fmt, F, Hp, g), QLinear(m.w_fmt, F, Hp, u), QLinear(m.w_fmt, Hp, F, d))
+                    u, d = (torch.zeros(n, k, dtype=m.act_dtype, device=dev) for n, k in ((F, Hp), (Hp, F)))
+                    u[: b.ff, :H], d[:H, : b.ff] = (w[mo + f"experts.{x}.{n}"].to(dev) for n in ("up", "down"))
+                    g = None
+                    if gated:
+                        g = torch.zeros_like(u)
+                        g[: b.ff, :H] = w[mo + f"experts.{x}.gate"].to(dev)
+                        g = QLinear(m.w_fmt, F, Hp, g)
+                    arena.write_expert(x, g, QLinear(m.w_fmt, F, Hp, u), QLinear(m.w_fmt, Hp, F, d))
                     arena.slot_of[x] = x
                 L["arena"] = arena
             if cfg.side_dim:
@@ -413,10 +554,13 @@ class BlockModel(ModelBase):
         z = lambda *s, dtype=torch.float32: torch.zeros(*s, dtype=dtype, device=self.device)
         self.block_table = z(n_slots, max_pages_per_seq, dtype=torch.int32)
         self.idx_block_table = self.block_table
-        for i, b in enumerate(self.cfg.blocks):
-            if b.recurrent:
+        for i, b in [(i, m) for i, L in enumerate(self.cfg.blocks) for m in L.mixers]:
+            if b.delta:
                 self.kda_state[i] = z(n_slots, b.heads, b.vdim, int(nat.call("lsb_delta_key_pad", b.dim)))
                 self.kda_conv[i] = z(n_slots, b.heads, 2 * b.dim + b.vdim, b.conv - 1)
+            elif b.kind == "time_mix":
+                self.kda_state[i] = z(n_slots, b.heads, b.vdim, int(nat.call("lsb_tmix_key_pad", b.dim)))
+                self.kda_conv[i] = z(n_slots, self.Hp)                   # the previous token's input
             elif b.latent:
                 if b.kv_from < 0:
                     self.kv_cache[i] = z(num_pages, self.page, self.latent_row(b), dtype=self.act_dtype)
@@ -425,27 +569,42 @@ class BlockModel(ModelBase):
 
     def cache_bytes_per_token(self) -> int:
         width = lambda b: ((self.latent_row(b) if b.kv_from < 0 else 0) if b.latent else b.kv_heads * (self.head_pad(b.dim) + self.head_pad(b.vdim)))
-        return sum(width(b) * (4 if self.f32 else 2) for b in self.cfg.blocks if not b.recurrent)
+        return sum(width(b) * (4 if self.f32 else 2) for L in self.cfg.blocks for b in L.mixers if not b.recurrent)
 
     # ------------------------------------------------------------------ forward
     def _resid_rows(self, ws, R: int, H: int) -> torch.Tensor:
-        return ws.resid[:R, :H]
+        return ws.streams[:R, :, :H].sum(1) if self.cfg.streams else ws.resid[:R, :H]
 
-    def _attention(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
+    def _mixer(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
+        """The layer's mixers, input projections to output projection: ``ws.sub`` (and ``ws.sub2`` of a second result that is normed on its own)."""
+        if L["in"] is not None:
+            L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
+        for x, M in zip(b.mixers, L["sides"]):
+            f = self._delta if x.delta else (self._time_mix if x.kind == "time_mix" else (self._latent if x.latent else self._attention))
+            f(i, x, M, ws, R, nseq, ws.mix.view(-1)[M["col"]:], L["mix_ld"])
+        if b.branches and b.join == "normed":
+            for M, sub in zip(L["sides"], (ws.sub, ws.sub2)):
+                M["out"](sub, ws.mix.view(-1)[M["col"]:], R, ldx=L["mix_ld"], ldo=self.Hp)
+        else:
+            L["out"](ws.sub, ws.mix, R, ldo=self.Hp)
+
+    def _attention(self, i: int, b: BlockSpec, M: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
         dkp, dvp, ldp = self.head_pad(b.dim), self.head_pad(b.vdim), self.max_proj
-        oq, ok, ov, og = L["meta"].offs
-        L["in"](ws.proj, ws.x, R, ldo=ldp)
-        mix = 0 if not b.v_mix else (1 if i == self.v_first_layer else 2)
-        nat.call("lsb_attn_prep", ws.proj, ldp, oq, ok, ov, L.get("q_norm"), L.get("k_norm"), self.cfg.rms_eps, ws.v_first if mix else None, mix,
-                 L.get("v_mix"), ws.q, self.kv_cache[i], self.block_table, self.max_pages, ws.row_seq, ws.row_pos, R, b.heads, b.kv_heads, b.dim, b.vdim,
-                 dkp, dvp, self.page, int(self.f32))
+        oq, ok, ov, og = M["meta"].offs
+        at = (ws.q, self.kv_cache[i], self.block_table, self.max_pages, ws.row_seq, ws.row_pos, R, b.heads, b.kv_heads, b.dim, b.vdim, dkp, dvp, self.page, int(self.f32))
+        if b.qkv_bias or b.head_norm or b.half_rot:
+            nat.call("lsb_attn_head_prep", ws.proj, ldp, oq, ok, ov, M.get("q_bias"), M.get("k_bias"), M.get("v_bias"), HEAD_NORM[b.head_norm], M.get("q_norm"),
+                     M.get("k_norm"), self.cfg.rms_eps, b.half_rot, M.get("inv_freq"), *at)
+        else:
+            mix = 0 if not b.v_mix else (1 if i == self.v_first_layer else 2)
+            nat.call("lsb_attn_prep", ws.proj, ldp, oq, ok, ov, M.get("q_norm"), M.get("k_norm"), self.cfg.rms_eps, ws.v_first if mix else None, mix, M.get("v_mix"), *at)
+        bias = M.get("bias")
         nat.call("lsb_attn", ws.q, self.kv_cache[i], self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
-                 max(ws.seq_rows), ws.proj, ldp, og, ws.mix, L["out"].K, ws.o_part, ws.ml_part, ws.splits[i], R, b.heads, b.kv_heads, b.dim, b.vdim, dkp, dvp,
-                 b.window, b.scale, L.get("slope"), int(self.f32))
+                 max(ws.seq_rows), ws.proj, ldp, og, out, ldo, ws.o_part, ws.ml_part, ws.splits[i], R, b.heads, b.kv_heads, b.dim, b.vdim, dkp, dvp,
+                 b.window, b.scale, M.get("slope"), int(b.head_gate), b.chunk, bias, bias.shape[1] if bias is not None else 0, b.out_scale, int(self.f32))
 
-    def _latent(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
+    def _latent(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
         cache = self.kv_cache[i if b.kv_from < 0 else b.kv_from]
-        L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
         # long runs one by one, what lies between them together
         rows, row0, j = ws.seq_rows, 0, 0
         while j < nseq:
@@ -461,7 +620,7 @@ class BlockModel(ModelBase):
     def _latent_rows(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, r0: int, R: int, j: int, k: int):
         """Step rows [r0, r0 + R) (sequences j .. k - 1 of the step) in the latent space."""
         oq, okv, og = L["meta"].offs
-        H, ld, K, f32, err = b.heads, self.max_proj, L["out"].K, int(self.f32), TcScratch.get(self.device).err
+        H, ld, K, f32, err = b.heads, self.max_proj, L["cols"], int(self.f32), TcScratch.get(self.device).err
         q, o_lat, proj, seq, pos = ws.q_lat[r0 * H * self.latent_row(b):], ws.o_lat[r0 * H * L["w_uv"].shape[2]:], ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
         nat.call("lsb_latent_query", proj, ld, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], q, ws.q_nope, cache, self.block_table,
                  self.max_pages, self.page, seq, pos, R, H, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank, f32, err)
@@ -476,7 +635,7 @@ class BlockModel(ModelBase):
     def _latent_run(self, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, r0: int, R: int, j: int):
         """Step rows [r0, r0 + R), a run of sequence j, over keys and values of every head, made for this step from the cached rows."""
         oq, okv, og = L["meta"].offs
-        H, ld, K, err, T = b.heads, self.max_proj, L["out"].K, TcScratch.get(self.device).err, ws.seq_end[j]
+        H, ld, K, err, T = b.heads, self.max_proj, L["cols"], TcScratch.get(self.device).err, ws.seq_end[j]
         dnw, dvp, drp = _align(b.dim, 16), self.head_pad(b.vdim), self.latent_pad(b.rot_dim)
         Tm, proj, seq, pos = _align(T, 256), ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
         q, lat, kv = self._expand_scratch(ws.R, R * H * (dnw + drp), Tm * self.latent_pad(b.kv_rank), Tm * (H * (dnw + dvp) + drp))
@@ -509,9 +668,8 @@ class BlockModel(ModelBase):
             at.append(at[-1] + _align(n, 64))
         return [self._expand[a: a + n] for a, n in zip(at, sizes)]
 
-    def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
+    def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
         mt = L["meta"]
-        L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
         rows = ws.seq_rows
         few = max(rows) <= FEW_ROWS and b.vdim <= nat.call("lsb_delta_few_max_dv", b.dim)
         scratch = chunk_ws = None
@@ -521,11 +679,32 @@ class BlockModel(ModelBase):
             chunks = sum((n + 63) // 64 for n in long_)
             scratch, chunk_ws = ws.delta_scratch(b, R, mt.ra, mt.rg, chunks)
         oq, ok, ov, ob, oa, og = mt.offs
-        nat.call("lsb_delta_forward", ws.proj, self.max_proj, oq, ok, ov, ob, oa, og, mt.ra, mt.rg, L["w_a"], L["w_g"], L.get("w_a2"), L.get("w_g2"),
+        nat.call("lsb_delta_forward", ws.proj, self.max_proj, oq, ok, ov, ob, oa, og, mt.ra, mt.rg, L.get("w_a"), L.get("w_g"), L.get("w_a2"), L.get("w_g2"),
                  L["conv_q"], L["conv_k"], L["conv_v"], L["a_exp"], L["dt_bias"], L["o_norm"], self.kda_state[i], self.kda_conv[i], ws.seq_row0,
-                 ws.seq_nrows, ws.seq_slot, ws.mix, L["out"].K, nseq, R, b.heads, b.kv_heads, b.dim, b.vdim, b.conv, 0 if b.decay == "softplus" else 1,
+                 ws.seq_nrows, ws.seq_slot, out, ldo, nseq, R, b.heads, b.kv_heads, b.dim, b.vdim, b.conv, 0 if b.decay == "softplus" else 1,
                  b.dim ** -0.5, b.decay_bound, self.cfg.rms_eps, int(self.f32), int(few), scratch, len(rows) - len(long_), len(long_), chunks, LONG_ROWS,
                  chunk_ws, TcScratch.get(self.device).err)
+
+    def _time_mix(self, i: int, b: BlockSpec, M: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
+        W, Hp, ldp, f32, err = M["shift"], self.Hp, self.max_proj, int(self.f32), TcScratch.get(self.device).err
+        seqs = (ws.seq_row0, ws.seq_nrows, ws.seq_slot)
+        nat.call("lsb_tmix_shift", ws.x, Hp, self.kda_conv[i], M["mu"], ws.xs, ws.xs.stride(0), *seqs, nseq, R, f32)
+        r, segs = M["seg_rows"].tolist(), M["segs"]
+        proj = ws.proj.view(-1)[M["at"]:]
+        if not f32 and R < 8 and Hp <= 16384:
+            nat.call("lsb_gemv_bf16_segs", proj, ws.xs, W.w, R, W.N, Hp, Hp, Hp, ldp, M["seg_rows"], 5, ws.xs.stride(0))
+        elif not f32 and R >= 8 and len(set(segs[:4])) == 1:
+            nat.call("lsb_gemm_bf16_tc_batched", proj, ws.xs, W.w, R, r[1], Hp, 4, Hp, ws.xs.stride(0), Hp, r[1] * Hp, ldp, r[1], 0, err)
+            QLinear(W.fmt, W.N - r[4], Hp, W.w[r[4]:])(proj[r[4]:], ws.xs[4], R, ldo=ldp)
+        else:
+            for j, end in enumerate(r[1:] + [W.N]):
+                QLinear(W.fmt, end - r[j], Hp, W.w[r[j]:])(proj[r[j]:], ws.xs[j], R, ldo=ldp)
+        few = max(ws.seq_rows) <= FEW_ROWS or b.dim > 128
+        rank = M["w2"].shape[1]
+        chunks = 0 if few else sum((n + 63) // 64 for n in ws.seq_rows)
+        scratch = None if few else ws.tmix_scratch(b, R, chunks, rank)
+        nat.call("lsb_tmix_forward", ws.proj, ldp, *M["meta"].offs, rank, M["w2"], M["w22"], M["w0"], M["u"], M["o_norm"], self.kda_state[i], self.kda_conv[i], ws.x, Hp,
+                 *seqs, out, ldo, nseq, R, b.heads, b.dim, b.vdim, self.cfg.rms_eps, f32, int(few), scratch, chunks, err)
 
     def _glu(self, L: dict, ws: BlockWorkspace, R: int, ff: int, offs, limit=0.0, alpha=1.0, shift=0.0):
         """Gated unit over columns of the projection in ``ws.proj`` and its down product into ``ws.sub``; ``offs``: gate, up, output gate (-1: none)."""
@@ -543,7 +722,7 @@ class BlockModel(ModelBase):
             self._glu(L, ws, R, b.shared_ff, L["ff_offs"][1:], b.shared_limit, b.act_alpha, b.act_shift)
         self.moe_prepare(L["arena"], mb, ws.x, R, b.experts)
         plain = b.act_alpha == 1.0 and b.act_shift == 0.0 and not b.scale_input
-        act = None if plain else (b.act_alpha, b.act_shift, mb.wts if b.scale_input else None)
+        act = "relu2" if b.unit == "relu2" else None if plain else (b.act_alpha, b.act_shift, mb.wts if b.scale_input else None)
         self.moe_experts(L["arena"], mb, ws.x, R, b.experts, b.limit, mb.miss, act)
         return mb
 
@@ -572,6 +751,11 @@ class BlockModel(ModelBase):
         """One step over the first ``R`` staged rows; logits of rows [logit_row0, logit_row0 + n_logit_rows)."""
         cfg, H, Hp, f32 = self.cfg, self.cfg.hidden, self.Hp, int(self.f32)
         run = [i for i in range(cfg.n_layers) if i not in self.skip_layers]
+        if cfg.streams:
+            self._forward_streams(ws, R, nseq, run)
+            if n_logit_rows:
+                self.emit_logits(ws, logit_row0, n_logit_rows)
+            return
         enters = dict(zip([-1] + run, [self.layers[i]["mix_in"] for i in run] + [NO_NORM]))       # norm in front of the layer that follows
         plain = enters[-1] is NO_NORM
         nat.call("lsb_embedding_scaled", ws.resid, ws.x if plain and not f32 else None, self.embed, ws.tok, R, Hp, 0, cfg.vocab, cfg.embed_scale)
@@ -583,8 +767,7 @@ class BlockModel(ModelBase):
             if i not in enters:
                 continue
             b, L = cfg.blocks[i], self.layers[i]
-            (self._delta if b.recurrent else (self._latent if b.latent else self._attention))(i, b, L, ws, R, nseq)
-            L["out"](ws.sub, ws.mix, R, ldo=Hp)
+            self._mixer(i, b, L, ws, R, nseq)
             last = NO_NORM if cfg.side_dim else enters[i]
             self._update(ws, R, L["mix_out"], L["ff_in"] if b.has_ff else last, ws.sub)
             if b.experts:
@@ -604,6 +787,42 @@ class BlockModel(ModelBase):
         if n_logit_rows:
             self.emit_logits(ws, logit_row0, n_logit_rows)
 
+    def _forward_streams(self, ws: BlockWorkspace, R: int, nseq: int, run: List[int]):
+        """The layers of a model with hyper-connections; leaves the sum of the streams in ``ws.resid``."""
+        cfg = self.cfg
+        subs = [(i, q) for i in run for q in ("mix", "ffn") if q == "mix" or cfg.blocks[i].has_ff]
+        enters = [(self.layers[i][q + "_hc"][0], self.layers[i]["mix_in" if q == "mix" else "ff_in"]) for i, q in subs] + [(None, NO_NORM)]
+        nat.call("lsb_embedding_scaled", ws.resid, None, self.embed, ws.tok, R, self.Hp, 0, cfg.vocab, cfg.embed_scale)
+        self._update_streams(ws, R, enters[0], first=ws.resid)
+        for (i, q), nxt in zip(subs, enters[1:]):
+            b, L = cfg.blocks[i], self.layers[i]
+            if q == "mix" and self.aux_capture is not None:
+                self._capture_aux(i, ws, R)
+            mb = None
+            if q == "mix":
+                self._mixer(i, b, L, ws, R, nseq)
+            elif b.experts:
+                mb = self._moe(i, b, L, ws, R)
+            else:
+                L["ff"](ws.proj, ws.x, R, ldo=self.max_proj)
+                self._glu(L, ws, R, b.dense_ff, (*L["ff_offs"], -1))
+            self._update_streams(ws, R, nxt, L[q + "_hc"], None if mb is not None and not b.shared_ff else ws.sub, mb, b, L, q == "mix" and b.join == "normed" and b.branches)
+            if self.drift is not None and (q == "ffn" or not b.has_ff):
+                self.drift[f"layer{i:03d}.resid"] = self._resid_rows(ws, R, cfg.hidden).float().cpu()
+        if self.aux_capture is not None:
+            self._capture_aux(cfg.n_layers, ws, R)
+
+    def _update_streams(self, ws: BlockWorkspace, R: int, nxt: tuple, hc: tuple = (None, None, None), sub=None, mb: Optional[MoeBuffers] = None, b=None, L=None,
+                        normed=False, first=None):
+        """Streams behind a sublayer with the weights ``hc``, and the input of the next one ``nxt`` = (its reading weights, its norm); behind the last
+        (reading weights None) the sum of the streams instead."""
+        Hp, y, last = self.Hp, (None, None, None, None, 0, 0, 0), nxt[0] is None
+        if mb is not None:
+            y = (mb.y, None if b.scale_input else mb.wts, mb.ids, L["arena"].slot_of, b.top, b.experts, L["arena"].ef.H)
+        sides = ([ws.sub2, Hp] + [M["out_norm"] for M in L["sides"]]) if normed else [None, Hp, None, None]
+        nat.call("lsb_stream_update", None if last else ws.x, Hp, ws.streams, Hp, self.cfg.streams, first, ws.resid if last else None, sub, *sides, hc[2], hc[1],
+                 self.cfg.residual_mult, nxt[0], *nxt[1], R, self.cfg.hidden, self.cfg.rms_eps, *y, int(self.f32))
+
     def emit_logits(self, ws: BlockWorkspace, row0: int, n: int, rows: Optional[torch.Tensor] = None):
         """Logits of step rows [row0, row0 + n), or of the ``n`` rows listed in ``rows`` (int32, device), after :meth:`forward`."""
         kind, nw, nb, alpha = self.final_norm
@@ -612,10 +831,22 @@ class BlockModel(ModelBase):
 
 
 class _Meta:
-    """Column offsets of a layer's fused input projection and the padded ranks of its low-rank gates."""
+    """Columns of a mixer's projections in the projection buffer (-1: it has none) and the padded ranks of its low-rank gates."""
 
     def __init__(self, offs: List[int], ra: int = 0, rg: int = 0):
         self.offs, self.ra, self.rg = offs, ra, rg
+
+    def shift(self, n: int):
+        self.offs = [o + n if o >= 0 else o for o in self.offs]
+
+
+def _offsets(parts) -> List[int]:
+    """Rows at which stacked projections start, each padded to a multiple of 8."""
+    offs, o = [], 0
+    for t in parts:
+        offs.append(o)
+        o += _align(t.shape[0], 8)
+    return offs
 
 
 def model_class(cfg: ModelConfig):

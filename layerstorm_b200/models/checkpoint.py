@@ -83,8 +83,20 @@ _RUBASUN_LAYER = {f"{c}.{k}": f + s for c, f in (("mix_norm", "norm1"), ("mix_po
     "side.gate": "side.gate", "side.proj": "side.proj", "side.norm": "side.norm",
 }
 _RUBASUN_TOP = _GAZUTAR_TOP | {"final_norm.alpha": "final.norm.alpha", "side_embed.weight": "side.embed"}
+# canonical suffix -> tensor name behind "l<N>." (Fasodra): the mixers' names stand alone or behind "left." / "right."
+_FASODRA_MIXERS = {
+    "attn.q": "q", "attn.k": "k", "attn.v": "v", "attn.g": "g", "attn.o": "o", "attn.q_bias": "q.b", "attn.k_bias": "k.b", "attn.v_bias": "v.b",
+    "attn.q_norm": "q.norm", "attn.k_norm": "k.norm", "attn.rel": "rel",
+    "kda.q": "q", "kda.k": "k", "kda.v": "v", "kda.beta": "b", "kda.a": "a", "kda.g": "g", "kda.conv_q": "q.conv", "kda.conv_k": "k.conv",
+    "kda.conv_v": "v.conv", "kda.a_log": "A_log", "kda.dt_bias": "dt_bias", "kda.o_norm": "norm", "kda.o": "o",
+    "tmix.w1": "w1", "tmix.w2": "w2", "tmix.w0": "w0", "tmix.u": "u", "tmix.o_norm": "norm", "tmix.o": "o",
+} | {f"tmix.{n}": n for n in "rkvg"} | {f"tmix.mu_{n}": f"mu.{n}" for n in "rkvgw"}
+_FASODRA_LAYER = {f"{side}{c}": f"mix.{side}{f}" for side in ("", "left.", "right.") for c, f in _FASODRA_MIXERS.items()} | {
+    "left.out_norm": "mix.left.out", "right.out_norm": "mix.right.out", "moe.router": "mlp.router",
+} | {f"{c}_norm.{k}": f + s for c, f in (("mix", "norm1"), ("ffn", "norm2")) for k, s in (("weight", ""), ("bias", ".b"))} | {
+    f"{c}_hc.{k}": f"{f}.{k}" for c, f in (("mix", "hc1"), ("ffn", "hc2")) for k in ("in", "out", "mix")}
 # checkpoints with tensor names of their own: architecture -> (layer names, names outside the layers)
-_NATIVE_NAMES = {"gazutar": (_GAZUTAR_LAYER, _GAZUTAR_TOP), "rubasun": (_RUBASUN_LAYER, _RUBASUN_TOP)}
+_NATIVE_NAMES = {"gazutar": (_GAZUTAR_LAYER, _GAZUTAR_TOP), "rubasun": (_RUBASUN_LAYER, _RUBASUN_TOP), "fasodra": (_FASODRA_LAYER, _GAZUTAR_TOP)}
 _LAYER_RE = re.compile(r"^layers\.(\d+)\.(.+)$")
 _EXPERT_RE = re.compile(r"^moe\.(experts|shared)\.(\d+)\.(gate|up|down)$")
 

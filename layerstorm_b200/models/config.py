@@ -16,14 +16,19 @@ import math
 from dataclasses import dataclass, field, asdict
 from typing import List, Optional
 
-ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun")
+ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun", "fasodra")
+
+RECURRENT_KINDS = ("channel_delta", "head_delta", "time_mix")
 
 
 @dataclass
 class BlockSpec:
     """One layer of a model that is described layer by layer (``ModelConfig.blocks``): a mixer and an optional feed-forward, dense or a
     mixture of experts, each with sizes of its own."""
-    kind: str = "attention"           # "attention" | "latent_attention" | "channel_delta" (gated delta rule with a decay per key channel)
+    # "attention" | "latent_attention" | "channel_delta" (gated delta rule, a decay per key channel and low-rank gates) | "head_delta" (gated delta
+    # rule, a decay per head and a full-rank silu gate) | "time_mix" (token shift, data-dependent decay per key channel, bonus for the current
+    # token) | "parallel" (two of the others side by side, see `branches`)
+    kind: str = "attention"
     heads: int = 0                    # query heads (attention) / value heads (delta)
     kv_heads: int = 0                 # key-value heads (attention) / query-key heads (delta); divides `heads`
     dim: int = 0                      # query / key head width
@@ -35,6 +40,12 @@ class BlockSpec:
     alibi: bool = False               # linear distance bias, slope 2^(-8 (h + 1) / heads)
     out_gate: bool = False            # heads times sigmoid(W_g h) in front of the output projection
     v_mix: bool = False               # values mixed with those of the first such layer
+    chunk: int = 0                    # chunked mask: a position sees the keys of its own chunk (0 = the whole prefix)
+    qkv_bias: bool = False            # biases on the q, k and v projections
+    head_norm: str = ""               # RMS norm of every q and k head: "" none | "plain" (no weight) | "weight" (one weight for all heads)
+    half_rot: int = 0                 # leading channels of q and k heads that are rotated (channel i with i + half_rot / 2), base rot_base
+    bias_rows: int = 0                # rows of a learned distance bias table (0: none): one per distance, then logarithmic up to bias_max
+    bias_max: int = 0
     # latent attention (one cached row of kv_rank + rot_dim per token for all heads)
     kv_rank: int = 0
     rot_dim: int = 0                  # rotated query / key channels per head, behind `dim` unrotated ones
@@ -45,6 +56,11 @@ class BlockSpec:
     conv: int = 0                     # taps of the short causal convolutions
     decay: str = "softplus"           # log decay: "softplus" -exp(A) softplus(x) | "bounded" decay_bound * sigmoid(exp(A) x)
     decay_bound: float = -5.0
+    # two mixers side by side over the same input: "scaled" a * left + b * right (each branch's out_scale), "normed" the mean of both
+    # results, each RMS-normed with a weight
+    branches: List["BlockSpec"] = field(default_factory=list)
+    join: str = "scaled"
+    out_scale: float = 1.0
     # feed-forward (dense_ff 0 and experts 0: none)
     dense_ff: int = 0                 # width of a dense gated unit
     experts: int = 0
@@ -56,6 +72,7 @@ class BlockSpec:
     # router: scores, selection correction; where a chosen expert's weight goes
     scoring: str = "softmax"          # softmax | sigmoid
     correction: bool = True
+    unit: str = "glu"                 # the experts' hidden unit: "glu" (gate and up) | "relu2" (square of relu of up, no gate)
     scale_input: bool = False         # the weight multiplies the expert's input instead of its output
     # the experts' gated unit min(g, limit) sigmoid(act_alpha g) (clamp(u, -limit, limit) + act_shift); limit 0: no clamps
     limit: float = 0.0
@@ -64,9 +81,26 @@ class BlockSpec:
     shared_ff: int = 0                # an expert for every token (same unit, own limit) times sigmoid of one number per token
     shared_limit: float = 0.0
 
+    def __post_init__(self):
+        self.branches = [b if isinstance(b, BlockSpec) else BlockSpec(**b) for b in self.branches]
+
+    @property
+    def mixers(self) -> List["BlockSpec"]:
+        """The layer's mixers: itself, or the two that run side by side."""
+        return self.branches or [self]
+
     @property
     def recurrent(self) -> bool:
-        return self.kind == "channel_delta"
+        """The mixer keeps a state per sequence instead of a cache."""
+        return self.kind in RECURRENT_KINDS
+
+    @property
+    def delta(self) -> bool:
+        return self.kind in ("channel_delta", "head_delta")
+
+    @property
+    def softmax(self) -> bool:
+        return self.kind == "attention"
 
     @property
     def latent(self) -> bool:
@@ -142,7 +176,9 @@ class ModelConfig:
     # models described layer by layer (models/block_model.py); empty for the MLA family
     blocks: List[BlockSpec] = field(default_factory=list)
     norm_kind: str = "rms"            # "rms" | "layer" (with bias) | "tanh" (dynamic tanh, element-wise): the norms of the residual stream
-    norm_place: str = "post"          # "post": on every sublayer's output | "sandwich": in front of every sublayer and on its output
+    norm_place: str = "post"          # "post": on every sublayer's output | "sandwich": in front of every sublayer and on its output | "pre": in front
+    streams: int = 0                  # hyper-connections: copies of the residual stream with learned static mixing (0: one plain stream)
+    residual_mult: float = 1.0        # factor on every sublayer's output (with `streams`)
     logit_scale: float = 1.0
     embed_scale: float = 1.0
     side_dim: int = 0                 # width of a layer's slice of the per-token side table (0: no such table)
@@ -157,6 +193,10 @@ class ModelConfig:
         assert len(self.layer_types) == self.n_layers
         assert self.architecture in ARCHITECTURES
         for i, b in enumerate(self.blocks):
+            if b.branches:
+                m = b.mixers
+                if b.kind != "parallel" or len(m) != 2 or any(x.branches or x.latent or x.v_mix for x in m) or sum(x.recurrent for x in m) > 1 or sum(x.softmax for x in m) > 1:
+                    raise ValueError(f"layer {i}: side by side go two mixers, at most one with a cache and one with a state")
             if b.kv_from >= 0:
                 src = self.blocks[b.kv_from] if b.kv_from < i else None
                 if src is None or not src.latent or src.kv_from >= 0 or (src.kv_rank, src.rot_dim, src.rot_base) != (b.kv_rank, b.rot_dim, b.rot_base):
@@ -185,8 +225,10 @@ class ModelConfig:
         return self.is_moe_layer(i) and i < self.num_hash_layers
 
     def is_kda_layer(self, i: int) -> bool:
-        """The layer keeps a recurrent state per sequence (KDA, or a delta-rule block) instead of a KV cache."""
-        return i < len(self.layer_types) and self.layer_types[i] in ("kda", "channel_delta")       # multi-token-prediction blocks (i >= n_layers) are MLA layers
+        """The layer keeps a recurrent state per sequence: KDA, a recurrent block, or a block with one beside attention."""
+        if i < len(self.blocks):
+            return any(b.recurrent for b in self.blocks[i].mixers)
+        return i < len(self.layer_types) and self.layer_types[i] == "kda"       # multi-token-prediction blocks (i >= n_layers) are MLA layers
 
     def mla_layers(self) -> List[int]:
         return [i for i in range(self.n_layers) if not self.is_kda_layer(i)]
@@ -353,7 +395,31 @@ def rubasun_flash() -> ModelConfig:
                     12288, 64, 8, 2048, 2048, (7.0, 7.0), 8, side=256)
 
 
+def _fasodra(name, width, vocab, heads, kv, dim, chunk, left, time, delta, experts, top, ff, n_layers, streams=2) -> ModelConfig:
+    """A Fasodra shape: chunked attention, attention beside time mixing, chunked attention, attention beside a delta rule, in turns."""
+    att = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "bias_max": chunk, "mask": {"size": chunk}}
+    lft = {"heads": left[0], "kv_heads": left[1], "dim": left[2], "vdim": left[2], "scale": left[2] ** -0.5, "rot": {"base": 1e5, "dims": left[2] // 2}}
+    par = {"left": lft, "right": {"heads": time[0], "dim": time[1]}, "left_scale": 0.7, "right_scale": 0.9}
+    par2 = {"left": lft, "right": {"heads": delta[0], "kv_heads": delta[1], "dim": delta[2], "vdim": delta[2], "conv": 4}}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    kinds = [("attention", att), ("parallel", par), ("attention", att), ("parallel_2", par2)]
+    return fasodra_config({"name": name, "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.8, "streams": streams,
+                           "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(n_layers)]})
+
+
+def tiny_fasodra() -> ModelConfig:
+    """A small Fasodra shape for tests and smoke runs."""
+    return _fasodra("tiny-fasodra", 192, 320, 6, 2, 32, 40, (4, 2, 48), (5, 24), (4, 2, 40), 6, 2, 80, 4, 3)
+
+
+def fasodra_flash() -> ModelConfig:
+    """A Fasodra shape with layers of a real model's size."""
+    return _fasodra("fasodra-flash", 4096, 154880, 32, 8, 128, 4096, (32, 8, 128), (64, 64), (32, 32, 128), 64, 8, 3072, 8)
+
+
 PRESETS = {
+    "tiny-fasodra": tiny_fasodra,
+    "fasodra-flash": fasodra_flash,
     "tiny-rubasun": tiny_rubasun,
     "rubasun-flash": rubasun_flash,
     "tiny-gazutar": tiny_gazutar,
@@ -440,8 +506,54 @@ def rubasun_config(c: dict) -> ModelConfig:
         n_shared=0, moe_inter=top("ff", moe), scoring="sigmoid", norm_topk_prob=False, max_position=int(c.get("max_position", 1 << 20)))
 
 
+def fasodra_config(c: dict) -> ModelConfig:
+    """Fasodra: layer norms in front of every sublayer, hyper-connections with static mixing; chunked attention with a learned distance bias, rotary
+    attention beside time mixing (a constant factor on each) or beside a delta rule (each result normed), and ungated squared-relu experts."""
+    def attention(m, **kw):
+        rot = m.get("rot") or {}
+        if int(rot.get("dims", 0)) % 2 or int(rot.get("dims", 0)) > m["dim"]:
+            raise ValueError(f"{rot['dims']} rotary channels in heads of {m['dim']}")
+        return BlockSpec(kind="attention", heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]), qkv_bias=True,
+                         half_rot=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)), **kw)
+
+    blocks = []
+    for i, L in enumerate(c["layers"]):
+        m = L["mixer"]
+        if L["type"] == "attention":
+            b = attention(m, head_norm="plain", chunk=int((m.get("mask") or {}).get("size", 0)), bias_rows=32, bias_max=int(m["bias_max"]))
+        elif L["type"] == "parallel":
+            r = m["right"]
+            b = BlockSpec(kind="parallel", join="scaled", branches=[
+                attention(m["left"], head_gate=True, out_scale=float(m["left_scale"])),
+                BlockSpec(kind="time_mix", heads=r["heads"], kv_heads=r["heads"], dim=r["dim"], vdim=r["dim"], out_scale=float(m["right_scale"]))])
+        elif L["type"] == "parallel_2":
+            r = m["right"]
+            b = BlockSpec(kind="parallel", join="normed", branches=[
+                attention(m["left"], head_norm="weight"),
+                BlockSpec(kind="head_delta", heads=r["heads"], kv_heads=r["kv_heads"], dim=r["dim"], vdim=r["vdim"], conv=int(r["conv"]))])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
+        mlp = L.get("mlp")
+        if mlp:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            b.experts, b.top, b.ff = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"])
+            b.correction, b.unit = False, "relu2"
+        blocks.append(b)
+    moe = [b for b in blocks if b.experts]
+    att = [x for b in blocks for x in b.mixers if not x.recurrent]
+    rec = [x for b in blocks for x in b.mixers if x.recurrent]
+    top = lambda key, of, least=0: max((getattr(b, key) for b in of), default=least)
+    return ModelConfig(
+        name=c.get("name", "Fasodra"), architecture="fasodra", hidden=c["width"], vocab=c["vocab"], rms_eps=float(c["norm"]["eps"]), norm_kind="layer",
+        norm_place="pre", streams=int(c.get("streams") or 1), residual_mult=float(c.get("residual_mult", 1.0)), blocks=blocks, n_heads=max(1, top("heads", att)),
+        q_lora=0, kv_lora=0, qk_nope=0, qk_rope=0, v_head=top("vdim", att), dense_inter=0, first_k_dense=0, n_routed=top("experts", moe), top_k=top("top", moe),
+        n_shared=0, moe_inter=top("ff", moe), norm_topk_prob=True, kda_heads=top("heads", rec), kda_head_dim=top("dim", rec),
+        max_position=int(c.get("max_position", 1 << 20)))
+
+
 # architectures whose config.json is described by its own keys ("architecture": name) rather than HuggingFace ones
-NATIVE_CONFIGS = {"gazutar": gazutar_config, "rubasun": rubasun_config}
+NATIVE_CONFIGS = {"gazutar": gazutar_config, "rubasun": rubasun_config, "fasodra": fasodra_config}
 
 
 def from_hf_config(path_or_dict) -> ModelConfig:

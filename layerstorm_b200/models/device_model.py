@@ -43,11 +43,13 @@ def _align(x, a):
     return (x + a - 1) // a * a
 
 
-def expert_layout(fmt: str, H: int, F: int, down_fmt: Optional[str] = None) -> ExpertFmt:
+def expert_layout(fmt: str, H: int, F: int, down_fmt: Optional[str] = None, gated: bool = True) -> ExpertFmt:
     """Byte layout of one expert slot (gate | up | down weights, then their scales, then a tail
     of per-tensor scales), slot stride 4096-aligned like the reference's prepacked slots
     (src/model/weight_pipeline/prepacked_format.h:44-52).  ``down_fmt``: GGUF files mix block types per tensor; the down
-    matrix may be another GGUF block type than gate / up."""
+    matrix may be another GGUF block type than gate / up.  ``gated`` False: experts of an up and a down matrix (bf16, fp32)."""
+    if not gated and fmt not in ("bf16", "f32"):
+        raise ValueError(f"experts without a gate are kept in bf16 or fp32, not in {fmt}")
     ef = ExpertFmt()
     ef.fmt, ef.H, ef.F = EXPERT_FMT[fmt], H, F
     if fmt in GGML_OF and (fmt != "gguf_q4_k" or (down_fmt or fmt) != fmt):
@@ -66,9 +68,9 @@ def expert_layout(fmt: str, H: int, F: int, down_fmt: Optional[str] = None) -> E
         raise ValueError("a separate down format is only supported between GGUF block types")
     if fmt in ("bf16", "f32"):
         wb = H * F * (2 if fmt == "bf16" else 4)
-        ef.off_gate, ef.off_up, ef.off_down = 0, wb, 2 * wb
-        ef.off_sg = ef.off_su = ef.off_sd = ef.off_tail = 3 * wb
-        end = 3 * wb
+        up = wb if gated else 0
+        ef.off_gate, ef.off_up, ef.off_down = 0, up, up + wb
+        ef.off_sg = ef.off_su = ef.off_sd = ef.off_tail = end = up + 2 * wb
     elif fmt == "fp8_e4m3":
         wb = H * F
         ef.off_gate, ef.off_up, ef.off_down = 0, wb, 2 * wb
@@ -454,15 +456,18 @@ class ExpertArena:
     def slot_view(self, slot: int) -> torch.Tensor:
         return self.data[slot]
 
-    def write_expert(self, slot: int, gate: QLinear, up: QLinear, down: QLinear):
+    def write_expert(self, slot: int, gate: Optional[QLinear], up: QLinear, down: QLinear):
+        """``gate`` None: an arena of experts without a gate."""
         ef, v = self.ef, self.data[slot]
 
         def put(off, t):
             b = t.contiguous().view(torch.uint8).reshape(-1)
             v[off: off + b.numel()] = b
 
-        put(ef.off_gate, gate.w); put(ef.off_up, up.w); put(ef.off_down, down.w)
-        if gate.scales is not None:
+        if gate is not None:
+            put(ef.off_gate, gate.w)
+        put(ef.off_up, up.w); put(ef.off_down, down.w)
+        if gate is not None and gate.scales is not None:
             put(ef.off_sg, gate.scales); put(ef.off_su, up.scales); put(ef.off_sd, down.scales)
         if ef.fmt == 2:
             put(ef.off_tail, torch.tensor([gate.alpha, up.alpha, down.alpha], dtype=torch.float32, device=v.device))
@@ -724,7 +729,8 @@ class ModelBase:
 
     def weight_bytes(self) -> int:
         tot = self.head.nbytes() + (self.embed.numel() * 2 if self.embed.is_cuda else 0)
-        for L in self.layers + self.mtp_layers:
+        layers = self.layers + self.mtp_layers
+        for L in layers + [M for L in layers for M in L.get("sides", ())]:           # (layers with mixers side by side: a dictionary for each)
             for v in L.values():
                 if isinstance(v, QLinear):
                     tot += v.nbytes()
@@ -759,8 +765,8 @@ class ModelBase:
             nat.call("lsb_moe_build_groups", ws.ids, R * S, E, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups, ws.counts)
 
     def moe_experts(self, arena: "ExpertArena", ws, x, R: int, E: int, limit: float, miss, act=None):
-        """gate/up + gated unit and down projections of every pair whose expert is resident (``arena.slot_of[e] >= 0``).  ``act``: (sigmoid slope,
-        shift of the linear half, input scale per pair or None) of another unit than SwiGLU."""
+        """gate/up + gated unit and down projections of every pair whose expert is resident (``arena.slot_of[e] >= 0``).  ``act``: another unit than SwiGLU,
+        (sigmoid slope, shift of the linear half, input scale per pair or None), or "relu2" for experts without a gate."""
         S = ws.S
         efp = ctypes.addressof(arena.ef)
         mode = self.moe_mode(arena, ws, R)
@@ -787,8 +793,8 @@ class ModelBase:
                 return
             up = (ws.tc_xs, ws.tc_xs.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n, ws.tc_cnt, ws.tc_sorted, ws.tc_act,
                   ws.tc_bn, tiles, limit)
-            if act is None:
-                nat.call("lsb_moe_tc_ffn", 1, *up, miss, err, None)
+            if act is None or act == "relu2":
+                nat.call("lsb_moe_tc_ffn", 1 if act is None else 2, *up, miss, err, None)
             else:
                 nat.call("lsb_moe_tc_gateup_act", *up, *act, miss, err)
             nat.call("lsb_moe_tc_ffn", 0, ws.tc_act, ws.tc_act.shape[0], arena.data, arena.slot_of, efp, ws.tc_tile_e, ws.tc_tile_r0, ws.tc_tile_n,
@@ -807,6 +813,8 @@ class ModelBase:
             up = (x, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups, ws.act, S, mg, limit)
             if act is None:
                 nat.call("lsb_moe_gateup", *up, miss, 0)
+            elif act == "relu2":
+                nat.call("lsb_moe_up", *up[:-1], miss)
             else:
                 nat.call("lsb_moe_gateup_act", *up, *act, miss, 0)
             nat.call("lsb_moe_down", ws.act, arena.data, arena.slot_of, efp, ws.group_expert, ws.group_n, ws.group_pairs, ws.n_groups,

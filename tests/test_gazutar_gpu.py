@@ -55,7 +55,7 @@ class Paged:
         nat.call("lsb_attn_prep", proj, proj.shape[1], oq, ok, ov, wq, wk, eps, vfirst, mix, lam, q, self.cache, self.bt, self.max_pages, seq, pos, R, H, G,
                  dk, dv, self.dkp, self.dvp, self.page, int(self.f32))
         nat.call("lsb_attn", q, self.cache, self.bt, self.max_pages, self.page, seq, pos, row0, i32(n), len(n), run_rows or max(n), proj, proj.shape[1],
-                 og if gate else -1, out, H * dv + 8, op, ml, NS, R, H, G, dk, dv, self.dkp, self.dvp, window, scale, slope, int(self.f32))
+                 og if gate else -1, out, H * dv + 8, op, ml, NS, R, H, G, dk, dv, self.dkp, self.dvp, window, scale, slope, 0, 0, None, 0, 1.0, int(self.f32))
         torch.cuda.synchronize()
         return out[:, : H * dv].float().cpu()
 
