@@ -215,3 +215,112 @@ def forward(cfg, w, tokens, want_layers=False):
         layers.append(sum(xs))
     lg = layer_norm(sum(xs), w["final.norm"], w["final.norm.b"], eps) @ w["head"].T
     return (lg, layers) if want_layers else lg
+
+
+# ------------------------------------------------------------------------------------------------ random models
+def random_model(cfg, seed=0, close_calls=True, rel_rows=(32, 10, 6), rank=12):
+    """Tensors for a configuration, spread so that every mechanism matters.  ``rel_rows``: rows of the distance bias tables, in turns.  Without
+    ``close_calls`` the bias of the norm in front of a router decides the choice (rounding cannot turn it)."""
+    g = torch.Generator().manual_seed(seed)
+    n = lambda *s: torch.randn(*s, generator=g)
+    u = lambda lo, hi, *s: lo + (hi - lo) * torch.rand(s, generator=g)
+    H, V, S, w = cfg["width"], cfg["vocab"], cfg["streams"], {}
+    lin = lambda o, i: n(o, i) / i ** 0.5
+
+    def norm(p):
+        w[p], w[p + ".b"] = 1.0 + 0.2 * n(H), 0.3 * n(H)
+
+    def attn(p, m, gate=False, weight=False):
+        for t, c in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
+            w[p + t], w[p + t + ".b"] = 1.5 * lin(c, H), 0.4 * n(c)
+        if weight:
+            w[p + "q.norm"], w[p + "k.norm"] = 1.5 * (1.0 + 0.2 * n(m["dim"])), 1.0 + 0.2 * n(m["dim"])
+        if gate:
+            w[p + "g"] = lin(m["heads"], H)
+        w[p + "o"] = lin(H, m["heads"] * m["vdim"])
+
+    def time(p, m):
+        c = m["heads"] * m["dim"]
+        for t in "rkvgw":
+            w[p + "mu." + t] = u(0.1, 0.9, H)
+        for t in "rkvg":
+            w[p + t] = lin(c, H)
+        w[p + "w1"], w[p + "w2"], w[p + "w0"], w[p + "u"] = lin(rank, H), 1.5 * lin(c, rank), u(-5.0, 0.5, c), 0.7 * n(m["heads"], m["dim"])
+        w[p + "norm"], w[p + "o"] = 1.0 + 0.2 * n(c), lin(H, c)
+
+    def delta(p, m):
+        h, k, v = m["heads"], m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+        for t, c in (("q", k), ("k", k), ("v", v)):
+            w[p + t], w[p + t + ".conv"] = lin(c, H), u(-1.0, 1.0, c, m["conv"])
+        w[p + "b"], w[p + "a"], w[p + "g"], w[p + "o"] = lin(h, H), lin(h, H), lin(v, H), lin(H, v)
+        w[p + "A_log"], w[p + "dt_bias"], w[p + "norm"] = u(-3.0, 0.5, h), u(-3.0, 0.0, h), 1.0 + 0.2 * n(m["vdim"])
+
+    w["embed"], w["head"] = n(V, H), lin(V, H)
+    norm("final.norm")
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        x = p + "mix."
+        norm(p + "norm1")
+        if L["type"] == "attention":
+            attn(x, m)
+            w[x + "rel"] = n(rel_rows[i % len(rel_rows)], m["heads"])
+        elif L["type"] == "parallel":
+            attn(x + "left.", m["left"], gate=True)
+            time(x + "right.", m["right"])
+        else:
+            attn(x + "left.", m["left"], weight=True)
+            delta(x + "right.", m["right"])
+            w[x + "left.out"], w[x + "right.out"] = 1.0 + 0.2 * n(H), 1.0 + 0.2 * n(H)
+        for q in (1, 2) if L.get("mlp") else (1,):
+            w[f"{p}hc{q}.in"], w[f"{p}hc{q}.out"], w[f"{p}hc{q}.mix"] = u(0.4, 1.2, S), u(0.5, 1.3, S), torch.eye(S) * 0.9 + 0.15 * n(S, S)
+        if L.get("mlp"):
+            norm(p + "norm2")
+            z, E, f = p + "mlp.", L["mlp"]["router"]["experts"], L["mlp"]["expert"]["ff"]
+            w[z + "router"] = 1.5 * lin(E, H)
+            if not close_calls:
+                b = w[p + "norm2.b"]
+                w[z + "router"] = 0.1 * lin(E, H) + (torch.randperm(E, generator=g).float() - E / 2)[:, None] * b / b.square().sum()
+            for j in range(E):
+                w[z + f"e{j}.up"], w[z + f"e{j}.down"] = lin(f, H), lin(H, f)
+    return w
+
+
+def att(heads, kv_heads, dim, vdim, chunk, reach, mlp=None, scale=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or round(2.0 / dim ** 0.5, 4), "bias_max": reach, "mask": {"size": chunk}}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def left(heads, kv_heads, dim, vdim, rot, base=10000.0):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": round(1.6 / dim ** 0.5, 4), "rot": {"base": base, "dims": rot}}
+
+
+def par(lft, heads, dim, scales=(0.8, 1.2), mlp=None):
+    return {"type": "parallel", "mixer": {"left": lft, "right": {"heads": heads, "dim": dim}, "left_scale": scales[0], "right_scale": scales[1]}, "mlp": mlp}
+
+
+def par2(lft, heads, kv_heads, dim, vdim, conv, mlp=None):
+    return {"type": "parallel_2", "mixer": {"left": lft, "right": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}, "mlp": mlp}
+
+
+def moe_spec(experts, top, ff):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+
+
+def model_cfg(width, vocab, streams, layers, eps=1e-5, mult=0.9):
+    return {"architecture": "Fasodra", "layers": layers, "norm": {"eps": eps}, "residual_mult": mult, "streams": streams, "vocab": vocab, "width": width}
+
+
+# several geometries: every kind first and last, layers without a feed-forward, sizes off the kernels' tiles and on them, sizes of one, key heads wider
+# than the chunked recurrences and the tensor-core attention take, one stream and many
+MODELS = {
+    "odd": lambda: model_cfg(136, 301, 3, [att(6, 2, 24, 40, 21, 50, moe_spec(5, 2, 40)), par(left(4, 2, 20, 12, 6, 500.0), 5, 12, mlp=moe_spec(7, 3, 24)),
+                                           par2(left(3, 3, 36, 20, 36), 4, 2, 24, 20, 3, moe_spec(4, 1, 56)), att(3, 1, 40, 9, 70, 20),
+                                           par(left(5, 1, 9, 24, 8, 77.0), 3, 40, (-0.6, 0.5)), par2(left(2, 1, 44, 30, 10), 6, 1, 40, 12, 5)], 3e-3, 0.7),
+    "tiles": lambda: model_cfg(384, 520, 2, [par2(left(4, 4, 128, 128, 64, 1e6), 4, 4, 128, 128, 4, moe_spec(12, 4, 128)), att(16, 2, 128, 64, 130, 128, moe_spec(12, 4, 128)),
+                                             par(left(8, 2, 64, 64, 32), 4, 64, mlp=moe_spec(12, 4, 256)), att(8, 1, 96, 32, 64, 40, moe_spec(8, 3, 128))]),
+    "ones": lambda: model_cfg(48, 40, 1, [par(left(1, 1, 2, 1, 2), 1, 1, (1.0, 1.0), moe_spec(1, 1, 1)), att(1, 1, 1, 2, 1, 9), par2(left(16, 1, 3, 1, 2, 3.0), 3, 3, 1, 1, 1, moe_spec(3, 3, 8)),
+                                          att(2, 2, 8, 8, 3, 17)], 1e-6, 1.0),
+    "wide": lambda: model_cfg(250, 200, 5, [att(33, 1, 24, 16, 90, 60, moe_spec(4, 1, 96)), par(left(2, 2, 200, 136, 100), 2, 160, mlp=moe_spec(6, 2, 64)),
+                                            par2(left(5, 1, 260, 24, 130), 2, 1, 160, 72, 4), par2(left(2, 2, 16, 272, 16), 2, 2, 48, 200, 2, moe_spec(6, 5, 32)),
+                                            par(left(70, 1, 8, 8, 4), 1, 128)], 1e-4, 1.1),
+}
