@@ -1,10 +1,11 @@
 """Prefill and decode throughput of a model design at layer sizes of a real model (random weights), beside the framework's closest other
 design at equal size, with the device time of every kernel launcher.
 
-    python bench.py --design gazutar|rubasun [--design-sizes 2048,4096]
+    python bench.py --design gazutar|rubasun|fasodra [--design-sizes 2048,4096]
 
 Gazutar's neighbour is a KDA + MLA model of the same width, heads, experts and layer pattern (plain residual stream, dense latent attention),
-Rubasun's an MLA + MoE model of the same width, heads, latent rows, experts and shared expert.
+Rubasun's an MLA + MoE model of the same width, heads, latent rows, experts and shared expert, Fasodra's the Gazutar model of the same width,
+attention heads and expert parameters.
 Per launcher: all its calls of one step, recorded from an eager pass and replayed back to back in a CUDA graph (other layers' operands in
 between, so that a layer's weights are not left over in L2), divided by the number of calls.  Fractions are of the measured peaks
 (MEASURED_PEAKS.json): bytes or FLOPs that the operation has to move or do, over the launcher's time.
@@ -18,7 +19,7 @@ import statistics
 import torch
 
 from ..models.block_model import model_class
-from ..models.config import ModelConfig, gazutar_config, rubasun_config
+from ..models.config import ModelConfig, fasodra_config, gazutar_config, rubasun_config
 from ..ops import _native as nat
 from ..runtime.engine import Engine
 
@@ -54,7 +55,23 @@ def rubasun_pair(hidden: int):
     return g, k
 
 
-DESIGNS = {"gazutar": gazutar_pair, "rubasun": rubasun_pair}
+def fasodra_pair(hidden: int):
+    """(Fasodra, neighbour) of one size: 128-wide attention heads, 64-wide time-mixing heads over the whole width, half as many delta heads as the
+    neighbour, ungated experts of the neighbour's parameter count.  Chunks of 5120: the 8k context ends 3072 tokens into one."""
+    heads, kv, experts, ff, vocab = hidden // 128, max(1, hidden // 512), hidden // 64, hidden * 3 // 4, 65536
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": TOP}}
+    base = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    lft = base | {"rot": {"base": 1e5, "dims": 64}}
+    kinds = [("attention", base | {"bias_max": 4096, "mask": {"size": 5120}}),
+             ("parallel", {"left": lft, "right": {"heads": hidden // 64, "dim": 64}, "left_scale": 0.7, "right_scale": 0.9}),
+             ("attention", base | {"bias_max": 4096, "mask": {"size": 5120}}),
+             ("parallel_2", {"left": lft, "right": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}})]
+    f = fasodra_config({"name": f"fasodra-{hidden}", "vocab": vocab, "width": hidden, "norm": {"eps": 1e-5}, "residual_mult": 0.8, "streams": 2,
+                        "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(N_LAYERS)]})
+    return f, gazutar_pair(hidden)[0]
+
+
+DESIGNS = {"gazutar": gazutar_pair, "rubasun": rubasun_pair, "fasodra": fasodra_pair}
 
 
 def _peaks():
@@ -121,7 +138,8 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
     per_tok = heads * (4 * 128 * 128 + 6 * 64 * 128) * 2            # chunk form: state products, pair products
     decode = rows == batch
     rec = ("bytes", state + gates + rows * heads * 128 * 18) if decode else ("flops", rows * per_tok)
-    att = next((x for x in cfg.blocks if not x.recurrent), None)
+    mixers = [x for b in cfg.blocks for x in b.mixers]
+    att = next((x for x in mixers if not x.recurrent), None)
     lat, rot, ah, dn, dv = cfg.kv_lora, cfg.qk_rope, cfg.n_heads, cfg.qk_nope, cfg.v_head
     seen = ctx - rows // 2                                          # keys a row of the chunk sees on average
     latent = ("bytes", batch * ctx * (lat + rot) * 2 + rows * ah * (2 * lat + rot) * 2) if decode else ("flops", 2 * rows * seen * ah * (2 * lat + rot))
@@ -135,13 +153,29 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
         out["lsb_resid_update"] = ("bytes", rows * H * 14)
         out["lsb_glu"] = ("bytes", rows * cfg.moe_inter * 10)
     elif att is not None:
-        b = att
-        seen = min(ctx, b.window)
-        out["lsb_delta_forward"] = rec
-        kv = b.kv_heads * (b.dim + b.vdim) * 2
-        out["lsb_attn"] = ("bytes", batch * seen * kv + rows * b.heads * b.vdim * 6) if decode else ("flops", 2 * rows * seen * b.heads * (b.dim + b.vdim))
-        out["lsb_attn_prep"] = ("bytes", rows * ((b.heads + b.kv_heads) * b.dim + b.kv_heads * b.vdim) * 6)
+        mean = lambda xs: sum(xs) / max(1, len(xs))
+        keys = lambda b: min(ctx % b.chunk or b.chunk if b.chunk else ctx, b.window or ctx)            # that a decoded token sees
+        per_row = lambda b: mean([min(p % b.chunk + 1 if b.chunk else p + 1, b.window or ctx) for p in range(ctx - rows, ctx)])
+        soft = [b for b in mixers if b.softmax]
+        kv = lambda b: b.kv_heads * (b.dim + b.vdim) * 2
+        out["lsb_attn"] = (("bytes", mean([batch * keys(b) * kv(b) + rows * b.heads * b.vdim * (6 if b.out_gate else 4) for b in soft])) if decode
+                           else ("flops", mean([2 * rows * per_row(b) * b.heads * (b.dim + b.vdim) for b in soft])))
+        out["lsb_attn_prep"] = out["lsb_attn_head_prep"] = ("bytes", mean([rows * ((b.heads + b.kv_heads) * b.dim + b.kv_heads * b.vdim) * 6 for b in soft]))
         out["lsb_resid_update"] = ("bytes", rows * H * (14 + TOP * 4) // 2 + rows * H * 7)
+        # chunk form: two state products and two (delta rule: six, with the solve) products over pairs of a chunk
+        dlt, tm = [b for b in mixers if b.delta], [b for b in mixers if b.kind == "time_mix"]
+        st = lambda b: 2 * batch * b.heads * b.dim * b.vdim * 4                                        # the state read and written once
+        if decode:
+            low = lambda b: b.heads * (b.dim + b.vdim) * 128 * 2 if b.kind == "channel_delta" else 0
+            out["lsb_delta_forward"] = ("bytes", mean([st(b) + low(b) + rows * b.heads * b.dim * 18 for b in dlt]))
+            out["lsb_tmix_forward"] = ("bytes", mean([st(b) + b.heads * b.dim * b.dim * 2 + rows * b.heads * b.dim * 18 for b in tm]))
+        else:
+            out["lsb_delta_forward"] = ("flops", mean([rows * b.heads * (4 * b.dim * b.vdim + 6 * 64 * b.dim) * 2 for b in dlt]))
+            out["lsb_tmix_forward"] = ("flops", mean([rows * b.heads * (2 * b.dim * b.vdim + 2 * 64 * b.dim) * 2 for b in tm]))
+        out["lsb_tmix_shift"] = ("bytes", rows * H * 12)
+        n = cfg.streams
+        ups = [rows * H * (4 + 4 * n + 2)] + [rows * H * (8 * n + 2 + s) for b in cfg.blocks for s in ((8 if b.join == "normed" and b.branches else 4), TOP * 4)]
+        out["lsb_stream_update"] = ("bytes", mean(ups))
     else:
         out["lsb_kda_forward"] = out["lsb_kda_forward_chunked"] = rec
         out["lsb_mla_decode"] = latent
@@ -151,10 +185,11 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
         out["lsb_mla_prep"] = ("bytes", rows * (cfg.q_lora + lat + rot) * 6)
     if rows == 1:                          # (how many experts a batch touches is the router's affair)
         by = experts * 3 * H * cfg.moe_inter * 2
+        out["lsb_moe_up"] = ("bytes", by / 3)
         out["lsb_moe_gateup"] = out["lsb_moe_gateup_act"] = ("bytes", by * 2 / 3)
         out["lsb_moe_down"] = ("bytes", by / 3)
     elif rows > 1024:
-        own = att is not None and att.scale_input                    # gate/up and down are launchers of their own, else halves of one launcher's calls
+        own = cfg.blocks and (cfg.blocks[-1].scale_input or cfg.blocks[-1].unit != "glu")      # up and down are one size, or gate/up is a launcher of its own
         out["lsb_moe_tc_ffn"] = ("flops", (2 if own else 3) * rows * experts * H * cfg.moe_inter)
         out["lsb_moe_tc_gateup_act"] = ("flops", 4 * rows * experts * H * cfg.moe_inter)
     return out
