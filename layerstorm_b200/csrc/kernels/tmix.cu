@@ -277,7 +277,7 @@ __global__ void __launch_bounds__(256) tmix_chunk_kernel(TmixParams p, TmixScrat
     float* sL = sK + kCh * kLdK;              // [t][c] log decay, then its sum over the sub-chunk up to and including t
     float* sA = sL + kCh * kLdK;              // [t][s] pair products
     float* sV = sA + kCh * kLdC;              // [v][t] values of a tile
-    float* sX = sV + kCh * kLdC;              // [16][kLdR] rescaled r rows of a sub-chunk
+    float* sX = sV + kCh * kLdC;              // [16][kLdR] rescaled r rows of a sub-chunk;  first, with sY: [64][kLdR] decay factors
     float* sY = sX + kSub * kLdR;             // [48][kLdR] rescaled earlier k rows
     const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, tx = tid & 15, ty = tid >> 4;
     pdl_wait();
@@ -286,6 +286,7 @@ __global__ void __launch_bounds__(256) tmix_chunk_kernel(TmixParams p, TmixScrat
     tmix_find(p, nseq, chunk, seq, row0, c0, cc);
     if (cc <= 0 || p.seq_slot[seq] < 0) return;
     const int r0 = row0 + c0, dk = p.dk;
+#pragma unroll 8
     for (int idx = tid; idx < kCh * kD; idx += 256) {
         const int t = idx / kD, c = idx % kD;
         float r = 0.f, k = 0.f, l = 0.f;
@@ -296,6 +297,7 @@ __global__ void __launch_bounds__(256) tmix_chunk_kernel(TmixParams p, TmixScrat
             l = tmix_log_decay(w.rawd[(size_t)(r0 + t) * p.H * dk + h * dk + c] + p.w0[(size_t)h * dk + c]);
         }
         sR[t * kLdK + c] = r; sK[t * kLdK + c] = k; sL[t * kLdK + c] = l;
+        sX[t * kLdR + c] = expf(l);
     }
     for (int idx = tid; idx < kCh * kLdC; idx += 256) sA[idx] = 0.f;
     __syncthreads();
@@ -306,28 +308,47 @@ __global__ void __launch_bounds__(256) tmix_chunk_kernel(TmixParams p, TmixScrat
     }
     __syncthreads();
     auto total = [&](int sub, int c) { return sL[(sub * kSub + kSub - 1) * kLdK + c]; };
-    // pair products: inside a sub-chunk one warp per pair; against earlier sub-chunks a product of two rescaled tiles
-    for (int I = 0; I < kCh / kSub; ++I) {
-        const int t0 = I * kSub;
-        if (t0 >= cc) break;                                   // block-uniform
-        for (int pidx = warp; pidx < kSub * (kSub + 1) / 2; pidx += 8) {
-            int dt = 0, ds = pidx;
-            while (ds > dt) { ds -= dt + 1; ++dt; }
-            const int t = t0 + dt, s = t0 + ds;
-            if (t >= cc) continue;                             // warp-uniform
-            float a = 0.f;
+    // pair products inside the sub-chunks: a warp takes a row t and walks back over its predecessors, the factors between them multiplied up in
+    // registers; the 16 sums over the lanes' channels are folded together, lane 2 d ends up with the one of distance d
+    for (int t = warp; t < cc; t += 8) {
+        const int dt = t % kSub;
+        float P[kD / 32], a[kSub];
+#pragma unroll
+        for (int i = 0; i < kD / 32; ++i) P[i] = sR[t * kLdK + lane + 32 * i];
+#pragma unroll
+        for (int d = 0; d < kSub; ++d) {
+            a[d] = 0.f;
+            if (d > dt) continue;                              // warp-uniform
 #pragma unroll
             for (int i = 0; i < kD / 32; ++i) {
                 const int c = lane + 32 * i;
-                float f;
-                if (ds == dt) f = c < dk ? p.u[(size_t)h * dk + c] : 0.f;
-                else f = __expf(fminf(sL[(t - 1) * kLdK + c] - sL[s * kLdK + c], 0.f));
-                a = fmaf(sR[t * kLdK + c] * f, sK[s * kLdK + c], a);
+                const float k = sK[(t - d) * kLdK + c];
+                if (d == 0) {
+                    a[d] = fmaf(P[i] * (c < dk ? p.u[(size_t)h * dk + c] : 0.f), k, a[d]);
+                } else {
+                    a[d] = fmaf(P[i], k, a[d]);
+                    P[i] *= sX[(t - d) * kLdR + c];
+                }
             }
-            a = warp_sum(a);
-            if (lane == 0) sA[t * kLdC + s] = a;
         }
-        if (I == 0) continue;
+#pragma unroll
+        for (int o = 16, n = kSub / 2; n >= 1; o >>= 1, n >>= 1) {
+#pragma unroll
+            for (int j = 0; j < kSub / 2; ++j) {
+                if (j >= n) break;
+                const float give = lane & o ? a[j] : a[j + n], keep = lane & o ? a[j + n] : a[j];
+                a[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+            }
+        }
+        a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
+        const int d = lane >> 1;
+        if ((lane & 1) == 0 && d <= dt) sA[t * kLdC + t - d] = a[0];
+    }
+    __syncthreads();                                           // sX and sY are refilled next
+    // against earlier sub-chunks: a product of two rescaled tiles
+    for (int I = 1; I < kCh / kSub; ++I) {
+        const int t0 = I * kSub;
+        if (t0 >= cc) break;                                   // block-uniform
         for (int idx = tid; idx < kSub * kD; idx += 256) {
             const int tt = idx / kD, c = idx % kD;
             sX[tt * kLdR + c] = sR[(t0 + tt) * kLdK + c] * (tt ? expf(sL[(t0 + tt - 1) * kLdK + c]) : 1.f);
@@ -352,6 +373,7 @@ __global__ void __launch_bounds__(256) tmix_chunk_kernel(TmixParams p, TmixScrat
     }
     __syncthreads();
     // r and k times the decays from the chunk's start and to its end; the chunk's whole decay
+#pragma unroll 4
     for (int idx = tid; idx < kCh * kD; idx += 256) {
         const int t = idx / kD, c = idx % kD, J = t / kSub;
         float before = t % kSub ? sL[(t - 1) * kLdK + c] : 0.f, after = total(J, c) - sL[t * kLdK + c];
@@ -363,6 +385,7 @@ __global__ void __launch_bounds__(256) tmix_chunk_kernel(TmixParams p, TmixScrat
     }
     __syncthreads();
     for (int v0 = 0; v0 < p.dv; v0 += kCh) {
+#pragma unroll 8
         for (int idx = tid; idx < kCh * kCh; idx += 256) {
             const int t = idx / kCh, v = idx % kCh;
             sV[v * kLdC + t] = t < cc && v0 + v < p.dv ? p.proj[(size_t)(r0 + t) * p.ldp + p.off_v + h * p.dv + v0 + v] : 0.f;
@@ -439,7 +462,8 @@ __global__ void __launch_bounds__(256) tmix_scan_kernel(TmixParams p, TmixScratc
     *st = S;
 }
 
-template <int kD, typename T>
+// ONE: value heads of up to 64 channels, whose outputs stay in registers up to the norm
+template <int kD, bool ONE, typename T>
 __global__ void __launch_bounds__(256) tmix_out_kernel(TmixParams p, TmixScratch w, int nseq) {
     constexpr int kLdK = TmixDims<kD>::kLdK;
     extern __shared__ __align__(16) float csm[];
@@ -452,41 +476,69 @@ __global__ void __launch_bounds__(256) tmix_out_kernel(TmixParams p, TmixScratch
     tmix_find(p, nseq, chunk, seq, row0, c0, cc);
     if (cc <= 0 || p.seq_slot[seq] < 0) return;
     const int r0 = row0 + c0;
+#pragma unroll
     for (int idx = tid; idx < kCh * (kD / 4); idx += 256) {
         const int t = idx / (kD / 4), c4 = idx % (kD / 4) * 4;
         *reinterpret_cast<float4*>(sQ + t * kLdK + c4) =
             t < cc ? *reinterpret_cast<const float4*>(w.qp + ((size_t)(r0 + t) * p.H + h) * kD + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    float acc[4][4], g[4][4];
     for (int v0 = 0; v0 < p.dv; v0 += kCh) {
+#pragma unroll
         for (int idx = tid; idx < kCh * (kD / 4); idx += 256) {
             const int v = idx / (kD / 4), c4 = idx % (kD / 4) * 4;
             *reinterpret_cast<float4*>(sS + v * kLdK + c4) =
                 v0 + v < p.dv ? *reinterpret_cast<const float4*>(w.kv + (((size_t)chunk * p.H + h) * p.dv + v0 + v) * kD + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
-        __syncthreads();
-        float acc[4][4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-        kda_mm_nt<kD>(sQ, kLdK, sS, kLdK, acc, tx, ty);
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int t = ty + 16 * i, v = v0 + tx + 16 * j;
-                if (t < cc && v < p.dv) w.o[((size_t)(r0 + t) * p.H + h) * p.dv + v] += acc[i][j];
+                const bool in = t < cc && v < p.dv;
+                acc[i][j] = in ? w.o[((size_t)(r0 + t) * p.H + h) * p.dv + v] : 0.f;
+                if (ONE) g[i][j] = in ? p.proj[(size_t)(r0 + t) * p.ldp + p.off_g + h * p.dv + v] : 0.f;
+            }
+        __syncthreads();
+        kda_mm_nt<kD>(sQ, kLdK, sS, kLdK, acc, tx, ty);
+        if (ONE) break;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int t = ty + 16 * i, v = v0 + tx + 16 * j;
+                if (t < cc && v < p.dv) w.o[((size_t)(r0 + t) * p.H + h) * p.dv + v] = acc[i][j];
             }
         __syncthreads();
     }
-    for (int t = warp; t < cc; t += 8) {
-        const float* o = w.o + ((size_t)(r0 + t) * p.H + h) * p.dv;
-        const float* g = p.proj + (size_t)(r0 + t) * p.ldp + p.off_g + h * p.dv;
-        float q = 0.f;
-        for (int c = lane; c < p.dv; c += 32) q = fmaf(o[c], o[c], q);
-        const float rs = 1.f / sqrtf(warp_sum(q) / (float)p.dv + p.eps);
-        for (int c = lane; c < p.dv; c += 32)
-            reinterpret_cast<T*>(p.out)[(size_t)(r0 + t) * p.ldo + (size_t)h * p.dv + c] = act_out<T>(o[c] * rs * p.onorm[(size_t)h * p.dv + c] * tmix_silu(g[c]));
+    if constexpr (ONE) {
+        float on[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) on[j] = tx + 16 * j < p.dv ? p.onorm[(size_t)h * p.dv + tx + 16 * j] : 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int t = ty + 16 * i;
+            float q = 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) q = fmaf(acc[i][j], acc[i][j], q);          // columns past dv hold zeros
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
+            const float rs = 1.f / sqrtf(q / (float)p.dv + p.eps);
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (t < cc && tx + 16 * j < p.dv)
+                    reinterpret_cast<T*>(p.out)[(size_t)(r0 + t) * p.ldo + (size_t)h * p.dv + tx + 16 * j] = act_out<T>(acc[i][j] * rs * on[j] * tmix_silu(g[i][j]));
+        }
+    } else {
+        for (int t = warp; t < cc; t += 8) {
+            const float* o = w.o + ((size_t)(r0 + t) * p.H + h) * p.dv;
+            const float* gr = p.proj + (size_t)(r0 + t) * p.ldp + p.off_g + h * p.dv;
+            float q = 0.f;
+            for (int c = lane; c < p.dv; c += 32) q = fmaf(o[c], o[c], q);
+            const float rs = 1.f / sqrtf(warp_sum(q) / (float)p.dv + p.eps);
+            for (int c = lane; c < p.dv; c += 32)
+                reinterpret_cast<T*>(p.out)[(size_t)(r0 + t) * p.ldo + (size_t)h * p.dv + c] = act_out<T>(o[c] * rs * p.onorm[(size_t)h * p.dv + c] * tmix_silu(gr[c]));
+        }
     }
     if (h == 0 && c0 + cc == p.seq_nrows[seq]) tmix_keep<T>(p, seq, p.seq_slot[seq]);
 }
@@ -509,12 +561,14 @@ static int launch_tmix_chunks(const TmixParams& p, const TmixScratch& w, int nse
     static bool attr = false;
     if (!attr) {
         cudaFuncSetAttribute(tmix_chunk_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TmixDims<DKP>::kChunkSmem);
-        cudaFuncSetAttribute(tmix_out_kernel<DKP, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TmixDims<DKP>::kOutSmem);
+        cudaFuncSetAttribute(tmix_out_kernel<DKP, true, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TmixDims<DKP>::kOutSmem);
+        cudaFuncSetAttribute(tmix_out_kernel<DKP, false, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TmixDims<DKP>::kOutSmem);
         attr = true;
     }
     launch_pdl((tmix_chunk_kernel<DKP>), dim3(nchunks, p.H), 256, TmixDims<DKP>::kChunkSmem, st, p, w, nseq);
     launch_pdl((tmix_scan_kernel), dim3((p.dv * DKP / 4 + 255) / 256, p.H, nseq), 256, 0, st, p, w, DKP);
-    launch_pdl((tmix_out_kernel<DKP, T>), dim3(nchunks, p.H), 256, TmixDims<DKP>::kOutSmem, st, p, w, nseq);
+    if (p.dv <= kCh) launch_pdl((tmix_out_kernel<DKP, true, T>), dim3(nchunks, p.H), 256, TmixDims<DKP>::kOutSmem, st, p, w, nseq);
+    else launch_pdl((tmix_out_kernel<DKP, false, T>), dim3(nchunks, p.H), 256, TmixDims<DKP>::kOutSmem, st, p, w, nseq);
     return (int)cudaGetLastError();
 }
 
