@@ -66,7 +66,8 @@ def kv_bytes_per_token(mc: ModelConfig, backend: str = "snapmla", tp: int = 1, k
     """All attention layers, one token, on one GPU.  Sharded mode keeps 1/tp of the rows per rank."""
     if mc.blocks:
         lat = lambda b: _align(b.kv_rank, 16) + _align(b.rot_dim, 16) if b.kv_from < 0 else 0       # (layers may read another layer's rows)
-        return float(sum(2 * (lat(b) if b.latent else b.kv_heads * (_head_pad(b.dim) + _head_pad(b.vdim))) for L in mc.blocks for b in L.mixers if not b.recurrent))
+        return float(sum(2 * (lat(b) if b.latent else b.kv_heads * (b.maps * _head_pad(b.dim) + _head_pad(b.vdim)))
+                         for i, _ in mc.layer_runs() for b in mc.blocks[i].mixers if not b.recurrent))
     mla = mc.mla_layers()
     idx_layers = len({mc.index_source_layer(i) for i in mla}) if mc.has_indexer else 0
     per = len(mla) * kv_row_bytes(mc, backend) + idx_layers * indexer_row_bytes(mc)
@@ -78,7 +79,8 @@ def recurrent_state_bytes_per_seq(mc: ModelConfig, tp: int = 1) -> int:
     if mc.blocks:
         pad = lambda d: next((p for p in (32, 64, 128) if d <= p), 256)
         kept = lambda b: _align(mc.hidden, 8) if b.kind == "time_mix" else b.heads * (2 * b.dim + b.vdim) * (b.conv - 1)      # previous input / convolutions
-        return sum((b.heads * b.vdim * pad(b.dim) + kept(b)) * 4 for L in mc.blocks for b in L.mixers if b.recurrent)
+        look_back = max(0, mc.input_conv - 1) * _align(mc.hidden, 8) * 4 * len(mc.layer_runs())                 # inputs of the mixers' convolutions
+        return look_back + sum((b.heads * b.vdim * pad(b.dim) + kept(b)) * 4 for i, _ in mc.layer_runs() for b in mc.blocks[i].mixers if b.recurrent)
     n_kda = sum(1 for t in mc.layer_types if t == "kda")
     if not n_kda:
         return 0
@@ -121,16 +123,19 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
             r.attention += w * 2 + ((2 * b.kv_heads * b.dim + b.heads * b.vdim) * b.conv + b.heads * b.dim) * 4
         elif b.latent:
             own = b.kv_rank + b.rot_dim if b.kv_from < 0 else 0
-            r.attention += ((b.heads * (b.dim + b.rot_dim + b.vdim + (1 if b.head_gate else 0)) + own) * H + b.heads * (b.dim + b.vdim) * b.kv_rank) * 2
+            q = b.heads * (b.dim + b.rot_dim)
+            r.attention += (((b.q_rank or q) + b.heads * (b.vdim * (2 if b.out_gate else 1) + (1 if b.head_gate else 0)) + own) * H + q * b.q_rank) * 2
+            r.attention += b.heads * (b.dim + b.vdim) * b.kv_rank * 2
         else:
-            r.attention += (b.heads * (b.dim + b.vdim * (2 if b.out_gate else 1) + (1 if b.head_gate else 0)) + b.kv_heads * (b.dim + b.vdim)) * H * 2
+            r.attention += (b.heads * (b.maps * b.dim + b.vdim * (2 if b.out_gate else 1) + (1 if b.head_gate else 0)) +
+                            b.kv_heads * (b.maps * b.dim + (0 if b.shared_kv else b.vdim))) * H * 2
             r.attention += (b.heads * (b.bias_max + 1) * 4 if b.bias_rows else 0) + ((b.heads * b.dim + b.kv_heads * (b.dim + b.vdim)) * 4 if b.qkv_bias else 0)
     for b in mc.blocks:
         r.dense_ffn += 3 * b.dense_ff * H * 2 + mc.side_dim * H * 2 * 2
         if b.experts:
             r.router += (b.experts + b.identity) * (2 * H + 4)
             r.shared_expert += (3 * b.shared_ff + (1 if b.shared_ff else 0)) * H * 2
-        r.norms += (4 if b.has_ff else 2) * H * 4 * (2 if mc.norm_place == "sandwich" else 1) + (H * 4 if mc.side_dim else 0)
+        r.norms += mc.input_conv * H * 4 + (4 if b.has_ff else 2) * H * 4 * (2 if mc.norm_place == "sandwich" else 1) + (H * 4 if mc.side_dim else 0)
         r.norms += (2 if b.has_ff else 1) * mc.streams * (mc.streams + 2) * 4 + (2 * H * 4 if b.branches and b.join == "normed" else 0)
     for i in range(0 if mc.blocks else mc.n_layers):
         if mc.is_kda_layer(i):
@@ -165,7 +170,7 @@ def resident_bytes(mc: ModelConfig, tp: int = 1, n_gpus: int = 1, embed_on_host:
             # two hyper-connection passes per layer: mixing matrix [(2n + n^2), n H] fp32, its base vector and three scales
             r.norms += 2 * ((2 * n + n * n) * (n * H + 1) + 3) * 4
     r.norms += H * 4                                                     # output norm
-    r.embedding = (0 if embed_on_host else mc.vocab * H * 2) + mc.vocab * mc.n_layers * mc.side_dim * 2
+    r.embedding = (0 if embed_on_host else mc.vocab * H * 2) + mc.vocab * mc.n_layers * mc.side_dim * 2 + (mc.bigram[0] + 1 if mc.bigram else 0) * H * 2
     r.head = int(mc.vocab * H * 2 / tp)
     return r
 

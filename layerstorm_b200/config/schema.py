@@ -13,7 +13,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any
 
-ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun", "fasodra")
+ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun", "fasodra", "nivasun")
 WEIGHT_QUANTS = ("nvfp4", "fp8_e4m3", "fp8_e5m2", "int4_symmetric", "int4_asymmetric", "bf16", "gguf", "gguf_q2_k",
                  "gguf_q3_k", "gguf_q4_k", "gguf_q5_k", "gguf_q6_k", "gguf_q8_0", "gguf_mxfp4")
 ATTENTION_BACKENDS = ("snapmla", "turboquant_mla", "csa_hca", "csa_hca_tq", "csa_hca_tq_mix")

@@ -8,12 +8,16 @@
 //   s_ij = scale q_i . k_j - slope_h (i - j) + bias_h[i - j],  0 <= i - j < window (window 0: the whole prefix), i and j in one chunk;
 //   o_i = softmax_j(s_ij) v_j
 //   out = o * sigmoid(gate)                                (gate offset < 0: none)
+//   a sink adds exp(sink_h) to the softmax's denominator; a temperature per head rides on the queries
+//   differential form: two maps per head over the same values, o = rms(o_1 - lambda o_2) (1 - diff) per head
 //
-// Cache row of a token: [G * dkp keys | G * dvp values], head widths padded with zeros to dkp / dvp.
-//   attn_prep      norms, value mixing, append to the cache;  attn_head_prep: biases, per-head norms, rotation, append
+// Cache row of a token: [G * dkp keys | G / maps * dvp values], head widths padded with zeros to dkp / dvp.  With several maps a "head" of the
+// attention kernels is one map of a query head; they are ordered [value head, map, head of the group].
+//   attn_prep      norms, value mixing, append to the cache;  attn_head_prep: biases, per-head norms, rotation, temperatures, append
 //   attn_decode    few rows: one block per (row, kv head, split of the visible keys); the heads of a group are the rows of mma.sync tiles, each
 //                  warp walks its own 16-key tiles; attn_combine merges the splits
 //   attn_prefill   runs of rows: 128 (token, head) rows of a sequence per block against 32-key tiles shared by eight warps
+//   attn_diff      difference of the two maps' results and its norm, merging the few-row form's splits
 //   attn_exact     fp32 cache and activations (and bf16 caches whose head widths the tensor-core kernels do not cover): CUDA cores
 // Scores, weights and the output sum are fp32; the tensor-core kernels split the weights into a bf16 (hi | lo) pair for the value product.
 #include "attn_core.cuh"
@@ -73,10 +77,13 @@ __global__ void __launch_bounds__(NT) attn_prep_kernel(const float* __restrict__
 }
 
 // One block per row, one warp per head: q and k = rot(norm(proj + bias)), v = proj + bias.  norm 0 none, 1 without a weight, 2 with wq / wk [dk].
+// Rotation of the leading `rot` channels: channel c with c + rot / 2, or (pairs) 2 i with 2 i + 1.  temp [H]: factor on a head's queries.  maps > 1: H
+// and G count maps, which the projection holds as [head, map]; queries are stored as [value head, map, head of the group].
 template <typename T, int NT>
 __global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restrict__ proj, int ldp, int off_q, int off_k, int off_v, const float* __restrict__ bq,
                                                              const float* __restrict__ bk, const float* __restrict__ bv, int norm, const float* __restrict__ wq,
-                                                             const float* __restrict__ wk, float eps, int rot, const double* __restrict__ inv_freq,
+                                                             const float* __restrict__ wk, float eps, int rot, int pairs, const double* __restrict__ inv_freq,
+                                                             const float* __restrict__ temp, int maps,
                                                              T* __restrict__ q_out, T* __restrict__ cache, const int* __restrict__ block_table, int max_pages,
                                                              const int* __restrict__ row_seq, const int* __restrict__ row_pos, int H, int G, int dk, int dv,
                                                              int dkp, int dvp, int page) {
@@ -89,8 +96,9 @@ __global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restr
     for (int i = threadIdx.x; i < half; i += NT) rotary_angle(pos, inv_freq[i], s_cs[half + i], s_cs[i]);
     __syncthreads();
     const float* pr = proj + (size_t)r * ldp;
-    T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * (dkp + dvp));
-    for (int j = warp; j < H + 2 * G; j += NT / 32) {
+    const int Gv = G / maps, hg = H / G;
+    T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * dkp + (size_t)Gv * dvp);
+    for (int j = warp; j < H + G + Gv; j += NT / 32) {
         if (j >= H + G) {
             const int g = j - H - G;
             for (int c = lane; c < dvp; c += 32)
@@ -111,16 +119,19 @@ __global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restr
             rs = 1.f / sqrtf(warp_sum(a) / (float)dk + eps);
         }
         auto at = [&](int c) { return (x[c] + (b ? b[c] : 0.f)) * rs * (norm == 2 ? w[c] : 1.f); };
-        T* d = isq ? q_out + ((size_t)r * H + h) * dkp : row + (size_t)h * dkp;
+        const int hq = h / maps, at_q = maps > 1 ? (hq / hg * maps + h % maps) * hg + hq % hg : h;
+        T* d = isq ? q_out + ((size_t)r * H + at_q) * dkp : row + (size_t)h * dkp;
+        const float f = isq && temp ? temp[hq] : 1.f;
 #pragma unroll 4
         for (int c = lane; c < dkp; c += 32) {
             float v = 0.f;
             if (c < dk) {
                 v = at(c);
-                if (c < half) v = v * s_cs[c] - at(c + half) * s_cs[half + c];
+                if (pairs) { if (c < rot) v = v * s_cs[c >> 1] + at(c ^ 1) * (c & 1 ? s_cs[half + (c >> 1)] : -s_cs[half + (c >> 1)]); }
+                else if (c < half) v = v * s_cs[c] - at(c + half) * s_cs[half + c];
                 else if (c < rot) v = v * s_cs[c - half] + at(c - half) * s_cs[c];
             }
-            d[c] = to_act<T>(v);
+            d[c] = to_act<T>(v * f);
         }
     }
 }
@@ -227,7 +238,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     const int lo = attn_low(p, pos);
     const int ntile = (pos - lo + 16) / 16;                       // 16-key tiles of the visible range
     const int per = (ntile + p.NS - 1) / p.NS, t0 = split * per, t1 = min(ntile, t0 + per);
-    const size_t ldc = (size_t)p.G * (p.dkp + p.dvp);
+    const size_t ldc = (size_t)p.ldc;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache);
     const int kc = p.dkp / 8, vc = DVP / 8;
     auto issue = [&](int tile, int buf) {
@@ -238,7 +249,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
             const int kr = lane >> 1, j = min(lo + tile * 16 + kr, pos);
             const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
             for (int c = lane & 1; c < kc; c += 2) cp16(dk_ + kr * ldk + c * 8, src + (size_t)g * p.dkp + c * 8);
-            for (int c = lane & 1; c < vc; c += 2) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.G * p.dkp + (size_t)g * p.dvp + c * 8);
+            for (int c = lane & 1; c < vc; c += 2) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)(g / p.maps) * p.dvp + c * 8);
         }
         cp_commit();
     };
@@ -297,7 +308,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
             }
         }
         if (p.NS == 1) {
-            O = O / L * attn_out_factor(p, r, h, c);
+            O *= attn_inv_sum(p, h, M, L);
+            if (p.out32) { p.out32[((size_t)r * p.H + h) * p.dvp + c] = O; continue; }
+            O *= attn_out_factor(p, r, h, c);
             reinterpret_cast<bf16*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = __float2bfloat16(O);
         } else {
             const size_t k = ((size_t)r * p.H + h) * p.NS + split;
@@ -317,12 +330,49 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(AttnParams p) {
     for (int s = 0; s < p.NS; ++s) M = fmaxf(M, p.ml_part[2 * (k0 + s)]);
     float L = 0.f;
     for (int s = 0; s < p.NS; ++s) L = fmaf(p.ml_part[2 * (k0 + s) + 1], ex2(p.ml_part[2 * (k0 + s)] - M), L);
+    const float inv = attn_inv_sum(p, h, M, L);
     for (int c = threadIdx.x; c < p.dv; c += 128) {
         float O = 0.f;
         for (int s = 0; s < p.NS; ++s) O = fmaf(p.o_part[(k0 + s) * p.dvp + c], ex2(p.ml_part[2 * (k0 + s)] - M), O);
-        O = O / L * attn_out_factor(p, r, h, c);
+        O = O * inv * attn_out_factor(p, r, h, c);
         reinterpret_cast<bf16*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = __float2bfloat16(O);
     }
+}
+
+// Differential heads: o_1 and o_2 of head h of a row (each the merge of NS split sums, or one normalised result: ml null) -> rms(o_1 - lambda o_2) factor.
+// One warp per (row, head); parts [rows, 2 H, NS, dvp] in the order [value head, map, head of the group].
+template <typename T>
+__global__ void __launch_bounds__(128) attn_diff_kernel(T* __restrict__ out, int ldo, const float* __restrict__ parts, const float* __restrict__ ml, int NS, int H, int hg,
+                                                        int dv, int dvp, float lambda, float eps, float factor, const int* __restrict__ row_seq) {
+    extern __shared__ float sdiff[];                               // [4][dv]
+    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y * 4 + warp;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (row_seq[r] < 0 || h >= H) return;
+    float* d = sdiff + warp * dv;
+    const size_t k[2] = {((size_t)r * 2 * H + h / hg * 2 * hg + h % hg) * NS, ((size_t)r * 2 * H + (h / hg * 2 + 1) * hg + h % hg) * NS};
+    float w[2];
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+        w[a] = 1.f;
+        if (ml) {
+            const float m = lane < NS ? ml[2 * (k[a] + lane)] : -INFINITY, l = lane < NS ? ml[2 * (k[a] + lane) + 1] : 0.f;
+            const float M = warp_max(m), e = m == -INFINITY ? 0.f : ex2(m - M);
+            w[a] = e / warp_sum(e * l);
+        }
+    }
+    w[1] *= -lambda;
+    float ss = 0.f;
+    for (int c0 = 0; c0 < dv; c0 += 32) {
+        const int c = min(c0 + lane, dv - 1);
+        float v = 0.f;
+#pragma unroll 4
+        for (int s = 0; s < NS; ++s)
+            v = fmaf(__shfl_sync(0xffffffffu, w[0], s), parts[(k[0] + s) * dvp + c], fmaf(__shfl_sync(0xffffffffu, w[1], s), parts[(k[1] + s) * dvp + c], v));
+        if (c0 + lane < dv) { d[c] = v; ss = fmaf(v, v, ss); }
+    }
+    const float f = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
+    for (int c = lane; c < dv; c += 32) out[(size_t)r * ldo + (size_t)h * dv + c] = to_act<T>(d[c] * f);
 }
 
 // ------------------------------------------------------------------------------------------------ prefill
@@ -359,7 +409,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         *reinterpret_cast<uint4*>(sq + m * ldk + c * 8) = v;
     }
     const int pos_last = pos0 + n - 1;
-    const int lo = attn_low(p, pos0) / kPreKeys * kPreKeys;
+    const int lo = max(attn_low(p, pos0) / kPreKeys * kPreKeys, p.key_base);
     const int ntile = (pos_last - lo) / kPreKeys + 1;
     const size_t ldc = (size_t)p.ldc;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache);
@@ -368,10 +418,10 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         if (tile < ntile) {
             bf16* dk_ = skv + (size_t)(tile & 1) * kPreKeys * (ldk + ldv);
             bf16* dv_ = dk_ + kPreKeys * ldk;
-            const int kr = t / kTpk, j = min(lo + tile * kPreKeys + kr, pos_last);
+            const int kr = t / kTpk, j = min(lo + tile * kPreKeys + kr, pos_last) - p.key_base;
             const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
             for (int c = t % kTpk; c < kc; c += kTpk) cp16(dk_ + kr * ldk + c * 8, src + (c * 8 < p.dkh ? (size_t)g * p.dkh + c * 8 : (size_t)p.off_ks + c * 8 - p.dkh));
-            for (int c = t % kTpk; c < vc; c += kTpk) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)g * p.dvp + c * 8);
+            for (int c = t % kTpk; c < vc; c += kTpk) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)(g / p.maps) * p.dvp + c * 8);
             if constexpr (BIAS) {
                 const int ldb = attn_bias_ld(tq), d0 = pos0 - (lo + tile * kPreKeys) - (kPreKeys - 1);       // distance of column 0
                 float* sb = sbias + (tile & 1) * hg * ldb;
@@ -426,7 +476,14 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
         const int tok = mr[row] / hg, h = g * hg + mr[row] % hg;
         if (tok >= n) continue;
         const size_t rr = (size_t)(r0 + tok);
-        const float inv = (p.off_gate >= 0 && p.head_gate ? gate_sigmoid(p.proj[rr * p.ldp + p.off_gate + h]) : 1.f) * p.out_scale / l[row];
+        const float norm = attn_inv_sum(p, h, m[row], l[row]);
+        if (p.out32) {
+            float* d = p.out32 + (rr * p.H + h) * p.dvp + (lane & 3) * 2;
+#pragma unroll
+            for (int i = 0; i < NV; ++i) *reinterpret_cast<float2*>(d + i * 8) = make_float2(o[i][2 * row] * norm, o[i][2 * row + 1] * norm);
+            continue;
+        }
+        const float inv = (p.off_gate >= 0 && p.head_gate ? gate_sigmoid(p.proj[rr * p.ldp + p.off_gate + h]) : 1.f) * p.out_scale * norm;
         bf16* d = reinterpret_cast<bf16*>(p.out) + rr * p.ldo + (size_t)h * p.dv;
         const float* gt = p.proj + rr * p.ldp + p.off_gate + (size_t)h * p.dv;
 #pragma unroll
@@ -458,7 +515,7 @@ static int launch_decode(const AttnParams& p, cudaStream_t st) {
     const dim3 grid(p.rows * p.G, p.NS, (p.H / p.G + 15) / 16);
     if (p.bias) launch_pdl((attn_decode_kernel<DVP, 1>), grid, 128, smem, st, p);
     else launch_pdl((attn_decode_kernel<DVP, 0>), grid, 128, smem, st, p);
-    if (p.NS > 1) launch_pdl((attn_combine_kernel), dim3(p.rows, p.H), 128, 0, st, p);
+    if (p.NS > 1 && p.maps == 1) launch_pdl((attn_combine_kernel), dim3(p.rows, p.H), 128, 0, st, p);
     return (int)cudaGetLastError();
 }
 template <int DVP>
@@ -477,9 +534,14 @@ static int launch_prefill(const AttnParams& p, const int* row0, const int* nrows
     return (int)cudaGetLastError();
 }
 
+static bool tensor_form(int dkp, int dvp, int f32) { return !f32 && dkp <= 256 && dvp <= 256; }
+static bool few_row_form(int run_rows, int H, int G, int dkp, int dvp, int f32) { return tensor_form(dkp, dvp, f32) && (run_rows < 8 || H / G > 128); }
+
 }  // namespace lsb
 using namespace lsb;
 
+// Split sums per (row, head) that lsb_attn leaves to lsb_attn_diff in a step with runs of up to run_rows rows (1: normalised results).
+LSB_API int lsb_attn_partials(int run_rows, int H, int G, int dkp, int dvp, int NS, int f32) { return few_row_form(run_rows, H, G, dkp, dvp, f32) ? NS : 1; }
 // padded head width of the cache and of the query buffer
 LSB_API int lsb_attn_head_pad(int d) { return d <= 32 ? 32 : (d <= 64 ? 64 : (d <= 128 ? 128 : (d + 127) / 128 * 128)); }
 
@@ -498,19 +560,19 @@ LSB_API int lsb_attn_prep(const void* proj, int ldp, int off_q, int off_k, int o
     LSB_CHECK_LAUNCH();
 }
 
-// Biases (null: none), per-head norms (norm 0 none, 1 plain, 2 with wq / wk [dk]), rotation of the leading `rot` channels (inv_freq: fp64 [rot / 2]) and
-// the cache append of every row.
+// Biases (null: none), per-head norms (norm 0 none, 1 plain, 2 with wq / wk [dk]), rotation of the leading `rot` channels (inv_freq: fp64 [rot / 2]; pairs:
+// adjacent channels, else halves), a factor per query head (temp, null: none) and the cache append of every row.  maps: see attn_head_prep_kernel.
 LSB_API int lsb_attn_head_prep(const void* proj, int ldp, int off_q, int off_k, int off_v, const void* bias_q, const void* bias_k, const void* bias_v, int norm,
-                               const void* wq, const void* wk, float eps, int rot, const void* inv_freq, void* q_out, void* cache, const void* block_table,
+                               const void* wq, const void* wk, float eps, int rot, int pairs, const void* inv_freq, const void* temp, int maps, void* q_out, void* cache, const void* block_table,
                                int max_pages, const void* row_seq, const void* row_pos, int rows, int H, int G, int dk, int dv, int dkp, int dvp, int page,
                                int f32, void* stream) {
     if (rows < 1 || H % G || dkp < dk || dvp < dv || dkp % 16 || dvp % 16 || rot < 0 || rot % 2 || rot > dk || (rot && !inv_freq) || norm < 0 || norm > 2 ||
-        (norm == 2 && (!wq || !wk)) || rot > 8192)
+        (norm == 2 && (!wq || !wk)) || rot > 8192 || maps < 1 || G % maps)
         return -1;
     cudaStream_t st = (cudaStream_t)stream;
     const bool wide = rows <= 64 && H + 2 * G >= 12;
 #define LSB_PREP(T, N) launch_pdl((attn_head_prep_kernel<T, N>), rows, N, (size_t)rot * 4, st, (const float*)proj, ldp, off_q, off_k, off_v, (const float*)bias_q, \
-                               (const float*)bias_k, (const float*)bias_v, norm, (const float*)wq, (const float*)wk, eps, rot, (const double*)inv_freq, (T*)q_out, \
+                               (const float*)bias_k, (const float*)bias_v, norm, (const float*)wq, (const float*)wk, eps, rot, pairs, (const double*)inv_freq, (const float*)temp, maps, (T*)q_out, \
                                (T*)cache, (const int*)block_table, max_pages, (const int*)row_seq, (const int*)row_pos, H, G, dk, dv, dkp, dvp, page)
     if (f32) LSB_PREP(float, 256); else if (wide) LSB_PREP(bf16, 1024); else LSB_PREP(bf16, 256);
 #undef LSB_PREP
@@ -520,21 +582,26 @@ LSB_API int lsb_attn_head_prep(const void* proj, int ldp, int off_q, int off_k, 
 // Attention of the step's rows.  run_rows: the largest number of rows a sequence has in this step (host knowledge; it selects the kernel form).
 // NS: key splits of the few-row form (o_part / ml_part sized for it).  off_gate < 0: no output gate; head_gate: one gate per head.  slope null: no linear
 // distance bias; bias [H, bias_len] (null: none): learned distance bias, not together with slopes.  chunk: size of the mask's chunks (0: none).
+// sink [H] (null: none).  maps > 1 (H and G count maps): the results stay in o_part for lsb_attn_diff, as split sums (NS > 1 and the few-row form) or
+// normalised ([rows, H, dvp]).
 LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
                      const void* seq_row0, const void* seq_nrows, int nseq, int run_rows, const void* proj, int ldp, int off_gate, void* out, int ldo,
                      void* o_part, void* ml_part, int NS, int rows, int H, int G, int dk, int dv, int dkp, int dvp, int window, float scale,
-                     const void* slope, int head_gate, int chunk, const void* bias, int bias_len, float out_scale, int f32, void* stream) {
-    if (rows < 1 || H % G || dkp % 16 || dvp % 16 || NS < 1 || (NS > 1 && (!o_part || !ml_part)) || chunk < 0 || (bias && (slope || bias_len < 1))) return -1;
+                     const void* slope, int head_gate, int chunk, const void* bias, int bias_len, float out_scale, const void* sink, int maps, int f32,
+                     void* stream) {
+    if (rows < 1 || H % G || dkp % 16 || dvp % 16 || NS < 1 || (NS > 1 && (!o_part || !ml_part)) || chunk < 0 || (bias && (slope || bias_len < 1)) ||
+        maps < 1 || G % maps || (maps > 1 && (!o_part || sink)))
+        return -1;
     AttnParams p;
     p.chunk = chunk; p.bias = (const float*)bias; p.bias_len = bias_len; p.out_scale = out_scale;
     p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
     p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = head_gate; p.out = out; p.ldo = ldo;
     p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.rows = rows; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = dkp; p.dvp = dvp;
-    p.ldc = G * (dkp + dvp); p.off_v = G * dkp; p.dkh = dkp; p.off_ks = 0; p.NS = NS; p.window = window; p.scale = scale; p.slope = (const float*)slope;
+    p.maps = maps; p.sink = (const float*)sink; p.out32 = maps > 1 ? (float*)o_part : nullptr;
+    p.ldc = G * dkp + G / maps * dvp; p.off_v = G * dkp; p.dkh = dkp; p.off_ks = 0; p.NS = NS; p.window = window; p.scale = scale; p.slope = (const float*)slope;
     cudaStream_t st = (cudaStream_t)stream;
-    const int hg = H / G;
-    const bool tc = !f32 && dkp <= 256 && dvp <= 256;
-    const bool prefill = tc && run_rows >= 8 && hg <= 128;
+    const bool tc = tensor_form(dkp, dvp, f32);
+    const bool prefill = tc && !few_row_form(run_rows, H, G, dkp, dvp, f32);
     if (!tc) {
         const size_t smem = (size_t)(dkp + 256 + dv) * 4;
         if (smem > 48 * 1024) return -1;
@@ -551,18 +618,31 @@ LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, 
     return -1;
 }
 
-// Attention of one run of rows (positions row_pos, causal) over keys and values written out per head and position: kv [positions, H dkh keys | H dvp values |
+// Differential heads from what lsb_attn (maps = 2) left in parts: H query heads in groups of hg, out [rows, ldo] heads side by side.  NS: split sums per map
+// (with ml) or 1 (ml null: normalised results).
+LSB_API int lsb_attn_diff(void* out, int ldo, const void* parts, const void* ml, int NS, int rows, int H, int hg, int dv, int dvp, float lambda, float eps, float factor,
+                          const void* row_seq, int f32, void* stream) {
+    if (rows < 1 || H < 1 || hg < 1 || H % hg || NS < 1 || NS > 32 || (NS > 1 && !ml) || dv < 1 || dv > dvp || dv > 3000) return -1;
+    const dim3 grid(rows, (H + 3) / 4);
+#define LSB_AD(T) launch_pdl((attn_diff_kernel<T>), grid, 128, (size_t)16 * dv, (cudaStream_t)stream, (T*)out, ldo, (const float*)parts, (const float*)(NS > 1 ? ml : nullptr), NS, \
+                             H, hg, dv, dvp, lambda, eps, factor, (const int*)row_seq)
+    if (f32) LSB_AD(float); else LSB_AD(bf16);
+#undef LSB_AD
+    LSB_CHECK_LAUNCH();
+}
+
+// Attention of one run of rows (positions row_pos, causal, sliding window or 0) over keys and values written out per head and position: kv [positions, H dkh keys | H dvp values |
 // dks key channels shared by all heads].  q: [rows, H, dkh + dks].  seq_row0 / seq_nrows: the run, as the other kernels take it; page0: a zero (the rows
-// are one page); off_gate: one gate per head (-1: none).
+// are one page; the first is position key_base); off_gate: one gate per head (head_gate) or value channel (-1: none).
 LSB_API int lsb_attn_run(const void* q, const void* kv, int positions, const void* page0, const void* row_seq, const void* row_pos, const void* seq_row0,
-                         const void* seq_nrows, const void* proj, int ldp, int off_gate, void* out, int ldo, int rows, int H, int dkh, int dks, int dv, int dvp,
-                         float scale, void* stream) {
-    if (rows < 1 || dkh % 16 || dks % 16 || dkh + dks > 256 || dv > dvp) return -1;
+                         const void* seq_nrows, const void* proj, int ldp, int off_gate, int head_gate, void* out, int ldo, int rows, int H, int dkh, int dks, int dv,
+                         int dvp, int window, int key_base, float scale, void* stream) {
+    if (key_base < 0 || rows < 1 || dkh % 16 || dks % 16 || dkh + dks > 256 || dv > dvp) return -1;
     AttnParams p;
     p.q = q; p.cache = kv; p.block_table = (const int*)page0; p.max_pages = 0; p.page = positions; p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos;
-    p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.out = out; p.ldo = ldo; p.o_part = p.ml_part = nullptr; p.rows = rows;
-    p.H = p.G = H; p.dk = p.dkp = dkh + dks; p.dv = dv; p.dvp = dvp; p.dkh = dkh; p.off_ks = H * (dkh + dvp); p.ldc = H * (dkh + dvp) + dks; p.off_v = H * dkh;
-    p.NS = 1; p.window = 0; p.scale = scale; p.slope = nullptr;
+    p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = head_gate; p.out = out; p.ldo = ldo; p.o_part = p.ml_part = nullptr; p.rows = rows;
+    p.key_base = key_base; p.H = p.G = H; p.dk = p.dkp = dkh + dks; p.dv = dv; p.dvp = dvp; p.dkh = dkh; p.off_ks = H * (dkh + dvp); p.ldc = H * (dkh + dvp) + dks; p.off_v = H * dkh;
+    p.NS = 1; p.window = window; p.scale = scale; p.slope = nullptr;
     switch (dvp) {
         case 32: return launch_prefill<32>(p, (const int*)seq_row0, (const int*)seq_nrows, 1, (cudaStream_t)stream);
         case 64: return launch_prefill<64>(p, (const int*)seq_row0, (const int*)seq_nrows, 1, (cudaStream_t)stream);

@@ -21,6 +21,10 @@ struct AttnParams {
     const float* bias = nullptr;      // [H, bias_len] added to the scores by distance, the last entry for all further ones; or null
     int bias_len = 0;
     float out_scale = 1.f;            // on the heads' outputs
+    int maps = 1;                     // consecutive groups that attend over one value head (G / maps value heads)
+    const float* sink = nullptr;      // [H] a term exp(sink) that only the softmax's denominator has, or null
+    float* out32 = nullptr;           // [rows, H, dvp] fp32 results in place of `out`, without gate and factor
+    int key_base = 0;                 // position of the cache's first row (caches that are one page)
 };
 
 // first key that position `pos` sees
@@ -38,6 +42,13 @@ __device__ __forceinline__ float gate_sigmoid(float x) { return 1.f / (1.f + exp
 // factor on value channel c of head h: output gate (if any) and constant
 __device__ __forceinline__ float attn_out_factor(const AttnParams& p, size_t r, int h, int c) {
     return p.off_gate >= 0 ? p.out_scale * gate_sigmoid(p.proj[r * p.ldp + p.off_gate + (p.head_gate ? (size_t)h : (size_t)h * p.dv + c)]) : p.out_scale;
+}
+
+// 1 / denominator, relative to the running maximum m (log2 units; never -inf) of head h's scores with sum l
+__device__ __forceinline__ float attn_inv_sum(const AttnParams& p, int h, float m, float l) {
+    if (!p.sink) return 1.f / l;
+    const float s = p.sink[h] * 1.4426950408889634f, M = fmaxf(m, s), f = exp2f(m - M);
+    return f / fmaf(l, f, exp2f(s - M));
 }
 
 // cosine and sine of pos * freq; the angle is reduced in fp64 so that far positions keep their phase
@@ -95,12 +106,14 @@ static __global__ void __launch_bounds__(128) attn_exact_kernel(AttnParams p) {
         const int n = min(128, pos - k0 + 1);
         for (int c = t; c < p.dv; c += 128) {
             float a = s_o[c] * corr;
-            for (int i = 0; i < n; ++i) a = fmaf(s_p[i], act_f(cache[(size_t)s_row[i] * ldc + (size_t)p.off_v + (size_t)g * p.dvp + c]), a);
+            for (int i = 0; i < n; ++i) a = fmaf(s_p[i], act_f(cache[(size_t)s_row[i] * ldc + (size_t)p.off_v + (size_t)(g / p.maps) * p.dvp + c]), a);
             s_o[c] = a;
         }
     }
+    const float inv = attn_inv_sum(p, h, m * 1.4426950408889634f, l);
     for (int c = t; c < p.dv; c += 128) {
-        const float o = s_o[c] / l * attn_out_factor(p, r, h, c);
+        if (p.out32) { p.out32[((size_t)r * p.H + h) * p.dvp + c] = s_o[c] * inv; continue; }
+        const float o = s_o[c] * inv * attn_out_factor(p, r, h, c);
         reinterpret_cast<T*>(p.out)[(size_t)r * p.ldo + (size_t)h * p.dv + c] = to_act<T>(o);
     }
 }

@@ -1,10 +1,11 @@
 // Latent attention over the paged cache, absorbed form, for models described layer by layer: one cached row [latent | rotated key part] per
-// token serves every head, whole causal prefix, fp32 scores and weights, per-head output gate.  All sizes are run-time parameters.
+// token serves every head, whole causal prefix or a sliding window, fp32 scores and weights, an output gate per head or per value channel.  All sizes
+// are run-time parameters; the rotated part may be missing.
 //
 //   c = RMSNorm(y[:dl]),  k_r = rot(y[dl:])                     y: the layer's latent projection (none: another layer's rows are read)
 //   q'_h = [ W_uk,h^T q_h | rot(q_r,h) ]                        the unrotated query moved into the latent space
 //   s_ij = scale q'_i . [c_j | k_r,j],  o_i = sum_j softmax_j(s_ij) c_j
-//   out_h = W_uv,h (sigmoid(g_h) o_h)
+//   out_h = W_uv,h (sigmoid(g_h) o_h), or sigmoid(g_h) * (W_uv,h o_h) with a gate per value channel
 //
 // Rotary pairs are adjacent channels.  Cache row of a token: [dlp latent | drp rotated], widths padded with zeros to multiples of 16.
 //   latent_query    few rows (and fp32): rotation, absorption and the cache append in one launch
@@ -29,7 +30,8 @@ namespace lsb {
 namespace cg = cooperative_groups;
 
 struct LatentPrep {
-    const float* proj; int ldp, off_q, off_kv;        // off_kv < 0: the layer has no latent projection of its own
+    const float* qsrc; int ldq;                       // queries, from their first column on
+    const float* proj; int ldp, off_kv;               // off_kv < 0: the layer has no latent projection of its own
     const float* kv_norm; float eps;
     const double* inv_freq;                           // [dr / 2]
     const void* w_uk;                                 // [H, dlp, dnp]
@@ -125,17 +127,17 @@ __global__ void __launch_bounds__(256) latent_query_kernel(LatentPrep p) {
     pdl_wait();
     pdl_launch_dependents();
     T* q = reinterpret_cast<T*>(p.q) + ((size_t)r0 * p.H + h) * D;
-    const float* src = p.proj + (size_t)r0 * p.ldp + p.off_q + (size_t)h * (p.dn + p.dr);
+    const float* src = p.qsrc + (size_t)r0 * p.ldq + (size_t)h * (p.dn + p.dr);
     if (blockIdx.x == gridDim.x - 1) {                        // rotations of this head; row m's append falls to head m
         for (int m = 0; m < nr; ++m)
-            rotated_tail(q + (size_t)m * p.H * D + p.dlp, src + (size_t)m * p.ldp + p.dn, p.dr, p.drp, p.row_pos[r0 + m], p.inv_freq, t, 256);
+            rotated_tail(q + (size_t)m * p.H * D + p.dlp, src + (size_t)m * p.ldq + p.dn, p.dr, p.drp, p.row_pos[r0 + m], p.inv_freq, t, 256);
         if (p.off_kv >= 0)
             for (int m = h; m < nr; m += p.H) append_row<T>(p, r0 + m, red);
         return;
     }
     for (int i = t; i < MT * p.dnp; i += 256) {
         const int m = i / p.dnp, c = i - m * p.dnp;
-        lsm[i] = m < nr && c < p.dn ? src[(size_t)m * p.ldp + c] : 0.f;
+        lsm[i] = m < nr && c < p.dn ? src[(size_t)m * p.ldq + c] : 0.f;
     }
     __syncthreads();
     small_products<T, MT>(reinterpret_cast<const T*>(p.w_uk) + (size_t)h * p.dlp * p.dnp, p.dnp, n0, n1, lsm, p.dnp, [&](int n, const float (&a)[MT]) {
@@ -147,6 +149,7 @@ __global__ void __launch_bounds__(256) latent_query_kernel(LatentPrep p) {
 
 // Rotated parts of all heads of a row (dst: rows of ld, src: rows of dn + dr); a thread keeps its rotary pair over the heads: one angle per pair.
 __device__ __forceinline__ void rotated_heads(bf16* dst, int ld, const float* src, const LatentPrep& p, int pos, int hp) {
+    if (hp == 0) return;
     const int t = threadIdx.x, w = min(hp, 256), step = 256 / w, h0 = t / w;
     for (int i = h0 < step ? t % w : hp; i < hp; i += w) {
         float cs = 1.f, sn = 0.f;
@@ -165,9 +168,9 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrep p) {
     pdl_wait();
     pdl_launch_dependents();
     const int pos = p.row_pos[r];
-    const float* src = p.proj + (size_t)r * p.ldp + p.off_q;
+    const float* src = p.qsrc + (size_t)r * p.ldq;
     bf16* qn = p.q_nope + (size_t)r * p.H * p.dnp;
-    if (p.dn == p.dnp && ((p.dn + p.dr) | p.off_q | p.ldp) % 4 == 0) {
+    if (p.dn == p.dnp && ((p.dn + p.dr) | p.ldq) % 4 == 0 && (reinterpret_cast<uintptr_t>(p.qsrc) & 15) == 0) {
         const int n4 = p.dn / 4;
         for (int i = t; i < p.H * n4; i += 256) {
             const int h = i / n4, c = (i - h * n4) * 4;
@@ -193,7 +196,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(LatentPrep p, int dnw)
     pdl_wait();
     pdl_launch_dependents();
     const int pos = p.row_pos[r];
-    const float* src = p.proj + (size_t)r * p.ldp + p.off_q;
+    const float* src = p.qsrc + (size_t)r * p.ldq;
     bf16* q = reinterpret_cast<bf16*>(p.q) + (size_t)r * p.H * K;
     for (int i = t; i < p.H * (dnw / 2); i += 256) {
         const int h = i / (dnw / 2), c = (i - h * (dnw / 2)) * 2;
@@ -204,19 +207,19 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(LatentPrep p, int dnw)
     if (p.off_kv >= 0) append_row<bf16>(p, r, red);
 }
 
-// Cached rows of positions [0, T) of one sequence: the latents to lat [T, dlp], the rotated part to column off_rot of kv's rows.  One warp per position.
+// Cached rows of positions [base, T) of one sequence: the latents to lat [T - base, dlp], the rotated part to column off_rot of kv's rows.  One warp per position.
 __global__ void __launch_bounds__(128) latent_gather_kernel(const bf16* __restrict__ cache, const int* __restrict__ block_table, int max_pages, int page,
-                                                            const int* __restrict__ row_seq, int T, int dlp, int drp, bf16* __restrict__ lat,
+                                                            const int* __restrict__ row_seq, int base, int T, int dlp, int drp, bf16* __restrict__ lat,
                                                             bf16* __restrict__ kv, int ldkv, int off_rot) {
-    const int j = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int j = base + blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     pdl_wait();
     pdl_launch_dependents();
     const int seq = row_seq[0];
     if (seq < 0 || j >= T) return;
     const uint4* src = reinterpret_cast<const uint4*>(cache + ((size_t)block_table[(size_t)seq * max_pages + j / page] * page + j % page) * (dlp + drp));
     for (int i = lane; i < (dlp + drp) / 8; i += 32) {
-        if (i < dlp / 8) reinterpret_cast<uint4*>(lat + (size_t)j * dlp)[i] = src[i];
-        else reinterpret_cast<uint4*>(kv + (size_t)j * ldkv + off_rot)[i - dlp / 8] = src[i];
+        if (i < dlp / 8) reinterpret_cast<uint4*>(lat + (size_t)(j - base) * dlp)[i] = src[i];
+        else reinterpret_cast<uint4*>(kv + (size_t)(j - base) * ldkv + off_rot)[i - dlp / 8] = src[i];
     }
 }
 
@@ -228,7 +231,7 @@ struct LatentAttn {
     const float* proj; int ldp, off_gate;
     bf16* out;                        // [rows, H, dlp]
     float* o_part; float* ml_part;    // [rows, H, NS / C, dlp], [rows, H, NS / C, 2]
-    int H, dlp, drp, NS, C;           // key splits, and how many of them form a cluster
+    int H, dlp, drp, window, NS, C;   // sliding window (0: none), key splits, and how many of them form a cluster
     float scale2;                     // log2 units
 };
 
@@ -285,7 +288,8 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
         if (m < nf) cp16(sq + m * ld + c * 8, p.q + ((size_t)row0 * p.H + f0 + m) * D + c * 8);
         else *reinterpret_cast<uint4*>(sq + m * ld + c * 8) = make_uint4(0, 0, 0, 0);
     }
-    const int ntile = pos_last / KT + 1, per = (ntile + p.NS - 1) / p.NS, t0 = (int)blockIdx.y * per, t1 = min(ntile, t0 + per);
+    auto low = [&](int pos) { return p.window > 0 ? max(0, pos - p.window + 1) : 0; };          // first key that a position sees
+    const int first = low(pos_first) / KT, end = pos_last / KT + 1, per = (end - first + p.NS - 1) / p.NS, t0 = first + (int)blockIdx.y * per, t1 = min(end, t0 + per);
     constexpr int TPK = 256 / KT;                                 // threads per key of a tile copy
     const int kr = t / TPK;
     const int* bt = p.block_table + (size_t)seq * p.max_pages;
@@ -304,11 +308,12 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
         cp_commit();
     };
     const int mi = warp % MG, ki = warp / MG;
-    int pr[2];
+    int pr[2], lo[2];
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
         const int m = mi * 16 + (lane >> 2) + 8 * u;
         pr[u] = m < nf ? pos0 + (f0 + m) / p.H : -1;              // -1: an idle row sees nothing
+        lo[u] = low(pr[u]);
     }
     float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[MG][NV][4];
 #pragma unroll
@@ -351,13 +356,14 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
         for (; k + 32 <= D; k += 32) { step(k, s[0]); step(k + 16, s[1]); }
         if (k < D) step(k, s[0]);
         float mt[2] = {-INFINITY, -INFINITY};
-        const bool full = kt * KT + KT - 1 <= pos_first && nf == BM;
+        const bool full = kt * KT + KT - 1 <= pos_first && nf == BM && kt * KT >= low(pos_last);
 #pragma unroll
         for (int i = 0; i < NT; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float v = (s[0][i][j] + s[1][i][j]) * p.scale2;
-                s[0][i][j] = full || kt * KT + ki * C::KW + i * 8 + (lane & 3) * 2 + (j & 1) <= pr[j >> 1] ? v : -INFINITY;
+                const int key = kt * KT + ki * C::KW + i * 8 + (lane & 3) * 2 + (j & 1);
+                s[0][i][j] = full || (key <= pr[j >> 1] && key >= lo[j >> 1]) ? v : -INFINITY;
                 mt[j >> 1] = fmaxf(mt[j >> 1], s[0][i][j]);
             }
 #pragma unroll
@@ -534,7 +540,7 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
 struct LatentOut {
     const void* o_lat;                // [rows, H, dlp], gated (NS == 1)
     const float* o_part; const float* ml_part; int NS;
-    const float* proj; int ldp, off_gate;
+    const float* proj; int ldp, off_gate, head_gate;      // gate per head (of the latent sums) or per value channel (of the result)
     const int* row_seq;
     int rows, H, dlp, dv;
 };
@@ -545,7 +551,7 @@ __device__ __forceinline__ void split_weights(const LatentOut& p, int r, int h, 
     const float m = lane < p.NS ? ml[2 * lane] : -INFINITY, l = lane < p.NS ? ml[2 * lane + 1] : 0.f;
     const float M = warp_max(m), e = m == -INFINITY ? 0.f : ex2(m - M);
     float f = 1.f / warp_sum(e * l);
-    if (p.off_gate >= 0) f *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + h]);
+    if (p.off_gate >= 0 && p.head_gate) f *= gate_sigmoid(p.proj[(size_t)r * p.ldp + p.off_gate + h]);
     w[lane] = e * f;
 }
 __device__ __forceinline__ float4 merged4(const LatentOut& p, int r, int h, int c, const float* w) {
@@ -603,8 +609,19 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentOut p, const T* _
     small_products<T, MT>(w_uv + (size_t)h * p.dv * p.dlp, p.dlp, n0, n1, lsm, p.dlp, [&](int n, const float (&a)[MT]) {
 #pragma unroll
         for (int m = 0; m < MT; ++m)
-            if (m < nr) out[(size_t)(r0 + m) * ldo + (size_t)h * p.dv + n] = to_act<T>(a[m]);
+            if (m < nr) {
+                const float g = p.off_gate >= 0 && !p.head_gate ? gate_sigmoid(p.proj[(size_t)(r0 + m) * p.ldp + p.off_gate + (size_t)h * p.dv + n]) : 1.f;
+                out[(size_t)(r0 + m) * ldo + (size_t)h * p.dv + n] = to_act<T>(a[m] * g);
+            }
     });
+}
+
+// x [rows, ldo] *= sigmoid(gate), column by column (the many-row form's gate per value channel)
+__global__ void __launch_bounds__(256) gate_rows_kernel(bf16* __restrict__ x, int ldo, const float* __restrict__ gate, int ldg, int n) {
+    const int r = blockIdx.y, i = blockIdx.x * 256 + threadIdx.x;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (i < n) x[(size_t)r * ldo + i] = __float2bfloat16(__bfloat162float(x[(size_t)r * ldo + i]) * gate_sigmoid(gate[(size_t)r * ldg + i]));
 }
 
 template <int NV, int MG>
@@ -632,11 +649,11 @@ static int launch_latent_rows(const LatentAttn& p, int mg, int tiles, cudaStream
     return mg == 1 ? launch_latent<NV, 1>(p, tiles, st) : (mg == 2 ? launch_latent<NV, 2>(p, tiles, st) : launch_latent<NV, 4>(p, tiles, st));
 }
 static int row_tiles(int run_rows, int H) { return run_rows * H <= 16 ? 1 : (run_rows * H <= 32 ? 2 : 4); }
-static LatentPrep latent_prep_params(const void* proj, int ldp, int off_q, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_uk, void* q,
+static LatentPrep latent_prep_params(const void* qsrc, int ldq, const void* proj, int ldp, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_uk, void* q,
                                      void* q_nope, void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
                                      int rows, int H, int dn, int dnp, int dr, int dl) {
     LatentPrep p;
-    p.proj = (const float*)proj; p.ldp = ldp; p.off_q = off_q; p.off_kv = off_kv; p.kv_norm = (const float*)kv_norm; p.eps = eps;
+    p.qsrc = (const float*)qsrc; p.ldq = ldq; p.proj = (const float*)proj; p.ldp = ldp; p.off_kv = off_kv; p.kv_norm = (const float*)kv_norm; p.eps = eps;
     p.inv_freq = (const double*)inv_freq; p.w_uk = w_uk; p.q = q; p.q_nope = (bf16*)q_nope; p.cache = cache; p.block_table = (const int*)block_table;
     p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos; p.rows = rows; p.H = H; p.dn = dn;
     p.dnp = dnp; p.dr = dr; p.drp = (dr + 15) / 16 * 16; p.dl = dl; p.dlp = (dl + 15) / 16 * 16;
@@ -669,12 +686,12 @@ LSB_API int lsb_latent_splits(int rows, int H, int dl, int dr, int seen, int f32
 // Partial sums per (row, head) that NS splits leave to lsb_latent_out (1: none, the attention kernel writes its result): o_part [rows, H, this, dlp].
 LSB_API int lsb_latent_partials(int NS) { return NS / cluster_of(NS); }
 
-// Queries in the latent space and the cache append.  w_uk: [H, dlp, dnp] (dn padded to dnp % 8 == 0 with zeros).  off_kv < 0: nothing is appended.
-LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_uk,
+// Queries (rows of ldq from qsrc on, heads of dn unrotated and dr rotated channels) in the latent space and the cache append.  w_uk: [H, dlp, dnp] (dn padded to dnp % 8 == 0 with zeros).  off_kv < 0: nothing is appended.
+LSB_API int lsb_latent_query(const void* qsrc, int ldq, const void* proj, int ldp, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_uk,
                              void* q, void* q_nope, void* cache, const void* block_table, int max_pages, int page, const void* row_seq,
                              const void* row_pos, int rows, int H, int dn, int dnp, int dr, int dl, int f32, void* err, void* stream) {
-    if (rows < 1 || dnp % 8 || dnp < dn || dr % 2 || dr < 1 || dl < 1) return -1;
-    const LatentPrep p = latent_prep_params(proj, ldp, off_q, off_kv, kv_norm, eps, inv_freq, w_uk, q, q_nope, cache, block_table, max_pages, page, row_seq, row_pos,
+    if (rows < 1 || dnp % 8 || dnp < dn || dr % 2 || dr < 0 || dl < 1) return -1;
+    const LatentPrep p = latent_prep_params(qsrc, ldq, proj, ldp, off_kv, kv_norm, eps, inv_freq, w_uk, q, q_nope, cache, block_table, max_pages, page, row_seq, row_pos,
                                             rows, H, dn, dnp, dr, dl);
     cudaStream_t st = (cudaStream_t)stream;
     if (!f32 && rows >= 8) {
@@ -696,17 +713,18 @@ LSB_API int lsb_latent_query(const void* proj, int ldp, int off_q, int off_kv, c
 
 // A run of rows of one sequence (row_pos consecutive, T positions in all after the append) with keys and values written out per head: q [rows, H, dnw + drp];
 // kv [Tm, H dnw unrotated keys | H dvp values | drp shared rotated part], read by lsb_attn_run.  w_kv: [H dnw + H dvp, dlp], padding rows and columns zero;
-// lat: scratch [Tm, dlp].  Tm >= T: positions the product runs over (those past T are never read).
-LSB_API int lsb_latent_expand(const void* proj, int ldp, int off_q, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_kv,
+// lat: scratch [Tm, dlp].  base: the first position that any row sees, row 0 of lat and kv.  Tm >= T - base: rows the product runs over (those past
+// T - base are never read).
+LSB_API int lsb_latent_expand(const void* qsrc, int ldq, const void* proj, int ldp, int off_kv, const void* kv_norm, float eps, const void* inv_freq, const void* w_kv,
                               void* q, void* lat, void* kv, void* cache, const void* block_table, int max_pages, int page, const void* row_seq,
-                              const void* row_pos, int rows, int T, int Tm, int H, int dn, int dnw, int dr, int dl, int dvp, void* err, void* stream) {
-    if (rows < 1 || T < rows || Tm < T || dnw % 16 || dnw < dn || dvp % 16 || dr % 2 || dr < 1 || dl < 1) return -1;
-    const LatentPrep p = latent_prep_params(proj, ldp, off_q, off_kv, kv_norm, eps, inv_freq, nullptr, q, nullptr, cache, block_table, max_pages, page, row_seq, row_pos,
+                              const void* row_pos, int rows, int base, int T, int Tm, int H, int dn, int dnw, int dr, int dl, int dvp, void* err, void* stream) {
+    if (rows < 1 || base < 0 || T - base < rows || Tm < T - base || dnw % 16 || dnw < dn || dvp % 16 || dr % 2 || dr < 0 || dl < 1) return -1;
+    const LatentPrep p = latent_prep_params(qsrc, ldq, proj, ldp, off_kv, kv_norm, eps, inv_freq, nullptr, q, nullptr, cache, block_table, max_pages, page, row_seq, row_pos,
                                             rows, H, dn, dnw, dr, dl);
     cudaStream_t st = (cudaStream_t)stream;
     const int N = H * (dnw + dvp), ldkv = N + p.drp;
     launch_pdl((latent_rows_kernel), rows, 256, 0, st, p, dnw);
-    launch_pdl((latent_gather_kernel), (T + 3) / 4, 128, 0, st, (const bf16*)cache, (const int*)block_table, max_pages, page, (const int*)row_seq, T, p.dlp, p.drp,
+    launch_pdl((latent_gather_kernel), (T - base + 3) / 4, 128, 0, st, (const bf16*)cache, (const int*)block_table, max_pages, page, (const int*)row_seq, base, T, p.dlp, p.drp,
                (bf16*)lat, (bf16*)kv, ldkv, N);
     const int rc = lsb_gemm_bf16_tc(kv, lat, w_kv, nullptr, Tm, N, p.dlp, p.dlp, p.dlp, ldkv, 1, nullptr, 0, err, nullptr, stream);
     return rc ? rc : (int)cudaGetLastError();
@@ -714,10 +732,11 @@ LSB_API int lsb_latent_expand(const void* proj, int ldp, int off_q, int off_kv, 
 
 // Attention of the step's rows.  NS: key splits (lsb_latent_splits; runs of rows use 1).  One partial sum: o_lat [rows, H, dlp], gated; more: o_part /
 // ml_part, merged by lsb_latent_out.  seq_row0 / seq_nrows: the step's sequences (consecutive positions each); run_rows: the largest number of rows one of them has.
+// window: sliding window (0: none); off_gate: one gate per head (-1: none, or none before lsb_latent_out).
 LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_table, int max_pages, int page, const void* row_seq, const void* row_pos,
                             const void* seq_row0, const void* seq_nrows, int nseq, int run_rows, const void* proj, int ldp, int off_gate, void* o_lat,
-                            void* o_part, void* ml_part, int NS, int rows, int H, int dl, int dr, float scale, int f32, void* stream) {
-    if (rows < 1 || !splits_ok(NS) || (lsb_latent_partials(NS) > 1 && (!o_part || !ml_part)) || dl < 1 || dr < 1) return -1;
+                            void* o_part, void* ml_part, int NS, int rows, int H, int dl, int dr, int window, float scale, int f32, void* stream) {
+    if (rows < 1 || !splits_ok(NS) || (lsb_latent_partials(NS) > 1 && (!o_part || !ml_part)) || dl < 1 || dr < 0 || window < 0) return -1;
     const int dlp = lsb_latent_pad(dl), drp = lsb_latent_pad(dr), D = dlp + drp;
     cudaStream_t st = (cudaStream_t)stream;
     if (latent_tc(dlp, drp, f32)) {
@@ -725,7 +744,7 @@ LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_
         p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page;
         p.row_seq = (const int*)row_seq; p.row_pos = (const int*)row_pos; p.seq_row0 = (const int*)seq_row0; p.seq_nrows = (const int*)seq_nrows;
         p.nseq = nseq; p.run_rows = run_rows; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.out = (bf16*)o_lat;
-        p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.H = H; p.dlp = dlp; p.drp = drp; p.NS = NS; p.C = cluster_of(NS); p.scale2 = scale * kLog2e;
+        p.o_part = (float*)o_part; p.ml_part = (float*)ml_part; p.H = H; p.dlp = dlp; p.drp = drp; p.window = window; p.NS = NS; p.C = cluster_of(NS); p.scale2 = scale * kLog2e;
         const int mg = row_tiles(run_rows, H), bm = 16 * mg;
         const long long tiles = run_rows == 1 ? (long long)rows * ((H + bm - 1) / bm) : (long long)rows * H / bm + nseq;
         if (tiles > 0x7fffffff) return -1;
@@ -740,7 +759,7 @@ LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_
     p.q = q; p.cache = cache; p.block_table = (const int*)block_table; p.max_pages = max_pages; p.page = page; p.row_seq = (const int*)row_seq;
     p.row_pos = (const int*)row_pos; p.proj = (const float*)proj; p.ldp = ldp; p.off_gate = off_gate; p.head_gate = 1; p.ldc = p.dkh = D; p.off_v = p.off_ks = 0;
     p.out = o_lat; p.ldo = H * dlp; p.o_part = p.ml_part = nullptr; p.rows = rows; p.H = H; p.G = 1; p.dk = p.dkp = D; p.dv = p.dvp = dlp; p.NS = 1;
-    p.window = 0; p.scale = scale; p.slope = nullptr;
+    p.window = window; p.scale = scale; p.slope = nullptr;
     const size_t smem = (size_t)(D + 256 + dlp) * 4;
     if (smem > 48 * 1024) return -1;
     if (f32) launch_pdl((attn_exact_kernel<float>), dim3(rows, H), 128, smem, st, p);
@@ -749,18 +768,22 @@ LSB_API int lsb_latent_attn(const void* q, const void* cache, const void* block_
 }
 
 // Value up-projection: out [rows, ldo] = W_uv o_lat, heads side by side; NS (partial sums) > 1: o_lat is first made from them (and gated).
-// w_uv: [H, dv, dlp].
+// w_uv: [H, dv, dlp].  off_gate: one gate per head (head_gate; applied here when NS > 1 only, otherwise the attention kernel has done it) or per value
+// channel (of the result), -1: none.
 LSB_API int lsb_latent_out(void* out, int ldo, void* o_lat, const void* o_part, const void* ml_part, int NS, const void* w_uv, const void* proj, int ldp,
-                           int off_gate, const void* row_seq, int rows, int H, int dl, int dv, int f32, void* err, void* stream) {
+                           int off_gate, int head_gate, const void* row_seq, int rows, int H, int dl, int dv, int f32, void* err, void* stream) {
     if (rows < 1 || NS < 1 || NS > 32 || (NS > 1 && (!o_part || !ml_part || f32)) || dl < 1 || dv < 1) return -1;
     const int dlp = lsb_latent_pad(dl);
     cudaStream_t st = (cudaStream_t)stream;
-    LatentOut o{o_lat, (const float*)o_part, (const float*)ml_part, NS, (const float*)proj, ldp, off_gate, (const int*)row_seq, rows, H, dlp, dv};
+    LatentOut o{o_lat, (const float*)o_part, (const float*)ml_part, NS, (const float*)proj, ldp, off_gate, head_gate, (const int*)row_seq, rows, H, dlp, dv};
     if (!f32 && rows >= 8) {
         if (NS > 1) launch_pdl((latent_combine_kernel), dim3(rows, H), 128, 0, st, o, (bf16*)o_lat);
         if (dv % 8 == 0 && ldo % 8 == 0) {
             const int rc = lsb_gemm_bf16_tc_batched(out, o_lat, w_uv, rows, dv, dlp, H, H * dlp, dlp, dlp, (long long)dv * dlp, ldo, dv, 1, err, stream);
-            return rc ? rc : (int)cudaGetLastError();
+            if (rc) return rc;
+            if (off_gate >= 0 && !head_gate)
+                launch_pdl((gate_rows_kernel), dim3((H * dv + 255) / 256, rows), 256, 0, st, (bf16*)out, ldo, (const float*)proj + off_gate, ldp, H * dv);
+            return (int)cudaGetLastError();
         }
         o.NS = 1;
     }

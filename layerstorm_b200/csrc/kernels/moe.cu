@@ -552,14 +552,14 @@ __global__ void moe_combine_kernel(float* __restrict__ out, const float* __restr
     pdl_launch_dependents();
 }
 
-// Dense gated unit over a fused fp32 projection (gate columns at off_g, up columns at off_u of rows of ld) -> [rows, ldo] bf16 / fp32; columns F .. ldo
+// Dense gated unit over a fused fp32 projection (gate columns at off_g, up columns at off_u of rows of ld) -> [rows, ldo] bf16 / fp32; columns F .. width
 // are zeroed.  off_s >= 0: the row's result times sigmoid of the projection's column off_s.
 template <typename T>
-__global__ void glu_kernel(T* __restrict__ out, int ldo, const float* __restrict__ z, int ld, int off_g, int off_u, int off_s, int F, GluAct ga) {
+__global__ void glu_kernel(T* __restrict__ out, int ldo, int width, const float* __restrict__ z, int ld, int off_g, int off_u, int off_s, int F, GluAct ga) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.y, f = blockIdx.x * blockDim.x + threadIdx.x;
-    if (f >= ldo) return;
+    if (f >= width) return;
     const float* zr = z + (size_t)r * ld;
     float v = 0.f;
     if (f < F) {
@@ -770,19 +770,19 @@ LSB_API int lsb_moe_combine(void* out, const void* y, const void* wts, const voi
 }
 
 LSB_API int lsb_swiglu(void* out, const void* gu, int rows, int F, float limit, void* stream) {
-    launch_pdl((glu_kernel<bf16>), dim3((F + 255) / 256, rows), 256, 0, (cudaStream_t)stream, (bf16*)out, F, (const float*)gu, 2 * F, 0, F, -1, F,
+    launch_pdl((glu_kernel<bf16>), dim3((F + 255) / 256, rows), 256, 0, (cudaStream_t)stream, (bf16*)out, F, F, (const float*)gu, 2 * F, 0, F, -1, F,
                GluAct{limit, 1.f, 0.f, nullptr});
     LSB_CHECK_LAUNCH();
 }
 
 // Gated unit of any two column blocks of a projection: see glu_kernel.  f32: fp32 output.
-LSB_API int lsb_glu(void* out, int ldo, const void* z, int ld, int off_g, int off_u, int off_s, int rows, int F, float limit, float alpha, float shift, int f32,
+LSB_API int lsb_glu(void* out, int ldo, int width, const void* z, int ld, int off_g, int off_u, int off_s, int rows, int F, float limit, float alpha, float shift, int f32,
                     void* stream) {
-    if (rows < 1 || rows > 65535 || F < 1 || ldo < F) return -1;
-    const dim3 grid((ldo + 255) / 256, rows);
+    if (rows < 1 || rows > 65535 || F < 1 || width < F || ldo < width) return -1;
+    const dim3 grid((width + 255) / 256, rows);
     const GluAct ga{limit, alpha, shift, nullptr};
-    if (f32) launch_pdl((glu_kernel<float>), grid, 256, 0, (cudaStream_t)stream, (float*)out, ldo, (const float*)z, ld, off_g, off_u, off_s, F, ga);
-    else launch_pdl((glu_kernel<bf16>), grid, 256, 0, (cudaStream_t)stream, (bf16*)out, ldo, (const float*)z, ld, off_g, off_u, off_s, F, ga);
+    if (f32) launch_pdl((glu_kernel<float>), grid, 256, 0, (cudaStream_t)stream, (float*)out, ldo, width, (const float*)z, ld, off_g, off_u, off_s, F, ga);
+    else launch_pdl((glu_kernel<bf16>), grid, 256, 0, (cudaStream_t)stream, (bf16*)out, ldo, width, (const float*)z, ld, off_g, off_u, off_s, F, ga);
     LSB_CHECK_LAUNCH();
 }
 

@@ -784,11 +784,15 @@ __device__ __forceinline__ float sum_slots(float a, const MoeSum& mo, const floa
     return a;
 }
 
-// resid[r] += post(sub[r] + MoE sum of the row), x[r] = pre(the new residual) in the activation type.  sub may be null.  Whole rows per block.
-// PLAIN: post is an RMS or layer norm and there is no pre norm.
+// Causal convolution over time on the sublayer's input h = x[r], added to it: xc = h + sum_j w[j] h_(t - taps + 1 + j).  state: a sequence slot's last
+// taps - 1 inputs, oldest first.  (As part of the residual update: steps of one row per sequence.)
+struct InputConv { void* xc; const float* w; float* state; const int* slot; int taps, ldw; };      // w [taps, ldw], state [slots, taps - 1, ldw]
+
+// resid[r] += post(sub[r] + MoE sum of the row) (+ step), x[r] = pre(the new residual) in the activation type.  sub may be null.  Whole rows per block.
+// PLAIN: post is an RMS or layer norm and there is no pre norm, no step and no convolution.
 template <typename T, bool MOE, bool PLAIN>
 __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds,
-                                                        NormW post, NormW pre, MoeSum mo) {
+                                                        NormW post, NormW pre, MoeSum mo, const float* __restrict__ step, InputConv ic) {
     __shared__ float red[33], s_w[32];
     __shared__ int s_id[32];
     extern __shared__ float row[];
@@ -824,7 +828,7 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int 
     }
     const bool again = norm_moments_needed(pre.kind);
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        const float v = rr[i] + norm_apply(row[i], i, post, mean, rstd, a_post);
+        const float v = rr[i] + norm_apply(row[i], i, post, mean, rstd, a_post) + (step ? step[i] : 0.f);
         rr[i] = v;
         if (again) row[i] = v;
         else xr[i] = as_act<T>(norm_apply(v, i, pre, 0.f, 1.f, a_pre));
@@ -832,7 +836,75 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int 
     if (!again) return;
     __syncthreads();
     norm_moments(row, pre, red, mean, rstd);
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) xr[i] = as_act<T>(norm_apply(row[i], i, pre, mean, rstd, a_pre));
+    if (!ic.xc) {
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) xr[i] = as_act<T>(norm_apply(row[i], i, pre, mean, rstd, a_pre));
+        return;
+    }
+    const int slot = ic.slot[r], K = ic.taps - 1;
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+        const T h = as_act<T>(norm_apply(row[i], i, pre, mean, rstd, a_pre));
+        const float v = (float)h;
+        float a = v * ic.w[(size_t)K * ic.ldw + i];
+        if (slot >= 0) {
+            float* s = ic.state + (size_t)slot * K * ic.ldw + i;
+            for (int j = 0; j < K; ++j) {
+                a = fmaf(s[(size_t)j * ic.ldw], ic.w[(size_t)j * ic.ldw + i], a);
+                s[(size_t)j * ic.ldw] = j + 1 < K ? s[(size_t)(j + 1) * ic.ldw] : v;
+            }
+        }
+        xr[i] = h;
+        reinterpret_cast<T*>(ic.xc)[(size_t)r * ldx + i] = as_act<T>(v + a);
+    }
+}
+
+// The input convolution of runs of rows: xc = x + conv(x), and every sequence's state moves on.  A block takes kConvRows rows of one sequence and 4 columns
+// per thread; the first block of a sequence alone touches its state (the rows it needs beyond its own are read from x).
+constexpr int kConvRows = 16;
+template <typename T>
+__global__ void __launch_bounds__(128) input_conv_kernel(const T* __restrict__ x, int ldx, InputConv ic, const int* __restrict__ seq_row0, const int* __restrict__ seq_nrows,
+                                                         const int* __restrict__ seq_slot, int nseq, int dim) {
+    pdl_wait();
+    pdl_launch_dependents();
+    int tile = blockIdx.y, s = 0, n = 0;
+    for (; s < nseq; ++s) {
+        n = seq_nrows[s];
+        const int nt = (n + kConvRows - 1) / kConvRows;
+        if (tile < nt) break;
+        tile -= nt;
+    }
+    const int i = (blockIdx.x * 128 + threadIdx.x) * 4, K = ic.taps - 1;
+    if (s == nseq || i >= dim) return;
+    const T* xs = x + (size_t)seq_row0[s] * ldx + i;
+    T* out = reinterpret_cast<T*>(ic.xc) + (size_t)seq_row0[s] * ldx + i;
+    float* st = ic.state + (size_t)seq_slot[s] * K * ic.ldw + i;
+    const float* w = ic.w + i;
+    auto load = [&](int t) {                                       // input of row t of the run; t < 0: before the run
+        if (t < 0) return *reinterpret_cast<const float4*>(st + (size_t)(K + t) * ic.ldw);
+        if constexpr (sizeof(T) == 4) return *reinterpret_cast<const float4*>(xs + (size_t)t * ldx);
+        else {
+            const uint2 u = *reinterpret_cast<const uint2*>(xs + (size_t)t * ldx);
+            const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&u.y));
+            return make_float4(a.x, a.y, b.x, b.y);
+        }
+    };
+    const int r0 = tile * kConvRows, r1 = min(n, r0 + kConvRows);
+#pragma unroll 4
+    for (int r = r0; r < r1; ++r) {
+        const float4 h = load(r), wk = *reinterpret_cast<const float4*>(w + (size_t)K * ic.ldw);
+        float4 a = make_float4(h.x * wk.x, h.y * wk.y, h.z * wk.z, h.w * wk.w);
+        for (int j = 0; j < K; ++j) {
+            const float4 v = load(r - K + j), c = *reinterpret_cast<const float4*>(w + (size_t)j * ic.ldw);
+            a.x = fmaf(v.x, c.x, a.x); a.y = fmaf(v.y, c.y, a.y); a.z = fmaf(v.z, c.z, a.z); a.w = fmaf(v.w, c.w, a.w);
+        }
+        a.x += h.x; a.y += h.y; a.z += h.z; a.w += h.w;
+        T* o = out + (size_t)r * ldx;
+        if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(o) = a;
+        else { reinterpret_cast<bf162*>(o)[0] = __floats2bfloat162_rn(a.x, a.y); reinterpret_cast<bf162*>(o)[1] = __floats2bfloat162_rn(a.z, a.w); }
+    }
+    // the block that reads the old state is the one that replaces it; oldest first, so that entries are read before they are overwritten.  (Tiles behind the
+    // first reach back at most into rows of the run when it has at least K rows in front of them.)
+    if (tile == 0)
+        for (int j = 0; j < K; ++j) *reinterpret_cast<float4*>(st + (size_t)j * ic.ldw) = load(n - K + j);
 }
 
 // The same with element-wise norms on both sides: columns spread over blocks, four per thread, nothing exchanged.
@@ -890,12 +962,13 @@ __global__ void __launch_bounds__(1024) norm_rows_kernel(T* __restrict__ out, in
 static int norm_threads(int dim, int rows) { return dim >= 2048 ? (rows <= 64 ? 1024 : 512) : (dim >= 512 ? 256 : 128); }
 
 static int residual_update(void* x, int ldx, void* resid, int ldr, const void* sub, int lds, const NormW& post, const NormW& pre, const MoeSum& mo, int rows,
-                           int f32, cudaStream_t st) {
+                           const float* step, const InputConv& ic, int f32, cudaStream_t st) {
     const int dim = post.dim;
     if (dim < 1 || dim > 12000 || rows < 1 || (mo.y && mo.S > 32)) return -1;
     for (const NormW* n : {&post, &pre})
         if (n->kind < 0 || n->kind > kNormNone || (n->kind != kNormNone && !n->w) || (n->kind == kNormTanh && !n->alpha)) return -1;
-    if (!norm_moments_needed(post.kind) && !norm_moments_needed(pre.kind) && dim % 4 == 0 && ldx % 4 == 0 && ldr % 4 == 0 && lds % 4 == 0 && mo.ldy % 4 == 0 && rows < 65536) {
+    if (ic.xc && (!norm_moments_needed(pre.kind) || ic.taps < 1 || !ic.w || (ic.taps > 1 && !ic.state) || !ic.slot)) return -1;
+    if (!step && !norm_moments_needed(post.kind) && !norm_moments_needed(pre.kind) && dim % 4 == 0 && ldx % 4 == 0 && ldr % 4 == 0 && lds % 4 == 0 && mo.ldy % 4 == 0 && rows < 65536) {
         const dim3 grid((dim / 4 + 127) / 128, rows);
 #define LSB_PW(T, M) launch_pdl((post_norm_wide_kernel<T, M>), grid, 128, 0, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
         if (f32) { if (mo.y) LSB_PW(float, true); else LSB_PW(float, false); }
@@ -903,9 +976,9 @@ static int residual_update(void* x, int ldx, void* resid, int ldr, const void* s
 #undef LSB_PW
         LSB_CHECK_LAUNCH();
     }
-    const bool plain = norm_moments_needed(post.kind) && pre.kind == kNormNone;
+    const bool plain = norm_moments_needed(post.kind) && pre.kind == kNormNone && !step;
 #define LSB_PN(T, M) if (plain) LSB_PM(T, M, true); else LSB_PM(T, M, false)
-#define LSB_PM(T, M, P) launch_pdl((post_norm_kernel<T, M, P>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
+#define LSB_PM(T, M, P) launch_pdl((post_norm_kernel<T, M, P>), rows, norm_threads(dim, rows), (size_t)dim * 4, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo, step, ic)
     if (f32) { if (mo.y) { LSB_PN(float, true); } else { LSB_PN(float, false); } }
     else { if (mo.y) { LSB_PN(bf16, true); } else { LSB_PN(bf16, false); } }
 #undef LSB_PN
@@ -916,15 +989,29 @@ static int residual_update(void* x, int ldx, void* resid, int ldr, const void* s
 
 // Residual update with a norm on either side: resid += post(sub + sum of the row's S expert outputs), x = pre(resid).  Kinds: 0 RMS, 1 layer norm,
 // 2 dynamic tanh (w, b, alpha: one number), 3 none (post: the sum as it is).  sub null: no dense part; y null: no experts; wts null: experts are
-// added as they are; ids >= experts: identity experts.
+// added as they are; ids >= experts: identity experts.  step [dim] (null: none) is added to the residual stream as well.  xc (null: none): the input
+// convolution of steps with one row per sequence (see InputConv); slots: per row, -1 for idle rows.
 LSB_API int lsb_resid_update(void* x, int ldx, void* resid, int ldr, const void* sub, int lds, int post_kind, const void* post_w, const void* post_b,
                              const void* post_alpha, int pre_kind, const void* pre_w, const void* pre_b, const void* pre_alpha, int rows, int dim,
-                             float eps, const void* y, const void* wts, const void* ids, const void* slot_of, int S, int experts, int ldy, int f32,
-                             void* stream) {
+                             float eps, const void* y, const void* wts, const void* ids, const void* slot_of, int S, int experts, int ldy, const void* step,
+                             void* xc, const void* conv_w, void* conv_state, const void* slots, int taps, int ldw, int f32, void* stream) {
     const NormW post{(const float*)post_w, (const float*)post_b, (const float*)post_alpha, dim, eps, post_kind};
     const NormW pre{(const float*)pre_w, (const float*)pre_b, (const float*)pre_alpha, dim, eps, pre_kind};
     const MoeSum mo{(const float*)y, (const float*)wts, (const int*)ids, (const int*)slot_of, S, experts, ldy};
-    return residual_update(x, ldx, resid, ldr, sub, lds, post, pre, mo, rows, f32, (cudaStream_t)stream);
+    return residual_update(x, ldx, resid, ldr, sub, lds, post, pre, mo, rows, (const float*)step, InputConv{xc, (const float*)conv_w, (float*)conv_state, (const int*)slots, taps, ldw}, f32,
+                           (cudaStream_t)stream);
+}
+
+// Input convolution of a step with runs of rows: xc = x + conv(x), rows of ldx; w [taps, ldw] fp32 (last tap: the current token), state [slots, taps - 1, ldw].
+LSB_API int lsb_input_conv(void* xc, const void* x, int ldx, const void* w, void* state, int taps, int ldw, const void* seq_row0, const void* seq_nrows, const void* seq_slot,
+                           int nseq, int rows, int dim, int f32, void* stream) {
+    if (rows < 1 || nseq < 1 || taps < 1 || taps - 1 > kConvRows || (taps > 1 && !state) || dim % 4 || ldx % 4 || ldw % 4 || ldw < dim) return -1;
+    const InputConv ic{xc, (const float*)w, (float*)state, nullptr, taps, ldw};
+    const dim3 grid((dim / 4 + 127) / 128, rows / kConvRows + nseq);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (f32) launch_pdl((input_conv_kernel<float>), grid, 128, 0, st, (const float*)x, ldx, ic, (const int*)seq_row0, (const int*)seq_nrows, (const int*)seq_slot, nseq, dim);
+    else launch_pdl((input_conv_kernel<bf16>), grid, 128, 0, st, (const bf16*)x, ldx, ic, (const int*)seq_row0, (const int*)seq_nrows, (const int*)seq_slot, nseq, dim);
+    LSB_CHECK_LAUNCH();
 }
 
 // out[j] = norm(resid[row]); kind as above.

@@ -11,7 +11,7 @@
 
 namespace lsb {
 
-enum { kScoreSigmoid = 0, kScoreSoftmax = 1, kScoreSqrtSoftplus = 2 };
+enum { kScoreSigmoid = 0, kScoreSoftmax = 1, kScoreSqrtSoftplus = 2, kScoreLogits = 3 };     // 3: the bias is part of the logits, the choice is by them, softmax weights
 enum { kGroupTop2 = 0, kGroupMax = 1 };       // a group's score: the sum of its two best biased scores, or its best one
 
 // floats of shared memory router_topk_block needs for E experts
@@ -32,22 +32,24 @@ __device__ __forceinline__ void router_topk_block(const float* __restrict__ lg, 
     float* red = pick_w + 32;                  // [34]
     const int t = threadIdx.x, nt = blockDim.x;
     float mx = 0.f, den = 1.f;
-    if (scoring == kScoreSoftmax) {
+    const bool by_logit = scoring == kScoreLogits;
+    auto logit = [&](int e) { return (CG ? __ldcg(lg + e) : lg[e]) + (by_logit && bias ? bias[e] : 0.f); };
+    if (scoring == kScoreSoftmax || by_logit) {
         float m = -INFINITY;
-        for (int e = t; e < E; e += nt) m = fmaxf(m, CG ? __ldcg(lg + e) : lg[e]);
+        for (int e = t; e < E; e += nt) m = fmaxf(m, logit(e));
         mx = block_max(m, red);
         float s = 0.f;
-        for (int e = t; e < E; e += nt) s += expf((CG ? __ldcg(lg + e) : lg[e]) - mx);
+        for (int e = t; e < E; e += nt) s += expf(logit(e) - mx);
         den = block_sum(s, red);
     }
     for (int e = t; e < E; e += nt) {
-        const float x = CG ? __ldcg(lg + e) : lg[e];
+        const float x = logit(e);
         float s;
         if (scoring == kScoreSigmoid) s = 1.f / (1.f + expf(-x));
-        else if (scoring == kScoreSoftmax) s = expf(x - mx) / den;
+        else if (scoring == kScoreSoftmax || by_logit) s = expf(x - mx) / den;
         else s = sqrtf(x > 20.f ? x : log1pf(expf(x)));
         score[e] = s;
-        sel[e] = s + (bias ? bias[e] : 0.f);
+        sel[e] = by_logit ? x : s + (bias ? bias[e] : 0.f);
     }
     if (t < 32) { pick_id[t] = 0; pick_w[t] = 0.f; }
     __syncthreads();

@@ -34,6 +34,36 @@ __global__ void embedding_kernel(float* __restrict__ out_f32, bf16* __restrict__
     pdl_launch_dependents();
 }
 
+// out[r] = scale * table[ids[r]] + pairs[(prev[r] * mul_prev + ids[r] * mul_cur) mod buckets], the last row (number `buckets`) of pairs for a row without
+// a previous token (prev < 0).
+__global__ void __launch_bounds__(256) embedding_bigram_kernel(float* __restrict__ out, const bf16* __restrict__ table, const bf16* __restrict__ pairs,
+                                                               const int* __restrict__ ids, const int* __restrict__ prev, int hidden, int vocab, float scale,
+                                                               int buckets, long long mul_prev, long long mul_cur) {
+    const int r = blockIdx.x;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int id = ids[r], p = prev[r];
+    const bool own = id >= 0 && id < vocab;
+    long long b = buckets;
+    if (p >= 0) {
+        // the terms are reduced one by one: neither product leaves 64 bits for tokens and multipliers of 31 bits
+        b = (p * mul_prev % buckets + (long long)id * mul_cur % buckets) % buckets;
+        if (b < 0) b += buckets;
+    }
+    const bf16* src = table + (size_t)(own ? id : 0) * hidden;
+    const bf16* add = pairs + (size_t)b * hidden;
+    for (int i = threadIdx.x; i < hidden; i += 256) out[(size_t)r * hidden + i] = own ? __bfloat162float(src[i]) * scale + __bfloat162float(add[i]) : 0.f;
+}
+
+// x <- cap * tanh(x / cap)
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int ld, int n, float cap) {
+    const int i = blockIdx.x * 256 + threadIdx.x;
+    pdl_wait();
+    pdl_launch_dependents();
+    float* p = x + (size_t)blockIdx.y * ld + i;
+    if (i < n) *p = cap * tanhf(*p / cap);
+}
+
 // packed (key, ~index): larger value wins, equal values -> lower index wins
 __device__ __forceinline__ unsigned long long pack_vi(float v, int i) {
     return ((unsigned long long)sortable_key(v) << 32) | (unsigned long long)(0xffffffffu - (uint32_t)i);
@@ -281,6 +311,21 @@ LSB_API int lsb_embedding_scaled(void* out_f32, void* out_bf16, const void* tabl
 LSB_API int lsb_embedding(void* out_f32, void* out_bf16, const void* table, const void* ids, int rows, int hidden,
                           int vocab_lo, int vocab_hi, void* stream) {
     return lsb_embedding_scaled(out_f32, out_bf16, table, ids, rows, hidden, vocab_lo, vocab_hi, 1.f, stream);
+}
+
+// Token embedding times a factor plus a learned row per pair of tokens (hashed into `buckets` rows; see embedding_bigram_kernel), fp32.
+LSB_API int lsb_embedding_bigram(void* out, const void* table, const void* pairs, const void* ids, const void* prev, int rows, int hidden, int vocab, float scale, int buckets,
+                                 long long mul_prev, long long mul_cur, void* stream) {
+    if (rows < 1 || buckets < 1 || !pairs || !prev) return -1;
+    launch_pdl((embedding_bigram_kernel), rows, 256, 0, (cudaStream_t)stream, (float*)out, (const bf16*)table, (const bf16*)pairs, (const int*)ids, (const int*)prev, hidden,
+               vocab, scale, buckets, mul_prev, mul_cur);
+    LSB_CHECK_LAUNCH();
+}
+// Soft cap of the logits, in place.
+LSB_API int lsb_softcap(void* logits, int ld, int rows, int V, float cap, void* stream) {
+    if (rows < 1 || rows > 65535 || V < 1 || !(cap > 0.f)) return -1;
+    launch_pdl((softcap_kernel), dim3((V + 255) / 256, rows), 256, 0, (cudaStream_t)stream, (float*)logits, ld, V, cap);
+    LSB_CHECK_LAUNCH();
 }
 
 // part: scratch u64 [rows, 64].  out_val may be null.  `base` is added to the index (vocab shard offset).

@@ -10,9 +10,14 @@ the stream and every sublayer reads and updates them through learned static weig
 
     u = sum_s in_s x_s,    y = residual_mult * f(n_in(u)),    x_t <- sum_s mix_st x_s + out_t y,    logits = head(norm(sum_t x_t)).
 
+With ``norm_place`` "parallel" both sublayers of a layer read one norm and their projections back are one product: x <- x + mixer(h + conv(h)) + ffn(h),
+h = n_in(x), where conv is a short causal convolution per channel (``input_conv``; any placement of the norms may have it).  A range of layers may run
+several times (``loop``): same weights, a cache and state per pass, a learned vector on the stream in front of each.
+
 Same engine, caches and step protocol as :class:`DeviceModel`: attention layers keep a paged cache (one row of all heads' keys and values per
 token; latent layers one row for all heads, which later layers may read instead of keeping their own), recurrent layers an fp32 state per sequence
-slot with the convolutions' history (delta rule) or the previous token's input (time mixing); layers with two mixers side by side have both.  Steps are any mixture of prompt portions and single tokens.
+slot with the convolutions' history (delta rule) or the previous token's input (time mixing); layers with two mixers side by side have both, and
+input convolutions the inputs they look back at.  Caches and states are numbered by layer run.  Steps are any mixture of prompt portions and single tokens.
 
 Two precisions.  ``bfloat16``: weights, activations and the cache in bf16, products accumulated in fp32; the residual stream, norms, routing,
 attention scores and weights, rotations and the whole recurrence in fp32.  ``float32``: everything in fp32 (FMA units, no reduced-precision
@@ -24,6 +29,7 @@ expert widths to the kernels' tiles; padding holds zeros and never reaches a res
 from __future__ import annotations
 
 import logging
+import math
 from typing import Dict, List, Optional
 
 import torch
@@ -38,6 +44,8 @@ EXPAND_ROWS = 128       # rows of a step of one sequence from which latent layer
 EXPAND_BYTES = 1 << 30  # ... while those of all its positions fit this much scratch
 NORM_KIND = {"rms": 0, "layer": 1, "tanh": 2}        # as the kernels number them; 3: none
 NO_NORM = (3, None, None, None)
+SCORING = {"sigmoid": 0, "softmax": 1}
+LOGIT_SCORES = 3        # the router's bias is part of the logits
 HEAD_NORM = {"": 0, "plain": 1, "weight": 2}
 
 
@@ -63,15 +71,18 @@ def _mixer_shapes(out: dict, p: str, b: BlockSpec, H: int, ranks: tuple):
                     k + "u": (b.heads, b.dim), k + "o_norm": (vw,), k + "o": (H, vw)} | {k + "mu_" + n: (H,) for n in "rkvgw"})
     elif b.latent:
         a = p + "attn."
-        out.update({a + "q": (b.heads * (b.dim + b.rot_dim), H), a + "k_b": (b.heads * b.dim, b.kv_rank), a + "v_b": (b.heads * b.vdim, b.kv_rank),
+        qw = b.heads * (b.dim + b.rot_dim)
+        out.update({a + "q_a": (b.q_rank, H), a + "q_a_norm": (b.q_rank,), a + "q_b": (qw, b.q_rank)} if b.q_rank else {a + "q": (qw, H)})
+        out.update({a + "k_b": (b.heads * b.dim, b.kv_rank), a + "v_b": (b.heads * b.vdim, b.kv_rank),
                     a + "o": (H, b.heads * b.vdim)})
         if b.kv_from < 0:
             out.update({a + "kv_a": (b.kv_rank + b.rot_dim, H), a + "kv_a_norm": (b.kv_rank,)})
-        if b.head_gate:
-            out[a + "g"] = (b.heads, H)
+        if b.out_gate or b.head_gate:
+            out[a + "g"] = (b.heads * (b.vdim if b.out_gate else 1), H)
     else:
-        a, qw, kw, vw = p + "attn.", b.heads * b.dim, b.kv_heads * b.dim, b.kv_heads * b.vdim
-        out.update({a + "q": (qw, H), a + "k": (kw, H), a + "v": (vw, H), a + "o": (H, b.heads * b.vdim)})
+        a, qw, kw, vw = p + "attn.", b.heads * b.maps * b.dim, b.kv_heads * b.maps * b.dim, b.kv_heads * b.vdim
+        out.update({a + "q": (qw, H), a + "k": (kw, H), a + "o": (H, b.heads * b.vdim)} | ({} if b.shared_kv else {a + "v": (vw, H)}))
+        out.update({a + n: (b.heads,) for n, has in (("temp", b.temp), ("sink", b.sink)) if has} | ({a + n: (b.dim,) for n in ("lq1", "lk1", "lq2", "lk2")} if b.maps > 1 else {}))
         if b.qkv_bias:
             out.update({a + "q_bias": (qw,), a + "k_bias": (kw,), a + "v_bias": (vw,)})
         if b.qk_norm:
@@ -104,13 +115,19 @@ def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = No
     """Canonical tensor names and shapes.  ``ranks``: {layer: (decay rank, gate rank)} of delta-rule layers (default: the key head width)."""
     H, out = cfg.hidden, {}
     extra = {"rms": (), "layer": ("bias",), "tanh": ("bias", "alpha")}[cfg.norm_kind]
-    norm = lambda p: out.update({p + ".weight": (H,)} | {f"{p}.{k}": () if k == "alpha" else (H,) for k in extra})
+    norm = lambda p: out.update({p + ".weight": () if cfg.norm_scalar else (H,)} | {f"{p}.{k}": () if k == "alpha" else (H,) for k in extra})
     out["embed.weight"] = out["head.weight"] = (cfg.vocab, H)
     if cfg.side_dim:
         out["side_embed.weight"] = (cfg.vocab, cfg.n_layers * cfg.side_dim)
+    if cfg.bigram:
+        out["bigram.weight"] = (cfg.bigram[0] + 1, H)
+    if cfg.loop:
+        out["loop_step"] = (cfg.loop[2], H)
     norm("final_norm")
     for i, b in enumerate(cfg.blocks):
         p = f"layers.{i}."
+        if cfg.input_conv:
+            out[p + "input_conv"] = (H, cfg.input_conv)
         norm(p + "mix_norm")
         if cfg.norm_place == "sandwich":
             norm(p + "mix_post_norm")
@@ -121,7 +138,7 @@ def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = No
         if cfg.streams:
             for q in ["mix_hc"] + (["ffn_hc"] if b.has_ff else []):
                 out.update({f"{p}{q}.in": (cfg.streams,), f"{p}{q}.out": (cfg.streams,), f"{p}{q}.mix": (cfg.streams, cfg.streams)})
-        if b.has_ff:
+        if b.has_ff and cfg.norm_place != "parallel":
             norm(p + "ffn_norm")
             if cfg.norm_place == "sandwich":
                 norm(p + "ffn_post_norm")
@@ -131,7 +148,7 @@ def block_weight_shapes(cfg: ModelConfig, ranks: Optional[Dict[int, tuple]] = No
         if b.experts:
             m = p + "moe."
             out[m + "router"] = (b.experts + b.identity, H)
-            if b.correction:
+            if b.correction or b.logit_bias:
                 out[m + "router_bias"] = (b.experts + b.identity,)
             for e in range(b.experts):
                 glu(m + f"experts.{e}.", b.ff)
@@ -155,8 +172,14 @@ def random_block_tensor(name: str, shape: tuple, gen: torch.Generator, device="c
         return t.uniform_(-3.0, 0.5, generator=gen)
     if leaf == "dt_bias":
         return t.uniform_(-3.0, -1.0, generator=gen)
-    if leaf.startswith("conv_"):
+    if leaf.startswith("conv_") or leaf == "input_conv":
         return t.uniform_(-0.7, 0.7, generator=gen)
+    if leaf == "temp":
+        return t.uniform_(0.5, 1.5, generator=gen)
+    if leaf in ("sink", "loop_step"):
+        return t.normal_(0.0, 0.5, generator=gen)
+    if leaf in ("lq1", "lk1", "lq2", "lk2"):
+        return t.normal_(0.0, 0.1, generator=gen)
     if leaf.startswith("mu_"):
         return t.uniform_(0.1, 0.9, generator=gen)
     if leaf == "w0":
@@ -174,7 +197,7 @@ def random_block_tensor(name: str, shape: tuple, gen: torch.Generator, device="c
     if leaf == "alpha":
         return t.uniform_(0.4, 1.0, generator=gen)
     if leaf == "weight":                                     # token tables, head
-        return t.normal_(0.0, 1.0 if "embed" in name else 0.5 / shape[1] ** 0.5, generator=gen)
+        return t.normal_(0.0, 1.0 if "embed" in name or "bigram" in name else 0.5 / shape[1] ** 0.5, generator=gen)
     return t.normal_(0.0, 1.0 / shape[1] ** 0.5, generator=gen)
 
 
@@ -198,7 +221,10 @@ class BlockWorkspace(StepBuffers):
     def __init__(self, m: "BlockModel", R: int, n_logit_rows: int, max_ctx: int):
         super().__init__(m, R, n_logit_rows)
         z, act, Hp = self.z, m.act_dtype, m.Hp
-        self.x = z(R, Hp, dtype=act)                 # the residual stream in the activation type: what every sublayer reads
+        # the residual stream in the activation type, what every sublayer reads; with input convolutions what the mixers read stands in front of it
+        self.x_pair = z(2, R, Hp, dtype=act) if m.cfg.input_conv else None
+        self.x = z(R, Hp, dtype=act) if self.x_pair is None else self.x_pair[1]
+        self.x_mix = self.x if self.x_pair is None else self.x_pair[0]
         self.resid = z(R, Hp)
         self.sub = z(R, Hp)
         self.xh = z(n_logit_rows, Hp, dtype=act)
@@ -209,29 +235,32 @@ class BlockWorkspace(StepBuffers):
         self.streams = z(R, m.cfg.streams, Hp) if m.cfg.streams else None
         self.sub2 = z(R, Hp) if any(b.join == "normed" and b.branches for b in m.cfg.blocks) else None
         self.xs = z(5, R, Hp, dtype=act) if any(b.kind == "time_mix" for L in m.cfg.blocks for b in L.mixers) else None      # token-shifted inputs
+        if any(b.q_rank for b in lat):
+            self.q_low = z(R * max(_align(b.q_rank, 8) for b in lat), dtype=act)
+            self.q_up = z(R * max(_align(b.heads * (b.dim + b.rot_dim), 8) for b in lat if b.q_rank))
         if lat:
             self.q_lat = z(R * max(b.heads * m.latent_row(b) for b in lat), dtype=act)
             self.q_nope = z(R * max(b.heads * _align(b.dim, 8) for b in lat), dtype=torch.bfloat16) if not m.f32 and R >= 8 else None
             self.o_lat = z(R * max(b.heads * m.latent_pad(b.kv_rank) for b in lat), dtype=act)
-            self.lat_splits = {i: 1 if R > 64 else int(nat.call("lsb_latent_splits", R, b.heads, b.kv_rank, b.rot_dim, max_ctx, int(m.f32)))
+            self.lat_splits = {i: 1 if R > 64 else int(nat.call("lsb_latent_splits", R, b.heads, b.kv_rank, b.rot_dim, min(b.window or max_ctx, max_ctx), int(m.f32)))
                                for i, b in enumerate(m.cfg.blocks) if b.latent}
             self.lat_parts = {i: int(nat.call("lsb_latent_partials", n)) for i, n in self.lat_splits.items()}
             ns = [(b.heads * self.lat_parts[i], m.latent_pad(b.kv_rank)) for i, b in enumerate(m.cfg.blocks) if self.lat_parts.get(i, 1) > 1]
             self.lat_o_part = z(R * max((n * w for n, w in ns), default=1))
             self.lat_ml_part = z(2 * R * max((n for n, _ in ns), default=1))
         dense = max((_align(max(b.dense_ff, b.shared_ff), 8) for b in m.cfg.blocks), default=0)
-        self.glu = z(R * dense, dtype=act) if dense else None
+        self.glu = z(R * dense, dtype=act) if dense and m.cfg.norm_place != "parallel" else None
         self.side = z(R, _align(m.cfg.side_dim, 8), dtype=act) if m.cfg.side_dim else None
         if att:
-            self.q = z(R * max(b.heads * m.head_pad(b.dim) for _, b in att), dtype=act)
+            self.q = z(R * max(b.heads * b.maps * m.head_pad(b.dim) for _, b in att), dtype=act)
             self.v_first = z(R, max([b.kv_heads * b.vdim for _, b in att if b.v_mix], default=1))
             # key splits of the few-row attention: about two blocks per SM, no split shorter than 64 visible keys
             self.splits = {}
             for i, b in att:
                 seen = min(b.window or max_ctx, b.chunk or max_ctx, max_ctx)
-                blocks = R * b.kv_heads * ((b.heads // b.kv_heads + 15) // 16)
+                blocks = R * b.kv_heads * b.maps * ((b.heads // b.kv_heads + 15) // 16)
                 self.splits[i] = 1 if (m.f32 or R > 64) else max(1, min(32, 296 // blocks, (seen + 63) // 64))
-            ns = [(b.heads * self.splits[i], m.head_pad(b.vdim)) for i, b in att if self.splits[i] > 1]
+            ns = [(b.heads * b.maps * self.splits[i], m.head_pad(b.vdim)) for i, b in att if self.splits[i] * b.maps > 1]
             self.o_part = z(R * max((n * w for n, w in ns), default=1))
             self.ml_part = z(2 * R * max((n for n, _ in ns), default=1))
         self.moe: Dict[tuple, MoeBuffers] = {}
@@ -294,10 +323,16 @@ class BlockModel(ModelBase):
             raise ValueError("layers that mix values must have the same number of value channels")
         if cfg.residual_mult != 1.0 and not cfg.streams or cfg.streams and cfg.norm_place != "pre" or cfg.streams > 8 or cfg.streams and cfg.side_dim:
             raise ValueError("hyper-connections (up to 8 streams) come with norms in front of the sublayers, a residual factor comes with hyper-connections")
+        if cfg.streams and (cfg.input_conv or cfg.loop) or cfg.loop and mixing or cfg.norm_place == "parallel" and any(b.branches for b in cfg.blocks) or cfg.input_conv > 17:
+            raise ValueError("input convolutions (of up to 17 taps) and loops come with one residual stream, loops without value mixing, parallel sublayers with one mixer")
+        if cfg.bigram and len(cfg.bigram) != 3:
+            raise ValueError("a bigram embedding has a number of buckets and two multipliers")
         for i, b in [(i, m) for i, L in enumerate(cfg.blocks) for m in L.mixers]:
+            if b.kind == "time_mix" and cfg.input_conv:
+                raise ValueError(f"layer {i}: time mixing behind an input convolution")
             if b.heads % max(b.kv_heads, 1) or min(b.heads, b.kv_heads, b.dim, b.vdim) < 1:
                 raise ValueError(f"layer {i}: {b.heads} heads over {b.kv_heads} groups of widths {b.dim} / {b.vdim}")
-            if b.latent and (b.kv_rank < 1 or b.rot_dim < 2 or b.rot_dim % 2):
+            if b.latent and (b.kv_rank < 1 or b.rot_dim < 0 or b.rot_dim % 2):
                 raise ValueError(f"layer {i}: latent rows of {b.kv_rank} + {b.rot_dim} channels")
             if b.recurrent and b.dim > 256:
                 raise ValueError(f"layer {i}: key heads of up to 256 channels, not {b.dim}")
@@ -381,10 +416,13 @@ class BlockModel(ModelBase):
         a = p + "attn."
         if b.latent:
             own = b.kv_from < 0
-            names = ["q"] + (["kv_a"] if own else []) + (["g"] if b.head_gate else [])
+            qn = "q_a" if b.q_rank else "q"
+            names = [qn] + (["kv_a"] if own else []) + (["g"] if b.out_gate or b.head_gate else [])
             parts = [w[a + n].to(dev) for n in names]
             at = dict(zip(names, _offsets(parts)))
-            M["meta"] = _Meta([at["q"], at.get("kv_a", -1), at.get("g", -1)])
+            M["meta"] = _Meta([at[qn], at.get("kv_a", -1), at.get("g", -1)])
+            if b.q_rank:
+                M["q_norm"], M["q_up"] = self._vec(w[a + "q_a_norm"]), self._mat(w[a + "q_b"].to(dev))
             dnp, dlp = _align(b.dim, 8), self.latent_pad(b.kv_rank)
             uk, uv = w[a + "k_b"].to(dev).view(b.heads, b.dim, b.kv_rank), w[a + "v_b"].to(dev).view(b.heads, b.vdim, b.kv_rank)
             M["w_uk"] = torch.zeros(b.heads, dlp, dnp, dtype=self.act_dtype, device=dev)
@@ -402,14 +440,22 @@ class BlockModel(ModelBase):
             M["inv_freq"] = self._inv_freq(b.rot_base, b.rot_dim)
             return parts, w[a + "o"].to(dev)
         gate = b.out_gate or b.head_gate
-        parts = [w[a + n].to(dev) for n in ("q", "k", "v")] + ([w[a + "g"].to(dev)] if gate else [])
-        M["meta"] = _Meta(_offsets(parts) + ([] if gate else [-1]))
+        names = ["q", "k"] + ([] if b.shared_kv else ["v"]) + (["g"] if gate else [])
+        parts = [w[a + n].to(dev) for n in names]
+        at = dict(zip(names, _offsets(parts)))
+        M["meta"] = _Meta([at["q"], at["k"], at.get("v", at["k"]), at.get("g", -1)])       # shared keys and values: one projection
+        for n in ("temp", "sink"):
+            if getattr(b, n):
+                M[n] = self._vec(w[a + n])
+        if b.maps > 1:
+            dot = lambda j: float((w[a + f"lq{j}"].double() * w[a + f"lk{j}"].double()).sum())
+            M["lambda"] = math.exp(dot(1)) - math.exp(dot(2)) + b.diff
         if b.qkv_bias:
             M["q_bias"], M["k_bias"], M["v_bias"] = (self._vec(w[a + n + "_bias"]) for n in "qkv")
         if b.qk_norm or b.head_norm == "weight":
             M["q_norm"], M["k_norm"] = self._vec(w[a + "q_norm"]), self._vec(w[a + "k_norm"])
-        if b.half_rot:
-            M["inv_freq"] = self._inv_freq(b.rot_base, b.half_rot)
+        if b.half_rot or b.pair_rot:
+            M["inv_freq"] = self._inv_freq(b.rot_base, b.half_rot or b.pair_rot)
         if b.bias_rows:
             rel = w[a + "rel"].to(dev).float()                 # one value per distance and head: the kernels know no buckets
             M["bias"] = rel[torch.tensor(distance_buckets(rel.shape[0], b.bias_max), device=dev)].T.contiguous()
@@ -440,7 +486,8 @@ class BlockModel(ModelBase):
         def norm(p, scale=1.0):
             """(kind, weight, bias, alpha) of a norm of the residual stream"""
             b, al = p + ".bias", p + ".alpha"
-            return kind, m._vec(w[p + ".weight"]) * scale, (m._vec(w[b]) * scale if b in w else None), (m._vec(w[al]) if al in w else None)
+            wt = m._vec(w[p + ".weight"]) * scale
+            return kind, wt.expand(H).contiguous() if cfg.norm_scalar else wt, (m._vec(w[b]) * scale if b in w else None), (m._vec(w[al]) if al in w else None)
 
         def stacked(parts, cols=Hp):
             """The parts as one projection and the row at which each starts."""
@@ -453,13 +500,25 @@ class BlockModel(ModelBase):
         m.head = m._mat(hw, cols=Hp)
         m.head.N = cfg.vocab                                   # padding rows of the matrix are never computed
         m.final_norm = norm("final_norm", cfg.logit_scale)     # the scale of the logits rides on the last norm
+        if cfg.bigram:
+            m.bigram = torch.zeros(cfg.bigram[0] + 1, Hp, dtype=torch.bfloat16, device=dev)
+            m.bigram[:, :H] = w["bigram.weight"].to(dev)
+        if cfg.loop:
+            m.loop_step = torch.zeros(cfg.loop[2], Hp, device=dev)
+            m.loop_step[:, :H] = w["loop_step"].to(dev)
         if cfg.side_dim:
             m.side_embed = w["side_embed.weight"].to(dev).to(torch.bfloat16).contiguous()
         for i, b in enumerate(cfg.blocks):
             p = f"layers.{i}."
             L: dict = {"mix_in": norm(p + "mix_norm"), "mix_out": norm(p + "mix_post_norm")} if sandwich else {"mix_in": NO_NORM, "mix_out": norm(p + "mix_norm")}
-            if cfg.norm_place == "pre":
+            if cfg.norm_place in ("pre", "parallel"):
                 L["mix_in"], L["mix_out"] = L["mix_out"], NO_NORM
+            if cfg.input_conv:
+                taps = w[p + "input_conv"].to(dev)
+                if tuple(taps.shape) != (H, cfg.input_conv):
+                    raise ValueError(f"{p}input_conv: shape {tuple(taps.shape)}")
+                L["conv_w"] = torch.zeros(cfg.input_conv, Hp, device=dev)
+                L["conv_w"][:, :H] = taps.float().T
             sides, cols = _sides(b), 0
             L["sides"] = [{} for _ in sides]
             parts, outs, base = [], [], 0
@@ -472,8 +531,23 @@ class BlockModel(ModelBase):
                 base += sum(_align(t.shape[0], 8) for t in own)
                 parts += own
                 outs.append(out)
-            L["mix_ld"] = cols
-            L["in"] = stacked(parts)[0] if parts else None
+            # one norm for both sublayers: what the feed-forward projects with follows the mixer's projections, its way back is part of the mixer's
+            both = cfg.norm_place == "parallel" and b.has_ff
+            glu_ff = (b.dense_ff or b.shared_ff) if both else 0
+            glu = ("mlp." if b.dense_ff else "moe.shared.0.") if glu_ff else ""
+            ff_parts = []
+            if both:
+                ff_parts = ([w[p + "moe.router"].to(dev)] if b.experts else []) + ([w[p + glu + n].to(dev) for n in ("gate", "up")] if glu else [])
+                ff_parts += [w[p + "moe.shared_gate"].to(dev)] if b.experts and b.shared_ff else []
+            L["mix_ld"] = cols + _align(glu_ff, 8)
+            L["glu_at"] = cols
+            L["in"] = stacked(parts + ff_parts)[0] if parts + ff_parts else None
+            if both:
+                W, n = L["in"], sum(_align(t.shape[0], 8) for t in parts)
+                L["halves"] = (QLinear(W.fmt, n, Hp, W.w[:n]), QLinear(W.fmt, W.N - n, Hp, W.w[n:]))
+                L["half_rows"] = torch.tensor([0, n], dtype=torch.int32)
+                L["ff_at"], L["ff_offs"] = n, [n + o for o in _offsets(ff_parts)]
+                base += W.N - n
             for M in L["sides"]:
                 if "shift" in M:                              # projections over inputs of their own, behind the others
                     M["meta"].shift(base)
@@ -486,17 +560,21 @@ class BlockModel(ModelBase):
                     M["out"].N = Hp
             else:
                 pad = torch.nn.functional.pad
-                L["out"] = m._mat(torch.cat([pad(t, (0, M["cols"] - t.shape[1])) for t, M in zip(outs, L["sides"])], 1))
+                wide = [pad(t, (0, M["cols"] - t.shape[1])) for t, M in zip(outs, L["sides"])]
+                if glu:
+                    t = w[p + glu + "down"].to(dev)
+                    wide.append(pad(t, (0, _align(t.shape[1], 8) - t.shape[1])))
+                L["out"] = m._mat(torch.cat(wide, 1))
                 L["out"].N = Hp
-            m.max_mix = max(m.max_mix, cols)
+            m.max_mix = max(m.max_mix, L["mix_ld"])
             if cfg.streams:
                 for q in ["mix_hc"] + (["ffn_hc"] if b.has_ff else []):
                     L[q] = tuple(m._vec(w[f"{p}{q}.{k}"]) for k in ("in", "out", "mix"))
-            if b.has_ff:
+            if b.has_ff and not both:
                 L["ff_in"], L["ff_out"] = (norm(p + "ffn_norm"), norm(p + "ffn_post_norm")) if sandwich else (NO_NORM, norm(p + "ffn_norm"))
                 if cfg.norm_place == "pre":
                     L["ff_in"], L["ff_out"] = L["ff_out"], NO_NORM
-            if b.dense_ff:
+            if b.dense_ff and not both:
                 L["ff"], L["ff_offs"] = stacked([w[p + f"mlp.{n}"].to(dev) for n in ("gate", "up")])
                 L["ff_down"] = m._mat(w[p + "mlp.down"].to(dev))
                 L["ff_down"].N = Hp
@@ -505,13 +583,14 @@ class BlockModel(ModelBase):
                 mo = p + "moe."
                 # the router and - where there is one - the shared expert's gate, up and output-gate rows are one product (values of the file's
                 # type: fp32-accumulated products are exact in them)
-                parts = [w[mo + "router"].to(dev)] + ([w[mo + n].to(dev) for n in ("shared.0.gate", "shared.0.up", "shared_gate")] if b.shared_ff else [])
-                L["router"], L["ff_offs"] = stacked(parts)
-                L["router_bias"] = m._vec(w[mo + "router_bias"]) if b.correction and (mo + "router_bias") in w else None
-                if b.shared_ff:
-                    L["ff_down"] = m._mat(w[mo + "shared.0.down"].to(dev))
-                    L["ff_down"].N = Hp
-                m.max_proj = max(m.max_proj, L["router"].N)
+                if not both:
+                    parts = [w[mo + "router"].to(dev)] + ([w[mo + n].to(dev) for n in ("shared.0.gate", "shared.0.up", "shared_gate")] if b.shared_ff else [])
+                    L["router"], L["ff_offs"] = stacked(parts)
+                    m.max_proj = max(m.max_proj, L["router"].N)
+                    if b.shared_ff:
+                        L["ff_down"] = m._mat(w[mo + "shared.0.down"].to(dev))
+                        L["ff_down"].N = Hp
+                L["router_bias"] = m._vec(w[mo + "router_bias"]) if (b.correction or b.logit_bias) and (mo + "router_bias") in w else None
                 # expert width padded to the tensor-core tile where the residual width allows that path
                 F = _align(b.ff, 128) if Hp % 128 == 0 else _align(b.ff, 8)
                 gated = b.unit == "glu"
@@ -554,7 +633,11 @@ class BlockModel(ModelBase):
         z = lambda *s, dtype=torch.float32: torch.zeros(*s, dtype=dtype, device=self.device)
         self.block_table = z(n_slots, max_pages_per_seq, dtype=torch.int32)
         self.idx_block_table = self.block_table
-        for i, b in [(i, m) for i, L in enumerate(self.cfg.blocks) for m in L.mixers]:
+        runs = self.cfg.layer_runs()
+        if self.cfg.input_conv > 1:
+            for k in range(len(runs)):                                      # the inputs that the run's convolution looks back at
+                self.kda_conv["input", k] = z(n_slots, self.cfg.input_conv - 1, self.Hp)
+        for i, b in [(k, m) for k, (i, _) in enumerate(runs) for m in self.cfg.blocks[i].mixers]:
             if b.delta:
                 self.kda_state[i] = z(n_slots, b.heads, b.vdim, int(nat.call("lsb_delta_key_pad", b.dim)))
                 self.kda_conv[i] = z(n_slots, b.heads, 2 * b.dim + b.vdim, b.conv - 1)
@@ -565,90 +648,128 @@ class BlockModel(ModelBase):
                 if b.kv_from < 0:
                     self.kv_cache[i] = z(num_pages, self.page, self.latent_row(b), dtype=self.act_dtype)
             else:
-                self.kv_cache[i] = z(num_pages, self.page, b.kv_heads * (self.head_pad(b.dim) + self.head_pad(b.vdim)), dtype=self.act_dtype)
+                self.kv_cache[i] = z(num_pages, self.page, b.kv_heads * (b.maps * self.head_pad(b.dim) + self.head_pad(b.vdim)), dtype=self.act_dtype)
 
     def cache_bytes_per_token(self) -> int:
-        width = lambda b: ((self.latent_row(b) if b.kv_from < 0 else 0) if b.latent else b.kv_heads * (self.head_pad(b.dim) + self.head_pad(b.vdim)))
-        return sum(width(b) * (4 if self.f32 else 2) for L in self.cfg.blocks for b in L.mixers if not b.recurrent)
+        width = lambda b: ((self.latent_row(b) if b.kv_from < 0 else 0) if b.latent else b.kv_heads * (b.maps * self.head_pad(b.dim) + self.head_pad(b.vdim)))
+        return sum(width(b) * (4 if self.f32 else 2) for i, _ in self.cfg.layer_runs() for b in self.cfg.blocks[i].mixers if not b.recurrent)
 
     # ------------------------------------------------------------------ forward
     def _resid_rows(self, ws, R: int, H: int) -> torch.Tensor:
         return ws.streams[:R, :, :H].sum(1) if self.cfg.streams else ws.resid[:R, :H]
 
-    def _mixer(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
-        """The layer's mixers, input projections to output projection: ``ws.sub`` (and ``ws.sub2`` of a second result that is normed on its own)."""
-        if L["in"] is not None:
-            L["in"](ws.proj, ws.x, R, ldo=self.max_proj)
+    def _mixer(self, k: int, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int):
+        """The mixers of layer i in its run k, input projections to output projection: ``ws.sub`` (and ``ws.sub2`` of a second result that is normed on its
+        own).  With both sublayers on one norm the feed-forward's projections and gated unit as well: all of the layer but its routed experts."""
+        if "halves" in L:
+            self._project_both(L, ws, R)
+        elif L["in"] is not None:
+            L["in"](ws.proj, ws.x_mix, R, ldo=self.max_proj)
         for x, M in zip(b.mixers, L["sides"]):
             f = self._delta if x.delta else (self._time_mix if x.kind == "time_mix" else (self._latent if x.latent else self._attention))
-            f(i, x, M, ws, R, nseq, ws.mix.view(-1)[M["col"]:], L["mix_ld"])
+            f(k, i, x, M, ws, R, nseq, ws.mix.view(-1)[M["col"]:], L["mix_ld"])
+        if "halves" in L and (b.dense_ff or b.shared_ff):
+            ff = b.dense_ff or b.shared_ff
+            g, u, s = (*L["ff_offs"], -1) if b.dense_ff else L["ff_offs"][1:]
+            nat.call("lsb_glu", ws.mix.view(-1)[L["glu_at"]:], L["mix_ld"], _align(ff, 8), ws.proj, self.max_proj, g, u, s, R, ff, 0.0 if b.dense_ff else b.shared_limit,
+                     *((1.0, 0.0) if b.dense_ff else (b.act_alpha, b.act_shift)), int(self.f32))
         if b.branches and b.join == "normed":
             for M, sub in zip(L["sides"], (ws.sub, ws.sub2)):
                 M["out"](sub, ws.mix.view(-1)[M["col"]:], R, ldx=L["mix_ld"], ldo=self.Hp)
         else:
             L["out"](ws.sub, ws.mix, R, ldo=self.Hp)
 
-    def _attention(self, i: int, b: BlockSpec, M: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
+    def _project_both(self, L: dict, ws: BlockWorkspace, R: int):
+        """The mixer's projections (of its own input) and the feed-forward's (of the norm as it is), side by side in ``ws.proj``."""
+        W, (mix, ff) = L["in"], L["halves"]
+        if ws.x_pair is None:
+            W(ws.proj, ws.x, R, ldo=self.max_proj)
+        elif not self.f32 and R < 8 and self.Hp <= 16384:
+            nat.call("lsb_gemv_bf16_segs", ws.proj, ws.x_pair, W.w, R, W.N, self.Hp, self.Hp, self.Hp, self.max_proj, L["half_rows"], 2, ws.x_pair.stride(0))
+        else:
+            mix(ws.proj, ws.x_mix, R, ldo=self.max_proj)
+            ff(ws.proj.view(-1)[L["ff_at"]:], ws.x, R, ldo=self.max_proj)
+
+    def _attention(self, k: int, i: int, b: BlockSpec, M: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
         dkp, dvp, ldp = self.head_pad(b.dim), self.head_pad(b.vdim), self.max_proj
         oq, ok, ov, og = M["meta"].offs
-        at = (ws.q, self.kv_cache[i], self.block_table, self.max_pages, ws.row_seq, ws.row_pos, R, b.heads, b.kv_heads, b.dim, b.vdim, dkp, dvp, self.page, int(self.f32))
-        if b.qkv_bias or b.head_norm or b.half_rot:
+        H, G = b.heads * b.maps, b.kv_heads * b.maps
+        at = (ws.q, self.kv_cache[k], self.block_table, self.max_pages, ws.row_seq, ws.row_pos, R, H, G, b.dim, b.vdim, dkp, dvp, self.page, int(self.f32))
+        if b.qkv_bias or b.head_norm or b.half_rot or b.pair_rot or b.temp or b.shared_kv or b.maps > 1:
             nat.call("lsb_attn_head_prep", ws.proj, ldp, oq, ok, ov, M.get("q_bias"), M.get("k_bias"), M.get("v_bias"), HEAD_NORM[b.head_norm], M.get("q_norm"),
-                     M.get("k_norm"), self.cfg.rms_eps, b.half_rot, M.get("inv_freq"), *at)
+                     M.get("k_norm"), self.cfg.rms_eps, b.half_rot or b.pair_rot, int(b.pair_rot > 0), M.get("inv_freq"), M.get("temp"), b.maps, *at)
         else:
             mix = 0 if not b.v_mix else (1 if i == self.v_first_layer else 2)
             nat.call("lsb_attn_prep", ws.proj, ldp, oq, ok, ov, M.get("q_norm"), M.get("k_norm"), self.cfg.rms_eps, ws.v_first if mix else None, mix, M.get("v_mix"), *at)
-        bias = M.get("bias")
-        nat.call("lsb_attn", ws.q, self.kv_cache[i], self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
-                 max(ws.seq_rows), ws.proj, ldp, og, out, ldo, ws.o_part, ws.ml_part, ws.splits[i], R, b.heads, b.kv_heads, b.dim, b.vdim, dkp, dvp,
-                 b.window, b.scale, M.get("slope"), int(b.head_gate), b.chunk, bias, bias.shape[1] if bias is not None else 0, b.out_scale, int(self.f32))
+        bias, run = M.get("bias"), max(ws.seq_rows)
+        nat.call("lsb_attn", ws.q, self.kv_cache[k], self.block_table, self.max_pages, self.page, ws.row_seq, ws.row_pos, ws.seq_row0, ws.seq_nrows, nseq,
+                 run, ws.proj, ldp, og, out, ldo, ws.o_part, ws.ml_part, ws.splits[i], R, H, G, b.dim, b.vdim, dkp, dvp,
+                 b.window, b.scale, M.get("slope"), int(b.head_gate), b.chunk, bias, bias.shape[1] if bias is not None else 0, b.out_scale, M.get("sink"), b.maps,
+                 int(self.f32))
+        if b.maps > 1:
+            n = nat.call("lsb_attn_partials", run, H, G, dkp, dvp, ws.splits[i], int(self.f32))
+            nat.call("lsb_attn_diff", out, ldo, ws.o_part, ws.ml_part, n, R, b.heads, b.heads // b.kv_heads, b.vdim, dvp, M["lambda"], self.cfg.rms_eps,
+                     b.out_scale * (1.0 - b.diff), ws.row_seq, int(self.f32))
 
-    def _latent(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
-        cache = self.kv_cache[i if b.kv_from < 0 else b.kv_from]
+    def _latent(self, k: int, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
+        cache = self.kv_cache[k if b.kv_from < 0 else b.kv_from]
+        q, ldq = ws.proj.view(-1)[L["meta"].offs[0]:], self.max_proj           # the heads' queries: straight from the projection or through a latent
+        if b.q_rank:
+            nat.call("lsb_norm_rows", ws.q_low, L["q_up"].K, q, ldq, None, 0, L["q_norm"], None, None, R, b.q_rank, self.cfg.rms_eps, NORM_KIND["rms"], int(self.f32))
+            q, ldq = ws.q_up, L["q_up"].N
+            L["q_up"](q, ws.q_low, R)
         # long runs one by one, what lies between them together
         rows, row0, j = ws.seq_rows, 0, 0
         while j < nseq:
-            k, n = j + 1, rows[j]
+            e, n = j + 1, rows[j]
+            at = (q[row0 * ldq:], ldq)
             if self._expands(b, rows[j], ws.seq_end[j]):
-                self._latent_run(b, L, ws, cache, row0, n, j)
+                self._latent_run(b, L, ws, cache, *at, row0, n, j, out, ldo)
             else:
-                while k < nseq and not self._expands(b, rows[k], ws.seq_end[k]):
-                    n, k = n + rows[k], k + 1
-                self._latent_rows(i, b, L, ws, cache, row0, n, j, k)
-            row0, j = row0 + n, k
+                while e < nseq and not self._expands(b, rows[e], ws.seq_end[e]):
+                    n, e = n + rows[e], e + 1
+                self._latent_rows(i, b, L, ws, cache, *at, row0, n, j, e, out, ldo)
+            row0, j = row0 + n, e
 
-    def _latent_rows(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, r0: int, R: int, j: int, k: int):
+    def _latent_rows(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, qsrc, ldq: int, r0: int, R: int, j: int, k: int, out, ldo: int):
         """Step rows [r0, r0 + R) (sequences j .. k - 1 of the step) in the latent space."""
-        oq, okv, og = L["meta"].offs
-        H, ld, K, f32, err = b.heads, self.max_proj, L["cols"], int(self.f32), TcScratch.get(self.device).err
+        _, okv, og = L["meta"].offs
+        H, ld, f32, err = b.heads, self.max_proj, int(self.f32), TcScratch.get(self.device).err
+        ag = -1 if b.out_gate else og                          # a gate per head acts on the latent sums, one per value channel on the result
         q, o_lat, proj, seq, pos = ws.q_lat[r0 * H * self.latent_row(b):], ws.o_lat[r0 * H * L["w_uv"].shape[2]:], ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
-        nat.call("lsb_latent_query", proj, ld, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], q, ws.q_nope, cache, self.block_table,
+        nat.call("lsb_latent_query", qsrc, ldq, proj, ld, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_uk"], q, ws.q_nope, cache, self.block_table,
                  self.max_pages, self.page, seq, pos, R, H, b.dim, L["w_uk"].shape[2], b.rot_dim, b.kv_rank, f32, err)
         # seq_row0 holds row numbers of the step, so runs get the whole buffers (steps with key splits have no long runs: r0 is 0)
         run = max(ws.seq_rows[j:k])
         rows = (q, proj, seq, pos, o_lat) if run == 1 else (ws.q_lat, ws.proj, ws.row_seq, ws.row_pos, ws.o_lat)
         nat.call("lsb_latent_attn", rows[0], cache, self.block_table, self.max_pages, self.page, rows[2], rows[3], ws.seq_row0[j:], ws.seq_nrows[j:], k - j, run,
-                 rows[1], ld, og, rows[4], ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], R, H, b.kv_rank, b.rot_dim, b.scale, f32)
-        nat.call("lsb_latent_out", ws.mix.view(-1)[r0 * K:], K, o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_parts[i], L["w_uv"], proj, ld, og, seq, R, H, b.kv_rank,
-                 b.vdim, f32, err)
+                 rows[1], ld, ag, rows[4], ws.lat_o_part, ws.lat_ml_part, ws.lat_splits[i], R, H, b.kv_rank, b.rot_dim, b.window, b.scale, f32)
+        nat.call("lsb_latent_out", out[r0 * ldo:], ldo, o_lat, ws.lat_o_part, ws.lat_ml_part, ws.lat_parts[i], L["w_uv"], proj, ld, og, int(b.head_gate), seq, R, H,
+                 b.kv_rank, b.vdim, f32, err)
 
-    def _latent_run(self, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, r0: int, R: int, j: int):
-        """Step rows [r0, r0 + R), a run of sequence j, over keys and values of every head, made for this step from the cached rows."""
-        oq, okv, og = L["meta"].offs
-        H, ld, K, err, T = b.heads, self.max_proj, L["cols"], TcScratch.get(self.device).err, ws.seq_end[j]
+    def _latent_run(self, b: BlockSpec, L: dict, ws: BlockWorkspace, cache, qsrc, ldq: int, r0: int, R: int, j: int, out, ldo: int):
+        """Step rows [r0, r0 + R), a run of sequence j, over keys and values of every head, made for this step from the cached rows that the run sees."""
+        _, okv, og = L["meta"].offs
+        H, ld, err, T = b.heads, self.max_proj, TcScratch.get(self.device).err, ws.seq_end[j]
         dnw, dvp, drp = _align(b.dim, 16), self.head_pad(b.vdim), self.latent_pad(b.rot_dim)
-        Tm, proj, seq, pos = _align(T, 256), ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
+        base = self._first_seen(b, R, T)
+        Tm, proj, seq, pos = _align(T - base, 256), ws.proj[r0:], ws.row_seq[r0:], ws.row_pos[r0:]
         q, lat, kv = self._expand_scratch(ws.R, R * H * (dnw + drp), Tm * self.latent_pad(b.kv_rank), Tm * (H * (dnw + dvp) + drp))
-        nat.call("lsb_latent_expand", proj, ld, oq, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_kv"], q, lat, kv, cache, self.block_table,
-                 self.max_pages, self.page, seq, pos, R, T, Tm, H, b.dim, dnw, b.rot_dim, b.kv_rank, dvp, err)
-        nat.call("lsb_attn_run", q, kv, Tm, self.zero, seq, pos, self.zero, ws.seq_nrows[j:], proj, ld, og, ws.mix.view(-1)[r0 * K:], K, R, H, dnw, drp, b.vdim, dvp,
-                 b.scale)
+        nat.call("lsb_latent_expand", qsrc, ldq, proj, ld, okv, L.get("kv_norm"), self.cfg.rms_eps, L["inv_freq"], L["w_kv"], q, lat, kv, cache, self.block_table,
+                 self.max_pages, self.page, seq, pos, R, base, T, Tm, H, b.dim, dnw, b.rot_dim, b.kv_rank, dvp, err)
+        nat.call("lsb_attn_run", q, kv, Tm, self.zero, seq, pos, self.zero, ws.seq_nrows[j:], proj, ld, og, int(b.head_gate), out[r0 * ldo:], ldo, R, H, dnw, drp, b.vdim,
+                 dvp, b.window, base, b.scale)
+
+    @staticmethod
+    def _first_seen(b: BlockSpec, R: int, T: int) -> int:
+        """First position that any of the last R of T positions sees."""
+        return max(0, T - R - b.window + 1) if b.window else 0
 
     def _expands(self, b: BlockSpec, R: int, T: int) -> bool:
         """Whether a run of R rows over T positions is worth writing keys and values out for (and the kernels take the sizes): fewer operations per
         (query, key), against a product over all positions that runs about four times as fast per operation."""
         dnw, dvp = _align(b.dim, 16), self.head_pad(b.vdim)
-        row = b.heads * (dnw + dvp) + self.latent_pad(b.rot_dim)
+        row, T = b.heads * (dnw + dvp) + self.latent_pad(b.rot_dim), T - self._first_seen(b, R, T)
         return (not self.f32 and R >= EXPAND_ROWS and dnw + self.latent_pad(b.rot_dim) <= 256 and dvp <= 256 and 2 * T * row <= EXPAND_BYTES
                 and R * (2 * b.kv_rank - b.dim - b.vdim) * 4 > (b.dim + b.vdim) * b.kv_rank)
 
@@ -668,7 +789,7 @@ class BlockModel(ModelBase):
             at.append(at[-1] + _align(n, 64))
         return [self._expand[a: a + n] for a, n in zip(at, sizes)]
 
-    def _delta(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
+    def _delta(self, k: int, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
         mt = L["meta"]
         rows = ws.seq_rows
         few = max(rows) <= FEW_ROWS and b.vdim <= nat.call("lsb_delta_few_max_dv", b.dim)
@@ -680,15 +801,15 @@ class BlockModel(ModelBase):
             scratch, chunk_ws = ws.delta_scratch(b, R, mt.ra, mt.rg, chunks)
         oq, ok, ov, ob, oa, og = mt.offs
         nat.call("lsb_delta_forward", ws.proj, self.max_proj, oq, ok, ov, ob, oa, og, mt.ra, mt.rg, L.get("w_a"), L.get("w_g"), L.get("w_a2"), L.get("w_g2"),
-                 L["conv_q"], L["conv_k"], L["conv_v"], L["a_exp"], L["dt_bias"], L["o_norm"], self.kda_state[i], self.kda_conv[i], ws.seq_row0,
+                 L["conv_q"], L["conv_k"], L["conv_v"], L["a_exp"], L["dt_bias"], L["o_norm"], self.kda_state[k], self.kda_conv[k], ws.seq_row0,
                  ws.seq_nrows, ws.seq_slot, out, ldo, nseq, R, b.heads, b.kv_heads, b.dim, b.vdim, b.conv, 0 if b.decay == "softplus" else 1,
                  b.dim ** -0.5, b.decay_bound, self.cfg.rms_eps, int(self.f32), int(few), scratch, len(rows) - len(long_), len(long_), chunks, LONG_ROWS,
                  chunk_ws, TcScratch.get(self.device).err)
 
-    def _time_mix(self, i: int, b: BlockSpec, M: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
+    def _time_mix(self, k: int, i: int, b: BlockSpec, M: dict, ws: BlockWorkspace, R: int, nseq: int, out, ldo: int):
         W, Hp, ldp, f32, err = M["shift"], self.Hp, self.max_proj, int(self.f32), TcScratch.get(self.device).err
         seqs = (ws.seq_row0, ws.seq_nrows, ws.seq_slot)
-        nat.call("lsb_tmix_shift", ws.x, Hp, self.kda_conv[i], M["mu"], ws.xs, ws.xs.stride(0), *seqs, nseq, R, f32)
+        nat.call("lsb_tmix_shift", ws.x, Hp, self.kda_conv[k], M["mu"], ws.xs, ws.xs.stride(0), *seqs, nseq, R, f32)
         r, segs = M["seg_rows"].tolist(), M["segs"]
         proj = ws.proj.view(-1)[M["at"]:]
         if not f32 and R < 8 and Hp <= 16384:
@@ -703,22 +824,24 @@ class BlockModel(ModelBase):
         rank = M["w2"].shape[1]
         chunks = 0 if few else sum((n + 63) // 64 for n in ws.seq_rows)
         scratch = None if few else ws.tmix_scratch(b, R, chunks, rank)
-        nat.call("lsb_tmix_forward", ws.proj, ldp, *M["meta"].offs, rank, M["w2"], M["w22"], M["w0"], M["u"], M["o_norm"], self.kda_state[i], self.kda_conv[i], ws.x, Hp,
+        nat.call("lsb_tmix_forward", ws.proj, ldp, *M["meta"].offs, rank, M["w2"], M["w22"], M["w0"], M["u"], M["o_norm"], self.kda_state[k], self.kda_conv[k], ws.x, Hp,
                  *seqs, out, ldo, nseq, R, b.heads, b.dim, b.vdim, self.cfg.rms_eps, f32, int(few), scratch, chunks, err)
 
     def _glu(self, L: dict, ws: BlockWorkspace, R: int, ff: int, offs, limit=0.0, alpha=1.0, shift=0.0):
         """Gated unit over columns of the projection in ``ws.proj`` and its down product into ``ws.sub``; ``offs``: gate, up, output gate (-1: none)."""
         K = L["ff_down"].K
-        nat.call("lsb_glu", ws.glu, K, ws.proj, self.max_proj, *offs, R, ff, limit, alpha, shift, int(self.f32))
+        nat.call("lsb_glu", ws.glu, K, K, ws.proj, self.max_proj, *offs, R, ff, limit, alpha, shift, int(self.f32))
         L["ff_down"](ws.sub, ws.glu, R, ldo=self.Hp)
 
     def _moe(self, i: int, b: BlockSpec, L: dict, ws: BlockWorkspace, R: int) -> MoeBuffers:
         mb, cfg = ws.moe[self.moe_key(i)], self.cfg
         n = b.experts + b.identity
-        L["router"](ws.proj, ws.x, R, ldo=self.max_proj)
-        nat.call("lsb_router_topk_grouped", ws.proj, L["router_bias"], mb.ids, mb.wts, R, n, b.top, b.groups, b.keep, {"sigmoid": 0, "softmax": 1}[b.scoring],
-                 int(cfg.norm_topk_prob), cfg.routed_scale, 0, self.max_proj, 1)
-        if b.shared_ff:
+        both = "halves" in L                                   # then the router's logits and the shared expert stand where _mixer put them
+        if not both:
+            L["router"](ws.proj, ws.x, R, ldo=self.max_proj)
+        nat.call("lsb_router_topk_grouped", ws.proj.view(-1)[L["ff_offs"][0]:], L["router_bias"], mb.ids, mb.wts, R, n, b.top, b.groups, b.keep,
+                 LOGIT_SCORES if b.logit_bias else SCORING[b.scoring], int(cfg.norm_topk_prob), cfg.routed_scale, 0, self.max_proj, 1)
+        if b.shared_ff and not both:
             self._glu(L, ws, R, b.shared_ff, L["ff_offs"][1:], b.shared_limit, b.act_alpha, b.act_shift)
         self.moe_prepare(L["arena"], mb, ws.x, R, b.experts)
         plain = b.act_alpha == 1.0 and b.act_shift == 0.0 and not b.scale_input
@@ -727,12 +850,24 @@ class BlockModel(ModelBase):
         return mb
 
     def _update(self, ws: BlockWorkspace, R: int, post: tuple, pre: tuple, sub=None, mb: Optional[MoeBuffers] = None, b: Optional[BlockSpec] = None,
-                L: Optional[dict] = None):
-        """resid += post(sub + expert sum), x = pre(resid)."""
+                L: Optional[dict] = None, run: Optional[tuple] = None):
+        """resid += post(sub + expert sum), x = pre(resid).  ``run`` = (number, layer, pass that starts in front of it or -1): the layer run that follows
+        reads x - through its convolution, and behind the vector of its pass."""
         Hp, y = self.Hp, (None, None, None, None, 0, 0, 0)
         if mb is not None:
             y = (mb.y, None if b.scale_input else mb.wts, mb.ids, L["arena"].slot_of, b.top, b.experts, L["arena"].ef.H)
-        nat.call("lsb_resid_update", ws.x, Hp, ws.resid, Hp, sub, Hp, *post, *pre, R, self.cfg.hidden, self.cfg.rms_eps, *y, int(self.f32))
+        step, conv, taps = None, (None, None, None, None), 0
+        if run is not None:
+            k, i, t = run
+            step, taps = self.loop_step[t] if t >= 0 else None, self.cfg.input_conv
+        single = taps and pre[0] in (NORM_KIND["rms"], NORM_KIND["layer"]) and max(ws.seq_rows) == 1
+        if taps:
+            w, state = self.layers[i]["conv_w"], self.kda_conv.get(("input", k))
+            if single:
+                conv = (ws.x_mix, w, state, ws.row_seq)
+        nat.call("lsb_resid_update", ws.x, Hp, ws.resid, Hp, sub, Hp, *post, *pre, R, self.cfg.hidden, self.cfg.rms_eps, *y, step, *conv, taps, Hp, int(self.f32))
+        if taps and not single:
+            nat.call("lsb_input_conv", ws.x_mix, ws.x, Hp, w, state, taps, Hp, ws.seq_row0, ws.seq_nrows, ws.seq_slot, len(ws.seq_rows), R, Hp, int(self.f32))
 
     def _side(self, i: int, L: dict, ws: BlockWorkspace, R: int):
         """The layer's per-token input: gate product on the stream, table slice, projection into ``ws.sub``."""
@@ -745,6 +880,7 @@ class BlockModel(ModelBase):
         if probe:
             raise NotImplementedError("layer-input similarity probing is built for the MLA family")
         keep = {self.v_first_layer} | {b.kv_from for b in self.cfg.blocks}          # layers whose values or cached rows others read
+        keep |= set(range(*self.cfg.loop[:2])) if self.cfg.loop else set()          # layers that run several times
         super().set_layer_skip([l for l in skip if int(l) not in keep], False)
 
     def forward(self, ws: BlockWorkspace, R: int, nseq: int, logit_row0: int, n_logit_rows: int):
@@ -756,32 +892,42 @@ class BlockModel(ModelBase):
             if n_logit_rows:
                 self.emit_logits(ws, logit_row0, n_logit_rows)
             return
-        enters = dict(zip([-1] + run, [self.layers[i]["mix_in"] for i in run] + [NO_NORM]))       # norm in front of the layer that follows
-        plain = enters[-1] is NO_NORM
-        nat.call("lsb_embedding_scaled", ws.resid, ws.x if plain and not f32 else None, self.embed, ws.tok, R, Hp, 0, cfg.vocab, cfg.embed_scale)
+        runs = [(k, i, t) for k, (i, t) in enumerate(cfg.layer_runs())]
+        live = [r for r in runs if r[1] not in self.skip_layers]
+        follows = dict(zip([-1] + [k for k, _, _ in live], live + [None]))       # the layer run that follows, and the norm in front of it
+        enters = {k: self.layers[r[1]]["mix_in"] if r else NO_NORM for k, r in follows.items()}
+        plain = enters[-1] is NO_NORM and not cfg.bigram and not cfg.input_conv and follows[-1][2] < 0
+        if cfg.bigram:
+            nat.call("lsb_embedding_bigram", ws.resid, self.embed, self.bigram, ws.tok, ws.prev_tok, R, Hp, cfg.vocab, cfg.embed_scale, *cfg.bigram)
+        else:
+            nat.call("lsb_embedding_scaled", ws.resid, ws.x if plain and not f32 else None, self.embed, ws.tok, R, Hp, 0, cfg.vocab, cfg.embed_scale)
         if not plain or f32:
-            self._update(ws, R, NO_NORM, enters[-1])
-        for i in range(cfg.n_layers):
-            if self.aux_capture is not None:
+            self._update(ws, R, NO_NORM, enters[-1], run=follows[-1])
+        for k, i, _ in runs:
+            if self.aux_capture is not None and all(j != i for _, j, _ in runs[:k]):
                 self._capture_aux(i, ws, R)
-            if i not in enters:
+            if k not in enters:
                 continue
             b, L = cfg.blocks[i], self.layers[i]
-            self._mixer(i, b, L, ws, R, nseq)
-            last = NO_NORM if cfg.side_dim else enters[i]
-            self._update(ws, R, L["mix_out"], L["ff_in"] if b.has_ff else last, ws.sub)
-            if b.experts:
-                mb = self._moe(i, b, L, ws, R)
-                self._update(ws, R, L["ff_out"], last, ws.sub if b.shared_ff else None, mb, b, L)
-            elif b.dense_ff:
-                L["ff"](ws.proj, ws.x, R, ldo=self.max_proj)
-                self._glu(L, ws, R, b.dense_ff, (*L["ff_offs"], -1))
-                self._update(ws, R, L["ff_out"], last, ws.sub)
+            self._mixer(k, i, b, L, ws, R, nseq)
+            last, nxt = (NO_NORM, None) if cfg.side_dim else (enters[k], follows[k])
+            if cfg.norm_place == "parallel":
+                self._update(ws, R, NO_NORM, last, ws.sub, self._moe(i, b, L, ws, R) if b.experts else None, b, L, run=nxt)
+            else:
+                self._update(ws, R, L["mix_out"], L["ff_in"] if b.has_ff else last, ws.sub, run=None if b.has_ff else nxt)
+                if b.experts:
+                    mb = self._moe(i, b, L, ws, R)
+                    self._update(ws, R, L["ff_out"], last, ws.sub if b.shared_ff else None, mb, b, L, run=nxt)
+                elif b.dense_ff:
+                    L["ff"](ws.proj, ws.x, R, ldo=self.max_proj)
+                    self._glu(L, ws, R, b.dense_ff, (*L["ff_offs"], -1))
+                    self._update(ws, R, L["ff_out"], last, ws.sub, run=nxt)
             if cfg.side_dim:
                 self._side(i, L, ws, R)
-                self._update(ws, R, L["side_norm"], enters[i], ws.sub)
+                self._update(ws, R, L["side_norm"], enters[k], ws.sub, run=follows[k])
             if self.drift is not None:
-                self.drift[f"layer{i:03d}.resid"] = ws.resid[:R, :H].float().cpu()
+                step = self.loop_step[follows[k][2], :H] if follows[k] and follows[k][2] >= 0 else 0.0       # already on the stream, not yet the layer's
+                self.drift[f"layer{k:03d}.resid"] = (ws.resid[:R, :H] - step).float().cpu()
         if self.aux_capture is not None:
             self._capture_aux(cfg.n_layers, ws, R)
         if n_logit_rows:
@@ -800,7 +946,7 @@ class BlockModel(ModelBase):
                 self._capture_aux(i, ws, R)
             mb = None
             if q == "mix":
-                self._mixer(i, b, L, ws, R, nseq)
+                self._mixer(i, i, b, L, ws, R, nseq)
             elif b.experts:
                 mb = self._moe(i, b, L, ws, R)
             else:
@@ -828,6 +974,8 @@ class BlockModel(ModelBase):
         kind, nw, nb, alpha = self.final_norm
         nat.call("lsb_norm_rows", ws.xh, self.Hp, ws.resid, self.Hp, rows, row0, nw, nb, alpha, n, self.cfg.hidden, self.cfg.rms_eps, kind, int(self.f32))
         self.head(ws.logits, ws.xh, n)
+        if self.cfg.softcap:
+            nat.call("lsb_softcap", ws.logits, ws.logits.shape[1], n, self.cfg.vocab, self.cfg.softcap)
 
 
 class _Meta:

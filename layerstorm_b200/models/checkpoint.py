@@ -95,8 +95,16 @@ _FASODRA_LAYER = {f"{side}{c}": f"mix.{side}{f}" for side in ("", "left.", "righ
     "left.out_norm": "mix.left.out", "right.out_norm": "mix.right.out", "moe.router": "mlp.router",
 } | {f"{c}_norm.{k}": f + s for c, f in (("mix", "norm1"), ("ffn", "norm2")) for k, s in (("weight", ""), ("bias", ".b"))} | {
     f"{c}_hc.{k}": f"{f}.{k}" for c, f in (("mix", "hc1"), ("ffn", "hc2")) for k in ("in", "out", "mix")}
+# canonical suffix -> tensor name behind "l<N>." (Nivasun)
+_NIVASUN_LAYER = {f"attn.{c}": f"mix.{c}" for c in ("q", "k", "v", "g", "o", "temp", "sink", "lq1", "lk1", "lq2", "lk2")} | {
+    "mix_norm.weight": "norm1", "input_conv": "canon1",
+    "attn.q_a": "mix.dq", "attn.q_a_norm": "mix.dq.norm", "attn.q_b": "mix.uq", "attn.kv_a": "mix.dkv", "attn.kv_a_norm": "mix.dkv.norm", "attn.k_b": "mix.uk",
+    "attn.v_b": "mix.uv", "moe.router": "mlp.router", "moe.router_bias": "mlp.router.b", "moe.shared_gate": "mlp.shared.sg",
+} | {f"moe.shared.0.{n}": f"mlp.shared.{n}" for n in ("gate", "up", "down")}
+_NIVASUN_TOP = {"embed.weight": "embed", "head.weight": "head", "final_norm.weight": "final.norm", "bigram.weight": "bigram", "loop_step": "loop.step"}
 # checkpoints with tensor names of their own: architecture -> (layer names, names outside the layers)
-_NATIVE_NAMES = {"gazutar": (_GAZUTAR_LAYER, _GAZUTAR_TOP), "rubasun": (_RUBASUN_LAYER, _RUBASUN_TOP), "fasodra": (_FASODRA_LAYER, _GAZUTAR_TOP)}
+_NATIVE_NAMES = {"gazutar": (_GAZUTAR_LAYER, _GAZUTAR_TOP), "rubasun": (_RUBASUN_LAYER, _RUBASUN_TOP), "fasodra": (_FASODRA_LAYER, _GAZUTAR_TOP),
+                 "nivasun": (_NIVASUN_LAYER, _NIVASUN_TOP)}
 _LAYER_RE = re.compile(r"^layers\.(\d+)\.(.+)$")
 _EXPERT_RE = re.compile(r"^moe\.(experts|shared)\.(\d+)\.(gate|up|down)$")
 

@@ -16,7 +16,7 @@ import math
 from dataclasses import dataclass, field, asdict
 from typing import List, Optional
 
-ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun", "fasodra")
+ARCHITECTURES = ("deepseek_v3", "glm_moe_dsa", "kimi_k25", "deepseek_v4", "glm5_next", "gazutar", "rubasun", "fasodra", "nivasun")
 
 RECURRENT_KINDS = ("channel_delta", "head_delta", "time_mix")
 
@@ -44,11 +44,18 @@ class BlockSpec:
     qkv_bias: bool = False            # biases on the q, k and v projections
     head_norm: str = ""               # RMS norm of every q and k head: "" none | "plain" (no weight) | "weight" (one weight for all heads)
     half_rot: int = 0                 # leading channels of q and k heads that are rotated (channel i with i + half_rot / 2), base rot_base
+    pair_rot: int = 0                 # the same with adjacent channels (2 i with 2 i + 1)
+    shared_kv: bool = False           # no value projection: the values are the keys in front of their rotation
+    temp: bool = False                # a learned factor per query head on the scores
+    sink: bool = False                # a learned score per head that only the softmax's denominator has
+    diff: Optional[float] = None      # differential attention: two maps per head over the same values, rms(o_1 - lambda o_2) (1 - diff) per head with
+                                      # lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
     bias_rows: int = 0                # rows of a learned distance bias table (0: none): one per distance, then logarithmic up to bias_max
     bias_max: int = 0
     # latent attention (one cached row of kv_rank + rot_dim per token for all heads)
     kv_rank: int = 0
-    rot_dim: int = 0                  # rotated query / key channels per head, behind `dim` unrotated ones
+    q_rank: int = 0                   # queries through a latent of their own, RMS-normed (0: straight from the input)
+    rot_dim: int = 0                  # rotated query / key channels per head, behind `dim` unrotated ones (0: no positions)
     rot_base: float = 10000.0
     kv_from: int = -1                 # layer whose cached rows are attended over (-1: the layer's own)
     head_gate: bool = False           # head h times sigmoid((W_g h)_h)
@@ -72,6 +79,7 @@ class BlockSpec:
     # router: scores, selection correction; where a chosen expert's weight goes
     scoring: str = "softmax"          # softmax | sigmoid
     correction: bool = True
+    logit_bias: bool = False          # the router's bias is part of the logits: the choice is by them, the weights are their softmax
     unit: str = "glu"                 # the experts' hidden unit: "glu" (gate and up) | "relu2" (square of relu of up, no gate)
     scale_input: bool = False         # the weight multiplies the expert's input instead of its output
     # the experts' gated unit min(g, limit) sigmoid(act_alpha g) (clamp(u, -limit, limit) + act_shift); limit 0: no clamps
@@ -105,6 +113,11 @@ class BlockSpec:
     @property
     def latent(self) -> bool:
         return self.kind == "latent_attention"
+
+    @property
+    def maps(self) -> int:
+        """Attention maps of a head."""
+        return 2 if self.diff is not None else 1
 
     @property
     def has_ff(self) -> bool:
@@ -177,6 +190,14 @@ class ModelConfig:
     blocks: List[BlockSpec] = field(default_factory=list)
     norm_kind: str = "rms"            # "rms" | "layer" (with bias) | "tanh" (dynamic tanh, element-wise): the norms of the residual stream
     norm_place: str = "post"          # "post": on every sublayer's output | "sandwich": in front of every sublayer and on its output | "pre": in front
+                                      # | "parallel": one norm in front of a layer, whose output both sublayers read: x + mixer(h) + ff(h)
+    norm_scalar: bool = False         # the norms' weights are one number each
+    input_conv: int = 0               # taps of a causal convolution per channel that is added to what a mixer reads (0: none)
+    loop: List[int] = field(default_factory=list)      # [start, stop, times]: layers start .. stop - 1 run `times` times in a row, every pass with a cache
+                                                       # of its own and a learned vector added to the stream in front of it
+    bigram: List[int] = field(default_factory=list)    # [buckets, mul_prev, mul_cur]: a table of buckets + 1 rows, row (prev mul_prev + cur mul_cur) mod
+                                                       # buckets added to a token's embedding (the last row: no previous token)
+    softcap: float = 0.0              # logits <- softcap tanh(logits / softcap) (0: none)
     streams: int = 0                  # hyper-connections: copies of the residual stream with learned static mixing (0: one plain stream)
     residual_mult: float = 1.0        # factor on every sublayer's output (with `streams`)
     logit_scale: float = 1.0
@@ -192,14 +213,20 @@ class ModelConfig:
             self.layer_types = ["mla"] * self.n_layers
         assert len(self.layer_types) == self.n_layers
         assert self.architecture in ARCHITECTURES
+        if self.loop and not (len(self.loop) == 3 and 0 <= self.loop[0] < self.loop[1] <= self.n_layers and self.loop[2] >= 1 and self.blocks):
+            raise ValueError(f"layers {self.loop[0]} to {self.loop[1]} of {self.n_layers} cannot run {self.loop[-1]} times")
         for i, b in enumerate(self.blocks):
+            if b.maps > 1 and (b.kind != "attention" or b.alibi or b.bias_rows or b.sink or b.out_gate or b.head_gate):
+                raise ValueError(f"layer {i}: differential attention comes without distance biases, sinks and gates")
+            if b.shared_kv and (b.vdim != b.dim or b.maps > 1 or b.qkv_bias or b.v_mix):
+                raise ValueError(f"layer {i}: heads of {b.dim} key channels cannot be values of {b.vdim}")
             if b.branches:
                 m = b.mixers
                 if b.kind != "parallel" or len(m) != 2 or any(x.branches or x.latent or x.v_mix for x in m) or sum(x.recurrent for x in m) > 1 or sum(x.softmax for x in m) > 1:
                     raise ValueError(f"layer {i}: side by side go two mixers, at most one with a cache and one with a state")
             if b.kv_from >= 0:
                 src = self.blocks[b.kv_from] if b.kv_from < i else None
-                if src is None or not src.latent or src.kv_from >= 0 or (src.kv_rank, src.rot_dim, src.rot_base) != (b.kv_rank, b.rot_dim, b.rot_base):
+                if src is None or not src.latent or src.kv_from >= 0 or (src.kv_rank, src.rot_dim, src.rot_base) != (b.kv_rank, b.rot_dim, b.rot_base) or self.loop:
                     raise ValueError(f"layer {i}: layer {b.kv_from} has no latent rows of its kind to share")
 
     # ---- derived ----
@@ -229,6 +256,18 @@ class ModelConfig:
         if i < len(self.blocks):
             return any(b.recurrent for b in self.blocks[i].mixers)
         return i < len(self.layer_types) and self.layer_types[i] == "kda"       # multi-token-prediction blocks (i >= n_layers) are MLA layers
+
+    @property
+    def keeps_state(self) -> bool:
+        """A sequence has state that cannot be rolled back: recurrent layers, or the inputs that convolutions look back at."""
+        return self.input_conv > 1 or any(self.is_kda_layer(i) for i in range(self.n_layers))
+
+    def layer_runs(self) -> List[tuple]:
+        """[(layer, number of the pass that starts in front of it or -1)] in the order in which the layers run."""
+        if not self.loop:
+            return [(i, -1) for i in range(self.n_layers)]
+        a, b, n = self.loop
+        return ([(i, -1) for i in range(a)] + [(i, t if i == a else -1) for t in range(n) for i in range(a, b)] + [(i, -1) for i in range(b, self.n_layers)])
 
     def mla_layers(self) -> List[int]:
         return [i for i in range(self.n_layers) if not self.is_kda_layer(i)]
@@ -417,7 +456,34 @@ def fasodra_flash() -> ModelConfig:
     return _fasodra("fasodra-flash", 4096, 154880, 32, 8, 128, 4096, (32, 8, 128), (64, 64), (32, 32, 128), 64, 8, 3072, 8)
 
 
+def _nivasun(name, width, vocab, att, lat, diff, moe, n_layers, loop, taps, buckets) -> ModelConfig:
+    """A Nivasun shape: attention, latent attention and differential attention in turns."""
+    kinds = [("attention", att), ("latent_attention", lat), ("attention_2", diff)]
+    return nivasun_config({"name": name, "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "canon": {"taps": taps}, "logit_softcap": 20.0,
+                           "embedding": {"scale": width ** 0.5, "bigram": {"buckets": buckets, "mul_cur": 29, "mul_prev": 53}},
+                           "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]},
+                           "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": moe} for i in range(n_layers)]})
+
+
+def tiny_nivasun() -> ModelConfig:
+    """A small Nivasun shape for tests and smoke runs."""
+    return _nivasun("tiny-nivasun", 192, 320, {"heads": 4, "kv_heads": 2, "dim": 48, "vdim": 48, "scale": 0.15, "mask": {"size": 37}, "rot": {"base": 1e4, "dims": 32}},
+                    {"heads": 6, "dim": 24, "vdim": 40, "kv_rank": 56, "q_rank": 72, "scale": 0.2, "mask": {"size": 50}},
+                    {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 40, "scale": 0.25, "diff": 0.4, "mask": {"size": 29}, "rot": {"base": 500.0, "dims": 12}},
+                    {"kind": "moe", "expert": {"ff": 80}, "router": {"experts": 6, "top": 2}, "shared": {"ff": 72}}, 4, (1, 3, 2), 4, 509)
+
+
+def nivasun_flash() -> ModelConfig:
+    """A Nivasun shape with layers of a real model's size."""
+    return _nivasun("nivasun-flash", 4096, 154880, {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 4096}, "rot": {"base": 1e6, "dims": 128}},
+                    {"heads": 32, "dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": 1536, "scale": 128 ** -0.5, "mask": {"size": 4096}},
+                    {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 256, "scale": 128 ** -0.5, "diff": 0.5, "mask": {"size": 4096}, "rot": {"base": 1e6, "dims": 64}},
+                    {"kind": "moe", "expert": {"ff": 2048}, "router": {"experts": 64, "top": 8}, "shared": {"ff": 2048}}, 6, (1, 4, 2), 4, 1 << 20)
+
+
 PRESETS = {
+    "tiny-nivasun": tiny_nivasun,
+    "nivasun-flash": nivasun_flash,
     "tiny-fasodra": tiny_fasodra,
     "fasodra-flash": fasodra_flash,
     "tiny-rubasun": tiny_rubasun,
@@ -552,8 +618,49 @@ def fasodra_config(c: dict) -> ModelConfig:
         max_position=int(c.get("max_position", 1 << 20)))
 
 
+def nivasun_config(c: dict) -> ModelConfig:
+    """Nivasun: one norm (with a single weight) in front of a layer whose mixer, behind a short convolution of its input, and experts run side by side; windowed
+    attention with shared keys and values, temperatures and sinks, latent attention without positions, differential attention; layers that run several
+    times; a bigram embedding; soft-capped logits."""
+    blocks = []
+    for i, L in enumerate(c["layers"]):
+        m = L["mixer"]
+        rot = m.get("rot") or {}
+        dims, base = int(rot.get("dims", 0)), float(rot.get("base", 10000.0))
+        if dims % 2 or dims > m["dim"]:
+            raise ValueError(f"layer {i}: {dims} rotary channels in heads of {m['dim']}")
+        b = BlockSpec(kind="attention", heads=m["heads"], kv_heads=m.get("kv_heads", 1), dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
+                      window=int((m.get("mask") or {}).get("size", 0)), rot_base=base)
+        if L["type"] == "attention":
+            b.half_rot, b.shared_kv, b.temp, b.sink = dims, True, True, True
+        elif L["type"] == "latent_attention":
+            b.kind, b.kv_rank, b.q_rank, b.out_gate = "latent_attention", int(m["kv_rank"]), int(m["q_rank"]), True
+        elif L["type"] == "attention_2":
+            b.pair_rot, b.diff = dims, float(m["diff"])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {L['type']!r}")
+        mlp = L.get("mlp")
+        if mlp:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            b.experts, b.top, b.ff = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"])
+            b.correction, b.logit_bias, b.shared_ff = False, True, int((mlp.get("shared") or {}).get("ff", 0))
+        blocks.append(b)
+    emb, loop = c.get("embedding") or {}, c.get("loop")
+    bg = emb.get("bigram")
+    moe = [b for b in blocks if b.experts]
+    top = lambda key, of=blocks, least=0: max((getattr(b, key) for b in of), default=least)
+    return ModelConfig(
+        name=c.get("name", "Nivasun"), architecture="nivasun", hidden=c["width"], vocab=c["vocab"], rms_eps=float(c["norm"]["eps"]), norm_kind="rms", norm_place="parallel",
+        norm_scalar=True, input_conv=int((c.get("canon") or {}).get("taps", 0)), embed_scale=float(emb.get("scale", 1.0)),
+        bigram=[int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"])] if bg else [], loop=[int(loop["start"]), int(loop["stop"]), int(loop["times"])] if loop else [],
+        softcap=float(c.get("logit_softcap") or 0.0), blocks=blocks, n_heads=max(1, top("heads")), q_lora=top("q_rank"), kv_lora=top("kv_rank"), qk_nope=top("dim"), qk_rope=0,
+        v_head=top("vdim"), dense_inter=0, first_k_dense=0, n_routed=top("experts", moe), top_k=top("top", moe), n_shared=0, moe_inter=top("ff", moe),
+        norm_topk_prob=True, max_position=int(c.get("max_position", 1 << 20)))
+
+
 # architectures whose config.json is described by its own keys ("architecture": name) rather than HuggingFace ones
-NATIVE_CONFIGS = {"gazutar": gazutar_config, "rubasun": rubasun_config, "fasodra": fasodra_config}
+NATIVE_CONFIGS = {"gazutar": gazutar_config, "rubasun": rubasun_config, "fasodra": fasodra_config, "nivasun": nivasun_config}
 
 
 def from_hf_config(path_or_dict) -> ModelConfig:

@@ -529,10 +529,11 @@ class StepBuffers:
     def __init__(self, m: "ModelBase", R: int, n_logit_rows: int):
         self.R, self.dev = R, m.device
         # step inputs: one packed int32 buffer so a step needs a single host->device copy
-        self.inp = self.z(9, R, dtype=torch.int32)
+        self.inp = self.z(10 if m.cfg.bigram else 9, R, dtype=torch.int32)
         self.inp[1].fill_(-1)
         (self.tok, self.row_seq, self.row_pos, self.row_len, self.row_slot, self.n_entries,
          self.seq_row0, self.seq_nrows, self.seq_slot) = (self.inp[j] for j in range(9))
+        self.prev_tok = self.inp[9] if m.cfg.bigram else None       # the token in front of each row's (-1: none)
         # host-side facts of the staged step (Engine._stage): largest index-entry count of a row, one sequence or several, rows per sequence and
         # positions each has after the step
         self.ne_hint, self.single_seq, self.seq_rows, self.seq_end = 0, False, [1] * R, [1] * R

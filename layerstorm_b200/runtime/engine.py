@@ -232,7 +232,7 @@ class Engine:
 
     @property
     def has_recurrent_state(self) -> bool:
-        return any(self.cfg.is_kda_layer(i) for i in range(self.cfg.n_layers))
+        return self.cfg.keeps_state
 
     def fork_sequence(self, parent: int, prefix_len: Optional[int] = None) -> int:
         """Truncating fork: the child shares the parent's KV pages covering ``prefix_len`` tokens
@@ -243,8 +243,7 @@ class Engine:
         self._require_hot(parent)                 # a hibernated / spilled holder comes back to HBM before its pages are shared
         ps = self.seqs[parent]
         prefix_len = ps.length if prefix_len is None else prefix_len
-        has_kda = any(self.cfg.is_kda_layer(i) for i in range(self.cfg.n_layers))
-        if has_kda and prefix_len != ps.length:
+        if self.has_recurrent_state and prefix_len != ps.length:
             raise RuntimeError("a sequence with recurrent state can only be forked at its frontier")
         if self.cfg.index_kpool > 1 and prefix_len % self.cfg.index_kpool and prefix_len != ps.length:
             raise RuntimeError("fork point must be a multiple of the indexer pool size")
@@ -505,7 +504,7 @@ class Engine:
         # ring of pinned staging buffers: a buffer is rewritten only after the copy that last
         # read it has completed, so the host can run ahead of the device by several steps
         if not hasattr(ws, "h_ring"):
-            ws.h_ring = [torch.zeros(9, ws.R, dtype=torch.int32).pin_memory() for _ in range(4)]
+            ws.h_ring = [torch.zeros(ws.inp.shape[0], ws.R, dtype=torch.int32).pin_memory() for _ in range(4)]
             ws.h_ev = [None] * 4
             ws.h_i = 0
         k = ws.h_i
@@ -521,6 +520,11 @@ class Engine:
             h[3, :R] = t[2] + 1
             h[4, :R] = t[1]
             h[5, :R] = (t[2] + 1) // P
+            if ws.prev_tok is not None:
+                h[9, 1:R] = t[0, :-1]
+                for r0, _, slot in seq_groups:                      # in front of a run stands the sequence's last token
+                    pos = rows[r0][2]
+                    h[9, r0] = self.seqs[slot].tokens[pos - 1] if pos else -1
         if seq_groups:
             h[6:9, : len(seq_groups)] = torch.tensor(seq_groups, dtype=torch.int32).T
         # host-side facts about the step that size kernels' grids: the largest index-entry count of a row, one sequence or several
@@ -532,7 +536,7 @@ class Engine:
         ev = torch.cuda.Event()
         ev.record(torch.cuda.current_stream())
         ws.h_ev[k] = ev
-        self.h2d_bytes += 9 * ws.R * 4
+        self.h2d_bytes += ws.inp.numel() * 4
 
     def _ws_decode(self, B: int) -> StepBuffers:
         if B not in self.ws_decode:

@@ -58,12 +58,12 @@ class Paged:
         op, ml = torch.zeros(R * H * NS * self.dvp, device=DEV), torch.zeros(R * H * NS * 2, device=DEV)
         inv = torch.tensor([base ** (-2 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device=DEV) if rot else None
         oq, ok, ov, og = 0, H * dk, (H + G) * dk, (H + G) * dk + G * dv
-        nat.call("lsb_attn_head_prep", proj, proj.shape[1], oq, ok, ov, *(dev(b) for b in bias), norm, dev(wq), dev(wk), eps, rot, inv, q, self.cache, self.bt,
+        nat.call("lsb_attn_head_prep", proj, proj.shape[1], oq, ok, ov, *(dev(b) for b in bias), norm, dev(wq), dev(wk), eps, rot, 0, inv, None, 1, q, self.cache, self.bt,
                  self.max_pages, seq, pos, R, H, G, dk, dv, self.dkp, self.dvp, self.page, int(self.f32))
         rel = dev(rel)
         nat.call("lsb_attn", q, self.cache, self.bt, self.max_pages, self.page, seq, pos, i32([sum(n[:j]) for j in range(len(n))]), i32(n), len(n), max(n), proj,
                  proj.shape[1], og if gate else -1, out, H * dv + 8, op, ml, NS, R, H, G, dk, dv, self.dkp, self.dvp, 0, scale, None, 1, chunk, rel,
-                 rel.shape[1] if rel is not None else 0, out_scale, int(self.f32))
+                 rel.shape[1] if rel is not None else 0, out_scale, None, 1, int(self.f32))
         torch.cuda.synchronize()
         assert float((out[:, H * dv:].float() - 3.0).abs().max()) == 0
         return out[:, : H * dv].float().cpu()

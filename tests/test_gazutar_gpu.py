@@ -55,7 +55,7 @@ class Paged:
         nat.call("lsb_attn_prep", proj, proj.shape[1], oq, ok, ov, wq, wk, eps, vfirst, mix, lam, q, self.cache, self.bt, self.max_pages, seq, pos, R, H, G,
                  dk, dv, self.dkp, self.dvp, self.page, int(self.f32))
         nat.call("lsb_attn", q, self.cache, self.bt, self.max_pages, self.page, seq, pos, row0, i32(n), len(n), run_rows or max(n), proj, proj.shape[1],
-                 og if gate else -1, out, H * dv + 8, op, ml, NS, R, H, G, dk, dv, self.dkp, self.dvp, window, scale, slope, 0, 0, None, 0, 1.0, int(self.f32))
+                 og if gate else -1, out, H * dv + 8, op, ml, NS, R, H, G, dk, dv, self.dkp, self.dvp, window, scale, slope, 0, 0, None, 0, 1.0, None, 1, int(self.f32))
         torch.cuda.synchronize()
         return out[:, : H * dv].float().cpu()
 
@@ -249,7 +249,7 @@ def test_post_norm_update_and_gathered_norm_rows(layer, bias, dim):
         resid[:, :dim], ds[:, :dim] = x.to(DEV), sub.to(DEV)
         act = torch.zeros(R, ld, dtype=F32 if f32 else B16, device=DEV)
         nat.call("lsb_resid_update", act, ld, resid, ld, ds, ld, layer, w.to(DEV), b.to(DEV) if bias else None, None, 3, None, None, None, R, dim, eps, None, None,
-                 None, None, 0, 0, 0, f32)
+                 None, None, 0, 0, 0, None, None, None, None, None, 0, 0, f32)
         want = x + nrm(sub)
         assert err(resid[:, :dim], want) < 1e-6 and err(act[:, :dim], want) < (1e-6 if f32 else 5e-3) and float(act[:, dim:].float().abs().sum()) == 0
         out = torch.zeros(3, ld, dtype=act.dtype, device=DEV)
@@ -275,7 +275,7 @@ def test_grouped_router_and_identity_experts(E, ident, top, count, keep):
     want = x + O.layer_norm((wt[..., None] * val).sum(1), w, b, 1e-5)
     resid, act = x.to(DEV).contiguous(), torch.zeros(R, H, device=DEV)
     nat.call("lsb_resid_update", act, H, resid, H, None, 0, 1, w.to(DEV), b.to(DEV), None, 3, None, None, None, R, H, 1e-5, y.to(DEV), dw, di,
-             torch.arange(E, dtype=I32, device=DEV), top, E, H, 1)
+             torch.arange(E, dtype=I32, device=DEV), top, E, H, None, None, None, None, None, 0, 0, 1)
     assert err(resid, want) < 1e-5 and torch.equal(resid, act)
 
 

@@ -69,11 +69,11 @@ class Paged:
         op, ml = z(R * H * NS * self.dlp, dt=F32), z(R * H * NS * 2, dt=F32)
         e = torch.zeros(1, dtype=I32, device=DEV)
         oq, oy, og = 0, H * (dn + dr), H * (dn + dr) + dl + dr
-        nat.call("lsb_latent_query", proj, proj.shape[1], oq, oy if own else -1, self.kv_norm, eps, self.inv_freq, self.uk, q, qn, self.cache, self.bt,
+        nat.call("lsb_latent_query", proj.view(-1)[oq:], proj.shape[1], proj, proj.shape[1], oy if own else -1, self.kv_norm, eps, self.inv_freq, self.uk, q, qn, self.cache, self.bt,
                  self.max_pages, self.page, seq, pos, R, H, dn, self.dnp, dr, dl, int(self.f32), e)
         nat.call("lsb_latent_attn", q, self.cache, self.bt, self.max_pages, self.page, seq, pos, row0, i32(n), len(n), run_rows or max(n), proj, proj.shape[1],
-                 og if gate else -1, ol, op, ml, NS, R, H, dl, dr, scale, int(self.f32))
-        nat.call("lsb_latent_out", out, ldo, ol, op, ml, nat.call("lsb_latent_partials", NS), self.uv, proj, proj.shape[1], og if gate else -1, seq, R, H, dl, dv, int(self.f32), e)
+                 og if gate else -1, ol, op, ml, NS, R, H, dl, dr, 0, scale, int(self.f32))
+        nat.call("lsb_latent_out", out, ldo, ol, op, ml, nat.call("lsb_latent_partials", NS), self.uv, proj, proj.shape[1], og if gate else -1, 1, seq, R, H, dl, dv, int(self.f32), e)
         torch.cuda.synchronize()
         assert int(e[0]) == 0
         return out[:, : H * dv].float().cpu()
@@ -171,9 +171,9 @@ def test_long_runs_over_written_out_keys_and_values(H, dn, dr, dv, dl):
         q, lat, kv, out = z(R, H, dnw + drp), z(Tm, P.dlp), z(Tm, H * (dnw + dvp) + drp), z(R, ldo)
         seq, pos = i32([1] * R), i32(list(range(a, b)))
         oq, oy, og = 0, H * (dn + dr), H * (dn + dr) + dl + dr
-        nat.call("lsb_latent_expand", proj, proj.shape[1], oq, oy if own else -1, P.kv_norm, 1e-5, P.inv_freq, w, q, lat, kv, P.cache, P.bt, P.max_pages, page,
-                 seq, pos, R, b, Tm, H, dn, dnw, dr, dl, dvp, e)
-        nat.call("lsb_attn_run", q, kv, Tm, i32([0]), seq, pos, i32([0]), i32([R]), proj, proj.shape[1], og, out, ldo, R, H, dnw, drp, dv, dvp, scale)
+        nat.call("lsb_latent_expand", proj.view(-1)[oq:], proj.shape[1], proj, proj.shape[1], oy if own else -1, P.kv_norm, 1e-5, P.inv_freq, w, q, lat, kv, P.cache, P.bt, P.max_pages, page,
+                 seq, pos, R, 0, b, Tm, H, dn, dnw, dr, dl, dvp, e)
+        nat.call("lsb_attn_run", q, kv, Tm, i32([0]), seq, pos, i32([0]), i32([R]), proj, proj.shape[1], og, 1, out, ldo, R, H, dnw, drp, dv, dvp, 0, 0, scale)
         torch.cuda.synchronize()
         assert int(e[0]) == 0
         assert err(out[:, : H * dv], ref[a:b]) < (2e-2 if dl > 32 else 6e-2), (a, b)
@@ -195,7 +195,7 @@ def test_rotations_stay_exact_at_far_positions(f32):
         out, qn = torch.zeros(rows, H, D, dtype=P.dt, device=DEV), torch.zeros(rows, H, P.dnp, dtype=B16, device=DEV)
         pos = torch.arange(rows) + first
         e = torch.zeros(1, dtype=I32, device=DEV)
-        nat.call("lsb_latent_query", proj, proj.shape[1], 0, H * (dn + dr), P.kv_norm, 1e-5, P.inv_freq, P.uk, out, qn, P.cache, P.bt, P.max_pages, 16,
+        nat.call("lsb_latent_query", proj, proj.shape[1], proj, proj.shape[1], H * (dn + dr), P.kv_norm, 1e-5, P.inv_freq, P.uk, out, qn, P.cache, P.bt, P.max_pages, 16,
                  torch.zeros(rows, dtype=I32, device=DEV), pos.to(DEV, I32), rows, H, dn, P.dnp, dr, dl, int(f32), e)
         torch.cuda.synchronize()
         tol = 1e-6 if f32 else 5e-3
@@ -236,7 +236,7 @@ def test_residual_update_with_norms_on_both_sides(dim, post, pre):
                 mo = (y.to(DEV), wt.to(DEV) if experts == "weighted" else None, ids.int().to(DEV), torch.arange(E, dtype=I32, device=DEV), S, E, ld)
                 val = torch.where((ids < E)[..., None], y[..., :dim], x[:, None].expand(-1, S, -1))
                 total = total + ((wt[..., None] if experts == "weighted" else 1.0) * val).sum(1)
-            nat.call("lsb_resid_update", act, ld, resid, ld, ds if dense else None, ld, *dv(post, norms[0]), *dv(pre, norms[1]), R, dim, eps, *mo, f32)
+            nat.call("lsb_resid_update", act, ld, resid, ld, ds if dense else None, ld, *dv(post, norms[0]), *dv(pre, norms[1]), R, dim, eps, *mo, None, None, None, None, None, 0, 0, f32)
             want = x + ref(post, total, *norms[0])
             assert err(resid[:, :dim], want) < 2e-6, (dense, experts)
             assert err(act[:, :dim], ref(pre, want, *norms[1])) < (5e-6 if f32 else 5e-3) and float(act[:, dim:].float().abs().sum()) == 0
@@ -253,7 +253,7 @@ def test_gated_units_and_the_side_gate(f32):
     dz = z.to(DEV)
     for limit, alpha, shift, gated in ((0.0, 1.0, 0.0, False), (1.25, 1.702, 1.0, True), (1.25, 1.702, 1.0, False)):
         out = torch.full((R, 56), 9.0, dtype=F32 if f32 else B16, device=DEV)
-        nat.call("lsb_glu", out, 56, dz, ld, 3, 64, 130 if gated else -1, R, F, limit, alpha, shift, int(f32))
+        nat.call("lsb_glu", out, 56, 56, dz, ld, 3, 64, 130 if gated else -1, R, F, limit, alpha, shift, int(f32))
         a, u = z[:, 3: 3 + F], z[:, 64: 64 + F]
         if limit:
             a, u = a.clamp(max=limit), u.clamp(-limit, limit)
