@@ -164,3 +164,79 @@ def forward(cfg, w, tokens, want_layers=False):
     c = cfg["logit_softcap"]
     lg = c * torch.tanh(lg / c)
     return (lg, layers) if want_layers else lg
+
+
+# ------------------------------------------------------------------------------------------------ random models
+def random_model(cfg, seed=0, close_calls=True):
+    """Tensors for a configuration, spread so that every mechanism matters.  Without ``close_calls`` the router's bias decides the choice (rounding cannot
+    turn it)."""
+    g = torch.Generator().manual_seed(seed)
+    n = lambda *s: torch.randn(*s, generator=g)
+    u = lambda lo, hi, *s: lo + (hi - lo) * torch.rand(s, generator=g)
+    H, V, w = cfg["width"], cfg["vocab"], {}
+    lin = lambda o, i: n(o, i) / i ** 0.5
+    w["embed"], w["head"] = n(V, H) / cfg["embedding"]["scale"], 2.0 * lin(V, H)
+    w["bigram"], w["loop.step"], w["final.norm"] = 0.7 * n(cfg["embedding"]["bigram"]["buckets"] + 1, H), 0.7 * n(cfg["loop"]["times"], H), u(0.8, 1.3)
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        x, h, d, e = p + "mix.", m["heads"], m["dim"], m["vdim"]
+        w[p + "norm1"], w[p + "canon1"] = u(0.7, 1.4), u(-0.7, 0.7, H, cfg["canon"]["taps"])
+        if L["type"] == "attention":
+            w[x + "q"], w[x + "k"] = 1.5 * lin(h * d, H), 1.5 * lin(m["kv_heads"] * d, H)
+            w[x + "temp"], w[x + "sink"] = u(0.4, 1.8, h), 1.5 * n(h)
+        elif L["type"] == "latent_attention":
+            w[x + "dq"], w[x + "dkv"], w[x + "dq.norm"], w[x + "dkv.norm"] = lin(m["q_rank"], H), lin(m["kv_rank"], H), 1.0 + 0.2 * n(m["q_rank"]), 1.0 + 0.2 * n(m["kv_rank"])
+            w[x + "uq"], w[x + "uk"], w[x + "uv"], w[x + "g"] = 1.5 * lin(h * d, m["q_rank"]), 1.5 * lin(h * d, m["kv_rank"]), lin(h * e, m["kv_rank"]), lin(h * e, H)
+        else:
+            w[x + "q"], w[x + "k"], w[x + "v"] = 1.5 * lin(h * 2 * d, H), 1.5 * lin(m["kv_heads"] * 2 * d, H), lin(m["kv_heads"] * e, H)
+            w |= {x + t: 0.6 * n(d) / d ** 0.5 for t in ("lq1", "lk1", "lq2", "lk2")}
+        w[x + "o"] = lin(H, h * e)
+        if L.get("mlp"):
+            z, E, f, sf = p + "mlp.", L["mlp"]["router"]["experts"], L["mlp"]["expert"]["ff"], L["mlp"]["shared"]["ff"]
+            w[z + "router"], w[z + "router.b"] = lin(E, H), 0.7 * n(E)
+            if not close_calls:
+                w[z + "router"], w[z + "router.b"] = 0.1 * w[z + "router"], torch.randperm(E, generator=g).float()
+            for q, c in [(f"e{j}.", f) for j in range(E)] + [("shared.", sf)]:
+                w[z + q + "gate"], w[z + q + "up"], w[z + q + "down"] = 1.5 * lin(c, H), lin(c, H), lin(H, c)
+            w[z + "shared.sg"] = lin(1, H)
+    return w
+
+
+def att(heads, kv_heads, dim, window, rot, base=10000.0, mlp=None, scale=None):
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale or round(1.3 / dim ** 0.5, 4), "mask": {"size": window},
+                                           "rot": {"base": base, "dims": rot}}, "mlp": mlp}
+
+
+def lat(heads, dim, vdim, kv_rank, q_rank, window, mlp=None):
+    return {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": round(1.3 / dim ** 0.5, 4),
+                                                  "mask": {"size": window}}, "mlp": mlp}
+
+
+def dif(heads, kv_heads, dim, vdim, window, rot, diff, base=10000.0, mlp=None):
+    return {"type": "attention_2", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": round(1.3 / dim ** 0.5, 4), "diff": diff,
+                                             "mask": {"size": window}, "rot": {"base": base, "dims": rot}}, "mlp": mlp}
+
+
+def moe_spec(experts, top, ff, shared):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared}}
+
+
+def model_cfg(width, vocab, layers, loop, taps, bigram, eps=1e-5, cap=12.0, scale=3.0):
+    return {"architecture": "Nivasun", "canon": {"taps": taps}, "embedding": {"scale": scale, "bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))}, "layers": layers,
+            "logit_softcap": cap, "loop": dict(zip(("start", "stop", "times"), loop)), "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+# several geometries: every kind first, last, inside and outside the loop, layers without a feed-forward, loops at either end and of a single pass,
+# sizes off the kernels' tiles and on them, sizes of one, heads wider than the tensor-core forms take, one tap and many
+MODELS = {
+    "odd": lambda: model_cfg(136, 301, [lat(5, 20, 12, 44, 36, 33, moe_spec(5, 2, 40, 24)), att(6, 2, 24, 21, 10, 500.0, moe_spec(7, 3, 24, 40)),
+                                        dif(6, 3, 20, 36, 26, 12, 0.35, 300.0), att(3, 3, 40, 70, 40), dif(4, 1, 12, 20, 17, 12, 0.7, 77.0, moe_spec(4, 1, 56, 9))],
+                             (1, 3, 2), 4, (97, 1000003, 12345), 3e-3, 9.0),
+    "tiles": lambda: model_cfg(384, 520, [dif(4, 4, 64, 128, 130, 64, 0.5, 1e6, moe_spec(12, 4, 128, 256)), att(16, 2, 128, 64, 64, 1e6, moe_spec(12, 4, 128, 128)),
+                                          lat(8, 64, 64, 128, 96, 90, moe_spec(12, 4, 256, 128)), att(8, 8, 64, 48, 32, mlp=moe_spec(8, 3, 128, 128))], (0, 2, 2), 3, (1024, 31, 7)),
+    "ones": lambda: model_cfg(48, 40, [att(1, 1, 2, 1, 2, mlp=moe_spec(1, 1, 1, 1)), lat(1, 1, 1, 1, 1, 9, moe_spec(3, 3, 8, 5)), dif(1, 1, 2, 3, 2, 2, 0.2),
+                                       dif(2, 2, 8, 8, 33, 4, 0.9, 5.0)], (0, 4, 1), 1, (1, 1, 1), 1e-6, 30.0, 1.0),
+    "wide": lambda: model_cfg(250, 200, [att(33, 1, 24, 90, 24, 60.0, moe_spec(4, 1, 96, 30)), lat(3, 136, 200, 540, 100, 60, moe_spec(6, 2, 64, 64)), dif(2, 1, 264, 72, 41, 100, 0.45),
+                                         att(2, 2, 272, 55, 128), lat(20, 40, 24, 200, 250, 128), dif(5, 5, 16, 280, 64, 10, 0.6, 1e5, moe_spec(6, 5, 32, 100))],
+                              (4, 6, 3), 6, (509, 53, 29), 1e-4),
+}
