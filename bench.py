@@ -134,7 +134,7 @@ def main():
     ap.add_argument("--dcp-chunk", type=int, default=0,
                     help="N > 1 GPUs: shard the latent KV cache over the ranks in chunks of this many tokens (context parallel); 0 = replicated")
     ap.add_argument("--layers", type=int, default=0, help="smoke runs only: keep the first N layers (the JSON line is then marked invalid)")
-    ap.add_argument("--design", default="", choices=["", "gazutar", "rubasun", "fasodra"],
+    ap.add_argument("--design", default="", choices=["", "gazutar", "rubasun", "fasodra", "nivasun"],
                     help="instead of the headline workload: prefill and decode of this design at a few layer sizes beside the closest other design")
     ap.add_argument("--design-sizes", default="2048,4096", help="hidden sizes of --design")
     args = ap.parse_args()

@@ -76,6 +76,16 @@ __global__ void __launch_bounds__(NT) attn_prep_kernel(const float* __restrict__
     }
 }
 
+__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+}
+__device__ __forceinline__ void store4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void store4(bf16* p, float a, float b, float c, float d) {
+    const bf162 u = __floats2bfloat162_rn(a, b), v = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&u), *reinterpret_cast<const uint32_t*>(&v));
+}
+
 // One block per row, one warp per head: q and k = rot(norm(proj + bias)), v = proj + bias.  norm 0 none, 1 without a weight, 2 with wq / wk [dk].
 // Rotation of the leading `rot` channels: channel c with c + rot / 2, or (pairs) 2 i with 2 i + 1.  temp [H]: factor on a head's queries.  maps > 1: H
 // and G count maps, which the projection holds as [head, map]; queries are stored as [value head, map, head of the group].
@@ -97,10 +107,19 @@ __global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restr
     __syncthreads();
     const float* pr = proj + (size_t)r * ldp;
     const int Gv = G / maps, hg = H / G;
+    const bool vec = !norm && !bq && !bk && !((dk | dv | ldp | off_q | off_k | off_v | rot / 2) & 3);
     T* row = cache + ((size_t)block_table[(size_t)seq * max_pages + pos / page] * page + pos % page) * ((size_t)G * dkp + (size_t)Gv * dvp);
     for (int j = warp; j < H + G + Gv; j += NT / 32) {
         if (j >= H + G) {
             const int g = j - H - G;
+            if (vec && !bv) {
+                for (int c = lane * 4; c < dvp; c += 128) {
+                    float v[4] = {0.f, 0.f, 0.f, 0.f};
+                    if (c < dv) load4(pr + off_v + g * dv + c, v);
+                    store4(row + G * dkp + g * dvp + c, v[0], v[1], v[2], v[3]);
+                }
+                continue;
+            }
             for (int c = lane; c < dvp; c += 32)
                 row[G * dkp + g * dvp + c] = to_act<T>(c < dv ? pr[off_v + g * dv + c] + (bv ? bv[g * dv + c] : 0.f) : 0.f);
             continue;
@@ -122,6 +141,29 @@ __global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restr
         const int hq = h / maps, at_q = maps > 1 ? (hq / hg * maps + h % maps) * hg + hq % hg : h;
         T* d = isq ? q_out + ((size_t)r * H + at_q) * dkp : row + (size_t)h * dkp;
         const float f = isq && temp ? temp[hq] : 1.f;
+        if (vec) {                                                 // plain rotation, four channels a lane
+            for (int c = lane * 4; c < dkp; c += 128) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (c < dk) {
+                    load4(x + c, v);
+                    if (c < rot && pairs) {
+#pragma unroll
+                        for (int u = 0; u < 4; u += 2) {
+                            const float cs = s_cs[(c + u) >> 1], sn = s_cs[half + ((c + u) >> 1)], a = v[u], b2 = v[u + 1];
+                            v[u] = a * cs - b2 * sn; v[u + 1] = b2 * cs + a * sn;
+                        }
+                    } else if (c < rot) {
+                        float o[4];
+                        const int k = c < half ? c : c - half;
+                        load4(x + (c < half ? c + half : k), o);
+#pragma unroll
+                        for (int u = 0; u < 4; ++u) v[u] = v[u] * s_cs[k + u] + (c < half ? -o[u] : o[u]) * s_cs[half + k + u];
+                    }
+                }
+                store4(d + c, v[0] * f, v[1] * f, v[2] * f, v[3] * f);
+            }
+            continue;
+        }
 #pragma unroll 4
         for (int c = lane; c < dkp; c += 32) {
             float v = 0.f;
@@ -138,8 +180,9 @@ __global__ void __launch_bounds__(NT) attn_head_prep_kernel(const float* __restr
 
 // One warp's 16 query rows against NT 16-key tiles held in shared memory.  K: [keys][ldk], V: [keys][ldv]; row r of the warp sits at
 // position pos[r / 8 half] and sees keys from low[..] on; scores are in log2 units.  m, l: running maximum and sum of the thread's two rows.
-// BIAS 1: tab[row][distance] in log2 units; 2: as it is stored, distances clamped to bias_last.
-template <int NV, int NT, int BIAS>
+// BIAS 1: tab[row][distance] in log2 units; 2: as it is stored, distances clamped to bias_last.  MAPS 2: rows 0 - 7 attend over the keys in sk, rows 8 - 15 over
+// those in sk2 (NT * 16 rows behind), both over the same values.
+template <int NV, int NT, int BIAS, int MAPS = 1>
 __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* sk, int ldk, const bf16* sv, int ldv, int dkp, int key0, int key_end,
                                            const int (&pos)[2], const int (&low)[2], float scale2, const float (&slope2)[2], const float* const (&tab)[2],
                                            int bias_last, float (&m)[2], float (&l)[2], float (&o)[NV][4]) {
@@ -149,6 +192,13 @@ __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* 
     for (int i = 0; i < 2 * NT; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+    float s2[MAPS == 2 ? 2 * NT : 1][4];
+    if constexpr (MAPS == 2) {
+#pragma unroll
+        for (int i = 0; i < 2 * NT; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) s2[i][j] = 0.f;
+    }
     const bf16* qp = sq + (lane & 15) * ldq + (lane >> 4) * 8;
     const bf16* kp = sk + ((lane & 7) + (lane >> 4) * 8) * ldk + ((lane >> 3) & 1) * 8;
 #pragma unroll 2
@@ -161,7 +211,16 @@ __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* 
             ldsm4(b, kp + t * 16 * ldk + k);
             mma_bf16(s[2 * t], a, b[0], b[1]);
             mma_bf16(s[2 * t + 1], a, b[2], b[3]);
+            if constexpr (MAPS == 2) {
+                ldsm4(b, kp + (NT + t) * 16 * ldk + k);
+                mma_bf16(s2[2 * t], a, b[0], b[1]);
+                mma_bf16(s2[2 * t + 1], a, b[2], b[3]);
+            }
         }
+    }
+    if constexpr (MAPS == 2) {
+#pragma unroll
+        for (int i = 0; i < 2 * NT; ++i) { s[i][2] = s2[i][2]; s[i][3] = s2[i][3]; }
     }
     float mt[2] = {m[0], m[1]};
 #pragma unroll
@@ -214,25 +273,28 @@ __device__ __forceinline__ void attn_tiles(const bf16* sq, int ldq, const bf16* 
 
 // ------------------------------------------------------------------------------------------------ decode
 constexpr int kDecStages = 3;
-template <int DVP, int BIAS>
+// MAPS 2: both maps of up to eight heads are the rows of one tile, their keys and the values they share one stage.
+template <int DVP, int BIAS, int MAPS>
 __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
-    constexpr int NV = DVP / 8;
+    constexpr int NV = DVP / 8, HB = 16 / MAPS;                    // heads of a tile
     extern __shared__ __align__(16) bf16 asm_[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = threadIdx.x;
-    const int r = blockIdx.x / p.G, g = blockIdx.x % p.G, split = blockIdx.y, hg = p.H / p.G, h0 = blockIdx.z * 16;
+    const int groups = p.G / MAPS, r = blockIdx.x / groups, g = blockIdx.x % groups, split = blockIdx.y, hg = p.H / p.G, h0 = blockIdx.z * HB;
     const int ldk = p.dkp + 8, ldv = DVP + 8;
     bf16* sq = asm_;                                              // [16][ldk]
-    bf16* st = sq + 16 * ldk + (size_t)warp * kDecStages * 16 * (ldk + ldv);
+    const int stage = 16 * (MAPS * ldk + ldv);
+    bf16* st = sq + 16 * ldk + (size_t)warp * kDecStages * stage;
     pdl_wait();
     pdl_launch_dependents();
     const int seq = p.row_seq[r], pos = p.row_pos[r];
     if (seq < 0) return;
-    const bf16* q = reinterpret_cast<const bf16*>(p.q) + ((size_t)r * p.H + (size_t)g * hg + h0) * p.dkp;
-    const int nh = min(16, hg - h0);
+    const bf16* q = reinterpret_cast<const bf16*>(p.q) + (size_t)r * p.H * p.dkp;
+    const int nh = min(HB, hg - h0);
+    auto head = [&](int row) { return (g * MAPS + row / HB) * hg + h0 + min(row % HB, nh - 1); };
     for (int i = t; i < 16 * (p.dkp / 8); i += 128) {
         const int hh = i / (p.dkp / 8), c = i % (p.dkp / 8);
         uint4 v = make_uint4(0, 0, 0, 0);
-        if (hh < nh) v = *reinterpret_cast<const uint4*>(q + (size_t)hh * p.dkp + c * 8);
+        if (hh % HB < nh) v = *reinterpret_cast<const uint4*>(q + (size_t)head(hh) * p.dkp + c * 8);
         *reinterpret_cast<uint4*>(sq + hh * ldk + c * 8) = v;
     }
     const int lo = attn_low(p, pos);
@@ -243,20 +305,22 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     const int kc = p.dkp / 8, vc = DVP / 8;
     auto issue = [&](int tile, int buf) {
         if (tile < t1) {
-            bf16* dk_ = st + (size_t)buf * 16 * (ldk + ldv);
-            bf16* dv_ = dk_ + 16 * ldk;
+            bf16* dk_ = st + (size_t)buf * stage;
+            bf16* dv_ = dk_ + MAPS * 16 * ldk;
             // two lanes per key, alternating 16-byte pieces; keys past the position are clamped (masked later)
             const int kr = lane >> 1, j = min(lo + tile * 16 + kr, pos);
             const bf16* src = cache + ((size_t)p.block_table[(size_t)seq * p.max_pages + j / p.page] * p.page + j % p.page) * ldc;
-            for (int c = lane & 1; c < kc; c += 2) cp16(dk_ + kr * ldk + c * 8, src + (size_t)g * p.dkp + c * 8);
-            for (int c = lane & 1; c < vc; c += 2) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)(g / p.maps) * p.dvp + c * 8);
+#pragma unroll
+            for (int m = 0; m < MAPS; ++m)
+                for (int c = lane & 1; c < kc; c += 2) cp16(dk_ + (m * 16 + kr) * ldk + c * 8, src + (size_t)(g * MAPS + m) * p.dkp + c * 8);
+            for (int c = lane & 1; c < vc; c += 2) cp16(dv_ + kr * ldv + c * 8, src + (size_t)p.off_v + (size_t)(MAPS == 2 ? g : g / p.maps) * p.dvp + c * 8);
         }
         cp_commit();
     };
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[NV][4];
 #pragma unroll
     for (int i = 0; i < NV; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
-    const int hr0 = g * hg + h0 + min(lane >> 2, nh - 1), hr1 = g * hg + h0 + min((lane >> 2) + 8, nh - 1);
+    const int hr0 = head(lane >> 2), hr1 = head((lane >> 2) + 8);
     const float slope2[2] = {p.slope ? p.slope[hr0] * kLog2e : 0.f, p.slope ? p.slope[hr1] * kLog2e : 0.f};
     const int pp[2] = {pos, pos}, low[2] = {lo, lo};
     const float* const tab[2] = {BIAS ? p.bias + (size_t)hr0 * p.bias_len : nullptr, BIAS ? p.bias + (size_t)hr1 * p.bias_len : nullptr};
@@ -268,8 +332,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         issue(tile + 4 * (kDecStages - 1), (buf + kDecStages - 1) % kDecStages);
         cp_wait<kDecStages - 1>();
         __syncwarp();
-        const bf16* dk_ = st + (size_t)buf * 16 * (ldk + ldv);
-        attn_tiles<NV, 1, BIAS ? 2 : 0>(sq, ldk, dk_, ldk, dk_ + 16 * ldk, ldv, p.dkp, lo + tile * 16, pos + 1, pp, low, p.scale * kLog2e, slope2, tab,
+        const bf16* dk_ = st + (size_t)buf * stage;
+        attn_tiles<NV, 1, BIAS ? 2 : 0, MAPS>(sq, ldk, dk_, ldk, dk_ + MAPS * 16 * ldk, ldv, p.dkp, lo + tile * 16, pos + 1, pp, low, p.scale * kLog2e, slope2, tab,
                                         p.bias_len - 1, m, l, o);
         __syncwarp();
         buf = (buf + 1) % kDecStages;
@@ -292,8 +356,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         if ((lane & 3) == 0) { d[DVP] = m[row]; d[DVP + 1] = l[row]; }
     }
     __syncthreads();
-    for (int i = t; i < nh * p.dv; i += 128) {
-        const int hh = i / p.dv, c = i - hh * p.dv, h = g * hg + h0 + hh;
+    for (int i = t; i < MAPS * nh * p.dv; i += 128) {
+        const int j = i / p.dv, c = i - j * p.dv, hh = j / nh * HB + j % nh, h = head(hh);
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) M = fmaxf(M, so[((size_t)w * 16 + hh) * LDO + DVP]);
@@ -339,40 +403,72 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(AttnParams p) {
     }
 }
 
-// Differential heads: o_1 and o_2 of head h of a row (each the merge of NS split sums, or one normalised result: ml null) -> rms(o_1 - lambda o_2) factor.
-// One warp per (row, head); parts [rows, 2 H, NS, dvp] in the order [value head, map, head of the group].
+// Differential heads: o_1 and o_2 of head h of a row -> rms(o_1 - lambda o_2) factor.  parts [rows, 2 H, NS, dvp] in the order [value head, map, head of the
+// group].  Normalised results (NS = 1): one warp per (row, head).
 template <typename T>
-__global__ void __launch_bounds__(128) attn_diff_kernel(T* __restrict__ out, int ldo, const float* __restrict__ parts, const float* __restrict__ ml, int NS, int H, int hg,
-                                                        int dv, int dvp, float lambda, float eps, float factor, const int* __restrict__ row_seq) {
+__global__ void __launch_bounds__(128) attn_diff_kernel(T* __restrict__ out, int ldo, const float* __restrict__ parts, int H, int hg, int dv, int dvp, float lambda, float eps,
+                                                        float factor, const int* __restrict__ row_seq) {
     extern __shared__ float sdiff[];                               // [4][dv]
     const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y * 4 + warp;
     pdl_wait();
     pdl_launch_dependents();
     if (row_seq[r] < 0 || h >= H) return;
     float* d = sdiff + warp * dv;
-    const size_t k[2] = {((size_t)r * 2 * H + h / hg * 2 * hg + h % hg) * NS, ((size_t)r * 2 * H + (h / hg * 2 + 1) * hg + h % hg) * NS};
-    float w[2];
-#pragma unroll
-    for (int a = 0; a < 2; ++a) {
-        w[a] = 1.f;
-        if (ml) {
-            const float m = lane < NS ? ml[2 * (k[a] + lane)] : -INFINITY, l = lane < NS ? ml[2 * (k[a] + lane) + 1] : 0.f;
-            const float M = warp_max(m), e = m == -INFINITY ? 0.f : ex2(m - M);
-            w[a] = e / warp_sum(e * l);
-        }
-    }
-    w[1] *= -lambda;
+    const float* p1 = parts + ((size_t)r * 2 * H + h / hg * 2 * hg + h % hg) * dvp;
+    const float* p2 = p1 + (size_t)hg * dvp;
     float ss = 0.f;
-    for (int c0 = 0; c0 < dv; c0 += 32) {
-        const int c = min(c0 + lane, dv - 1);
-        float v = 0.f;
 #pragma unroll 4
-        for (int s = 0; s < NS; ++s)
-            v = fmaf(__shfl_sync(0xffffffffu, w[0], s), parts[(k[0] + s) * dvp + c], fmaf(__shfl_sync(0xffffffffu, w[1], s), parts[(k[1] + s) * dvp + c], v));
-        if (c0 + lane < dv) { d[c] = v; ss = fmaf(v, v, ss); }
+    for (int c = lane; c < dv; c += 32) {
+        const float v = fmaf(-lambda, p2[c], p1[c]);
+        d[c] = v;
+        ss = fmaf(v, v, ss);
     }
     const float f = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
+#pragma unroll 4
     for (int c = lane; c < dv; c += 32) out[(size_t)r * ldo + (size_t)h * dv + c] = to_act<T>(d[c] * f);
+}
+
+// The same from split sums (maxima and sums in ml): one block per (row, head); a thread takes four channels of every ng-th split of both maps.
+template <typename T>
+__global__ void __launch_bounds__(256) attn_diff_merge_kernel(T* __restrict__ out, int ldo, const float* __restrict__ parts, const float* __restrict__ ml, int NS, int ng, int H,
+                                                              int hg, int dv, int dvp, float lambda, float eps, float factor, const int* __restrict__ row_seq) {
+    extern __shared__ __align__(16) float sdiff[];                 // [ng][4 nq]
+    __shared__ float sw[2][32], red[33];
+    const int r = blockIdx.x, h = blockIdx.y, t = threadIdx.x, lane = t & 31, nq = (dv + 3) / 4;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (row_seq[r] < 0) return;
+    const size_t k1 = ((size_t)r * 2 * H + h / hg * 2 * hg + h % hg) * NS, k2 = k1 + (size_t)hg * NS;
+    if (t < 64) {
+        const size_t k = t < 32 ? k1 : k2;
+        const float m = lane < NS ? ml[2 * (k + lane)] : -INFINITY, l = lane < NS ? ml[2 * (k + lane) + 1] : 0.f;
+        const float M = warp_max(m), e = m == -INFINITY ? 0.f : ex2(m - M);
+        sw[t >> 5][lane] = e / warp_sum(e * l) * (t < 32 ? 1.f : -lambda);
+    }
+    __syncthreads();
+    for (int i = t; i < nq * ng; i += 256) {
+        const int g = i / nq, q = i - g * nq;
+        const float4* p1 = reinterpret_cast<const float4*>(parts + k1 * dvp) + q;
+        const float4* p2 = reinterpret_cast<const float4*>(parts + k2 * dvp) + q;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int s = g; s < NS; s += ng) {
+            const float4 x = p1[(size_t)s * (dvp / 4)], y = p2[(size_t)s * (dvp / 4)];
+            const float u = sw[0][s], v = sw[1][s];
+            a.x = fmaf(u, x.x, fmaf(v, y.x, a.x)); a.y = fmaf(u, x.y, fmaf(v, y.y, a.y)); a.z = fmaf(u, x.z, fmaf(v, y.z, a.z)); a.w = fmaf(u, x.w, fmaf(v, y.w, a.w));
+        }
+        reinterpret_cast<float4*>(sdiff)[i] = a;
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int c = t; c < dv; c += 256) {
+        float v = sdiff[c];
+        for (int g = 1; g < ng; ++g) v += sdiff[g * 4 * nq + c];
+        sdiff[c] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float f = factor / sqrtf(block_sum(ss, red) / (float)dv + eps);
+    for (int c = t; c < dv; c += 256) out[(size_t)r * ldo + (size_t)h * dv + c] = to_act<T>(sdiff[c] * f);
 }
 
 // ------------------------------------------------------------------------------------------------ prefill
@@ -500,21 +596,26 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
     }
 }
 
+// the few-row form takes both maps of a differential head at once when two stages' worth of their keys fit an SM
+static bool two_map_form(int maps, int dkp, int dvp) { return maps == 2 && (16 * (dkp + 8) + 4 * kDecStages * 16 * (2 * (dkp + 8) + dvp + 8)) * 2 <= 224 * 1024; }
 template <int DVP>
 static int launch_decode(const AttnParams& p, cudaStream_t st) {
     const int ldk = p.dkp + 8, ldv = DVP + 8;
-    size_t smem = (size_t)(16 * ldk + 4 * kDecStages * 16 * (ldk + ldv)) * 2;
+    const bool both = two_map_form(p.maps, p.dkp, DVP) && !p.bias;
+    size_t smem = (size_t)(16 * ldk + 4 * kDecStages * 16 * ((both ? 2 : 1) * ldk + ldv)) * 2;
     const size_t merge = (size_t)4 * 16 * (DVP + 2) * 4;
     if (merge > smem) smem = merge;
     static bool attr = false;
     if (!attr) {
-        cudaFuncSetAttribute(attn_decode_kernel<DVP, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
-        cudaFuncSetAttribute(attn_decode_kernel<DVP, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<DVP, 0, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<DVP, 1, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<DVP, 0, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
         attr = true;
     }
     const dim3 grid(p.rows * p.G, p.NS, (p.H / p.G + 15) / 16);
-    if (p.bias) launch_pdl((attn_decode_kernel<DVP, 1>), grid, 128, smem, st, p);
-    else launch_pdl((attn_decode_kernel<DVP, 0>), grid, 128, smem, st, p);
+    if (both) launch_pdl((attn_decode_kernel<DVP, 0, 2>), dim3(p.rows * (p.G / 2), p.NS, (p.H / p.G + 7) / 8), 128, smem, st, p);
+    else if (p.bias) launch_pdl((attn_decode_kernel<DVP, 1, 1>), grid, 128, smem, st, p);
+    else launch_pdl((attn_decode_kernel<DVP, 0, 1>), grid, 128, smem, st, p);
     if (p.NS > 1 && p.maps == 1) launch_pdl((attn_combine_kernel), dim3(p.rows, p.H), 128, 0, st, p);
     return (int)cudaGetLastError();
 }
@@ -542,6 +643,10 @@ using namespace lsb;
 
 // Split sums per (row, head) that lsb_attn leaves to lsb_attn_diff in a step with runs of up to run_rows rows (1: normalised results).
 LSB_API int lsb_attn_partials(int run_rows, int H, int G, int dkp, int dvp, int NS, int f32) { return few_row_form(run_rows, H, G, dkp, dvp, f32) ? NS : 1; }
+// Blocks of the few-row form per row and key split
+LSB_API int lsb_attn_blocks(int H, int G, int maps, int dkp, int dvp) {
+    return two_map_form(maps, dkp, dvp) ? G / 2 * ((H / G + 7) / 8) : G * ((H / G + 15) / 16);
+}
 // padded head width of the cache and of the query buffer
 LSB_API int lsb_attn_head_pad(int d) { return d <= 32 ? 32 : (d <= 64 ? 64 : (d <= 128 ? 128 : (d + 127) / 128 * 128)); }
 
@@ -623,10 +728,16 @@ LSB_API int lsb_attn(const void* q, const void* cache, const void* block_table, 
 LSB_API int lsb_attn_diff(void* out, int ldo, const void* parts, const void* ml, int NS, int rows, int H, int hg, int dv, int dvp, float lambda, float eps, float factor,
                           const void* row_seq, int f32, void* stream) {
     if (rows < 1 || H < 1 || hg < 1 || H % hg || NS < 1 || NS > 32 || (NS > 1 && !ml) || dv < 1 || dv > dvp || dv > 3000) return -1;
-    const dim3 grid(rows, (H + 3) / 4);
-#define LSB_AD(T) launch_pdl((attn_diff_kernel<T>), grid, 128, (size_t)16 * dv, (cudaStream_t)stream, (T*)out, ldo, (const float*)parts, (const float*)(NS > 1 ? ml : nullptr), NS, \
-                             H, hg, dv, dvp, lambda, eps, factor, (const int*)row_seq)
-    if (f32) LSB_AD(float); else LSB_AD(bf16);
+    cudaStream_t st = (cudaStream_t)stream;
+    const int nq = (dv + 3) / 4;
+    int ng = 256 / nq;
+    ng = ng < 1 ? 1 : (ng < NS ? ng : NS);
+#define LSB_AD(T)                                                                                                                                                    \
+    if (NS > 1) launch_pdl((attn_diff_merge_kernel<T>), dim3(rows, H), 256, (size_t)ng * nq * 16, st, (T*)out, ldo, (const float*)parts, (const float*)ml, NS, ng, H, hg,  \
+                           dv, dvp, lambda, eps, factor, (const int*)row_seq);                                                                                       \
+    else launch_pdl((attn_diff_kernel<T>), dim3(rows, (H + 3) / 4), 128, (size_t)16 * dv, st, (T*)out, ldo, (const float*)parts, H, hg, dv, dvp, lambda, eps, factor,      \
+                    (const int*)row_seq)
+    if (f32) { LSB_AD(float); } else { LSB_AD(bf16); }
 #undef LSB_AD
     LSB_CHECK_LAUNCH();
 }

@@ -289,12 +289,12 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
         else *reinterpret_cast<uint4*>(sq + m * ld + c * 8) = make_uint4(0, 0, 0, 0);
     }
     auto low = [&](int pos) { return p.window > 0 ? max(0, pos - p.window + 1) : 0; };          // first key that a position sees
-    const int first = low(pos_first) / KT, end = pos_last / KT + 1, per = (end - first + p.NS - 1) / p.NS, t0 = first + (int)blockIdx.y * per, t1 = min(end, t0 + per);
+    const int key0 = low(pos_first), ntile = (pos_last - key0) / KT + 1, per = (ntile + p.NS - 1) / p.NS, t0 = (int)blockIdx.y * per, t1 = min(ntile, t0 + per);
     constexpr int TPK = 256 / KT;                                 // threads per key of a tile copy
     const int kr = t / TPK;
     const int* bt = p.block_table + (size_t)seq * p.max_pages;
     auto locate = [&](int kt) {                                   // cache row of this thread's key in tile kt
-        const int j = min(kt * KT + kr, pos_last);                // keys past the tile's last position are clamped (masked later)
+        const int j = min(key0 + kt * KT + kr, pos_last);                // keys past the tile's last position are clamped (masked later)
         return kt < t1 ? (size_t)bt[j / p.page] * p.page + j % p.page : 0;
     };
     size_t ahead = locate(t0);                                    // looked up one tile early: the copies do not wait for the table
@@ -356,13 +356,13 @@ __global__ void __launch_bounds__(256, 1) latent_attn_kernel(LatentAttn p) {
         for (; k + 32 <= D; k += 32) { step(k, s[0]); step(k + 16, s[1]); }
         if (k < D) step(k, s[0]);
         float mt[2] = {-INFINITY, -INFINITY};
-        const bool full = kt * KT + KT - 1 <= pos_first && nf == BM && kt * KT >= low(pos_last);
+        const bool full = key0 + kt * KT + KT - 1 <= pos_first && nf == BM && key0 + kt * KT >= low(pos_last);
 #pragma unroll
         for (int i = 0; i < NT; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float v = (s[0][i][j] + s[1][i][j]) * p.scale2;
-                const int key = kt * KT + ki * C::KW + i * 8 + (lane & 3) * 2 + (j & 1);
+                const int key = key0 + kt * KT + ki * C::KW + i * 8 + (lane & 3) * 2 + (j & 1);
                 s[0][i][j] = full || (key <= pr[j >> 1] && key >= lo[j >> 1]) ? v : -INFINITY;
                 mt[j >> 1] = fmaxf(mt[j >> 1], s[0][i][j]);
             }

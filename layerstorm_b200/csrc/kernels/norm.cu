@@ -784,6 +784,22 @@ __device__ __forceinline__ float sum_slots(float a, const MoeSum& mo, const floa
     return a;
 }
 
+// 16 bytes of activations as fp32 and back; four of them
+__device__ __forceinline__ void load_act16(const float* p, float (&v)[4]) { *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void load_act16(const bf16* p, float (&v)[8]) { unpack_bf16x8(*reinterpret_cast<const uint4*>(p), v); }
+__device__ __forceinline__ void store_act4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store_act4(bf16* p, const float* v) {
+    const bf162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+__device__ __forceinline__ void store_act16(float* p, const float (&v)[4]) { store_act4(p, v); }
+__device__ __forceinline__ void store_act16(bf16* p, const float (&v)[8]) {
+    bf162 h[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) h[u] = __floats2bfloat162_rn(v[2 * u], v[2 * u + 1]);
+    *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(h);
+}
+
 // Causal convolution over time on the sublayer's input h = x[r], added to it: xc = h + sum_j w[j] h_(t - taps + 1 + j).  state: a sequence slot's last
 // taps - 1 inputs, oldest first.  (As part of the residual update: steps of one row per sequence.)
 struct InputConv { void* xc; const float* w; float* state; const int* slot; int taps, ldw; };      // w [taps, ldw], state [slots, taps - 1, ldw]
@@ -857,12 +873,77 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(T* __restrict__ x, int 
     }
 }
 
-// The input convolution of runs of rows: xc = x + conv(x), and every sequence's state moves on.  A block takes kConvRows rows of one sequence and 4 columns
-// per thread; the first block of a sequence alone touches its state (the rows it needs beyond its own are read from x).
+// x = norm(resid), xc = x + conv(x) behind the residual update of steps with one row per sequence, for norms of the sum (RMS, layer norm) behind a plain update:
+// a row per block, four columns per thread kept in registers; everything that the previous kernel does not write is fetched in front of the dependency wait.
+template <typename T, bool MOE, int TAPS>
+__global__ void __launch_bounds__(1024) norm_conv_kernel(T* __restrict__ x, int ldx, float* __restrict__ resid, int ldr, const float* __restrict__ sub, int lds, NormW pre,
+                                                         MoeSum mo, const float* __restrict__ step, InputConv ic) {
+    __shared__ float red[33], s_w[32];
+    __shared__ int s_id[32];
+    constexpr int K = TAPS - 1;
+    const int r = blockIdx.x, i = threadIdx.x * 4, slot = ic.slot[r];
+    const bool in = i < pre.dim;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto ld = [&](const float* p) { return p && in ? *reinterpret_cast<const float4*>(p + i) : zero; };
+    float* s0 = ic.state + (size_t)max(slot, 0) * K * ic.ldw + i;
+    const float4 nw = ld(pre.w), nb = ld(pre.b);
+    float4 cw[TAPS], st[K ? K : 1], v = ld(step);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) cw[j] = ld(ic.w + (size_t)j * ic.ldw);
+#pragma unroll
+    for (int j = 0; j < K; ++j) st[j] = slot >= 0 && in ? *reinterpret_cast<const float4*>(s0 + (size_t)j * ic.ldw) : zero;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (MOE) load_slots(mo, r, s_id, s_w);
+    if (in) {
+        float* rr = resid + (size_t)r * ldr;
+        const float4 o = *reinterpret_cast<const float4*>(rr + i);
+        float4 a = ld(sub ? sub + (size_t)r * lds : nullptr);
+        if (MOE) a = sum_slots4(a, mo, mo.y + (size_t)r * mo.S * mo.ldy, rr, i, s_id, s_w);
+        v.x += o.x + a.x; v.y += o.y + a.y; v.z += o.z + a.z; v.w += o.w + a.w;
+        *reinterpret_cast<float4*>(rr + i) = v;
+    }
+    if (pre.kind == kNormLayer) {
+        const float mean = block_sum(v.x + v.y + v.z + v.w, red) / (float)pre.dim;
+        if (in) { v.x -= mean; v.y -= mean; v.z -= mean; v.w -= mean; }
+    }
+    const float rstd = 1.f / sqrtf(block_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))), red) / (float)pre.dim + pre.eps);
+    if (!in) return;
+    const float n[4] = {v.x * rstd * nw.x + nb.x, v.y * rstd * nw.y + nb.y, v.z * rstd * nw.z + nb.z, v.w * rstd * nw.w + nb.w};
+    float h[4], c[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+        h[u] = (float)as_act<T>(n[u]);
+        float a = h[u] * reinterpret_cast<const float*>(&cw[K])[u];
+#pragma unroll
+        for (int j = 0; j < K; ++j) a = fmaf(reinterpret_cast<const float*>(&st[j])[u], reinterpret_cast<const float*>(&cw[j])[u], a);
+        c[u] = h[u] + a;
+    }
+    store_act4(x + (size_t)r * ldx + i, h);
+    store_act4(reinterpret_cast<T*>(ic.xc) + (size_t)r * ldx + i, c);
+    if (slot >= 0) {
+#pragma unroll
+        for (int j = 0; j < K; ++j) *reinterpret_cast<float4*>(s0 + (size_t)j * ic.ldw) = j + 1 < K ? st[j + 1] : make_float4(h[0], h[1], h[2], h[3]);
+    }
+}
+
+// The input convolution of runs of rows: xc = x + conv(x), and every sequence's state moves on.  A block takes kConvRows rows of one sequence and V columns
+// per thread (16 bytes); the inputs that the convolution looks back at stay in registers (TAPS; 0: any number of taps, read again per tap).  The first block
+// of a sequence alone touches its state (the rows that the others need beyond their own are read from x).
 constexpr int kConvRows = 16;
-template <typename T>
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) input_conv_kernel(const T* __restrict__ x, int ldx, InputConv ic, const int* __restrict__ seq_row0, const int* __restrict__ seq_nrows,
                                                          const int* __restrict__ seq_slot, int nseq, int dim) {
+    constexpr int V = 16 / (int)sizeof(T);
+    const int i = (blockIdx.x * 128 + threadIdx.x) * V, K = TAPS ? TAPS - 1 : ic.taps - 1;
+    const float* w = ic.w + i;
+    float cw[TAPS ? TAPS : 1][V];
+    if (TAPS && i < dim) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int u = 0; u < V; u += 4) *reinterpret_cast<float4*>(&cw[j][u]) = *reinterpret_cast<const float4*>(w + (size_t)j * ic.ldw + u);
+    }
     pdl_wait();
     pdl_launch_dependents();
     int tile = blockIdx.y, s = 0, n = 0;
@@ -872,39 +953,60 @@ __global__ void __launch_bounds__(128) input_conv_kernel(const T* __restrict__ x
         if (tile < nt) break;
         tile -= nt;
     }
-    const int i = (blockIdx.x * 128 + threadIdx.x) * 4, K = ic.taps - 1;
     if (s == nseq || i >= dim) return;
     const T* xs = x + (size_t)seq_row0[s] * ldx + i;
     T* out = reinterpret_cast<T*>(ic.xc) + (size_t)seq_row0[s] * ldx + i;
     float* st = ic.state + (size_t)seq_slot[s] * K * ic.ldw + i;
-    const float* w = ic.w + i;
-    auto load = [&](int t) {                                       // input of row t of the run; t < 0: before the run
-        if (t < 0) return *reinterpret_cast<const float4*>(st + (size_t)(K + t) * ic.ldw);
-        if constexpr (sizeof(T) == 4) return *reinterpret_cast<const float4*>(xs + (size_t)t * ldx);
-        else {
-            const uint2 u = *reinterpret_cast<const uint2*>(xs + (size_t)t * ldx);
-            const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&u.y));
-            return make_float4(a.x, a.y, b.x, b.y);
-        }
+    auto load = [&](int t, float (&v)[V]) {                        // input of row t of the run; t < 0: before the run
+        if (t >= 0) { load_act16(xs + (size_t)t * ldx, v); return; }
+#pragma unroll
+        for (int u = 0; u < V; u += 4) *reinterpret_cast<float4*>(&v[u]) = *reinterpret_cast<const float4*>(st + (size_t)(K + t) * ic.ldw + u);
     };
     const int r0 = tile * kConvRows, r1 = min(n, r0 + kConvRows);
-#pragma unroll 4
-    for (int r = r0; r < r1; ++r) {
-        const float4 h = load(r), wk = *reinterpret_cast<const float4*>(w + (size_t)K * ic.ldw);
-        float4 a = make_float4(h.x * wk.x, h.y * wk.y, h.z * wk.z, h.w * wk.w);
-        for (int j = 0; j < K; ++j) {
-            const float4 v = load(r - K + j), c = *reinterpret_cast<const float4*>(w + (size_t)j * ic.ldw);
-            a.x = fmaf(v.x, c.x, a.x); a.y = fmaf(v.y, c.y, a.y); a.z = fmaf(v.z, c.z, a.z); a.w = fmaf(v.w, c.w, a.w);
+    if constexpr (TAPS > 0) {
+        float b[TAPS][V];                                          // the last inputs, row r in b[(r - r0 + K) % TAPS]
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) load(r0 - K + j, b[j]);
+#pragma unroll
+        for (int rr = 0; rr < kConvRows; ++rr) {
+            if (r0 + rr >= r1) break;
+            load(r0 + rr, b[(rr + TAPS - 1) % TAPS]);
+            float a[V];
+#pragma unroll
+            for (int u = 0; u < V; ++u) {
+                const float h = b[(rr + TAPS - 1) % TAPS][u];
+                a[u] = h * cw[TAPS - 1][u];
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) a[u] = fmaf(b[(rr + j) % TAPS][u], cw[j][u], a[u]);
+                a[u] += h;
+            }
+            store_act16(out + (size_t)(r0 + rr) * ldx, a);
         }
-        a.x += h.x; a.y += h.y; a.z += h.z; a.w += h.w;
-        T* o = out + (size_t)r * ldx;
-        if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(o) = a;
-        else { reinterpret_cast<bf162*>(o)[0] = __floats2bfloat162_rn(a.x, a.y); reinterpret_cast<bf162*>(o)[1] = __floats2bfloat162_rn(a.z, a.w); }
+    } else {
+        for (int r = r0; r < r1; ++r) {
+            float h[V], a[V], b[V];
+            load(r, h);
+#pragma unroll
+            for (int u = 0; u < V; ++u) a[u] = h[u] * w[(size_t)K * ic.ldw + u];
+            for (int j = 0; j < K; ++j) {
+                load(r - K + j, b);
+#pragma unroll
+                for (int u = 0; u < V; ++u) a[u] = fmaf(b[u], w[(size_t)j * ic.ldw + u], a[u]);
+            }
+#pragma unroll
+            for (int u = 0; u < V; ++u) a[u] += h[u];
+            store_act16(out + (size_t)r * ldx, a);
+        }
     }
     // the block that reads the old state is the one that replaces it; oldest first, so that entries are read before they are overwritten.  (Tiles behind the
-    // first reach back at most into rows of the run when it has at least K rows in front of them.)
+    // first reach back into rows of the run only: it has at least K rows in front of them.)
     if (tile == 0)
-        for (int j = 0; j < K; ++j) *reinterpret_cast<float4*>(st + (size_t)j * ic.ldw) = load(n - K + j);
+        for (int j = 0; j < K; ++j) {
+            float v[V];
+            load(n - K + j, v);
+#pragma unroll
+            for (int u = 0; u < V; u += 4) *reinterpret_cast<float4*>(st + (size_t)j * ic.ldw + u) = *reinterpret_cast<const float4*>(&v[u]);
+        }
 }
 
 // The same with element-wise norms on both sides: columns spread over blocks, four per thread, nothing exchanged.
@@ -968,6 +1070,16 @@ static int residual_update(void* x, int ldx, void* resid, int ldr, const void* s
     for (const NormW* n : {&post, &pre})
         if (n->kind < 0 || n->kind > kNormNone || (n->kind != kNormNone && !n->w) || (n->kind == kNormTanh && !n->alpha)) return -1;
     if (ic.xc && (!norm_moments_needed(pre.kind) || ic.taps < 1 || !ic.w || (ic.taps > 1 && !ic.state) || !ic.slot)) return -1;
+    if (ic.xc && post.kind == kNormNone && ic.taps <= 4 && dim <= 4096 && !((dim | ldx | ldr | lds | ic.ldw) & 3) && (!mo.y || mo.ldy % 4 == 0)) {
+        const int threads = (dim / 4 + 31) / 32 * 32;
+#define LSB_NC(T, M, N) launch_pdl((norm_conv_kernel<T, M, N>), rows, threads, 0, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, pre, mo, step, ic)
+#define LSB_NM(T, M) switch (ic.taps) { case 1: LSB_NC(T, M, 1); break; case 2: LSB_NC(T, M, 2); break; case 3: LSB_NC(T, M, 3); break; default: LSB_NC(T, M, 4); }
+        if (f32) { if (mo.y) { LSB_NM(float, true) } else { LSB_NM(float, false) } }
+        else { if (mo.y) { LSB_NM(bf16, true) } else { LSB_NM(bf16, false) } }
+#undef LSB_NM
+#undef LSB_NC
+        LSB_CHECK_LAUNCH();
+    }
     if (!step && !norm_moments_needed(post.kind) && !norm_moments_needed(pre.kind) && dim % 4 == 0 && ldx % 4 == 0 && ldr % 4 == 0 && lds % 4 == 0 && mo.ldy % 4 == 0 && rows < 65536) {
         const dim3 grid((dim / 4 + 127) / 128, rows);
 #define LSB_PW(T, M) launch_pdl((post_norm_wide_kernel<T, M>), grid, 128, 0, st, (T*)x, ldx, (float*)resid, ldr, (const float*)sub, lds, post, pre, mo)
@@ -1005,12 +1117,16 @@ LSB_API int lsb_resid_update(void* x, int ldx, void* resid, int ldr, const void*
 // Input convolution of a step with runs of rows: xc = x + conv(x), rows of ldx; w [taps, ldw] fp32 (last tap: the current token), state [slots, taps - 1, ldw].
 LSB_API int lsb_input_conv(void* xc, const void* x, int ldx, const void* w, void* state, int taps, int ldw, const void* seq_row0, const void* seq_nrows, const void* seq_slot,
                            int nseq, int rows, int dim, int f32, void* stream) {
-    if (rows < 1 || nseq < 1 || taps < 1 || taps - 1 > kConvRows || (taps > 1 && !state) || dim % 4 || ldx % 4 || ldw % 4 || ldw < dim) return -1;
+    if (rows < 1 || nseq < 1 || taps < 1 || taps - 1 > kConvRows || (taps > 1 && !state) || dim % 8 || ldx % 8 || ldw % 4 || ldw < dim) return -1;
     const InputConv ic{xc, (const float*)w, (float*)state, nullptr, taps, ldw};
-    const dim3 grid((dim / 4 + 127) / 128, rows / kConvRows + nseq);
+    const int v = f32 ? 4 : 8;
+    const dim3 grid((dim / v + 127) / 128, rows / kConvRows + nseq);
     cudaStream_t st = (cudaStream_t)stream;
-    if (f32) launch_pdl((input_conv_kernel<float>), grid, 128, 0, st, (const float*)x, ldx, ic, (const int*)seq_row0, (const int*)seq_nrows, (const int*)seq_slot, nseq, dim);
-    else launch_pdl((input_conv_kernel<bf16>), grid, 128, 0, st, (const bf16*)x, ldx, ic, (const int*)seq_row0, (const int*)seq_nrows, (const int*)seq_slot, nseq, dim);
+#define LSB_IT(T, N) launch_pdl((input_conv_kernel<T, N>), grid, 128, 0, st, (const T*)x, ldx, ic, (const int*)seq_row0, (const int*)seq_nrows, (const int*)seq_slot, nseq, dim)
+#define LSB_IC(T) switch (taps) { case 2: LSB_IT(T, 2); break; case 3: LSB_IT(T, 3); break; case 4: LSB_IT(T, 4); break; default: LSB_IT(T, 0); }
+    if (f32) { LSB_IC(float) } else { LSB_IC(bf16) }
+#undef LSB_IC
+#undef LSB_IT
     LSB_CHECK_LAUNCH();
 }
 

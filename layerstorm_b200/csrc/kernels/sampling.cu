@@ -57,11 +57,15 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(float* __restrict
 
 // x <- cap * tanh(x / cap)
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int ld, int n, float cap) {
-    const int i = blockIdx.x * 256 + threadIdx.x;
+    float* p = x + (size_t)blockIdx.y * ld;
+    const int i0 = blockIdx.x * 1024 + threadIdx.x;
     pdl_wait();
     pdl_launch_dependents();
-    float* p = x + (size_t)blockIdx.y * ld + i;
-    if (i < n) *p = cap * tanhf(*p / cap);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int i = i0 + j * 256;
+        if (i < n) p[i] = cap * tanhf(p[i] / cap);
+    }
 }
 
 // packed (key, ~index): larger value wins, equal values -> lower index wins
@@ -324,7 +328,7 @@ LSB_API int lsb_embedding_bigram(void* out, const void* table, const void* pairs
 // Soft cap of the logits, in place.
 LSB_API int lsb_softcap(void* logits, int ld, int rows, int V, float cap, void* stream) {
     if (rows < 1 || rows > 65535 || V < 1 || !(cap > 0.f)) return -1;
-    launch_pdl((softcap_kernel), dim3((V + 255) / 256, rows), 256, 0, (cudaStream_t)stream, (float*)logits, ld, V, cap);
+    launch_pdl((softcap_kernel), dim3((V + 1023) / 1024, rows), 256, 0, (cudaStream_t)stream, (float*)logits, ld, V, cap);
     LSB_CHECK_LAUNCH();
 }
 

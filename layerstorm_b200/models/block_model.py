@@ -258,7 +258,7 @@ class BlockWorkspace(StepBuffers):
             self.splits = {}
             for i, b in att:
                 seen = min(b.window or max_ctx, b.chunk or max_ctx, max_ctx)
-                blocks = R * b.kv_heads * b.maps * ((b.heads // b.kv_heads + 15) // 16)
+                blocks = R * int(nat.call("lsb_attn_blocks", b.heads * b.maps, b.kv_heads * b.maps, b.maps, m.head_pad(b.dim), m.head_pad(b.vdim)))
                 self.splits[i] = 1 if (m.f32 or R > 64) else max(1, min(32, 296 // blocks, (seen + 63) // 64))
             ns = [(b.heads * b.maps * self.splits[i], m.head_pad(b.vdim)) for i, b in att if self.splits[i] * b.maps > 1]
             self.o_part = z(R * max((n * w for n, w in ns), default=1))

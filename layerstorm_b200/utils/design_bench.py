@@ -1,11 +1,12 @@
 """Prefill and decode throughput of a model design at layer sizes of a real model (random weights), beside the framework's closest other
 design at equal size, with the device time of every kernel launcher.
 
-    python bench.py --design gazutar|rubasun|fasodra [--design-sizes 2048,4096]
+    python bench.py --design gazutar|rubasun|fasodra|nivasun [--design-sizes 2048,4096]
 
 Gazutar's neighbour is a KDA + MLA model of the same width, heads, experts and layer pattern (plain residual stream, dense latent attention),
 Rubasun's an MLA + MoE model of the same width, heads, latent rows, experts and shared expert, Fasodra's the Gazutar model of the same width,
-attention heads and expert parameters.
+attention heads and expert parameters, Nivasun's the Rubasun model (latent attention, gated shared expert) and the Gazutar model (windowed
+attention) of the same width, heads and experts.
 Per launcher: all its calls of one step, recorded from an eager pass and replayed back to back in a CUDA graph (other layers' operands in
 between, so that a layer's weights are not left over in L2), divided by the number of calls.  Fractions are of the measured peaks
 (MEASURED_PEAKS.json): bytes or FLOPs that the operation has to move or do, over the launcher's time.
@@ -19,7 +20,7 @@ import statistics
 import torch
 
 from ..models.block_model import model_class
-from ..models.config import ModelConfig, fasodra_config, gazutar_config, rubasun_config
+from ..models.config import ModelConfig, fasodra_config, gazutar_config, nivasun_config, rubasun_config
 from ..ops import _native as nat
 from ..runtime.engine import Engine
 
@@ -71,7 +72,22 @@ def fasodra_pair(hidden: int):
     return f, gazutar_pair(hidden)[0]
 
 
-DESIGNS = {"gazutar": gazutar_pair, "rubasun": rubasun_pair, "fasodra": fasodra_pair}
+def nivasun_set(hidden: int):
+    """(Nivasun, neighbours) of one size: 128-wide heads, attention, latent attention and differential attention (half the heads, two maps and 256 value
+    channels each) in turns over windows of half the context; six layers, the second and third run twice, so that there are as many layer runs as layers in
+    the neighbours."""
+    heads, kv, experts, ff, vocab = hidden // 128, max(1, hidden // 512), hidden // 64, hidden // 2, 65536
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": TOP}, "shared": {"ff": ff}}
+    rot, base = {"base": 1e5, "dims": 128}, {"dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 4096}}
+    kinds = [("attention", base | {"heads": heads, "kv_heads": kv, "rot": rot}), ("latent_attention", base | {"heads": heads, "kv_rank": 512, "q_rank": hidden * 3 // 8}),
+             ("attention_2", base | {"heads": heads // 2, "kv_heads": max(1, kv // 2), "vdim": 256, "diff": 0.5, "rot": rot})]
+    n = nivasun_config({"name": f"nivasun-{hidden}", "vocab": vocab, "width": hidden, "norm": {"eps": 1e-5}, "canon": {"taps": 4}, "logit_softcap": 30.0,
+                        "embedding": {"scale": 1.0, "bigram": {"buckets": vocab, "mul_prev": 31, "mul_cur": 17}}, "loop": {"start": 1, "stop": 3, "times": 2},
+                        "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(N_LAYERS - 2)]})
+    return n, rubasun_pair(hidden)[0], gazutar_pair(hidden)[0]
+
+
+DESIGNS = {"gazutar": gazutar_pair, "rubasun": rubasun_pair, "fasodra": fasodra_pair, "nivasun": nivasun_set}
 
 
 def _peaks():
@@ -138,29 +154,32 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
     per_tok = heads * (4 * 128 * 128 + 6 * 64 * 128) * 2            # chunk form: state products, pair products
     decode = rows == batch
     rec = ("bytes", state + gates + rows * heads * 128 * 18) if decode else ("flops", rows * per_tok)
-    mixers = [x for b in cfg.blocks for x in b.mixers]
+    mixers = [x for i, _ in cfg.layer_runs() for x in cfg.blocks[i].mixers] if cfg.blocks else []
     att = next((x for x in mixers if not x.recurrent), None)
     lat, rot, ah, dn, dv = cfg.kv_lora, cfg.qk_rope, cfg.n_heads, cfg.qk_nope, cfg.v_head
-    seen = ctx - rows // 2                                          # keys a row of the chunk sees on average
-    latent = ("bytes", batch * ctx * (lat + rot) * 2 + rows * ah * (2 * lat + rot) * 2) if decode else ("flops", 2 * rows * seen * ah * (2 * lat + rot))
+    lw = min([b.window or ctx for b in mixers if b.latent], default=ctx)
+    seen = sum(min(p + 1, lw) for p in range(ctx - rows, ctx)) / rows      # keys a row of the chunk sees on average
+    latent = ("bytes", batch * min(ctx, lw) * (lat + rot) * 2 + rows * ah * (2 * lat + rot) * 2) if decode else ("flops", 2 * rows * seen * ah * (2 * lat + rot))
     # the queries' way into the latent space and the values' way out of it: weights and activations, or products
     absorb, up = ((("bytes", ah * lat * d * 2 + rows * ah * (lat + d) * 2) if decode else ("flops", 2 * rows * ah * lat * d)) for d in (dn, dv))
     experts = TOP + cfg.n_shared
-    if att is not None and att.latent:
+    if any(b.latent for b in mixers):
         out["lsb_latent_attn"], out["lsb_latent_query"], out["lsb_latent_out"] = latent, absorb, up
-        out["lsb_latent_expand"] = ("flops", 2 * ctx * ah * lat * (dn + dv))
+        out["lsb_latent_expand"] = ("flops", 2 * min(ctx, lw + rows) * ah * lat * (dn + dv))
         out["lsb_attn_run"] = ("flops", 2 * rows * seen * ah * (dn + rot + dv))
         out["lsb_resid_update"] = ("bytes", rows * H * 14)
         out["lsb_glu"] = ("bytes", rows * cfg.moe_inter * 10)
-    elif att is not None:
+    if any(b.softmax for b in mixers):
         mean = lambda xs: sum(xs) / max(1, len(xs))
         keys = lambda b: min(ctx % b.chunk or b.chunk if b.chunk else ctx, b.window or ctx)            # that a decoded token sees
         per_row = lambda b: mean([min(p % b.chunk + 1 if b.chunk else p + 1, b.window or ctx) for p in range(ctx - rows, ctx)])
         soft = [b for b in mixers if b.softmax]
-        kv = lambda b: b.kv_heads * (b.dim + b.vdim) * 2
+        kv = lambda b: b.kv_heads * (b.maps * b.dim + b.vdim) * 2
         out["lsb_attn"] = (("bytes", mean([batch * keys(b) * kv(b) + rows * b.heads * b.vdim * (6 if b.out_gate else 4) for b in soft])) if decode
-                           else ("flops", mean([2 * rows * per_row(b) * b.heads * (b.dim + b.vdim) for b in soft])))
-        out["lsb_attn_prep"] = out["lsb_attn_head_prep"] = ("bytes", mean([rows * ((b.heads + b.kv_heads) * b.dim + b.kv_heads * b.vdim) * 6 for b in soft]))
+                           else ("flops", mean([2 * rows * per_row(b) * b.heads * b.maps * (b.dim + b.vdim) for b in soft])))
+        out["lsb_attn_prep"] = out["lsb_attn_head_prep"] = ("bytes", mean([rows * ((b.heads + b.kv_heads) * b.maps * b.dim * 6 + b.kv_heads * b.vdim * (2 if b.shared_kv else 6))
+                                                                          for b in soft]))
+        out["lsb_attn_diff"] = ("bytes", mean([rows * b.heads * b.vdim * 10 for b in soft if b.maps > 1]))
         out["lsb_resid_update"] = ("bytes", rows * H * (14 + TOP * 4) // 2 + rows * H * 7)
         # chunk form: two state products and two (delta rule: six, with the solve) products over pairs of a chunk
         dlt, tm = [b for b in mixers if b.delta], [b for b in mixers if b.kind == "time_mix"]
@@ -176,7 +195,12 @@ def work(cfg, rows: int, ctx: int, batch: int) -> dict:
         n = cfg.streams
         ups = [rows * H * (4 + 4 * n + 2)] + [rows * H * (8 * n + 2 + s) for b in cfg.blocks for s in ((8 if b.join == "normed" and b.branches else 4), TOP * 4)]
         out["lsb_stream_update"] = ("bytes", mean(ups))
-    else:
+    if cfg.norm_place == "parallel":
+        # one update per layer run and one in front of the first; steps of single tokens have the convolution in it (its state read and written)
+        out["lsb_resid_update"] = ("bytes", rows * H * (14 + TOP * 4 + ((2 + 8 * (cfg.input_conv - 1)) if decode else 0)))
+        out["lsb_input_conv"] = ("bytes", rows * H * 4)
+        out["lsb_glu"] = ("bytes", rows * cfg.moe_inter * 10)
+    if att is None:
         out["lsb_kda_forward"] = out["lsb_kda_forward_chunked"] = rec
         out["lsb_mla_decode"] = latent
         out["lsb_batched_gemv_bf16"] = (absorb[0], (absorb[1] + up[1]) / 2)

@@ -157,7 +157,7 @@ def test_a_sink_counts_once_and_takes_no_part_in_the_values():
 
 @pytest.mark.parametrize("f32", [True, False])
 @pytest.mark.parametrize("H,G,dk,dv,rot,window", [(4, 4, 32, 64, 8, 40), (6, 3, 20, 36, 12, 26), (8, 2, 64, 128, 64, 64), (4, 1, 128, 128, 128, 33), (2, 1, 264, 72, 100, 41), (5, 5, 16, 280, 10, 64),
-                                                  (40, 1, 24, 16, 24, 90), (1, 1, 2, 1, 2, 1), (3, 3, 96, 256, 32, 500)])
+                                                  (40, 1, 24, 16, 24, 90), (1, 1, 2, 1, 2, 1), (3, 3, 96, 256, 32, 500), (4, 2, 200, 250, 64, 45)])
 def test_differential_attention_forms(H, G, dk, dv, rot, window, f32):
     """The two maps of a head look at different keys, at the window's ends and page borders, over one set of values."""
     if f32 and (H, G) not in ((6, 3), (4, 1)):
@@ -282,7 +282,7 @@ def test_long_runs_over_written_out_keys_start_at_the_first_visible_one(H, dn, d
 # ------------------------------------------------------------------------------------------------ input convolution, residual update, embedding, router, logits
 @pytest.mark.parametrize("f32", [True, False])
 @pytest.mark.parametrize("taps", [1, 2, 3, 4, 6, 17])
-@pytest.mark.parametrize("width", [12, 136, 1024])
+@pytest.mark.parametrize("width", [16, 136, 1024])
 def test_input_convolution_across_portions(width, taps, f32):
     """Runs of every short length on interleaved slots, single rows through the residual update, against the whole sequence."""
     g = torch.Generator().manual_seed(width + taps)
