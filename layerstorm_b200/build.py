@@ -18,6 +18,7 @@ from __future__ import annotations
 
 import concurrent.futures as cf
 import hashlib
+import itertools
 import os
 import shutil
 import subprocess
@@ -41,8 +42,17 @@ CXX_FLAGS = ["-O2", "-g", "-std=c++20", "-fPIC", "-Wall", "-Wno-unused-function"
              "-I", str(CSRC / "include"), "-I", str(CSRC / "runtime")]
 
 
-# kernel files of a model family (models described layer by layer run without the MLA-family, indexer, hyper-connection and expert-parallel kernels)
-FAMILIES = {"blocks": ("attn", "delta", "gemm_tc", "gemv", "latent", "moe", "moe_tc", "norm", "sampling", "tmix")}
+# kernel files of a model family: models described layer by layer run without the MLA-family, indexer, hyper-connection and expert-parallel kernels, and
+# without those of the mixers that they do not have
+MIXER_FILES = {"delta": ("channel_delta", "head_delta"), "latent": ("latent_attention",), "tmix": ("time_mix",)}
+FAMILIES = {"blocks" + "".join(f"_{f}" for f in extra): ("attn", "gemm_tc", "gemv", "moe", "moe_tc", "norm", "sampling") + extra
+            for n in range(len(MIXER_FILES) + 1) for extra in itertools.combinations(MIXER_FILES, n)}
+
+
+def family_of(cfg) -> str | None:
+    """The family of a model described layer by layer (None: the MLA family, which takes the whole library)."""
+    kinds = {m.kind for b in cfg.blocks for m in b.mixers}
+    return "blocks" + "".join(f"_{f}" for f, k in MIXER_FILES.items() if kinds & set(k)) if cfg.blocks else None
 
 
 def _rel(p) -> str:
@@ -147,7 +157,7 @@ def ensure_for(cfg) -> Path:
     """Compile what the model needs (nothing when it is there already) and make the bindings load it; returns the kernel library's path."""
     from .ops import _native
     full = LIB / "liblsb200_kernels.so"
-    family = "blocks" if cfg.blocks else None
+    family = family_of(cfg)
     if family and not _linked([_obj_path(s, "cu") for s in _kernel_sources()], full):
         out = build_all(family=family)
     else:

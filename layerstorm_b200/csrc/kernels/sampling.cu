@@ -58,14 +58,10 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(float* __restrict
 // x <- cap * tanh(x / cap)
 __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int ld, int n, float cap) {
     float* p = x + (size_t)blockIdx.y * ld;
-    const int i0 = blockIdx.x * 1024 + threadIdx.x;
     pdl_wait();
     pdl_launch_dependents();
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-        const int i = i0 + j * 256;
-        if (i < n) p[i] = cap * tanhf(p[i] / cap);
-    }
+#pragma unroll 4
+    for (int i = blockIdx.x * 256 + threadIdx.x; i < n; i += gridDim.x * 256) p[i] = cap * tanhf(p[i] / cap);
 }
 
 // packed (key, ~index): larger value wins, equal values -> lower index wins
@@ -328,7 +324,8 @@ LSB_API int lsb_embedding_bigram(void* out, const void* table, const void* pairs
 // Soft cap of the logits, in place.
 LSB_API int lsb_softcap(void* logits, int ld, int rows, int V, float cap, void* stream) {
     if (rows < 1 || rows > 65535 || V < 1 || !(cap > 0.f)) return -1;
-    launch_pdl((softcap_kernel), dim3((V + 1023) / 1024, rows), 256, 0, (cudaStream_t)stream, (float*)logits, ld, V, cap);
+    const int want = (V + 255) / 256, most = rows < 1184 ? 1184 / rows : 1;      // eight blocks per SM in all, a thread takes several columns
+    launch_pdl((softcap_kernel), dim3(want < most ? want : most, rows), 256, 0, (cudaStream_t)stream, (float*)logits, ld, V, cap);
     LSB_CHECK_LAUNCH();
 }
 

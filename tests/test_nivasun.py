@@ -87,6 +87,13 @@ def test_server_resolves_a_native_checkpoint_directory(tmp_path):
     assert r.embedding == (301 + 98) * 136 * 2
 
 
+def test_a_tool_compiles_the_files_of_the_mixers_that_a_model_has():
+    from layerstorm_b200 import build
+    fam = {n: build.family_of(get_preset(n)) for n in ("tiny-nivasun", "tiny-rubasun", "tiny-fasodra", "tiny-gazutar", "tiny-mla-moe")}
+    assert list(fam.values()) == ["blocks_latent", "blocks_latent", "blocks_delta_tmix", "blocks_delta", None]
+    assert {p.stem for p in build._kernel_sources("blocks_latent")} == set(build.FAMILIES["blocks"]) | {"latent"}
+
+
 def test_the_previous_token_is_staged_with_the_step():
     """In front of a run's first row stands the sequence's last token, in front of a sequence's first token nothing."""
     from types import SimpleNamespace
