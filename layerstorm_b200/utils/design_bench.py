@@ -82,7 +82,7 @@ def nivasun_set(hidden: int):
     kinds = [("attention", base | {"heads": heads, "kv_heads": kv, "rot": rot}), ("latent_attention", base | {"heads": heads, "kv_rank": 512, "q_rank": hidden * 3 // 8}),
              ("attention_2", base | {"heads": heads // 2, "kv_heads": max(1, kv // 2), "vdim": 256, "diff": 0.5, "rot": rot})]
     n = nivasun_config({"name": f"nivasun-{hidden}", "vocab": vocab, "width": hidden, "norm": {"eps": 1e-5}, "canon": {"taps": 4}, "logit_softcap": 30.0,
-                        "embedding": {"scale": 1.0, "bigram": {"buckets": vocab, "mul_prev": 31, "mul_cur": 17}}, "loop": {"start": 1, "stop": 3, "times": 2},
+                        "embedding": {"scale": 1.0, "bigram": {"buckets": vocab, "mul_prev": 53, "mul_cur": 29}}, "loop": {"start": 1, "stop": 3, "times": 2},
                         "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(N_LAYERS - 2)]})
     return n, rubasun_pair(hidden)[0], gazutar_pair(hidden)[0]
 

@@ -233,7 +233,7 @@ MODELS = {
                                         dif(6, 3, 20, 36, 26, 12, 0.35, 300.0), att(3, 3, 40, 70, 40), dif(4, 1, 12, 20, 17, 12, 0.7, 77.0, moe_spec(4, 1, 56, 9))],
                              (1, 3, 2), 4, (97, 1000003, 12345), 3e-3, 9.0),
     "tiles": lambda: model_cfg(384, 520, [dif(4, 4, 64, 128, 130, 64, 0.5, 1e6, moe_spec(12, 4, 128, 256)), att(16, 2, 128, 64, 64, 1e6, moe_spec(12, 4, 128, 128)),
-                                          lat(8, 64, 64, 128, 96, 90, moe_spec(12, 4, 256, 128)), att(8, 8, 64, 48, 32, mlp=moe_spec(8, 3, 128, 128))], (0, 2, 2), 3, (1024, 31, 7)),
+                                          lat(8, 64, 96, 128, 112, 90, moe_spec(12, 4, 256, 128)), att(8, 8, 64, 48, 32, mlp=moe_spec(8, 3, 128, 128))], (0, 2, 2), 3, (1024, 31, 7)),
     "ones": lambda: model_cfg(48, 40, [att(1, 1, 2, 1, 2, mlp=moe_spec(1, 1, 1, 1)), lat(1, 1, 1, 1, 1, 9, moe_spec(3, 3, 8, 5)), dif(1, 1, 2, 3, 2, 2, 0.2),
                                        dif(2, 2, 8, 8, 33, 4, 0.9, 5.0)], (0, 4, 1), 1, (1, 1, 1), 1e-6, 30.0, 1.0),
     "wide": lambda: model_cfg(250, 200, [att(33, 1, 24, 90, 24, 60.0, moe_spec(4, 1, 96, 30)), lat(3, 136, 200, 540, 100, 60, moe_spec(6, 2, 64, 64)), dif(2, 1, 264, 72, 41, 100, 0.45),
