@@ -599,7 +599,7 @@ __global__ void __launch_bounds__(256, DVP <= 128 ? 2 : 1) attn_prefill_kernel(A
     }
 }
 
-// the few-row form takes both maps of a differential head at once when two stages' worth of their keys fit an SM
+// the few-row form takes both maps of a differential head at once when its stages with both maps' keys fit an SM
 static bool two_map_form(int maps, int dkp, int dvp) { return maps == 2 && (16 * (dkp + 8) + 4 * kDecStages * 16 * (2 * (dkp + 8) + dvp + 8)) * 2 <= 224 * 1024; }
 template <int DVP>
 static int launch_decode(const AttnParams& p, cudaStream_t st) {
